@@ -1034,7 +1034,7 @@ def test_weights_keeper_maps_device_weights_into_another_process(tmp_path):
     import os
     import subprocess
     import sys
-    from uniserve_v1_b200.__main__ import _qwen3_model
+    from uniserve_v1_b200.__main__ import _paged_model
     from uniserve_v1_b200.config.policy import Package
     from uniserve_v1_b200.engine.engine import LLMEngine
     from uniserve_v1_b200.engine.types import SamplingParams
@@ -1056,10 +1056,10 @@ def test_weights_keeper_maps_device_weights_into_another_process(tmp_path):
         dev = torch.device("cuda", 0)
         prompts = [[(3 * i + j) % 1000 for i in range(n)] for j, n in enumerate((9, 30))]
         sp = SamplingParams(temperature=0.0, max_tokens=6, ignore_eos=True)
-        _, own, _ = _qwen3_model(pkg, None, dev, BF, None)
+        _, own, _ = _paged_model(pkg, "qwen3_moe", None, dev, BF, None)
         want = LLMEngine(own, num_pages=64, max_num_seqs=4, max_model_len=128).generate(prompts, sp)
         before = torch.cuda.memory_allocated()
-        _, mapped, _ = _qwen3_model(pkg, None, dev, BF, None, sock)
+        _, mapped, _ = _paged_model(pkg, "qwen3_moe", None, dev, BF, None, sock)
         assert mapped.weights_from["keeper_pid"] == proc.pid
         assert torch.cuda.memory_allocated() - before < own.weight_bytes() // 4   # mapped, not copied
         assert torch.equal(mapped.embed, own.embed)

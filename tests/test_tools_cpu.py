@@ -1009,7 +1009,7 @@ def test_weights_keeper_serves_weights_to_restarting_engines(tmp_path):
     import os
     import subprocess
     import sys
-    from uniserve_v1_b200.__main__ import _qwen3_model
+    from uniserve_v1_b200.__main__ import _paged_model
     from uniserve_v1_b200.config.policy import Package
     from uniserve_v1_b200.engine.engine import LLMEngine
     from uniserve_v1_b200.engine.types import SamplingParams
@@ -1032,11 +1032,11 @@ def test_weights_keeper_serves_weights_to_restarting_engines(tmp_path):
         pkg = Package.load(str(pkg_dir))
         prompts = [[(3 * i + j) % 1000 for i in range(n)] for j, n in enumerate((9, 30))]
         sp = SamplingParams(temperature=0.0, max_tokens=6, ignore_eos=True)
-        _, own, _ = _qwen3_model(pkg, None, torch.device("cpu"), torch.float32, None)
+        _, own, _ = _paged_model(pkg, "qwen3_moe", None, torch.device("cpu"), torch.float32, None)
         want = LLMEngine(own, num_pages=64, max_num_seqs=4, max_model_len=128,
                          use_graphs=False).generate(prompts, sp)
         for _ in range(2):                                   # an engine, then its restart
-            _, mapped, _ = _qwen3_model(pkg, None, torch.device("cpu"), torch.float32, None, sock)
+            _, mapped, _ = _paged_model(pkg, "qwen3_moe", None, torch.device("cpu"), torch.float32, None, sock)
             assert mapped.weights_from["keeper_pid"] == proc.pid
             assert torch.equal(mapped.embed, own.embed) and mapped.embed.data_ptr() != own.embed.data_ptr()
             assert (mapped.lm_head is mapped.embed) == (own.lm_head is own.embed)

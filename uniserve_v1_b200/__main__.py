@@ -66,6 +66,8 @@ def serve(args) -> int:
         family = "minimax_h3"
     elif pkg.model and "qwen4_exp" in pkg.model.lower():
         family = "qwen4_exp"
+    elif pkg.model and "nepevik" in pkg.model.lower():
+        family = "nepevik"
     name = pkg.served_model_name or (pkg.model or "model").split("/")[-1]
     shutdown = None
     if family == "minimax_h3":
@@ -266,15 +268,17 @@ def serve(args) -> int:
         shutdown = front.shutdown
         app = create_app(package=pkg, engine=front, tokenizer=tok, served_model_name=name)
     else:
+        # decoders of the paged engine (models/registry.py)
         from .engine.engine import LLMEngine
-        from .models.qwen3_moe import Qwen3MoeConfig, Qwen3MoeModel
         from .server.tokenizer import load_tokenizer
         ctx = None
+        if world > 1 and family != "qwen3_moe":
+            raise SystemExit(f"{family} is served on one GPU")
         if world > 1:
             pp = axes.get("layer", 1) if world % axes.get("layer", 1) == 0 else 1
             ctx = ParallelContext.from_world(tensor=world // pp, layer=pp,
                                              expert_over_tensor=world // pp > 1)
-        cfg, model, ld = _qwen3_model(pkg, directory, device, dtype, ctx,
+        cfg, model, ld = _paged_model(pkg, family, directory, device, dtype, ctx,
                                       getattr(args, "weights_socket", None))
         if pkg.profiling_config.expert_load and hasattr(model, "enable_expert_load") and \
                 (device.type == "cpu" or "expert_order" in pkg.programs
@@ -446,20 +450,20 @@ def serve(args) -> int:
     return 0
 
 
-def _qwen3_model(pkg, directory, device, dtype, ctx, weights_socket=None):
-    """The package's Qwen3 model: mapped from a weights keeper when one answers on
-    ``weights_socket`` with this model's identity, else read from the checkpoint (or drawn
-    at random for ``random:`` models).  Returns (config, model, checkpoint loader or None)."""
-    from .models.qwen3_moe import Qwen3MoeConfig, Qwen3MoeModel
+def _paged_model(pkg, family, directory, device, dtype, ctx, weights_socket=None):
+    """The package's decoder for the paged engine: mapped from a weights keeper when one
+    answers on ``weights_socket`` with this model's identity, else read from the checkpoint (or
+    drawn at random for ``random:`` models).  Returns (config, model, loader or None)."""
+    from .models.registry import PAGED_DECODERS
+    entry = PAGED_DECODERS[family]
     ld = None
     if directory:
         from .checkpoint.quantized import open_checkpoint
         ld = open_checkpoint(directory, dtype)       # NVFP4 / FP8 exports expand on read
-        cfg = Qwen3MoeConfig.from_hf(ld.config)
+        cfg = entry.config(ld.config)
     else:
-        cfg = Qwen3MoeConfig.tiny() if (pkg.model or "").endswith(":tiny") \
-            else Qwen3MoeConfig.qwen3_30b_a3b()
-    model = Qwen3MoeModel(cfg, device, dtype, ctx)
+        cfg = entry.named_config("tiny" if (pkg.model or "").endswith(":tiny") else None)
+    model = entry.model(cfg, device, dtype, ctx)
     if weights_socket:
         from .server.weights_keeper import attach
         if attach(model, weights_socket):
@@ -486,7 +490,13 @@ def keep(args) -> int:
     directory = pkg.model_dir or None
     if directory is None and pkg.model and not pkg.model.startswith("random:"):
         directory = str(resolve_hub(pkg.model))
-    _cfg, model, _ld = _qwen3_model(pkg, directory, device, dtype, None)
+    family = "qwen3_moe"
+    if directory:
+        from .checkpoint.safetensors_io import resolve_family
+        family = resolve_family(directory)
+    elif "nepevik" in (pkg.model or "").lower():
+        family = "nepevik"
+    _cfg, model, _ld = _paged_model(pkg, family, directory, device, dtype, None)
     keeper = WeightsKeeper(model, args.socket)
 
     def ready():

@@ -12,7 +12,11 @@ reference compiles kernel packages at first start
 (crates/build-server, reference project path); here the libraries are built once
 and loaded with ctypes.
 
-Usage: ``python -m uniserve_v1_b200.build [--force] [--verbose]``
+A *group* is the subset of sources one family needs (``GROUPS``): ``build(group=...)`` compiles
+and links only those, into libraries of its own (``libus_kernels-<group>.so``), from the same
+object files, so a tool that serves one model in a fresh checkout does not wait for the rest.
+
+Usage: ``python -m uniserve_v1_b200.build [--force] [--verbose] [--group NAME]``
 """
 from __future__ import annotations
 
@@ -37,6 +41,12 @@ NVCC_FLAGS = [
     "--expt-relaxed-constexpr",
     "-Xptxas", "-v",
 ]
+# Sources of the families that can be built alone: (csrc/**.cu, csrc/host/*.cpp).
+GROUPS = {
+    "nepevik": (("runtime.cu", "gemm_tc05.cu", "linear_decode.cu", "gemm_f32.cu", "moe_route.cu",
+                 "misc.cu", "sampler.cu", "row_ops.cu", "vector_delta.cu", "head_mix_attn.cu"),
+                ("block_manager.cpp",)),
+}
 CXX_FLAGS = ["-O3", "-std=c++17", "-fPIC", "-fvisibility=hidden", "-pthread", "-Wall"]
 
 
@@ -73,14 +83,42 @@ def _compile_one(src: Path, flags: list[str], compiler: str, stamp: dict, force:
     return obj, True, log
 
 
-def build(force: bool = False, verbose: bool = False) -> dict:
-    """Compile what changed and link both libraries; returns the paths."""
+def library_paths(group: str | None = None) -> tuple[Path, Path]:
+    """(kernel library, host library) of the whole package or of one group."""
+    tail = f"-{group}" if group else ""
+    return LIB / f"libus_kernels{tail}.so", LIB / f"libus_host{tail}.so"
+
+
+def _sources(group: str | None) -> tuple[list, list]:
+    if group is None:
+        return (sorted(CSRC.glob("*.cu")) + sorted((CSRC / "fused").glob("*.cu")),
+                sorted((CSRC / "host").glob("*.cpp")))
+    cu, cpp = GROUPS[group]
+    return [CSRC / n for n in cu], [CSRC / "host" / n for n in cpp]
+
+
+def _link(cmd: list, out: Path, objs: list, stamp: dict, force: bool) -> None:
+    """Links ``objs`` into ``out`` unless it was linked from the same object digests."""
+    dig = hashlib.sha256("".join(stamp[o.name] for o in objs).encode()).hexdigest()
+    if not force and out.exists() and stamp.get(out.name) == dig:
+        return
+    tmp = out.with_suffix(f".so.tmp{os.getpid()}")       # linked aside, then moved into place at once
+    proc = subprocess.run([*cmd, "-o", str(tmp), *[str(o) for o in objs]], capture_output=True,
+                          text=True)
+    if proc.returncode != 0:
+        raise RuntimeError(f"link failed: {proc.stdout}{proc.stderr}")
+    os.replace(tmp, out)
+    stamp[out.name] = dig
+
+
+def build(force: bool = False, verbose: bool = False, group: str | None = None) -> dict:
+    """Compile what changed and link both libraries (of the package, or of one ``group``);
+    returns the paths."""
     OBJ.mkdir(parents=True, exist_ok=True)
     stamp_path = OBJ / "stamp.json"
     stamp = json.loads(stamp_path.read_text()) if stamp_path.exists() else {}
+    cu, cpp = _sources(group)
     nvcc = _nvcc()
-    cu = sorted(CSRC.glob("*.cu")) + sorted((CSRC / "fused").glob("*.cu"))
-    cpp = sorted((CSRC / "host").glob("*.cpp"))
     logs = {}
     with ThreadPoolExecutor(max_workers=max(1, (os.cpu_count() or 4))) as pool:
         cu_jobs = [pool.submit(_compile_one, s, NVCC_FLAGS, nvcc, stamp, force, verbose) for s in cu]
@@ -90,33 +128,17 @@ def build(force: bool = False, verbose: bool = False) -> dict:
         cpp_res = [j.result() for j in cpp_jobs]
     for (obj, _, log), src in zip(cu_res, cu):
         logs[src.name] = log
+    kern, host = library_paths(group)
+    _link([nvcc, "-shared", "-gencode", "arch=compute_100a,code=sm_100a", "-lcudart"], kern,
+          [o for o, _, _ in cu_res], stamp, force)
+    _link(["g++", "-shared", "-pthread"], host, [o for o, _, _ in cpp_res], stamp, force)
     stamp_path.write_text(json.dumps(stamp, indent=0))
-    out = {}
-    kern = LIB / "libus_kernels.so"
-    if cu_res and (force or not kern.exists() or any(c for _, c, _ in cu_res)):
-        tmp = kern.with_suffix(".so.tmp")       # linked aside, then moved into place at once
-        cmd = [nvcc, "-shared", "-o", str(tmp), *[str(o) for o, _, _ in cu_res],
-               "-gencode", "arch=compute_100a,code=sm_100a", "-lcudart"]
-        proc = subprocess.run(cmd, capture_output=True, text=True)
-        if proc.returncode != 0:
-            raise RuntimeError(f"link failed: {proc.stdout}{proc.stderr}")
-        os.replace(tmp, kern)
-    out["kernels"] = kern
-    host = LIB / "libus_host.so"
-    if cpp_res and (force or not host.exists() or any(c for _, c, _ in cpp_res)):
-        tmp = host.with_suffix(".so.tmp")
-        cmd = ["g++", "-shared", "-o", str(tmp), *[str(o) for o, _, _ in cpp_res], "-pthread"]
-        proc = subprocess.run(cmd, capture_output=True, text=True)
-        if proc.returncode != 0:
-            raise RuntimeError(f"link failed: {proc.stdout}{proc.stderr}")
-        os.replace(tmp, host)
-    out["host"] = host
-    out["logs"] = logs
-    return out
+    return {"kernels": kern, "host": host, "logs": logs}
 
 
 def main(argv: list[str]) -> int:
-    res = build(force="--force" in argv, verbose="--verbose" in argv)
+    group = argv[argv.index("--group") + 1] if "--group" in argv else None
+    res = build(force="--force" in argv, verbose="--verbose" in argv, group=group)
     print("built:", res["kernels"], res["host"])
     return 0
 

@@ -181,14 +181,16 @@ FAMILIES = {
     "Qwen4ExpForConditionalGeneration": "qwen4_exp", "Qwen4ExpForCausalLM": "qwen4_exp",
     "MiniMaxH3Pipeline": "minimax_h3", "FastH3Pipeline": "minimax_h3",
     "MiniMaxH3Transformer3DModel": "minimax_h3",
+    "Nepevik": "nepevik",
 }
 
 
 def resolve_family(directory) -> str:
-    """Family of a checkpoint: transformers ``config.json`` -> ``architectures[0]``;
-    diffusers ``model_index.json`` / ``modular_model_index.json`` -> ``_class_name``."""
+    """Family of a checkpoint: ``config.json`` -> ``architectures[0]`` (transformers) or
+    ``architecture``; diffusers ``model_index.json`` / ``modular_model_index.json`` -> ``_class_name``."""
     d = Path(directory)
-    for fn, key in (("config.json", "architectures"), ("model_index.json", "_class_name"),
+    for fn, key in (("config.json", "architectures"), ("config.json", "architecture"),
+                    ("model_index.json", "_class_name"),
                     ("modular_model_index.json", "_class_name")):
         p = d / fn
         if p.exists():

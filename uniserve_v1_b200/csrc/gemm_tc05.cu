@@ -787,6 +787,10 @@ gemm_wx_pair_kernel(const __grid_constant__ CUtensorMap tmA,
               if (f0 + c + j < M)
                 x[j] += bias_f ? bias_f[f0 + c + j] : us::bf2f(bias_h[f0 + c + j]);
           }
+          if (SWAP == 2 && act == 3) {
+#pragma unroll
+            for (int j = 0; j < 16; ++j) x[j] = gelu_erf_f(x[j]);
+          }
           if (lines) {
             const int ch = (c & 63) >> 3;     // first of this piece's two 16-byte chunks
             uint32_t o[8];

@@ -15,6 +15,7 @@ struct GemmArgs {
   int stages;
   int early;        // dense: weight tiles of the first stages are fetched before the PDL wait
   int act;          // dual: 0 = silu fused rounding, 1 = silu stepwise rounding, 2 = gelu-tanh
+                    // single: 0 = none, 3 = gelu (erf) of the biased value
   int out_dtype;    // 0 = bf16, 1 = fp32
   int bias_dtype;   // 0 = bf16, 1 = fp32
   long long ldo;
@@ -82,6 +83,10 @@ __device__ __forceinline__ float silu_f(float x) { return x / (1.f + __expf(-x))
 __device__ __forceinline__ float gelu_tanh_f(float x) {
   const float k0 = 0.7978845608028654f, k1 = 0.044715f;
   return 0.5f * x * (1.f + tanhf(k0 * (x + k1 * x * x * x)));
+}
+
+__device__ __forceinline__ float gelu_erf_f(float x) {
+  return 0.5f * x * (1.f + erff(x * 0.70710678118654752f));
 }
 
 template <int BN>
@@ -168,6 +173,7 @@ struct Epilogue {
       }
     }
     val += bias;
+    if (!DUAL && act == 3) val = gelu_erf_f(val);
     if (route_rows != nullptr) return val * route_w[route_rows[r]];
     if (scale_rows != nullptr && !scale_first) val *= scale_rows[r];
     return val;
@@ -210,7 +216,7 @@ struct Epilogue {
     }
     const uint32_t buf = tc::smem_u32(stage) + (uint32_t)(chunk & 1) * (kEpiStageBytes / 2);
     // fast path: nothing per row but the gated activation and the bias
-    const bool plain = scale_rows == nullptr && route_rows == nullptr;
+    const bool plain = scale_rows == nullptr && route_rows == nullptr && (DUAL || act == 0);
     if (esz == 2) {
 #pragma unroll
       for (int j = 0; j < 16; ++j) {

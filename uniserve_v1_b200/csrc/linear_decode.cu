@@ -52,13 +52,17 @@ __device__ __forceinline__ void cp_async16(void* smem, const void* gmem, bool va
                : "memory");
 }
 
+__device__ __forceinline__ float gelu_erf(float x) {
+  return 0.5f * x * (1.f + erff(x * 0.70710678118654752f));
+}
+
 // MT = 16-row tiles of the activation (rows <= 16 * MT).
 template <int MT>
 __global__ void __launch_bounds__(256)
 linear_decode_kernel(const __nv_bfloat16* __restrict__ W, const __nv_bfloat16* __restrict__ X,
                      void* __restrict__ out, const void* __restrict__ bias, int rows, int M, int K,
                      long long ldw, long long ldx, long long ldo, int out_f32, int bias_f32,
-                     int ksplit) {
+                     int ksplit, int act) {
   // Weights are never written by a kernel: the first loads go out before the wait on the
   // kernels that produce the activation.
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
@@ -181,6 +185,7 @@ linear_decode_kernel(const __nv_bfloat16* __restrict__ W, const __nv_bfloat16* _
         if (bias)
           v += bias_f32 ? reinterpret_cast<const float*>(bias)[col]
                         : us::bf2f(reinterpret_cast<const __nv_bfloat16*>(bias)[col]);
+        if (act == 3) v = gelu_erf(v);
         if (out_f32)
           reinterpret_cast<float*>(out)[(long long)r * ldo + col] = v;
         else
@@ -200,6 +205,7 @@ linear_decode_kernel(const __nv_bfloat16* __restrict__ W, const __nv_bfloat16* _
     if (bias)
       v += bias_f32 ? reinterpret_cast<const float*>(bias)[col]
                     : us::bf2f(reinterpret_cast<const __nv_bfloat16*>(bias)[col]);
+    if (act == 3) v = gelu_erf(v);
     if (out_f32)
       reinterpret_cast<float*>(out)[(long long)r * ldo + col] = v;
     else
@@ -209,11 +215,11 @@ linear_decode_kernel(const __nv_bfloat16* __restrict__ W, const __nv_bfloat16* _
 
 }  // namespace
 
-// rows <= 64, K a multiple of 256, 16-byte aligned rows of W and X.  Returns
+// act: 0 none, 3 gelu (erf) of the biased value.  rows <= 64, K a multiple of 256, 16-byte aligned rows of W and X.  Returns
 // US_ERR_UNSUPPORTED for other shapes (the caller then takes the tcgen05 kernel).
 US_API int us_linear_decode(const void* W, const void* X, void* out, const void* bias, int rows,
                             int M, int K, long long ldw, long long ldx, long long ldo,
-                            int out_f32, int bias_f32, void* stream_) {
+                            int out_f32, int bias_f32, int act, void* stream_) {
   US_REQUIRE(W && X && out && rows >= 1 && M >= 1 && K >= 1);
   if (rows > 64 || (K % kIterK) != 0 || (ldw % 8) != 0 || (ldx % 8) != 0 ||
       ((uintptr_t)W % 16) != 0 || ((uintptr_t)X % 16) != 0)
@@ -265,7 +271,7 @@ US_API int us_linear_decode(const void* W, const void* X, void* out, const void*
     cfg.attrs = attr;
     cfg.numAttrs = ksplit > 1 ? 2 : 1;
     return cudaLaunchKernelEx(&cfg, kernel, w, x, out, bias, rows, M, K, ldw, ldx, ldo, out_f32,
-                              bias_f32, ksplit);
+                              bias_f32, ksplit, act);
   };
   // kStages buffers x (16 MT) rows x 512 bytes
   if (rows <= 16)

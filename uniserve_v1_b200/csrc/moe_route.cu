@@ -217,6 +217,32 @@ moe_sort_kernel(const int* __restrict__ ids, int R, int e_lo, int E, int block_n
               tile_group, tile_row0, tile_rows, num_tiles, status);
 }
 
+// Routing by a table over token ids, for the routed layers of a whole forward pass at once (the
+// choice depends on nothing a layer computes): CTA l looks up layer l's experts of every token
+// and sorts its routes.  Buffers of consecutive layers follow one another.
+__global__ void __launch_bounds__(1024)
+table_route_sort_kernel(const int* __restrict__ tokens, const int* __restrict__ tables, int T,
+                        int top, int vocab, int E, int block_n, int max_tiles, int* ids,
+                        int* sorted_route, int* perm_of_route, int* expert_offsets,
+                        int* tile_group, int* tile_row0, int* tile_rows, int* num_tiles,
+                        unsigned int* status) {
+  US_PDL_PROLOGUE();
+  const long long l = blockIdx.x;
+  const int R = T * top;
+  const int* table = tables + l * vocab * top;
+  int* mine = ids + l * R;
+  for (int i = threadIdx.x; i < R; i += blockDim.x) {
+    const int t = i / top, tok = tokens[t];
+    const bool ok = tok >= 0 && tok < vocab;
+    if (!ok) us_dev_fail(status, US_DEV_BOUNDS);
+    mine[i] = ok ? table[(long long)tok * top + (i - t * top)] : 0;
+  }
+  __syncthreads();
+  sort_routes(mine, R, 0, E, block_n, max_tiles, sorted_route + l * R, perm_of_route + l * R,
+              expert_offsets + l * (E + 1), tile_group + l * max_tiles, tile_row0 + l * max_tiles,
+              tile_rows + l * max_tiles, num_tiles + l, status);
+}
+
 // The same sort by a cluster of kSortCtas CTAs for prefill-sized route lists: CTA c counts
 // and scatters the routes [c * chunk, (c + 1) * chunk).  After the local histograms every
 // CTA reads its peers' counts through distributed shared memory: their sum gives the expert
@@ -594,6 +620,23 @@ US_API int us_moe_sort(const int* ids, int R, int e_lo, int E, int block_n, int 
   us::launch_pdl(moe_sort_kernel, dim3(1), dim3(1024), 0, (cudaStream_t)stream_, ids, R, e_lo, E, block_n, max_tiles, sorted_route, perm_of_route, expert_offsets, tile_group,
       tile_row0, tile_rows, num_tiles, us_status_ptr());
   US_LAUNCH_CHECK();
+  return US_OK;
+}
+
+// tokens [T], tables [layers, vocab, top]; outputs per layer as us_moe_sort's, ids [layers, T, top].
+US_API int us_table_route_sort(const int* tokens, const int* tables, int layers, int T, int top,
+                               int vocab, int E, int block_n, int max_tiles, int* ids,
+                               int* sorted_route, int* perm_of_route, int* expert_offsets,
+                               int* tile_group, int* tile_row0, int* tile_rows, int* num_tiles,
+                               void* stream_) {
+  US_REQUIRE(tokens && tables && layers >= 1 && T >= 1 && top >= 1 && vocab >= 1 && E >= 1 &&
+             E <= kMaxExperts && block_n >= 1 && max_tiles >= 1);
+  US_REQUIRE(ids && sorted_route && perm_of_route && expert_offsets && tile_group && tile_row0 &&
+             tile_rows && num_tiles);
+  US_CUDA_CHECK(us::launch_pdl(table_route_sort_kernel, dim3(layers), dim3(1024), 0,
+                               (cudaStream_t)stream_, tokens, tables, T, top, vocab, E, block_n,
+                               max_tiles, ids, sorted_route, perm_of_route, expert_offsets,
+                               tile_group, tile_row0, tile_rows, num_tiles, us_status_ptr()));
   return US_OK;
 }
 

@@ -1,0 +1,599 @@
+// Recurrent mixers whose decay is a vector over the key channels of a head, for packed batches
+// of sequences with their state in slots of a pool:
+//
+//   channel rule   S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;       o = S^T q
+//   general rule   S <- diag(w) S - (a*n)(n^T S) + k v^T  (both read the old S);  o = S^T q
+//
+// with S [D, V] FP32 per (sequence, head).  Three kernels:
+//
+//   us_channel_delta_prep   short causal convolutions + silu of q, k, v, unit q and k, the decay
+//                           g = exp(-exp(A_log) softplus(low + dt_bias)) and beta = sigmoid(b)
+//   us_general_delta_prep   decay w = exp(-c sigmoid(low + w0)), unit key n, removal a * n
+//   us_vector_delta_rule    the recurrence
+//   us_head_norm_gate       per-head RMS norm of o, weight, sigmoid gate
+//
+// The preparation is parallel over tokens, so the recurrence reads finished FP32 vectors and
+// does nothing but its multiply-adds.  A sequence whose first packed row stands at position 0
+// starts from a zero state whatever its slot holds: slots are handed on without being cleared,
+// and nothing has to be launched when a request is admitted.  A negative slot marks padding.
+//
+// Rule kernel: a CTA owns 32 value columns of one head of one sequence.  Four warps compute:
+// a lane holds D/16 rows x 4 columns of S in registers (16 lanes span the rows, so one 16-byte
+// access per row moves 4 columns, and 4 independent chains hide the FMA latency); the two
+// D-long reductions of a token fold 4 columns over 16 lanes in five shuffles.  Four more warps
+// stage the vectors of the next tokens into the other half of shared memory meanwhile.  The
+// state crosses HBM once per call.
+#include "include/us_common.cuh"
+
+namespace {
+
+__device__ __forceinline__ float ld_any(const void* base, long long idx, int bf16) {
+  return bf16 ? us::bf2f(reinterpret_cast<const __nv_bfloat16*>(base)[idx])
+              : reinterpret_cast<const float*>(base)[idx];
+}
+__device__ __forceinline__ void st_any(void* base, long long idx, int bf16, float v) {
+  if (bf16) reinterpret_cast<__nv_bfloat16*>(base)[idx] = us::f2bf(v);
+  else reinterpret_cast<float*>(base)[idx] = v;
+}
+__device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
+__device__ __forceinline__ float softplus_f(float x) {
+  return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x)));
+}
+
+// e^x of a decay.  Hundreds of factors just below one multiply along a sequence, so a bias of
+// half an ulp each would add up: near zero the rounding of 1 + (e^x - 1) is the nearest one.
+__device__ __forceinline__ float decay_exp(float x) { return x > -0.5f ? 1.f + expm1f(x) : expf(x); }
+
+// sequence that holds packed row t (cu is ascending, cu[0] = 0, cu[B] = rows)
+__device__ __forceinline__ int seq_of(const int* cu, int B, int t) {
+  int lo = 0, hi = B - 1;
+  while (lo < hi) {
+    const int mid = (lo + hi + 1) >> 1;
+    if (cu[mid] <= t) lo = mid; else hi = mid - 1;
+  }
+  return lo;
+}
+
+constexpr int kMaxTaps = 8;
+constexpr int kMaxDim = 256;      // key channels per head
+constexpr int kPrepTokens = 4;    // consecutive rows of one warp in the prefill form
+
+struct ChannelPrep {
+  const void* x;                // projection rows, element type = bf16 flag
+  long long ldx;
+  int off_q, off_k, off_v, off_b;
+  const float *cq, *ck, *cv;    // taps [channels, K]
+  const float* low;             // [rows, H * D]
+  long long ldlow;
+  const float *A_log, *dt_bias; // [H], [H * D]
+  void* conv;                   // [slots, K - 1, C], C = 2 Hk D + H V
+  float *q, *k, *v, *g, *beta;  // [rows, Hk, D] x 2, [rows, H, V], [rows, H, D], [rows, H]
+  const int *cu, *slots, *pos;
+  int B, rows, H, Hk, D, V, K, bf16, one_token;
+};
+
+// A warp owns one head of q, of k, of v or of the decay for kPrepTokens rows (prefill) or one
+// row (every sequence brings one token: the warp then also shifts its channels' window).
+__global__ void __launch_bounds__(256) channel_prep_kernel(const ChannelPrep a) {
+  US_PDL_PROLOGUE();
+  const int lane = threadIdx.x & 31;
+  const int unit = blockIdx.y * 8 + (threadIdx.x >> 5);
+  const int units = 2 * a.Hk + 2 * a.H;
+  if (unit >= units) return;
+  const int per = a.one_token ? 1 : kPrepTokens;
+  const int t0 = blockIdx.x * per, t1 = min(a.rows, t0 + per);
+  if (unit >= 2 * a.Hk + a.H) {                       // decay and step size
+    const int h = unit - 2 * a.Hk - a.H;
+    const float A = expf(a.A_log[h]);
+    for (int t = t0; t < t1; ++t) {
+      const float* lo = a.low + (long long)t * a.ldlow + (long long)h * a.D;
+      float* g = a.g + ((long long)t * a.H + h) * a.D;
+      for (int d = lane; d < a.D; d += 32)
+        g[d] = decay_exp(-A * softplus_f(lo[d] + a.dt_bias[h * a.D + d]));
+      if (lane == 0)
+        a.beta[(long long)t * a.H + h] =
+            sigmoid_f(ld_any(a.x, (long long)t * a.ldx + a.off_b + h, a.bf16));
+    }
+    return;
+  }
+  int head, dim, off, cbase;
+  const float* taps;
+  if (unit < a.Hk) {
+    head = unit; dim = a.D; off = a.off_q + head * a.D; taps = a.cq + (long long)head * a.D * a.K;
+    cbase = head * a.D;
+  } else if (unit < 2 * a.Hk) {
+    head = unit - a.Hk; dim = a.D; off = a.off_k + head * a.D;
+    taps = a.ck + (long long)head * a.D * a.K;
+    cbase = a.Hk * a.D + head * a.D;
+  } else {
+    head = unit - 2 * a.Hk; dim = a.V; off = a.off_v + head * a.V;
+    taps = a.cv + (long long)head * a.V * a.K;
+    cbase = 2 * a.Hk * a.D + head * a.V;
+  }
+  const long long C = 2LL * a.Hk * a.D + (long long)a.H * a.V;
+  for (int t = t0; t < t1; ++t) {
+    const int s = seq_of(a.cu, a.B, t);
+    const int start = a.cu[s], slot = a.slots[s];
+    if (slot < 0) continue;
+    const bool fresh = a.pos[start] == 0;
+    const long long sbase = (long long)slot * (a.K - 1) * C + cbase;
+    float y[kMaxDim / 32];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < kMaxDim / 32; ++i) {
+      const int d = i * 32 + lane;
+      y[i] = 0.f;
+      if (d >= dim) continue;
+      float acc = 0.f;
+      for (int j = 0; j < a.K; ++j) {
+        const int src = t - (a.K - 1) + j;            // packed row of the tap
+        float xv;
+        if (src >= start)
+          xv = ld_any(a.x, (long long)src * a.ldx + off + d, a.bf16);
+        else
+          xv = fresh ? 0.f
+                     : ld_any(a.conv, sbase + (long long)(src - start + a.K - 1) * C + d, a.bf16);
+        acc += taps[(long long)d * a.K + j] * xv;
+        // one token per sequence: entry j of the old window becomes entry j - 1 of the new
+        if (a.one_token && j > 0) st_any(a.conv, sbase + (long long)(j - 1) * C + d, a.bf16, xv);
+      }
+      y[i] = acc / (1.f + expf(-acc));
+      ss += y[i] * y[i];
+    }
+    if (unit < 2 * a.Hk) {
+      float inv = 1.f / sqrtf(us::warp_sum(ss) + 1e-6f);
+      if (unit < a.Hk) inv *= 1.f / sqrtf((float)a.D);
+      float* dst = (unit < a.Hk ? a.q : a.k) + ((long long)t * a.Hk + head) * a.D;
+#pragma unroll
+      for (int i = 0; i < kMaxDim / 32; ++i)
+        if (i * 32 + lane < dim) dst[i * 32 + lane] = y[i] * inv;
+    } else {
+      float* dst = a.v + ((long long)t * a.H + head) * a.V;
+#pragma unroll
+      for (int i = 0; i < kMaxDim / 32; ++i)
+        if (i * 32 + lane < dim) dst[i * 32 + lane] = y[i];
+    }
+  }
+}
+
+// New window of every sequence: the last K - 1 rows of [old window; rows of this call].  A
+// thread owns one channel and walks the entries upwards, so each is read before it is written.
+__global__ void __launch_bounds__(256) conv_window_kernel(const ChannelPrep a) {
+  US_PDL_PROLOGUE();
+  const int c = blockIdx.x * 256 + threadIdx.x;
+  const int nq = a.Hk * a.D, C = 2 * nq + a.H * a.V;
+  if (c >= C) return;
+  const int s = blockIdx.y;
+  const int start = a.cu[s], T = a.cu[s + 1] - start, slot = a.slots[s];
+  if (slot < 0 || T <= 0) return;
+  const bool fresh = a.pos[start] == 0;
+  const int col = c < nq ? a.off_q + c : c < 2 * nq ? a.off_k + c - nq : a.off_v + c - 2 * nq;
+  const long long base = (long long)slot * (a.K - 1) * C + c;
+  for (int j = 0; j < a.K - 1; ++j) {
+    const int src = T + j;
+    float v;
+    if (src < a.K - 1) v = fresh ? 0.f : ld_any(a.conv, base + (long long)src * C, a.bf16);
+    else v = ld_any(a.x, (long long)(start + src - (a.K - 1)) * a.ldx + col, a.bf16);
+    st_any(a.conv, base + (long long)j * C, a.bf16, v);
+  }
+}
+
+struct GeneralPrep {
+  const void* x;
+  long long ldx;
+  int off_k, off_a;
+  const float* low;             // [rows, H * D] (before w0)
+  long long ldlow;
+  const float *w0, *a_bias;     // [H * D]
+  float *w, *n, *p;             // [rows, H, D]
+  int rows, H, D, bf16;
+  float rate;                   // w = exp(-rate * sigmoid(.))
+};
+
+// One warp per (row, head).
+__global__ void __launch_bounds__(256) general_prep_kernel(const GeneralPrep a) {
+  US_PDL_PROLOGUE();
+  const long long r = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  if (r >= (long long)a.rows * a.H) return;
+  const int t = (int)(r / a.H), h = (int)(r - (long long)t * a.H);
+  const long long xr = (long long)t * a.ldx + (long long)h * a.D;
+  float kv[kMaxDim / 32], ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < kMaxDim / 32; ++i) {
+    const int d = i * 32 + lane;
+    kv[i] = d < a.D ? ld_any(a.x, xr + a.off_k + d, a.bf16) : 0.f;
+    ss += kv[i] * kv[i];
+  }
+  const float inv = 1.f / sqrtf(us::warp_sum(ss) + 1e-6f);
+#pragma unroll
+  for (int i = 0; i < kMaxDim / 32; ++i) {
+    const int d = i * 32 + lane;
+    if (d >= a.D) continue;
+    const int hd = h * a.D + d;
+    const float n = kv[i] * inv;
+    a.w[r * a.D + d] =
+        decay_exp(-a.rate * sigmoid_f(a.low[(long long)t * a.ldlow + hd] + a.w0[hd]));
+    a.n[r * a.D + d] = n;
+    a.p[r * a.D + d] = n * sigmoid_f(ld_any(a.x, xr + a.off_a + d, a.bf16) + a.a_bias[hd]);
+  }
+}
+
+constexpr int kCols = 32;         // value columns per CTA
+constexpr int kChunk = 8;         // tokens staged per round
+constexpr int kComputeThreads = 128;
+
+struct RuleArgs {
+  const void *q, *k, *v;          // element (t, h, i) at t * ld + h * hs + i
+  long long ldq, ldk, ldv;
+  int hsq, hsk, hsv;
+  int q_bf16, k_bf16, v_bf16;
+  const float* g;                 // decay [rows, H, D]
+  const float* n;                 // general: removal direction [rows, H, D]
+  const float* p;                 // general: removal rate * direction [rows, H, D]
+  const float* beta;              // channel: [rows, H]
+  float* state;                   // [slots, H, D, V]
+  float* out;                     // [rows, H, V]
+  const int *cu, *slots, *pos;
+  int H, Hk, D, V;
+};
+
+// Folds four per-lane column sums over the 16 lanes that span the rows: afterwards every lane
+// holds the sum of column ((lane >> 3) & 1) * 2 + ((lane >> 2) & 1).
+__device__ __forceinline__ float fold16(float c0, float c1, float c2, float c3, int lane) {
+  const bool up = lane & 8;
+  const float a0 = up ? c2 : c0, a1 = up ? c3 : c1, b0 = up ? c0 : c2, b1 = up ? c1 : c3;
+  const float s0 = a0 + __shfl_xor_sync(0xffffffffu, b0, 8);
+  const float s1 = a1 + __shfl_xor_sync(0xffffffffu, b1, 8);
+  const bool odd = lane & 4;
+  float s = (odd ? s1 : s0) + __shfl_xor_sync(0xffffffffu, odd ? s0 : s1, 4);
+  s += __shfl_xor_sync(0xffffffffu, s, 2);
+  s += __shfl_xor_sync(0xffffffffu, s, 1);
+  return s;
+}
+
+
+template <int W>
+__device__ __forceinline__ void lds_vec(float (&o)[W], const float* p) {
+  if (W == 4) {
+    const float4 v = *reinterpret_cast<const float4*>(p);
+    o[0] = v.x; o[1 % W] = v.y; o[2 % W] = v.z; o[3 % W] = v.w;
+  } else if (W == 2) {
+    const float2 v = *reinterpret_cast<const float2*>(p);
+    o[0] = v.x; o[1 % W] = v.y;
+  } else {
+    o[0] = p[0];
+  }
+}
+
+// Vectors of token slot i in shared memory: kVecs rows of DP floats, then 32 columns of v.
+template <int DP, bool GENERAL>
+struct Stage {
+  static constexpr int kVecs = GENERAL ? 5 : 3;       // g, k, q (, n, p)
+  static constexpr int kToken = kVecs * DP + kCols + 4;
+  static constexpr int kFloats = kChunk * kToken;
+};
+
+template <int DP, bool GENERAL>
+__device__ __forceinline__ void stage_tokens(const RuleArgs& a, float* buf, int start, int c0, int n,
+                                             int h, int hk, int col0, int tid, int nthreads) {
+  using St = Stage<DP, GENERAL>;
+  const bool quad = (a.D & 3) == 0;
+  if (quad && !a.q_bf16 && !a.k_bf16 && ((a.ldq | a.ldk | a.hsq | a.hsk) & 3) == 0) {
+    constexpr int kQ = DP / 4;
+    for (int e = tid; e < n * St::kVecs * kQ; e += nthreads) {
+      const int i = e / (St::kVecs * kQ), rest = e - i * St::kVecs * kQ;
+      const int vec = rest / kQ, d = (rest - vec * kQ) * 4;
+      const long long row = start + c0 + i;
+      float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (d < a.D) {
+        const float* src;
+        if (vec == 1) src = (const float*)a.k + row * a.ldk + (long long)hk * a.hsk + d;
+        else if (vec == 2) src = (const float*)a.q + row * a.ldq + (long long)hk * a.hsq + d;
+        else src = (vec == 0 ? a.g : vec == 3 ? a.n : a.p) + (row * a.H + h) * a.D + d;
+        x = *reinterpret_cast<const float4*>(src);
+      }
+      *reinterpret_cast<float4*>(buf + i * St::kToken + vec * DP + d) = x;
+    }
+  } else {
+    for (int e = tid; e < n * St::kVecs * DP; e += nthreads) {
+      const int i = e / (St::kVecs * DP), rest = e - i * St::kVecs * DP;
+      const int vec = rest / DP, d = rest - vec * DP;
+      const long long row = start + c0 + i;
+      float x = 0.f;
+      if (d < a.D) {
+        if (vec == 1) x = ld_any(a.k, row * a.ldk + (long long)hk * a.hsk + d, a.k_bf16);
+        else if (vec == 2) x = ld_any(a.q, row * a.ldq + (long long)hk * a.hsq + d, a.q_bf16);
+        else x = (vec == 0 ? a.g : vec == 3 ? a.n : a.p)[(row * a.H + h) * a.D + d];
+      }
+      buf[i * St::kToken + vec * DP + d] = x;
+    }
+  }
+  for (int e = tid; e < n * (kCols + 1); e += nthreads) {
+    const int i = e / (kCols + 1), c = e - i * (kCols + 1);
+    const long long row = start + c0 + i;
+    float x = 0.f;
+    if (c == kCols) x = GENERAL ? 0.f : a.beta[row * a.H + h];
+    else if (col0 + c < a.V) x = ld_any(a.v, row * a.ldv + (long long)h * a.hsv + col0 + c, a.v_bf16);
+    buf[i * St::kToken + St::kVecs * DP + c] = x;
+  }
+}
+
+template <int DP, bool GENERAL>
+__global__ void __launch_bounds__(256) vector_delta_kernel(const RuleArgs a) {
+  US_PDL_PROLOGUE();
+  using St = Stage<DP, GENERAL>;
+  constexpr int R = DP / 16;                          // rows per lane
+  constexpr int W = R >= 4 ? 4 : R;                   // rows per shared-memory access
+  constexpr int NG = R / W;
+  extern __shared__ __align__(16) float sm[];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int h = blockIdx.y, s = blockIdx.z;
+  const int hk = h / (a.H / a.Hk);
+  const int col0 = blockIdx.x * kCols;
+  const int start = a.cu[s], T = a.cu[s + 1] - start, slot = a.slots[s];
+  if (T <= 0) return;
+  if (slot < 0) {                                     // padding: defined rows, no state
+    for (int e = tid; e < T * kCols; e += 256) {
+      const int t = e / kCols, c = col0 + e - t * kCols;
+      if (c < a.V) a.out[((long long)(start + t) * a.H + h) * a.V + c] = 0.f;
+    }
+    return;
+  }
+  const bool loader = warp >= kComputeThreads / 32;
+  const int rl = lane & 15;
+  const int my = ((lane >> 3) & 1) * 2 + ((lane >> 2) & 1);        // column a fold leaves here
+  const int cb = (warp & 3) * 8 + (lane >> 4) * 4;                 // first of the lane's columns
+  float* Sg = a.state + (((long long)slot * a.H + h) * a.D) * a.V + col0 + cb;
+  const bool wide = (a.V & 3) == 0;
+  float S[R][4];
+  if (loader) {
+    stage_tokens<DP, GENERAL>(a, sm, start, 0, min(kChunk, T), h, hk, col0, tid - kComputeThreads,
+                              256 - kComputeThreads);
+  } else {
+    const bool fresh = a.pos[start] == 0;
+#pragma unroll
+    for (int j = 0; j < NG; ++j)
+#pragma unroll
+      for (int e = 0; e < W; ++e) {
+        const int row = (j * 16 + rl) * W + e;
+        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (!fresh && row < a.D) {
+          const float* p = Sg + (long long)row * a.V;
+          if (wide) {
+            if (col0 + cb < a.V) x = *reinterpret_cast<const float4*>(p);
+          } else {
+            if (col0 + cb < a.V) x.x = p[0];
+            if (col0 + cb + 1 < a.V) x.y = p[1];
+            if (col0 + cb + 2 < a.V) x.z = p[2];
+            if (col0 + cb + 3 < a.V) x.w = p[3];
+          }
+        }
+        S[j * W + e][0] = x.x; S[j * W + e][1] = x.y; S[j * W + e][2] = x.z; S[j * W + e][3] = x.w;
+      }
+  }
+  __syncthreads();
+  int buf = 0;
+  for (int c0 = 0; c0 < T; c0 += kChunk, buf ^= 1) {
+    const int n = min(kChunk, T - c0);
+    if (loader) {
+      if (c0 + kChunk < T)
+        stage_tokens<DP, GENERAL>(a, sm + (buf ^ 1) * St::kFloats, start, c0 + kChunk,
+                                  min(kChunk, T - c0 - kChunk), h, hk, col0, tid - kComputeThreads,
+                                  256 - kComputeThreads);
+    } else {
+      const float* base = sm + buf * St::kFloats;
+      for (int t = 0; t < n; ++t, base += St::kToken) {
+        const float* gs = base;
+        const float* ks = base + DP;
+        const float* qs = base + 2 * DP;
+        const float* vs = base + St::kVecs * DP;
+        float y0 = 0.f, y1 = 0.f, y2 = 0.f, y3 = 0.f;
+#pragma unroll
+        for (int j = 0; j < NG; ++j) {
+          const int r0 = (j * 16 + rl) * W;
+          float m[W];
+          if (GENERAL) {
+            lds_vec<W>(m, base + 3 * DP + r0);
+          } else {
+            float g[W];
+            lds_vec<W>(m, ks + r0);
+            lds_vec<W>(g, gs + r0);
+#pragma unroll
+            for (int e = 0; e < W; ++e) {
+              // the state is decayed first; what the key sees is the decayed state
+              S[j * W + e][0] *= g[e]; S[j * W + e][1] *= g[e];
+              S[j * W + e][2] *= g[e]; S[j * W + e][3] *= g[e];
+            }
+          }
+#pragma unroll
+          for (int e = 0; e < W; ++e) {
+            y0 = fmaf(S[j * W + e][0], m[e], y0);
+            y1 = fmaf(S[j * W + e][1], m[e], y1);
+            y2 = fmaf(S[j * W + e][2], m[e], y2);
+            y3 = fmaf(S[j * W + e][3], m[e], y3);
+          }
+        }
+        const float seen = fold16(y0, y1, y2, y3, lane);
+        float c = seen;                               // general: n^T S of this lane's column
+        if (!GENERAL) c = vs[kCols] * (vs[cb + my] - seen);
+        const int half = lane & 16;
+        const float u0 = __shfl_sync(0xffffffffu, c, half);
+        const float u1 = __shfl_sync(0xffffffffu, c, half | 4);
+        const float u2 = __shfl_sync(0xffffffffu, c, half | 8);
+        const float u3 = __shfl_sync(0xffffffffu, c, half | 12);
+        float4 vv;
+        if (GENERAL) vv = *reinterpret_cast<const float4*>(vs + cb);
+        float o0 = 0.f, o1 = 0.f, o2 = 0.f, o3 = 0.f;
+#pragma unroll
+        for (int j = 0; j < NG; ++j) {
+          const int r0 = (j * 16 + rl) * W;
+          float k[W], q[W];
+          lds_vec<W>(k, ks + r0);
+          lds_vec<W>(q, qs + r0);
+          if (GENERAL) {
+            float g[W], p[W];
+            lds_vec<W>(g, gs + r0);
+            lds_vec<W>(p, base + 4 * DP + r0);
+#pragma unroll
+            for (int e = 0; e < W; ++e) {
+              float* x = S[j * W + e];
+              x[0] = fmaf(k[e], vv.x, fmaf(-p[e], u0, g[e] * x[0]));
+              x[1] = fmaf(k[e], vv.y, fmaf(-p[e], u1, g[e] * x[1]));
+              x[2] = fmaf(k[e], vv.z, fmaf(-p[e], u2, g[e] * x[2]));
+              x[3] = fmaf(k[e], vv.w, fmaf(-p[e], u3, g[e] * x[3]));
+            }
+          } else {
+#pragma unroll
+            for (int e = 0; e < W; ++e) {
+              float* x = S[j * W + e];
+              x[0] = fmaf(k[e], u0, x[0]); x[1] = fmaf(k[e], u1, x[1]);
+              x[2] = fmaf(k[e], u2, x[2]); x[3] = fmaf(k[e], u3, x[3]);
+            }
+          }
+#pragma unroll
+          for (int e = 0; e < W; ++e) {
+            o0 = fmaf(S[j * W + e][0], q[e], o0);
+            o1 = fmaf(S[j * W + e][1], q[e], o1);
+            o2 = fmaf(S[j * W + e][2], q[e], o2);
+            o3 = fmaf(S[j * W + e][3], q[e], o3);
+          }
+        }
+        const float o = fold16(o0, o1, o2, o3, lane);
+        if ((lane & 3) == 0 && col0 + cb + my < a.V)
+          a.out[((long long)(start + c0 + t) * a.H + h) * a.V + col0 + cb + my] = o;
+      }
+    }
+    __syncthreads();
+  }
+  if (loader) return;
+#pragma unroll
+  for (int j = 0; j < NG; ++j)
+#pragma unroll
+    for (int e = 0; e < W; ++e) {
+      const int row = (j * 16 + rl) * W + e;
+      if (row >= a.D) continue;
+      float* p = Sg + (long long)row * a.V;
+      const float* x = S[j * W + e];
+      if (wide) {
+        if (col0 + cb < a.V) *reinterpret_cast<float4*>(p) = make_float4(x[0], x[1], x[2], x[3]);
+      } else {
+        for (int i = 0; i < 4; ++i)
+          if (col0 + cb + i < a.V) p[i] = x[i];
+      }
+    }
+}
+
+// y = o / rms(o over V) * w * sigmoid(gate), one warp per (row, head); columns past H * V of
+// the (padded) output row are zeroed by the last head's warp.
+__global__ void __launch_bounds__(256)
+head_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ w, int w_head_stride,
+                      const void* __restrict__ gate, long long ldg, void* __restrict__ y,
+                      long long ldy, int rows, int H, int V, float eps, int bf16, int gate_bf16) {
+  US_PDL_PROLOGUE();
+  const long long r = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  if (r >= (long long)rows * H) return;
+  const int t = (int)(r / H), h = (int)(r - (long long)t * H);
+  const float* x = o + r * V;
+  float ss = 0.f;
+  for (int c = lane; c < V; c += 32) ss += x[c] * x[c];
+  const float inv = 1.f / sqrtf(us::warp_sum(ss) / (float)V + eps);
+  for (int c = lane; c < V; c += 32) {
+    const float gv = ld_any(gate, (long long)t * ldg + h * V + c, gate_bf16);
+    st_any(y, (long long)t * ldy + h * V + c, bf16,
+           x[c] * inv * w[h * w_head_stride + c] * sigmoid_f(gv));
+  }
+  if (h == H - 1)
+    for (long long c = (long long)H * V + lane; c < ldy; c += 32)
+      st_any(y, (long long)t * ldy + c, bf16, 0.f);
+}
+
+template <int DP, bool GENERAL>
+int launch_rule(const RuleArgs& a, int B, cudaStream_t stream) {
+  constexpr size_t smem = 2 * Stage<DP, GENERAL>::kFloats * sizeof(float);
+  static bool configured = false;
+  if (!configured && smem > 48 * 1024) {
+    US_CUDA_CHECK(cudaFuncSetAttribute(vector_delta_kernel<DP, GENERAL>,
+                                       cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  }
+  configured = true;
+  US_CUDA_CHECK(us::launch_pdl(vector_delta_kernel<DP, GENERAL>,
+                               dim3((a.V + kCols - 1) / kCols, a.H, B), dim3(256), smem, stream, a));
+  return US_OK;
+}
+
+}  // namespace
+
+// x: projection rows holding q at off_q, k at off_k, v at off_v and the step size at off_b.
+// one_token: every sequence of the batch brings exactly one row (rows == B).
+US_API int us_channel_delta_prep(const void* x, long long ldx, int off_q, int off_k, int off_v,
+                                 int off_b, const float* cq, const float* ck, const float* cv,
+                                 const float* low, long long ldlow, const float* A_log,
+                                 const float* dt_bias, void* conv, float* q, float* k, float* v,
+                                 float* g, float* beta, const int* cu, const int* slots,
+                                 const int* pos, int B, int rows, int H, int Hk, int D, int V, int K,
+                                 int bf16, int one_token, void* stream_) {
+  US_REQUIRE(x && cq && ck && cv && low && A_log && dt_bias && q && k && v && g && beta && cu &&
+             slots && pos && B >= 1 && rows >= 1 && H >= 1 && Hk >= 1 && H % Hk == 0);
+  US_REQUIRE(K == 1 || conv);
+  US_REQUIRE(!one_token || rows == B);
+  if (K < 1 || K > kMaxTaps || D < 1 || D > kMaxDim || V < 1 || V > kMaxDim)
+    return US_ERR_UNSUPPORTED;
+  ChannelPrep a{x, ldx, off_q, off_k, off_v, off_b, cq, ck, cv, low, ldlow, A_log, dt_bias, conv,
+                q, k, v, g, beta, cu, slots, pos, B, rows, H, Hk, D, V, K, bf16, one_token};
+  cudaStream_t stream = (cudaStream_t)stream_;
+  const int per = one_token ? 1 : kPrepTokens;
+  const int units = 2 * Hk + 2 * H;
+  US_CUDA_CHECK(us::launch_pdl(channel_prep_kernel, dim3((rows + per - 1) / per, (units + 7) / 8),
+                               dim3(256), 0, stream, a));
+  if (!one_token && K > 1)
+    US_CUDA_CHECK(us::launch_pdl(conv_window_kernel, dim3((2 * Hk * D + H * V + 255) / 256, B),
+                                 dim3(256), 0, stream, a));
+  return US_OK;
+}
+
+US_API int us_general_delta_prep(const void* x, long long ldx, int off_k, int off_a,
+                                 const float* low, long long ldlow, const float* w0,
+                                 const float* a_bias, float* w, float* n, float* p, int rows, int H,
+                                 int D, float rate, int bf16, void* stream_) {
+  US_REQUIRE(x && low && w0 && a_bias && w && n && p && rows >= 1 && H >= 1);
+  if (D < 1 || D > kMaxDim) return US_ERR_UNSUPPORTED;
+  GeneralPrep a{x, ldx, off_k, off_a, low, ldlow, w0, a_bias, w, n, p, rows, H, D, bf16, rate};
+  const long long warps = (long long)rows * H;
+  US_CUDA_CHECK(us::launch_pdl(general_prep_kernel, dim3((unsigned)((warps + 7) / 8)), dim3(256), 0,
+                               (cudaStream_t)stream_, a));
+  return US_OK;
+}
+
+// general = 0: the channel rule (g, beta); 1: the general rule (g, n, p).  q and k heads serve
+// H / Hk value heads each.
+US_API int us_vector_delta_rule(int general, const void* q, const void* k, const void* v,
+                                long long ldq, long long ldk, long long ldv, int hsq, int hsk,
+                                int hsv, int q_bf16, int k_bf16, int v_bf16, const float* g,
+                                const float* n, const float* p, const float* beta, float* state,
+                                float* out, const int* cu, const int* slots, const int* pos, int B,
+                                int H, int Hk, int D, int V, void* stream_) {
+  US_REQUIRE(q && k && v && g && state && out && cu && slots && pos && B >= 1 && B <= 65535);
+  US_REQUIRE(general ? (n && p) : (beta != nullptr));
+  US_REQUIRE(H >= 1 && Hk >= 1 && H % Hk == 0 && H <= 65535 && D >= 1 && V >= 1);
+  RuleArgs a{q, k, v, ldq, ldk, ldv, hsq, hsk, hsv, q_bf16, k_bf16, v_bf16, g, n, p, beta, state,
+             out, cu, slots, pos, H, Hk, D, V};
+  cudaStream_t stream = (cudaStream_t)stream_;
+#define US_VD(DP) \
+  if (D <= DP) return general ? launch_rule<DP, true>(a, B, stream) : launch_rule<DP, false>(a, B, stream);
+  US_VD(16) US_VD(32) US_VD(64) US_VD(128) US_VD(256)
+#undef US_VD
+  return US_ERR_UNSUPPORTED;
+}
+
+US_API int us_head_norm_gate(const float* o, const float* w, int w_head_stride, const void* gate,
+                             long long ldg, void* y, long long ldy, int rows, int H, int V,
+                             float eps, int bf16, int gate_bf16, void* stream_) {
+  US_REQUIRE(o && w && gate && y && rows >= 1 && H >= 1 && V >= 1 && ldy >= (long long)H * V);
+  const long long warps = (long long)rows * H;
+  US_CUDA_CHECK(us::launch_pdl(head_norm_gate_kernel, dim3((unsigned)((warps + 7) / 8)), dim3(256),
+                               0, (cudaStream_t)stream_, o, w, w_head_stride, gate, ldg, y, ldy, rows,
+                               H, V, eps, bf16, gate_bf16));
+  return US_OK;
+}

@@ -53,6 +53,7 @@ class BlockManager:
         self.num_pages = num_pages
         self.kv_events = None        # server.export.KvEventPublisher of this scheduler
         self.page_size = page_size
+        self.prefix_cache_allowed = True     # False: the model cannot continue from pages alone
         self.enable_prefix_cache = enable_prefix_cache
         self.identity = weights_identity
         self.h = self.lib.us_bm_create(num_pages, page_size)
@@ -66,6 +67,14 @@ class BlockManager:
                 self.h = None
         except Exception:
             pass
+
+    @property
+    def enable_prefix_cache(self) -> bool:
+        return self._prefix_cache and self.prefix_cache_allowed
+
+    @enable_prefix_cache.setter
+    def enable_prefix_cache(self, on: bool) -> None:
+        self._prefix_cache = bool(on)
 
     # -------------------------------------------------------------- host tier --
     def enable_host_tier(self, slots: int) -> None:

@@ -114,6 +114,9 @@ class LLMEngine:
                  host_reserve_gib: Optional[float] = None):
         self.model = model
         self.device = model.device
+        self.recurrent = bool(getattr(model, "recurrent_state", False))
+        if self.recurrent and kv_dtype not in (None, "auto", "bf16", "bfloat16"):
+            raise ValueError(f"kv cache dtype {kv_dtype!r} is not served for this model")
         if kv_dtype in ("fp8", "fp8_e4m3", "e4m3"):
             model.kv_dtype = "fp8"       # E4M3 pages, one FP32 scale per page and plane
         elif kv_dtype not in (None, "auto", "bf16", "bfloat16"):
@@ -131,16 +134,23 @@ class LLMEngine:
         self._quota_items = {
             "weights": _weights_on(model, self.device),
             "graph_pool": GRAPH_POOL_BYTES if (self.device.type == "cuda" and use_graphs) else 0,
-            "cache_segment": int(num_pages) * int(model.kv_bytes_per_page(page_size))}
+            "cache_segment": int(num_pages) * int(model.kv_bytes_per_page(page_size)) +
+            self._state_bytes(max_num_seqs)}
         self.quota.state_fraction(self.quota_holder, min(1.0, max(1e-6, mem_fraction_static)))
         weakref.finalize(self, self.quota.release, self.quota_holder)
         self._reserve_quota(("weights", "graph_pool", "cache_segment"))
+        if self.recurrent:
+            # a prompt's pages do not hold its recurrent state: prefixes are not shared, and
+            # copies of pages alone (host tier) cannot bring a request back
+            enable_prefix_cache, host_kv_pages, host_kv_ratio = False, 0, 0.0
         self.blocks = BlockManager(num_pages, page_size, weights_identity, enable_prefix_cache)
+        self.blocks.prefix_cache_allowed = not self.recurrent
         self.config = SchedulerConfig(max_num_seqs=max_num_seqs,
                                       max_num_batched_tokens=max_num_batched_tokens,
                                       chunked_prefill_size=max_num_batched_tokens,
                                       max_model_len=max_model_len, page_size=page_size,
-                                      eos_token_id=model.cfg.eos_token_id)
+                                      eos_token_id=model.cfg.eos_token_id,
+                                      mixed_batches=bool(getattr(model, "mixed_batches", False)))
         self.scheduler = Scheduler(self.blocks, self.config, policy)
         self.runner = CausalLmRunner(model, num_pages, page_size, max_num_seqs, max_model_len,
                                      use_graphs)
@@ -202,16 +212,21 @@ class LLMEngine:
         Returns the bytes released."""
         return self.quota.release(self.quota_holder)
 
+    def _state_bytes(self, max_num_seqs: int) -> int:
+        """Bytes of the recurrent layers' state pools (one slot per running request)."""
+        return max_num_seqs * int(self.model.state_bytes_per_slot()) if self.recurrent else 0
+
     def _divide_memory(self, fraction, page_size, max_num_seqs, max_model_len) -> int:
         """Quota division: what is left of ``fraction`` of the device after the
         weights goes to KV pages (crates/engine/src/memory/division.rs, reference)."""
-        per_page = self.model.kv_bytes_per_page(page_size)
+        per_page = max(1, self.model.kv_bytes_per_page(page_size))
         want = max_num_seqs * ((max_model_len + page_size - 1) // page_size) + 1
         if self.device.type != "cuda":
             return min(want, 4096)
         free, total = torch.cuda.mem_get_info(self.device)
         used_by_us = total - free
         budget = int(total * fraction) - used_by_us - GRAPH_POOL_BYTES   # graphs + workspaces
+        budget -= self._state_bytes(max_num_seqs)
         pages = max(64, budget // per_page)
         return int(min(pages, want))
 
@@ -262,6 +277,9 @@ class LLMEngine:
                 if t is not None:
                     freed += t.numel() * t.element_size()
         self.runner.kv_caches = None
+        for t in (t for pool in (self.runner.states or []) for t in pool if t is not None):
+            freed += t.numel() * t.element_size()
+        self.runner.states = None
         self._parked = []
         if level >= 2:
             hosts = {}                          # one host copy per tensor (tied weights alias)
@@ -299,6 +317,8 @@ class LLMEngine:
             _set_tensor(holder, name, back[key])
         self._parked, self._parked_hosts = [], {}
         self.runner.kv_caches = self.model.new_kv_caches(self.blocks.num_pages, self.config.page_size)
+        if self.recurrent:
+            self.runner.states = self.model.new_state_pools(self.config.max_num_seqs)
         if self.device.type == "cuda":
             torch.cuda.synchronize(self.device)
         level, self.asleep = self.asleep, 0
@@ -419,6 +439,43 @@ class LLMEngine:
                 errors[rid] = f"{ErrorClass.NUMERICAL_FAULT.value}: sampled token {tok}"
         return self.scheduler.update(batch, sampled, lps, errors)
 
+    def forced_step(self, entries: list, end=()) -> Optional[torch.Tensor]:
+        """One step over given tokens (a replayed trace) instead of sampled ones: ``entries``
+        are (request id, tokens, want) triples run as one batch - new ids are admitted, known
+        ones continue - and the logits at the places ``want`` of each entry's tokens come back
+        in order (None when nothing is wanted).  ``end``: ids released after the step."""
+        if self.failed:
+            raise RuntimeError(f"engine stopped: {self.failed}")
+        sch, V = self.scheduler, self.model.cfg.vocab_size
+        pairs, want = [], []
+        for rid, tokens, places in entries:
+            if not tokens or any((t < 0 or t >= V) for t in tokens):
+                raise ValueError(f"input_error: {rid}: no tokens, or an id outside the vocabulary")
+            if any((w < 0 or w >= len(tokens)) for w in places):
+                raise ValueError(f"input_error: {rid}: a wanted place outside its tokens")
+            req = sch.requests.get(rid)
+            if req is None:
+                req = Request(rid, [], SamplingParams(temperature=0.0))
+            if req.num_tokens + len(tokens) > self.config.max_model_len:
+                raise ValueError(f"input_error: {rid}: longer than {self.config.max_model_len}")
+            pairs.append((req, tokens))
+            want.append(list(places))
+        logits = None
+        if pairs:
+            batch = sch.force(pairs)
+            self.watchdog.begin(f"forced {batch.kind} step {batch.step_id}")
+            try:
+                logits = self.runner.batch_logits(batch, want)
+            except Exception as e:
+                self.failed = f"{ErrorClass.FATAL_WORKER_FAILURE.value}: {e}"
+                raise
+            finally:
+                self.watchdog.end()
+            sch.update(batch, {})
+        for rid in end:
+            sch.release(rid)
+        return logits
+
     def decode_burst(self, steps: int) -> list:
         """Multi-step decode: when every running request is decoding, ensures
         pages for ``steps`` more tokens, replays the decode graph ``steps`` times
@@ -457,6 +514,8 @@ class LLMEngine:
         agreed prefix plus one token; otherwise an ordinary step runs."""
         from .scheduler import Batch, Chunk
         from .speculation import accept
+        if self.recurrent:          # a refused draft cannot be taken back out of the state
+            return self.step()
         sch = self.scheduler
         stateful = getattr(drafter, "needs_hidden", False)
         if stateful and getattr(self.runner, "hidden_tap", None) is None and hasattr(drafter, "tap"):

@@ -219,6 +219,8 @@ def export_request(engine, request_id: str, release: bool = True) -> Handoff:
     """Lends ``request_id`` (running, at least its prompt computed).  With ``release``
     the request ends here (its pages go back to the pool, committed prefix pages stay
     in the prefix cache)."""
+    if getattr(engine, "recurrent", False):
+        raise ValueError("input_error: a request with recurrent state is not handed between engines")
     sch, runner = engine.scheduler, engine.runner
     req = sch.requests[request_id]
     assert not req.finished and req.num_computed >= len(req.prompt_ids), \
@@ -340,6 +342,8 @@ def import_request(engine, handoffs) -> str:
     of every exporting rank's (head ranges are re-cut for this rank)."""
     hs = handoffs if isinstance(handoffs, (list, tuple)) else [handoffs]
     h = hs[0]
+    if getattr(engine, "recurrent", False):
+        raise ValueError("input_error: a request with recurrent state is not handed between engines")
     sch, runner, model = engine.scheduler, engine.runner, engine.model
     for x in hs:
         x.validate_for(engine)

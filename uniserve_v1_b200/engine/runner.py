@@ -110,6 +110,11 @@ class CausalLmRunner:
         self.max_model_len = max_model_len
         self.max_pages = (max_model_len + page_size - 1) // page_size
         self.kv_caches = model.new_kv_caches(num_pages, page_size)
+        # recurrent layers: one slot per running request (the scheduler's slot), in fixed pools
+        self.recurrent = bool(getattr(model, "recurrent_state", False))
+        self.attends_pages = bool(getattr(model, "attends_pages", False))
+        self.states = model.new_state_pools(max_num_seqs) if self.recurrent else None
+        self._row_cu: dict = {}
         self.use_graphs = use_graphs and self.device.type == "cuda"
         self.buckets = [b for b in DECODE_BUCKETS if b < max_num_seqs] + [max_num_seqs]
         self.history_steps = history_steps
@@ -141,7 +146,7 @@ class CausalLmRunner:
             blk = InputBlock([
                 ("input_ids", i32, (B,)), ("positions", i32, (B,)), ("slots", i32, (B,)),
                 ("seq_lens", i32, (B,)), ("live", i32, (1,)), ("step", i32, (1,)),
-                ("page_table", i32, (B, self.max_pages)),
+                ("page_table", i32, (B, self.max_pages)), ("state_slots", i32, (B,)),
                 ("temperature", f32, (B,)), ("top_p", f32, (B,)), ("min_p", f32, (B,)),
                 ("top_k", i32, (B,)), ("seeds", i64, (B,)), ("sample_pos", i64, (B,)),
             ], self.device)
@@ -163,13 +168,18 @@ class CausalLmRunner:
         """The one forward function: eager, rehearsal and capture all run this."""
         d = blk.d
         max_len = self.max_model_len
-        splits = F.decode_splits(B, self.model.Hkv, max_len) if self.device.type == "cuda" else 1
-        if self._persist_attention(B):
-            splits = F.PERSIST_SPLITS
-        scratch, counters = self._attn_scratch(B, splits)
-        meta = AttnMeta(kind="decode", slots=d["slots"], page_table=d["page_table"],
-                        seq_lens=d["seq_lens"], splits=splits, live=d["live"], scratch=scratch,
-                        counters=counters)
+        if self.attends_pages:             # the model brings its own attention over pages
+            meta = AttnMeta(kind="decode", slots=d["slots"], page_table=d["page_table"],
+                            seq_lens=d["seq_lens"], live=d["live"], cu_q=self._arange(B),
+                            state_slots=d["state_slots"], states=self.states, max_k=max_len)
+        else:
+            splits = F.decode_splits(B, self.model.Hkv, max_len) if self.device.type == "cuda" else 1
+            if self._persist_attention(B):
+                splits = F.PERSIST_SPLITS
+            scratch, counters = self._attn_scratch(B, splits)
+            meta = AttnMeta(kind="decode", slots=d["slots"], page_table=d["page_table"],
+                            seq_lens=d["seq_lens"], splits=splits, live=d["live"], scratch=scratch,
+                            counters=counters)
         hidden = self.model.forward(d["input_ids"], d["positions"], meta, self.kv_caches)
         logits = None
         if variant == "greedy" and hasattr(self.model, "greedy_tokens"):
@@ -196,6 +206,13 @@ class CausalLmRunner:
                           step=d["step"])
         d["sample_pos"].add_(1)
         return logits, sampled
+
+    def _arange(self, B: int) -> torch.Tensor:
+        """0 .. B (int32, on the device): the row offsets of one-token sequences."""
+        t = self._row_cu.get(B)
+        if t is None:
+            t = self._row_cu[B] = torch.arange(B + 1, dtype=torch.int32, device=self.device)
+        return t
 
     def _persist_attention(self, B: int) -> bool:
         """Whether this runner's decode steps use the persistent attention kernel."""
@@ -274,6 +291,8 @@ class CausalLmRunner:
         # Inert inputs: no row is live, no cache slot is written.
         blk.dev.zero_()
         blk.d["slots"].fill_(-1)
+        blk.d["state_slots"].fill_(-1)
+        self._arange(B)
         torch.cuda.synchronize()
         self.announce(self._decode_kind("eager", B), B)
         with torch.cuda.stream(s):
@@ -344,6 +363,7 @@ class CausalLmRunner:
         h["seq_lens"][:n] = pos
         h["seq_lens"][:n] += 1
         h["slots"][:n] = slots
+        h["state_slots"][:n] = [req.slot for req in rows]
         h["temperature"][:n] = temp
         h["top_k"][:n] = top_k
         h["top_p"][:n] = top_p
@@ -356,6 +376,7 @@ class CausalLmRunner:
             h["positions"][n:] = 0
             h["seq_lens"][n:] = 0
             h["slots"][n:] = -1
+            h["state_slots"][n:] = -1
             h["temperature"][n:] = 1.0
             h["top_k"][n:] = 1
             h["top_p"][n:] = 1.0
@@ -630,8 +651,60 @@ class CausalLmRunner:
         chunks that sample, in chunk order, on the host; logprob info).  ``capacity`` pads
         the rows to an agreed count (padding rows write no cache slot and route nowhere)."""
         dev = self.device
+        hidden, cu_q = self._prefill_rows(chunks, capacity)
+        last_rows = [cu_q[i + 1] - 1 for i, c in enumerate(chunks) if c.sample]
+        sample_rows = [c.request for c in chunks if c.sample]
+        if not sample_rows:
+            return None, None, []
+        rows_idx = torch.tensor(last_rows, dtype=torch.int32, device=dev)
+        last = F.gather_rows(hidden, rows_idx)
+        logits = self.model.logits(last)
+        if self.variant_for(sample_rows) == "greedy":
+            toks = F.argmax(logits)
+            host = self._to_host(toks) if dev.type == "cuda" else toks
+            return host, None, sample_rows
+        host, info = self._shape_and_sample(logits, sample_rows)
+        return host, info, sample_rows
+
+    def batch_logits(self, batch: Batch, want: list) -> Optional[torch.Tensor]:
+        """Runs a batch and returns the logits (FP32, on the host) at the places ``want[i]``
+        among chunk i's tokens, in order; None when nothing is wanted.  A batch of one token
+        per request replays the decode graph, any other runs the prefill path."""
+        dev = self.device
+        if batch.kind == "decode":
+            rows = [c.request for c in batch.chunks]
+            B = self.bucket_for(len(rows))
+            blk = self._decode_block(B)
+            self._fill_decode(blk, rows, B)
+            g = self._graph(B, "logits")
+            self.h2d_bytes += blk.upload()
+            if g is not None:
+                g.graph.replay()
+                N.launch_count += g.launches
+                logits = g.logits
+            else:
+                logits, _ = self._decode_body(blk, B, "logits")
+            idx = [i for i, w in enumerate(want) for _ in w]
+            logits = logits[torch.tensor(idx, dtype=torch.long, device=dev)] if idx else None
+        else:
+            hidden, cu_q = self._prefill_rows(batch.chunks)
+            idx = [cu_q[i] + j for i, w in enumerate(want) for j in w]
+            logits = self.model.logits(F.gather_rows(
+                hidden, torch.tensor(idx, dtype=torch.int32, device=dev))) if idx else None
+        if dev.type != "cuda":
+            return logits
+        if logits is None:
+            self._queue_status_copy()
+            self._wait(torch.cuda.current_stream().synchronize, "to_host")
+            self.check_device_status()
+            return None
+        return self._to_host(logits)
+
+    def _prefill_rows(self, chunks: list, capacity: Optional[int] = None):
+        """The forward of ``prefill``: (hidden rows, row offset of every chunk)."""
+        dev = self.device
         ps = self.page_size
-        ids, pos, slots, cu_q, cu_k, ctx, last_rows, sample_rows = [], [], [], [0], [0], [], [], []
+        ids, pos, slots, cu_q, cu_k, ctx = [], [], [], [0], [0], []
         max_q = max_k = 0
         for c in chunks:
             req = c.request
@@ -645,9 +718,6 @@ class CausalLmRunner:
             ctx.append(c.start)
             max_q = max(max_q, c.length)
             max_k = max(max_k, c.start + c.length)
-            if c.sample:
-                last_rows.append(cu_q[-1] - 1)
-                sample_rows.append(req)
         T_real = len(ids)
         live = None
         if capacity is not None:
@@ -657,21 +727,22 @@ class CausalLmRunner:
             live = torch.tensor([T_real], dtype=torch.int32, device=dev)
         T = len(ids)
         i32 = torch.int32
-        packed = torch.tensor(ids + pos + slots + cu_q + cu_k, dtype=i32,
-                              pin_memory=dev.type == "cuda")
+        packed = torch.tensor(ids + pos + slots + cu_q + cu_k + [c.request.slot for c in chunks],
+                              dtype=i32, pin_memory=dev.type == "cuda")
         d = packed.to(dev, non_blocking=True)
         self.h2d_bytes += packed.numel() * 4
         nq = len(cu_q)
         page_table = None
-        if any(c > 0 for c in ctx):
+        if self.attends_pages or any(c > 0 for c in ctx):
             page_table = torch.zeros(len(chunks), self.max_pages, dtype=i32)
             for i, c in enumerate(chunks):
                 page_table[i, :len(c.request.pages)] = torch.tensor(c.request.pages, dtype=i32)
             page_table = page_table.to(dev)
         meta = AttnMeta(kind="prefill", slots=d[2 * T:3 * T], cu_q=d[3 * T:3 * T + nq],
                         cu_k=d[3 * T + nq:3 * T + 2 * nq], max_q=max_q, max_k=max_k,
-                        context_lens=ctx, page_table=page_table, live=live, rows_real=T_real)
-        if page_table is not None and dev.type == "cuda":
+                        context_lens=ctx, page_table=page_table, live=live, rows_real=T_real,
+                        state_slots=d[3 * T + 2 * nq:], states=self.states)
+        if page_table is not None and dev.type == "cuda" and not self.attends_pages:
             from ..ops.attention import context_tables
             meta.ctx_tables = context_tables(ctx, cu_q, cu_k, dev)
             self.h2d_bytes += 4 * len(cu_q) + 8 * T_real
@@ -681,17 +752,7 @@ class CausalLmRunner:
         if tap is not None:          # a drafter that feeds on the target's states (MTP head)
             for i, c in enumerate(chunks):
                 tap(c.request, c.start, hidden[cu_q[i]:cu_q[i + 1]])
-        if not sample_rows:
-            return None, None, []
-        rows_idx = torch.tensor(last_rows, dtype=i32, device=dev)
-        last = F.gather_rows(hidden, rows_idx)
-        logits = self.model.logits(last)
-        if self.variant_for(sample_rows) == "greedy":
-            toks = F.argmax(logits)
-            host = self._to_host(toks) if dev.type == "cuda" else toks
-            return host, None, sample_rows
-        host, info = self._shape_and_sample(logits, sample_rows)
-        return host, info, sample_rows
+        return hidden, cu_q
 
     # ----------------------------------------------------------------- verify --
     def verify(self, rows: list, drafts: list, want_hidden: bool = False):

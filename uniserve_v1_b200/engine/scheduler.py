@@ -34,6 +34,7 @@ class SchedulerConfig:
     page_size: int = 16
     eos_token_id: Optional[int] = None
     decode_lookahead: int = 1               # pages are ensured this many tokens ahead
+    mixed_batches: bool = False             # decoded tokens ride along with prompt portions
 
 
 class Policy:
@@ -220,8 +221,10 @@ class Scheduler:
             chunks.append(Chunk(req, req.num_computed, take,
                                 req.num_computed + take == req.num_tokens))
             budget -= take
+        if chunks and cfg.mixed_batches:
+            chunks += self._riding_decodes({id(c.request) for c in chunks})
         if chunks:
-            self.stats["prefill_tokens"] += sum(c.length for c in chunks)
+            self.stats["prefill_tokens"] += sum(c.length for c in chunks if not self._decodes(c))
             b = Batch("prefill", chunks, self.step_id)
             b.validate(cfg.page_size)
             return b
@@ -259,6 +262,58 @@ class Scheduler:
         b = Batch("decode", chunks, self.step_id)
         b.validate(cfg.page_size)
         return b
+
+    @staticmethod
+    def _decodes(c: Chunk) -> bool:
+        return c.length == 1 and bool(c.request.output_ids) and c.start == c.request.num_tokens - 1
+
+    def _riding_decodes(self, taken: set) -> list:
+        """One-token chunks of the decoding requests that join a batch of prompt portions, as
+        far as free pages go (nobody is preempted for them: they decode again next step)."""
+        out = []
+        for r in self.running:
+            if id(r) in taken or not r.output_ids or r.num_computed != r.num_tokens - 1:
+                continue
+            pages = self.blocks.allocate(self._pages_needed(r, r.num_tokens))
+            if pages is None:
+                continue
+            r.pages.extend(pages)
+            out.append(Chunk(r, r.num_tokens - 1, 1, True))
+        self.stats["decode_tokens"] += len(out)
+        return out
+
+    # -------------------------------------------------------- forced batches --
+    def force(self, entries: list) -> Batch:
+        """A batch that runs given tokens instead of scheduled ones: ``entries`` are (request,
+        tokens) pairs, the tokens following what the request has computed.  New requests are
+        admitted, pages come from the pool as for any batch; nothing is sampled."""
+        chunks = []
+        for req, tokens in entries:
+            if req.state != RequestState.RUNNING:
+                self.requests[req.request_id] = req
+                if not self._admit(req):
+                    raise RuntimeError(f"{req.request_id}: no free slot "
+                                       f"({self.config.max_num_seqs} requests are live)")
+                self.running.append(req)
+            assert req.num_computed == req.num_tokens, "earlier tokens have not run"
+            req.prompt_ids.extend(int(t) for t in tokens)
+            pages = self.blocks.allocate(self._pages_needed(req, req.num_tokens))
+            if pages is None:
+                raise RuntimeError(f"{req.request_id}: the cache pool has no page left")
+            req.pages.extend(pages)
+            chunks.append(Chunk(req, req.num_computed, len(tokens), False))
+        self.step_id += 1
+        batch = Batch("decode" if all(c.length == 1 for c in chunks) else "prefill", chunks,
+                      self.step_id)
+        batch.validate(self.config.page_size)
+        return batch
+
+    def release(self, request_id: str) -> None:
+        """Ends a request of forced batches and drops its record."""
+        req = self.requests[request_id]
+        if not req.finished:
+            self._finish(req, FinishReason.STOP)
+        del self.requests[request_id]
 
     # --------------------------------------------------------------- update --
     def _commit_pages(self, req: Request) -> None:

@@ -153,6 +153,8 @@ class AttnMeta:
     rows_real: Optional[int] = None             # prefill padded to a capacity: rows before the padding
     ctx_tables: Optional[tuple] = None          # ops.attention.context_tables(...) when sequences
                                                 # have cached context (GPU: no host sync in prefill)
+    state_slots: Optional[torch.Tensor] = None  # [B] int32 state-pool slot per sequence, -1 padding
+    states: Optional[list] = None               # state pools of a model with recurrent layers
 
 
 class Qwen3MoeModel:

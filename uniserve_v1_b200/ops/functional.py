@@ -302,12 +302,27 @@ def _block_n(rows: int, dual: bool) -> int:
     return 128 if dual else 256
 
 
-def linear(x, w, bias=None, out_dtype=None, out=None, block_n=None):
-    """y[rows, M] = x[rows, K] @ w[M, K]^T (+ bias).  bf16 operands, FP32
-    accumulation in tensor memory, output bf16 or fp32."""
+_ACT1 = {None: 0, "gelu_erf": 3}       # activations of a single (ungated) product
+
+
+def linear(x, w, bias=None, out_dtype=None, out=None, block_n=None, act=None):
+    """y[rows, M] = act(x[rows, K] @ w[M, K]^T (+ bias)).  bf16 operands, FP32
+    accumulation in tensor memory, output bf16 or fp32; FP32 operands run in true 32-bit.
+    ``act``: None or "gelu_erf"."""
     out_dtype = out_dtype or x.dtype
     if not _cuda(x):
-        return R.linear(x, w, bias, out_dtype)
+        y = R.linear(x, w, bias, torch.float32 if act else out_dtype)
+        return R.gelu_erf(y).to(out_dtype) if act else y
+    acode = _ACT1[act]
+    if x.dtype == torch.float32:
+        assert w.dtype == torch.float32 and w.stride(1) == 1 and out_dtype == torch.float32
+        x2 = x.reshape(-1, x.shape[-1])
+        if out is None:
+            out = torch.empty(x2.shape[0], w.shape[0], dtype=torch.float32, device=x.device)
+        N.call("us_gemm_f32", N.ptr(w), N.ptr(x2), N.ptr(out), 1, w.shape[0], w.shape[0],
+               x2.shape[1], x2.shape[0], w.stride(0), x2.stride(0), out.stride(0), acode,
+               N.ptr(bias), None, None, None, None, 0, N.stream())
+        return out.view(*x.shape[:-1], w.shape[0])
     assert x.dtype == BF16 and w.dtype == BF16
     x2 = x.reshape(-1, x.shape[-1])
     if x2.stride(-1) != 1 or x2.stride(0) % 8:
@@ -331,11 +346,11 @@ def linear(x, w, bias=None, out_dtype=None, out=None, block_n=None):
         # decode-size projection: weight-streaming kernel (latency-bound shape)
         N.call("us_linear_decode", N.ptr(w), N.ptr(x2), N.ptr(out), N.ptr(bias), rows, M, K,
                w.stride(0), x2.stride(0), out.stride(0), int(out.dtype == torch.float32),
-               0 if (bias is None or bias.dtype == BF16) else 1, N.stream())
+               0 if (bias is None or bias.dtype == BF16) else 1, acode, N.stream())
         return out.view(*x.shape[:-1], M)
     bn = block_n or _block_n(rows, False)
     N.call("us_gemm_wx", N.ptr(w), N.ptr(x2), N.ptr(out), 1, M, M, K, rows, w.stride(0),
-           x2.stride(0), out.stride(0), 0, 0, 0, 0 if out.dtype == BF16 else 1, N.ptr(bias),
+           x2.stride(0), out.stride(0), 0, 0, acode, 0 if out.dtype == BF16 else 1, N.ptr(bias),
            0 if (bias is None or bias.dtype == BF16) else 1, None, None, None, None, None, None,
            0, bn, N.stream())
     return out.view(*x.shape[:-1], M)
@@ -527,6 +542,157 @@ def moe_experts(x, ids, weights, w13, w2, e_lo=0, act="silu", stepwise=False, ws
     return out
 
 
+@dataclass
+class TableRoutes:
+    """Routes of one layer chosen by token id: the sorted route list and the expert tile list."""
+    ids: torch.Tensor             # [T, top] expert of every route
+    sorted_route: torch.Tensor
+    perm: torch.Tensor            # [T, top] permuted row of every route
+    expert_offsets: torch.Tensor
+    tile_group: torch.Tensor
+    tile_row0: torch.Tensor
+    tile_rows: torch.Tensor
+    num_tiles: torch.Tensor
+    block_n: int
+    max_tiles: int
+    live_tiles: int
+
+
+def table_routes(tokens, tables, E):
+    """``tables`` [layers, vocab, top] (int32): the experts of every token id, layer by layer.
+    Routes and their sort of all layers in one launch (they depend on the token ids only);
+    returns a ``TableRoutes`` per layer."""
+    Ln, V, top = tables.shape
+    T = tokens.shape[0]
+    if not _cuda(tokens):
+        return [R.table_routes(tokens, tables[i]) for i in range(Ln)]
+    R_ = T * top
+    avg = max(1, R_ // E)
+    block_n = 16 if avg <= 16 else 32 if avg <= 32 else 64 if avg <= 64 else 128
+    if avg >= MOE_PAIR_MIN_ROWS:
+        block_n = 256
+    max_tiles = min(R_, E) + R_ // block_n + 1
+    widths = (R_, R_, R_, E + 1, max_tiles, max_tiles, max_tiles, 1)
+    buf = torch.empty(Ln * sum(widths), dtype=torch.int32, device=tokens.device)
+    parts, off = [], 0
+    for w in widths:
+        parts.append(buf[off:off + Ln * w].view(Ln, w))
+        off += Ln * w
+    N.call("us_table_route_sort", N.ptr(tokens), N.ptr(tables), Ln, T, top, V, E, block_n, max_tiles,
+           *[N.ptr(p) for p in parts], N.stream())
+    live = MoeWorkspace._expected_tiles(R_, E, E, block_n)
+    return [TableRoutes(parts[0][i].view(T, top), parts[1][i], parts[2][i].view(T, top), parts[3][i],
+                        parts[4][i], parts[5][i], parts[6][i], parts[7][i], block_n, max_tiles, live)
+            for i in range(Ln)]
+
+
+def routed_mlp(x, routes, w_up, w_down, act="gelu_erf"):
+    """Ungated experts W_down act(W_up x) over sorted routes: gather, two grouped products with
+    the activation in the first one's epilogue.  w_up [E, I, H], w_down [E, H, I].  Returns the
+    expert rows in permuted order; ``routes.perm`` says where a token's are."""
+    if not _cuda(x):
+        return R.routed_mlp(x, routes, w_up, w_down)
+    T, H = x.shape
+    E, I_, _ = w_up.shape
+    top = routes.perm.shape[1]
+    R_ = T * top
+    dev, st, code = x.device, N.stream(), _ACT1[act]
+    xp = torch.empty(R_, H, dtype=x.dtype, device=dev)
+    h = torch.empty(R_, I_, dtype=x.dtype, device=dev)
+    y = torch.empty(R_, H, dtype=x.dtype, device=dev)
+    wide = 1 if x.dtype == BF16 else 2          # the gather moves 16-bit units
+    N.call("us_moe_gather", N.ptr(x), N.ptr(routes.sorted_route), N.ptr(routes.expert_offsets[E:]),
+           R_, top, H * wide, N.ptr(xp), st)
+    tiles = (N.ptr(routes.tile_group), N.ptr(routes.tile_row0), N.ptr(routes.tile_rows),
+             N.ptr(routes.num_tiles), routes.max_tiles)
+    for w, a, o, M, K, c in ((w_up, xp, h, I_, H, code), (w_down, h, y, H, I_, 0)):
+        if x.dtype == torch.float32:
+            N.call("us_gemm_f32", N.ptr(w), N.ptr(a), N.ptr(o), E, M, M, K, R_, K, K, M, c, None,
+                   *tiles, st)
+            continue
+        if routes.live_tiles:
+            N.kernels().us_gemm_wx_hint(routes.live_tiles * ((M + 127) // 128))
+        N.call("us_gemm_wx", N.ptr(w), N.ptr(a), N.ptr(o), E, M, M, K, R_, K, K, M, 0, 0, c, 0, None,
+               0, None, None, *tiles, routes.block_n, st)
+    return y
+
+
+# ------------------------------------------------- output-normed residual --
+def embed_rows(ids, table):
+    """(FP32 residual rows, the same rows in the table's type)."""
+    if not _cuda(table):
+        x = table[ids.long()]
+        return x.float(), x
+    T, W = ids.shape[0], table.shape[1]
+    res = torch.empty(T, W, dtype=torch.float32, device=table.device)
+    x = torch.empty(T, W, dtype=table.dtype, device=table.device)
+    N.call("us_embed_rows", N.ptr(ids), N.ptr(table), N.ptr(res), N.ptr(x), T, W, table.shape[0],
+           int(table.dtype == BF16), N.stream())
+    return res, x
+
+
+def output_norm_add_(y, residual, gain, eps, width, routed=None, shared=None, shared_gate=None,
+                     final_gain=None, dtype=None):
+    """The sublayer output (``y``, or ``routed = (expert rows, perm, weight)`` summed per token,
+    plus ``shared`` rows times sigmoid(residual . shared_gate)) divided by its root mean square,
+    times ``gain``, added to the FP32 ``residual`` in place.  Returns the new residual in the
+    model's type or, with ``final_gain``, its norm (the model's last one)."""
+    src = y if y is not None else routed[0]
+    if not _cuda(residual):
+        return R.output_norm_add_(y, residual, gain, eps, width, routed, shared, shared_gate,
+                                  final_gain).to(src.dtype)
+    T, W = residual.shape
+    x = torch.empty(T, W, dtype=src.dtype, device=residual.device)
+    yp, perm, rw = routed if routed is not None else (None, None, 0.0)
+    N.call("us_output_norm_add", N.ptr(y), N.ptr(yp), N.ptr(perm), rw,
+           perm.shape[1] if perm is not None else 0, N.ptr(shared), N.ptr(shared_gate),
+           N.ptr(residual), N.ptr(x), gain, final_gain or 0.0, int(final_gain is not None), T, W,
+           width, eps, int(src.dtype == BF16), N.stream())
+    return x
+
+
+def row_norm_kv_(x, offs, dims, wq, wk, slots, kcache, vcache, eps):
+    """``x`` [T, ld] holds q, k, v at columns ``offs``, ``dims`` wide.  q (in place) and k are
+    normalised over their whole row (all heads together) with weights wq, wk; k and v go to the
+    cache rows ``slots``.  A k width of 0: the layer has no keys of its own."""
+    nq, nk, nv = dims
+    if not _cuda(x):
+        return R.row_norm_kv_(x, offs, dims, wq, wk, slots, kcache, vcache, eps)
+    N.call("us_row_norm_kv", N.ptr(x), x.stride(0), *offs, nq, nk, nv, N.ptr(wq), N.ptr(wk),
+           N.ptr(slots), N.ptr(kcache), N.ptr(vcache), x.shape[0], eps, int(x.dtype == BF16),
+           N.stream())
+
+
+def tanh_cols_(x, off, n):
+    if not _cuda(x):
+        x[:, off:off + n] = torch.tanh(x[:, off:off + n].float()).to(x.dtype)
+        return
+    N.call("us_tanh_cols", N.ptr(x), x.stride(0), off, n, x.shape[0], int(x.dtype == BF16),
+           N.stream())
+
+
+def head_mix_attention(q, H, kcache, vcache, talk, cu, positions, page_table, scale, size=0,
+                       keep=0, seq_lens=None, ldo=None):
+    """Causal attention whose heads' softmax weights are mixed by ``talk`` [H, H] (FP32) before
+    the values: q [T, H * D] (row-strided view), pages [n, page, G, D] and [n, page, G, V], rows
+    of sequence s at cu[s] .. cu[s + 1], keys up to a row's own position read through
+    ``page_table``.  ``size`` / ``keep``: sliding window and always-visible first keys (0: off).
+    Returns [T, ldo] rows (columns past H * V zero)."""
+    T = q.shape[0]
+    _, page, G, D = kcache.shape
+    V = vcache.shape[3]
+    ldo = ldo or H * V
+    if not _cuda(q):
+        return R.head_mix_attention(q, H, kcache, vcache, talk, cu, positions, page_table, scale,
+                                    size, keep, ldo)
+    out = torch.empty(T, ldo, dtype=q.dtype, device=q.device)
+    N.call("us_head_mix_attention", N.ptr(q), N.ptr(kcache), N.ptr(vcache), N.ptr(talk), N.ptr(out),
+           N.ptr(cu), N.ptr(positions), N.ptr(page_table), N.ptr(seq_lens), q.stride(0), ldo, T,
+           cu.shape[0] - 1, H, G, D, V, page, page_table.shape[1], size, keep, scale,
+           int(q.dtype == BF16), N.stream())
+    return out
+
+
 # --------------------------------------------------------------- sampling --
 def argmax(logits, out=None):
     if not _cuda(logits):
@@ -596,7 +762,9 @@ def gather_rows(src, idx, out=None):
     H = src.shape[1]
     if out is None:
         out = torch.empty(M, H, dtype=src.dtype, device=src.device)
-    N.call("us_gather_rows", N.ptr(src), N.ptr(idx), M, H, src.stride(0), N.ptr(out), N.stream())
+    wide = src.element_size() // 2              # rows move as 16-bit units
+    N.call("us_gather_rows", N.ptr(src), N.ptr(idx), M, H * wide, src.stride(0) * wide, N.ptr(out),
+           N.stream())
     return out
 
 

@@ -39,7 +39,21 @@ _SIGNATURES = {
     "us_device_info": (I, [P, P, P, P]),
     "us_gemm_wx": (I, [P, P, P, I, I, I, I, I, L, L, L, I, I, I, I, P, I, P, P, P, P, P, P, I, I, P]),
     "us_gemm_wx_hint": (I, [I]),
-    "us_linear_decode": (I, [P, P, P, P, I, I, I, L, L, L, I, I, P]),
+    "us_linear_decode": (I, [P, P, P, P, I, I, I, L, L, L, I, I, I, P]),
+    "us_gemm_f32": (I, [P, P, P, I, I, I, I, I, L, L, L, I, P, P, P, P, P, I, P]),
+    "us_channel_delta_prep": (I, [P, L, I, I, I, I, P, P, P, P, L, P, P, P, P, P, P, P, P, P, P, P,
+                                  I, I, I, I, I, I, I, I, I, P]),
+    "us_general_delta_prep": (I, [P, L, I, I, P, L, P, P, P, P, P, I, I, I, F, I, P]),
+    "us_vector_delta_rule": (I, [I, P, P, P, L, L, L, I, I, I, I, I, I, P, P, P, P, P, P, P, P, P,
+                                 I, I, I, I, I, P]),
+    "us_head_norm_gate": (I, [P, P, I, P, L, P, L, I, I, I, F, I, I, P]),
+    "us_embed_rows": (I, [P, P, P, P, I, I, I, I, P]),
+    "us_output_norm_add": (I, [P, P, P, F, I, P, P, P, P, F, F, I, I, I, I, F, I, P]),
+    "us_row_norm_kv": (I, [P, L, I, I, I, I, I, I, P, P, P, P, P, I, F, I, P]),
+    "us_tanh_cols": (I, [P, L, I, I, I, I, P]),
+    "us_head_mix_attention": (I, [P, P, P, P, P, P, P, P, P, L, L, I, I, I, I, I, I, I, I, I, I, F,
+                                  I, P]),
+    "us_table_route_sort": (I, [P, P, I, I, I, I, I, I, I, P, P, P, P, P, P, P, P, P]),
     "us_kv_write_scaled": (I, [P, P, L, L, P, P, P, P, P, I, I, I, I, P]),
     "us_kv_gather": (I, [P, P, P, P, P, I, P, P, I, I, I, I, I, P, P, L, I, P]),
     "us_paged_decode_attention_fp8": (I, [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I,
@@ -86,12 +100,24 @@ class NativeMissing(RuntimeError):
     pass
 
 
+_group = ""       # "-<group>": libraries built for one family alone
+
+
+def use_group(name: str | None) -> None:
+    """Loads the libraries of one family's build group instead of the whole package's (before
+    anything else of the library is used)."""
+    global _group
+    if _kernels is not None or _host is not None:
+        raise RuntimeError("the native libraries are already loaded")
+    _group = f"-{name}" if name else ""
+
+
 def kernels_path() -> Path:
-    return _LIB_DIR / "libus_kernels.so"
+    return _LIB_DIR / f"libus_kernels{_group}.so"
 
 
 def host_path() -> Path:
-    return _LIB_DIR / "libus_host.so"
+    return _LIB_DIR / f"libus_host{_group}.so"
 
 
 def _bind(lib, table, strict=False):

@@ -402,3 +402,84 @@ def persist_merge_slots(seq_lens, Hkv: int, n_cta: int, b: int, hk: int, tile: i
     begin = Hkv * pre[b] + hk * tiles[b]
     last = begin + tiles[b] - 1
     return [(c, 0 if start(c) >= begin else 1) for c in range(cta_of(begin), cta_of(last) + 1)]
+
+
+# ------------------------------------------------- output-normed residual --
+def gelu_erf(x):
+    return torch.nn.functional.gelu(x.float())
+
+
+def table_routes(tokens, table):
+    """Experts of every token [T, top] (the CPU form of a layer's routes)."""
+    return table[tokens.long()].long()
+
+
+def routed_mlp(x, routes, w_up, w_down):
+    """Expert rows in route order (row t * top + k belongs to token t's k-th expert)."""
+    T, top = routes.shape
+    y = torch.zeros(T * top, w_down.shape[1], dtype=x.dtype)
+    flat = routes.reshape(-1)
+    tok = torch.arange(T).repeat_interleave(top)
+    for e in flat.unique().tolist():
+        sel = (flat == e).nonzero(as_tuple=True)[0]
+        h = gelu_erf(linear(x[tok[sel]], w_up[e], None, torch.float32)).to(x.dtype)
+        y[sel] = linear(h, w_down[e], None, x.dtype)
+    return y
+
+
+def output_norm_add_(y, residual, gain, eps, width, routed=None, shared=None, shared_gate=None,
+                     final_gain=None):
+    T = residual.shape[0]
+    if y is None:
+        rows, routes, w = routed
+        y = rows.float().view(T, routes.shape[1], -1).sum(1) * w
+    y = y.float()
+    if shared is not None:
+        g = 1.0 if shared_gate is None else torch.sigmoid(residual @ shared_gate)[:, None]
+        y = y + g * shared.float()
+    residual += y * (gain * torch.rsqrt(y.pow(2).sum(-1, keepdim=True) / width + eps))
+    if final_gain is None:
+        return residual
+    return residual * (final_gain *
+                       torch.rsqrt(residual.pow(2).sum(-1, keepdim=True) / width + eps))
+
+
+def row_norm_kv_(x, offs, dims, wq, wk, slots, kcache, vcache, eps):
+    (oq, ok, ov), (nq, nk, nv) = offs, dims
+    q = x[:, oq:oq + nq].float()
+    x[:, oq:oq + nq] = (q * torch.rsqrt(q.pow(2).mean(-1, keepdim=True) + eps) * wq).to(x.dtype)
+    if nk == 0:
+        return
+    k = x[:, ok:ok + nk].float()
+    k = (k * torch.rsqrt(k.pow(2).mean(-1, keepdim=True) + eps) * wk).to(x.dtype)
+    sel = slots >= 0
+    at = slots[sel].long()
+    kcache.view(-1, nk)[at] = k[sel]
+    vcache.view(-1, nv)[at] = x[:, ov:ov + nv][sel]
+
+
+def head_mix_attention(q, H, kcache, vcache, talk, cu, positions, page_table, scale, size, keep,
+                       ldo):
+    T = q.shape[0]
+    _, page, G, D = kcache.shape
+    V = vcache.shape[3]
+    out = torch.zeros(T, ldo, dtype=q.dtype)
+    cu = cu.tolist()
+    for s in range(len(cu) - 1):
+        lo, hi = cu[s], cu[s + 1]
+        if hi == lo:
+            continue
+        pos = positions[lo:hi].long()
+        n = int(pos.max()) + 1
+        pg = page_table[s, :(n + page - 1) // page].long()
+        k = kcache[pg].reshape(-1, G, D)[:n].float().repeat_interleave(H // G, 1)
+        v = vcache[pg].reshape(-1, G, V)[:n].float().repeat_interleave(H // G, 1)
+        sc = torch.einsum("thd,nhd->htn", q[lo:hi].reshape(hi - lo, H, D).float(), k) * scale
+        j = torch.arange(n)[None, :]
+        see = j <= pos[:, None]
+        if size > 0:
+            see = see & ((pos[:, None] - j < size) | (j < keep))
+        w = sc.masked_fill(~see[None], float("-inf")).softmax(-1)
+        w = torch.einsum("hg,gtn->htn", talk.float(), w)
+        out[lo:hi, :H * V] = torch.einsum("htn,nhv->thv", w, v).reshape(hi - lo, H * V).to(q.dtype)
+    return out

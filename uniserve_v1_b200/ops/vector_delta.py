@@ -1,0 +1,148 @@
+"""Recurrent mixers whose decay is a vector over the key channels of a head.
+
+    channel rule:  S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;   o = S^T q
+    general rule:  S <- diag(w) S - (a n)(n^T S) + k v^T (both on the old S); o = S^T q
+
+Batches are packed: rows of sequence s are cu[s] .. cu[s + 1], its state lives in slot
+``slots[s]`` of a pool and is updated in place; a sequence whose first row stands at position 0
+starts from zero whatever the slot holds, a negative slot marks padding.  On a GPU the entry
+points run ``csrc/vector_delta.cu``; on the CPU the same recurrences run step by step in FP32.
+"""
+from __future__ import annotations
+
+import math
+from dataclasses import dataclass
+
+import torch
+
+from . import native as N
+
+BF16 = torch.bfloat16
+UNIT_EPS = 1e-6
+GENERAL_DECAY_RATE = math.exp(-0.5)     # the general rule's w = exp(-rate * sigmoid(.))
+
+
+@dataclass
+class SeqMeta:
+    """Where the packed rows belong."""
+    cu: torch.Tensor            # [B + 1] int32
+    slots: torch.Tensor         # [B] int32 state slot of every sequence
+    positions: torch.Tensor     # [T] int32
+    one_token: bool             # every sequence brings exactly one row
+
+
+def _spans(m: SeqMeta):
+    cu, slots = m.cu.tolist(), m.slots.tolist()
+    for s, slot in enumerate(slots):
+        if slot >= 0 and cu[s + 1] > cu[s]:
+            yield cu[s], cu[s + 1], slot, int(m.positions[cu[s]]) == 0
+
+
+def _unit(x):
+    return x * torch.rsqrt((x * x).sum(-1, keepdim=True) + UNIT_EPS)
+
+
+def channel_prep(x, offs, low, w, conv, m: SeqMeta, H, Hk, D, V):
+    """Projection rows ``x`` (q, k, v and the step size at columns ``offs``) and the decay's
+    low-rank rows ``low`` [T, H * D] (FP32) to what the rule reads: unit q (scaled) and k
+    [T, Hk, D], v [T, H, V], decay g [T, H, D], beta [T, H], all FP32.  ``conv`` [slots, K - 1, C]
+    holds the last inputs of the short convolutions and is advanced."""
+    oq, ok, ov, ob = offs
+    T, K, dev = x.shape[0], w["conv_q"].shape[1], x.device
+    if x.is_cuda:
+        f = dict(dtype=torch.float32, device=dev)
+        q, k = torch.empty(T, Hk, D, **f), torch.empty(T, Hk, D, **f)
+        v, g = torch.empty(T, H, V, **f), torch.empty(T, H, D, **f)
+        beta = torch.empty(T, H, **f)
+        N.call("us_channel_delta_prep", N.ptr(x), x.stride(0), oq, ok, ov, ob, N.ptr(w["conv_q"]),
+               N.ptr(w["conv_k"]), N.ptr(w["conv_v"]), N.ptr(low), low.stride(0), N.ptr(w["A_log"]),
+               N.ptr(w["dt_bias"]), N.ptr(conv), N.ptr(q), N.ptr(k), N.ptr(v), N.ptr(g),
+               N.ptr(beta), N.ptr(m.cu), N.ptr(m.slots), N.ptr(m.positions), m.slots.shape[0], T, H,
+               Hk, D, V, K, int(x.dtype == BF16), int(m.one_token), N.stream(),
+               launches=1 if m.one_token or K == 1 else 2)
+        return q, k, v, g, beta
+    nq, nv = Hk * D, H * V
+    taps = torch.cat([w["conv_q"], w["conv_k"], w["conv_v"]], 0)
+    cols = torch.cat([x[:, oq:oq + nq], x[:, ok:ok + nq], x[:, ov:ov + nv]], 1)
+    y = torch.zeros(T, 2 * nq + nv)
+    for lo, hi, slot, fresh in _spans(m):
+        old = torch.zeros(K - 1, cols.shape[1], dtype=x.dtype) if fresh else conv[slot]
+        full = torch.cat([old, cols[lo:hi]], 0)
+        y[lo:hi] = (full.float().unfold(0, K, 1) * taps[None]).sum(-1)
+        if K > 1:
+            conv[slot] = full[-(K - 1):]
+    y = torch.nn.functional.silu(y)
+    q = _unit(y[:, :nq].view(T, Hk, D)) * D ** -0.5
+    k = _unit(y[:, nq:2 * nq].view(T, Hk, D))
+    g = torch.exp(-w["A_log"].exp()[None, :, None] *
+                  torch.nn.functional.softplus(low + w["dt_bias"]).view(T, H, D))
+    return q, k, y[:, 2 * nq:].view(T, H, V), g, torch.sigmoid(x[:, ob:ob + H].float())
+
+
+def general_prep(x, offs, low, w, H, D):
+    """Decay w, unit key n and removal a * n of the general rule, [T, H, D] FP32 each; ``offs``
+    are the columns of k and of the removal rate, ``low`` the decay's low-rank rows (FP32)."""
+    ok, oa = offs
+    T = x.shape[0]
+    if x.is_cuda:
+        out = torch.empty(3, T, H, D, dtype=torch.float32, device=x.device)
+        N.call("us_general_delta_prep", N.ptr(x), x.stride(0), ok, oa, N.ptr(low), low.stride(0),
+               N.ptr(w["w0"]), N.ptr(w["a_bias"]), N.ptr(out[0]), N.ptr(out[1]), N.ptr(out[2]), T, H,
+               D, GENERAL_DECAY_RATE, int(x.dtype == BF16), N.stream())
+        return out[0], out[1], out[2]
+    n = _unit(x[:, ok:ok + H * D].float().view(T, H, D))
+    a = torch.sigmoid(x[:, oa:oa + H * D].float() + w["a_bias"]).view(T, H, D)
+    return torch.exp(-GENERAL_DECAY_RATE * torch.sigmoid(low + w["w0"])).view(T, H, D), n, a * n
+
+
+def vector_delta_rule(q, k, v, g, state, m: SeqMeta, beta=None, n=None, p=None):
+    """The recurrence.  q, k [T, Hk, D] and v [T, H, V] may be strided views (last dimension
+    dense, bf16 or FP32), g / n / p [T, H, D] and beta [T, H] are FP32; ``beta`` selects the
+    channel rule, ``n`` and ``p`` the general one.  ``state`` [slots, H, D, V] FP32 is updated
+    in place.  Returns o [T, H, V] FP32."""
+    T, H, D = g.shape
+    Hk, V = q.shape[1], v.shape[2]
+    general = beta is None
+    if q.is_cuda:
+        assert state.dtype == torch.float32 and state.is_contiguous() and g.is_contiguous()
+        out = torch.empty(T, H, V, dtype=torch.float32, device=q.device)
+        b = [int(t.dtype == BF16) for t in (q, k, v)]
+        N.call("us_vector_delta_rule", int(general), N.ptr(q), N.ptr(k), N.ptr(v), q.stride(0),
+               k.stride(0), v.stride(0), q.stride(1), k.stride(1), v.stride(1), *b, N.ptr(g),
+               N.ptr(n), N.ptr(p), N.ptr(beta), N.ptr(state), N.ptr(out), N.ptr(m.cu),
+               N.ptr(m.slots), N.ptr(m.positions), m.slots.shape[0], H, Hk, D, V, N.stream())
+        return out
+    q, k, v = (t.float() for t in (q, k, v))
+    q, k = (t.repeat_interleave(H // Hk, 1) for t in (q, k))
+    out = torch.zeros(T, H, V)
+    for lo, hi, slot, fresh in _spans(m):
+        S = torch.zeros_like(state[slot]) if fresh else state[slot]
+        for t in range(lo, hi):
+            if general:
+                seen = torch.einsum("hkv,hk->hv", S, n[t])
+                S = g[t][:, :, None] * S - p[t][:, :, None] * seen[:, None] + \
+                    k[t][:, :, None] * v[t][:, None]
+            else:
+                S = g[t][:, :, None] * S
+                u = beta[t][:, None] * (v[t] - torch.einsum("hkv,hk->hv", S, k[t]))
+                S = S + k[t][:, :, None] * u[:, None]
+            out[t] = torch.einsum("hkv,hk->hv", S, q[t])
+        state[slot] = S
+    return out
+
+
+def head_norm_gate(o, w, gate, eps, ldo, dtype):
+    """o [T, H, V] divided by its root mean square per head, times ``w`` ([V] shared by the
+    heads or [H * V]) and sigmoid(gate [T, H * V]); rows ``ldo`` wide (zero past H * V)."""
+    T, H, V = o.shape
+    if o.is_cuda:
+        y = torch.empty(T, ldo, dtype=dtype, device=o.device)
+        N.call("us_head_norm_gate", N.ptr(o), N.ptr(w), 0 if w.numel() == V else V, N.ptr(gate),
+               gate.stride(0), N.ptr(y), ldo, T, H, V, eps, int(dtype == BF16),
+               int(gate.dtype == BF16), N.stream())
+        return y
+    y = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps)
+    y = y * (w if w.numel() == V else w.view(H, V))
+    out = torch.zeros(T, ldo, dtype=dtype)
+    out[:, :H * V] = (y.reshape(T, H * V) * torch.sigmoid(gate.float())).to(dtype)
+    return out
