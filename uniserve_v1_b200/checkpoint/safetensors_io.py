@@ -64,7 +64,7 @@ def save_file(tensors: dict, path, metadata: Optional[dict] = None) -> None:
         header["__metadata__"] = {k: str(v) for k, v in metadata.items()}
     for name, t in tensors.items():
         t = t.detach().cpu().contiguous()
-        raw = t.view(torch.uint8).numpy().tobytes() if t.numel() else b""
+        raw = t.reshape(-1).view(torch.uint8).numpy().tobytes() if t.numel() else b""
         header[name] = {"dtype": _NAMES[t.dtype], "shape": list(t.shape),
                         "data_offsets": [off, off + len(raw)]}
         off += len(raw)

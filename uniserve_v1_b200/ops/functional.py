@@ -622,7 +622,7 @@ def embed_rows(ids, table):
     """(FP32 residual rows, the same rows in the table's type)."""
     if not _cuda(table):
         x = table[ids.long()]
-        return x.float(), x
+        return x.to(torch.float32, copy=True), x
     T, W = ids.shape[0], table.shape[1]
     res = torch.empty(T, W, dtype=torch.float32, device=table.device)
     x = torch.empty(T, W, dtype=table.dtype, device=table.device)
@@ -640,7 +640,7 @@ def output_norm_add_(y, residual, gain, eps, width, routed=None, shared=None, sh
     src = y if y is not None else routed[0]
     if not _cuda(residual):
         return R.output_norm_add_(y, residual, gain, eps, width, routed, shared, shared_gate,
-                                  final_gain).to(src.dtype)
+                                  final_gain).to(src.dtype, copy=True)
     T, W = residual.shape
     x = torch.empty(T, W, dtype=src.dtype, device=residual.device)
     yp, perm, rw = routed if routed is not None else (None, None, 0.0)
@@ -672,7 +672,7 @@ def tanh_cols_(x, off, n):
 
 
 def head_mix_attention(q, H, kcache, vcache, talk, cu, positions, page_table, scale, size=0,
-                       keep=0, seq_lens=None, ldo=None):
+                       keep=0, seq_lens=None, ldo=None, max_q=0, max_k=0):
     """Causal attention whose heads' softmax weights are mixed by ``talk`` [H, H] (FP32) before
     the values: q [T, H * D] (row-strided view), pages [n, page, G, D] and [n, page, G, V], rows
     of sequence s at cu[s] .. cu[s + 1], keys up to a row's own position read through

@@ -66,7 +66,7 @@ def channel_prep(x, offs, low, w, conv, m: SeqMeta, H, Hk, D, V):
     cols = torch.cat([x[:, oq:oq + nq], x[:, ok:ok + nq], x[:, ov:ov + nv]], 1)
     y = torch.zeros(T, 2 * nq + nv)
     for lo, hi, slot, fresh in _spans(m):
-        old = torch.zeros(K - 1, cols.shape[1], dtype=x.dtype) if fresh else conv[slot]
+        old = cols[:0] if K == 1 else torch.zeros_like(conv[slot]) if fresh else conv[slot]
         full = torch.cat([old, cols[lo:hi]], 0)
         y[lo:hi] = (full.float().unfold(0, K, 1) * taps[None]).sum(-1)
         if K > 1:
