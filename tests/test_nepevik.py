@@ -507,7 +507,7 @@ def test_mixed_head_attention_alone(form, H, G, D, V, size, keep):
         ldo = (H * V + 7) // 8 * 8
         out = F.head_mix_attention(to(form, rows.reshape(-1, H * D)), H, kc, vc, talk.to(dev), i32(cu),
                                    i32(pos), pt, scale, size, keep, seq_lens=seq_lens, ldo=ldo,
-                                   max_q=max(hi - lo for lo, hi in spans), max_k=max(hi for _, hi in spans))
+                                   max_k=max(hi for _, hi in spans))
         ref = torch.cat([a[lo:hi] for a, (lo, hi) in zip(want, spans)]).reshape(-1, H * V)
         close(out[:, :H * V], ref, form[1], f"spans {spans}", 1.5)
         assert ldo == H * V or float(out[:, H * V:].float().abs().max()) == 0.0

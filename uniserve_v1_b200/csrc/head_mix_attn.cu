@@ -9,10 +9,23 @@
 // weight of a key before any head's value product, so the softmax statistics (maximum and sum
 // per head) of all heads come first and the scores are formed a second time for the product.
 //
-// General form (any head width, bf16 or FP32 pages): one CTA per query row, all heads.  Keys
-// are read through the page table, the key list of a query being its kept keys followed by its
-// window.  All arithmetic is FP32.
+// Keys are read through the page table; the key list of a query is its kept keys followed by its
+// window.  Three forms:
+//
+// * row form (any head width, bf16 or FP32 pages): one CTA per query row, all heads, FP32 FMAs;
+// * decode form (bf16, one row per sequence): CTAs per (key split, kv head, sequence) write the
+//   scores and their statistics, then CTAs of the same shape turn every head's scores of their
+//   keys into mixed weights (FP32) and form the value product; the splits of a sequence are one
+//   thread-block cluster that sums its partial outputs in a fixed order.  Keys and values cross
+//   HBM once;
+// * tile form (bf16 prompts): a CTA takes 16 consecutive query rows and all heads.  A first sweep
+//   over the keys finds the statistics, a second one forms the probabilities, mixes them and
+//   multiplies the values, 16 keys at a time, on warp-level tensor instructions (every product
+//   of this operator is 16 rows high: an output head's weights exist only after all heads' scores
+//   of the same 16 x 16 tile do).  Probabilities and mixed weights enter the products as the sum
+//   of two bf16 values, which keeps 16 bits of their fraction; T is a bf16 tensor and exact.
 #include "include/us_common.cuh"
+#include "include/us_tc05.cuh"
 
 namespace {
 
@@ -139,7 +152,691 @@ __global__ void __launch_bounds__(kThreads) head_mix_row_kernel(const MixArgs a)
     st1(a.out, orow + c, a.bf16, c < H * V ? os[c] : 0.f);
 }
 
+// ------------------------------------------------------------------ decode --
+__device__ __forceinline__ void mma16816(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2,
+                                         uint32_t a3, uint32_t b0, uint32_t b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, "
+      "{%8,%9}, {%0,%1,%2,%3};"
+      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+      : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+
+struct StepArgs {
+  const __nv_bfloat16* q;
+  const __nv_bfloat16 *kc, *vc;
+  const float* talk;
+  __nv_bfloat16* out;
+  float* scores;              // [B, H, cap]
+  float* stats;               // [B, H, splits, 2]: maximum, sum of exponentials
+  const int *pos, *page_table, *seq_lens;
+  long long ldq, ldo;
+  int B, H, G, D, V, page, max_pages, size, keep, cap, splits;
+  float scale;
+};
+
+struct KeyList {
+  int n, lo, kept;
+  __device__ __forceinline__ int key(int x) const { return x < kept ? x : lo + x - kept; }
+};
+__device__ __forceinline__ KeyList key_list(int pos, int size, int keep, int cap) {
+  KeyList k;
+  k.lo = size > 0 ? max(0, pos - size + 1) : 0;
+  k.kept = min(max(keep, 0), k.lo);
+  k.n = min(cap, k.kept + pos - k.lo + 1);
+  return k;
+}
+
+constexpr int kStepThreads = 128;
+
+// Scores of one split's keys for the heads of one kv head.  A warp takes 8 keys per product: a
+// lane's 16-byte piece of a key row feeds two instructions, the queries' rows (at most 16 heads)
+// sit in registers in the same order of channels.  kD8 = 16-byte pieces per lane.
+template <int kD8>
+__global__ void __launch_bounds__(kStepThreads) head_mix_scores_kernel(const StepArgs a) {
+  US_PDL_PROLOGUE();
+  extern __shared__ __align__(16) float sc[];            // [rep][keys of the split]
+  const int split = blockIdx.x, u = blockIdx.y, b = blockIdx.z;
+  if (a.seq_lens[b] <= 0) return;
+  const int rep = a.H / a.G;
+  const KeyList kl = key_list(a.pos[b], a.size, a.keep, a.cap);
+  const int per = (kl.n + a.splits - 1) / a.splits;
+  const int k0 = min(kl.n, split * per), nk = min(kl.n, k0 + per) - k0;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int row = lane >> 2, kq = lane & 3;
+  uint4 qa[kD8], qb[kD8];
+  const __nv_bfloat16* qr = a.q + (long long)b * a.ldq + (long long)u * rep * a.D;
+#pragma unroll
+  for (int i = 0; i < kD8; ++i) {
+    const int d = (i * 4 + kq) * 8;
+    const uint4 z = make_uint4(0, 0, 0, 0);
+    qa[i] = (d < a.D && row < rep) ? *reinterpret_cast<const uint4*>(qr + (long long)row * a.D + d) : z;
+    qb[i] = (d < a.D && row + 8 < rep) ? *reinterpret_cast<const uint4*>(qr + (long long)(row + 8) * a.D + d) : z;
+  }
+  const int* pt = a.page_table + (long long)b * a.max_pages;
+  float* srow = a.scores + ((long long)b * a.H + (long long)u * rep) * a.cap;
+  for (int j0 = warp * 8; j0 < nk; j0 += kStepThreads / 4) {
+    const int x = min(k0 + j0 + row, kl.n - 1);
+    const int key = kl.key(x);
+    const __nv_bfloat16* kr =
+        a.kc + (((long long)pt[key / a.page] * a.page + key % a.page) * a.G + u) * a.D;
+    uint4 kv[kD8];
+#pragma unroll
+    for (int i = 0; i < kD8; ++i) {
+      const int d = (i * 4 + kq) * 8;
+      kv[i] = d < a.D ? *reinterpret_cast<const uint4*>(kr + d) : make_uint4(0, 0, 0, 0);
+    }
+    float c[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+    for (int i = 0; i < kD8; ++i) {
+      mma16816(c, qa[i].x, qb[i].x, qa[i].y, qb[i].y, kv[i].x, kv[i].y);
+      mma16816(c, qa[i].z, qb[i].z, qa[i].w, qb[i].w, kv[i].z, kv[i].w);
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int h = row + (e >> 1) * 8, j = j0 + kq * 2 + (e & 1);
+      if (h < rep && j < nk) {
+        const float v = c[e] * a.scale;
+        sc[h * per + j] = v;
+        srow[(long long)h * a.cap + k0 + j] = v;
+      }
+    }
+  }
+  __syncthreads();
+  for (int h = warp; h < rep; h += kStepThreads / 32) {
+    float m = -INFINITY, l = 0.f;
+    for (int j = lane; j < nk; j += 32) m = fmaxf(m, sc[h * per + j]);
+    m = us::warp_max(m);
+    for (int j = lane; j < nk; j += 32) l += expf(sc[h * per + j] - m);
+    l = us::warp_sum(l);
+    if (lane == 0) {
+      float* st = a.stats + (((long long)b * a.H + u * rep + h) * a.splits + split) * 2;
+      st[0] = m;
+      st[1] = l;
+    }
+  }
+}
+
+constexpr int kStepTile = 32;
+
+// Mixed weights and value product of one split's keys for the heads of one kv head.  Warp w
+// takes keys w, w + 4, ... of a tile, a lane VPL value columns of up to RM heads.
+template <int VPL, int RM>
+__global__ void __launch_bounds__(kStepThreads) head_mix_apply_kernel(const StepArgs a) {
+  US_PDL_PROLOGUE();
+  extern __shared__ __align__(16) float sm[];
+  const int split = blockIdx.x, u = blockIdx.y, b = blockIdx.z;
+  const int rep = a.H / a.G, H = a.H;
+  float* mx = sm;                              // [H] maximum
+  float* inv = mx + H;                         // [H] 1 / sum
+  float* tk = inv + H;                         // [rep][H]
+  float* ps = tk + rep * H;                    // [H][kStepTile]
+  float* ws = ps + H * kStepTile;              // [kStepTile][RM]
+  float* os = ws + kStepTile * RM;             // [4 warps][rep][V]
+  __shared__ long long where[kStepTile];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const bool live = a.seq_lens[b] > 0;         // the same in the whole cluster
+  float acc[RM][VPL];
+#pragma unroll
+  for (int r = 0; r < RM; ++r)
+#pragma unroll
+    for (int i = 0; i < VPL; ++i) acc[r][i] = 0.f;
+  if (live) {
+    const KeyList kl = key_list(a.pos[b], a.size, a.keep, a.cap);
+    const int per = (kl.n + a.splits - 1) / a.splits;
+    const int k0 = min(kl.n, split * per), k1 = min(kl.n, k0 + per);
+    const int* pt = a.page_table + (long long)b * a.max_pages;
+    for (int g = tid; g < H; g += kStepThreads) {
+      const float* st = a.stats + ((long long)b * H + g) * a.splits * 2;
+      float m = -INFINITY, l = 0.f;
+      for (int s = 0; s < a.splits; ++s) m = fmaxf(m, st[2 * s]);
+      for (int s = 0; s < a.splits; ++s)
+        if (st[2 * s + 1] > 0.f) l += st[2 * s + 1] * expf(st[2 * s] - m);
+      mx[g] = m;
+      inv[g] = 1.f / l;
+    }
+    for (int e = tid; e < rep * H; e += kStepThreads) tk[e] = a.talk[(long long)u * rep * H + e];
+    const float* srow = a.scores + (long long)b * H * a.cap;
+    for (int j0 = k0; j0 < k1; j0 += kStepTile) {
+      const int nj = min(kStepTile, k1 - j0);
+      __syncthreads();
+      if (tid < nj) {
+        const int key = kl.key(j0 + tid);
+        where[tid] = (long long)pt[key / a.page] * a.page + key % a.page;
+      }
+      for (int g = warp; g < H; g += kStepThreads / 32)
+        ps[g * kStepTile + lane] =
+            lane < nj ? expf(srow[(long long)g * a.cap + j0 + lane] - mx[g]) * inv[g] : 0.f;
+      __syncthreads();
+      for (int r = warp; r < RM; r += kStepThreads / 32) {
+        float w = 0.f;
+        if (r < rep)
+          for (int g = 0; g < H; ++g) w = fmaf(tk[r * H + g], ps[g * kStepTile + lane], w);
+        ws[lane * RM + r] = w;
+      }
+      __syncthreads();
+#pragma unroll 4
+      for (int j = warp; j < nj; j += kStepThreads / 32) {
+        const int c = lane * VPL;
+        float v[VPL];
+#pragma unroll
+        for (int i = 0; i < VPL; ++i) v[i] = 0.f;
+        if (c < a.V) {
+          const __nv_bfloat16* vr = a.vc + (where[j] * a.G + u) * a.V + c;
+          if (VPL == 4) {
+            us::Pack8 p;
+            p.u = *reinterpret_cast<const uint2*>(vr);
+#pragma unroll
+            for (int i = 0; i < VPL; ++i) v[i] = us::bf2f(p.b[i & 3]);
+          } else {
+            const __nv_bfloat162 p = *reinterpret_cast<const __nv_bfloat162*>(vr);
+            v[0] = us::bf2f(p.x);
+            v[1 % VPL] = us::bf2f(p.y);
+          }
+        }
+        const float* wr = ws + j * RM;
+#pragma unroll
+        for (int r = 0; r < RM; ++r)
+#pragma unroll
+          for (int i = 0; i < VPL; ++i) acc[r][i] = fmaf(wr[r], v[i], acc[r][i]);
+      }
+    }
+  }
+#pragma unroll
+  for (int r = 0; r < RM; ++r)
+#pragma unroll
+    for (int i = 0; i < VPL; ++i)
+      if (r < rep && lane * VPL + i < a.V) os[(warp * rep + r) * a.V + lane * VPL + i] = acc[r][i];
+  __syncthreads();
+  const int n = rep * a.V;
+  for (int e = tid; e < n; e += kStepThreads) os[e] = os[e] + os[n + e] + os[2 * n + e] + os[3 * n + e];
+  if (a.splits > 1) tc::cluster_sync();
+  // every CTA of the cluster finishes a share of the outputs, adding the splits in order
+  for (int e = tid + split * kStepThreads; e < n; e += kStepThreads * a.splits) {
+    float v = os[e];
+    if (a.splits > 1) {
+      const uint32_t local = (uint32_t)__cvta_generic_to_shared(&os[e]);
+      v = 0.f;
+      for (int p = 0; p < a.splits; ++p) v += tc::ld_dsmem_f32(tc::map_to_cta(local, (uint32_t)p));
+    }
+    a.out[(long long)b * a.ldo + (long long)u * n + e] = us::f2bf(v);
+  }
+  if (u == 0 && split == 0)
+    for (long long c = (long long)H * a.V + tid; c < a.ldo; c += kStepThreads)
+      a.out[(long long)b * a.ldo + c] = us::f2bf(0.f);
+  if (a.splits > 1) tc::cluster_sync();        // nobody leaves while its sums may still be read
+}
+
+template <int VPL, int RM>
+int launch_apply(const StepArgs& a, cudaStream_t stream) {
+  const int rep = a.H / a.G;
+  const size_t smem = (size_t)(2 * a.H + rep * a.H + a.H * kStepTile + kStepTile * RM + 4 * rep * a.V) * 4;
+  if (smem > 200 * 1024) return US_ERR_LIMIT;
+  static bool configured = false;
+  if (!configured) {
+    US_CUDA_CHECK(cudaFuncSetAttribute(head_mix_apply_kernel<VPL, RM>,
+                                       cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    configured = true;
+  }
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3(a.splits, a.G, a.B);
+  cfg.blockDim = dim3(kStepThreads);
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = stream;
+  cudaLaunchAttribute attr[2];
+  attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[0].val.programmaticStreamSerializationAllowed = us::pdl_enabled() ? 1 : 0;
+  attr[1].id = cudaLaunchAttributeClusterDimension;
+  attr[1].val.clusterDim.x = a.splits;
+  attr[1].val.clusterDim.y = 1;
+  attr[1].val.clusterDim.z = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = a.splits > 1 ? 2 : 1;
+  US_CUDA_CHECK(cudaLaunchKernelEx(&cfg, head_mix_apply_kernel<VPL, RM>, a));
+  return US_OK;
+}
+
+template <int kD8>
+int launch_scores(const StepArgs& a, cudaStream_t stream) {
+  const int rep = a.H / a.G;
+  const size_t smem = (size_t)rep * ((a.cap + a.splits - 1) / a.splits) * 4;
+  static bool configured = false;
+  if (!configured) {
+    US_CUDA_CHECK(cudaFuncSetAttribute(head_mix_scores_kernel<kD8>,
+                                       cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024));
+    configured = true;
+  }
+  US_CUDA_CHECK(us::launch_pdl(head_mix_scores_kernel<kD8>, dim3(a.splits, a.G, a.B),
+                               dim3(kStepThreads), smem, stream, a));
+  return US_OK;
+}
+
+// ------------------------------------------------------------------- tiles --
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void cp16(uint32_t dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+}
+__device__ __forceinline__ uint32_t pack_bf(float a, float b) {
+  __nv_bfloat162 p = __floats2bfloat162_rn(a, b);
+  return *reinterpret_cast<uint32_t*>(&p);
+}
+// x = hi + lo with both halves bf16
+__device__ __forceinline__ void split_bf(float x, float y, uint32_t& hi, uint32_t& lo) {
+  const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
+  hi = *reinterpret_cast<const uint32_t*>(&h);
+  lo = pack_bf(x - us::bf2f(h.x), y - us::bf2f(h.y));
+}
+
+struct TileArgs {
+  const __nv_bfloat16* q;
+  const __nv_bfloat16 *kc, *vc;
+  const float* talk;
+  __nv_bfloat16* out;
+  const int *cu, *pos, *page_table;
+  long long ldq, ldo;
+  int B, H, G, D, V, page, max_pages, size, keep;
+  float scale_log2;
+  int bufs;                   // key / value buffers (1 or 2)
+};
+
+constexpr int kTileThreads = 256;
+constexpr int kKeys = 16;             // keys per step
+constexpr int kOutHeads = 16;         // output heads per CTA (the mixture's 16 rows)
+constexpr int kPRow = 16 * kKeys * 2 + 16;   // bytes of a head's probabilities (16 x 16 bf16, padded)
+
+// byte offset of 16-byte piece c of row r in a tile whose rows hold `pieces` pieces (8 or 16):
+// pieces are XOR-swizzled by row so that 8 consecutive rows read 8 different bank groups
+template <int PIECES>
+__device__ __forceinline__ uint32_t swz(int r, int c) {
+  return (uint32_t)(r * PIECES + (c ^ (r & 7))) * 16u;
+}
+
+// HP: heads padded to 8, 16 or 32 (8 warps x HP / 8 heads); DP, VP: head widths padded to 64 or
+// 128.  blockIdx.x: query tile, blockIdx.y: group of 16 output heads.
+template <int HP, int DP, int VP>
+__global__ void __launch_bounds__(kTileThreads, 1) head_mix_tile_kernel(const TileArgs a) {
+  US_PDL_PROLOGUE();
+  constexpr int HW = HP / 8;                       // score heads per warp
+  constexpr int OW = HP >= 16 ? 2 : 1;             // output heads per warp
+  constexpr int DC = DP / 8, VC = VP / 8;          // 16-byte pieces per row
+  extern __shared__ __align__(1024) uint8_t smem[];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  // the query tile: 16 consecutive rows of one sequence
+  int tile = blockIdx.x, s = 0, row0 = 0, nrows = 0;
+  for (; s < a.B; ++s) {
+    const int lo = a.cu[s], n = a.cu[s + 1] - lo, t = (n + 15) >> 4;
+    if (tile < t) {
+      row0 = lo + tile * 16;
+      nrows = min(16, lo + n - row0);
+      break;
+    }
+    tile -= t;
+  }
+  if (nrows == 0) return;
+  const int rep = a.H / a.G;
+  const int h_out0 = blockIdx.y * kOutHeads;
+  const int n_out = min(kOutHeads, a.H - h_out0);
+  const int u_lo = h_out0 / rep, u_n = (h_out0 + n_out - 1) / rep - u_lo + 1;   // value heads needed
+  const uint32_t sq = tc::smem_u32(smem);                      // [HP][16][DC]
+  const uint32_t sk = sq + HP * 16 * DP * 2;                   // bufs x [G][16][DC]
+  const uint32_t k_bytes = (uint32_t)a.G * kKeys * DP * 2;
+  const uint32_t sv = sk + a.bufs * k_bytes;                   // bufs x [u_n][16][VC]
+  const uint32_t v_bytes = (uint32_t)u_n * kKeys * VP * 2;
+  const uint32_t sp = sv + a.bufs * v_bytes;                        // [2: hi, lo][HP16][kPRow]
+  constexpr int HK = HP < 16 ? 16 : HP;                        // mixture's inner extent
+  const uint32_t p_half = HK * kPRow;
+  // queries (heads past H, rows past the tile and channels past D are zero)
+  for (int e = tid; e < HP * 16 * DC; e += kTileThreads) {
+    const int h = e / (16 * DC), r = (e / DC) & 15, c = e & (DC - 1);
+    const uint32_t dst = sq + h * 16 * DP * 2 + swz<DC>(r, c);
+    if (h < a.H && r < nrows && c * 8 < a.D)
+      cp16(dst, a.q + (long long)(row0 + r) * a.ldq + (long long)h * a.D + c * 8);
+    else
+      asm volatile("st.shared.v4.u32 [%0], {%1,%1,%1,%1};" ::"r"(dst), "r"(0) : "memory");
+  }
+  if constexpr (HP < 16) {        // inner rows without a head
+    for (int e = tid; e < 2 * (16 - HP) * kPRow / 4; e += kTileThreads) {
+      const int half = e / ((16 - HP) * kPRow / 4), x = e - half * ((16 - HP) * kPRow / 4);
+      asm volatile("st.shared.u32 [%0], %1;" ::"r"(sp + half * p_half + HP * kPRow + x * 4), "r"(0) : "memory");
+    }
+  }
+  const int p0 = a.pos[row0], p1 = p0 + nrows - 1;
+  // keys of the tile: [0, keep) then [lo, p1], or one run from 0 when they meet
+  int lo = a.size > 0 ? max(0, p0 - a.size + 1) : 0;
+  int kept = max(a.keep, 0);
+  if (kept >= lo) { kept = 0; lo = 0; }
+  const int kt = (kept + kKeys - 1) / kKeys, steps = kt + (p1 - lo + kKeys) / kKeys;
+  const int* pt = a.page_table + (long long)s * a.max_pages;
+  auto first_key = [&](int st) { return st < kt ? st * kKeys : lo + (st - kt) * kKeys; };
+  auto end_key = [&](int st) { return st < kt ? kept : p1 + 1; };
+  auto load = [&](int st, int buf, bool values) {
+    const int k0 = first_key(st), k1 = end_key(st);
+    for (int e = tid; e < a.G * kKeys * DC; e += kTileThreads) {
+      const int r = e / (a.G * DC), x = e - r * a.G * DC, u = x / DC, c = x & (DC - 1);
+      const int key = k0 + r;
+      const uint32_t dst = sk + buf * k_bytes + u * kKeys * DP * 2 + swz<DC>(r, c);
+      if (key < k1 && c * 8 < a.D)
+        cp16(dst, a.kc + (((long long)pt[key / a.page] * a.page + key % a.page) * a.G + u) * a.D + c * 8);
+      else
+        asm volatile("st.shared.v4.u32 [%0], {%1,%1,%1,%1};" ::"r"(dst), "r"(0) : "memory");
+    }
+    if (values)
+      for (int e = tid; e < u_n * kKeys * VC; e += kTileThreads) {
+        const int r = e / (u_n * VC), x = e - r * u_n * VC, u = x / VC, c = x & (VC - 1);
+        const int key = k0 + r;
+        const uint32_t dst = sv + buf * v_bytes + u * kKeys * VP * 2 + swz<VC>(r, c);
+        if (key < k1 && c * 8 < a.V)
+          cp16(dst, a.vc + (((long long)pt[key / a.page] * a.page + key % a.page) * a.G + u_lo + u) * a.V + c * 8);
+        else
+          asm volatile("st.shared.v4.u32 [%0], {%1,%1,%1,%1};" ::"r"(dst), "r"(0) : "memory");
+      }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  const int lrow = lane & 15, lhalf = lane >> 4;     // ldmatrix row / 8-column half of this lane
+  const int r0 = lane >> 2, cq = (lane & 3) * 2;     // accumulator row and first column
+  // scores of the warp's heads for one step: S[16 rows][16 keys] per head, columns cq, cq + 1
+  // of the two 8-key halves
+  auto scores = [&](int buf, float (&sc)[HW][2][4]) {
+#pragma unroll
+    for (int i = 0; i < HW; ++i)
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) sc[i][n][e] = 0.f;
+    const int g0 = warp * HW;
+#pragma unroll
+    for (int k = 0; k < DC / 2; ++k) {
+      int u_prev = -1;
+      uint32_t bk[4];
+#pragma unroll
+      for (int i = 0; i < HW; ++i) {
+        if (g0 + i >= a.H) break;
+        const int u = (g0 + i) / rep;
+        if (u != u_prev) {
+          // keys are the instruction's columns: rows lrow of the tile, channel halves
+          ldsm4(bk, sk + buf * k_bytes + u * kKeys * DP * 2 + swz<DC>(lrow, 2 * k + lhalf));
+          u_prev = u;
+        }
+        uint32_t aq[4];
+        ldsm4(aq, sq + (g0 + i) * 16 * DP * 2 + swz<DC>(lrow, 2 * k + lhalf));
+        mma16816(sc[i][0], aq[0], aq[1], aq[2], aq[3], bk[0], bk[2]);
+        mma16816(sc[i][1], aq[0], aq[1], aq[2], aq[3], bk[1], bk[3]);
+      }
+    }
+  };
+  // whether row r0 (+8) of the tile sees the key behind accumulator element (n, e)
+  auto sees = [&](int k0, int k1, int n, int e) {
+    const int i = p0 + r0 + (e >> 1) * 8, j = k0 + n * 8 + cq + (e & 1);
+    return j < k1 && j <= i && (a.size <= 0 || i - j < a.size || j < a.keep);
+  };
+  // ---- first sweep: maximum and sum of every (row, head), in the log2 domain ----
+  float mx[HW][2], sum[HW][2];
+#pragma unroll
+  for (int i = 0; i < HW; ++i) {
+    mx[i][0] = mx[i][1] = -INFINITY;
+    sum[i][0] = sum[i][1] = 0.f;
+  }
+  // A step's keys (and values) are fetched while the step before computes, into the other
+  // buffer; with one buffer (shapes whose tiles do not fit twice) they are fetched in between.
+  const bool two = a.bufs == 2;
+  auto next_step = [&](int st, bool values) -> int {
+    if (!two) {
+      __syncthreads();                      // the step before is done with the buffer
+      load(st, 0, values);
+    } else if (st == 0) {
+      __syncthreads();
+      load(0, 0, values);
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();                        // visible to all; everybody has left the step before
+    if (two && st + 1 < steps) load(st + 1, (st + 1) & 1, values);
+    return two ? st & 1 : 0;
+  };
+  for (int st = 0; st < steps; ++st) {
+    const int buf = next_step(st, false);
+    float sc[HW][2][4];
+    scores(buf, sc);
+    const int k0 = first_key(st), k1 = end_key(st);
+#pragma unroll
+    for (int i = 0; i < HW; ++i)
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        float v[4], m = mx[i][r];
+#pragma unroll
+        for (int x = 0; x < 4; ++x) {
+          const int n = x >> 1, e = r * 2 + (x & 1);
+          v[x] = sees(k0, k1, n, e) ? sc[i][n][e] * a.scale_log2 : -INFINITY;
+          m = fmaxf(m, v[x]);
+        }
+        if (m == -INFINITY) continue;
+        float l = sum[i][r] * exp2f(mx[i][r] - m);
+#pragma unroll
+        for (int x = 0; x < 4; ++x) l += exp2f(v[x] - m);
+        sum[i][r] = l;
+        mx[i][r] = m;
+      }
+  }
+#pragma unroll
+  for (int i = 0; i < HW; ++i)
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+#pragma unroll
+      for (int o = 1; o < 4; o <<= 1) {
+        const float m2 = __shfl_xor_sync(0xffffffffu, mx[i][r], o);
+        const float l2 = __shfl_xor_sync(0xffffffffu, sum[i][r], o);
+        const float m = fmaxf(mx[i][r], m2);
+        if (m != -INFINITY) sum[i][r] = sum[i][r] * exp2f(mx[i][r] - m) + l2 * exp2f(m2 - m);
+        mx[i][r] = m;
+      }
+      sum[i][r] = sum[i][r] > 0.f ? 1.f / sum[i][r] : 0.f;
+    }
+  // ---- the mixture's rows T[h_out0 + 0..15][g] as operand fragments ----
+  uint32_t tf[HK / 16][4];
+#pragma unroll
+  for (int k = 0; k < HK / 16; ++k)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int h = r0 + (e & 1) * 8, g = k * 16 + cq + (e >> 1) * 8;
+      const float* t = a.talk + (long long)(h_out0 + h) * a.H + g;
+      tf[k][e] = pack_bf(h < n_out && g < a.H ? t[0] : 0.f, h < n_out && g + 1 < a.H ? t[1] : 0.f);
+    }
+  float o[OW][VP / 8][4];
+#pragma unroll
+  for (int i = 0; i < OW; ++i)
+#pragma unroll
+    for (int n = 0; n < VP / 8; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) o[i][n][e] = 0.f;
+  // ---- second sweep ----
+  for (int st = 0; st < steps; ++st) {
+    const int buf = next_step(st, true);    // (the step before has read its mixed weights)
+    {
+      float sc[HW][2][4];
+      scores(buf, sc);
+      const int k0 = first_key(st), k1 = end_key(st);
+#pragma unroll
+      for (int i = 0; i < HW; ++i)
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+          for (int r = 0; r < 2; ++r) {
+            const int g = warp * HW + i;
+            const float x = sees(k0, k1, n, r * 2) ? exp2f(sc[i][n][r * 2] * a.scale_log2 - mx[i][r]) * sum[i][r] : 0.f;
+            const float y = sees(k0, k1, n, r * 2 + 1) ? exp2f(sc[i][n][r * 2 + 1] * a.scale_log2 - mx[i][r]) * sum[i][r] : 0.f;
+            uint32_t hi, low;
+            split_bf(g < a.H ? x : 0.f, g < a.H ? y : 0.f, hi, low);
+            const uint32_t dst = sp + g * kPRow + ((r0 + r * 8) * kKeys + n * 8 + cq) * 2;
+            asm volatile("st.shared.u32 [%0], %1;" ::"r"(dst), "r"(hi) : "memory");
+            asm volatile("st.shared.u32 [%0], %1;" ::"r"(dst + p_half), "r"(low) : "memory");
+          }
+    }
+    __syncthreads();
+    // mixture: the warp's 32 columns (2 query rows x 16 keys) of all heads, written back in place
+    {
+      float w[4][4];
+#pragma unroll
+      for (int n = 0; n < 4; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) w[n][e] = 0.f;
+#pragma unroll
+      for (int k = 0; k < HK / 16; ++k)
+#pragma unroll
+        for (int part = 0; part < 2; ++part)
+#pragma unroll
+          for (int n2 = 0; n2 < 2; ++n2) {
+            uint32_t bp[4];
+            ldsm4t(bp, sp + part * p_half + (k * 16 + lrow) * kPRow + (warp * 32 + n2 * 16 + lhalf * 8) * 2);
+            mma16816(w[n2 * 2], tf[k][0], tf[k][1], tf[k][2], tf[k][3], bp[0], bp[1]);
+            mma16816(w[n2 * 2 + 1], tf[k][0], tf[k][1], tf[k][2], tf[k][3], bp[2], bp[3]);
+          }
+      __syncwarp();
+#pragma unroll
+      for (int n = 0; n < 4; ++n)
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+          if (HP < 16 && r == 1) continue;
+          uint32_t hi, low;
+          split_bf(w[n][r * 2], w[n][r * 2 + 1], hi, low);
+          const uint32_t dst = sp + (r0 + r * 8) * kPRow + (warp * 32 + n * 8 + cq) * 2;
+          asm volatile("st.shared.u32 [%0], %1;" ::"r"(dst), "r"(hi) : "memory");
+          asm volatile("st.shared.u32 [%0], %1;" ::"r"(dst + p_half), "r"(low) : "memory");
+        }
+    }
+    __syncthreads();
+    // value product of the warp's output heads
+#pragma unroll
+    for (int i = 0; i < OW; ++i) {
+      const int h = warp * OW + i;
+      if (h >= n_out) break;
+      uint32_t wh[4], wl[4];
+      ldsm4(wh, sp + h * kPRow + (lrow * kKeys + lhalf * 8) * 2);
+      ldsm4(wl, sp + p_half + h * kPRow + (lrow * kKeys + lhalf * 8) * 2);
+      const uint32_t vb = sv + buf * v_bytes + ((h_out0 + h) / rep - u_lo) * kKeys * VP * 2;
+#pragma unroll
+      for (int n2 = 0; n2 < VC / 2; ++n2) {
+        uint32_t bv[4];
+        ldsm4t(bv, vb + swz<VC>(lrow, 2 * n2 + lhalf));
+        mma16816(o[i][2 * n2], wh[0], wh[1], wh[2], wh[3], bv[0], bv[1]);
+        mma16816(o[i][2 * n2 + 1], wh[0], wh[1], wh[2], wh[3], bv[2], bv[3]);
+        mma16816(o[i][2 * n2], wl[0], wl[1], wl[2], wl[3], bv[0], bv[1]);
+        mma16816(o[i][2 * n2 + 1], wl[0], wl[1], wl[2], wl[3], bv[2], bv[3]);
+      }
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < OW; ++i) {
+    const int h = warp * OW + i;
+    if (h >= n_out) break;
+#pragma unroll
+    for (int n = 0; n < VP / 8; ++n)
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        const int c = n * 8 + cq, row = r0 + r * 8;
+        if (row < nrows && c < a.V)
+          *reinterpret_cast<uint32_t*>(a.out + (long long)(row0 + row) * a.ldo + (long long)(h_out0 + h) * a.V + c) =
+              pack_bf(o[i][n][r * 2], o[i][n][r * 2 + 1]);
+      }
+  }
+  if (blockIdx.y == 0)
+    for (int r = 0; r < nrows; ++r)
+      for (long long c = (long long)a.H * a.V + tid; c < a.ldo; c += kTileThreads)
+        a.out[(long long)(row0 + r) * a.ldo + c] = us::f2bf(0.f);
+}
+
+template <int HP, int DP, int VP>
+int launch_tile(TileArgs a, int tiles, cudaStream_t stream) {
+  const int rep = a.H / a.G;
+  int u_n = 1;
+  for (int h0 = 0; h0 < a.H; h0 += kOutHeads) {
+    const int last = (a.H < h0 + kOutHeads ? a.H : h0 + kOutHeads) - 1;
+    const int n = last / rep - h0 / rep + 1;
+    u_n = n > u_n ? n : u_n;
+  }
+  const size_t fixed = (size_t)HP * 16 * DP * 2 + 2 * (size_t)(HP < 16 ? 16 : HP) * kPRow;
+  const size_t tile = (size_t)a.G * kKeys * DP * 2 + (size_t)u_n * kKeys * VP * 2;
+  a.bufs = fixed + 2 * tile <= 227 * 1024 ? 2 : 1;
+  const size_t smem = fixed + a.bufs * tile;
+  if (smem > 227 * 1024) return US_ERR_LIMIT;
+  static bool configured = false;
+  if (!configured) {
+    US_CUDA_CHECK(cudaFuncSetAttribute(head_mix_tile_kernel<HP, DP, VP>,
+                                       cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
+    configured = true;
+  }
+  US_CUDA_CHECK(us::launch_pdl(head_mix_tile_kernel<HP, DP, VP>,
+                               dim3(tiles, (a.H + kOutHeads - 1) / kOutHeads), dim3(kTileThreads), smem,
+                               stream, a));
+  return US_OK;
+}
+
 }  // namespace
+
+// Bytes of scratch of the decode form for rows whose key lists hold at most `cap` keys.
+US_API long long us_head_mix_decode_scratch(int B, int H, int cap, int splits) {
+  return 4LL * B * H * ((long long)cap + 2LL * splits);
+}
+
+// One bf16 row per sequence; US_ERR_UNSUPPORTED / US_ERR_LIMIT for shapes of the row form.
+US_API int us_head_mix_decode(const void* q, const void* kc, const void* vc, const float* talk,
+                              void* out, const int* pos, const int* page_table, const int* seq_lens,
+                              void* scratch, long long ldq, long long ldo, int B, int H, int G, int D,
+                              int V, int page, int max_pages, int size, int keep, int cap, int splits,
+                              float scale, void* stream_) {
+  US_REQUIRE(q && kc && vc && talk && out && pos && page_table && seq_lens && scratch && B >= 1);
+  US_REQUIRE(H >= 1 && G >= 1 && H % G == 0 && page >= 1 && cap >= 1 && splits >= 1 && splits <= 8);
+  US_REQUIRE(ldo >= (long long)H * V && ((uintptr_t)q % 16) == 0 && ((uintptr_t)kc % 16) == 0 &&
+             ((uintptr_t)vc % 16) == 0 && (ldq % 8) == 0);
+  const int rep = H / G;
+  if ((D % 8) || D > 256 || (V % 4) || V > 128 || rep > 16 || B > 65535) return US_ERR_UNSUPPORTED;
+  if ((long long)rep * ((cap + splits - 1) / splits) * 4 > 100 * 1024) return US_ERR_LIMIT;
+  StepArgs a{(const __nv_bfloat16*)q, (const __nv_bfloat16*)kc, (const __nv_bfloat16*)vc, talk,
+             (__nv_bfloat16*)out, (float*)scratch, (float*)scratch + (long long)B * H * cap, pos,
+             page_table, seq_lens, ldq, ldo, B, H, G, D, V, page, max_pages, size, keep, cap, splits,
+             scale};
+  cudaStream_t stream = (cudaStream_t)stream_;
+  int rc = D <= 64 ? launch_scores<2>(a, stream) : D <= 128 ? launch_scores<4>(a, stream)
+                                                            : launch_scores<8>(a, stream);
+  if (rc) return rc;
+#define US_HM(VPL) \
+  return rep <= 4 ? launch_apply<VPL, 4>(a, stream) : rep <= 8 ? launch_apply<VPL, 8>(a, stream) : launch_apply<VPL, 16>(a, stream);
+  if (V <= 64) { US_HM(2) }
+  US_HM(4)
+#undef US_HM
+}
+
+// bf16 rows of packed sequences; `rows` bounds the tiles.
+US_API int us_head_mix_prefill(const void* q, const void* kc, const void* vc, const float* talk,
+                               void* out, const int* cu, const int* pos, const int* page_table,
+                               long long ldq, long long ldo, int rows, int B, int H, int G, int D,
+                               int V, int page, int max_pages, int size, int keep, float scale,
+                               void* stream_) {
+  US_REQUIRE(q && kc && vc && talk && out && cu && pos && page_table && rows >= 1 && B >= 1);
+  US_REQUIRE(H >= 1 && G >= 1 && H % G == 0 && page >= 1 && ldo >= (long long)H * V);
+  US_REQUIRE(((uintptr_t)q % 16) == 0 && ((uintptr_t)kc % 16) == 0 && ((uintptr_t)vc % 16) == 0 &&
+             (ldq % 8) == 0 && (ldo % 2) == 0);
+  if ((D % 8) || D > 128 || (V % 8) || V > 128 || H > 32) return US_ERR_UNSUPPORTED;
+  TileArgs a{(const __nv_bfloat16*)q, (const __nv_bfloat16*)kc, (const __nv_bfloat16*)vc, talk,
+             (__nv_bfloat16*)out, cu, pos, page_table, ldq, ldo, B, H, G, D, V, page, max_pages, size,
+             keep, scale * 1.4426950408889634f, 2};
+  cudaStream_t stream = (cudaStream_t)stream_;
+  const int tiles = rows / 16 + B;
+#define US_HT2(HP, DP) \
+  return V <= 64 ? launch_tile<HP, DP, 64>(a, tiles, stream) : launch_tile<HP, DP, 128>(a, tiles, stream);
+#define US_HT(HP) \
+  if (D <= 64) { US_HT2(HP, 64) } else { US_HT2(HP, 128) }
+  if (H <= 8) { US_HT(8) }
+  if (H <= 16) { US_HT(16) }
+  US_HT(32)
+#undef US_HT
+#undef US_HT2
+}
 
 // q [rows, H * D] (row stride ldq) of the packed sequences cu [B + 1], positions pos [rows];
 // every key up to a row's own position is in the pages already.  Output rows are ldo wide

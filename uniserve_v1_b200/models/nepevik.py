@@ -403,7 +403,7 @@ class NepevikModel:
                            self.cfg.eps)
         att = F.head_mix_attention(proj[:, :H * D], H, kc, vc, w["talk"], m.cu, positions,
                                    meta.page_table, s.scale, s.window, s.keep_first,
-                                   seq_lens=meta.seq_lens, ldo=w["o"].shape[1])
+                                   seq_lens=meta.seq_lens, ldo=w["o"].shape[1], max_k=meta.max_k)
         return F.linear(att, w["o"])
 
     def forward(self, input_ids, positions, meta, kv_caches) -> torch.Tensor:

@@ -671,13 +671,37 @@ def tanh_cols_(x, off, n):
            N.stream())
 
 
+def _mix_splits(B, H, G, cap):
+    """Key splits of the decode form of head-mixed attention: enough CTAs for every SM, at least
+    64 keys each, scores of a split within shared memory (None: they never are)."""
+    rep = H // G
+    fit = -(-rep * cap * 4 // (100 * 1024))
+    want = max(1, min(-(-592 // (B * G)), cap // 64, 8))
+    splits = max(want, fit)
+    while splits <= 8 and rep * (-(-cap // splits)) * 4 > 100 * 1024:
+        splits += 1
+    return splits if splits <= 8 else None
+
+
+def _mix_tile_fits(H, G, D, V):
+    """Whether the tile form's operands fit a CTA's shared memory (one key / value buffer)."""
+    HP, DP, VP = (8 if H <= 8 else 16 if H <= 16 else 32), (64 if D <= 64 else 128), (64 if V <= 64 else 128)
+    rep = H // G
+    u_n = max((min(H, h0 + 16) - 1) // rep - h0 // rep + 1 for h0 in range(0, H, 16))
+    return HP * 16 * DP * 2 + 2 * max(HP, 16) * 528 + 16 * 2 * (G * DP + u_n * VP) <= 227 * 1024
+
+
 def head_mix_attention(q, H, kcache, vcache, talk, cu, positions, page_table, scale, size=0,
-                       keep=0, seq_lens=None, ldo=None, max_q=0, max_k=0):
+                       keep=0, seq_lens=None, ldo=None, max_k=0):
     """Causal attention whose heads' softmax weights are mixed by ``talk`` [H, H] (FP32) before
     the values: q [T, H * D] (row-strided view), pages [n, page, G, D] and [n, page, G, V], rows
     of sequence s at cu[s] .. cu[s + 1], keys up to a row's own position read through
     ``page_table``.  ``size`` / ``keep``: sliding window and always-visible first keys (0: off).
-    Returns [T, ldo] rows (columns past H * V zero)."""
+    With ``seq_lens`` every sequence brings one row (length 0: padding) and ``max_k`` bounds the
+    keys of a sequence.  Returns [T, ldo] rows (columns past H * V zero).
+
+    bf16 rows take the decode or the tile form of the kernel, FP32 rows and unusual head widths
+    the row form (``csrc/head_mix_attn.cu``)."""
     T = q.shape[0]
     _, page, G, D = kcache.shape
     V = vcache.shape[3]
@@ -686,10 +710,32 @@ def head_mix_attention(q, H, kcache, vcache, talk, cu, positions, page_table, sc
         return R.head_mix_attention(q, H, kcache, vcache, talk, cu, positions, page_table, scale,
                                     size, keep, ldo)
     out = torch.empty(T, ldo, dtype=q.dtype, device=q.device)
+    if T == 0:
+        return out
+    B, max_pages = cu.shape[0] - 1, page_table.shape[1]
+    if q.dtype == BF16 and D % 8 == 0 and q.stride(0) % 8 == 0:
+        if seq_lens is not None and D <= 256 and V % 4 == 0 and V <= 128 and H // G <= 16:
+            cap = max_k or page * max_pages
+            if size > 0:
+                cap = min(cap, size + max(keep, 0))
+            splits = _mix_splits(B, H, G, cap)
+            if splits is not None:
+                scratch = torch.empty(N.kernels().us_head_mix_decode_scratch(B, H, cap, splits),
+                                      dtype=torch.uint8, device=q.device)
+                N.call("us_head_mix_decode", N.ptr(q), N.ptr(kcache), N.ptr(vcache), N.ptr(talk),
+                       N.ptr(out), N.ptr(positions), N.ptr(page_table), N.ptr(seq_lens),
+                       N.ptr(scratch), q.stride(0), ldo, B, H, G, D, V, page, max_pages, size, keep,
+                       cap, splits, scale, N.stream(), launches=2)
+                return out
+        if seq_lens is None and D <= 128 and V <= 128 and V % 8 == 0 and H <= 32 and \
+                _mix_tile_fits(H, G, D, V):
+            N.call("us_head_mix_prefill", N.ptr(q), N.ptr(kcache), N.ptr(vcache), N.ptr(talk),
+                   N.ptr(out), N.ptr(cu), N.ptr(positions), N.ptr(page_table), q.stride(0), ldo, T, B,
+                   H, G, D, V, page, max_pages, size, keep, scale, N.stream())
+            return out
     N.call("us_head_mix_attention", N.ptr(q), N.ptr(kcache), N.ptr(vcache), N.ptr(talk), N.ptr(out),
-           N.ptr(cu), N.ptr(positions), N.ptr(page_table), N.ptr(seq_lens), q.stride(0), ldo, T,
-           cu.shape[0] - 1, H, G, D, V, page, page_table.shape[1], size, keep, scale,
-           int(q.dtype == BF16), N.stream())
+           N.ptr(cu), N.ptr(positions), N.ptr(page_table), N.ptr(seq_lens), q.stride(0), ldo, T, B, H,
+           G, D, V, page, max_pages, size, keep, scale, int(q.dtype == BF16), N.stream())
     return out
 
 

@@ -53,6 +53,10 @@ _SIGNATURES = {
     "us_tanh_cols": (I, [P, L, I, I, I, I, P]),
     "us_head_mix_attention": (I, [P, P, P, P, P, P, P, P, P, L, L, I, I, I, I, I, I, I, I, I, I, F,
                                   I, P]),
+    "us_head_mix_decode_scratch": (L, [I, I, I, I]),
+    "us_head_mix_decode": (I, [P, P, P, P, P, P, P, P, P, L, L, I, I, I, I, I, I, I, I, I, I, I, F,
+                               P]),
+    "us_head_mix_prefill": (I, [P, P, P, P, P, P, P, P, L, L, I, I, I, I, I, I, I, I, I, I, F, P]),
     "us_table_route_sort": (I, [P, P, I, I, I, I, I, I, I, P, P, P, P, P, P, P, P, P]),
     "us_kv_write_scaled": (I, [P, P, L, L, P, P, P, P, P, I, I, I, I, P]),
     "us_kv_gather": (I, [P, P, P, P, P, I, P, P, I, I, I, I, I, P, P, L, I, P]),

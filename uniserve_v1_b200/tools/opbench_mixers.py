@@ -1,0 +1,182 @@
+"""Kernels of the vector-decay, head-mixing and table-routed layers beside the like kernels of
+the hybrid and Qwen3 decoders at equal sizes, each with its roofline fraction.
+
+    python -m uniserve_v1_b200.tools.opbench_mixers [--only NAME,...] [--batch 64] [--rows 8192]
+
+One JSON line per case.  ``bytes`` / ``flops`` are the algorithm's (every operand once), the
+fraction is of the measured copy bandwidth or cuBLAS bf16 throughput (see ``opbench``); L2 is
+flushed between iterations.
+"""
+from __future__ import annotations
+
+import argparse
+import json
+
+import torch
+
+from ..ops import functional as F
+from ..ops import gated_delta as GD
+from ..ops import vector_delta as VD
+from .opbench import peaks, timeit
+
+
+def main():
+    ap = argparse.ArgumentParser()
+    ap.add_argument("--only", default="")
+    ap.add_argument("--batch", type=int, default=64, help="sequences of a decode step")
+    ap.add_argument("--rows", type=int, default=8192, help="tokens of a prompt")
+    ap.add_argument("--iters", type=int, default=7)
+    a = ap.parse_args()
+    dev, bf = torch.device("cuda"), torch.bfloat16
+    torch.manual_seed(0)
+    tbs, tfl, tag = peaks()
+    only = [x for x in a.only.split(",") if x]
+    f32 = dict(dtype=torch.float32, device=dev)
+
+    def rnd(*s, dtype=bf):
+        return torch.randn(*s, device=dev).to(dtype)
+
+    def i32(x):
+        return torch.tensor(x, dtype=torch.int32, device=dev)
+
+    def case(name, fn, bytes_=None, flops=None, **info):
+        if only and not any(name.startswith(x) for x in only):
+            return
+        fn()
+        torch.cuda.synchronize()
+        graph = torch.cuda.CUDAGraph()      # launch latency of the host left out
+        with torch.cuda.graph(graph):
+            fn()
+        ms = timeit(graph.replay, a.iters)
+        out = {"case": name, "ms": round(ms, 4)}
+        if bytes_:
+            out["frac_memory"] = round(bytes_ / ms / 1e9 / tbs, 3)
+        if flops:
+            out["frac_tensor"] = round(flops / ms / 1e9 / tfl, 3)
+        out.update(info, roofline=tag)
+        print(json.dumps(out), flush=True)
+
+    B, T = a.batch, a.rows
+    metas = {"decode": (B, VD.SeqMeta(i32(list(range(B + 1))), i32(list(range(B))),
+                                      torch.full((B,), 2000, dtype=torch.int32, device=dev), True)),
+             "prefill": (T, VD.SeqMeta(i32([0, T]), i32([0]),
+                                       torch.arange(T, dtype=torch.int32, device=dev), False))}
+    H, Hk, D, V, K, W = 32, 16, 128, 128, 4, 2048
+    # ---- recurrences ----
+    pool = torch.zeros(B, H, D, V, **f32)
+    for kind, (n, m) in metas.items():
+        state = 2.0 * (B if kind == "decode" else 1) * H * D * V * 4
+        q, k, v = rnd(n, Hk, D, dtype=torch.float32), rnd(n, Hk, D, dtype=torch.float32), rnd(n, H, V, dtype=torch.float32)
+        k = k / k.norm(dim=-1, keepdim=True)
+        g, beta = torch.rand(n, H, D, device=dev) * 0.1 + 0.9, torch.rand(n, H, device=dev)
+        vec = 4.0 * n * (2 * Hk * D + H * (D + 2 * V) + H)
+        case(f"channel_rule_{kind}", lambda: VD.vector_delta_rule(q, k, v, g, pool, m, beta=beta),
+             state + vec)
+        D2 = 64
+        pool2 = pool.view(-1)[:B * H * D2 * D2].view(B, H, D2, D2)
+        r2, k2, v2 = rnd(n, H, D2), rnd(n, H, D2), rnd(n, H, D2)
+        u2 = k2.float() / k2.float().norm(dim=-1, keepdim=True)
+        g2, p2 = torch.rand(n, H, D2, device=dev) * 0.1 + 0.9, u2 * 0.5
+        k2 = (k2.float() * 0.1).to(bf)
+        case(f"general_rule_{kind}", lambda: VD.vector_delta_rule(r2, k2, v2, g2, pool2, m, n=u2, p=p2),
+             2.0 * (B if kind == "decode" else 1) * H * D2 * D2 * 4 + n * H * D2 * (3 * 4 + 3 * 2 + 4.0))
+        qb, kb, vb = rnd(n, Hk, D), rnd(n, Hk, D), rnd(n, H, V)
+        ar, br, A, dtb = rnd(n, H), rnd(n, H), -torch.rand(H, device=dev) - 0.2, torch.rand(H, device=dev)
+        case(f"gated_rule_{kind} (like)", lambda: GD.gated_delta_rule_packed(
+            qb, kb, vb, pool, m.cu, m.slots, raw=(ar, br, A, dtb)),
+            state + n * (2 * Hk * D + H * V + 2 * H) * 2.0 + n * H * V * 4.0)
+        # ---- preparation (convolutions, unit vectors, decay) ----
+        C = 2 * Hk * D + H * V
+        x, low = rnd(n, C + 64), rnd(n, H * D, dtype=torch.float32)
+        w = {"conv_q": rnd(Hk * D, K, dtype=torch.float32), "conv_k": rnd(Hk * D, K, dtype=torch.float32),
+             "conv_v": rnd(H * V, K, dtype=torch.float32), "A_log": rnd(H, dtype=torch.float32),
+             "dt_bias": rnd(H * D, dtype=torch.float32), "w0": rnd(H * D2, dtype=torch.float32),
+             "a_bias": rnd(H * D2, dtype=torch.float32)}
+        conv = torch.zeros(B, K - 1, C, dtype=bf, device=dev)
+        case(f"channel_prep_{kind}", lambda: VD.channel_prep(x, (0, Hk * D, 2 * Hk * D, C), low, w, conv, m, H, Hk, D, V),
+             n * (2.0 * C + 4 * H * D) + vec - n * H * V * 4.0 + (2 * B * (K - 1) * C * 2.0 if kind == "decode" else 0))
+        xc = rnd(n, C)
+        wc = rnd(C, K, dtype=torch.float32)
+        case(f"causal_conv1d_{kind} (like)", lambda: GD.causal_conv1d(xc, wc, conv, cu=m.cu, slots=m.slots),
+             4.0 * n * C + (2 * B * (K - 1) * C * 2.0 if kind == "decode" else 0))
+        xg, lowg = rnd(n, 5 * H * D2), rnd(n, H * D2, dtype=torch.float32)
+        case(f"general_prep_{kind}", lambda: VD.general_prep(xg, (H * D2, 4 * H * D2), lowg, w, H, D2),
+             n * H * D2 * (2 * 2 + 4 + 12.0))
+        o, gate, hw = rnd(n, H, V, dtype=torch.float32), rnd(n, H * V), rnd(V, dtype=torch.float32)
+        case(f"head_norm_gate_{kind}", lambda: VD.head_norm_gate(o, hw, gate, 1e-6, H * V, bf), n * H * V * 8.0)
+        zz = gate.view(n, H, V)
+        case(f"rmsnorm_gated_{kind} (like)", lambda: GD.rmsnorm_gated(o, hw, zz, 1e-6), n * H * V * 8.0)
+        # ---- residual rows ----
+        y, res = rnd(n, W), rnd(n, W, dtype=torch.float32)
+        case(f"output_norm_add_{kind}", lambda: F.output_norm_add_(y, res, 0.5, 1e-6, W), n * W * (2 + 4 + 4 + 2.0))
+        nw = rnd(W)
+        case(f"add_rmsnorm_{kind} (like)", lambda: F.add_rmsnorm(y, res, nw), n * W * (2 + 4 + 4 + 2.0))
+        top, E, I = 4, 64, 768
+        rows, shared = rnd(n * top, W), rnd(n, W)
+        perm = torch.randperm(n * top, device=dev).view(n, top).to(torch.int32)
+        sg = rnd(W, dtype=torch.float32) * 0.01
+        case(f"output_norm_add_routed_{kind}", lambda: F.output_norm_add_(
+            None, res, 0.5, 1e-6, W, routed=(rows, perm, 0.25), shared=shared, shared_gate=sg),
+            n * W * (2 * top + 2 + 4 + 4 + 2.0))
+        wts = torch.rand(n, top, device=dev)
+        case(f"unpermute_add_rmsnorm_{kind} (like)", lambda: F.unpermute_add_rmsnorm(rows, perm, wts, res, nw),
+             n * W * (2 * top + 4 + 4 + 2.0))
+        # ---- routing and experts ----
+        tok = torch.randint(0, 50000, (n,), device=dev, dtype=torch.int32)
+        tables = torch.rand(8, 50000, E, device=dev).argsort(-1)[:, :, :top].to(torch.int32).contiguous()
+        case(f"table_routes_8_layers_{kind}", lambda: F.table_routes(tok, tables, E))
+        routes = F.table_routes(tok, tables, E)[0]
+        up, down = rnd(E, I, W), rnd(E, W, I)
+        wb = 2.0 * E * I * W * 2 if n * top >= 2 * E else 2.0 * n * top * I * W * 2
+        case(f"routed_mlp_{kind}", lambda: F.routed_mlp(y, routes, up, down),
+             wb + n * top * (2 * W + I) * 2.0, 4.0 * n * top * I * W)
+        w13 = rnd(E, 2 * I, W)
+        ws = F.MoeWorkspace.create(n, top, E, W, I, dev)
+        ids = routes.ids.contiguous()
+        case(f"moe_experts_{kind} (like)", lambda: F.moe_experts(y, ids, wts, w13, down, ws=ws, defer_unpermute=True),
+             1.5 * wb + n * top * (2 * W + I) * 2.0, 6.0 * n * top * I * W)
+        # ---- attention over pages: window 1024 + 4 first keys ----
+        Hq, G, page, size, keep = 32, 4, 16, 1024, 4
+        ctx = 2048 if kind == "decode" else n
+        seqs = B if kind == "decode" else 1
+        per = (ctx + page - 1) // page
+        kc, vc = rnd(seqs * per + 1, page, G, D), rnd(seqs * per + 1, page, G, V)
+        pt = (torch.randperm(seqs * per, device=dev).view(seqs, per) + 1).to(torch.int32)
+        pos = torch.full((B,), ctx - 1, dtype=torch.int32, device=dev) if kind == "decode" else m.positions
+        talk = torch.randn(Hq, Hq, device=dev) * 0.2
+        q2 = rnd(n, Hq * D)
+        sl = torch.full((B,), ctx, dtype=torch.int32, device=dev)
+        seen = (size + keep) * B if kind == "decode" else sum(min(i + 1, size + min(keep, max(0, i + 1 - size))) for i in range(n))
+        byts = 2.0 * (B * (size + keep) if kind == "decode" else n) * G * (D + V)
+        case(f"head_mix_attention_{kind}", lambda: F.head_mix_attention(
+            q2, Hq, kc, vc, talk, m.cu, pos, pt, 0.088, size, keep, seq_lens=sl if kind == "decode" else None,
+            max_k=ctx),
+            byts, seen * Hq * 2.0 * (D + V + Hq))
+        if kind == "decode":
+            splits = F.decode_splits(B, G, size + keep)
+            sl2 = torch.full((B,), size + keep, dtype=torch.int32, device=dev)
+            case("paged_decode_attention (like)", lambda: F.paged_decode_attention(
+                q2.view(B, Hq, D), kc, vc, pt, sl2, 0.088, splits), byts)
+        else:
+            kk, vv = rnd(n, G, D), rnd(n, G, D)
+            case("flash_causal_prefill (like)", lambda: F_flash(q2.view(n, Hq, D), kk, vv, m.cu, n),
+                 None, 4.0 * Hq * D * n * n / 2)
+        xr = rnd(n, (Hq + 2 * G) * D)
+        wq, wk = rnd(Hq * D, dtype=torch.float32), rnd(G * D, dtype=torch.float32)
+        slots = torch.arange(n, dtype=torch.int32, device=dev) % (kc.shape[0] * page)
+        case(f"row_norm_kv_{kind}", lambda: F.row_norm_kv_(
+            xr, (0, Hq * D, (Hq + G) * D), (Hq * D, G * D, G * D), wq, wk, slots, kc, vc, 1e-6),
+            n * (2 * Hq * D + 4 * G * D) * 2.0)
+        inv = torch.rand(64, device=dev)
+        case(f"qk_norm_rope_kv_{kind} (like)", lambda: F.qk_norm_rope_kv_(
+            xr, nw[:D].contiguous(), nw[:D].contiguous(), pos, inv, slots, kc, vc, Hq, G, D),
+            n * (2 * Hq * D + 4 * G * D) * 2.0)
+
+
+def F_flash(q, k, v, cu, n):
+    from ..ops.flash import flash_attn_varlen
+    return flash_attn_varlen(q, k, v, cu, cu, n, n, 0.088, True)
+
+
+if __name__ == "__main__":
+    main()
