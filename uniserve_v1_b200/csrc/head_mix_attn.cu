@@ -458,6 +458,52 @@ __device__ __forceinline__ uint32_t swz(int r, int c) {
   return (uint32_t)(r * PIECES + (c ^ (r & 7))) * 16u;
 }
 
+// 16-byte piece of a head's weights that holds row q, keys 8 n .. 8 n + 7 (rows 4 apart take
+// opposite halves, so the eight rows of an accumulator store hit different banks; the mixture
+// works column by column and needs no order)
+__device__ __forceinline__ int ppiece(int q, int n) { return q * 2 + (n ^ ((q >> 2) & 1)); }
+
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+// Scores of a warp's HW heads for one step of 16 keys: S[16 rows][16 keys] per head, a lane's
+// columns in the two 8-key halves.  Keys are the instruction's columns (row lrow of the tile,
+// channel half lhalf); the query fragments come from registers (REG) or shared memory.
+template <int HW, int DC, bool REG>
+__device__ __forceinline__ void tile_scores(float (&sc)[HW][2][4], const uint32_t (&qf)[HW][DC / 2][4],
+                                            uint32_t sq, uint32_t kb, int g0, int H, int rep,
+                                            bool one_kv, int lrow, int lhalf) {
+  constexpr uint32_t kTileBytes = 16 * DC * 16;
+#pragma unroll
+  for (int i = 0; i < HW; ++i)
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) sc[i][n][e] = 0.f;
+#pragma unroll
+  for (int k = 0; k < DC / 2; ++k) {
+    const uint32_t off = swz<DC>(lrow, 2 * k + lhalf);
+    uint32_t bk[4];
+    if (one_kv) ldsm4(bk, kb + (uint32_t)(min(g0, H - 1) / rep) * kTileBytes + off);
+#pragma unroll
+    for (int i = 0; i < HW; ++i) {
+      if (!one_kv) ldsm4(bk, kb + (uint32_t)(min(g0 + i, H - 1) / rep) * kTileBytes + off);
+      if (REG) {
+        mma16816(sc[i][0], qf[i][k][0], qf[i][k][1], qf[i][k][2], qf[i][k][3], bk[0], bk[2]);
+        mma16816(sc[i][1], qf[i][k][0], qf[i][k][1], qf[i][k][2], qf[i][k][3], bk[1], bk[3]);
+      } else {
+        uint32_t aq[4];
+        ldsm4(aq, sq + (uint32_t)(g0 + i) * kTileBytes + off);
+        mma16816(sc[i][0], aq[0], aq[1], aq[2], aq[3], bk[0], bk[2]);
+        mma16816(sc[i][1], aq[0], aq[1], aq[2], aq[3], bk[1], bk[3]);
+      }
+    }
+  }
+}
+
 // HP: heads padded to 8, 16 or 32 (8 warps x HP / 8 heads); DP, VP: head widths padded to 64 or
 // 128.  blockIdx.x: query tile, blockIdx.y: group of 16 output heads.
 template <int HP, int DP, int VP>
@@ -514,67 +560,65 @@ __global__ void __launch_bounds__(kTileThreads, 1) head_mix_tile_kernel(const Ti
   if (kept >= lo) { kept = 0; lo = 0; }
   const int kt = (kept + kKeys - 1) / kKeys, steps = kt + (p1 - lo + kKeys) / kKeys;
   const int* pt = a.page_table + (long long)s * a.max_pages;
+  const int page_shift = (a.page & (a.page - 1)) == 0 ? __ffs(a.page) - 1 : -1;
+  auto slot_of = [&](int key) -> long long {
+    const int p = page_shift >= 0 ? key >> page_shift : key / a.page;
+    return (long long)pt[p] * a.page + (key - p * a.page);
+  };
   auto first_key = [&](int st) { return st < kt ? st * kKeys : lo + (st - kt) * kKeys; };
   auto end_key = [&](int st) { return st < kt ? kept : p1 + 1; };
+  // a thread fetches piece c of key row r for every (second, fourth) kv head
   auto load = [&](int st, int buf, bool values) {
     const int k0 = first_key(st), k1 = end_key(st);
-    for (int e = tid; e < a.G * kKeys * DC; e += kTileThreads) {
-      const int r = e / (a.G * DC), x = e - r * a.G * DC, u = x / DC, c = x & (DC - 1);
-      const int key = k0 + r;
-      const uint32_t dst = sk + buf * k_bytes + u * kKeys * DP * 2 + swz<DC>(r, c);
-      if (key < k1 && c * 8 < a.D)
-        cp16(dst, a.kc + (((long long)pt[key / a.page] * a.page + key % a.page) * a.G + u) * a.D + c * 8);
-      else
-        asm volatile("st.shared.v4.u32 [%0], {%1,%1,%1,%1};" ::"r"(dst), "r"(0) : "memory");
-    }
-    if (values)
-      for (int e = tid; e < u_n * kKeys * VC; e += kTileThreads) {
-        const int r = e / (u_n * VC), x = e - r * u_n * VC, u = x / VC, c = x & (VC - 1);
-        const int key = k0 + r;
-        const uint32_t dst = sv + buf * v_bytes + u * kKeys * VP * 2 + swz<VC>(r, c);
-        if (key < k1 && c * 8 < a.V)
-          cp16(dst, a.vc + (((long long)pt[key / a.page] * a.page + key % a.page) * a.G + u_lo + u) * a.V + c * 8);
-        else
-          asm volatile("st.shared.v4.u32 [%0], {%1,%1,%1,%1};" ::"r"(dst), "r"(0) : "memory");
+    {
+      const int c = tid & (DC - 1), r = (tid / DC) & (kKeys - 1), key = k0 + r;
+      constexpr int kStride = kTileThreads / (kKeys * DC);
+      uint32_t dst = sk + buf * k_bytes + swz<DC>(r, c) + (tid / (kKeys * DC)) * (kKeys * DP * 2);
+      const bool ok = key < k1 && c * 8 < a.D;
+      const __nv_bfloat16* src = a.kc;
+      if (ok) src += (slot_of(key) * a.G + tid / (kKeys * DC)) * a.D + c * 8;
+      for (int u = tid / (kKeys * DC); u < a.G; u += kStride) {
+        if (ok) cp16(dst, src);
+        else asm volatile("st.shared.v4.u32 [%0], {%1,%1,%1,%1};" ::"r"(dst), "r"(0) : "memory");
+        dst += kStride * kKeys * DP * 2;
+        src += kStride * a.D;
       }
+    }
+    if (values) {
+      const int c = tid & (VC - 1), r = (tid / VC) & (kKeys - 1), key = k0 + r;
+      constexpr int kStride = kTileThreads / (kKeys * VC);
+      uint32_t dst = sv + buf * v_bytes + swz<VC>(r, c) + (tid / (kKeys * VC)) * (kKeys * VP * 2);
+      const bool ok = key < k1 && c * 8 < a.V;
+      const __nv_bfloat16* src = a.vc;
+      if (ok) src += (slot_of(key) * a.G + u_lo + tid / (kKeys * VC)) * a.V + c * 8;
+      for (int u = tid / (kKeys * VC); u < u_n; u += kStride) {
+        if (ok) cp16(dst, src);
+        else asm volatile("st.shared.v4.u32 [%0], {%1,%1,%1,%1};" ::"r"(dst), "r"(0) : "memory");
+        dst += kStride * kKeys * VP * 2;
+        src += kStride * a.V;
+      }
+    }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   const int lrow = lane & 15, lhalf = lane >> 4;     // ldmatrix row / 8-column half of this lane
   const int r0 = lane >> 2, cq = (lane & 3) * 2;     // accumulator row and first column
-  // scores of the warp's heads for one step: S[16 rows][16 keys] per head, columns cq, cq + 1
-  // of the two 8-key halves
-  auto scores = [&](int buf, float (&sc)[HW][2][4]) {
+  const int g0 = warp * HW;
+  const bool one_kv = min(g0, a.H - 1) / rep == min(g0 + HW - 1, a.H - 1) / rep;
+  // bit n * 4 + e: row r0 (+8) of the tile sees the key behind accumulator element (n, e)
+  auto seen_bits = [&](int st) -> uint32_t {
+    const int k0 = first_key(st), k1 = end_key(st);
+    // a step every row sees whole: nothing to test
+    if (k0 + kKeys <= k1 && k0 + kKeys - 1 <= p0 &&
+        (a.size <= 0 || p0 + 15 - k0 < a.size || k0 + kKeys <= a.keep)) return 0xffu;
+    uint32_t bits = 0;
 #pragma unroll
-    for (int i = 0; i < HW; ++i)
+    for (int n = 0; n < 2; ++n)
 #pragma unroll
-      for (int n = 0; n < 2; ++n)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) sc[i][n][e] = 0.f;
-    const int g0 = warp * HW;
-#pragma unroll
-    for (int k = 0; k < DC / 2; ++k) {
-      int u_prev = -1;
-      uint32_t bk[4];
-#pragma unroll
-      for (int i = 0; i < HW; ++i) {
-        if (g0 + i >= a.H) break;
-        const int u = (g0 + i) / rep;
-        if (u != u_prev) {
-          // keys are the instruction's columns: rows lrow of the tile, channel halves
-          ldsm4(bk, sk + buf * k_bytes + u * kKeys * DP * 2 + swz<DC>(lrow, 2 * k + lhalf));
-          u_prev = u;
-        }
-        uint32_t aq[4];
-        ldsm4(aq, sq + (g0 + i) * 16 * DP * 2 + swz<DC>(lrow, 2 * k + lhalf));
-        mma16816(sc[i][0], aq[0], aq[1], aq[2], aq[3], bk[0], bk[2]);
-        mma16816(sc[i][1], aq[0], aq[1], aq[2], aq[3], bk[1], bk[3]);
+      for (int e = 0; e < 4; ++e) {
+        const int i = p0 + r0 + (e >> 1) * 8, j = k0 + n * 8 + cq + (e & 1);
+        if (j < k1 && j <= i && (a.size <= 0 || i - j < a.size || j < a.keep)) bits |= 1u << (n * 4 + e);
       }
-    }
-  };
-  // whether row r0 (+8) of the tile sees the key behind accumulator element (n, e)
-  auto sees = [&](int k0, int k1, int n, int e) {
-    const int i = p0 + r0 + (e >> 1) * 8, j = k0 + n * 8 + cq + (e & 1);
-    return j < k1 && j <= i && (a.size <= 0 || i - j < a.size || j < a.keep);
+    return bits;
   };
   // ---- first sweep: maximum and sum of every (row, head), in the log2 domain ----
   float mx[HW][2], sum[HW][2];
@@ -599,29 +643,39 @@ __global__ void __launch_bounds__(kTileThreads, 1) head_mix_tile_kernel(const Ti
     if (two && st + 1 < steps) load(st + 1, (st + 1) & 1, values);
     return two ? st & 1 : 0;
   };
-  for (int st = 0; st < steps; ++st) {
-    const int buf = next_step(st, false);
-    float sc[HW][2][4];
-    scores(buf, sc);
-    const int k0 = first_key(st), k1 = end_key(st);
+  {
+    uint32_t qf[HW][DC / 2][4];             // the queries stay in registers during this sweep
+    for (int st = 0; st < steps; ++st) {
+      const int buf = next_step(st, false);
+      if (st == 0) {
 #pragma unroll
-    for (int i = 0; i < HW; ++i)
+        for (int i = 0; i < HW; ++i)
 #pragma unroll
-      for (int r = 0; r < 2; ++r) {
-        float v[4], m = mx[i][r];
-#pragma unroll
-        for (int x = 0; x < 4; ++x) {
-          const int n = x >> 1, e = r * 2 + (x & 1);
-          v[x] = sees(k0, k1, n, e) ? sc[i][n][e] * a.scale_log2 : -INFINITY;
-          m = fmaxf(m, v[x]);
-        }
-        if (m == -INFINITY) continue;
-        float l = sum[i][r] * exp2f(mx[i][r] - m);
-#pragma unroll
-        for (int x = 0; x < 4; ++x) l += exp2f(v[x] - m);
-        sum[i][r] = l;
-        mx[i][r] = m;
+          for (int k = 0; k < DC / 2; ++k)
+            ldsm4(qf[i][k], sq + (g0 + i) * 16 * DP * 2 + swz<DC>(lrow, 2 * k + lhalf));
       }
+      float sc[HW][2][4];
+      tile_scores<HW, DC, true>(sc, qf, sq, sk + buf * k_bytes, g0, a.H, rep, one_kv, lrow, lhalf);
+      const uint32_t bits = seen_bits(st);
+#pragma unroll
+      for (int i = 0; i < HW; ++i)
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+          float v[4], m = mx[i][r];
+#pragma unroll
+          for (int x = 0; x < 4; ++x) {
+            const int n = x >> 1, e = r * 2 + (x & 1);
+            v[x] = (bits >> (n * 4 + e)) & 1u ? sc[i][n][e] * a.scale_log2 : -INFINITY;
+            m = fmaxf(m, v[x]);
+          }
+          const float base = m == -INFINITY ? 0.f : m;      // nothing seen yet: every term is zero
+          float l = sum[i][r] * ex2(mx[i][r] - base);
+#pragma unroll
+          for (int x = 0; x < 4; ++x) l += ex2(v[x] - base);
+          sum[i][r] = l;
+          mx[i][r] = m;
+        }
+    }
   }
 #pragma unroll
   for (int i = 0; i < HW; ++i)
@@ -632,7 +686,7 @@ __global__ void __launch_bounds__(kTileThreads, 1) head_mix_tile_kernel(const Ti
         const float m2 = __shfl_xor_sync(0xffffffffu, mx[i][r], o);
         const float l2 = __shfl_xor_sync(0xffffffffu, sum[i][r], o);
         const float m = fmaxf(mx[i][r], m2);
-        if (m != -INFINITY) sum[i][r] = sum[i][r] * exp2f(mx[i][r] - m) + l2 * exp2f(m2 - m);
+        if (m != -INFINITY) sum[i][r] = sum[i][r] * ex2(mx[i][r] - m) + l2 * ex2(m2 - m);
         mx[i][r] = m;
       }
       sum[i][r] = sum[i][r] > 0.f ? 1.f / sum[i][r] : 0.f;
@@ -659,20 +713,23 @@ __global__ void __launch_bounds__(kTileThreads, 1) head_mix_tile_kernel(const Ti
     const int buf = next_step(st, true);    // (the step before has read its mixed weights)
     {
       float sc[HW][2][4];
-      scores(buf, sc);
-      const int k0 = first_key(st), k1 = end_key(st);
+      uint32_t none[HW][DC / 2][4];
+      tile_scores<HW, DC, false>(sc, none, sq, sk + buf * k_bytes, g0, a.H, rep, one_kv, lrow, lhalf);
+      const uint32_t bits = seen_bits(st);
 #pragma unroll
       for (int i = 0; i < HW; ++i)
 #pragma unroll
         for (int n = 0; n < 2; ++n)
 #pragma unroll
           for (int r = 0; r < 2; ++r) {
-            const int g = warp * HW + i;
-            const float x = sees(k0, k1, n, r * 2) ? exp2f(sc[i][n][r * 2] * a.scale_log2 - mx[i][r]) * sum[i][r] : 0.f;
-            const float y = sees(k0, k1, n, r * 2 + 1) ? exp2f(sc[i][n][r * 2 + 1] * a.scale_log2 - mx[i][r]) * sum[i][r] : 0.f;
+            const int g = g0 + i, b0 = n * 4 + r * 2;
+            float x = ex2(sc[i][n][r * 2] * a.scale_log2 - mx[i][r]) * sum[i][r];
+            float y = ex2(sc[i][n][r * 2 + 1] * a.scale_log2 - mx[i][r]) * sum[i][r];
+            if (!((bits >> b0) & 1u) || g >= a.H) x = 0.f;
+            if (!((bits >> (b0 + 1)) & 1u) || g >= a.H) y = 0.f;
             uint32_t hi, low;
-            split_bf(g < a.H ? x : 0.f, g < a.H ? y : 0.f, hi, low);
-            const uint32_t dst = sp + g * kPRow + ((r0 + r * 8) * kKeys + n * 8 + cq) * 2;
+            split_bf(x, y, hi, low);
+            const uint32_t dst = sp + g * kPRow + ppiece(r0 + r * 8, n) * 16 + cq * 2;
             asm volatile("st.shared.u32 [%0], %1;" ::"r"(dst), "r"(hi) : "memory");
             asm volatile("st.shared.u32 [%0], %1;" ::"r"(dst + p_half), "r"(low) : "memory");
           }
@@ -716,8 +773,8 @@ __global__ void __launch_bounds__(kTileThreads, 1) head_mix_tile_kernel(const Ti
       const int h = warp * OW + i;
       if (h >= n_out) break;
       uint32_t wh[4], wl[4];
-      ldsm4(wh, sp + h * kPRow + (lrow * kKeys + lhalf * 8) * 2);
-      ldsm4(wl, sp + p_half + h * kPRow + (lrow * kKeys + lhalf * 8) * 2);
+      ldsm4(wh, sp + h * kPRow + ppiece(lrow, lhalf) * 16);
+      ldsm4(wl, sp + p_half + h * kPRow + ppiece(lrow, lhalf) * 16);
       const uint32_t vb = sv + buf * v_bytes + ((h_out0 + h) / rep - u_lo) * kKeys * VP * 2;
 #pragma unroll
       for (int n2 = 0; n2 < VC / 2; ++n2) {
