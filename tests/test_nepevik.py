@@ -487,7 +487,7 @@ def test_mixed_head_attention_alone(form, H, G, D, V, size, keep):
         k[0][j] = k[0][j] * 0.1 + pat * 3.0
     if form[1] == torch.bfloat16:
         q, k, v = ([t.bfloat16().float() for t in x] for x in (q, k, v))
-    talk = torch.eye(H) * 0.6 + rnd(g, H, H, std=0.5)
+    talk = (torch.eye(H) * 0.6 + rnd(g, H, H, std=0.5)).bfloat16().float()
     want = [P.mixed_head_attention(a, b, c, scale, win, keep, talk) for a, b, c in zip(q, k, v)]
     dev = form[0]
     kc, vc, pt = paged(k, v, 3, page, dev, form[1], g)

@@ -162,6 +162,41 @@ __device__ __forceinline__ void mma16816(float (&c)[4], uint32_t a0, uint32_t a1
       : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
 
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void cp16(uint32_t dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+}
+__device__ __forceinline__ uint32_t pack_bf(float a, float b) {
+  __nv_bfloat162 p = __floats2bfloat162_rn(a, b);
+  return *reinterpret_cast<uint32_t*>(&p);
+}
+// x = hi + lo with both halves bf16
+__device__ __forceinline__ void split_bf(float x, float y, uint32_t& hi, uint32_t& lo) {
+  const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
+  hi = *reinterpret_cast<const uint32_t*>(&h);
+  lo = pack_bf(x - us::bf2f(h.x), y - us::bf2f(h.y));
+}
+
+// byte offset of 16-byte piece c of row r in a tile whose rows hold `pieces` pieces (8 or 16):
+// pieces are XOR-swizzled by row so that 8 consecutive rows read 8 different bank groups
+template <int PIECES>
+__device__ __forceinline__ uint32_t swz(int r, int c) {
+  return (uint32_t)(r * PIECES + (c ^ (r & 7))) * 16u;
+}
+
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
 struct StepArgs {
   const __nv_bfloat16* q;
   const __nv_bfloat16 *kc, *vc;
@@ -188,6 +223,11 @@ __device__ __forceinline__ KeyList key_list(int pos, int size, int keep, int cap
 }
 
 constexpr int kStepThreads = 128;
+constexpr int kStepTile = 32;         // keys per step of the value product
+// keys of one split: whole tiles
+__host__ __device__ __forceinline__ int split_keys(int n, int splits) {
+  return ((n + splits - 1) / splits + kStepTile - 1) / kStepTile * kStepTile;
+}
 
 // Scores of one split's keys for the heads of one kv head.  A warp takes 8 keys per product: a
 // lane's 16-byte piece of a key row feeds two instructions, the queries' rows (at most 16 heads)
@@ -200,7 +240,7 @@ __global__ void __launch_bounds__(kStepThreads) head_mix_scores_kernel(const Ste
   if (a.seq_lens[b] <= 0) return;
   const int rep = a.H / a.G;
   const KeyList kl = key_list(a.pos[b], a.size, a.keep, a.cap);
-  const int per = (kl.n + a.splits - 1) / a.splits;
+  const int per = split_keys(kl.n, a.splits);
   const int k0 = min(kl.n, split * per), nk = min(kl.n, k0 + per) - k0;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int row = lane >> 2, kq = lane & 3;
@@ -215,17 +255,24 @@ __global__ void __launch_bounds__(kStepThreads) head_mix_scores_kernel(const Ste
   }
   const int* pt = a.page_table + (long long)b * a.max_pages;
   float* srow = a.scores + ((long long)b * a.H + (long long)u * rep) * a.cap;
-  for (int j0 = warp * 8; j0 < nk; j0 += kStepThreads / 4) {
-    const int x = min(k0 + j0 + row, kl.n - 1);
-    const int key = kl.key(x);
+  auto fetch = [&](int j0, uint4 (&kv)[kD8]) {
+    const int key = kl.key(min(k0 + j0 + row, kl.n - 1));
     const __nv_bfloat16* kr =
         a.kc + (((long long)pt[key / a.page] * a.page + key % a.page) * a.G + u) * a.D;
-    uint4 kv[kD8];
 #pragma unroll
     for (int i = 0; i < kD8; ++i) {
       const int d = (i * 4 + kq) * 8;
       kv[i] = d < a.D ? *reinterpret_cast<const uint4*>(kr + d) : make_uint4(0, 0, 0, 0);
     }
+  };
+  constexpr int kStride = kStepThreads / 4;      // 4 warps x 8 keys
+  uint4 ahead[kD8];
+  if (warp * 8 < nk) fetch(warp * 8, ahead);
+  for (int j0 = warp * 8; j0 < nk; j0 += kStride) {
+    uint4 kv[kD8];
+#pragma unroll
+    for (int i = 0; i < kD8; ++i) kv[i] = ahead[i];
+    if (j0 + kStride < nk) fetch(j0 + kStride, ahead);
     float c[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
     for (int i = 0; i < kD8; ++i) {
@@ -257,99 +304,166 @@ __global__ void __launch_bounds__(kStepThreads) head_mix_scores_kernel(const Ste
   }
 }
 
-constexpr int kStepTile = 32;
+constexpr int kWRow = kStepTile * 2 + 16;    // bytes of a head's 32 weights (bf16, padded)
 
-// Mixed weights and value product of one split's keys for the heads of one kv head.  Warp w
-// takes keys w, w + 4, ... of a tile, a lane VPL value columns of up to RM heads.
-template <int VPL, int RM>
+// Mixed weights and value product of one split's keys for the heads of one kv head, 32 keys a
+// step on warp-level tensor instructions.  Probabilities P [H][32] and mixed weights W [16][32]
+// are the sum of two bf16 values.  For the mixture a warp takes 8 keys, for the value product a
+// quarter of the value columns.  The next step's values (cp.async) and scores (registers) are on
+// their way while a step computes.  NK: 16-head steps of the mixture, VP: value width padded.
+template <int NK, int VP>
 __global__ void __launch_bounds__(kStepThreads) head_mix_apply_kernel(const StepArgs a) {
   US_PDL_PROLOGUE();
-  extern __shared__ __align__(16) float sm[];
+  constexpr int VC = VP / 8, HK = NK * 16, NP = HK / 8, NT = VP / 32;
+  extern __shared__ __align__(1024) uint8_t dsm[];
   const int split = blockIdx.x, u = blockIdx.y, b = blockIdx.z;
   const int rep = a.H / a.G, H = a.H;
-  float* mx = sm;                              // [H] maximum
-  float* inv = mx + H;                         // [H] 1 / sum
-  float* tk = inv + H;                         // [rep][H]
-  float* ps = tk + rep * H;                    // [H][kStepTile]
-  float* ws = ps + H * kStepTile;              // [kStepTile][RM]
-  float* os = ws + kStepTile * RM;             // [4 warps][rep][V]
-  __shared__ long long where[kStepTile];
+  const uint32_t sv = tc::smem_u32(dsm);                     // 2 x [32 keys][VC pieces]
+  constexpr uint32_t kVBytes = kStepTile * VP * 2;
+  const uint32_t sp = sv + 2 * kVBytes;                      // [2: hi, lo][HK][kWRow]
+  constexpr uint32_t kPHalf = HK * kWRow;
+  const uint32_t sw = sp + 2 * kPHalf;                       // [2][16][kWRow]
+  constexpr uint32_t kWHalf = 16 * kWRow;
+  float* os = reinterpret_cast<float*>(dsm + 2 * kVBytes + 2 * kPHalf + 2 * kWHalf);   // [rep][V]
+  __shared__ float mx[HK], inv[HK];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int lrow = lane & 15, lhalf = lane >> 4, r0 = lane >> 2, cq = (lane & 3) * 2;
   const bool live = a.seq_lens[b] > 0;         // the same in the whole cluster
-  float acc[RM][VPL];
+  float o[NT][4];
 #pragma unroll
-  for (int r = 0; r < RM; ++r)
+  for (int n = 0; n < NT; ++n)
 #pragma unroll
-    for (int i = 0; i < VPL; ++i) acc[r][i] = 0.f;
+    for (int e = 0; e < 4; ++e) o[n][e] = 0.f;
   if (live) {
     const KeyList kl = key_list(a.pos[b], a.size, a.keep, a.cap);
-    const int per = (kl.n + a.splits - 1) / a.splits;
+    const int per = split_keys(kl.n, a.splits);
     const int k0 = min(kl.n, split * per), k1 = min(kl.n, k0 + per);
     const int* pt = a.page_table + (long long)b * a.max_pages;
-    for (int g = tid; g < H; g += kStepThreads) {
-      const float* st = a.stats + ((long long)b * H + g) * a.splits * 2;
-      float m = -INFINITY, l = 0.f;
-      for (int s = 0; s < a.splits; ++s) m = fmaxf(m, st[2 * s]);
-      for (int s = 0; s < a.splits; ++s)
-        if (st[2 * s + 1] > 0.f) l += st[2 * s + 1] * expf(st[2 * s] - m);
-      mx[g] = m;
-      inv[g] = 1.f / l;
-    }
-    for (int e = tid; e < rep * H; e += kStepThreads) tk[e] = a.talk[(long long)u * rep * H + e];
     const float* srow = a.scores + (long long)b * H * a.cap;
-    for (int j0 = k0; j0 < k1; j0 += kStepTile) {
-      const int nj = min(kStepTile, k1 - j0);
-      __syncthreads();
-      if (tid < nj) {
-        const int key = kl.key(j0 + tid);
-        where[tid] = (long long)pt[key / a.page] * a.page + key % a.page;
-      }
-      for (int g = warp; g < H; g += kStepThreads / 32)
-        ps[g * kStepTile + lane] =
-            lane < nj ? expf(srow[(long long)g * a.cap + j0 + lane] - mx[g]) * inv[g] : 0.f;
-      __syncthreads();
-      for (int r = warp; r < RM; r += kStepThreads / 32) {
-        float w = 0.f;
-        if (r < rep)
-          for (int g = 0; g < H; ++g) w = fmaf(tk[r * H + g], ps[g * kStepTile + lane], w);
-        ws[lane * RM + r] = w;
-      }
-      __syncthreads();
-#pragma unroll 4
-      for (int j = warp; j < nj; j += kStepThreads / 32) {
-        const int c = lane * VPL;
-        float v[VPL];
+    const int kp = (tid & 15) * 2, pg = tid >> 4;            // this thread's key pair, first head
+    float2 ahead[NP];
+    auto fetch_scores = [&](int j0) {
 #pragma unroll
-        for (int i = 0; i < VPL; ++i) v[i] = 0.f;
-        if (c < a.V) {
-          const __nv_bfloat16* vr = a.vc + (where[j] * a.G + u) * a.V + c;
-          if (VPL == 4) {
-            us::Pack8 p;
-            p.u = *reinterpret_cast<const uint2*>(vr);
+      for (int i = 0; i < NP; ++i) {
+        const int g = pg + i * 8;
+        ahead[i] = (g < H && j0 + kp < k1)
+                       ? *reinterpret_cast<const float2*>(srow + (long long)g * a.cap + j0 + kp)
+                       : make_float2(-INFINITY, -INFINITY);
+      }
+    };
+    auto fetch_values = [&](int j0, int buf) {
+      constexpr int kRows = kStepThreads / VC;
+      const int c = tid & (VC - 1);
 #pragma unroll
-            for (int i = 0; i < VPL; ++i) v[i] = us::bf2f(p.b[i & 3]);
-          } else {
-            const __nv_bfloat162 p = *reinterpret_cast<const __nv_bfloat162*>(vr);
-            v[0] = us::bf2f(p.x);
-            v[1 % VPL] = us::bf2f(p.y);
-          }
+      for (int i = 0; i < kStepTile / kRows; ++i) {
+        const int r = tid / VC + i * kRows;
+        const uint32_t dst = sv + buf * kVBytes + swz<VC>(r, c);
+        if (j0 + r < k1 && c * 8 < a.V) {
+          const int key = kl.key(j0 + r), p = key / a.page;
+          cp16(dst, a.vc + (((long long)pt[p] * a.page + (key - p * a.page)) * a.G + u) * a.V + c * 8);
+        } else {
+          asm volatile("st.shared.v4.u32 [%0], {%1,%1,%1,%1};" ::"r"(dst), "r"(0) : "memory");
         }
-        const float* wr = ws + j * RM;
+      }
+      asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    if (k0 < k1) {
+      fetch_values(k0, 0);
+      fetch_scores(k0);
+    }
+    for (int g = tid; g < HK; g += kStepThreads) {
+      float m = -INFINITY, l = 0.f;
+      if (g < H) {
+        const float2* st = reinterpret_cast<const float2*>(a.stats) + ((long long)b * H + g) * a.splits;
+        float2 v[8];
 #pragma unroll
-        for (int r = 0; r < RM; ++r)
+        for (int s = 0; s < 8; ++s) v[s] = s < a.splits ? st[s] : make_float2(-INFINITY, 0.f);
 #pragma unroll
-          for (int i = 0; i < VPL; ++i) acc[r][i] = fmaf(wr[r], v[i], acc[r][i]);
+        for (int s = 0; s < 8; ++s) m = fmaxf(m, v[s].x);
+#pragma unroll
+        for (int s = 0; s < 8; ++s)
+          if (v[s].y > 0.f) l += v[s].y * expf(v[s].x - m);
+      }
+      mx[g] = g < H ? m : 0.f;
+      inv[g] = g < H ? 1.f / l : 0.f;
+    }
+    uint32_t tf[NK][4];                                       // T[u * rep + 0..15][g]
+#pragma unroll
+    for (int k = 0; k < NK; ++k)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int h = r0 + (e & 1) * 8, g = k * 16 + cq + (e >> 1) * 8;
+        const float* t = a.talk + (long long)(u * rep + h) * H + g;
+        tf[k][e] = pack_bf(h < rep && g < H ? t[0] : 0.f, h < rep && g + 1 < H ? t[1] : 0.f);
+      }
+    __syncthreads();
+    float mg[NP], ig[NP];
+#pragma unroll
+    for (int i = 0; i < NP; ++i) {
+      mg[i] = mx[pg + i * 8];
+      ig[i] = inv[pg + i * 8];
+    }
+    int buf = 0;
+    for (int j0 = k0; j0 < k1; j0 += kStepTile, buf ^= 1) {
+#pragma unroll
+      for (int i = 0; i < NP; ++i) {
+        const float x = expf(ahead[i].x - mg[i]) * ig[i];
+        const float y = j0 + kp + 1 < k1 ? expf(ahead[i].y - mg[i]) * ig[i] : 0.f;
+        uint32_t hi, low;
+        split_bf(x, y, hi, low);
+        const uint32_t dst = sp + (pg + i * 8) * kWRow + kp * 2;
+        asm volatile("st.shared.u32 [%0], %1;" ::"r"(dst), "r"(hi) : "memory");
+        asm volatile("st.shared.u32 [%0], %1;" ::"r"(dst + kPHalf), "r"(low) : "memory");
+      }
+      asm volatile("cp.async.wait_group 0;" ::: "memory");
+      __syncthreads();                         // P and this step's values; the other buffer is free
+      if (j0 + kStepTile < k1) {
+        fetch_values(j0 + kStepTile, buf ^ 1);
+        fetch_scores(j0 + kStepTile);
+      }
+      float w[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+      for (int k = 0; k < NK; ++k) {
+        uint32_t bp[4];                        // hi (first two) and lo of 16 heads x the warp's 8 keys
+        ldsm4t(bp, sp + lhalf * kPHalf + (k * 16 + lrow) * kWRow + warp * 16);
+        mma16816(w, tf[k][0], tf[k][1], tf[k][2], tf[k][3], bp[0], bp[1]);
+        mma16816(w, tf[k][0], tf[k][1], tf[k][2], tf[k][3], bp[2], bp[3]);
+      }
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        uint32_t hi, low;
+        split_bf(w[r * 2], w[r * 2 + 1], hi, low);
+        const uint32_t dst = sw + (r0 + r * 8) * kWRow + (warp * 8 + cq) * 2;
+        asm volatile("st.shared.u32 [%0], %1;" ::"r"(dst), "r"(hi) : "memory");
+        asm volatile("st.shared.u32 [%0], %1;" ::"r"(dst + kWHalf), "r"(low) : "memory");
+      }
+      __syncthreads();
+#pragma unroll
+      for (int k = 0; k < 2; ++k) {
+        uint32_t wh[4], wl[4];
+        ldsm4(wh, sw + lrow * kWRow + (k * 16 + lhalf * 8) * 2);
+        ldsm4(wl, sw + kWHalf + lrow * kWRow + (k * 16 + lhalf * 8) * 2);
+#pragma unroll
+        for (int n2 = 0; n2 < NT / 2; ++n2) {
+          uint32_t bv[4];
+          ldsm4t(bv, sv + buf * kVBytes + swz<VC>(k * 16 + lrow, warp * NT + 2 * n2 + lhalf));
+          mma16816(o[2 * n2], wh[0], wh[1], wh[2], wh[3], bv[0], bv[1]);
+          mma16816(o[2 * n2 + 1], wh[0], wh[1], wh[2], wh[3], bv[2], bv[3]);
+          mma16816(o[2 * n2], wl[0], wl[1], wl[2], wl[3], bv[0], bv[1]);
+          mma16816(o[2 * n2 + 1], wl[0], wl[1], wl[2], wl[3], bv[2], bv[3]);
+        }
       }
     }
   }
 #pragma unroll
-  for (int r = 0; r < RM; ++r)
+  for (int n = 0; n < NT; ++n)
 #pragma unroll
-    for (int i = 0; i < VPL; ++i)
-      if (r < rep && lane * VPL + i < a.V) os[(warp * rep + r) * a.V + lane * VPL + i] = acc[r][i];
+    for (int e = 0; e < 4; ++e) {
+      const int h = r0 + (e >> 1) * 8, c = (warp * NT + n) * 8 + cq + (e & 1);
+      if (h < rep && c < a.V) os[h * a.V + c] = o[n][e];
+    }
   __syncthreads();
   const int n = rep * a.V;
-  for (int e = tid; e < n; e += kStepThreads) os[e] = os[e] + os[n + e] + os[2 * n + e] + os[3 * n + e];
   if (a.splits > 1) tc::cluster_sync();
   // every CTA of the cluster finishes a share of the outputs, adding the splits in order
   for (int e = tid + split * kStepThreads; e < n; e += kStepThreads * a.splits) {
@@ -367,15 +481,14 @@ __global__ void __launch_bounds__(kStepThreads) head_mix_apply_kernel(const Step
   if (a.splits > 1) tc::cluster_sync();        // nobody leaves while its sums may still be read
 }
 
-template <int VPL, int RM>
+template <int NK, int VP>
 int launch_apply(const StepArgs& a, cudaStream_t stream) {
   const int rep = a.H / a.G;
-  const size_t smem = (size_t)(2 * a.H + rep * a.H + a.H * kStepTile + kStepTile * RM + 4 * rep * a.V) * 4;
-  if (smem > 200 * 1024) return US_ERR_LIMIT;
+  const size_t smem = 2 * kStepTile * VP * 2 + 2 * (NK * 16 + 16) * kWRow + (size_t)rep * a.V * 4;
   static bool configured = false;
   if (!configured) {
-    US_CUDA_CHECK(cudaFuncSetAttribute(head_mix_apply_kernel<VPL, RM>,
-                                       cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    US_CUDA_CHECK(cudaFuncSetAttribute(head_mix_apply_kernel<NK, VP>,
+                                       cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(48 * 1024)));
     configured = true;
   }
   cudaLaunchConfig_t cfg = {};
@@ -392,14 +505,14 @@ int launch_apply(const StepArgs& a, cudaStream_t stream) {
   attr[1].val.clusterDim.z = 1;
   cfg.attrs = attr;
   cfg.numAttrs = a.splits > 1 ? 2 : 1;
-  US_CUDA_CHECK(cudaLaunchKernelEx(&cfg, head_mix_apply_kernel<VPL, RM>, a));
+  US_CUDA_CHECK(cudaLaunchKernelEx(&cfg, head_mix_apply_kernel<NK, VP>, a));
   return US_OK;
 }
 
 template <int kD8>
 int launch_scores(const StepArgs& a, cudaStream_t stream) {
   const int rep = a.H / a.G;
-  const size_t smem = (size_t)rep * ((a.cap + a.splits - 1) / a.splits) * 4;
+  const size_t smem = (size_t)rep * split_keys(a.cap, a.splits) * 4;
   static bool configured = false;
   if (!configured) {
     US_CUDA_CHECK(cudaFuncSetAttribute(head_mix_scores_kernel<kD8>,
@@ -412,28 +525,6 @@ int launch_scores(const StepArgs& a, cudaStream_t stream) {
 }
 
 // ------------------------------------------------------------------- tiles --
-__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ void cp16(uint32_t dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
-}
-__device__ __forceinline__ uint32_t pack_bf(float a, float b) {
-  __nv_bfloat162 p = __floats2bfloat162_rn(a, b);
-  return *reinterpret_cast<uint32_t*>(&p);
-}
-// x = hi + lo with both halves bf16
-__device__ __forceinline__ void split_bf(float x, float y, uint32_t& hi, uint32_t& lo) {
-  const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
-  hi = *reinterpret_cast<const uint32_t*>(&h);
-  lo = pack_bf(x - us::bf2f(h.x), y - us::bf2f(h.y));
-}
-
 struct TileArgs {
   const __nv_bfloat16* q;
   const __nv_bfloat16 *kc, *vc;
@@ -451,23 +542,10 @@ constexpr int kKeys = 16;             // keys per step
 constexpr int kOutHeads = 16;         // output heads per CTA (the mixture's 16 rows)
 constexpr int kPRow = 16 * kKeys * 2 + 16;   // bytes of a head's probabilities (16 x 16 bf16, padded)
 
-// byte offset of 16-byte piece c of row r in a tile whose rows hold `pieces` pieces (8 or 16):
-// pieces are XOR-swizzled by row so that 8 consecutive rows read 8 different bank groups
-template <int PIECES>
-__device__ __forceinline__ uint32_t swz(int r, int c) {
-  return (uint32_t)(r * PIECES + (c ^ (r & 7))) * 16u;
-}
-
 // 16-byte piece of a head's weights that holds row q, keys 8 n .. 8 n + 7 (rows 4 apart take
 // opposite halves, so the eight rows of an accumulator store hit different banks; the mixture
 // works column by column and needs no order)
 __device__ __forceinline__ int ppiece(int q, int n) { return q * 2 + (n ^ ((q >> 2) & 1)); }
-
-__device__ __forceinline__ float ex2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
 
 // Scores of a warp's HW heads for one step of 16 keys: S[16 rows][16 keys] per head, a lane's
 // columns in the two 8-key halves.  Keys are the instruction's columns (row lrow of the tile,
@@ -851,8 +929,9 @@ US_API int us_head_mix_decode(const void* q, const void* kc, const void* vc, con
   US_REQUIRE(ldo >= (long long)H * V && ((uintptr_t)q % 16) == 0 && ((uintptr_t)kc % 16) == 0 &&
              ((uintptr_t)vc % 16) == 0 && (ldq % 8) == 0);
   const int rep = H / G;
-  if ((D % 8) || D > 256 || (V % 4) || V > 128 || rep > 16 || B > 65535) return US_ERR_UNSUPPORTED;
-  if ((long long)rep * ((cap + splits - 1) / splits) * 4 > 100 * 1024) return US_ERR_LIMIT;
+  if ((D % 8) || D > 256 || (V % 8) || V > 128 || rep > 16 || H > 64 || (cap % 2) || B > 65535)
+    return US_ERR_UNSUPPORTED;
+  if ((long long)rep * split_keys(cap, splits) * 4 > 100 * 1024) return US_ERR_LIMIT;
   StepArgs a{(const __nv_bfloat16*)q, (const __nv_bfloat16*)kc, (const __nv_bfloat16*)vc, talk,
              (__nv_bfloat16*)out, (float*)scratch, (float*)scratch + (long long)B * H * cap, pos,
              page_table, seq_lens, ldq, ldo, B, H, G, D, V, page, max_pages, size, keep, cap, splits,
@@ -861,9 +940,10 @@ US_API int us_head_mix_decode(const void* q, const void* kc, const void* vc, con
   int rc = D <= 64 ? launch_scores<2>(a, stream) : D <= 128 ? launch_scores<4>(a, stream)
                                                             : launch_scores<8>(a, stream);
   if (rc) return rc;
-#define US_HM(VPL) \
-  return rep <= 4 ? launch_apply<VPL, 4>(a, stream) : rep <= 8 ? launch_apply<VPL, 8>(a, stream) : launch_apply<VPL, 16>(a, stream);
-  if (V <= 64) { US_HM(2) }
+#define US_HM(NK) \
+  return V <= 64 ? launch_apply<NK, 64>(a, stream) : launch_apply<NK, 128>(a, stream);
+  if (H <= 16) { US_HM(1) }
+  if (H <= 32) { US_HM(2) }
   US_HM(4)
 #undef US_HM
 }

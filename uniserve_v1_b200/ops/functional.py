@@ -673,12 +673,12 @@ def tanh_cols_(x, off, n):
 
 def _mix_splits(B, H, G, cap):
     """Key splits of the decode form of head-mixed attention: enough CTAs for every SM, at least
-    64 keys each, scores of a split within shared memory (None: they never are)."""
-    rep = H // G
-    fit = -(-rep * cap * 4 // (100 * 1024))
-    want = max(1, min(-(-592 // (B * G)), cap // 64, 8))
-    splits = max(want, fit)
-    while splits <= 8 and rep * (-(-cap // splits)) * 4 > 100 * 1024:
+    64 keys each, the scores of a split (whole 32-key tiles) within shared memory (None: they
+    never are)."""
+    def fits(s):
+        return H // G * ((-(-cap // s) + 31) // 32 * 32) * 4 <= 100 * 1024
+    splits = max(1, min(-(-592 // (B * G)), cap // 64, 8))
+    while splits <= 8 and not fits(splits):
         splits += 1
     return splits if splits <= 8 else None
 
@@ -714,10 +714,11 @@ def head_mix_attention(q, H, kcache, vcache, talk, cu, positions, page_table, sc
         return out
     B, max_pages = cu.shape[0] - 1, page_table.shape[1]
     if q.dtype == BF16 and D % 8 == 0 and q.stride(0) % 8 == 0:
-        if seq_lens is not None and D <= 256 and V % 4 == 0 and V <= 128 and H // G <= 16:
+        if seq_lens is not None and D <= 256 and V % 8 == 0 and V <= 128 and H // G <= 16 and H <= 64:
             cap = max_k or page * max_pages
             if size > 0:
                 cap = min(cap, size + max(keep, 0))
+            cap += cap % 2
             splits = _mix_splits(B, H, G, cap)
             if splits is not None:
                 scratch = torch.empty(N.kernels().us_head_mix_decode_scratch(B, H, cap, splits),
