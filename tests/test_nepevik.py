@@ -370,7 +370,7 @@ def test_channel_delta_alone(form, H, Hk, D, V, K):
                       P.softplus(low[lo:hi] + w["dt_bias"]).view(-1, H, D))
         want.append(P.channel_delta_rule(q[:, of], k[:, of], v, d, P.sigmoid(x[lo:hi, 2 * nq + nv:])))
     dev, wd = form[0], {n: t.to(form[0]) for n, t in w.items()}
-    conv = torch.full((5, max(K - 1, 0), 2 * nq + nv), 9.0, device=dev, dtype=form[1])  # left-overs
+    conv = torch.full((5, K, 2 * nq + nv), 9.0, device=dev, dtype=form[1])  # left-overs
     S = torch.full((5, H, D, V), 7.0, device=dev)
     slots, done, got = [3, 0, 4], [0, 0, 0], [[], [], []]
     for step in ([5, 1, 0], [1, 1, 1], [7, 0, 6]):
@@ -398,7 +398,7 @@ def test_channel_delta_alone(form, H, Hk, D, V, K):
 
 
 @pytest.mark.parametrize("form", FORMS)
-@pytest.mark.parametrize("H,D", [(3, 12), (2, 64), (2, 100), (1, 136), (2, 32)])
+@pytest.mark.parametrize("H,D", [(3, 12), (2, 64), (2, 100), (1, 136), (2, 32), (3, 13)])
 def test_general_delta_alone(form, H, D):
     g = gen(D)
     T, n = 19, H * D
@@ -416,8 +416,7 @@ def test_general_delta_alone(form, H, D):
     for lo, hi in ((0, 9), (9, 10), (10, 12), (12, 19)):
         m = seq_meta([hi - lo], [lo], [1], dev)
         rows = xs[lo:hi]
-        d, nn, p = VD.general_prep(rows, (n, 4 * n), ls[lo:hi], wd, H, D)
-        rr, kk, vv = (rows[:, i * n:(i + 1) * n].unflatten(1, (H, D)) for i in (0, 1, 2))
+        d, nn, p, kk, rr, vv = VD.general_prep(rows, (0, n, 2 * n, 4 * n), ls[lo:hi], wd, H, D)
         got.append(VD.vector_delta_rule(rr, kk, vv, d, S, m, n=nn, p=p).cpu())
     close(torch.cat(got), want, torch.float32, "general rule", 4.0)
     settled(dev)

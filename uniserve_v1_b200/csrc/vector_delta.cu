@@ -17,12 +17,11 @@
 // starts from a zero state whatever its slot holds: slots are handed on without being cleared,
 // and nothing has to be launched when a request is admitted.  A negative slot marks padding.
 //
-// Rule kernel: a CTA owns 32 value columns of one head of one sequence.  Four warps compute:
-// a lane holds D/16 rows x 4 columns of S in registers (16 lanes span the rows, so one 16-byte
-// access per row moves 4 columns, and 4 independent chains hide the FMA latency); the two
-// D-long reductions of a token fold 4 columns over 16 lanes in five shuffles.  Four more warps
-// stage the vectors of the next tokens into the other half of shared memory meanwhile.  The
-// state crosses HBM once per call.
+// Rule kernel: a CTA owns 32 value columns of one head of one sequence.  A lane holds D/16 rows
+// x 4 columns of S in registers (16 lanes span the rows, so one 16-byte access per row moves 4
+// columns, and 4 independent chains hide the FMA latency); the two D-long reductions of a token
+// fold 4 columns over 16 lanes in five shuffles.  The vectors of the next 16 tokens are copied
+// into the other half of shared memory meanwhile.  The state crosses HBM once per call.
 #include "include/us_common.cuh"
 
 namespace {
@@ -66,14 +65,18 @@ struct ChannelPrep {
   const float* low;             // [rows, H * D]
   long long ldlow;
   const float *A_log, *dt_bias; // [H], [H * D]
-  void* conv;                   // [slots, K - 1, C], C = 2 Hk D + H V
+  void* conv;                   // [slots, K, C], C = 2 Hk D + H V: input of position p in entry p % K
   float *q, *k, *v, *g, *beta;  // [rows, Hk, D] x 2, [rows, H, V], [rows, H, D], [rows, H]
   const int *cu, *slots, *pos;
   int B, rows, H, Hk, D, V, K, bf16, one_token;
 };
 
+// The last inputs of a sequence's convolutions are a ring of K entries addressed by position:
+// a token reads K - 1 entries and writes another one, so nothing is shifted and the readers of
+// one token never meet its writer.  Positions before the sequence are zero.
+
 // A warp owns one head of q, of k, of v or of the decay for kPrepTokens rows (prefill) or one
-// row (every sequence brings one token: the warp then also shifts its channels' window).
+// row (every sequence brings one token: the warp then also stores its channels' inputs).
 __global__ void __launch_bounds__(256) channel_prep_kernel(const ChannelPrep a) {
   US_PDL_PROLOGUE();
   const int lane = threadIdx.x & 31;
@@ -115,8 +118,8 @@ __global__ void __launch_bounds__(256) channel_prep_kernel(const ChannelPrep a) 
     const int s = seq_of(a.cu, a.B, t);
     const int start = a.cu[s], slot = a.slots[s];
     if (slot < 0) continue;
-    const bool fresh = a.pos[start] == 0;
-    const long long sbase = (long long)slot * (a.K - 1) * C + cbase;
+    const int p0 = a.pos[start];
+    const long long sbase = (long long)slot * a.K * C + cbase;
     float y[kMaxDim / 32];
     float ss = 0.f;
 #pragma unroll
@@ -127,15 +130,13 @@ __global__ void __launch_bounds__(256) channel_prep_kernel(const ChannelPrep a) 
       float acc = 0.f;
       for (int j = 0; j < a.K; ++j) {
         const int src = t - (a.K - 1) + j;            // packed row of the tap
-        float xv;
-        if (src >= start)
-          xv = ld_any(a.x, (long long)src * a.ldx + off + d, a.bf16);
-        else
-          xv = fresh ? 0.f
-                     : ld_any(a.conv, sbase + (long long)(src - start + a.K - 1) * C + d, a.bf16);
+        const int sp = p0 + src - start;              // its position
+        float xv = 0.f;
+        if (src >= start) xv = ld_any(a.x, (long long)src * a.ldx + off + d, a.bf16);
+        else if (sp >= 0) xv = ld_any(a.conv, sbase + (long long)(sp % a.K) * C + d, a.bf16);
         acc += taps[(long long)d * a.K + j] * xv;
-        // one token per sequence: entry j of the old window becomes entry j - 1 of the new
-        if (a.one_token && j > 0) st_any(a.conv, sbase + (long long)(j - 1) * C + d, a.bf16, xv);
+        if (a.one_token && a.K > 1 && j == a.K - 1)
+          st_any(a.conv, sbase + (long long)(p0 % a.K) * C + d, a.bf16, xv);
       }
       y[i] = acc / (1.f + expf(-acc));
       ss += y[i] * y[i];
@@ -156,9 +157,8 @@ __global__ void __launch_bounds__(256) channel_prep_kernel(const ChannelPrep a) 
   }
 }
 
-// New window of every sequence: the last K - 1 rows of [old window; rows of this call].  A
-// thread owns one channel and walks the entries upwards, so each is read before it is written.
-__global__ void __launch_bounds__(256) conv_window_kernel(const ChannelPrep a) {
+// Inputs of every sequence's last K - 1 rows into its ring, after the rows' convolutions.
+__global__ void __launch_bounds__(256) conv_ring_kernel(const ChannelPrep a) {
   US_PDL_PROLOGUE();
   const int c = blockIdx.x * 256 + threadIdx.x;
   const int nq = a.Hk * a.D, C = 2 * nq + a.H * a.V;
@@ -166,26 +166,21 @@ __global__ void __launch_bounds__(256) conv_window_kernel(const ChannelPrep a) {
   const int s = blockIdx.y;
   const int start = a.cu[s], T = a.cu[s + 1] - start, slot = a.slots[s];
   if (slot < 0 || T <= 0) return;
-  const bool fresh = a.pos[start] == 0;
+  const int p0 = a.pos[start];
   const int col = c < nq ? a.off_q + c : c < 2 * nq ? a.off_k + c - nq : a.off_v + c - 2 * nq;
-  const long long base = (long long)slot * (a.K - 1) * C + c;
-  for (int j = 0; j < a.K - 1; ++j) {
-    const int src = T + j;
-    float v;
-    if (src < a.K - 1) v = fresh ? 0.f : ld_any(a.conv, base + (long long)src * C, a.bf16);
-    else v = ld_any(a.x, (long long)(start + src - (a.K - 1)) * a.ldx + col, a.bf16);
-    st_any(a.conv, base + (long long)j * C, a.bf16, v);
-  }
+  for (int t = max(0, T - (a.K - 1)); t < T; ++t)
+    st_any(a.conv, ((long long)slot * a.K + (p0 + t) % a.K) * C + c, a.bf16,
+           ld_any(a.x, (long long)(start + t) * a.ldx + col, a.bf16));
 }
 
 struct GeneralPrep {
   const void* x;
   long long ldx;
-  int off_k, off_a;
+  int off_r, off_k, off_v, off_a;
   const float* low;             // [rows, H * D] (before w0)
   long long ldlow;
   const float *w0, *a_bias;     // [H * D]
-  float *w, *n, *p;             // [rows, H, D]
+  float *w, *n, *p, *k, *r, *v;  // [rows, H, D]
   int rows, H, D, bf16;
   float rate;                   // w = exp(-rate * sigmoid(.))
 };
@@ -212,6 +207,9 @@ __global__ void __launch_bounds__(256) general_prep_kernel(const GeneralPrep a) 
     if (d >= a.D) continue;
     const int hd = h * a.D + d;
     const float n = kv[i] * inv;
+    a.k[r * a.D + d] = kv[i];
+    a.r[r * a.D + d] = ld_any(a.x, xr + a.off_r + d, a.bf16);
+    a.v[r * a.D + d] = ld_any(a.x, xr + a.off_v + d, a.bf16);
     a.w[r * a.D + d] =
         decay_exp(-a.rate * sigmoid_f(a.low[(long long)t * a.ldlow + hd] + a.w0[hd]));
     a.n[r * a.D + d] = n;
@@ -220,14 +218,10 @@ __global__ void __launch_bounds__(256) general_prep_kernel(const GeneralPrep a) 
 }
 
 constexpr int kCols = 32;         // value columns per CTA
-constexpr int kChunk = 8;         // tokens staged per round
-constexpr int kComputeThreads = 128;
+constexpr int kRuleThreads = 128;
 
 struct RuleArgs {
-  const void *q, *k, *v;          // element (t, h, i) at t * ld + h * hs + i
-  long long ldq, ldk, ldv;
-  int hsq, hsk, hsv;
-  int q_bf16, k_bf16, v_bf16;
+  const float *q, *k, *v;         // [rows, Hk, D] x 2, [rows, H, V]
   const float* g;                 // decay [rows, H, D]
   const float* n;                 // general: removal direction [rows, H, D]
   const float* p;                 // general: removal rate * direction [rows, H, D]
@@ -252,7 +246,6 @@ __device__ __forceinline__ float fold16(float c0, float c1, float c2, float c3, 
   return s;
 }
 
-
 template <int W>
 __device__ __forceinline__ void lds_vec(float (&o)[W], const float* p) {
   if (W == 4) {
@@ -266,61 +259,52 @@ __device__ __forceinline__ void lds_vec(float (&o)[W], const float* p) {
   }
 }
 
-// Vectors of token slot i in shared memory: kVecs rows of DP floats, then 32 columns of v.
+template <int BYTES>
+__device__ __forceinline__ void cp_async(float* dst, const float* src) {
+  const uint32_t d = (uint32_t)__cvta_generic_to_shared(dst);
+  if (BYTES == 16) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(d), "l"(src) : "memory");
+  else asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(d), "l"(src) : "memory");
+}
+
+// A token in shared memory: kVecs vectors of DP floats (g, k, q and, general, n, p), then 32
+// columns of v and beta.
 template <int DP, bool GENERAL>
 struct Stage {
-  static constexpr int kVecs = GENERAL ? 5 : 3;       // g, k, q (, n, p)
+  static constexpr int kVecs = GENERAL ? 5 : 3;
   static constexpr int kToken = kVecs * DP + kCols + 4;
+  static constexpr int kChunk = DP > 128 ? 8 : 16;    // tokens per round
   static constexpr int kFloats = kChunk * kToken;
 };
 
-template <int DP, bool GENERAL>
-__device__ __forceinline__ void stage_tokens(const RuleArgs& a, float* buf, int start, int c0, int n,
-                                             int h, int hk, int col0, int tid, int nthreads) {
+// Asynchronous copies of n tokens' vectors, U floats at a time.
+template <int DP, bool GENERAL, int U>
+__device__ __forceinline__ void stage_tokens(const RuleArgs& a, float* buf, long long row0, int n,
+                                             int h, int hk, int col0) {
   using St = Stage<DP, GENERAL>;
-  const bool quad = (a.D & 3) == 0;
-  if (quad && !a.q_bf16 && !a.k_bf16 && ((a.ldq | a.ldk | a.hsq | a.hsk) & 3) == 0) {
-    constexpr int kQ = DP / 4;
-    for (int e = tid; e < n * St::kVecs * kQ; e += nthreads) {
-      const int i = e / (St::kVecs * kQ), rest = e - i * St::kVecs * kQ;
-      const int vec = rest / kQ, d = (rest - vec * kQ) * 4;
-      const long long row = start + c0 + i;
-      float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (d < a.D) {
-        const float* src;
-        if (vec == 1) src = (const float*)a.k + row * a.ldk + (long long)hk * a.hsk + d;
-        else if (vec == 2) src = (const float*)a.q + row * a.ldq + (long long)hk * a.hsq + d;
-        else src = (vec == 0 ? a.g : vec == 3 ? a.n : a.p) + (row * a.H + h) * a.D + d;
-        x = *reinterpret_cast<const float4*>(src);
-      }
-      *reinterpret_cast<float4*>(buf + i * St::kToken + vec * DP + d) = x;
-    }
-  } else {
-    for (int e = tid; e < n * St::kVecs * DP; e += nthreads) {
-      const int i = e / (St::kVecs * DP), rest = e - i * St::kVecs * DP;
-      const int vec = rest / DP, d = rest - vec * DP;
-      const long long row = start + c0 + i;
-      float x = 0.f;
-      if (d < a.D) {
-        if (vec == 1) x = ld_any(a.k, row * a.ldk + (long long)hk * a.hsk + d, a.k_bf16);
-        else if (vec == 2) x = ld_any(a.q, row * a.ldq + (long long)hk * a.hsq + d, a.q_bf16);
-        else x = (vec == 0 ? a.g : vec == 3 ? a.n : a.p)[(row * a.H + h) * a.D + d];
-      }
-      buf[i * St::kToken + vec * DP + d] = x;
-    }
+  constexpr int kP = DP / U, kV = kCols / U;
+  for (int e = threadIdx.x; e < n * St::kVecs * kP; e += kRuleThreads) {
+    const int i = e / (St::kVecs * kP), rest = e - i * (St::kVecs * kP);
+    const int vec = rest / kP, d = (rest - vec * kP) * U;
+    if (d >= a.D) continue;
+    const long long row = row0 + i;
+    const float* src = vec == 1 ? a.k : vec == 2 ? a.q : vec == 0 ? a.g : vec == 3 ? a.n : a.p;
+    src += (vec == 1 || vec == 2 ? row * a.Hk + hk : row * a.H + h) * a.D + d;
+    cp_async<U * 4>(buf + i * St::kToken + vec * DP + d, src);
   }
-  for (int e = tid; e < n * (kCols + 1); e += nthreads) {
-    const int i = e / (kCols + 1), c = e - i * (kCols + 1);
-    const long long row = start + c0 + i;
-    float x = 0.f;
-    if (c == kCols) x = GENERAL ? 0.f : a.beta[row * a.H + h];
-    else if (col0 + c < a.V) x = ld_any(a.v, row * a.ldv + (long long)h * a.hsv + col0 + c, a.v_bf16);
-    buf[i * St::kToken + St::kVecs * DP + c] = x;
+  for (int e = threadIdx.x; e < n * kV; e += kRuleThreads) {
+    const int i = e / kV, c = (e - i * kV) * U;
+    if (col0 + c < a.V)
+      cp_async<U * 4>(buf + i * St::kToken + St::kVecs * DP + c,
+                      a.v + ((row0 + i) * a.H + h) * a.V + col0 + c);
   }
+  if (!GENERAL)
+    for (int i = threadIdx.x; i < n; i += kRuleThreads)
+      cp_async<4>(buf + i * St::kToken + St::kVecs * DP + kCols, a.beta + (row0 + i) * a.H + h);
+  asm volatile("cp.async.commit_group;" ::: "memory");
 }
 
 template <int DP, bool GENERAL>
-__global__ void __launch_bounds__(256) vector_delta_kernel(const RuleArgs a) {
+__global__ void __launch_bounds__(kRuleThreads) vector_delta_kernel(const RuleArgs a) {
   US_PDL_PROLOGUE();
   using St = Stage<DP, GENERAL>;
   constexpr int R = DP / 16;                          // rows per lane
@@ -334,139 +318,144 @@ __global__ void __launch_bounds__(256) vector_delta_kernel(const RuleArgs a) {
   const int start = a.cu[s], T = a.cu[s + 1] - start, slot = a.slots[s];
   if (T <= 0) return;
   if (slot < 0) {                                     // padding: defined rows, no state
-    for (int e = tid; e < T * kCols; e += 256) {
+    for (int e = tid; e < T * kCols; e += kRuleThreads) {
       const int t = e / kCols, c = col0 + e - t * kCols;
       if (c < a.V) a.out[((long long)(start + t) * a.H + h) * a.V + c] = 0.f;
     }
     return;
   }
-  const bool loader = warp >= kComputeThreads / 32;
   const int rl = lane & 15;
   const int my = ((lane >> 3) & 1) * 2 + ((lane >> 2) & 1);        // column a fold leaves here
-  const int cb = (warp & 3) * 8 + (lane >> 4) * 4;                 // first of the lane's columns
+  const int cb = warp * 8 + (lane >> 4) * 4;                       // first of the lane's columns
   float* Sg = a.state + (((long long)slot * a.H + h) * a.D) * a.V + col0 + cb;
-  const bool wide = (a.V & 3) == 0;
+  const bool wide = (a.V & 3) == 0, quad = wide && (a.D & 3) == 0;
+  const bool fresh = a.pos[start] == 0;
   float S[R][4];
-  if (loader) {
-    stage_tokens<DP, GENERAL>(a, sm, start, 0, min(kChunk, T), h, hk, col0, tid - kComputeThreads,
-                              256 - kComputeThreads);
-  } else {
-    const bool fresh = a.pos[start] == 0;
 #pragma unroll
-    for (int j = 0; j < NG; ++j)
+  for (int j = 0; j < NG; ++j)
 #pragma unroll
-      for (int e = 0; e < W; ++e) {
-        const int row = (j * 16 + rl) * W + e;
-        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (!fresh && row < a.D) {
-          const float* p = Sg + (long long)row * a.V;
-          if (wide) {
-            if (col0 + cb < a.V) x = *reinterpret_cast<const float4*>(p);
-          } else {
-            if (col0 + cb < a.V) x.x = p[0];
-            if (col0 + cb + 1 < a.V) x.y = p[1];
-            if (col0 + cb + 2 < a.V) x.z = p[2];
-            if (col0 + cb + 3 < a.V) x.w = p[3];
-          }
+    for (int e = 0; e < W; ++e) {
+      const int row = (j * 16 + rl) * W + e;
+      float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (!fresh && row < a.D) {
+        const float* p = Sg + (long long)row * a.V;
+        if (wide) {
+          if (col0 + cb < a.V) x = *reinterpret_cast<const float4*>(p);
+        } else {
+          if (col0 + cb < a.V) x.x = p[0];
+          if (col0 + cb + 1 < a.V) x.y = p[1];
+          if (col0 + cb + 2 < a.V) x.z = p[2];
+          if (col0 + cb + 3 < a.V) x.w = p[3];
         }
-        S[j * W + e][0] = x.x; S[j * W + e][1] = x.y; S[j * W + e][2] = x.z; S[j * W + e][3] = x.w;
       }
-  }
-  __syncthreads();
-  int buf = 0;
-  for (int c0 = 0; c0 < T; c0 += kChunk, buf ^= 1) {
-    const int n = min(kChunk, T - c0);
-    if (loader) {
-      if (c0 + kChunk < T)
-        stage_tokens<DP, GENERAL>(a, sm + (buf ^ 1) * St::kFloats, start, c0 + kChunk,
-                                  min(kChunk, T - c0 - kChunk), h, hk, col0, tid - kComputeThreads,
-                                  256 - kComputeThreads);
-    } else {
-      const float* base = sm + buf * St::kFloats;
-      for (int t = 0; t < n; ++t, base += St::kToken) {
-        const float* gs = base;
-        const float* ks = base + DP;
-        const float* qs = base + 2 * DP;
-        const float* vs = base + St::kVecs * DP;
-        float y0 = 0.f, y1 = 0.f, y2 = 0.f, y3 = 0.f;
-#pragma unroll
-        for (int j = 0; j < NG; ++j) {
-          const int r0 = (j * 16 + rl) * W;
-          float m[W];
-          if (GENERAL) {
-            lds_vec<W>(m, base + 3 * DP + r0);
-          } else {
-            float g[W];
-            lds_vec<W>(m, ks + r0);
-            lds_vec<W>(g, gs + r0);
-#pragma unroll
-            for (int e = 0; e < W; ++e) {
-              // the state is decayed first; what the key sees is the decayed state
-              S[j * W + e][0] *= g[e]; S[j * W + e][1] *= g[e];
-              S[j * W + e][2] *= g[e]; S[j * W + e][3] *= g[e];
-            }
-          }
-#pragma unroll
-          for (int e = 0; e < W; ++e) {
-            y0 = fmaf(S[j * W + e][0], m[e], y0);
-            y1 = fmaf(S[j * W + e][1], m[e], y1);
-            y2 = fmaf(S[j * W + e][2], m[e], y2);
-            y3 = fmaf(S[j * W + e][3], m[e], y3);
-          }
-        }
-        const float seen = fold16(y0, y1, y2, y3, lane);
-        float c = seen;                               // general: n^T S of this lane's column
-        if (!GENERAL) c = vs[kCols] * (vs[cb + my] - seen);
-        const int half = lane & 16;
-        const float u0 = __shfl_sync(0xffffffffu, c, half);
-        const float u1 = __shfl_sync(0xffffffffu, c, half | 4);
-        const float u2 = __shfl_sync(0xffffffffu, c, half | 8);
-        const float u3 = __shfl_sync(0xffffffffu, c, half | 12);
-        float4 vv;
-        if (GENERAL) vv = *reinterpret_cast<const float4*>(vs + cb);
-        float o0 = 0.f, o1 = 0.f, o2 = 0.f, o3 = 0.f;
-#pragma unroll
-        for (int j = 0; j < NG; ++j) {
-          const int r0 = (j * 16 + rl) * W;
-          float k[W], q[W];
-          lds_vec<W>(k, ks + r0);
-          lds_vec<W>(q, qs + r0);
-          if (GENERAL) {
-            float g[W], p[W];
-            lds_vec<W>(g, gs + r0);
-            lds_vec<W>(p, base + 4 * DP + r0);
-#pragma unroll
-            for (int e = 0; e < W; ++e) {
-              float* x = S[j * W + e];
-              x[0] = fmaf(k[e], vv.x, fmaf(-p[e], u0, g[e] * x[0]));
-              x[1] = fmaf(k[e], vv.y, fmaf(-p[e], u1, g[e] * x[1]));
-              x[2] = fmaf(k[e], vv.z, fmaf(-p[e], u2, g[e] * x[2]));
-              x[3] = fmaf(k[e], vv.w, fmaf(-p[e], u3, g[e] * x[3]));
-            }
-          } else {
-#pragma unroll
-            for (int e = 0; e < W; ++e) {
-              float* x = S[j * W + e];
-              x[0] = fmaf(k[e], u0, x[0]); x[1] = fmaf(k[e], u1, x[1]);
-              x[2] = fmaf(k[e], u2, x[2]); x[3] = fmaf(k[e], u3, x[3]);
-            }
-          }
-#pragma unroll
-          for (int e = 0; e < W; ++e) {
-            o0 = fmaf(S[j * W + e][0], q[e], o0);
-            o1 = fmaf(S[j * W + e][1], q[e], o1);
-            o2 = fmaf(S[j * W + e][2], q[e], o2);
-            o3 = fmaf(S[j * W + e][3], q[e], o3);
-          }
-        }
-        const float o = fold16(o0, o1, o2, o3, lane);
-        if ((lane & 3) == 0 && col0 + cb + my < a.V)
-          a.out[((long long)(start + c0 + t) * a.H + h) * a.V + col0 + cb + my] = o;
-      }
+      S[j * W + e][0] = x.x; S[j * W + e][1] = x.y; S[j * W + e][2] = x.z; S[j * W + e][3] = x.w;
     }
+  if (a.D < DP || col0 + kCols > a.V) {               // places that no copy fills
+    for (int e = tid; e < 2 * St::kFloats; e += kRuleThreads) sm[e] = 0.f;
     __syncthreads();
   }
-  if (loader) return;
+  auto stage = [&](int c0, int buf) {
+    float* dst = sm + buf * St::kFloats;
+    const int n = min(St::kChunk, T - c0);
+    if (quad) stage_tokens<DP, GENERAL, 4>(a, dst, start + c0, n, h, hk, col0);
+    else stage_tokens<DP, GENERAL, 1>(a, dst, start + c0, n, h, hk, col0);
+  };
+  stage(0, 0);
+  float* op = a.out + ((long long)start * a.H + h) * a.V + col0 + cb + my;
+  const bool writes = (lane & 3) == 0 && col0 + cb + my < a.V;
+  const long long ostep = (long long)a.H * a.V;
+  // the read-out of a token is folded beside the next token's first reduction: two independent
+  // shuffle chains instead of one after the other
+  float o0 = 0.f, o1 = 0.f, o2 = 0.f, o3 = 0.f;
+  bool pending = false;
+  int buf = 0;
+  for (int c0 = 0; c0 < T; c0 += St::kChunk, buf ^= 1) {
+    const int n = min(St::kChunk, T - c0);
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+    if (c0 + St::kChunk < T) stage(c0 + St::kChunk, buf ^ 1);
+    const float* base = sm + buf * St::kFloats;
+    for (int t = 0; t < n; ++t, base += St::kToken) {
+      const float* vs = base + St::kVecs * DP;
+      float y0 = 0.f, y1 = 0.f, y2 = 0.f, y3 = 0.f;
+#pragma unroll
+      for (int j = 0; j < NG; ++j) {
+        const int r0 = (j * 16 + rl) * W;
+        float m[W];
+        if (GENERAL) {
+          lds_vec<W>(m, base + 3 * DP + r0);
+        } else {
+          float g[W];
+          lds_vec<W>(m, base + DP + r0);
+          lds_vec<W>(g, base + r0);
+#pragma unroll
+          for (int e = 0; e < W; ++e) {
+            // the state is decayed first; what the key sees is the decayed state
+            float* x = S[j * W + e];
+            x[0] *= g[e]; x[1] *= g[e]; x[2] *= g[e]; x[3] *= g[e];
+          }
+        }
+#pragma unroll
+        for (int e = 0; e < W; ++e) {
+          const float* x = S[j * W + e];
+          y0 = fmaf(x[0], m[e], y0); y1 = fmaf(x[1], m[e], y1);
+          y2 = fmaf(x[2], m[e], y2); y3 = fmaf(x[3], m[e], y3);
+        }
+      }
+      const float seen = fold16(y0, y1, y2, y3, lane);
+      const float o = fold16(o0, o1, o2, o3, lane);
+      if (pending) {
+        if (writes) *op = o;
+        op += ostep;
+      }
+      pending = true;
+      float c = seen;                               // general: n^T S of this lane's column
+      if (!GENERAL) c = vs[kCols] * (vs[cb + my] - seen);
+      const int half = lane & 16;
+      const float u0 = __shfl_sync(0xffffffffu, c, half);
+      const float u1 = __shfl_sync(0xffffffffu, c, half | 4);
+      const float u2 = __shfl_sync(0xffffffffu, c, half | 8);
+      const float u3 = __shfl_sync(0xffffffffu, c, half | 12);
+      float4 vv;
+      if (GENERAL) vv = *reinterpret_cast<const float4*>(vs + cb);
+      o0 = o1 = o2 = o3 = 0.f;
+#pragma unroll
+      for (int j = 0; j < NG; ++j) {
+        const int r0 = (j * 16 + rl) * W;
+        float k[W], q[W];
+        lds_vec<W>(k, base + DP + r0);
+        lds_vec<W>(q, base + 2 * DP + r0);
+        if (GENERAL) {
+          float g[W], p[W];
+          lds_vec<W>(g, base + r0);
+          lds_vec<W>(p, base + 4 * DP + r0);
+#pragma unroll
+          for (int e = 0; e < W; ++e) {
+            float* x = S[j * W + e];
+            x[0] = fmaf(k[e], vv.x, fmaf(-p[e], u0, g[e] * x[0]));
+            x[1] = fmaf(k[e], vv.y, fmaf(-p[e], u1, g[e] * x[1]));
+            x[2] = fmaf(k[e], vv.z, fmaf(-p[e], u2, g[e] * x[2]));
+            x[3] = fmaf(k[e], vv.w, fmaf(-p[e], u3, g[e] * x[3]));
+          }
+        } else {
+#pragma unroll
+          for (int e = 0; e < W; ++e) {
+            float* x = S[j * W + e];
+            x[0] = fmaf(k[e], u0, x[0]); x[1] = fmaf(k[e], u1, x[1]);
+            x[2] = fmaf(k[e], u2, x[2]); x[3] = fmaf(k[e], u3, x[3]);
+          }
+        }
+#pragma unroll
+        for (int e = 0; e < W; ++e) {
+          const float* x = S[j * W + e];
+          o0 = fmaf(x[0], q[e], o0); o1 = fmaf(x[1], q[e], o1);
+          o2 = fmaf(x[2], q[e], o2); o3 = fmaf(x[3], q[e], o3);
+        }
+      }
+    }
+  }
+  const float o = fold16(o0, o1, o2, o3, lane);
+  if (writes) *op = o;
 #pragma unroll
   for (int j = 0; j < NG; ++j)
 #pragma unroll
@@ -519,7 +508,8 @@ int launch_rule(const RuleArgs& a, int B, cudaStream_t stream) {
   }
   configured = true;
   US_CUDA_CHECK(us::launch_pdl(vector_delta_kernel<DP, GENERAL>,
-                               dim3((a.V + kCols - 1) / kCols, a.H, B), dim3(256), smem, stream, a));
+                               dim3((a.V + kCols - 1) / kCols, a.H, B), dim3(kRuleThreads), smem,
+                               stream, a));
   return US_OK;
 }
 
@@ -548,37 +538,38 @@ US_API int us_channel_delta_prep(const void* x, long long ldx, int off_q, int of
   US_CUDA_CHECK(us::launch_pdl(channel_prep_kernel, dim3((rows + per - 1) / per, (units + 7) / 8),
                                dim3(256), 0, stream, a));
   if (!one_token && K > 1)
-    US_CUDA_CHECK(us::launch_pdl(conv_window_kernel, dim3((2 * Hk * D + H * V + 255) / 256, B),
+    US_CUDA_CHECK(us::launch_pdl(conv_ring_kernel, dim3((2 * Hk * D + H * V + 255) / 256, B),
                                  dim3(256), 0, stream, a));
   return US_OK;
 }
 
-US_API int us_general_delta_prep(const void* x, long long ldx, int off_k, int off_a,
-                                 const float* low, long long ldlow, const float* w0,
-                                 const float* a_bias, float* w, float* n, float* p, int rows, int H,
-                                 int D, float rate, int bf16, void* stream_) {
-  US_REQUIRE(x && low && w0 && a_bias && w && n && p && rows >= 1 && H >= 1);
+// out: six [rows, H, D] arrays one behind another: decay, unit key, removal, key, read-out, value.
+US_API int us_general_delta_prep(const void* x, long long ldx, int off_r, int off_k, int off_v,
+                                 int off_a, const float* low, long long ldlow, const float* w0,
+                                 const float* a_bias, float* out, int rows, int H, int D, float rate,
+                                 int bf16, void* stream_) {
+  US_REQUIRE(x && low && w0 && a_bias && out && rows >= 1 && H >= 1);
   if (D < 1 || D > kMaxDim) return US_ERR_UNSUPPORTED;
-  GeneralPrep a{x, ldx, off_k, off_a, low, ldlow, w0, a_bias, w, n, p, rows, H, D, bf16, rate};
-  const long long warps = (long long)rows * H;
+  const long long warps = (long long)rows * H, n = warps * D;
+  GeneralPrep a{x, ldx, off_r, off_k, off_v, off_a, low, ldlow, w0, a_bias, out, out + n, out + 2 * n,
+                out + 3 * n, out + 4 * n, out + 5 * n, rows, H, D, bf16, rate};
   US_CUDA_CHECK(us::launch_pdl(general_prep_kernel, dim3((unsigned)((warps + 7) / 8)), dim3(256), 0,
                                (cudaStream_t)stream_, a));
   return US_OK;
 }
 
 // general = 0: the channel rule (g, beta); 1: the general rule (g, n, p).  q and k heads serve
-// H / Hk value heads each.
-US_API int us_vector_delta_rule(int general, const void* q, const void* k, const void* v,
-                                long long ldq, long long ldk, long long ldv, int hsq, int hsk,
-                                int hsv, int q_bf16, int k_bf16, int v_bf16, const float* g,
-                                const float* n, const float* p, const float* beta, float* state,
-                                float* out, const int* cu, const int* slots, const int* pos, int B,
-                                int H, int Hk, int D, int V, void* stream_) {
+// H / Hk value heads each; all vectors dense FP32.
+US_API int us_vector_delta_rule(int general, const float* q, const float* k, const float* v,
+                                const float* g, const float* n, const float* p, const float* beta,
+                                float* state, float* out, const int* cu, const int* slots,
+                                const int* pos, int B, int H, int Hk, int D, int V, void* stream_) {
   US_REQUIRE(q && k && v && g && state && out && cu && slots && pos && B >= 1 && B <= 65535);
   US_REQUIRE(general ? (n && p) : (beta != nullptr));
   US_REQUIRE(H >= 1 && Hk >= 1 && H % Hk == 0 && H <= 65535 && D >= 1 && V >= 1);
-  RuleArgs a{q, k, v, ldq, ldk, ldv, hsq, hsk, hsv, q_bf16, k_bf16, v_bf16, g, n, p, beta, state,
-             out, cu, slots, pos, H, Hk, D, V};
+  US_REQUIRE((D & 3) || (V & 3) || (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)g | (uintptr_t)n |
+               (uintptr_t)p | (uintptr_t)state) % 16) == 0);
+  RuleArgs a{q, k, v, g, n, p, beta, state, out, cu, slots, pos, H, Hk, D, V};
   cudaStream_t stream = (cudaStream_t)stream_;
 #define US_VD(DP) \
   if (D <= DP) return general ? launch_rule<DP, true>(a, B, stream) : launch_rule<DP, false>(a, B, stream);

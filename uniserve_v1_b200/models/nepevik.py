@@ -336,7 +336,7 @@ class NepevikModel:
                    if s.kind == "attention" and s.kv_from is None)
 
     def new_state_pools(self, slots: int) -> list:
-        """Per layer (last convolution inputs [slots, K - 1, C] or None, S [slots, H, D, V])."""
+        """Per layer (ring of the last convolution inputs [slots, K, C] or None, S [slots, H, D, V])."""
         out = []
         for L in self.cfg.layers:
             s = L.mixer
@@ -345,7 +345,7 @@ class NepevikModel:
                 continue
             conv = None
             if s.kind == "channel_delta" and s.conv > 1:
-                conv = torch.zeros(slots, s.conv - 1,
+                conv = torch.zeros(slots, s.conv,
                                    2 * s.kv_heads * s.dim + s.heads * s.vdim, dtype=self.dtype,
                                    device=self.device)
             V = s.vdim if s.kind == "channel_delta" else s.dim
@@ -357,7 +357,8 @@ class NepevikModel:
         e, n = torch.empty(0, dtype=self.dtype).element_size(), 0
         for s in (L.mixer for L in self.cfg.layers):
             if s.kind == "channel_delta":
-                n += (s.conv - 1) * (2 * s.kv_heads * s.dim + s.heads * s.vdim) * e
+                if s.conv > 1:
+                    n += s.conv * (2 * s.kv_heads * s.dim + s.heads * s.vdim) * e
                 n += 4 * s.heads * s.dim * s.vdim
             elif s.kind == "general_delta":
                 n += 4 * s.heads * s.dim * s.dim
@@ -384,8 +385,7 @@ class NepevikModel:
         proj = F.linear(x, w["proj"])
         F.tanh_cols_(proj, ow, w["w2"].shape[1])
         low = F.linear(proj[:, ow:ow + w["w2"].shape[1]], w["w2"], out_dtype=torch.float32)
-        g, n, p = VD.general_prep(proj, (ok, oa), low[:, :H * D], w, H, D)
-        r, k, v = (proj[:, a:a + H * D].unflatten(1, (H, D)) for a in (orr, ok, ov))
+        g, n, p, k, r, v = VD.general_prep(proj, (orr, ok, ov, oa), low[:, :H * D], w, H, D)
         o = VD.vector_delta_rule(r, k, v, g, S, m, n=n, p=p)
         y = VD.head_norm_gate(o, w["norm"], proj[:, og:og + H * D], self.cfg.eps, w["o"].shape[1],
                               x.dtype)

@@ -43,9 +43,8 @@ _SIGNATURES = {
     "us_gemm_f32": (I, [P, P, P, I, I, I, I, I, L, L, L, I, P, P, P, P, P, I, P]),
     "us_channel_delta_prep": (I, [P, L, I, I, I, I, P, P, P, P, L, P, P, P, P, P, P, P, P, P, P, P,
                                   I, I, I, I, I, I, I, I, I, P]),
-    "us_general_delta_prep": (I, [P, L, I, I, P, L, P, P, P, P, P, I, I, I, F, I, P]),
-    "us_vector_delta_rule": (I, [I, P, P, P, L, L, L, I, I, I, I, I, I, P, P, P, P, P, P, P, P, P,
-                                 I, I, I, I, I, P]),
+    "us_general_delta_prep": (I, [P, L, I, I, I, I, P, L, P, P, P, I, I, I, F, I, P]),
+    "us_vector_delta_rule": (I, [I, P, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, P]),
     "us_head_norm_gate": (I, [P, P, I, P, L, P, L, I, I, I, F, I, I, P]),
     "us_embed_rows": (I, [P, P, P, P, I, I, I, I, P]),
     "us_output_norm_add": (I, [P, P, P, F, I, P, P, P, P, F, F, I, I, I, I, F, I, P]),

@@ -45,8 +45,9 @@ def _unit(x):
 def channel_prep(x, offs, low, w, conv, m: SeqMeta, H, Hk, D, V):
     """Projection rows ``x`` (q, k, v and the step size at columns ``offs``) and the decay's
     low-rank rows ``low`` [T, H * D] (FP32) to what the rule reads: unit q (scaled) and k
-    [T, Hk, D], v [T, H, V], decay g [T, H, D], beta [T, H], all FP32.  ``conv`` [slots, K - 1, C]
-    holds the last inputs of the short convolutions and is advanced."""
+    [T, Hk, D], v [T, H, V], decay g [T, H, D], beta [T, H], all FP32.  ``conv`` [slots, K, C]
+    holds the last inputs of the short convolutions, the input of position p in entry p % K, and
+    is advanced."""
     oq, ok, ov, ob = offs
     T, K, dev = x.shape[0], w["conv_q"].shape[1], x.device
     if x.is_cuda:
@@ -65,12 +66,15 @@ def channel_prep(x, offs, low, w, conv, m: SeqMeta, H, Hk, D, V):
     taps = torch.cat([w["conv_q"], w["conv_k"], w["conv_v"]], 0)
     cols = torch.cat([x[:, oq:oq + nq], x[:, ok:ok + nq], x[:, ov:ov + nv]], 1)
     y = torch.zeros(T, 2 * nq + nv)
-    for lo, hi, slot, fresh in _spans(m):
-        old = cols[:0] if K == 1 else torch.zeros_like(conv[slot]) if fresh else conv[slot]
+    for lo, hi, slot, _ in _spans(m):
+        p0 = int(m.positions[lo])
+        old = cols.new_zeros(K - 1, cols.shape[1])
+        for j in range(min(K - 1, p0)):
+            old[K - 2 - j] = conv[slot, (p0 - 1 - j) % K]
         full = torch.cat([old, cols[lo:hi]], 0)
         y[lo:hi] = (full.float().unfold(0, K, 1) * taps[None]).sum(-1)
-        if K > 1:
-            conv[slot] = full[-(K - 1):]
+        for t in range(max(lo, hi - (K - 1)), hi):
+            conv[slot, (p0 + t - lo) % K] = cols[t]
     y = torch.nn.functional.silu(y)
     q = _unit(y[:, :nq].view(T, Hk, D)) * D ** -0.5
     k = _unit(y[:, nq:2 * nq].view(T, Hk, D))
@@ -80,39 +84,38 @@ def channel_prep(x, offs, low, w, conv, m: SeqMeta, H, Hk, D, V):
 
 
 def general_prep(x, offs, low, w, H, D):
-    """Decay w, unit key n and removal a * n of the general rule, [T, H, D] FP32 each; ``offs``
-    are the columns of k and of the removal rate, ``low`` the decay's low-rank rows (FP32)."""
-    ok, oa = offs
+    """What the general rule reads, [T, H, D] FP32 each: decay w, unit key n, removal a * n, key k,
+    read-out r, value v.  ``offs`` are the columns of r, k, v and the removal rate in the
+    projection rows, ``low`` the decay's low-rank rows (FP32)."""
+    orr, ok, ov, oa = offs
     T = x.shape[0]
     if x.is_cuda:
-        out = torch.empty(3, T, H, D, dtype=torch.float32, device=x.device)
-        N.call("us_general_delta_prep", N.ptr(x), x.stride(0), ok, oa, N.ptr(low), low.stride(0),
-               N.ptr(w["w0"]), N.ptr(w["a_bias"]), N.ptr(out[0]), N.ptr(out[1]), N.ptr(out[2]), T, H,
-               D, GENERAL_DECAY_RATE, int(x.dtype == BF16), N.stream())
-        return out[0], out[1], out[2]
-    n = _unit(x[:, ok:ok + H * D].float().view(T, H, D))
+        out = torch.empty(6, T, H, D, dtype=torch.float32, device=x.device)
+        N.call("us_general_delta_prep", N.ptr(x), x.stride(0), orr, ok, ov, oa, N.ptr(low),
+               low.stride(0), N.ptr(w["w0"]), N.ptr(w["a_bias"]), N.ptr(out), T, H, D,
+               GENERAL_DECAY_RATE, int(x.dtype == BF16), N.stream())
+        return tuple(out)
+    r, k, v = (x[:, o:o + H * D].float().view(T, H, D) for o in (orr, ok, ov))
+    n = _unit(k)
     a = torch.sigmoid(x[:, oa:oa + H * D].float() + w["a_bias"]).view(T, H, D)
-    return torch.exp(-GENERAL_DECAY_RATE * torch.sigmoid(low + w["w0"])).view(T, H, D), n, a * n
+    return torch.exp(-GENERAL_DECAY_RATE * torch.sigmoid(low + w["w0"])).view(T, H, D), n, a * n, k, r, v
 
 
 def vector_delta_rule(q, k, v, g, state, m: SeqMeta, beta=None, n=None, p=None):
-    """The recurrence.  q, k [T, Hk, D] and v [T, H, V] may be strided views (last dimension
-    dense, bf16 or FP32), g / n / p [T, H, D] and beta [T, H] are FP32; ``beta`` selects the
-    channel rule, ``n`` and ``p`` the general one.  ``state`` [slots, H, D, V] FP32 is updated
-    in place.  Returns o [T, H, V] FP32."""
+    """The recurrence.  q, k [T, Hk, D], v [T, H, V], g / n / p [T, H, D] and beta [T, H] are dense
+    FP32; ``beta`` selects the channel rule, ``n`` and ``p`` the general one.  ``state``
+    [slots, H, D, V] FP32 is updated in place.  Returns o [T, H, V] FP32."""
     T, H, D = g.shape
     Hk, V = q.shape[1], v.shape[2]
     general = beta is None
     if q.is_cuda:
-        assert state.dtype == torch.float32 and state.is_contiguous() and g.is_contiguous()
+        for t in (q, k, v, g, state):
+            assert t.dtype == torch.float32 and t.is_contiguous()
         out = torch.empty(T, H, V, dtype=torch.float32, device=q.device)
-        b = [int(t.dtype == BF16) for t in (q, k, v)]
-        N.call("us_vector_delta_rule", int(general), N.ptr(q), N.ptr(k), N.ptr(v), q.stride(0),
-               k.stride(0), v.stride(0), q.stride(1), k.stride(1), v.stride(1), *b, N.ptr(g),
-               N.ptr(n), N.ptr(p), N.ptr(beta), N.ptr(state), N.ptr(out), N.ptr(m.cu),
-               N.ptr(m.slots), N.ptr(m.positions), m.slots.shape[0], H, Hk, D, V, N.stream())
+        N.call("us_vector_delta_rule", int(general), N.ptr(q), N.ptr(k), N.ptr(v), N.ptr(g), N.ptr(n),
+               N.ptr(p), N.ptr(beta), N.ptr(state), N.ptr(out), N.ptr(m.cu), N.ptr(m.slots),
+               N.ptr(m.positions), m.slots.shape[0], H, Hk, D, V, N.stream())
         return out
-    q, k, v = (t.float() for t in (q, k, v))
     q, k = (t.repeat_interleave(H // Hk, 1) for t in (q, k))
     out = torch.zeros(T, H, V)
     for lo, hi, slot, fresh in _spans(m):

@@ -74,12 +74,12 @@ def main():
              state + vec)
         D2 = 64
         pool2 = pool.view(-1)[:B * H * D2 * D2].view(B, H, D2, D2)
-        r2, k2, v2 = rnd(n, H, D2), rnd(n, H, D2), rnd(n, H, D2)
-        u2 = k2.float() / k2.float().norm(dim=-1, keepdim=True)
+        r2, k2, v2 = (rnd(n, H, D2, dtype=torch.float32) for _ in range(3))
+        u2 = k2 / k2.norm(dim=-1, keepdim=True)
         g2, p2 = torch.rand(n, H, D2, device=dev) * 0.1 + 0.9, u2 * 0.5
-        k2 = (k2.float() * 0.1).to(bf)
+        k2 = k2 * 0.1
         case(f"general_rule_{kind}", lambda: VD.vector_delta_rule(r2, k2, v2, g2, pool2, m, n=u2, p=p2),
-             2.0 * (B if kind == "decode" else 1) * H * D2 * D2 * 4 + n * H * D2 * (3 * 4 + 3 * 2 + 4.0))
+             2.0 * (B if kind == "decode" else 1) * H * D2 * D2 * 4 + n * H * D2 * 7 * 4.0)
         qb, kb, vb = rnd(n, Hk, D), rnd(n, Hk, D), rnd(n, H, V)
         ar, br, A, dtb = rnd(n, H), rnd(n, H), -torch.rand(H, device=dev) - 0.2, torch.rand(H, device=dev)
         case(f"gated_rule_{kind} (like)", lambda: GD.gated_delta_rule_packed(
@@ -92,16 +92,16 @@ def main():
              "conv_v": rnd(H * V, K, dtype=torch.float32), "A_log": rnd(H, dtype=torch.float32),
              "dt_bias": rnd(H * D, dtype=torch.float32), "w0": rnd(H * D2, dtype=torch.float32),
              "a_bias": rnd(H * D2, dtype=torch.float32)}
-        conv = torch.zeros(B, K - 1, C, dtype=bf, device=dev)
+        conv = torch.zeros(B, K, C, dtype=bf, device=dev)
         case(f"channel_prep_{kind}", lambda: VD.channel_prep(x, (0, Hk * D, 2 * Hk * D, C), low, w, conv, m, H, Hk, D, V),
              n * (2.0 * C + 4 * H * D) + vec - n * H * V * 4.0 + (2 * B * (K - 1) * C * 2.0 if kind == "decode" else 0))
-        xc = rnd(n, C)
+        xc, conv3 = rnd(n, C), torch.zeros(B, K - 1, C, dtype=bf, device=dev)
         wc = rnd(C, K, dtype=torch.float32)
-        case(f"causal_conv1d_{kind} (like)", lambda: GD.causal_conv1d(xc, wc, conv, cu=m.cu, slots=m.slots),
+        case(f"causal_conv1d_{kind} (like)", lambda: GD.causal_conv1d(xc, wc, conv3, cu=m.cu, slots=m.slots),
              4.0 * n * C + (2 * B * (K - 1) * C * 2.0 if kind == "decode" else 0))
         xg, lowg = rnd(n, 5 * H * D2), rnd(n, H * D2, dtype=torch.float32)
-        case(f"general_prep_{kind}", lambda: VD.general_prep(xg, (H * D2, 4 * H * D2), lowg, w, H, D2),
-             n * H * D2 * (2 * 2 + 4 + 12.0))
+        case(f"general_prep_{kind}", lambda: VD.general_prep(
+            xg, (0, H * D2, 2 * H * D2, 4 * H * D2), lowg, w, H, D2), n * H * D2 * (4 * 2 + 4 + 24.0))
         o, gate, hw = rnd(n, H, V, dtype=torch.float32), rnd(n, H * V), rnd(V, dtype=torch.float32)
         case(f"head_norm_gate_{kind}", lambda: VD.head_norm_gate(o, hw, gate, 1e-6, H * V, bf), n * H * V * 8.0)
         zz = gate.view(n, H, V)
