@@ -436,6 +436,48 @@ def test_head_norm_gate_alone(form, shared):
     settled(form[0])
 
 
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16], ids=["f32", "bf16"])
+@pytest.mark.parametrize("H,Hk,D,V,K", [(4, 2, 128, 128, 4), (2, 1, 64, 256, 2), (3, 3, 16, 8, 1),
+                                        (6, 2, 100, 68, 8)])
+def test_one_launch_decode_step_equals_the_separate_kernels(H, Hk, D, V, K, dtype):
+    """Tokens of several sequences at different positions (one of them fresh, one row padding)."""
+    g, dev, eps = gen(D), "cuda", 1e-4
+    nq, nv, B = Hk * D, H * V, 5
+    w = {"conv_q": rnd(g, nq, K), "conv_k": rnd(g, nq, K), "conv_v": rnd(g, nv, K),
+         "A_log": rnd(g, H, std=0.5), "dt_bias": rnd(g, H * D), "norm": rnd(g, V) + 1.0}
+    gw = {"w0": rnd(g, H * D) - 2.0, "a_bias": rnd(g, H * D), "norm": rnd(g, H * D) + 1.0}
+    w, gw = ({n: t.to(dev) for n, t in d.items()} for d in (w, gw))
+    slots, starts = [2, 5, -1, 0, 3], [0, 7, 0, 1, 300]
+    pools = [(rnd(g, 6, K, 2 * nq + nv).to(dev, dtype), rnd(g, 6, H, D, V).to(dev), rnd(g, 6, H, D, D).to(dev))] * 2
+    pools = [tuple(t.clone() for t in p) for p in pools]
+    for step in range(3):
+        m = seq_meta([1] * B, [s + step for s in starts], slots, dev)
+        x, low = rnd(g, B, 2 * nq + nv + H).to(dev, dtype), rnd(g, B, H * D).to(dev)
+        gate = rnd(g, B, H * V).to(dev, dtype)
+        offs = (0, nq, 2 * nq, 2 * nq + nv)
+        conv, S, S2 = pools[0]
+        got = VD.channel_step(x, offs, low, w, conv, S, gate, m, H, Hk, D, V, eps)
+        conv, S, _ = pools[1]
+        q, k, v, d, b = VD.channel_prep(x, offs, low, w, conv, m, H, Hk, D, V)
+        o = VD.vector_delta_rule(q, k, v, d, S, m, beta=b)
+        want = VD.head_norm_gate(o, w["norm"], gate, eps, H * V, dtype)
+        live = [0, 1, 3, 4]
+        close(got[live], want[live], dtype, f"channel step {step}")
+        assert float(got[2].float().abs().max()) == 0.0
+        if VD.step_fits(H, D, D, H * D):
+            x, gate = rnd(g, B, 5 * H * D, std=0.7).to(dev, dtype), rnd(g, B, H * D).to(dev, dtype)
+            offs = (0, H * D, 2 * H * D, 4 * H * D)
+            got = VD.general_step(x, offs, low, gw, S2, gate, m, H, D, eps)
+            d, n, p, k, r, v = VD.general_prep(x, offs, low, gw, H, D)
+            o = VD.vector_delta_rule(r, k, v, d, pools[1][2], m, n=n, p=p)
+            want = VD.head_norm_gate(o, gw["norm"], gate, eps, H * D, dtype)
+            close(got[live], want[live], dtype, f"general step {step}")
+    for a, b in zip(*pools):
+        close(a.flatten(1), b.flatten(1), torch.float32, "pools", 2.0)
+    settled(dev)
+
+
 def paged(k, v, starts_free, page, dev, dtype, g):
     """Pages (shuffled, with noise in the unused rows) holding k / v [n, G, D] of each sequence;
     returns (key pages, value pages, page table)."""

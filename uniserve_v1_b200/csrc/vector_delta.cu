@@ -11,6 +11,7 @@
 //   us_general_delta_prep   decay w = exp(-c sigmoid(low + w0)), unit key n, removal a * n
 //   us_vector_delta_rule    the recurrence
 //   us_head_norm_gate       per-head RMS norm of o, weight, sigmoid gate
+//   us_{channel,general}_delta_step   all of these for one token of every sequence in one launch
 //
 // The preparation is parallel over tokens, so the recurrence reads finished FP32 vectors and
 // does nothing but its multiply-adds.  A sequence whose first packed row stands at position 0
@@ -498,6 +499,208 @@ head_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ w, 
       st_any(y, (long long)t * ldy + c, bf16, 0.f);
 }
 
+// ------------------------------------------------------------- decode step --
+struct StepArgs {
+  const void* x;                  // projection rows
+  long long ldx;
+  int off_q, off_k, off_v, off_b; // general: read-out, key, value, removal rate
+  const float *cq, *ck, *cv;      // channel: taps
+  const float* low;               // [B, H * D]
+  long long ldlow;
+  const float *A_log, *bias;      // channel: [H], dt_bias [H * D]; general: null, w0 [H * D]
+  const float* a_bias;            // general: [H * D]
+  void* conv;                     // channel: ring [slots, K, C]
+  float* state;                   // [slots, H, D, V]
+  const float* nw;                // norm weight
+  int nw_head_stride;
+  const void* gate;               // [B, H * V] at ldg
+  long long ldg;
+  void* y;                        // [B, ldy]
+  long long ldy;
+  const int *slots, *pos;
+  int H, Hk, D, V, K, bf16, gate_bf16;
+  float eps, rate;
+};
+
+constexpr int kStepThreads = 256;
+
+// One token of every sequence through a whole mixer between its input and output projections:
+// convolutions (channel) or key norm (general), decay, recurrence, per-head norm and gate.  A CTA
+// owns one head of one sequence.  A thread holds R rows x 4 columns of S, a warp reading whole
+// rows; the state is on its way while the vectors are formed in shared memory.  LQ threads span
+// the value columns.  Sums over key channels meet in shared memory.
+template <int R, int LQ, bool GENERAL>
+__global__ void __launch_bounds__(kStepThreads) vector_delta_step_kernel(const StepArgs a) {
+  US_PDL_PROLOGUE();
+  constexpr int RG = kStepThreads / LQ;               // row groups
+  __shared__ float qs[kMaxDim], ks[kMaxDim], gs[kMaxDim], ps[GENERAL ? kMaxDim : 1], vs[LQ * 4];
+  __shared__ __align__(16) float red[RG][LQ * 4];
+  __shared__ float scal[4];
+  const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int slot = a.slots[b], H = a.H, D = a.D, V = a.V;
+  if (slot < 0) {
+    for (int c = tid; c < V; c += kStepThreads) st_any(a.y, b * a.ldy + h * V + c, a.bf16, 0.f);
+    return;
+  }
+  const int p0 = a.pos[b], cq4 = (tid % LQ) * 4, rg = tid / LQ;
+  const bool on = cq4 < V;
+  float* Sg = a.state + ((long long)slot * H + h) * D * V + cq4;
+  float4 S[R];
+#pragma unroll
+  for (int i = 0; i < R; ++i) {
+    const int row = rg + i * RG;
+    S[i] = (p0 > 0 && on && row < D) ? *reinterpret_cast<const float4*>(Sg + (long long)row * V)
+                                     : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  const long long xb = b * a.ldx;
+  const int hk = h / (H / a.Hk);
+  // ---- vectors ----
+  for (int e = tid; e < 3 * D + V; e += kStepThreads) {
+    const int what = e < D ? 0 : e < 2 * D ? 1 : e < 3 * D ? 2 : 3;       // q, k, decay, v
+    const int d = e - what * D;
+    if (what == 2) {
+      const float lo = a.low[b * a.ldlow + h * D + d] + a.bias[h * D + d];
+      if (GENERAL) {
+        gs[d] = decay_exp(-a.rate * sigmoid_f(lo));
+        ps[d] = sigmoid_f(ld_any(a.x, xb + a.off_b + h * D + d, a.bf16) + a.a_bias[h * D + d]);
+      } else {
+        gs[d] = decay_exp(-expf(a.A_log[h]) * softplus_f(lo));
+      }
+      continue;
+    }
+    float v;
+    if (GENERAL) {
+      const int off = what == 0 ? a.off_q : what == 1 ? a.off_k : a.off_v;
+      v = ld_any(a.x, xb + off + h * (what == 3 ? V : D) + d, a.bf16);
+    } else {
+      const int nq = a.Hk * D, C = 2 * nq + H * V;
+      const int ch = what == 3 ? h * V + d : hk * D + d;                  // channel of q, k or v
+      const int col = (what == 0 ? a.off_q : what == 1 ? a.off_k : a.off_v) + ch;
+      const float* taps = (what == 0 ? a.cq : what == 1 ? a.ck : a.cv) + (long long)ch * a.K;
+      const long long ring = (long long)slot * a.K * C + (what == 3 ? 2 * nq : what == 1 ? nq : 0) + ch;
+      const float cur = ld_any(a.x, xb + col, a.bf16);
+      float acc = taps[a.K - 1] * cur;
+#pragma unroll
+      for (int j = 1; j < kMaxTaps; ++j)
+        if (j < a.K && p0 - j >= 0)
+          acc += taps[a.K - 1 - j] * ld_any(a.conv, ring + (long long)((p0 - j) % a.K) * C, a.bf16);
+      // the entry written is one that no reader of this token touches
+      if (a.K > 1 && (what == 3 || h % (H / a.Hk) == 0))
+        st_any(a.conv, ring + (long long)(p0 % a.K) * C, a.bf16, cur);
+      v = acc / (1.f + expf(-acc));
+    }
+    (what == 0 ? qs : what == 1 ? ks : vs)[d] = v;
+  }
+  __syncthreads();
+  if (warp < 2) {                                      // unit lengths of q and k
+    const float* x = warp ? ks : qs;
+    float ss = 0.f;
+    for (int d = lane; d < D; d += 32) ss += x[d] * x[d];
+    ss = us::warp_sum(ss);
+    if (lane == 0) scal[warp] = 1.f / sqrtf(ss + 1e-6f);
+  } else if (!GENERAL && tid == 64) {
+    scal[2] = sigmoid_f(ld_any(a.x, xb + a.off_b + h, a.bf16));
+  }
+  __syncthreads();
+  const float kinv = scal[1];
+  // ---- what the key sees ----
+  float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+  for (int i = 0; i < R; ++i) {
+    const int row = rg + i * RG;
+    if (row >= D) break;
+    const float k = ks[row] * kinv;
+    if (!GENERAL) {
+      const float g = gs[row];
+      S[i].x *= g; S[i].y *= g; S[i].z *= g; S[i].w *= g;
+    }
+    acc.x = fmaf(S[i].x, k, acc.x); acc.y = fmaf(S[i].y, k, acc.y);
+    acc.z = fmaf(S[i].z, k, acc.z); acc.w = fmaf(S[i].w, k, acc.w);
+  }
+  auto gather = [&](float4 x) {                        // sum over the row groups
+    *reinterpret_cast<float4*>(&red[rg][cq4]) = x;
+    __syncthreads();
+    float4 t = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int r = 0; r < RG; ++r) {
+      const float4 e = *reinterpret_cast<const float4*>(&red[r][cq4]);
+      t.x += e.x; t.y += e.y; t.z += e.z; t.w += e.w;
+    }
+    return t;
+  };
+  const float4 seen = gather(acc);
+  float4 vv = make_float4(0.f, 0.f, 0.f, 0.f), u = seen;
+  if (on) vv = make_float4(vs[cq4], vs[cq4 + 1], vs[cq4 + 2], vs[cq4 + 3]);
+  if (!GENERAL) {
+    const float beta = scal[2];
+    u = make_float4(beta * (vv.x - seen.x), beta * (vv.y - seen.y), beta * (vv.z - seen.z),
+                    beta * (vv.w - seen.w));
+  }
+  acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+  for (int i = 0; i < R; ++i) {
+    const int row = rg + i * RG;
+    if (row >= D) break;
+    float4& x = S[i];
+    if (GENERAL) {
+      const float g = gs[row], k = ks[row], p = ps[row] * (k * kinv);
+      x.x = fmaf(k, vv.x, fmaf(-p, u.x, g * x.x)); x.y = fmaf(k, vv.y, fmaf(-p, u.y, g * x.y));
+      x.z = fmaf(k, vv.z, fmaf(-p, u.z, g * x.z)); x.w = fmaf(k, vv.w, fmaf(-p, u.w, g * x.w));
+    } else {
+      const float k = ks[row] * kinv;
+      x.x = fmaf(k, u.x, x.x); x.y = fmaf(k, u.y, x.y);
+      x.z = fmaf(k, u.z, x.z); x.w = fmaf(k, u.w, x.w);
+    }
+    const float q = qs[row];
+    acc.x = fmaf(x.x, q, acc.x); acc.y = fmaf(x.y, q, acc.y);
+    acc.z = fmaf(x.z, q, acc.z); acc.w = fmaf(x.w, q, acc.w);
+    if (on) *reinterpret_cast<float4*>(Sg + (long long)row * V) = x;
+  }
+  __syncthreads();                                     // the first sum has been read
+  float4 o = gather(acc);
+  const float qscale = GENERAL ? 1.f : scal[0] / sqrtf((float)D);
+  o.x *= qscale; o.y *= qscale; o.z *= qscale; o.w *= qscale;
+  // ---- norm over the head's values, weight, gate ----
+  if (warp >= (LQ + 31) / 32) return;                  // the first LQ threads hold the head once
+  float ss = (tid < LQ && on) ? o.x * o.x + o.y * o.y + o.z * o.z + o.w * o.w : 0.f;
+  ss = us::warp_sum(ss);
+  if (LQ > 32) {
+    if (lane == 0) scal[2 + warp] = ss;                // (beta has been read)
+    asm volatile("bar.sync 1, 64;" ::: "memory");
+    ss = scal[2] + scal[3];
+  }
+  if (tid >= LQ || !on) return;
+  const float inv = 1.f / sqrtf(ss / (float)V + a.eps);
+  const float r[4] = {o.x, o.y, o.z, o.w};
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int c = h * V + cq4 + i;
+    st_any(a.y, b * a.ldy + c, a.bf16,
+           r[i] * inv * a.nw[h * a.nw_head_stride + cq4 + i] * sigmoid_f(ld_any(a.gate, b * a.ldg + c, a.gate_bf16)));
+  }
+}
+
+template <int LQ, bool GENERAL>
+int launch_step(const StepArgs& a, int B, cudaStream_t stream) {
+  const int rows = (a.D + kStepThreads / LQ - 1) / (kStepThreads / LQ);
+  const dim3 grid(a.H, B), block(kStepThreads);
+  if (rows <= 4) US_CUDA_CHECK(us::launch_pdl(vector_delta_step_kernel<4, LQ, GENERAL>, grid, block, 0, stream, a));
+  else if (rows <= 8) US_CUDA_CHECK(us::launch_pdl(vector_delta_step_kernel<8, LQ, GENERAL>, grid, block, 0, stream, a));
+  else if (rows <= 16) US_CUDA_CHECK(us::launch_pdl(vector_delta_step_kernel<16, LQ, GENERAL>, grid, block, 0, stream, a));
+  else return US_ERR_UNSUPPORTED;
+  return US_OK;
+}
+
+template <bool GENERAL>
+int step_impl(const StepArgs& a, int B, cudaStream_t stream) {
+  US_REQUIRE(a.x && a.low && a.bias && a.state && a.nw && a.gate && a.y && a.slots && a.pos && B >= 1 &&
+             B <= 65535 && a.H >= 1 && a.ldy == (long long)a.H * a.V && ((uintptr_t)a.state % 16) == 0);
+  if (a.D < 1 || a.D > kMaxDim || (a.V & 3) || a.V > 256) return US_ERR_UNSUPPORTED;
+  if (a.V <= 64) return launch_step<16, GENERAL>(a, B, stream);
+  if (a.V <= 128) return launch_step<32, GENERAL>(a, B, stream);
+  return launch_step<64, GENERAL>(a, B, stream);
+}
+
 template <int DP, bool GENERAL>
 int launch_rule(const RuleArgs& a, int B, cudaStream_t stream) {
   constexpr size_t smem = 2 * Stage<DP, GENERAL>::kFloats * sizeof(float);
@@ -587,4 +790,36 @@ US_API int us_head_norm_gate(const float* o, const float* w, int w_head_stride, 
                                0, (cudaStream_t)stream_, o, w, w_head_stride, gate, ldg, y, ldy, rows,
                                H, V, eps, bf16, gate_bf16));
   return US_OK;
+}
+
+// One token of every sequence: projection rows x (q, k, v, step size at their columns), decay rows
+// low and gate rows in, y [B, H * V] (input of the output projection) out; ring and state advance.
+// US_ERR_UNSUPPORTED: the caller takes the separate kernels.
+US_API int us_channel_delta_step(const void* x, long long ldx, int off_q, int off_k, int off_v,
+                                 int off_b, const float* cq, const float* ck, const float* cv,
+                                 const float* low, long long ldlow, const float* A_log,
+                                 const float* dt_bias, void* conv, float* state, const float* nw,
+                                 int nw_head_stride, const void* gate, long long ldg, void* y,
+                                 long long ldy, const int* slots, const int* pos, int B, int H, int Hk,
+                                 int D, int V, int K, float eps, int bf16, int gate_bf16,
+                                 void* stream_) {
+  US_REQUIRE(cq && ck && cv && A_log && Hk >= 1 && H % Hk == 0 && K >= 1 && (K == 1 || conv));
+  if (K > kMaxTaps) return US_ERR_UNSUPPORTED;
+  StepArgs a{x, ldx, off_q, off_k, off_v, off_b, cq, ck, cv, low, ldlow, A_log, dt_bias, nullptr, conv,
+             state, nw, nw_head_stride, gate, ldg, y, ldy, slots, pos, H, Hk, D, V, K, bf16, gate_bf16,
+             eps, 0.f};
+  return step_impl<false>(a, B, (cudaStream_t)stream_);
+}
+
+US_API int us_general_delta_step(const void* x, long long ldx, int off_r, int off_k, int off_v,
+                                 int off_a, const float* low, long long ldlow, const float* w0,
+                                 const float* a_bias, float* state, const float* nw,
+                                 int nw_head_stride, const void* gate, long long ldg, void* y,
+                                 long long ldy, const int* slots, const int* pos, int B, int H, int D,
+                                 float rate, float eps, int bf16, int gate_bf16, void* stream_) {
+  US_REQUIRE(a_bias);
+  StepArgs a{x, ldx, off_r, off_k, off_v, off_a, nullptr, nullptr, nullptr, low, ldlow, nullptr, w0,
+             a_bias, nullptr, state, nw, nw_head_stride, gate, ldg, y, ldy, slots, pos, H, H, D, D, 1,
+             bf16, gate_bf16, eps, rate};
+  return step_impl<true>(a, B, (cudaStream_t)stream_);
 }

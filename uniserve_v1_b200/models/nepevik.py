@@ -372,6 +372,10 @@ class NepevikModel:
         proj = F.linear(x, w["proj"])
         low = F.linear(proj[:, oa:oa + w["a2"].shape[1]], w["a2"], out_dtype=torch.float32)
         gate = F.linear(proj[:, og:og + w["g2"].shape[1]], w["g2"])
+        if x.is_cuda and m.one_token and VD.step_fits(H, D, V, w["o"].shape[1]):
+            y = VD.channel_step(proj, (oq, ok, ov, ob), low, w, conv, S, gate, m, H, Hk, D, V,
+                                self.cfg.eps)
+            return F.linear(y, w["o"])
         q, k, v, g, beta = VD.channel_prep(proj, (oq, ok, ov, ob), low[:, :H * D], w, conv, m, H, Hk,
                                            D, V)
         o = VD.vector_delta_rule(q, k, v, g, S, m, beta=beta)
@@ -385,10 +389,13 @@ class NepevikModel:
         proj = F.linear(x, w["proj"])
         F.tanh_cols_(proj, ow, w["w2"].shape[1])
         low = F.linear(proj[:, ow:ow + w["w2"].shape[1]], w["w2"], out_dtype=torch.float32)
+        gate = proj[:, og:og + H * D]
+        if x.is_cuda and m.one_token and VD.step_fits(H, D, D, w["o"].shape[1]):
+            y = VD.general_step(proj, (orr, ok, ov, oa), low, w, S, gate, m, H, D, self.cfg.eps)
+            return F.linear(y, w["o"])
         g, n, p, k, r, v = VD.general_prep(proj, (orr, ok, ov, oa), low[:, :H * D], w, H, D)
         o = VD.vector_delta_rule(r, k, v, g, S, m, n=n, p=p)
-        y = VD.head_norm_gate(o, w["norm"], proj[:, og:og + H * D], self.cfg.eps, w["o"].shape[1],
-                              x.dtype)
+        y = VD.head_norm_gate(o, w["norm"], gate, self.cfg.eps, w["o"].shape[1], x.dtype)
         return F.linear(y, w["o"])
 
     def _attention(self, s: MixerSpec, w, x, m, meta, positions, caches):

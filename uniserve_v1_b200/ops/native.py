@@ -45,6 +45,10 @@ _SIGNATURES = {
                                   I, I, I, I, I, I, I, I, I, P]),
     "us_general_delta_prep": (I, [P, L, I, I, I, I, P, L, P, P, P, I, I, I, F, I, P]),
     "us_vector_delta_rule": (I, [I, P, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, P]),
+    "us_channel_delta_step": (I, [P, L, I, I, I, I, P, P, P, P, L, P, P, P, P, P, I, P, L, P, L, P, P,
+                                  I, I, I, I, I, I, F, I, I, P]),
+    "us_general_delta_step": (I, [P, L, I, I, I, I, P, L, P, P, P, P, I, P, L, P, L, P, P, I, I, I, F,
+                                  F, I, I, P]),
     "us_head_norm_gate": (I, [P, P, I, P, L, P, L, I, I, I, F, I, I, P]),
     "us_embed_rows": (I, [P, P, P, P, I, I, I, I, P]),
     "us_output_norm_add": (I, [P, P, P, F, I, P, P, P, P, F, F, I, I, I, I, F, I, P]),

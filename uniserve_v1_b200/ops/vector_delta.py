@@ -149,3 +149,36 @@ def head_norm_gate(o, w, gate, eps, ldo, dtype):
     out = torch.zeros(T, ldo, dtype=dtype)
     out[:, :H * V] = (y.reshape(T, H * V) * torch.sigmoid(gate.float())).to(dtype)
     return out
+
+
+def step_fits(H, D, V, ldo) -> bool:
+    """Whether the one-launch decode step serves these sizes (else: the separate kernels)."""
+    groups = 256 // (16 if V <= 64 else 32 if V <= 128 else 64)
+    return V % 4 == 0 and V <= 256 and D <= 256 and -(-D // groups) <= 16 and ldo == H * V
+
+
+def channel_step(x, offs, low, w, conv, state, gate, m: SeqMeta, H, Hk, D, V, eps):
+    """``channel_prep``, ``vector_delta_rule`` and ``head_norm_gate`` for one token of every
+    sequence in one launch (GPU, ``step_fits``)."""
+    B = x.shape[0]
+    y = torch.empty(B, H * V, dtype=x.dtype, device=x.device)
+    N.call("us_channel_delta_step", N.ptr(x), x.stride(0), *offs, N.ptr(w["conv_q"]),
+           N.ptr(w["conv_k"]), N.ptr(w["conv_v"]), N.ptr(low), low.stride(0), N.ptr(w["A_log"]),
+           N.ptr(w["dt_bias"]), N.ptr(conv), N.ptr(state), N.ptr(w["norm"]),
+           0 if w["norm"].numel() == V else V, N.ptr(gate), gate.stride(0), N.ptr(y), H * V,
+           N.ptr(m.slots), N.ptr(m.positions), B, H, Hk, D, V, w["conv_q"].shape[1], eps,
+           int(x.dtype == BF16), int(gate.dtype == BF16), N.stream())
+    return y
+
+
+def general_step(x, offs, low, w, state, gate, m: SeqMeta, H, D, eps):
+    """``general_prep``, ``vector_delta_rule`` and ``head_norm_gate`` for one token of every
+    sequence in one launch (GPU, ``step_fits``)."""
+    B = x.shape[0]
+    y = torch.empty(B, H * D, dtype=x.dtype, device=x.device)
+    N.call("us_general_delta_step", N.ptr(x), x.stride(0), *offs, N.ptr(low), low.stride(0),
+           N.ptr(w["w0"]), N.ptr(w["a_bias"]), N.ptr(state), N.ptr(w["norm"]),
+           0 if w["norm"].numel() == D else D, N.ptr(gate), gate.stride(0), N.ptr(y), H * D,
+           N.ptr(m.slots), N.ptr(m.positions), B, H, D, GENERAL_DECAY_RATE, eps,
+           int(x.dtype == BF16), int(gate.dtype == BF16), N.stream())
+    return y

@@ -104,6 +104,15 @@ def main():
             xg, (0, H * D2, 2 * H * D2, 4 * H * D2), lowg, w, H, D2), n * H * D2 * (4 * 2 + 4 + 24.0))
         o, gate, hw = rnd(n, H, V, dtype=torch.float32), rnd(n, H * V), rnd(V, dtype=torch.float32)
         case(f"head_norm_gate_{kind}", lambda: VD.head_norm_gate(o, hw, gate, 1e-6, H * V, bf), n * H * V * 8.0)
+        if kind == "decode":
+            w.update(norm=hw)
+            case("channel_step_decode", lambda: VD.channel_step(x, (0, Hk * D, 2 * Hk * D, C), low, w, conv, pool,
+                                                                gate, m, H, Hk, D, V, 1e-6),
+                 state + n * (2.0 * C * (K + 1) + 4 * H * D + 4 * H * V))
+            w2 = dict(w, norm=rnd(H * D2, dtype=torch.float32))
+            case("general_step_decode", lambda: VD.general_step(xg, (0, H * D2, 2 * H * D2, 4 * H * D2), lowg, w2,
+                                                                pool2, xg[:, 3 * H * D2:4 * H * D2], m, H, D2, 1e-6),
+                 2.0 * B * H * D2 * D2 * 4 + n * H * D2 * (5 * 2 + 4 + 2.0))
         zz = gate.view(n, H, V)
         case(f"rmsnorm_gated_{kind} (like)", lambda: GD.rmsnorm_gated(o, hw, zz, 1e-6), n * H * V * 8.0)
         # ---- residual rows ----
