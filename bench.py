@@ -629,11 +629,146 @@ def qwen3_record(job: Job) -> dict:
     return rec
 
 
+# ------------------------------------------------------------------ Nepevik --
+def nepevik_record(job: Job) -> dict:
+    """Prefill and decode throughput of the Nepevik decoder at a production-like layer size
+    (random weights) through ``LLMEngine``, beside two existing models of equal size: the
+    Qwen3.5-style hybrid (gated delta net, dense-state engine) and Qwen3-MoE (attention in every
+    layer, the same paged engine).  One GPU.
+
+    ``value``: output tokens/s of the device-timed decode step of all concurrent requests (graph
+    replays); ``sizes``: the same and the prompt throughput per (requests, prompt length)."""
+    import torch
+    from uniserve_v1_b200.engine.dense_state import DenseStateEngine
+    from uniserve_v1_b200.engine.engine import LLMEngine
+    from uniserve_v1_b200.engine.types import SamplingParams
+    from uniserve_v1_b200.models.nepevik import NepevikConfig, NepevikModel
+    from uniserve_v1_b200.models.qwen3_5 import Qwen35Config, Qwen35MoeModel
+    from uniserve_v1_b200.models.qwen3_moe import Qwen3MoeConfig, Qwen3MoeModel
+    from uniserve_v1_b200.ops import native
+
+    args, dev = job.args, job.dev
+    assert job.world == 1, "this workload runs on one GPU"
+    K, W = args.steps, args.warmup
+    layers, vocab = args.layers or 8, 32000
+    sizes = [(args.concurrency, args.prompt_len)] if args.concurrency and args.prompt_len \
+        else [(64, 1024), (8, 4096), (1, 4096)]
+    ncfg = NepevikConfig.bench(layers)
+    ncfg.vocab_size = vocab
+    hcfg = Qwen35Config(vocab_size=vocab, hidden_size=2048, num_hidden_layers=layers,
+                        num_attention_heads=32, num_key_value_heads=4, head_dim=128,
+                        linear_num_key_heads=16, linear_num_value_heads=32, num_experts=64,
+                        num_experts_per_tok=4, moe_intermediate_size=768,
+                        shared_expert_intermediate_size=1024, eos_token_id=vocab - 1)
+    qcfg = Qwen3MoeConfig(vocab_size=vocab, num_hidden_layers=layers, num_experts=64,
+                          num_experts_per_tok=4, eos_token_id=vocab - 1)
+    g = torch.Generator().manual_seed(5)
+
+    def prompts(n, length):
+        return [torch.randint(0, vocab - 1, (length,), generator=g).tolist() for _ in range(n)]
+
+    def measure(make_engine, n, length, graph_steps):
+        """(prompt tokens/s, decode ms per step, launches per step) of one engine."""
+        sp = SamplingParams(temperature=0.0, max_tokens=K + W + 12, ignore_eos=True)
+        eng = make_engine(n, length)
+        run = getattr(eng, "scheduler", eng)
+        for p in prompts(min(n, max(1, 8192 // length)), length):    # warm-up at the batch's size
+            eng.add_request(p, SamplingParams(temperature=0.0, max_tokens=4, ignore_eos=True))
+        while eng.has_work():
+            eng.step()
+        for p in prompts(n, length):
+            eng.add_request(p, sp)
+
+        def prefill():
+            while run.waiting or any(not r.output_ids for r in run.running):
+                eng.step()
+        pre_ms, _, _ = job.timed(prefill)
+        if not graph_steps:                 # eager engine: its own steps
+            for _ in range(W):
+                eng.step()
+            l0 = native.launch_count
+            ms, _, _ = job.timed(lambda: [eng.step() for _ in range(K)])
+            return n * length / pre_ms * 1e3, ms / K, (native.launch_count - l0) // K, None, eng
+        for _ in range(W):
+            eng.step()
+        h0, d0 = eng.runner.h2d_bytes, eng.runner.d2h_bytes
+        e_ms, _, _ = job.timed(lambda: [eng.step() for _ in range(K)])
+        e2e = {"value": n * K / (e_ms / 1e3), "unit": "output tokens/s", "ms_per_step": e_ms / K,
+               "h2d_bytes_per_step": (eng.runner.h2d_bytes - h0) // K,
+               "d2h_bytes_per_step": (eng.runner.d2h_bytes - d0) // K}
+        rows, runner = list(eng.scheduler.running), eng.runner
+        for r in rows:
+            r.pages.extend(eng.blocks.allocate(eng.scheduler._pages_needed(r, r.num_tokens + K + W + 2)))
+        B = runner.bucket_for(len(rows))
+        blk = runner._decode_block(B)
+        runner._fill_decode(blk, rows, B)
+        graph = runner._graph(B, "greedy")
+        blk.upload()
+        for _ in range(W):
+            graph.graph.replay()
+
+        def replays():
+            for _ in range(K):
+                graph.graph.replay()
+        ms, _, _ = job.timed(replays)
+        native.launch_count += graph.launches * K
+        return n * length / pre_ms * 1e3, ms / K, graph.launches, e2e, eng
+
+    def paged(model):
+        return lambda n, length: LLMEngine(model, max_num_seqs=n, max_model_len=length + 128,
+                                           max_num_batched_tokens=8192, enable_prefix_cache=False)
+
+    out, clocks, launches, head = [], None, 0, None
+    for name, build_model, make, graphs in (
+            ("nepevik", lambda: NepevikModel(ncfg, dev).init_random(0), paged, True),
+            ("qwen3.5-style hybrid", lambda: Qwen35MoeModel(hcfg, dev).init_random(0, std=0.02),
+             lambda m: lambda n, length: DenseStateEngine(m, max_num_seqs=n, max_model_len=length + 128,
+                                                          prefill_chunk=8192, state_cache_entries=0), False),
+            ("qwen3-moe", lambda: Qwen3MoeModel(qcfg, dev).init_random(0), paged, True)):
+        if args.only_nepevik and name != "nepevik":
+            continue
+        model = build_model()
+        for n, length in sizes:
+            sampler = ClockSampler(job.local, period_ms=50)
+            if name == "nepevik" and head is None:
+                sampler.start()
+            l0 = native.launch_count
+            pre, ms, per_step, e2e, eng = measure(make(model), n, length, graphs)
+            if name == "nepevik" and head is None:
+                clocks, launches = sampler.stop(), native.launch_count - l0
+                head = (n, length, ms, e2e, per_step)
+            native.raise_on_device_error()
+            out.append({"model": name, "requests": n, "prompt_tokens": length,
+                        "prefill_tokens_per_s": round(pre), "decode_ms_per_step": round(ms, 4),
+                        "decode_tokens_per_s": round(n / ms * 1e3), "launches_per_step": per_step,
+                        "end_to_end_tokens_per_s": e2e and round(e2e["value"])})
+            if hasattr(eng, "runner"):
+                eng.runner.release_graphs()
+            del eng
+            release_device_memory()
+        del model
+        release_device_memory()
+    n, length, ms, e2e, per_step = head
+    return {"metric": "Nepevik output tokens/s", "value": n / ms * 1e3, "unit": "tokens/s", "n_gpus": 1,
+            "steps": K, "warmup": W, "ms_per_step": ms, "higher_is_better": True, "scaling": "strong",
+            "vs_baseline": None, "dtype": "bf16",
+            "data": "synthetic (uniform-random prompt ids, random-init weights)",
+            "config": {"model": "Nepevik, layer sizes of NepevikConfig.bench", "layers": layers, "hidden": 2048,
+                       "vocab": vocab, "global_batch": n, "seq_len": length, "parallelism": "tp1",
+                       "step": "one decode step of all concurrent requests",
+                       "l2": "inputs larger than L2 (weights and state read per step >> 126 MB)"},
+            "clocks": clocks, "e2e": e2e, "gpu_launches": launches, "launches_per_step": per_step,
+            "sizes": out}
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--workload", default="all", choices=["all", "qwen3-moe", "fasth3"],
+    ap.add_argument("--workload", default="all", choices=["all", "qwen3-moe", "fasth3", "nepevik"],
                     help="all (default): the FastH3 clip latency as the headline with the "
-                         "Qwen3-MoE record nested; or one of the two alone")
+                         "Qwen3-MoE record nested; or one of the two alone; nepevik: that decoder's "
+                         "throughput beside models of equal size (one GPU, not part of all)")
+    ap.add_argument("--only-nepevik", action="store_true",
+                    help="nepevik: without the models it is compared with")
     ap.add_argument("--frames", type=int, default=0, help="fasth3: frame count (rule 17n + 5)")
     ap.add_argument("--mlp-fp8", action="store_true",
                     help="fasth3: feed-forward projections in FP8 (per-tensor weights, per-row "
@@ -689,6 +824,8 @@ def main() -> int:
             line["metric"] = "FastH3 8-step clip latency (s); Qwen3-MoE output tokens/s nested"
             line["qwen3_moe"] = q
             line["gpu_launches"] = line["gpu_launches"] + q.get("gpu_launches", 0)
+    if args.workload == "nepevik":
+        line = nepevik_record(job)
     if job.rank == 0 and line:
         print(json.dumps(line))
     job.mark("line printed")
