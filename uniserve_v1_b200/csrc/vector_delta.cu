@@ -18,11 +18,12 @@
 // starts from a zero state whatever its slot holds: slots are handed on without being cleared,
 // and nothing has to be launched when a request is admitted.  A negative slot marks padding.
 //
-// Rule kernel: a CTA owns 32 value columns of one head of one sequence.  A lane holds D/16 rows
-// x 4 columns of S in registers (16 lanes span the rows, so one 16-byte access per row moves 4
-// columns, and 4 independent chains hide the FMA latency); the two D-long reductions of a token
-// fold 4 columns over 16 lanes in five shuffles.  The vectors of the next 16 tokens are copied
-// into the other half of shared memory meanwhile.  The state crosses HBM once per call.
+// Rule kernel: a CTA owns 32 value columns of one head of one sequence.  A lane holds D/8 rows x 2
+// columns of S in registers as row pairs (packed FP32 instructions), so the two D-long reductions
+// of a token are short chains and three shuffles; the read-out's is folded beside the next token's
+// first one.  A token depends on the one before through one reduction and one update: that chain
+// is what a long prompt costs.  The vectors of the next rounds of 8 tokens are on their way into
+// a ring in shared memory meanwhile (four warps multiply, one fetches).  The state crosses HBM once per call.
 #include "include/us_common.cuh"
 
 namespace {
@@ -56,7 +57,7 @@ __device__ __forceinline__ int seq_of(const int* cu, int B, int t) {
 
 constexpr int kMaxTaps = 8;
 constexpr int kMaxDim = 256;      // key channels per head
-constexpr int kPrepTokens = 4;    // consecutive rows of one warp in the prefill form
+constexpr int kPrepTokens = 16;   // consecutive rows of one warp in the prefill form
 
 struct ChannelPrep {
   const void* x;                // projection rows, element type = bf16 flag
@@ -76,8 +77,11 @@ struct ChannelPrep {
 // a token reads K - 1 entries and writes another one, so nothing is shifted and the readers of
 // one token never meet its writer.  Positions before the sequence are zero.
 
-// A warp owns one head of q, of k, of v or of the decay for kPrepTokens rows (prefill) or one
-// row (every sequence brings one token: the warp then also stores its channels' inputs).
+// A warp owns one head of q, of k, of v or of the decay for kPrepTokens consecutive rows (prefill)
+// or one row (every sequence brings one token: the warp then also stores its channels' inputs).
+// The window of a channel stays in registers from row to row (KT >= K taps, leading ones zero).
+// NI: channels per lane.
+template <int KT, int NI>
 __global__ void __launch_bounds__(256) channel_prep_kernel(const ChannelPrep a) {
   US_PDL_PROLOGUE();
   const int lane = threadIdx.x & 31;
@@ -89,6 +93,7 @@ __global__ void __launch_bounds__(256) channel_prep_kernel(const ChannelPrep a) 
   if (unit >= 2 * a.Hk + a.H) {                       // decay and step size
     const int h = unit - 2 * a.Hk - a.H;
     const float A = expf(a.A_log[h]);
+#pragma unroll 2
     for (int t = t0; t < t1; ++t) {
       const float* lo = a.low + (long long)t * a.ldlow + (long long)h * a.D;
       float* g = a.g + ((long long)t * a.H + h) * a.D;
@@ -115,44 +120,73 @@ __global__ void __launch_bounds__(256) channel_prep_kernel(const ChannelPrep a) 
     cbase = 2 * a.Hk * a.D + head * a.V;
   }
   const long long C = 2LL * a.Hk * a.D + (long long)a.H * a.V;
-  for (int t = t0; t < t1; ++t) {
-    const int s = seq_of(a.cu, a.B, t);
-    const int start = a.cu[s], slot = a.slots[s];
-    if (slot < 0) continue;
-    const int p0 = a.pos[start];
-    const long long sbase = (long long)slot * a.K * C + cbase;
-    float y[kMaxDim / 32];
-    float ss = 0.f;
+  float w[NI][KT], win[NI][KT];                       // win[KT - 1]: the current row
 #pragma unroll
-    for (int i = 0; i < kMaxDim / 32; ++i) {
-      const int d = i * 32 + lane;
-      y[i] = 0.f;
-      if (d >= dim) continue;
-      float acc = 0.f;
-      for (int j = 0; j < a.K; ++j) {
-        const int src = t - (a.K - 1) + j;            // packed row of the tap
-        const int sp = p0 + src - start;              // its position
-        float xv = 0.f;
-        if (src >= start) xv = ld_any(a.x, (long long)src * a.ldx + off + d, a.bf16);
-        else if (sp >= 0) xv = ld_any(a.conv, sbase + (long long)(sp % a.K) * C + d, a.bf16);
-        acc += taps[(long long)d * a.K + j] * xv;
-        if (a.one_token && a.K > 1 && j == a.K - 1)
-          st_any(a.conv, sbase + (long long)(p0 % a.K) * C + d, a.bf16, xv);
+  for (int i = 0; i < NI; ++i)
+#pragma unroll
+    for (int j = 0; j < KT; ++j) {
+      const int d = i * 32 + lane, c = j - (KT - a.K);
+      w[i][j] = (c >= 0 && d < dim) ? taps[(long long)d * a.K + c] : 0.f;
+    }
+  int s = seq_of(a.cu, a.B, t0), end = t0, slot = -1;
+  for (int t = t0; t < t1; ++t) {
+    if (t >= end) {                                   // first row here, or of the next sequence
+      while (a.cu[s + 1] <= t) ++s;
+      const int start = a.cu[s], p0 = a.pos[start];
+      end = a.cu[s + 1];
+      slot = a.slots[s];
+      const long long sbase = (long long)max(slot, 0) * a.K * C + cbase;
+#pragma unroll
+      for (int j = 1; j < KT; ++j) {                  // entry of the row KT - j back, before t
+        const int src = t - (KT - j), pos = p0 + src - start;
+        const bool in_x = src >= start, in_ring = !in_x && pos >= 0 && KT - j < a.K && slot >= 0;
+        const long long at = in_ring ? sbase + (long long)(pos % a.K) * C : 0;
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+          const int d = i * 32 + lane;
+          float v = 0.f;
+          if (d < dim) {
+            if (in_x) v = ld_any(a.x, (long long)src * a.ldx + off + d, a.bf16);
+            else if (in_ring) v = ld_any(a.conv, at + d, a.bf16);
+          }
+          win[i][j] = v;
+        }
       }
+      if (a.one_token && a.K > 1 && slot >= 0) {
+        const long long at1 = sbase + (long long)(p0 % a.K) * C;
+#pragma unroll
+        for (int i = 0; i < NI; ++i)
+          if (i * 32 + lane < dim)
+            st_any(a.conv, at1 + i * 32 + lane, a.bf16,
+                   ld_any(a.x, (long long)t * a.ldx + off + i * 32 + lane, a.bf16));
+      }
+    }
+    // the window moves on: entries 1 .. KT - 1 become the older ones of this row
+    float y[NI], ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      const int d = i * 32 + lane;
+#pragma unroll
+      for (int j = 0; j + 1 < KT; ++j) win[i][j] = win[i][j + 1];
+      win[i][KT - 1] = d < dim ? ld_any(a.x, (long long)t * a.ldx + off + d, a.bf16) : 0.f;
+      float acc = 0.f;
+#pragma unroll
+      for (int j = 0; j < KT; ++j) acc = fmaf(w[i][j], win[i][j], acc);
       y[i] = acc / (1.f + expf(-acc));
       ss += y[i] * y[i];
     }
+    if (slot < 0) continue;
     if (unit < 2 * a.Hk) {
       float inv = 1.f / sqrtf(us::warp_sum(ss) + 1e-6f);
       if (unit < a.Hk) inv *= 1.f / sqrtf((float)a.D);
       float* dst = (unit < a.Hk ? a.q : a.k) + ((long long)t * a.Hk + head) * a.D;
 #pragma unroll
-      for (int i = 0; i < kMaxDim / 32; ++i)
+      for (int i = 0; i < NI; ++i)
         if (i * 32 + lane < dim) dst[i * 32 + lane] = y[i] * inv;
     } else {
       float* dst = a.v + ((long long)t * a.H + head) * a.V;
 #pragma unroll
-      for (int i = 0; i < kMaxDim / 32; ++i)
+      for (int i = 0; i < NI; ++i)
         if (i * 32 + lane < dim) dst[i * 32 + lane] = y[i];
     }
   }
@@ -219,7 +253,9 @@ __global__ void __launch_bounds__(256) general_prep_kernel(const GeneralPrep a) 
 }
 
 constexpr int kCols = 32;         // value columns per CTA
-constexpr int kRuleThreads = 128;
+constexpr int kRuleCompute = 128, kRuleCopy = 32;    // threads that multiply / that fetch vectors
+constexpr int kRuleThreads = kRuleCompute + kRuleCopy;
+constexpr int kRuleBufs = 4;                         // rounds of vectors in shared memory
 
 struct RuleArgs {
   const float *q, *k, *v;         // [rows, Hk, D] x 2, [rows, H, V]
@@ -233,31 +269,44 @@ struct RuleArgs {
   int H, Hk, D, V;
 };
 
-// Folds four per-lane column sums over the 16 lanes that span the rows: afterwards every lane
-// holds the sum of column ((lane >> 3) & 1) * 2 + ((lane >> 2) & 1).
-__device__ __forceinline__ float fold16(float c0, float c1, float c2, float c3, int lane) {
-  const bool up = lane & 8;
-  const float a0 = up ? c2 : c0, a1 = up ? c3 : c1, b0 = up ? c0 : c2, b1 = up ? c1 : c3;
-  const float s0 = a0 + __shfl_xor_sync(0xffffffffu, b0, 8);
-  const float s1 = a1 + __shfl_xor_sync(0xffffffffu, b1, 8);
-  const bool odd = lane & 4;
-  float s = (odd ? s1 : s0) + __shfl_xor_sync(0xffffffffu, odd ? s0 : s1, 4);
+// Folds two per-lane column sums over the 8 lanes that span the rows: afterwards lanes 0 .. 3 hold
+// column 0's sum, lanes 4 .. 7 column 1's.
+__device__ __forceinline__ float fold8(float c0, float c1, bool up) {
+  float s = (up ? c1 : c0) + __shfl_xor_sync(0xffffffffu, up ? c0 : c1, 4);
   s += __shfl_xor_sync(0xffffffffu, s, 2);
   s += __shfl_xor_sync(0xffffffffu, s, 1);
   return s;
 }
 
-template <int W>
-__device__ __forceinline__ void lds_vec(float (&o)[W], const float* p) {
-  if (W == 4) {
-    const float4 v = *reinterpret_cast<const float4*>(p);
-    o[0] = v.x; o[1 % W] = v.y; o[2 % W] = v.z; o[3 % W] = v.w;
-  } else if (W == 2) {
-    const float2 v = *reinterpret_cast<const float2*>(p);
-    o[0] = v.x; o[1 % W] = v.y;
-  } else {
-    o[0] = p[0];
-  }
+// Packed FP32 pairs (two rows of one state column per instruction).
+typedef unsigned long long f2;
+__device__ __forceinline__ f2 pack2(float a, float b) {
+  f2 r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+  return r;
+}
+__device__ __forceinline__ float lo2(f2 r) { return __uint_as_float((uint32_t)r); }
+__device__ __forceinline__ float hi2(f2 r) { return __uint_as_float((uint32_t)(r >> 32)); }
+__device__ __forceinline__ f2 fma2(f2 a, f2 b, f2 c) {
+  f2 d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ f2 mul2(f2 a, f2 b) {
+  f2 d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+__device__ __forceinline__ f2 add2(f2 a, f2 b) {
+  f2 d;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+// four consecutive floats as two pairs
+__device__ __forceinline__ void lds_vec(f2 (&o)[2], const float* p) {
+  const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(p);
+  o[0] = v.x;
+  o[1] = v.y;
 }
 
 template <int BYTES>
@@ -273,44 +322,90 @@ template <int DP, bool GENERAL>
 struct Stage {
   static constexpr int kVecs = GENERAL ? 5 : 3;
   static constexpr int kToken = kVecs * DP + kCols + 4;
-  static constexpr int kChunk = DP > 128 ? 8 : 16;    // tokens per round
+  static constexpr int kChunk = 8;                    // tokens per round
   static constexpr int kFloats = kChunk * kToken;
 };
 
-// Asynchronous copies of n tokens' vectors, U floats at a time.
-template <int DP, bool GENERAL, int U>
-__device__ __forceinline__ void stage_tokens(const RuleArgs& a, float* buf, long long row0, int n,
-                                             int h, int hk, int col0) {
+// Asynchronous copies of tokens' vectors by the copying threads.  Widths that are multiples of
+// four move as 16-byte pieces: a thread owns the same pieces of every token and only advances its
+// pointers (address arithmetic per piece would cost as much as the recurrence).
+template <int DP, bool GENERAL>
+struct Copier {
   using St = Stage<DP, GENERAL>;
-  constexpr int kP = DP / U, kV = kCols / U;
-  for (int e = threadIdx.x; e < n * St::kVecs * kP; e += kRuleThreads) {
-    const int i = e / (St::kVecs * kP), rest = e - i * (St::kVecs * kP);
-    const int vec = rest / kP, d = (rest - vec * kP) * U;
-    if (d >= a.D) continue;
-    const long long row = row0 + i;
-    const float* src = vec == 1 ? a.k : vec == 2 ? a.q : vec == 0 ? a.g : vec == 3 ? a.n : a.p;
-    src += (vec == 1 || vec == 2 ? row * a.Hk + hk : row * a.H + h) * a.D + d;
-    cp_async<U * 4>(buf + i * St::kToken + vec * DP + d, src);
+  static constexpr int kQ = DP / 4;
+  static constexpr int kPieces = St::kVecs * kQ + kCols / 4;
+  static constexpr int kMine = (kPieces + kRuleCopy - 1) / kRuleCopy;
+  const float* src[kMine];
+  int step[kMine], dst[kMine];          // floats per token, place in the token (-1: nothing)
+  const float* beta;
+  int tid, heads;
+  bool quad;
+  __device__ __forceinline__ void init(const RuleArgs& a, int tid_, long long row0, int h, int hk, int col0) {
+    tid = tid_;
+    heads = a.H;
+    quad = (a.V & 3) == 0 && (a.D & 3) == 0;
+    beta = GENERAL ? nullptr : a.beta + row0 * a.H + h;
+#pragma unroll
+    for (int i = 0; i < kMine; ++i) {
+      const int e = tid + i * kRuleCopy, vec = e / kQ, d = (e - vec * kQ) * 4;
+      dst[i] = -1;
+      src[i] = nullptr;
+      step[i] = 0;
+      if (e < St::kVecs * kQ) {
+        if (d >= a.D) continue;
+        const bool shared = vec == 1 || vec == 2;
+        const int heads_ = shared ? a.Hk : a.H, hh = shared ? hk : h;
+        src[i] = (vec == 1 ? a.k : vec == 2 ? a.q : vec == 0 ? a.g : vec == 3 ? a.n : a.p) +
+                 (row0 * heads_ + hh) * a.D + d;
+        step[i] = heads_ * a.D;
+        dst[i] = vec * DP + d;
+      } else if (e < kPieces) {
+        const int c = (e - St::kVecs * kQ) * 4;
+        if (col0 + c >= a.V) continue;
+        src[i] = a.v + (row0 * a.H + h) * a.V + col0 + c;
+        step[i] = a.H * a.V;
+        dst[i] = St::kVecs * DP + c;
+      }
+    }
   }
-  for (int e = threadIdx.x; e < n * kV; e += kRuleThreads) {
-    const int i = e / kV, c = (e - i * kV) * U;
-    if (col0 + c < a.V)
-      cp_async<U * 4>(buf + i * St::kToken + St::kVecs * DP + c,
-                      a.v + ((row0 + i) * a.H + h) * a.V + col0 + c);
+  // the next n tokens into buf (row0: their first row, for widths that are not multiples of 4)
+  __device__ __forceinline__ void fetch(const RuleArgs& a, float* buf, int n, long long row0, int h, int hk,
+                                        int col0) {
+    if (quad) {
+      for (int t = 0; t < n; ++t, buf += St::kToken) {
+#pragma unroll
+        for (int i = 0; i < kMine; ++i)
+          if (dst[i] >= 0) {
+            cp_async<16>(buf + dst[i], src[i]);
+            src[i] += step[i];
+          }
+        if (!GENERAL && tid == 0) {
+          cp_async<4>(buf + St::kVecs * DP + kCols, beta);
+          beta += heads;
+        }
+      }
+    } else {
+      for (int t = 0; t < n; ++t, buf += St::kToken) {
+        const long long row = row0 + t;
+        for (int e = tid; e < St::kVecs * a.D; e += kRuleCopy) {
+          const int vec = e / a.D, d = e - vec * a.D;
+          const bool shared = vec == 1 || vec == 2;
+          const float* from = vec == 1 ? a.k : vec == 2 ? a.q : vec == 0 ? a.g : vec == 3 ? a.n : a.p;
+          cp_async<4>(buf + vec * DP + d, from + (shared ? row * a.Hk + hk : row * a.H + h) * a.D + d);
+        }
+        for (int c = tid; c < kCols && col0 + c < a.V; c += kRuleCopy)
+          cp_async<4>(buf + St::kVecs * DP + c, a.v + (row * a.H + h) * a.V + col0 + c);
+        if (!GENERAL && tid == 0) cp_async<4>(buf + St::kVecs * DP + kCols, a.beta + row * a.H + h);
+      }
+    }
   }
-  if (!GENERAL)
-    for (int i = threadIdx.x; i < n; i += kRuleThreads)
-      cp_async<4>(buf + i * St::kToken + St::kVecs * DP + kCols, a.beta + (row0 + i) * a.H + h);
-  asm volatile("cp.async.commit_group;" ::: "memory");
-}
+};
 
 template <int DP, bool GENERAL>
-__global__ void __launch_bounds__(kRuleThreads) vector_delta_kernel(const RuleArgs a) {
+__global__ void __launch_bounds__(kRuleThreads, DP > 128 ? 1 : 3) vector_delta_kernel(const RuleArgs a) {
   US_PDL_PROLOGUE();
   using St = Stage<DP, GENERAL>;
-  constexpr int R = DP / 16;                          // rows per lane
-  constexpr int W = R >= 4 ? 4 : R;                   // rows per shared-memory access
-  constexpr int NG = R / W;
+  constexpr int NG = DP / 32;                         // groups of four rows per lane
   extern __shared__ __align__(16) float sm[];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int h = blockIdx.y, s = blockIdx.z;
@@ -325,151 +420,161 @@ __global__ void __launch_bounds__(kRuleThreads) vector_delta_kernel(const RuleAr
     }
     return;
   }
-  const int rl = lane & 15;
-  const int my = ((lane >> 3) & 1) * 2 + ((lane >> 2) & 1);        // column a fold leaves here
-  const int cb = warp * 8 + (lane >> 4) * 4;                       // first of the lane's columns
+  const bool gaps = a.D < DP || col0 + kCols > a.V;    // places that no copy fills: zero
+  if (gaps) {
+    for (int e = tid; e < kRuleBufs * St::kFloats; e += kRuleThreads) sm[e] = 0.f;
+    __syncthreads();
+  }
+  if (tid >= kRuleCompute) {                          // the copying threads stay one round ahead
+    Copier<DP, GENERAL> cp;
+    cp.init(a, tid - kRuleCompute, start, h, hk, col0);
+    const int rounds = (T + St::kChunk - 1) / St::kChunk;
+    auto fetch = [&](int r) {                         // (an empty group past the end)
+      if (r < rounds)
+        cp.fetch(a, sm + (r % kRuleBufs) * St::kFloats, min(St::kChunk, T - r * St::kChunk),
+                 start + r * St::kChunk, h, hk, col0);
+      asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+#pragma unroll 1
+    for (int r = 0; r < kRuleBufs - 1; ++r) fetch(r);
+#pragma unroll 1
+    for (int r = 0; r < rounds; ++r) {
+      asm volatile("cp.async.wait_group %0;" ::"n"(kRuleBufs - 2) : "memory");
+      __syncthreads();                                // round r is there, round r - 1 consumed
+      fetch(r + kRuleBufs - 1);
+    }
+    return;
+  }
+  const int kq = lane & 7;                                         // lane's share of the rows
+  const bool up = kq >= 4;                                         // a fold leaves column 1 here
+  const int cb = warp * 8 + (lane >> 3) * 2;                       // the lane's two columns
   float* Sg = a.state + (((long long)slot * a.H + h) * a.D) * a.V + col0 + cb;
-  const bool wide = (a.V & 3) == 0, quad = wide && (a.D & 3) == 0;
+  const bool wide = (a.V & 1) == 0;
   const bool fresh = a.pos[start] == 0;
-  float S[R][4];
+  const bool c0ok = col0 + cb < a.V, c1ok = col0 + cb + 1 < a.V;
+  f2 S[NG * 2][2];                                    // row pairs x 2 columns
 #pragma unroll
   for (int j = 0; j < NG; ++j)
 #pragma unroll
-    for (int e = 0; e < W; ++e) {
-      const int row = (j * 16 + rl) * W + e;
-      float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (!fresh && row < a.D) {
-        const float* p = Sg + (long long)row * a.V;
-        if (wide) {
-          if (col0 + cb < a.V) x = *reinterpret_cast<const float4*>(p);
-        } else {
-          if (col0 + cb < a.V) x.x = p[0];
-          if (col0 + cb + 1 < a.V) x.y = p[1];
-          if (col0 + cb + 2 < a.V) x.z = p[2];
-          if (col0 + cb + 3 < a.V) x.w = p[3];
+    for (int e = 0; e < 2; ++e) {
+      float2 x[2];
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const int row = (j * 8 + kq) * 4 + e * 2 + i;
+        x[i] = make_float2(0.f, 0.f);
+        if (!fresh && row < a.D) {
+          const float* p = Sg + (long long)row * a.V;
+          if (wide && c0ok) {
+            x[i] = *reinterpret_cast<const float2*>(p);
+          } else {
+            if (c0ok) x[i].x = p[0];
+            if (c1ok) x[i].y = p[1];
+          }
         }
       }
-      S[j * W + e][0] = x.x; S[j * W + e][1] = x.y; S[j * W + e][2] = x.z; S[j * W + e][3] = x.w;
+      S[j * 2 + e][0] = pack2(x[0].x, x[1].x);
+      S[j * 2 + e][1] = pack2(x[0].y, x[1].y);
     }
-  if (a.D < DP || col0 + kCols > a.V) {               // places that no copy fills
-    for (int e = tid; e < 2 * St::kFloats; e += kRuleThreads) sm[e] = 0.f;
-    __syncthreads();
-  }
-  auto stage = [&](int c0, int buf) {
-    float* dst = sm + buf * St::kFloats;
-    const int n = min(St::kChunk, T - c0);
-    if (quad) stage_tokens<DP, GENERAL, 4>(a, dst, start + c0, n, h, hk, col0);
-    else stage_tokens<DP, GENERAL, 1>(a, dst, start + c0, n, h, hk, col0);
-  };
-  stage(0, 0);
-  float* op = a.out + ((long long)start * a.H + h) * a.V + col0 + cb + my;
-  const bool writes = (lane & 3) == 0 && col0 + cb + my < a.V;
+  float* op = a.out + ((long long)start * a.H + h) * a.V + col0 + cb + (up ? 1 : 0);
+  const bool writes = (lane & 3) == 0 && (up ? c1ok : c0ok);
   const long long ostep = (long long)a.H * a.V;
   // the read-out of a token is folded beside the next token's first reduction: two independent
   // shuffle chains instead of one after the other
-  float o0 = 0.f, o1 = 0.f, o2 = 0.f, o3 = 0.f;
+  float o0 = 0.f, o1 = 0.f;
   bool pending = false;
   int buf = 0;
-  for (int c0 = 0; c0 < T; c0 += St::kChunk, buf ^= 1) {
+  for (int c0 = 0; c0 < T; c0 += St::kChunk, buf = buf + 1 == kRuleBufs ? 0 : buf + 1) {
     const int n = min(St::kChunk, T - c0);
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
-    __syncthreads();
-    if (c0 + St::kChunk < T) stage(c0 + St::kChunk, buf ^ 1);
+    __syncthreads();                                  // this round's vectors are there
     const float* base = sm + buf * St::kFloats;
     for (int t = 0; t < n; ++t, base += St::kToken) {
       const float* vs = base + St::kVecs * DP;
-      float y0 = 0.f, y1 = 0.f, y2 = 0.f, y3 = 0.f;
+      f2 y[2][2] = {{0ull, 0ull}, {0ull, 0ull}};
 #pragma unroll
       for (int j = 0; j < NG; ++j) {
-        const int r0 = (j * 16 + rl) * W;
-        float m[W];
+        const int r0 = (j * 8 + kq) * 4;
+        f2 m[2];
         if (GENERAL) {
-          lds_vec<W>(m, base + 3 * DP + r0);
+          lds_vec(m, base + 3 * DP + r0);
         } else {
-          float g[W];
-          lds_vec<W>(m, base + DP + r0);
-          lds_vec<W>(g, base + r0);
+          f2 g[2];
+          lds_vec(m, base + DP + r0);
+          lds_vec(g, base + r0);
 #pragma unroll
-          for (int e = 0; e < W; ++e) {
-            // the state is decayed first; what the key sees is the decayed state
-            float* x = S[j * W + e];
-            x[0] *= g[e]; x[1] *= g[e]; x[2] *= g[e]; x[3] *= g[e];
-          }
+          for (int e = 0; e < 2; ++e)
+#pragma unroll
+            for (int c = 0; c < 2; ++c)     // the key sees the decayed state
+              S[j * 2 + e][c] = mul2(S[j * 2 + e][c], g[e]);
         }
 #pragma unroll
-        for (int e = 0; e < W; ++e) {
-          const float* x = S[j * W + e];
-          y0 = fmaf(x[0], m[e], y0); y1 = fmaf(x[1], m[e], y1);
-          y2 = fmaf(x[2], m[e], y2); y3 = fmaf(x[3], m[e], y3);
-        }
+        for (int e = 0; e < 2; ++e)
+#pragma unroll
+          for (int c = 0; c < 2; ++c) y[c][e] = fma2(S[j * 2 + e][c], m[e], y[c][e]);
       }
-      const float seen = fold16(y0, y1, y2, y3, lane);
-      const float o = fold16(o0, o1, o2, o3, lane);
+      y[0][0] = add2(y[0][0], y[0][1]);
+      y[1][0] = add2(y[1][0], y[1][1]);
+      const float seen = fold8(lo2(y[0][0]) + hi2(y[0][0]), lo2(y[1][0]) + hi2(y[1][0]), up);
+      const float o = fold8(o0, o1, up);
       if (pending) {
         if (writes) *op = o;
         op += ostep;
       }
       pending = true;
       float c = seen;                               // general: n^T S of this lane's column
-      if (!GENERAL) c = vs[kCols] * (vs[cb + my] - seen);
-      const int half = lane & 16;
-      const float u0 = __shfl_sync(0xffffffffu, c, half);
-      const float u1 = __shfl_sync(0xffffffffu, c, half | 4);
-      const float u2 = __shfl_sync(0xffffffffu, c, half | 8);
-      const float u3 = __shfl_sync(0xffffffffu, c, half | 12);
-      float4 vv;
-      if (GENERAL) vv = *reinterpret_cast<const float4*>(vs + cb);
-      o0 = o1 = o2 = o3 = 0.f;
+      if (!GENERAL) c = vs[kCols] * (vs[cb + (up ? 1 : 0)] - seen);
+      const float other = __shfl_xor_sync(0xffffffffu, c, 4);
+      const float u0 = up ? other : c, u1 = up ? c : other;
+      f2 uu[2], vv[2];
+      if (GENERAL) {
+        const float2 v2 = *reinterpret_cast<const float2*>(vs + cb);
+        uu[0] = pack2(-u0, -u0); uu[1] = pack2(-u1, -u1);
+        vv[0] = pack2(v2.x, v2.x); vv[1] = pack2(v2.y, v2.y);
+      } else {
+        uu[0] = pack2(u0, u0); uu[1] = pack2(u1, u1);
+      }
+      f2 oo[2][2] = {{0ull, 0ull}, {0ull, 0ull}};
 #pragma unroll
       for (int j = 0; j < NG; ++j) {
-        const int r0 = (j * 16 + rl) * W;
-        float k[W], q[W];
-        lds_vec<W>(k, base + DP + r0);
-        lds_vec<W>(q, base + 2 * DP + r0);
+        const int r0 = (j * 8 + kq) * 4;
+        f2 k[2], q[2], g[2], p[2];
+        lds_vec(k, base + DP + r0);
+        lds_vec(q, base + 2 * DP + r0);
         if (GENERAL) {
-          float g[W], p[W];
-          lds_vec<W>(g, base + r0);
-          lds_vec<W>(p, base + 4 * DP + r0);
-#pragma unroll
-          for (int e = 0; e < W; ++e) {
-            float* x = S[j * W + e];
-            x[0] = fmaf(k[e], vv.x, fmaf(-p[e], u0, g[e] * x[0]));
-            x[1] = fmaf(k[e], vv.y, fmaf(-p[e], u1, g[e] * x[1]));
-            x[2] = fmaf(k[e], vv.z, fmaf(-p[e], u2, g[e] * x[2]));
-            x[3] = fmaf(k[e], vv.w, fmaf(-p[e], u3, g[e] * x[3]));
-          }
-        } else {
-#pragma unroll
-          for (int e = 0; e < W; ++e) {
-            float* x = S[j * W + e];
-            x[0] = fmaf(k[e], u0, x[0]); x[1] = fmaf(k[e], u1, x[1]);
-            x[2] = fmaf(k[e], u2, x[2]); x[3] = fmaf(k[e], u3, x[3]);
-          }
+          lds_vec(g, base + r0);
+          lds_vec(p, base + 4 * DP + r0);
         }
 #pragma unroll
-        for (int e = 0; e < W; ++e) {
-          const float* x = S[j * W + e];
-          o0 = fmaf(x[0], q[e], o0); o1 = fmaf(x[1], q[e], o1);
-          o2 = fmaf(x[2], q[e], o2); o3 = fmaf(x[3], q[e], o3);
-        }
+        for (int e = 0; e < 2; ++e)
+#pragma unroll
+          for (int c = 0; c < 2; ++c) {
+            f2& x = S[j * 2 + e][c];
+            if (GENERAL) x = fma2(k[e], vv[c], fma2(p[e], uu[c], mul2(g[e], x)));
+            else x = fma2(k[e], uu[c], x);
+            oo[c][e] = fma2(x, q[e], oo[c][e]);
+          }
       }
+      oo[0][0] = add2(oo[0][0], oo[0][1]);
+      oo[1][0] = add2(oo[1][0], oo[1][1]);
+      o0 = lo2(oo[0][0]) + hi2(oo[0][0]);
+      o1 = lo2(oo[1][0]) + hi2(oo[1][0]);
     }
   }
-  const float o = fold16(o0, o1, o2, o3, lane);
+  const float o = fold8(o0, o1, up);
   if (writes) *op = o;
 #pragma unroll
   for (int j = 0; j < NG; ++j)
 #pragma unroll
-    for (int e = 0; e < W; ++e) {
-      const int row = (j * 16 + rl) * W + e;
+    for (int e = 0; e < 4; ++e) {
+      const int row = (j * 8 + kq) * 4 + e;
       if (row >= a.D) continue;
       float* p = Sg + (long long)row * a.V;
-      const float* x = S[j * W + e];
-      if (wide) {
-        if (col0 + cb < a.V) *reinterpret_cast<float4*>(p) = make_float4(x[0], x[1], x[2], x[3]);
+      const f2 s0 = S[j * 2 + e / 2][0], s1 = S[j * 2 + e / 2][1];
+      const float x0 = (e & 1) ? hi2(s0) : lo2(s0), x1 = (e & 1) ? hi2(s1) : lo2(s1);
+      if (wide && c0ok) {
+        *reinterpret_cast<float2*>(p) = make_float2(x0, x1);
       } else {
-        for (int i = 0; i < 4; ++i)
-          if (col0 + cb + i < a.V) p[i] = x[i];
+        if (c0ok) p[0] = x0;
+        if (c1ok) p[1] = x1;
       }
     }
 }
@@ -703,7 +808,7 @@ int step_impl(const StepArgs& a, int B, cudaStream_t stream) {
 
 template <int DP, bool GENERAL>
 int launch_rule(const RuleArgs& a, int B, cudaStream_t stream) {
-  constexpr size_t smem = 2 * Stage<DP, GENERAL>::kFloats * sizeof(float);
+  constexpr size_t smem = kRuleBufs * Stage<DP, GENERAL>::kFloats * sizeof(float);
   static bool configured = false;
   if (!configured && smem > 48 * 1024) {
     US_CUDA_CHECK(cudaFuncSetAttribute(vector_delta_kernel<DP, GENERAL>,
@@ -738,8 +843,14 @@ US_API int us_channel_delta_prep(const void* x, long long ldx, int off_q, int of
   cudaStream_t stream = (cudaStream_t)stream_;
   const int per = one_token ? 1 : kPrepTokens;
   const int units = 2 * Hk + 2 * H;
-  US_CUDA_CHECK(us::launch_pdl(channel_prep_kernel, dim3((rows + per - 1) / per, (units + 7) / 8),
-                               dim3(256), 0, stream, a));
+  const dim3 grid((rows + per - 1) / per, (units + 7) / 8);
+  const int widest = D > V ? D : V;
+#define US_PREP(KT)                                                                               \
+  if (widest <= 64) US_CUDA_CHECK(us::launch_pdl(channel_prep_kernel<KT, 2>, grid, dim3(256), 0, stream, a));       \
+  else if (widest <= 128) US_CUDA_CHECK(us::launch_pdl(channel_prep_kernel<KT, 4>, grid, dim3(256), 0, stream, a)); \
+  else US_CUDA_CHECK(us::launch_pdl(channel_prep_kernel<KT, 8>, grid, dim3(256), 0, stream, a));
+  if (K <= 4) { US_PREP(4) } else { US_PREP(8) }
+#undef US_PREP
   if (!one_token && K > 1)
     US_CUDA_CHECK(us::launch_pdl(conv_ring_kernel, dim3((2 * Hk * D + H * V + 255) / 256, B),
                                  dim3(256), 0, stream, a));
@@ -776,7 +887,7 @@ US_API int us_vector_delta_rule(int general, const float* q, const float* k, con
   cudaStream_t stream = (cudaStream_t)stream_;
 #define US_VD(DP) \
   if (D <= DP) return general ? launch_rule<DP, true>(a, B, stream) : launch_rule<DP, false>(a, B, stream);
-  US_VD(16) US_VD(32) US_VD(64) US_VD(128) US_VD(256)
+  US_VD(32) US_VD(64) US_VD(128) US_VD(256)
 #undef US_VD
   return US_ERR_UNSUPPORTED;
 }
