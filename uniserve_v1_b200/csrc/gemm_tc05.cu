@@ -23,7 +23,7 @@
 
 namespace {
 
-template <int BN, bool DUAL>
+template <int BN, bool DUAL, bool GELU>
 __global__ void __launch_bounds__(192)
 gemm_wx_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ BMaps tmBs,
                const GemmArgs args) {
@@ -194,7 +194,7 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
         }
       } else {
         // The pipeline stages are idle: their first 16 KiB stage the stores.
-        Epilogue<DUAL> epi(args, group, m_tile * kBlockM, ml, row0);
+        Epilogue<DUAL, GELU> epi(args, group, m_tile * kBlockM, ml, row0);
         int chunk = 0;
 #pragma unroll 1
         for (int c = 0; c < BN; c += 16, ++chunk) {
@@ -218,7 +218,7 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
       const int q = warp & 3;
       const int ml = q * 32 + lane;
       const uint32_t my_rank = tc::cluster_ctarank();
-      Epilogue<false> epi(args, group, m_tile * kBlockM, ml, row0);
+      Epilogue<false, GELU> epi(args, group, m_tile * kBlockM, ml, row0);
       const uint32_t local = tc::smem_u32(smem) + (uint32_t)ml * 4u;
       for (int r = (int)my_rank; r < nrows; r += args.splits) {
         float acc = 0.f;
@@ -469,7 +469,7 @@ __device__ __forceinline__ void swapped_tile(int t, int m_pairs, int n_tiles, in
 // per CTA) and every epilogue thread owns one activation row, whose features it
 // stores from registers as 32-byte pieces - no staging tile, and every destination
 // (plain, row-mapped, a peer's buffer by feature block or by row interval, the
-// token owner's combine buffer) is one pointer per thread.  SWAP = 2 (dense): the
+// token owner's combine buffer) is one pointer per thread.  SWAP = 2 (dense; 3: with gelu): the
 // other side is 256 weight rows, 128 per CTA.  SWAP = 1 (gated): 128 value rows in
 // the even CTA and the matching 128 gate rows in the odd CTA, so one N = 256
 // instruction produces both halves and a thread finds value j in column j and its
@@ -515,7 +515,7 @@ gemm_wx_pair_kernel(const __grid_constant__ CUtensorMap tmA,
     return grouped ? args.tile_row0[mp] + (int)rank * kBlockM : (2 * mp + (int)rank) * kBlockM;
   };
   auto b_off_of = [&](int mp) -> int { return grouped ? args.tile_group[mp] * args.group_rows : 0; };
-  constexpr int kFeat = SWAP == 2 ? 2 * kBlockM : kBlockM;   // features per swapped tile
+  constexpr int kFeat = SWAP >= 2 ? 2 * kBlockM : kBlockM;   // features per swapped tile
   const int n_tiles = SWAP ? (args.M + kFeat - 1) / kFeat : (args.rows + BN - 1) / BN;
   const int total = m_pairs * n_tiles;
   const int num_k = (args.K + kKC * kBK - 1) / (kKC * kBK);   // stages of K
@@ -574,7 +574,7 @@ gemm_wx_pair_kernel(const __grid_constant__ CUtensorMap tmA,
         if (SWAP) swapped_tile(t, m_pairs, n_tiles, mp, nt);
         const int m_tile = 2 * mp + (int)rank;
         const int row0 = SWAP == 1   ? nt * kBlockM + (rank ? args.dual_offset : 0)
-                         : SWAP == 2 ? nt * kFeat + (int)rank * kBlockM
+                         : SWAP >= 2 ? nt * kFeat + (int)rank * kBlockM
                                      : nt * BN + (int)rank * (BN / 2);
         const int a_row = SWAP ? a_row_of(mp) : 0;
         const int b_off = SWAP ? b_off_of(mp) : 0;
@@ -787,7 +787,7 @@ gemm_wx_pair_kernel(const __grid_constant__ CUtensorMap tmA,
               if (f0 + c + j < M)
                 x[j] += bias_f ? bias_f[f0 + c + j] : us::bf2f(bias_h[f0 + c + j]);
           }
-          if (SWAP == 2 && act == 3) {
+          if (SWAP == 3) {
 #pragma unroll
             for (int j = 0; j < 16; ++j) x[j] = gelu_erf_f(x[j]);
           }
@@ -970,7 +970,7 @@ int launch_persist(const CUtensorMap& tmA, const BMaps& tmB, GemmArgs a, int til
 // Live CTAs expected of the next grouped launch of this thread (us_gemm_wx_hint); 0 = none.
 thread_local int g_cta_hint = 0;
 
-template <int BN, bool DUAL>
+template <int BN, bool DUAL, bool GELU = false>
 int launch(const CUtensorMap& tmA, const BMaps& tmB, GemmArgs a, int m_tiles, int n_tiles,
            cudaStream_t stream) {
   constexpr int kBTile = BN * kBlockK * 2;
@@ -1038,7 +1038,7 @@ int launch(const CUtensorMap& tmA, const BMaps& tmB, GemmArgs a, int m_tiles, in
   const size_t smem = (size_t)stages * kStageBytes + (2 * stages + 1) * 8 + 16 + 1024;
   static bool configured = false;
   if (!configured) {
-    US_CUDA_CHECK(cudaFuncSetAttribute(gemm_wx_kernel<BN, DUAL>,
+    US_CUDA_CHECK(cudaFuncSetAttribute(gemm_wx_kernel<BN, DUAL, GELU>,
                                        cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
     configured = true;
   }
@@ -1059,7 +1059,7 @@ int launch(const CUtensorMap& tmA, const BMaps& tmB, GemmArgs a, int m_tiles, in
   attr[1].val.programmaticStreamSerializationAllowed = us::pdl_enabled() ? 1 : 0;
   cfg.attrs = attr;
   cfg.numAttrs = 2;
-  US_CUDA_CHECK(cudaLaunchKernelEx(&cfg, gemm_wx_kernel<BN, DUAL>, tmA, tmB, a));
+  US_CUDA_CHECK(cudaLaunchKernelEx(&cfg, gemm_wx_kernel<BN, DUAL, GELU>, tmA, tmB, a));
   return US_OK;
 }
 
@@ -1116,7 +1116,9 @@ int gemm_impl(const void* W, const void* X, void* out, int G, int w_rows, int M,
   if (num_tiles) US_REQUIRE(tile_group && tile_row0 && tile_rows && max_tiles >= 1);
 
   // Dense problems of more than one wave run on CTA pairs (US_GEMM_PAIR=0: single CTAs).
-  const bool pair = pair_enabled() && num_tiles == nullptr && G == 1 && !ps.x_peers &&
+  const bool gelu = !dual && act == 3;    // single-CTA and swapped kernels only
+  US_REQUIRE(dual || act == 0 || gelu);
+  const bool pair = pair_enabled() && (!gelu || pair_mode() == 1) && num_tiles == nullptr && G == 1 && !ps.x_peers &&
                     (K % kBlockK) == 0 &&
                     (dual ? block_n == 128 : block_n == 256) &&
                     (long long)((M + kBlockM - 1) / kBlockM) * ((x_rows + block_n - 1) / block_n) >
@@ -1126,9 +1128,9 @@ int gemm_impl(const void* W, const void* X, void* out, int G, int w_rows, int M,
   const bool gpair = pair_enabled() && pair_mode() == 1 && num_tiles != nullptr && block_n == 256 &&
                      !ps.x_peers && !ps.out_peers && (K % kBlockK) == 0 && bias == nullptr &&
                      ldw == K;
-  const uint32_t box_n = (uint32_t)(pair ? block_n / 2 : block_n);
   // operands swapped: one activation row per epilogue thread
   const bool swap = (pair && pair_mode() == 1) || gpair;
+  const uint32_t box_n = (uint32_t)(pair ? block_n / 2 : block_n);
 
   CUtensorMap tmA;
   BMaps tmB;
@@ -1272,6 +1274,7 @@ int gemm_impl(const void* W, const void* X, void* out, int G, int w_rows, int M,
     const int x_pairs = gpair ? max_tiles : ((x_rows + kBlockM - 1) / kBlockM + 1) / 2;
     if (dual)
       return launch_pair<256, false, false, 1>(tmA, tmB, a, x_pairs * ((M + 127) / 128), stream);
+    if (gelu) return launch_pair<256, false, false, 3>(tmA, tmB, a, x_pairs * ((M + 255) / 256), stream);
     return launch_pair<256, false, false, 2>(tmA, tmB, a, x_pairs * ((M + 255) / 256), stream);
   }
   if (pair) {
@@ -1279,7 +1282,7 @@ int gemm_impl(const void* W, const void* X, void* out, int G, int w_rows, int M,
     if (dual) return launch_pair<128, true>(tmA, tmB, a, pair_tiles, stream);
     return launch_pair<256, false>(tmA, tmB, a, pair_tiles, stream);
   }
-  if (!no_persist && num_tiles == nullptr && G == 1 && m_tiles * n_tiles > 148 &&
+  if (!no_persist && !gelu && num_tiles == nullptr && G == 1 && m_tiles * n_tiles > 148 &&
       (dual ? block_n == 128 : (block_n == 128 || block_n == 256))) {
     const int tiles = m_tiles * n_tiles;
     if (dual) return launch_persist<128, true>(tmA, tmB, a, tiles, stream);
@@ -1288,8 +1291,9 @@ int gemm_impl(const void* W, const void* X, void* out, int G, int w_rows, int M,
   }
 #define US_GEMM_CASE(BN)                                                              \
   case BN:                                                                            \
-    return dual ? launch<BN, true>(tmA, tmB, a, m_tiles, n_tiles, stream)             \
-                : launch<BN, false>(tmA, tmB, a, m_tiles, n_tiles, stream);
+    return dual   ? launch<BN, true>(tmA, tmB, a, m_tiles, n_tiles, stream)             \
+           : gelu ? launch<BN, false, true>(tmA, tmB, a, m_tiles, n_tiles, stream)      \
+                  : launch<BN, false>(tmA, tmB, a, m_tiles, n_tiles, stream);
   switch (block_n) {
     US_GEMM_CASE(16)
     US_GEMM_CASE(32)

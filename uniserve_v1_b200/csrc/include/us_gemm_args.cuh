@@ -105,7 +105,9 @@ constexpr int kEpiStageBytes = 16 * 1024;   // two staging tiles of 16 rows x 12
 // so that every row leaves as contiguous 16-byte pieces (256 B per row for bf16)
 // whatever the destination: the plain output, a row-mapped output, a peer's buffer
 // (scatter by feature, reduce-scatter by row) or the token owner's combine buffer.
-template <bool DUAL>
+// GELU: gelu (erf) of the biased value, a form of its own so that the other products' epilogues
+// do not carry its code.
+template <bool DUAL, bool GELU = false>
 struct Epilogue {
   // Everything the per-element code needs is copied out of the argument block
   // once: the block lives in parameter memory, and reading it per element (after
@@ -173,7 +175,7 @@ struct Epilogue {
       }
     }
     val += bias;
-    if (!DUAL && act == 3) val = gelu_erf_f(val);
+    if (GELU) val = gelu_erf_f(val);
     if (route_rows != nullptr) return val * route_w[route_rows[r]];
     if (scale_rows != nullptr && !scale_first) val *= scale_rows[r];
     return val;
@@ -216,7 +218,7 @@ struct Epilogue {
     }
     const uint32_t buf = tc::smem_u32(stage) + (uint32_t)(chunk & 1) * (kEpiStageBytes / 2);
     // fast path: nothing per row but the gated activation and the bias
-    const bool plain = scale_rows == nullptr && route_rows == nullptr && (DUAL || act == 0);
+    const bool plain = scale_rows == nullptr && route_rows == nullptr && !GELU;
     if (esz == 2) {
 #pragma unroll
       for (int j = 0; j < 16; ++j) {

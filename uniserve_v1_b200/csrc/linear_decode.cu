@@ -57,12 +57,12 @@ __device__ __forceinline__ float gelu_erf(float x) {
 }
 
 // MT = 16-row tiles of the activation (rows <= 16 * MT).
-template <int MT>
+template <int MT, bool GELU>
 __global__ void __launch_bounds__(256)
 linear_decode_kernel(const __nv_bfloat16* __restrict__ W, const __nv_bfloat16* __restrict__ X,
                      void* __restrict__ out, const void* __restrict__ bias, int rows, int M, int K,
                      long long ldw, long long ldx, long long ldo, int out_f32, int bias_f32,
-                     int ksplit, int act) {
+                     int ksplit) {
   // Weights are never written by a kernel: the first loads go out before the wait on the
   // kernels that produce the activation.
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
@@ -185,7 +185,7 @@ linear_decode_kernel(const __nv_bfloat16* __restrict__ W, const __nv_bfloat16* _
         if (bias)
           v += bias_f32 ? reinterpret_cast<const float*>(bias)[col]
                         : us::bf2f(reinterpret_cast<const __nv_bfloat16*>(bias)[col]);
-        if (act == 3) v = gelu_erf(v);
+        if (GELU) v = gelu_erf(v);
         if (out_f32)
           reinterpret_cast<float*>(out)[(long long)r * ldo + col] = v;
         else
@@ -205,7 +205,7 @@ linear_decode_kernel(const __nv_bfloat16* __restrict__ W, const __nv_bfloat16* _
     if (bias)
       v += bias_f32 ? reinterpret_cast<const float*>(bias)[col]
                     : us::bf2f(reinterpret_cast<const __nv_bfloat16*>(bias)[col]);
-    if (act == 3) v = gelu_erf(v);
+    if (GELU) v = gelu_erf(v);
     if (out_f32)
       reinterpret_cast<float*>(out)[(long long)r * ldo + col] = v;
     else
@@ -230,12 +230,12 @@ US_API int us_linear_decode(const void* W, const void* X, void* out, const void*
   const __nv_bfloat16* x = (const __nv_bfloat16*)X;
   static bool configured = false;
   if (!configured) {
-    US_CUDA_CHECK(cudaFuncSetAttribute(linear_decode_kernel<4>,
-                                       cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                       4 * kStages * 8192));
-    US_CUDA_CHECK(cudaFuncSetAttribute(linear_decode_kernel<2>,
-                                       cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                       2 * kStages * 8192));
+    for (auto k : {linear_decode_kernel<4, false>, linear_decode_kernel<4, true>})
+      US_CUDA_CHECK(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                         4 * kStages * 8192));
+    for (auto k : {linear_decode_kernel<2, false>, linear_decode_kernel<2, true>})
+      US_CUDA_CHECK(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                         2 * kStages * 8192));
     configured = true;
   }
   // K split over a cluster when one CTA per 16 features would leave most SMs idle
@@ -271,14 +271,16 @@ US_API int us_linear_decode(const void* W, const void* X, void* out, const void*
     cfg.attrs = attr;
     cfg.numAttrs = ksplit > 1 ? 2 : 1;
     return cudaLaunchKernelEx(&cfg, kernel, w, x, out, bias, rows, M, K, ldw, ldx, ldo, out_f32,
-                              bias_f32, ksplit, act);
+                              bias_f32, ksplit);
   };
   // kStages buffers x (16 MT) rows x 512 bytes
+  US_REQUIRE(act == 0 || act == 3);
+  const bool gelu = act == 3;
   if (rows <= 16)
-    US_CUDA_CHECK(launch(linear_decode_kernel<1>, kStages * 8192));
+    US_CUDA_CHECK(launch(gelu ? linear_decode_kernel<1, true> : linear_decode_kernel<1, false>, kStages * 8192));
   else if (rows <= 32)
-    US_CUDA_CHECK(launch(linear_decode_kernel<2>, 2 * kStages * 8192));
+    US_CUDA_CHECK(launch(gelu ? linear_decode_kernel<2, true> : linear_decode_kernel<2, false>, 2 * kStages * 8192));
   else
-    US_CUDA_CHECK(launch(linear_decode_kernel<4>, 4 * kStages * 8192));
+    US_CUDA_CHECK(launch(gelu ? linear_decode_kernel<4, true> : linear_decode_kernel<4, false>, 4 * kStages * 8192));
   return US_OK;
 }
