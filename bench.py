@@ -672,7 +672,7 @@ def nepevik_record(job: Job) -> dict:
         sp = SamplingParams(temperature=0.0, max_tokens=K + W + 12, ignore_eos=True)
         eng = make_engine(n, length)
         run = getattr(eng, "scheduler", eng)
-        for p in prompts(min(n, max(1, 8192 // length)), length):    # warm-up at the batch's size
+        for p in prompts(n, length):        # warm-up: the whole batch once (allocator, graphs)
             eng.add_request(p, SamplingParams(temperature=0.0, max_tokens=4, ignore_eos=True))
         while eng.has_work():
             eng.step()

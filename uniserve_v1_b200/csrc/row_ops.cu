@@ -147,32 +147,54 @@ struct RowNormKv {
   int bf16;
 };
 
+// Both sums in one pass over the row and one exchange.  VEC: every width is a multiple of 4.
+template <bool VEC>
 __global__ void __launch_bounds__(kThreads) row_norm_kv_kernel(const RowNormKv a) {
   US_PDL_PROLOGUE();
-  __shared__ float scratch[33];
+  constexpr int U = VEC ? 4 : 1;
+  __shared__ float2 part[kThreads / 32];
   const long long base = (long long)blockIdx.x * a.ldx;
+  const int tid = threadIdx.x;
+  auto load = [&](long long i) -> float4 {
+    return VEC ? ld4(a.x, base + i, a.bf16) : make_float4(ld1(a.x, base + i, a.bf16), 0.f, 0.f, 0.f);
+  };
+  auto weight = [&](const float* w, int c) -> float4 {
+    return VEC ? *reinterpret_cast<const float4*>(w + c) : make_float4(w[c], 0.f, 0.f, 0.f);
+  };
+  auto store = [&](void* dst, long long i, float4 v) {
+    if (VEC) st4(dst, i, a.bf16, v);
+    else st1(dst, i, a.bf16, v.x);
+  };
+  const long long slot = a.nk ? a.slots[blockIdx.x] : -1;
   float sq = 0.f, sk = 0.f;
-  for (int c = threadIdx.x; c < a.nq; c += kThreads) {
-    const float v = ld1(a.x, base + a.off_q + c, a.bf16);
-    sq += v * v;
+  for (int c = tid * U; c < a.nq; c += kThreads * U) sq += sq4(load(a.off_q + c));
+  for (int c = tid * U; c < a.nk; c += kThreads * U) sk += sq4(load(a.off_k + c));
+  sq = us::warp_sum(sq);
+  sk = us::warp_sum(sk);
+  if ((tid & 31) == 0) part[tid >> 5] = make_float2(sq, sk);
+  __syncthreads();
+  sq = sk = 0.f;
+#pragma unroll
+  for (int w = 0; w < kThreads / 32; ++w) {
+    sq += part[w].x;
+    sk += part[w].y;
   }
-  for (int c = threadIdx.x; c < a.nk; c += kThreads) {
-    const float v = ld1(a.x, base + a.off_k + c, a.bf16);
-    sk += v * v;
-  }
-  sq = us::block_sum(sq, scratch);
   const float iq = 1.f / sqrtf(sq / (float)a.nq + a.eps);
-  for (int c = threadIdx.x; c < a.nq; c += kThreads)
-    st1(a.x, base + a.off_q + c, a.bf16, ld1(a.x, base + a.off_q + c, a.bf16) * iq * a.wq[c]);
-  if (a.nk == 0) return;
-  sk = us::block_sum(sk, scratch);
-  const long long slot = a.slots[blockIdx.x];
+  for (int c = tid * U; c < a.nq; c += kThreads * U) {
+    float4 v = load(a.off_q + c);
+    const float4 w = weight(a.wq, c);
+    v.x *= iq * w.x; v.y *= iq * w.y; v.z *= iq * w.z; v.w *= iq * w.w;
+    store(a.x, base + a.off_q + c, v);
+  }
   if (slot < 0) return;
   const float ik = 1.f / sqrtf(sk / (float)a.nk + a.eps);
-  for (int c = threadIdx.x; c < a.nk; c += kThreads)
-    st1(a.kc, slot * a.nk + c, a.bf16, ld1(a.x, base + a.off_k + c, a.bf16) * ik * a.wk[c]);
-  for (int c = threadIdx.x; c < a.nv; c += kThreads)
-    st1(a.vc, slot * a.nv + c, a.bf16, ld1(a.x, base + a.off_v + c, a.bf16));
+  for (int c = tid * U; c < a.nk; c += kThreads * U) {
+    float4 v = load(a.off_k + c);
+    const float4 w = weight(a.wk, c);
+    v.x *= ik * w.x; v.y *= ik * w.y; v.z *= ik * w.z; v.w *= ik * w.w;
+    store(a.kc, slot * a.nk + c, v);
+  }
+  for (int c = tid * U; c < a.nv; c += kThreads * U) store(a.vc, slot * a.nv + c, load(a.off_v + c));
 }
 
 // tanh over a column range of the rows, in place.
@@ -225,8 +247,10 @@ US_API int us_row_norm_kv(void* x, long long ldx, int off_q, int off_k, int off_
   US_REQUIRE(nk == 0 || (nv >= 1 && wk && slots && kc && vc));
   if (T == 0) return US_OK;
   RowNormKv a{x, ldx, off_q, off_k, off_v, nq, nk, nv, wq, wk, slots, kc, vc, eps, bf16};
-  US_CUDA_CHECK(us::launch_pdl(row_norm_kv_kernel, dim3(T), dim3(kThreads), 0,
-                               (cudaStream_t)stream_, a));
+  const bool vec = ((nq | nk | nv | off_q | off_k | off_v) & 3) == 0 && (ldx & 3) == 0 &&
+                   (((uintptr_t)x | (uintptr_t)kc | (uintptr_t)vc | (uintptr_t)wq | (uintptr_t)wk) % 16) == 0;
+  US_CUDA_CHECK(us::launch_pdl(vec ? row_norm_kv_kernel<true> : row_norm_kv_kernel<false>, dim3(T),
+                               dim3(kThreads), 0, (cudaStream_t)stream_, a));
   return US_OK;
 }
 
