@@ -346,7 +346,7 @@ def to(form, t):
 
 @pytest.mark.parametrize("form", FORMS)
 @pytest.mark.parametrize("H,Hk,D,V,K", [(2, 2, 16, 32, 4), (6, 2, 24, 40, 3), (4, 1, 128, 64, 2),
-                                        (3, 3, 65, 33, 1), (2, 1, 200, 8, 8), (4, 2, 64, 128, 5)])
+                                        (3, 3, 65, 33, 1), (2, 1, 200, 8, 8), (4, 2, 64, 128, 5), (2, 2, 32, 48, 11)])
 def test_channel_delta_alone(form, H, Hk, D, V, K):
     """Convolution windows, unit vectors, decay, step size and state over a packed batch run in
     pieces, with a padding sequence and slots out of order."""
@@ -439,7 +439,7 @@ def test_head_norm_gate_alone(form, shared):
 @pytest.mark.gpu
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16], ids=["f32", "bf16"])
 @pytest.mark.parametrize("H,Hk,D,V,K", [(4, 2, 128, 128, 4), (2, 1, 64, 256, 2), (3, 3, 16, 8, 1),
-                                        (6, 2, 100, 68, 8)])
+                                        (6, 2, 100, 68, 8), (2, 1, 32, 32, 12)])
 def test_one_launch_decode_step_equals_the_separate_kernels(H, Hk, D, V, K, dtype):
     """Tokens of several sequences at different positions (one of them fresh, one row padding)."""
     g, dev, eps = gen(D), "cuda", 1e-4
@@ -501,7 +501,10 @@ def paged(k, v, starts_free, page, dev, dtype, g):
 @pytest.mark.parametrize("H,G,D,V,size,keep", [(4, 2, 32, 24, 20, 3), (6, 2, 20, 28, 17, 0),
                                                (8, 8, 64, 64, 33, 40), (2, 1, 128, 16, 0, 0),
                                                (3, 3, 80, 130, 1, 2), (16, 4, 128, 128, 48, 4),
-                                               (32, 4, 64, 64, 100, 2), (8, 2, 128, 128, 0, 0)])
+                                               (32, 4, 64, 64, 100, 2), (8, 2, 128, 128, 0, 0),
+                                               (6, 2, 48, 96, 25, 7), (12, 3, 40, 72, 30, 2),
+                                               (24, 8, 96, 104, 60, 16), (40, 4, 32, 40, 12, 1),
+                                               (32, 8, 128, 128, 21, 3), (5, 1, 64, 8, 150, 4)])
 def test_mixed_head_attention_alone(form, H, G, D, V, size, keep):
     """Random keys plus, per probed query, one key whose score stands out: just inside and just
     outside the window, the last kept key and the next one, page borders, far away."""

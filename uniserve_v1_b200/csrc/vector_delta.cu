@@ -55,7 +55,7 @@ __device__ __forceinline__ int seq_of(const int* cu, int B, int t) {
   return lo;
 }
 
-constexpr int kMaxTaps = 8;
+constexpr int kMaxTaps = 16;
 constexpr int kMaxDim = 256;      // key channels per head
 constexpr int kPrepTokens = 16;   // consecutive rows of one warp in the prefill form
 
@@ -849,7 +849,7 @@ US_API int us_channel_delta_prep(const void* x, long long ldx, int off_q, int of
   if (widest <= 64) US_CUDA_CHECK(us::launch_pdl(channel_prep_kernel<KT, 2>, grid, dim3(256), 0, stream, a));       \
   else if (widest <= 128) US_CUDA_CHECK(us::launch_pdl(channel_prep_kernel<KT, 4>, grid, dim3(256), 0, stream, a)); \
   else US_CUDA_CHECK(us::launch_pdl(channel_prep_kernel<KT, 8>, grid, dim3(256), 0, stream, a));
-  if (K <= 4) { US_PREP(4) } else { US_PREP(8) }
+  if (K <= 4) { US_PREP(4) } else if (K <= 8) { US_PREP(8) } else { US_PREP(16) }
 #undef US_PREP
   if (!one_token && K > 1)
     US_CUDA_CHECK(us::launch_pdl(conv_ring_kernel, dim3((2 * Hk * D + H * V + 255) / 256, B),
