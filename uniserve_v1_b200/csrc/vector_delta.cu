@@ -22,7 +22,7 @@
 // columns of S in registers as row pairs (packed FP32 instructions), so the two D-long reductions
 // of a token are short chains and three shuffles; the read-out's is folded beside the next token's
 // first one.  A token depends on the one before through one reduction and one update: that chain
-// is what a long prompt costs.  The vectors of the next rounds of 8 tokens are on their way into
+// is what a long prompt costs.  The vectors of the next chunks of 8 tokens are on their way into
 // a ring in shared memory meanwhile (four warps multiply, one fetches).  The state crosses HBM once per call.
 #include "include/us_common.cuh"
 
@@ -255,7 +255,7 @@ __global__ void __launch_bounds__(256) general_prep_kernel(const GeneralPrep a) 
 constexpr int kCols = 32;         // value columns per CTA
 constexpr int kRuleCompute = 128, kRuleCopy = 32;    // threads that multiply / that fetch vectors
 constexpr int kRuleThreads = kRuleCompute + kRuleCopy;
-constexpr int kRuleBufs = 4;                         // rounds of vectors in shared memory
+constexpr int kRuleBufs = 4;                         // chunks of vectors in shared memory
 
 struct RuleArgs {
   const float *q, *k, *v;         // [rows, Hk, D] x 2, [rows, H, V]
@@ -322,7 +322,7 @@ template <int DP, bool GENERAL>
 struct Stage {
   static constexpr int kVecs = GENERAL ? 5 : 3;
   static constexpr int kToken = kVecs * DP + kCols + 4;
-  static constexpr int kChunk = 8;                    // tokens per round
+  static constexpr int kChunk = 8;                    // tokens per chunk
   static constexpr int kFloats = kChunk * kToken;
 };
 
@@ -425,12 +425,12 @@ __global__ void __launch_bounds__(kRuleThreads, DP > 128 ? 1 : 3) vector_delta_k
     for (int e = tid; e < kRuleBufs * St::kFloats; e += kRuleThreads) sm[e] = 0.f;
     __syncthreads();
   }
-  if (tid >= kRuleCompute) {                          // the copying threads stay one round ahead
+  if (tid >= kRuleCompute) {                          // the copying threads stay one chunk ahead
     Copier<DP, GENERAL> cp;
     cp.init(a, tid - kRuleCompute, start, h, hk, col0);
-    const int rounds = (T + St::kChunk - 1) / St::kChunk;
+    const int chunks = (T + St::kChunk - 1) / St::kChunk;
     auto fetch = [&](int r) {                         // (an empty group past the end)
-      if (r < rounds)
+      if (r < chunks)
         cp.fetch(a, sm + (r % kRuleBufs) * St::kFloats, min(St::kChunk, T - r * St::kChunk),
                  start + r * St::kChunk, h, hk, col0);
       asm volatile("cp.async.commit_group;" ::: "memory");
@@ -438,9 +438,9 @@ __global__ void __launch_bounds__(kRuleThreads, DP > 128 ? 1 : 3) vector_delta_k
 #pragma unroll 1
     for (int r = 0; r < kRuleBufs - 1; ++r) fetch(r);
 #pragma unroll 1
-    for (int r = 0; r < rounds; ++r) {
+    for (int r = 0; r < chunks; ++r) {
       asm volatile("cp.async.wait_group %0;" ::"n"(kRuleBufs - 2) : "memory");
-      __syncthreads();                                // round r is there, round r - 1 consumed
+      __syncthreads();                                // chunk r is there, chunk r - 1 consumed
       fetch(r + kRuleBufs - 1);
     }
     return;
@@ -485,7 +485,7 @@ __global__ void __launch_bounds__(kRuleThreads, DP > 128 ? 1 : 3) vector_delta_k
   int buf = 0;
   for (int c0 = 0; c0 < T; c0 += St::kChunk, buf = buf + 1 == kRuleBufs ? 0 : buf + 1) {
     const int n = min(St::kChunk, T - c0);
-    __syncthreads();                                  // this round's vectors are there
+    __syncthreads();                                  // this chunk's vectors are there
     const float* base = sm + buf * St::kFloats;
     for (int t = 0; t < n; ++t, base += St::kToken) {
       const float* vs = base + St::kVecs * DP;
