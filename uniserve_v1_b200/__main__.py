@@ -20,6 +20,7 @@ def serve(args) -> int:
     import uvicorn
 
     from .checkpoint.safetensors_io import CheckpointLoader, resolve_family, resolve_hub
+    from .models.registry import named_family
     from .config.policy import Package
     from .server.app import create_app
 
@@ -66,8 +67,8 @@ def serve(args) -> int:
         family = "minimax_h3"
     elif pkg.model and "qwen4_exp" in pkg.model.lower():
         family = "qwen4_exp"
-    elif pkg.model and "nepevik" in pkg.model.lower():
-        family = "nepevik"
+    else:
+        family = named_family(pkg.model or "") or family
     name = pkg.served_model_name or (pkg.model or "model").split("/")[-1]
     shutdown = None
     if family == "minimax_h3":
@@ -494,8 +495,9 @@ def keep(args) -> int:
     if directory:
         from .checkpoint.safetensors_io import resolve_family
         family = resolve_family(directory)
-    elif "nepevik" in (pkg.model or "").lower():
-        family = "nepevik"
+    else:
+        from .models.registry import named_family
+        family = named_family(pkg.model or "") or family
     _cfg, model, _ld = _paged_model(pkg, family, directory, device, dtype, None)
     keeper = WeightsKeeper(model, args.socket)
 

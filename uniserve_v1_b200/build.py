@@ -46,6 +46,9 @@ GROUPS = {
     "nepevik": (("runtime.cu", "gemm_tc05.cu", "linear_decode.cu", "gemm_f32.cu", "moe_route.cu",
                  "misc.cu", "sampler.cu", "row_ops.cu", "vector_delta.cu", "head_mix_attn.cu"),
                 ("block_manager.cpp",)),
+    "zonopel": (("runtime.cu", "gemm_tc05.cu", "linear_decode.cu", "gemm_f32.cu", "misc.cu", "sampler.cu",
+                 "stream_rows.cu", "state_space.cu", "latent_attn.cu"),
+                ("block_manager.cpp",)),
 }
 CXX_FLAGS = ["-O3", "-std=c++17", "-fPIC", "-fvisibility=hidden", "-pthread", "-Wall"]
 

@@ -1,0 +1,358 @@
+// Rows of the FP32 residual stream between two sublayers, in one launch:
+//
+//   source   r(t) = rms(embed[id] * scale + table2[row]) * w              start of the stream
+//            r(t) = residual(t) + rms(y(t)) * w                           output norm and add
+//   output   h(t) = rms(r(t)) * w_out                                     input norm
+//            x(t) = h(t)   or   h(t) + (h(t - 1) - h(t)) * mu             token shift
+//
+// with rms(v) = v / sqrt(mean(v^2) + eps).  r goes to a second residual buffer (the one that is
+// read stays as it is), because a shifted row needs its neighbour's h: a CTA takes up to kRows
+// consecutive rows of one sequence and forms the row before its first one itself.  The h before a
+// sequence's first row of the batch comes from the state slot; the CTA that reads it also forms
+// the h of the sequence's last row and stores it there, so no other CTA meets the slot.
+//
+//   bigram_rows   table rows hashed from a token and the one before it (its own slot of state)
+//   poly_norm     a N(z) + b N(z^2) + c N(z^3) + e,  N(v) = v / sqrt(mean(v^2) + eps) over the row
+//
+// Rows are padded to a multiple of 8 columns with zeros; `width` is the true column count.
+// Element types: 1 = bf16, 0 = fp32.  All arithmetic is FP32.
+#include "include/us_common.cuh"
+
+namespace {
+
+constexpr int kRows = 8;          // rows of a sequence per CTA
+
+__device__ __forceinline__ float4 ld4(const void* base, long long i, int bf16) {
+  if (bf16) {
+    us::Pack8 p;
+    p.u = *reinterpret_cast<const uint2*>(reinterpret_cast<const __nv_bfloat16*>(base) + i);
+    return make_float4(us::bf2f(p.b[0]), us::bf2f(p.b[1]), us::bf2f(p.b[2]), us::bf2f(p.b[3]));
+  }
+  return *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(base) + i);
+}
+__device__ __forceinline__ void st4(void* base, long long i, int bf16, float4 v) {
+  if (bf16) {
+    us::Pack8 p;
+    p.b[0] = us::f2bf(v.x); p.b[1] = us::f2bf(v.y); p.b[2] = us::f2bf(v.z); p.b[3] = us::f2bf(v.w);
+    *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(base) + i) = p.u;
+  } else {
+    *reinterpret_cast<float4*>(reinterpret_cast<float*>(base) + i) = v;
+  }
+}
+__device__ __forceinline__ float sq4(float4 v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
+__device__ __forceinline__ float4 mul4(float4 a, float4 b, float s) {
+  return make_float4(a.x * s * b.x, a.y * s * b.y, a.z * s * b.z, a.w * s * b.w);
+}
+__device__ __forceinline__ float4 add4(float4 a, float4 b) {
+  return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w);
+}
+__device__ __forceinline__ float4 mix4(float4 h, float4 before, float4 mu) {
+  return make_float4(h.x + (before.x - h.x) * mu.x, h.y + (before.y - h.y) * mu.y,
+                     h.z + (before.z - h.z) * mu.z, h.w + (before.w - h.w) * mu.w);
+}
+
+// Sum over the block; `buf` holds 2 x 32 floats used in turns, so one barrier per sum suffices.
+__device__ __forceinline__ float turn_sum(float v, float* buf, int& turn) {
+  v = us::warp_sum(v);
+  float* b = buf + (turn ^= 32);
+  if ((threadIdx.x & 31) == 0) b[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float s = 0.f;
+  for (int w = 0; w < (int)(blockDim.x >> 5); ++w) s += b[w];
+  return s;
+}
+
+struct StreamRows {
+  const int *ids, *rows2;     // start of the stream: token ids, rows of the second table (or null)
+  const void *table, *table2;
+  float scale;
+  int vocab, n2;
+  const void* y;              // [T, W] sublayer output (null: start of the stream)
+  const float* residual;      // [T, W]
+  const float* w;             // [W]
+  float* residual_out;        // [T, W]
+  const float* w_out;         // [W]
+  const float* mu;            // [W] or null: no token shift
+  float* state;               // [slots, W]: h of a sequence's last token
+  const int *cu, *slots, *pos;
+  void* x;                    // [T, W]
+  int B, T, W, width, bf16, one_token;
+  float eps;
+  unsigned int* status;
+};
+
+template <int NV>
+__global__ void __launch_bounds__(256) stream_rows_kernel(const StreamRows a) {
+  US_PDL_PROLOGUE();
+  __shared__ float buf[64];
+  int turn = 0;
+  const int W = a.W, step = blockDim.x * 4, c0 = threadIdx.x * 4;
+  const float inv_n = 1.f / (float)a.width;
+  // rows of this CTA: t0 .. t1 of sequence s
+  int s = -1, t0, t1, start = 0, end = 0;
+  if (!a.mu) {
+    t0 = blockIdx.x * kRows;
+    t1 = min(a.T, t0 + kRows);
+  } else if (a.one_token) {
+    s = start = t0 = blockIdx.x;
+    end = t1 = t0 + 1;
+  } else {
+    int tile = blockIdx.x;
+    t0 = t1 = 0;
+    for (s = 0; s < a.B; ++s) {
+      start = a.cu[s];
+      end = a.cu[s + 1];
+      const int n = (end - start + kRows - 1) / kRows;
+      if (tile < n) {
+        t0 = start + tile * kRows;
+        t1 = min(end, t0 + kRows);
+        break;
+      }
+      tile -= n;
+    }
+    if (t0 == t1) return;
+  }
+  auto source = [&](int t, float4 (&v)[NV]) {
+    const long long base = (long long)t * W;
+    float ss = 0.f;
+    if (a.y) {
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int c = c0 + i * step;
+        v[i] = c < W ? ld4(a.y, base + c, a.bf16) : make_float4(0.f, 0.f, 0.f, 0.f);
+        ss += sq4(v[i]);
+      }
+    } else {
+      const int id = a.ids[t], r2 = a.rows2 ? a.rows2[t] : 0;
+      const bool ok = id >= 0 && id < a.vocab && r2 >= 0 && (!a.rows2 || r2 < a.n2);
+      if (!ok && threadIdx.x == 0) us_dev_fail(a.status, US_DEV_BOUNDS);
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int c = c0 + i * step;
+        v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (ok && c < W) {
+          const float4 e = ld4(a.table, (long long)id * W + c, a.bf16);
+          v[i] = make_float4(e.x * a.scale, e.y * a.scale, e.z * a.scale, e.w * a.scale);
+          if (a.rows2) v[i] = add4(v[i], ld4(a.table2, (long long)r2 * W + c, a.bf16));
+        }
+        ss += sq4(v[i]);
+      }
+    }
+    const float inv = 1.f / sqrtf(turn_sum(ss, buf, turn) * inv_n + a.eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = c0 + i * step;
+      if (c >= W) continue;
+      v[i] = mul4(v[i], *reinterpret_cast<const float4*>(a.w + c), inv);
+      if (a.y) v[i] = add4(v[i], *reinterpret_cast<const float4*>(a.residual + base + c));
+    }
+  };
+  auto norm = [&](float4 (&v)[NV]) {
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) ss += sq4(v[i]);
+    const float inv = 1.f / sqrtf(turn_sum(ss, buf, turn) * inv_n + a.eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = c0 + i * step;
+      if (c < W) v[i] = mul4(v[i], *reinterpret_cast<const float4*>(a.w_out + c), inv);
+    }
+  };
+  float4 before[NV];
+  float* kept = nullptr;            // this CTA's state slot (it holds the sequence's first row)
+  if (a.mu) {
+#pragma unroll
+    for (int i = 0; i < NV; ++i) before[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (t0 > start) {
+      source(t0 - 1, before);
+      norm(before);
+    } else if (a.slots[s] >= 0) {
+      kept = a.state + (long long)a.slots[s] * W;
+      if (a.pos[start] > 0) {
+#pragma unroll
+        for (int i = 0; i < NV; ++i)
+          if (c0 + i * step < W) before[i] = *reinterpret_cast<const float4*>(kept + c0 + i * step);
+      }
+    }
+  }
+  float4 v[NV];
+  for (int t = t0; t < t1; ++t) {
+    source(t, v);
+    const long long base = (long long)t * W;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = c0 + i * step;
+      if (c < W) *reinterpret_cast<float4*>(a.residual_out + base + c) = v[i];
+    }
+    norm(v);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = c0 + i * step;
+      if (c >= W) continue;
+      float4 o = v[i];
+      if (a.mu) {
+        o = mix4(v[i], before[i], *reinterpret_cast<const float4*>(a.mu + c));
+        before[i] = v[i];
+      }
+      st4(a.x, base + c, a.bf16, o);
+    }
+  }
+  if (!kept) return;
+  if (t1 < end) {
+    source(end - 1, v);
+    norm(v);
+  }
+#pragma unroll
+  for (int i = 0; i < NV; ++i)
+    if (c0 + i * step < W) *reinterpret_cast<float4*>(kept + c0 + i * step) = v[i];
+}
+
+// A thread per row; the thread of a sequence's first row reads the token before it and leaves the
+// sequence's last token in its place.
+__global__ void __launch_bounds__(128)
+bigram_rows_kernel(const int* __restrict__ ids, int* __restrict__ last, const int* __restrict__ cu,
+                   const int* __restrict__ slots, const int* __restrict__ pos, int* __restrict__ out,
+                   int B, int T, int one_token, long long mul_prev, long long mul_cur, int buckets) {
+  US_PDL_PROLOGUE();
+  const int t = blockIdx.x * 128 + threadIdx.x;
+  if (t >= T) return;
+  int s = t, start = t, end = t + 1;
+  if (!one_token) {
+    int lo = 0, hi = B - 1;
+    while (lo < hi) {
+      const int mid = (lo + hi + 1) >> 1;
+      if (cu[mid] <= t) lo = mid; else hi = mid - 1;
+    }
+    s = lo;
+    start = cu[s];
+    end = cu[s + 1];
+  }
+  long long prev = -1;
+  if (t > start) {
+    prev = ids[t - 1];
+  } else if (slots[s] >= 0) {
+    if (pos[t] > 0) prev = last[slots[s]];
+    last[slots[s]] = ids[end - 1];
+  }
+  out[t] = prev < 0 ? buckets : (int)((prev * mul_prev + (long long)ids[t] * mul_cur) % buckets);
+}
+
+template <int NV>
+__global__ void __launch_bounds__(256)
+poly_norm_kernel(const void* __restrict__ z, long long ldz, const float* __restrict__ act,
+                 void* __restrict__ out, long long ldo, int W, int width, float eps, int bf16) {
+  US_PDL_PROLOGUE();
+  __shared__ float part[3][8];
+  const int step = blockDim.x * 4, c0 = threadIdx.x * 4;
+  const long long zi = (long long)blockIdx.x * ldz, oi = (long long)blockIdx.x * ldo;
+  float4 v[NV];
+  float s2 = 0.f, s4 = 0.f, s6 = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = c0 + i * step;
+    v[i] = c < W ? ld4(z, zi + c, bf16) : make_float4(0.f, 0.f, 0.f, 0.f);
+    const float* p = reinterpret_cast<const float*>(&v[i]);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float q = p[e] * p[e];
+      s2 += q;
+      s4 += q * q;
+      s6 += q * q * q;
+    }
+  }
+  s2 = us::warp_sum(s2);
+  s4 = us::warp_sum(s4);
+  s6 = us::warp_sum(s6);
+  if ((threadIdx.x & 31) == 0) {
+    part[0][threadIdx.x >> 5] = s2;
+    part[1][threadIdx.x >> 5] = s4;
+    part[2][threadIdx.x >> 5] = s6;
+  }
+  __syncthreads();
+  s2 = s4 = s6 = 0.f;
+  for (int w = 0; w < (int)(blockDim.x >> 5); ++w) {
+    s2 += part[0][w];
+    s4 += part[1][w];
+    s6 += part[2][w];
+  }
+  const float n = 1.f / (float)width;
+  const float a = act[0] / sqrtf(s2 * n + eps), b = act[1] / sqrtf(s4 * n + eps),
+              c3 = act[2] / sqrtf(s6 * n + eps), e0 = act[3];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = c0 + i * step;
+    if (c >= W) continue;
+    float4 o;
+    const float* p = reinterpret_cast<const float*>(&v[i]);
+    float* q = reinterpret_cast<float*>(&o);
+#pragma unroll
+    for (int e = 0; e < 4; ++e)
+      q[e] = c + e < width ? fmaf(fmaf(fmaf(c3, p[e], b), p[e], a), p[e], e0) : 0.f;
+    st4(out, oi + c, bf16, o);
+  }
+}
+
+int block_threads(int W) { return min(256, (W / 4 + 31) / 32 * 32); }
+
+}  // namespace
+
+// Start of the stream (y null) or output norm and add, then the next sublayer's input rows.
+US_API int us_stream_rows(const int* ids, const int* rows2, const void* table, const void* table2,
+                          float scale, int vocab, int n2, const void* y, const float* residual,
+                          const float* w, float* residual_out, const float* w_out, const float* mu,
+                          float* state, const int* cu, const int* slots, const int* pos, void* x,
+                          int B, int T, int W, int width, int bf16, int one_token, float eps,
+                          void* stream_) {
+  US_REQUIRE(w && residual_out && w_out && x && T >= 0 && W >= 8 && (W % 8) == 0 && width >= 1 &&
+             width <= W);
+  US_REQUIRE(y ? residual != nullptr && residual != residual_out : (ids && table && (!rows2 || table2)));
+  US_REQUIRE(!mu || (state && cu && slots && pos && B >= 1 && (!one_token || B == T)));
+  if (T == 0) return US_OK;
+  StreamRows a{ids, rows2, table, table2, scale, vocab, n2, y, residual, w, residual_out, w_out, mu,
+               state, cu, slots, pos, x, B, T, W, width, bf16, one_token, eps, us_status_ptr()};
+  const int grid = !mu ? us::ceil_div(T, kRows) : one_token ? T : T / kRows + B;
+  const dim3 block(block_threads(W));
+  const int nv = us::ceil_div(W, 1024);
+#define US_STREAM(N)                                                                              \
+  US_CUDA_CHECK(us::launch_pdl(stream_rows_kernel<N>, dim3(grid), block, 0, (cudaStream_t)stream_, a))
+  if (nv <= 1) US_STREAM(1);
+  else if (nv <= 2) US_STREAM(2);
+  else if (nv <= 4) US_STREAM(4);
+  else if (nv <= 8) US_STREAM(8);
+  else if (nv <= 16) US_STREAM(16);
+  else return US_ERR_LIMIT;
+#undef US_STREAM
+  return US_OK;
+}
+
+US_API int us_bigram_rows(const int* ids, int* last, const int* cu, const int* slots, const int* pos,
+                          int* out, int B, int T, int one_token, long long mul_prev,
+                          long long mul_cur, int buckets, void* stream_) {
+  US_REQUIRE(ids && last && cu && slots && pos && out && B >= 1 && T >= 0 && buckets >= 1);
+  US_REQUIRE(!one_token || B == T);
+  if (T == 0) return US_OK;
+  US_CUDA_CHECK(us::launch_pdl(bigram_rows_kernel, dim3((T + 127) / 128), dim3(128), 0,
+                               (cudaStream_t)stream_, ids, last, cu, slots, pos, out, B, T, one_token,
+                               mul_prev, mul_cur, buckets));
+  return US_OK;
+}
+
+US_API int us_poly_norm(const void* z, long long ldz, const float* act, void* out, long long ldo,
+                        int T, int W, int width, float eps, int bf16, void* stream_) {
+  US_REQUIRE(z && act && out && T >= 0 && W >= 4 && (W % 4) == 0 && width >= 1 && width <= W &&
+             (ldz % 4) == 0 && (ldo % 4) == 0);
+  if (T == 0) return US_OK;
+  const dim3 block(block_threads(W));
+  const int nv = us::ceil_div(W, 1024);
+#define US_POLY(N)                                                                                \
+  US_CUDA_CHECK(us::launch_pdl(poly_norm_kernel<N>, dim3(T), block, 0, (cudaStream_t)stream_, z, ldz, \
+                               act, out, ldo, W, width, eps, bf16))
+  if (nv <= 1) US_POLY(1);
+  else if (nv <= 2) US_POLY(2);
+  else if (nv <= 4) US_POLY(4);
+  else if (nv <= 8) US_POLY(8);
+  else if (nv <= 16) US_POLY(16);
+  else return US_ERR_LIMIT;
+#undef US_POLY
+  return US_OK;
+}

@@ -1,0 +1,94 @@
+"""What decoders made of a list of unlike layers share: padded and stacked weights, random
+checkpoints, the output projection.
+
+Projections that read the same rows are stacked into one product; stacked sections and row
+widths are padded with zeros to multiples of 8 so that every operand row starts on a 16-byte
+boundary."""
+from __future__ import annotations
+
+from typing import Optional
+
+import torch
+
+from ..ops import functional as F
+
+
+def pad8(n: int) -> int:
+    return (n + 7) // 8 * 8
+
+
+class LayeredDecoder:
+    recurrent_state = True       # running requests own a slot of the state pools
+    mixed_batches = True         # prompt portions and decoded tokens may share a forward
+    attends_pages = True         # prefill reads its keys through the page table as well
+
+    def __init__(self, cfg, device="cpu", dtype=torch.bfloat16):
+        if dtype not in (torch.bfloat16, torch.float32):
+            raise ValueError(f"this family is served in bfloat16 or float32, not {dtype}")
+        self.cfg, self.device, self.dtype = cfg, torch.device(device), dtype
+        self.kv_dtype = None
+        self.Wp = pad8(cfg.hidden_size)
+        self.layers: list = []              # per layer a dict of tensors
+        self.embed = self.lm_head = None
+        self.residual_tap: Optional[list] = None     # receives the residual after every layer
+
+    def _put(self, t, dtype=None):
+        return t.to(device=self.device, dtype=dtype or self.dtype)
+
+    def _matrix(self, t, rows=None, cols=None):
+        """``t`` [out, in] zero-padded to [rows, cols] (each up to a multiple of 8)."""
+        rows, cols = pad8(rows or t.shape[0]), pad8(cols or t.shape[1])
+        out = torch.zeros(rows, cols, device=self.device, dtype=self.dtype)
+        out[:t.shape[0], :t.shape[1]] = self._put(t)
+        return out
+
+    def _table(self, t):
+        """Rows of ``t`` as they are, columns zero-padded to a multiple of 8."""
+        return self._matrix(t)[:t.shape[0]]
+
+    def _vector(self, t, width=None):
+        """FP32 vector, zero-padded to ``width``."""
+        out = torch.zeros(width or t.shape[0], device=self.device)
+        out[:t.shape[0]] = self._put(t, torch.float32)
+        return out
+
+    def _stack(self, parts):
+        """Rows of several projections of the same input as one matrix: (matrix, offsets)."""
+        offs, mats, at = [], [], 0
+        for t in parts:
+            m = self._matrix(t)
+            offs.append(at)
+            mats.append(m)
+            at += m.shape[0]
+        return torch.cat(mats, 0), offs
+
+    @staticmethod
+    def _getter(loader):
+        """(get, need): tensors by name; ``need`` also compares the shape with the configuration's."""
+        get = loader.get
+
+        def need(n, *shape):
+            t = get(n)
+            if tuple(t.shape) != shape:
+                raise ValueError(f"tensor {n!r} has shape {tuple(t.shape)}, the configuration "
+                                 f"says {shape}")
+            return t
+        return get, need
+
+    def init_random(self, seed: int = 0, **kw):
+        state = self.random_state(seed, **kw)
+
+        class _Dict:
+            get = staticmethod(state.__getitem__)
+        return self.load_state(_Dict())
+
+    def logits(self, hidden_rows: torch.Tensor) -> torch.Tensor:
+        return F.linear(hidden_rows, self.lm_head, out_dtype=torch.float32)
+
+    def weight_bytes(self) -> int:
+        seen = {}
+        for w in [vars(self)] + self.layers:
+            for t in w.values():
+                if torch.is_tensor(t):
+                    seen[(t.data_ptr(), t.numel())] = t.numel() * t.element_size()
+        return sum(seen.values())

@@ -21,9 +21,6 @@ shared expert scaled by a sigmoid of the residual.
 
 The model runs in the paged engine: attention layers own cache pages, recurrent layers own one
 slot per running request in a state pool (``new_state_pools``).  bf16, or FP32 throughout.
-Projections that read the same rows are stacked into one product; stacked sections, low-rank
-widths and row widths are padded with zeros to multiples of 8 so that every operand row starts
-on a 16-byte boundary.
 """
 from __future__ import annotations
 
@@ -34,12 +31,9 @@ import torch
 
 from ..ops import functional as F
 from ..ops import vector_delta as VD
+from .layered import LayeredDecoder
 
 MIXERS = ("channel_delta", "general_delta", "attention")
-
-
-def _pad8(n: int) -> int:
-    return (n + 7) // 8 * 8
 
 
 @dataclass
@@ -145,61 +139,23 @@ class NepevikConfig:
                                      LayerSpec(at, mlp), LayerSpec(share, mlp)])
 
 
-class NepevikModel:
-    recurrent_state = True       # running requests own a slot of the state pools
-    mixed_batches = True         # prompt portions and decoded tokens may share a forward
-    attends_pages = True         # prefill reads its keys through the page table as well
-
+class NepevikModel(LayeredDecoder):
     def __init__(self, cfg: NepevikConfig, device="cpu", dtype=torch.bfloat16):
-        if dtype not in (torch.bfloat16, torch.float32):
-            raise ValueError(f"this family is served in bfloat16 or float32, not {dtype}")
-        self.cfg, self.device, self.dtype = cfg, torch.device(device), dtype
-        self.kv_dtype = None
-        self.Wp = _pad8(cfg.hidden_size)
-        self.layers: list = []              # per layer a dict of tensors
+        super().__init__(cfg, device, dtype)
         self.gains: list = []               # per layer (norm1, norm2)
-        self.embed = self.lm_head = None
         self.final_gain = 1.0
         self.tables: list = []              # (stacked tables [n, V, top], layer indices)
-        self.residual_tap: Optional[list] = None     # receives the residual after every layer
 
     # ------------------------------------------------------------- weights --
-    def _put(self, t, dtype=None):
-        return t.to(device=self.device, dtype=dtype or self.dtype)
-
-    def _matrix(self, t, rows=None, cols=None):
-        """``t`` [out, in] zero-padded to [rows, cols] (each up to a multiple of 8)."""
-        rows, cols = _pad8(rows or t.shape[0]), _pad8(cols or t.shape[1])
-        out = torch.zeros(rows, cols, device=self.device, dtype=self.dtype)
-        out[:t.shape[0], :t.shape[1]] = self._put(t)
-        return out
-
-    def _stack(self, parts):
-        """Rows of several projections of the same input as one matrix: (matrix, offsets)."""
-        offs, mats, at = [], [], 0
-        for t in parts:
-            m = self._matrix(t)
-            offs.append(at)
-            mats.append(m)
-            at += m.shape[0]
-        return torch.cat(mats, 0), offs
-
     def load_state(self, loader) -> "NepevikModel":
         c, dev = self.cfg, self.device
-        get = loader.get
+        get, need = self._getter(loader)
 
         def f32(n):
             return self._put(get(n), torch.float32).contiguous()
-
-        def need(n, *shape):
-            t = get(n)
-            if tuple(t.shape) != shape:
-                raise ValueError(f"tensor {n!r} has shape {tuple(t.shape)}, the configuration "
-                                 f"says {shape}")
-            return t
         W = c.hidden_size
-        self.embed = self._matrix(need("embed", c.vocab_size, W), rows=c.vocab_size)[:c.vocab_size]
-        self.lm_head = self._matrix(need("head", c.vocab_size, W), rows=c.vocab_size)[:c.vocab_size]
+        self.embed = self._table(need("embed", c.vocab_size, W))
+        self.lm_head = self._table(need("head", c.vocab_size, W))
         self.final_gain = float(get("final.norm"))
         tables: dict = {}
         for i, L in enumerate(c.layers):
@@ -307,13 +263,6 @@ class NepevikModel:
                     out[m + "shared.up"], out[m + "shared.down"] = lin(e.shared_ff, W), lin(W, e.shared_ff)
                     out[m + "shared.sg"] = lin(1, W)
         return out
-
-    def init_random(self, seed: int = 0, rank: Optional[int] = None) -> "NepevikModel":
-        state = self.random_state(seed, rank)
-
-        class _Dict:
-            get = staticmethod(state.__getitem__)
-        return self.load_state(_Dict())
 
     # ------------------------------------------------------------- caches --
     def new_kv_caches(self, num_pages: int, page_size: int = 16):
@@ -448,10 +397,3 @@ class NepevikModel:
             if self.residual_tap is not None:
                 self.residual_tap.append(res[:, :c.hidden_size].clone())
         return x
-
-    def logits(self, hidden_rows: torch.Tensor) -> torch.Tensor:
-        return F.linear(hidden_rows, self.lm_head, out_dtype=torch.float32)
-
-    def weight_bytes(self) -> int:
-        return sum(t.numel() * t.element_size() for w in [vars(self)] + self.layers
-                   for t in w.values() if torch.is_tensor(t))

@@ -50,8 +50,32 @@ def _nepevik_model(cfg, device, dtype, ctx=None):
     return NepevikModel(cfg, device, dtype)
 
 
+def _zonopel_config(d):
+    from .zonopel import ZonopelConfig
+    return ZonopelConfig.from_json(d)
+
+
+def _zonopel_named(name):
+    from .zonopel import ZonopelConfig
+    return ZonopelConfig.tiny() if name == "tiny" else ZonopelConfig.bench()
+
+
+def _zonopel_model(cfg, device, dtype, ctx=None):
+    from .zonopel import ZonopelModel
+    if ctx is not None and ctx.world_size > 1:
+        raise ValueError("this family is served on one GPU")
+    return ZonopelModel(cfg, device, dtype)
+
+
 PAGED_DECODERS = {
     "qwen3_moe": PagedDecoder(_qwen3_config, _qwen3_named, _qwen3_model, (torch.bfloat16,)),
     "nepevik": PagedDecoder(_nepevik_config, _nepevik_named, _nepevik_model,
                             (torch.bfloat16, torch.float32), "nepevik"),
+    "zonopel": PagedDecoder(_zonopel_config, _zonopel_named, _zonopel_model,
+                            (torch.bfloat16, torch.float32), "zonopel"),
 }
+
+
+def named_family(model: str) -> Optional[str]:
+    """Paged decoder that a model name without a checkpoint (``random:<family>[:tiny]``) names."""
+    return next((f for f in PAGED_DECODERS if f in model.lower()), None)

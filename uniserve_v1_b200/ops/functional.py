@@ -651,6 +651,78 @@ def output_norm_add_(y, residual, gain, eps, width, routed=None, shared=None, sh
     return x
 
 
+# ------------------------------------------- rows between two sublayers --
+@dataclass
+class NextRows:
+    """What follows a residual row: the next sublayer's input norm and, with ``shift``, the token
+    shift h + (h' - h) * shift, h' being the row before (``state`` [slots, W] FP32 keeps the last
+    one of every sequence of the packed batch ``meta``)."""
+    weight: torch.Tensor
+    shift: Optional[torch.Tensor] = None
+    state: Optional[torch.Tensor] = None
+    meta: object = None
+
+
+def _stream_rows(embed, y, residual, w, nxt, eps, width, dtype, T, W):
+    dev, m = w.device, nxt.meta
+    res = torch.empty(T, W, dtype=torch.float32, device=dev)
+    x = torch.empty(T, W, dtype=dtype, device=dev)
+    shift = nxt.shift is not None
+    ids, rows2, table, table2, scale = embed or (None, None, None, None, 0.0)
+    N.call("us_stream_rows", N.ptr(ids), N.ptr(rows2), N.ptr(table), N.ptr(table2), scale,
+           table.shape[0] if embed else 0, table2.shape[0] if table2 is not None else 0, N.ptr(y),
+           N.ptr(residual), N.ptr(w), N.ptr(res), N.ptr(nxt.weight), N.ptr(nxt.shift), N.ptr(nxt.state),
+           *([N.ptr(m.cu), N.ptr(m.slots), N.ptr(m.positions)] if shift else [None] * 3), N.ptr(x),
+           m.slots.shape[0] if shift else 1, T, W, width, int(dtype == BF16),
+           int(shift and m.one_token), eps, N.stream())
+    return res, x
+
+
+def embed_norm_rows(ids, table, scale, w, nxt: NextRows, eps, width, second=None):
+    """Start of the stream: rms(table row * scale + second row) * w in FP32, and the next sublayer's
+    rows in the table's type.  ``second``: (rows [T] int32, table) added without the scale."""
+    if not _cuda(table):
+        e = table[ids.long()].float() * scale
+        if second is not None:
+            e = e + second[1][second[0].long()].float()
+        return R.stream_rows(e, None, w, nxt, eps, width, table.dtype)
+    rows2, table2 = second or (None, None)
+    return _stream_rows((ids, rows2, table, table2, scale), None, None, w, nxt, eps, width, table.dtype,
+                        ids.shape[0], table.shape[1])
+
+
+def add_norm_rows(y, residual, w, nxt: NextRows, eps, width):
+    """(residual + rms(y) * w, the next sublayer's rows in y's type).  The residual handed in stays
+    as it is."""
+    if not _cuda(y):
+        return R.stream_rows(y.float(), residual, w, nxt, eps, width, y.dtype)
+    assert y.is_contiguous() and y.shape == residual.shape
+    return _stream_rows(None, y, residual, w, nxt, eps, width, y.dtype, *y.shape)
+
+
+def bigram_rows(ids, last, m, mul_prev, mul_cur, buckets):
+    """Rows (previous token * mul_prev + token * mul_cur) mod buckets of a bigram table [T] int32, row
+    ``buckets`` for a sequence's first token.  ``last`` [slots] int32: last token of every sequence."""
+    if not _cuda(ids):
+        return R.bigram_rows(ids, last, m, mul_prev, mul_cur, buckets)
+    T = ids.shape[0]
+    out = torch.empty(T, dtype=torch.int32, device=ids.device)
+    N.call("us_bigram_rows", N.ptr(ids), N.ptr(last), N.ptr(m.cu), N.ptr(m.slots), N.ptr(m.positions),
+           N.ptr(out), m.slots.shape[0], T, int(m.one_token), mul_prev, mul_cur, buckets, N.stream())
+    return out
+
+
+def poly_norm_(z, act, width, eps):
+    """a N(z) + b N(z^2) + c N(z^3) + e in place, N dividing a row by its root mean square over the first
+    ``width`` columns; ``act`` = (a, b, c, e) FP32.  Columns past ``width`` become zero."""
+    if not _cuda(z):
+        z.copy_(R.poly_norm(z, act, width, eps))
+        return z
+    N.call("us_poly_norm", N.ptr(z), z.stride(0), N.ptr(act), N.ptr(z), z.stride(0), z.shape[0], z.shape[1],
+           width, eps, int(z.dtype == BF16), N.stream())
+    return z
+
+
 def row_norm_kv_(x, offs, dims, wq, wk, slots, kcache, vcache, eps):
     """``x`` [T, ld] holds q, k, v at columns ``offs``, ``dims`` wide.  q (in place) and k are
     normalised over their whole row (all heads together) with weights wq, wk; k and v go to the

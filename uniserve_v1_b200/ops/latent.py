@@ -1,0 +1,143 @@
+"""Latent attention: every cached token is one normed latent c and one rotated key part shared
+by all heads; a head's unrotated keys and its values are linear images of c.
+
+    score_h(i, j) = scale (q_h(i) . W_uk,h c_j + r_h(i) . kr_j)        softmax over j visible to i
+    out_h(i)      = W_uv,h sum_j p_h(i, j) c_j
+
+*Absorbed form*: q W_uk is formed once per query, so attention runs over the latents alone, as
+with one key head of width rank + rot_dim whose values are its first ``rank`` columns.
+
+Pages hold ``[page, 1, rank]`` latents and ``[page, 1, rot_dim]`` rotated parts (each padded to a
+multiple of 8).  On a GPU the entry points run ``csrc/latent_attn.cu``, on the CPU FP32 formulas."""
+from __future__ import annotations
+
+from dataclasses import dataclass
+
+import torch
+
+from . import native as N
+from .vector_delta import BF16, SeqMeta
+
+P, I, L, F = N.P, N.I, N.L, N.F
+N.register_signatures({
+    "us_latent_prep": (I, [P, L, I, I, I, I, I, I, P, P, P, I, P, P, P, I, P, I, I, F, I, P]),
+    "us_rotate_heads": (I, [P, L, I, I, I, P, I, P, I, I, P]),
+    "us_head_linear": (I, [P, P, P, L, L, L, L, L, L, I, I, I, I, I, P]),
+    "us_latent_attention_rows": (I, [P, L, I, P, L, I, P, I, P, I, P, L, I, P, P, P, P, I, I, I, I, I, I,
+                                     I, I, F, I, P]),
+})
+
+
+@dataclass(frozen=True)
+class LatentDims:
+    heads: int
+    dim: int            # unrotated query / key width per head
+    rot_dim: int        # rotated query / key width
+    vdim: int
+    kv_rank: int
+    q_rank: int
+    scale: float
+    window: int         # keys a query sees, itself included (0: every earlier one)
+
+
+def frequencies(dims: int, base: float, device) -> torch.Tensor:
+    """Angle per position of every channel pair, FP64: its product with a far position is reduced
+    before anything is rounded to FP32."""
+    i = torch.arange(dims // 2, dtype=torch.float64)
+    return (float(base) ** (-2.0 * i / dims)).to(device)
+
+
+def _turned(x, positions, freq):
+    """Channel 2i turned with channel 2i + 1 of the last axis (x [T, ..., n] FP32)."""
+    n = freq.shape[0]
+    a = positions.double()[:, None] * freq[None]
+    c, s = torch.cos(a).float(), torch.sin(a).float()
+    while c.dim() < x.dim():
+        c, s = c[:, None], s[:, None]
+    u, v = x[..., 0:2 * n:2], x[..., 1:2 * n:2]
+    out = x.clone()
+    out[..., 0:2 * n:2], out[..., 1:2 * n:2] = u * c - v * s, v * c + u * s
+    return out
+
+
+def _rms(x, w, eps):
+    return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w
+
+
+def latent_prep_(x, offs, d: LatentDims, wq, wc, freq, positions, slots, cpages, rpages, eps):
+    """``x`` holds the query latent, the key latent and the rotated key part at columns ``offs``.
+    Norms the query latent in place; the normed key latent and the turned part go to the cache
+    rows ``slots`` (negative: not written)."""
+    oq, oc, orr = offs
+    nc, nr = cpages.shape[-1], rpages.shape[-1]
+    if x.is_cuda:
+        N.call("us_latent_prep", N.ptr(x), x.stride(0), oq, oc, orr, d.q_rank, d.kv_rank, d.rot_dim,
+               N.ptr(wq), N.ptr(wc), N.ptr(freq), freq.shape[0], N.ptr(positions), N.ptr(slots),
+               N.ptr(cpages), nc, N.ptr(rpages), nr, x.shape[0], eps, int(x.dtype == BF16), N.stream())
+        return
+    x[:, oq:oq + d.q_rank] = _rms(x[:, oq:oq + d.q_rank].float(), wq, eps).to(x.dtype)
+    c = _rms(x[:, oc:oc + d.kv_rank].float(), wc, eps).to(x.dtype)
+    r = _turned(x[:, orr:orr + d.rot_dim].float(), positions, freq).to(x.dtype)
+    sel = slots >= 0
+    at = slots[sel].long()
+    cpages.view(-1, nc)[at, :d.kv_rank] = c[sel]
+    rpages.view(-1, nr)[at, :d.rot_dim] = r[sel]
+
+
+def rotate_heads_(x, off, positions, freq):
+    """Turns the channel pairs that start at channel ``off`` of every head of x [T, H, n] in place."""
+    T, H, n = x.shape
+    if x.is_cuda:
+        N.call("us_rotate_heads", N.ptr(x), x.stride(0), off, x.stride(1), H, N.ptr(freq), freq.shape[0],
+               N.ptr(positions), T, int(x.dtype == BF16), N.stream())
+        return
+    x[..., off:] = _turned(x[..., off:].float(), positions, freq).to(x.dtype)
+
+
+def head_linear(w, x, out):
+    """out[t, h, :M] = w[h] x[t, h, :K]: w [H, M, K] contiguous, x [T, H, >= K] and out [T, H, >= M] with any
+    row and head strides (bf16: multiples of 8 for x)."""
+    H, M, K = w.shape
+    if x.is_cuda:
+        N.call("us_head_linear", N.ptr(w), N.ptr(x), N.ptr(out), M * K, K, x.stride(0), x.stride(1),
+               out.stride(0), out.stride(1), H, min(M, out.shape[2]), K, x.shape[0], int(x.dtype == BF16),
+               N.stream())
+        return out
+    M = min(M, out.shape[2])
+    out[..., :M] = torch.einsum("hmk,thk->thm", w[:, :M].float(), x[..., :K].float()).to(out.dtype)
+    return out
+
+
+def latent_attention(ql, qr, cpages, rpages, m: SeqMeta, page_table, d: LatentDims, seq_lens=None):
+    """Absorbed form over pages: ql [T, H, Rp], qr [T, H, >= rot_dim] (strided views) -> mixtures of
+    latents [T, H, Rp].  ``seq_lens``: one row per sequence, length 0 marks padding."""
+    T, H = ql.shape[:2]
+    page, Rp, RDp = cpages.shape[1], cpages.shape[-1], rpages.shape[-1]
+    R, RD = d.kv_rank, d.rot_dim
+    if ql.is_cuda:
+        out = torch.empty(T, H, Rp, dtype=ql.dtype, device=ql.device)
+        N.call("us_latent_attention_rows", N.ptr(ql), ql.stride(0), ql.stride(1), N.ptr(qr), qr.stride(0),
+               qr.stride(1), N.ptr(cpages), Rp, N.ptr(rpages), RDp, N.ptr(out), H * Rp, Rp, N.ptr(m.cu),
+               N.ptr(m.positions), N.ptr(seq_lens), N.ptr(page_table), T, m.cu.shape[0] - 1, H, R, RD, page,
+               page_table.shape[1], d.window, d.scale, int(ql.dtype == BF16), N.stream())
+        return out
+    out = torch.zeros(T, H, Rp, dtype=ql.dtype)
+    cu = m.cu.tolist()
+    for s in range(len(cu) - 1):
+        lo, hi = cu[s], cu[s + 1]
+        if hi == lo or (seq_lens is not None and int(seq_lens[s]) <= 0):
+            continue
+        pos = m.positions[lo:hi].long()
+        n = int(pos.max()) + 1
+        pg = page_table[s, :(n + page - 1) // page].long()
+        c = cpages[pg].reshape(-1, Rp)[:n, :R].float()
+        r = rpages[pg].reshape(-1, RDp)[:n, :RD].float()
+        sc = (torch.einsum("thr,nr->htn", ql[lo:hi, :, :R].float(), c) +
+              torch.einsum("thr,nr->htn", qr[lo:hi, :, :RD].float(), r)) * d.scale
+        gap = pos[:, None] - torch.arange(n)[None, :]
+        see = gap >= 0
+        if d.window > 0:
+            see = see & (gap < d.window)
+        p = sc.masked_fill(~see[None], float("-inf")).softmax(-1)
+        out[lo:hi, :, :R] = torch.einsum("htn,nr->thr", p, c).to(out.dtype)
+    return out

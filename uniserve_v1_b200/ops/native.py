@@ -52,6 +52,9 @@ _SIGNATURES = {
     "us_head_norm_gate": (I, [P, P, I, P, L, P, L, I, I, I, F, I, I, P]),
     "us_embed_rows": (I, [P, P, P, P, I, I, I, I, P]),
     "us_output_norm_add": (I, [P, P, P, F, I, P, P, P, P, F, F, I, I, I, I, F, I, P]),
+    "us_stream_rows": (I, [P, P, P, P, F, I, I, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, P]),
+    "us_bigram_rows": (I, [P, P, P, P, P, P, I, I, I, L, L, I, P]),
+    "us_poly_norm": (I, [P, L, P, P, L, I, I, I, F, I, P]),
     "us_row_norm_kv": (I, [P, L, I, I, I, I, I, I, P, P, P, P, P, I, F, I, P]),
     "us_tanh_cols": (I, [P, L, I, I, I, I, P]),
     "us_head_mix_attention": (I, [P, P, P, P, P, P, P, P, P, L, L, I, I, I, I, I, I, I, I, I, I, F,

@@ -483,3 +483,55 @@ def head_mix_attention(q, H, kcache, vcache, talk, cu, positions, page_table, sc
         w = torch.einsum("hg,gtn->htn", talk.float(), w)
         out[lo:hi, :H * V] = torch.einsum("htn,nhv->thv", w, v).reshape(hi - lo, H * V).to(q.dtype)
     return out
+
+
+# ------------------------------------------------- rows between two sublayers --
+def _rms(x, width, eps):
+    return x * torch.rsqrt(x.pow(2).sum(-1, keepdim=True) / width + eps)
+
+
+def stream_rows(source, residual, w, nxt, eps, width, dtype):
+    """(new residual, next rows): ``residual`` + rms(source) * w, then the next input norm and, when
+    ``nxt`` has one, the token shift with its state."""
+    r = _rms(source, width, eps) * w
+    if residual is not None:
+        r = residual + r
+    h = _rms(r, width, eps) * nxt.weight
+    if nxt.shift is None:
+        return r, h.to(dtype)
+    before = torch.zeros_like(h)
+    before[1:] = h[:-1]
+    cu, slots = nxt.meta.cu.tolist(), nxt.meta.slots.tolist()
+    for s, slot in enumerate(slots):
+        lo, hi = cu[s], cu[s + 1]
+        if hi == lo:
+            continue
+        fresh = slot < 0 or int(nxt.meta.positions[lo]) == 0
+        before[lo] = 0.0 if fresh else nxt.state[slot]
+        if slot >= 0:
+            nxt.state[slot] = h[hi - 1]
+    return r, (h + (before - h) * nxt.shift).to(dtype)
+
+
+def bigram_rows(ids, last, m, mul_prev, mul_cur, buckets):
+    ids = ids.long()
+    prev = torch.full_like(ids, -1)
+    prev[1:] = ids[:-1]
+    cu, slots = m.cu.tolist(), m.slots.tolist()
+    for s, slot in enumerate(slots):
+        lo, hi = cu[s], cu[s + 1]
+        if hi == lo:
+            continue
+        prev[lo] = -1 if slot < 0 or int(m.positions[lo]) == 0 else int(last[slot])
+        if slot >= 0:
+            last[slot] = ids[hi - 1].to(last.dtype)
+    rows = (prev * mul_prev + ids * mul_cur) % buckets
+    return torch.where(prev < 0, torch.full_like(rows, buckets), rows).to(torch.int32)
+
+
+def poly_norm(z, act, width, eps):
+    v = z.float()
+    out = act[0] * _rms(v, width, eps) + act[1] * _rms(v * v, width, eps) + \
+        act[2] * _rms(v * v * v, width, eps) + act[3]
+    out[:, width:] = 0.0
+    return out.to(z.dtype)

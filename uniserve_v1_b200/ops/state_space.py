@@ -1,0 +1,130 @@
+"""State-space mixer with a scalar decay per head (Mamba-2, state-space duality):
+
+    dt <- softplus(dt + bias)
+    S <- exp(-exp(A_log) dt) S + dt B x^T          S [N, V] per head, FP32
+    y  = S^T C + D x
+    out = rms_groups(y * silu(z)) * w
+
+x, B and C come from one short causal convolution (with bias) and silu; heads share B and C in
+groups.  Batches are packed and states live in slots as described in ``vector_delta``.  On a GPU
+the entry points run ``csrc/state_space.cu``; on the CPU the same recurrence runs in FP32."""
+from __future__ import annotations
+
+from dataclasses import dataclass
+
+import torch
+
+from . import native as N
+from .vector_delta import BF16, SeqMeta, _spans
+
+P, I, L, F = N.P, N.I, N.L, N.F
+N.register_signatures({
+    "us_short_conv": (I, [P, L, I, P, P, P, P, L, P, P, P, I, I, I, I, I, I, P]),
+    "us_state_space_scan": (I, [P, L, P, L, I, P, P, P, P, P, L, P, P, P, I, I, I, I, I, I, I, P]),
+    "us_group_norm_gate": (I, [P, L, P, L, I, P, P, L, I, I, I, F, I, P]),
+})
+
+
+@dataclass(frozen=True)
+class StateSpaceDims:
+    heads: int
+    vdim: int
+    state: int
+    groups: int         # of heads that share B and C
+    norm_groups: int    # of channels that share a root mean square
+    taps: int
+
+    @property
+    def inner(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def channels(self) -> int:          # of the convolution: x, B, C
+        return self.inner + 2 * self.groups * self.state
+
+
+def tiles(m: SeqMeta, rows: int) -> int:
+    """Upper bound of the row tiles (16 rows of one sequence each) of a packed batch."""
+    return rows if m.one_token else rows // 16 + m.slots.shape[0]
+
+
+def short_conv(x, off, taps, bias, ring, m: SeqMeta):
+    """Causal convolution per channel, bias, silu: columns ``off`` .. ``off`` + C of the projection
+    rows ``x``; ``taps`` [C, K], ``bias`` [C] FP32.  ``ring`` [slots, K, C] holds the last inputs
+    of every sequence, the input of position p in entry p % K, and is advanced (K = 1: None).
+    Returns [T, C] rows in x's type."""
+    T, (C, K) = x.shape[0], taps.shape
+    if x.is_cuda:
+        ld = (C + 7) // 8 * 8
+        y = torch.empty(T, ld, dtype=x.dtype, device=x.device)
+        N.call("us_short_conv", N.ptr(x), x.stride(0), off, N.ptr(taps), N.ptr(bias), N.ptr(ring),
+               N.ptr(y), ld, N.ptr(m.cu), N.ptr(m.slots), N.ptr(m.positions), m.slots.shape[0], T, C, K,
+               int(x.dtype == BF16), int(m.one_token), N.stream())
+        return y[:, :C]
+    y = torch.zeros(T, C)
+    cols = x[:, off:off + C]
+    for lo, hi, slot, _ in _spans(m):
+        p0 = int(m.positions[lo])
+        old = cols.new_zeros(K - 1, C)
+        for j in range(min(K - 1, p0)):
+            old[K - 2 - j] = ring[slot, (p0 - 1 - j) % K]
+        full = torch.cat([old, cols[lo:hi]], 0)
+        y[lo:hi] = (full.float().unfold(0, K, 1) * taps[None]).sum(-1) + bias
+        if K > 1:
+            for t in range(max(lo, hi - (K - 1)), hi):
+                ring[slot, (p0 + t - lo) % K] = cols[t]
+    return torch.nn.functional.silu(y).to(x.dtype)
+
+
+def state_space_scan(u, proj, off_dt, w, state, m: SeqMeta, d: StateSpaceDims):
+    """The recurrence and its read-out.  ``u`` [T, channels]: convolved x | B | C; the step sizes
+    stand at column ``off_dt`` of ``proj`` before their bias.  ``state`` [slots, H, N, V] FP32 is
+    updated in place.  Returns y [T, inner] in u's type."""
+    T, H, V, S_, G = u.shape[0], d.heads, d.vdim, d.state, d.groups
+    if u.is_cuda:
+        assert state.is_contiguous() and state.dtype == torch.float32
+        ld = (d.inner + 7) // 8 * 8
+        y = torch.empty(T, ld, dtype=u.dtype, device=u.device)
+        N.call("us_state_space_scan", N.ptr(u), u.stride(0), N.ptr(proj), proj.stride(0), off_dt,
+               N.ptr(w["dt_bias"]), N.ptr(w["A_log"]), N.ptr(w["D"]), N.ptr(state), N.ptr(y), ld,
+               N.ptr(m.cu), N.ptr(m.slots), N.ptr(m.positions), m.slots.shape[0], T, H, V, S_, G,
+               int(u.dtype == BF16), N.stream())
+        return y[:, :d.inner]
+    x = u[:, :d.inner].float().view(T, H, V)
+    B, C = (u[:, d.inner + i * G * S_:d.inner + (i + 1) * G * S_].float().view(T, G, S_)
+            .repeat_interleave(H // G, 1) for i in (0, 1))
+    dt = torch.nn.functional.softplus(proj[:, off_dt:off_dt + H].float() + w["dt_bias"], threshold=1e9)
+    decay = torch.exp(-w["A_log"].exp() * dt)
+    y = torch.zeros(T, H, V)
+    for lo, hi, slot, fresh in _spans(m):
+        S = torch.zeros_like(state[slot]) if fresh else state[slot]
+        for t in range(lo, hi):
+            S = decay[t][:, None, None] * S + (dt[t][:, None] * B[t])[:, :, None] * x[t][:, None, :]
+            y[t] = torch.einsum("hnv,hn->hv", S, C[t]) + w["D"][:, None] * x[t]
+        state[slot] = S
+    return y.view(T, d.inner).to(u.dtype)
+
+
+def group_norm_gate(y, z, w, groups, eps, ldo):
+    """y * silu(z), each of ``groups`` equal parts of a row divided by its own root mean square,
+    times ``w`` (FP32); rows ``ldo`` wide (zero past the end)."""
+    T, n = y.shape
+    if y.is_cuda:
+        out = torch.empty(T, ldo, dtype=y.dtype, device=y.device)
+        N.call("us_group_norm_gate", N.ptr(y), y.stride(0), N.ptr(z), z.stride(0), groups, N.ptr(w),
+               N.ptr(out), ldo, T, n, int(y.dtype == BF16), eps, int(z.dtype == BF16), N.stream())
+        return out
+    g = (y.float() * torch.nn.functional.silu(z.float())).view(T, groups, n // groups)
+    g = g * torch.rsqrt(g.pow(2).mean(-1, keepdim=True) + eps)
+    out = torch.zeros(T, ldo, dtype=y.dtype)
+    out[:, :n] = (g.view(T, n) * w).to(y.dtype)
+    return out
+
+
+def mixer(x, w, ring, state, m: SeqMeta, d: StateSpaceDims, eps):
+    """Everything between the input projection's rows and the output projection's: ``x`` holds
+    z | x B C | dt at the columns ``w['offs']``."""
+    oz, oc, odt = w["offs"]
+    u = short_conv(x, oc, w["conv"], w["conv_b"], ring, m)
+    y = state_space_scan(u, x, odt, w, state, m, d)
+    return group_norm_gate(y, x[:, oz:oz + d.inner], w["norm"], d.norm_groups, eps, w["o"].shape[1])
