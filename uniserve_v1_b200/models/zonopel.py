@@ -141,8 +141,8 @@ class ZonopelModel(LayeredDecoder):
         c, W, Wp = self.cfg, self.cfg.hidden_size, self.Wp
         get, need = self._getter(loader)
 
-        def norm(n, width=W, padded=None):
-            return self._vector(need(n, width), padded or pad8(width))
+        def norm(n, width=None):         # of the residual's width (padded), or of any other one
+            return self._vector(need(n, width or W), width or Wp)
         self.embed = self._table(need("embed", c.vocab_size, W))
         self.lm_head = self._table(need("head", c.vocab_size, W))
         self.embed_norm, self.final_norm = norm("embed.norm"), norm("final.norm")
@@ -172,7 +172,7 @@ class ZonopelModel(LayeredDecoder):
                 w["norm2"], w["norm2b"] = norm(f"l{i}.norm2"), norm(f"l{i}.norm2b")
                 w["up"] = self._matrix(need(m + "up", L.ff, W))
                 w["down"] = self._matrix(need(m + "down", W, L.ff))
-                w["act"] = norm(m + "act", 4, 4)
+                w["act"] = norm(m + "act", 4)
             own[i] = w
         self.layers = [own[i if L.weights_of is None else L.weights_of] for i, L in enumerate(c.layers)]
         return self
