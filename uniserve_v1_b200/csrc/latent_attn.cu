@@ -13,6 +13,7 @@
 // Channel 2i turns with channel 2i + 1.  The angle is formed and reduced to a fraction of a turn in
 // FP64, so far positions lose nothing before the FP32 sine and cosine.
 #include "include/us_common.cuh"
+#include "include/us_mma.cuh"
 #include "include/us_tc05.cuh"
 
 namespace {
@@ -166,27 +167,6 @@ __global__ void __launch_bounds__(256) head_linear_f32_kernel(const HeadLinear a
         out[(long long)(r0 + ty * 4 + i) * a.ldo + m0 + tx * 4 + j] = acc[i][j];
 }
 
-__device__ __forceinline__ void mma16816(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2,
-                                         uint32_t a3, uint32_t b0, uint32_t b1) {
-  asm volatile(
-      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, "
-      "{%8,%9}, {%0,%1,%2,%3};"
-      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-      : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ void cp16(uint32_t dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
-}
-__device__ __forceinline__ void zero16(uint32_t dst) {
-  asm volatile("st.shared.v4.u32 [%0], {%1,%1,%1,%1};" ::"r"(dst), "r"(0) : "memory");
-}
-// byte offset of 16-byte piece c of row r in a tile with 8 pieces (64 columns) per row
-__device__ __forceinline__ uint32_t swz8(int r, int c) { return (uint32_t)(r * 8 + (c ^ (r & 7))) * 16u; }
-
 // 64 rows x 64 features of one head; a warp takes 16 rows.  K in steps of 64, the next step's
 // tiles on their way (cp.async) while one multiplies.
 __global__ void __launch_bounds__(128) head_linear_kernel(const HeadLinear a) {
@@ -200,32 +180,32 @@ __global__ void __launch_bounds__(128) head_linear_kernel(const HeadLinear a) {
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const int r = (tid >> 3) + i * 16, c = tid & 7, k = k0 + c * 8;
-      const uint32_t dx = tc::smem_u32(sm[buf][0]) + swz8(r, c), dw = tc::smem_u32(sm[buf][1]) + swz8(r, c);
-      if (r0 + r < a.rows && k < a.K) cp16(dx, X + (long long)(r0 + r) * a.ldx + k);
-      else zero16(dx);
-      if (m0 + r < a.M && k < a.K) cp16(dw, W + (long long)(m0 + r) * a.ldw + k);
-      else zero16(dw);
+      const uint32_t dx = tc::smem_u32(sm[buf][0]) + us::swz(r, c, 8), dw = tc::smem_u32(sm[buf][1]) + us::swz(r, c, 8);
+      if (r0 + r < a.rows && k < a.K) us::cp16(dx, X + (long long)(r0 + r) * a.ldx + k);
+      else us::zero16(dx);
+      if (m0 + r < a.M && k < a.K) us::cp16(dw, W + (long long)(m0 + r) * a.ldw + k);
+      else us::zero16(dw);
     }
-    asm volatile("cp.async.commit_group;" ::: "memory");
+    us::cp_commit();
   };
   float acc[8][4] = {};
   fetch(0, 0);
   int buf = 0;
   for (int k0 = 0; k0 < a.K; k0 += 64, buf ^= 1) {
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    us::cp_wait<0>();
     __syncthreads();
     if (k0 + 64 < a.K) fetch(k0 + 64, buf ^ 1);
     const uint32_t sx = tc::smem_u32(sm[buf][0]), sw = tc::smem_u32(sm[buf][1]);
 #pragma unroll
     for (int k = 0; k < 4; ++k) {
       uint32_t x[4];
-      ldsm4(x, sx + swz8(warp * 16 + lrow, 2 * k + lhalf));
+      us::ldsm4(x, sx + us::swz(warp * 16 + lrow, 2 * k + lhalf, 8));
 #pragma unroll
       for (int n = 0; n < 4; ++n) {
         uint32_t w[4];
-        ldsm4(w, sw + swz8(n * 16 + lrow, 2 * k + lhalf));
-        mma16816(acc[2 * n], x[0], x[1], x[2], x[3], w[0], w[2]);
-        mma16816(acc[2 * n + 1], x[0], x[1], x[2], x[3], w[1], w[3]);
+        us::ldsm4(w, sw + us::swz(n * 16 + lrow, 2 * k + lhalf, 8));
+        us::mma16816(acc[2 * n], x[0], x[1], x[2], x[3], w[0], w[2]);
+        us::mma16816(acc[2 * n + 1], x[0], x[1], x[2], x[3], w[1], w[3]);
       }
     }
   }

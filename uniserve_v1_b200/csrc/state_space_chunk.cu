@@ -1,0 +1,372 @@
+// Chunked form of the state-space recurrence (see state_space.cu) for bf16 prompts: 64 tokens at a
+// time as products on the tensor cores instead of 64 dependent updates.  With a_t = -exp(A_log)
+// dt_t, c_t its running sum inside the chunk and S the state before it:
+//
+//   y_t  = e^{c_t} S^T C_t + sum_{s <= t} (C_t . B_s) e^{c_t - c_s} dt_s x_s + D x_t
+//   S'   = e^{c_63} S + sum_s B_s (e^{c_63 - c_s} dt_s x_s)^T
+//
+// The recurrence stays a 32-bit one: B, C and x are bf16 values and exact operands, and every FP32
+// operand (S, the decayed scores, the weighted x) enters as the sum of three bf16 values, which
+// holds all 24 bits; products accumulate in FP32 and S lives in FP32 accumulators across chunks.
+// Running sums of a are FP64, kept as two floats: differences of far exponents stay exact.
+//
+// A CTA takes 32 state columns of one head of one sequence and walks its chunks; the next chunk's
+// operands (cp.async) and exponents are formed while one multiplies.  8 warps: scores and outputs
+// by (16 tokens, half of the summed axis), the state by 16 rows.
+#include "include/us_common.cuh"
+#include "include/us_mma.cuh"
+#include "include/us_tc05.cuh"
+
+namespace {
+
+constexpr int kThreads = 256;
+constexpr int kQ = 64;              // tokens per chunk
+constexpr int kV = 32;              // state columns per CTA
+constexpr int kYRow = kV + 4;
+
+struct ChunkArgs {
+  const __nv_bfloat16* u;           // [T, ldu]: x (H V) | B (G N) | C (G N)
+  long long ldu;
+  const __nv_bfloat16* dt;          // raw step sizes, column h of rows at lddt
+  long long lddt;
+  const float *dt_bias, *A_log, *D;
+  float* state;                     // [slots, H, N, V]
+  __nv_bfloat16* y;
+  long long ldy;
+  const int *cu, *slots, *pos;
+  int H, V, N, G;
+};
+
+struct Exponents {                  // of a chunk's tokens
+  float hi[kQ], lo[kQ];             // running sum c_t as two floats
+  float dt[kQ], w[kQ], e[kQ];       // dt_t, e^{c_63 - c_t} dt_t, e^{c_t}
+  float all;                        // e^{c_63}
+};
+
+__device__ __forceinline__ float softplus_f(float x) {
+  return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x)));
+}
+// byte offset of piece c (of four) of row r: 8 rows of one piece hit 8 bank groups
+__device__ __forceinline__ uint32_t swz4(int r, int c) { return (uint32_t)(r * 4 + (c ^ ((r >> 1) & 3))) * 16u; }
+
+// (x, y) = sum of three bf16 pairs
+__device__ __forceinline__ void split3(float x, float y, uint32_t (&o)[3]) {
+#pragma unroll
+  for (int i = 0; i < 3; ++i) {
+    const __nv_bfloat162 p = __floats2bfloat162_rn(x, y);
+    o[i] = *reinterpret_cast<const uint32_t*>(&p);
+    x -= us::bf2f(p.x);
+    y -= us::bf2f(p.y);
+  }
+}
+
+// One warp: exponents of the chunk whose raw step sizes its lanes hold (tokens 2 lane, 2 lane + 1).
+__device__ __forceinline__ void form_exponents(Exponents& x, float raw0, float raw1, int n, float A,
+                                               float bias) {
+  const int lane = threadIdx.x & 31, t = 2 * lane;
+  const float d0 = t < n ? softplus_f(raw0 + bias) : 0.f, d1 = t + 1 < n ? softplus_f(raw1 + bias) : 0.f;
+  const double a0 = -(double)(A * d0), a1 = -(double)(A * d1);
+  double s = a0 + a1;
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const double b = __shfl_up_sync(0xffffffffu, s, o);
+    if (lane >= o) s += b;
+  }
+  const double total = __shfl_sync(0xffffffffu, s, 31), c1 = s, c0 = s - a1;
+  x.hi[t] = (float)c0;
+  x.lo[t] = (float)(c0 - (double)(float)c0);
+  x.hi[t + 1] = (float)c1;
+  x.lo[t + 1] = (float)(c1 - (double)(float)c1);
+  x.dt[t] = d0;
+  x.dt[t + 1] = d1;
+  x.w[t] = expf((float)(total - c0)) * d0;
+  x.w[t + 1] = expf((float)(total - c1)) * d1;
+  x.e[t] = expf((float)c0);
+  x.e[t + 1] = expf((float)c1);
+  if (lane == 0) x.all = expf((float)total);
+}
+
+template <int NP>
+__global__ void __launch_bounds__(kThreads, 1) state_space_chunk_kernel(const ChunkArgs a) {
+  US_PDL_PROLOGUE();
+  constexpr int PC = NP / 8;                          // 16-byte pieces of a B or C row
+  constexpr uint32_t kBC = kQ * NP * 2, kX = kQ * kV * 2, kS = NP * kV * 2;
+  constexpr uint32_t kBuf = 2 * kBC + kX;             // B, C, x of a chunk
+  constexpr int MB = NP / 16, WN = 8 / MB, SN = 4 / WN;   // state: row blocks, warps per block, col tiles
+  extern __shared__ __align__(1024) uint8_t sm[];
+  const uint32_t sb = tc::smem_u32(sm);               // 2 buffers
+  const uint32_t sx = sb + 2 * kBuf;                  // [3] weighted x
+  const uint32_t ss = sx + 3 * kX;                    // [3] state
+  float* yp = reinterpret_cast<float*>(sm + 2 * kBuf + 3 * kX + 3 * kS);    // [kQ][kYRow]
+  Exponents* ex = reinterpret_cast<Exponents*>(yp + kQ * kYRow);            // [2]
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int lrow = lane & 15, lhalf = lane >> 4, r0 = lane >> 2, cq = (lane & 3) * 2;
+  const int h = blockIdx.y, s = blockIdx.z, g = h / (a.H / a.G), v0 = blockIdx.x * kV;
+  const int start = a.cu[s], T = a.cu[s + 1] - start, slot = a.slots[s];
+  if (T <= 0) return;
+  if (slot < 0) {
+    for (int e = tid; e < T * kV; e += kThreads)
+      if (v0 + e % kV < a.V)
+        a.y[(long long)(start + e / kV) * a.ldy + (long long)h * a.V + v0 + e % kV] = us::f2bf(0.f);
+    return;
+  }
+  const bool fresh = a.pos[start] == 0;
+  float* Sg = a.state + ((long long)slot * a.H + h) * a.N * a.V;
+  const float A = expf(a.A_log[h]), bias = a.dt_bias[h], D = a.D[h];
+  const __nv_bfloat16* xg = a.u + (long long)start * a.ldu + (long long)h * a.V + v0;
+  const __nv_bfloat16* bg = a.u + (long long)start * a.ldu + (long long)a.H * a.V + (long long)g * a.N;
+  const __nv_bfloat16* cg = bg + (long long)a.G * a.N;
+
+  auto fetch = [&](int c, int buf) {
+    const uint32_t dst = sb + buf * kBuf;
+    const int n = min(kQ, T - c * kQ);
+    for (int e = tid; e < kQ * PC; e += kThreads) {
+      const int r = e / PC, p = e % PC;
+      const long long row = (long long)(c * kQ + r) * a.ldu;
+      const uint32_t d = dst + us::swz(r, p, PC);
+      if (r < n && p * 8 < a.N) {
+        us::cp16(d, bg + row + p * 8);
+        us::cp16(d + kBC, cg + row + p * 8);
+      } else {
+        us::zero16(d);
+        us::zero16(d + kBC);
+      }
+    }
+    {
+      const int r = tid >> 2, p = tid & 3;
+      const uint32_t d = dst + 2 * kBC + swz4(r, p);
+      if (r < n && v0 + p * 8 < a.V) us::cp16(d, xg + (long long)(c * kQ + r) * a.ldu + p * 8);
+      else us::zero16(d);
+    }
+    us::cp_commit();
+  };
+  const int chunks = (T + kQ - 1) / kQ;
+  float raw0 = 0.f, raw1 = 0.f;
+  auto fetch_steps = [&](int c) {                     // warp 0's lanes: two tokens each
+    const int t = c * kQ + 2 * lane;
+    raw0 = t < T ? us::bf2f(a.dt[(long long)(start + t) * a.lddt + h]) : 0.f;
+    raw1 = t + 1 < T ? us::bf2f(a.dt[(long long)(start + t + 1) * a.lddt + h]) : 0.f;
+  };
+  fetch(0, 0);
+  if (warp == 0) {
+    fetch_steps(0);
+    form_exponents(ex[0], raw0, raw1, min(kQ, T), A, bias);
+    if (chunks > 1) fetch_steps(1);
+  }
+  // state: warp (block m, part) holds rows 16 m .. and SN column tiles
+  const int sm_ = (warp % MB) * 16, sn = (warp / MB) * SN;
+  float S[SN][4];
+#pragma unroll
+  for (int x = 0; x < SN; ++x)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int row = sm_ + r0 + (e >> 1) * 8, col = v0 + (sn + x) * 8 + cq + (e & 1);
+      S[x][e] = (!fresh && row < a.N && col < a.V) ? Sg[(long long)row * a.V + col] : 0.f;
+    }
+  const int tm = (warp >> 1) * 16, half = warp & 1;   // outputs: tokens tm .., half of the summed axis
+
+  for (int c = 0; c < chunks; ++c) {
+    const int buf = c & 1, n = min(kQ, T - c * kQ);
+    const uint32_t B = sb + buf * kBuf, C = B + kBC, X = B + 2 * kBC;
+    const Exponents& x = ex[buf];
+    us::cp_wait<0>();
+    __syncthreads();                                  // chunk c is there, chunk c - 1 is done
+    if (c + 1 < chunks) fetch(c + 1, buf ^ 1);
+    // weighted x and the state, three bf16 parts each
+    {
+      const int r = tid >> 2, p = tid & 3;
+      us::Pack16 v;
+      const uint32_t at = swz4(r, p);
+      v.u = *reinterpret_cast<const uint4*>(sm + (X - sb) + at);
+      const float w = x.w[r];
+      uint32_t o[3][4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        uint32_t q[3];
+        split3(us::bf2f(v.b[2 * e]) * w, us::bf2f(v.b[2 * e + 1]) * w, q);
+#pragma unroll
+        for (int i = 0; i < 3; ++i) o[i][e] = q[i];
+      }
+#pragma unroll
+      for (int i = 0; i < 3; ++i)
+        asm volatile("st.shared.v4.u32 [%0], {%1,%2,%3,%4};" ::"r"(sx + i * kX + at), "r"(o[i][0]),
+                     "r"(o[i][1]), "r"(o[i][2]), "r"(o[i][3]) : "memory");
+#pragma unroll
+      for (int t = 0; t < SN; ++t)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          uint32_t q[3];
+          split3(S[t][2 * e], S[t][2 * e + 1], q);
+          const uint32_t d = ss + swz4(sm_ + r0 + e * 8, sn + t) + cq * 2;
+#pragma unroll
+          for (int i = 0; i < 3; ++i)
+            asm volatile("st.shared.u32 [%0], %1;" ::"r"(d + i * kS), "r"(q[i]) : "memory");
+        }
+    }
+    __syncthreads();
+    // the next chunk's exponents, while the other warps multiply
+    if (warp == 0 && c + 1 < chunks) {
+      form_exponents(ex[buf ^ 1], raw0, raw1, min(kQ, T - (c + 1) * kQ), A, bias);
+      if (c + 2 < chunks) fetch_steps(c + 2);
+    }
+    float acc[4][4];
+#pragma unroll
+    for (int t = 0; t < 4; ++t)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[t][e] = 0.f;
+    const bool within = tm + 15 >= half * 32;         // some s <= t in this warp's half
+    float sc[4][4];
+#pragma unroll
+    for (int t = 0; t < 4; ++t)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) sc[t][e] = 0.f;
+#pragma unroll
+    for (int k = 0; k < NP / 16; ++k) {
+      uint32_t cf[4];
+      us::ldsm4(cf, C + us::swz(tm + lrow, 2 * k + lhalf, PC));
+      if (within) {                                   // scores C_t . B_s of 16 x 32 pairs
+#pragma unroll
+        for (int y = 0; y < 2; ++y) {
+          uint32_t b[4];
+          us::ldsm4(b, B + us::swz(half * 32 + y * 16 + lrow, 2 * k + lhalf, PC));
+          us::mma16816(sc[2 * y], cf[0], cf[1], cf[2], cf[3], b[0], b[2]);
+          us::mma16816(sc[2 * y + 1], cf[0], cf[1], cf[2], cf[3], b[1], b[3]);
+        }
+      }
+      if (k / (NP / 32) == half) {                    // S^T C_t over this warp's half of the rows
+#pragma unroll
+        for (int i = 0; i < 3; ++i)
+#pragma unroll
+          for (int y = 0; y < 2; ++y) {
+            uint32_t b[4];
+            us::ldsm4t(b, ss + i * kS + swz4(k * 16 + lrow, 2 * y + lhalf));
+            us::mma16816(acc[2 * y], cf[0], cf[1], cf[2], cf[3], b[0], b[1]);
+            us::mma16816(acc[2 * y + 1], cf[0], cf[1], cf[2], cf[3], b[2], b[3]);
+          }
+      }
+    }
+    const int ta = tm + r0, tb = ta + 8;
+    {
+      const float ea = x.e[ta], eb = x.e[tb];
+#pragma unroll
+      for (int t = 0; t < 4; ++t) {
+        acc[t][0] *= ea;
+        acc[t][1] *= ea;
+        acc[t][2] *= eb;
+        acc[t][3] *= eb;
+      }
+    }
+    if (within) {
+      const float ha = x.hi[ta], la = x.lo[ta], hb = x.hi[tb], lb = x.lo[tb];
+#pragma unroll
+      for (int k = 0; k < 2; ++k) {                   // 16 tokens s per step
+        uint32_t m[4][3];                             // operand registers: rows t, t + 8; s, s + 8
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int s0 = half * 32 + k * 16 + e * 8 + cq;
+          const float h0 = x.hi[s0], l0 = x.lo[s0], h1 = x.hi[s0 + 1], l1 = x.lo[s0 + 1];
+          const float d0 = x.dt[s0], d1 = x.dt[s0 + 1];
+          const float (&q)[4] = sc[2 * k + e];
+          split3(s0 <= ta ? q[0] * (expf((ha - h0) + (la - l0)) * d0) : 0.f,
+                 s0 + 1 <= ta ? q[1] * (expf((ha - h1) + (la - l1)) * d1) : 0.f, m[2 * e]);
+          split3(s0 <= tb ? q[2] * (expf((hb - h0) + (lb - l0)) * d0) : 0.f,
+                 s0 + 1 <= tb ? q[3] * (expf((hb - h1) + (lb - l1)) * d1) : 0.f, m[2 * e + 1]);
+        }
+#pragma unroll
+        for (int y = 0; y < 2; ++y) {
+          uint32_t b[4];
+          us::ldsm4t(b, X + swz4(half * 32 + k * 16 + lrow, 2 * y + lhalf));
+#pragma unroll
+          for (int i = 0; i < 3; ++i) {
+            us::mma16816(acc[2 * y], m[0][i], m[1][i], m[2][i], m[3][i], b[0], b[1]);
+            us::mma16816(acc[2 * y + 1], m[0][i], m[1][i], m[2][i], m[3][i], b[2], b[3]);
+          }
+        }
+      }
+    }
+    if (half == 1) {
+#pragma unroll
+      for (int t = 0; t < 4; ++t) {
+        *reinterpret_cast<float2*>(yp + ta * kYRow + t * 8 + cq) = make_float2(acc[t][0], acc[t][1]);
+        *reinterpret_cast<float2*>(yp + tb * kYRow + t * 8 + cq) = make_float2(acc[t][2], acc[t][3]);
+      }
+    }
+    // state after the chunk
+#pragma unroll
+    for (int t = 0; t < SN; ++t)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) S[t][e] *= x.all;
+#pragma unroll
+    for (int k = 0; k < kQ / 16; ++k) {
+      uint32_t b[4];                                  // B^T: rows of the state, 16 tokens
+      us::ldsm4t(b, B + us::swz(k * 16 + (lane & 7) + (lhalf << 3), sm_ / 8 + ((lane >> 3) & 1), PC));
+#pragma unroll
+      for (int i = 0; i < 3; ++i)
+#pragma unroll
+        for (int y = 0; y < (SN + 1) / 2; ++y) {
+          uint32_t w[4];
+          us::ldsm4t(w, sx + i * kX + swz4(k * 16 + lrow, sn + 2 * y + lhalf));
+          us::mma16816(S[2 * y], b[0], b[1], b[2], b[3], w[0], w[1]);
+          us::mma16816(S[2 * y + 1], b[0], b[1], b[2], b[3], w[2], w[3]);
+        }
+    }
+    __syncthreads();
+    if (half == 0) {
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int t = ta + e * 8;
+        if (t >= n) continue;
+        __nv_bfloat16* yr = a.y + (long long)(start + c * kQ + t) * a.ldy + (long long)h * a.V + v0;
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
+          if (v0 + q * 8 >= a.V) continue;
+          const float2 o = *reinterpret_cast<const float2*>(yp + t * kYRow + q * 8 + cq);
+          const __nv_bfloat162 xv = *reinterpret_cast<const __nv_bfloat162*>(sm + (X - sb) + swz4(t, q) + cq * 2);
+          *reinterpret_cast<__nv_bfloat162*>(yr + q * 8 + cq) = __floats2bfloat162_rn(
+              fmaf(D, us::bf2f(xv.x), acc[q][2 * e] + o.x), fmaf(D, us::bf2f(xv.y), acc[q][2 * e + 1] + o.y));
+        }
+      }
+    }
+  }
+#pragma unroll
+  for (int x = 0; x < SN; ++x)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int row = sm_ + r0 + (e >> 1) * 8, col = v0 + (sn + x) * 8 + cq + (e & 1);
+      if (row < a.N && col < a.V) Sg[(long long)row * a.V + col] = S[x][e];
+    }
+}
+
+template <int NP>
+int launch_chunk(const ChunkArgs& a, int B, cudaStream_t stream) {
+  constexpr size_t smem = 2 * (2 * kQ * NP * 2 + kQ * kV * 2) + 3 * kQ * kV * 2 + 3 * NP * kV * 2 +
+                          kQ * kYRow * 4 + 2 * sizeof(Exponents);
+  static bool configured = false;
+  if (!configured) {
+    US_CUDA_CHECK(cudaFuncSetAttribute(state_space_chunk_kernel<NP>,
+                                       cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    configured = true;
+  }
+  US_CUDA_CHECK(us::launch_pdl(state_space_chunk_kernel<NP>, dim3(us::ceil_div(a.V, kV), a.H, B),
+                               dim3(kThreads), smem, stream, a));
+  return US_OK;
+}
+
+}  // namespace
+
+// Widths N <= 128 and V, every offset a multiple of 8.
+US_API int us_state_space_chunks(const void* u, long long ldu, const void* proj, long long ldp,
+                                 int off_dt, const float* dt_bias, const float* A_log, const float* D,
+                                 float* state, void* y, long long ldy, const int* cu,
+                                 const int* slots, const int* pos, int B, int T, int H, int V, int N,
+                                 int G, void* stream_) {
+  US_REQUIRE(u && proj && dt_bias && A_log && D && state && y && cu && slots && pos);
+  US_REQUIRE(B >= 1 && T >= 0 && H >= 1 && V >= 1 && N >= 1 && G >= 1 && H % G == 0);
+  US_REQUIRE((V % 8) == 0 && (N % 8) == 0 && (ldu % 8) == 0 && (ldy % 2) == 0 && ((uintptr_t)u % 16) == 0 &&
+             ((uintptr_t)y % 4) == 0);
+  if (N > 128) return US_ERR_LIMIT;
+  if (T == 0) return US_OK;
+  ChunkArgs a{(const __nv_bfloat16*)u, ldu, (const __nv_bfloat16*)proj + off_dt, ldp, dt_bias, A_log, D,
+              state, (__nv_bfloat16*)y, ldy, cu, slots, pos, H, V, N, G};
+  return N <= 64 ? launch_chunk<64>(a, B, (cudaStream_t)stream_) : launch_chunk<128>(a, B, (cudaStream_t)stream_);
+}

@@ -78,6 +78,7 @@ struct StreamRows {
   void* x;                    // [T, W]
   int B, T, W, width, bf16, one_token;
   float eps;
+  int rows;                   // rows per CTA without a shift
   unsigned int* status;
 };
 
@@ -91,8 +92,8 @@ __global__ void __launch_bounds__(256) stream_rows_kernel(const StreamRows a) {
   // rows of this CTA: t0 .. t1 of sequence s
   int s = -1, t0, t1, start = 0, end = 0;
   if (!a.mu) {
-    t0 = blockIdx.x * kRows;
-    t1 = min(a.T, t0 + kRows);
+    t0 = blockIdx.x * a.rows;
+    t1 = min(a.T, t0 + a.rows);
   } else if (a.one_token) {
     s = start = t0 = blockIdx.x;
     end = t1 = t0 + 1;
@@ -309,8 +310,8 @@ US_API int us_stream_rows(const int* ids, const int* rows2, const void* table, c
   US_REQUIRE(!mu || (state && cu && slots && pos && B >= 1 && (!one_token || B == T)));
   if (T == 0) return US_OK;
   StreamRows a{ids, rows2, table, table2, scale, vocab, n2, y, residual, w, residual_out, w_out, mu,
-               state, cu, slots, pos, x, B, T, W, width, bf16, one_token, eps, us_status_ptr()};
-  const int grid = !mu ? us::ceil_div(T, kRows) : one_token ? T : T / kRows + B;
+               state, cu, slots, pos, x, B, T, W, width, bf16, one_token, eps, T >= 2048 ? 2 : 1, us_status_ptr()};
+  const int grid = !mu ? us::ceil_div(T, a.rows) : one_token ? T : T / kRows + B;
   const dim3 block(block_threads(W));
   const int nv = us::ceil_div(W, 1024);
 #define US_STREAM(N)                                                                              \

@@ -287,7 +287,8 @@ class ZonopelModel(LayeredDecoder):
         q = F.linear(proj[:, oq:oq + pad8(s.q_rank)], w["uq"]).view(T, H, Dp + RDp)
         LA.rotate_heads_(q, Dp, m.positions, w["freq"])
         ql = LA.head_linear(w["absorb"], q, torch.empty(T, H, cp.shape[-1], dtype=q.dtype, device=q.device))
-        lat = LA.latent_attention(ql, q[:, :, Dp:], cp, rp, m, meta.page_table, s, seq_lens=meta.seq_lens)
+        lat = LA.latent_attention(ql, q[:, :, Dp:], cp, rp, m, meta.page_table, s, seq_lens=meta.seq_lens,
+                                  max_k=meta.max_k)
         n, ldo = H * s.vdim, w["o"].shape[1]
         att = (torch.empty if ldo == n else torch.zeros)(T, ldo, dtype=x.dtype, device=x.device)
         LA.head_linear(w["uv"], lat, att[:, :n].unflatten(1, (H, s.vdim)))

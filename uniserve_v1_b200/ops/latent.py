@@ -25,6 +25,8 @@ N.register_signatures({
     "us_head_linear": (I, [P, P, P, L, L, L, L, L, L, I, I, I, I, I, P]),
     "us_latent_attention_rows": (I, [P, L, I, P, L, I, P, I, P, I, P, L, I, P, P, P, P, I, I, I, I, I, I,
                                      I, I, F, I, P]),
+    "us_latent_decode": (I, [P, L, I, P, L, I, P, I, P, I, P, L, I, P, P, P, P, P, I, I, I, I, I, I, I, I, I,
+                             F, P]),
 })
 
 
@@ -108,14 +110,39 @@ def head_linear(w, x, out):
     return out
 
 
-def latent_attention(ql, qr, cpages, rpages, m: SeqMeta, page_table, d: LatentDims, seq_lens=None):
+def decode_fits(ql, cpages, rpages) -> bool:
+    """Whether single rows take the tensor-instruction form."""
+    return ql.dtype == BF16 and cpages.shape[-1] <= 512 and rpages.shape[-1] <= 64
+
+
+def decode_splits(rows: int, heads: int, keys: int) -> int:
+    """Key splits per row: up to two CTAs per SM, at least 64 keys each."""
+    ctas = rows * -(-heads // (16 if heads <= 16 else 32))
+    return max(1, min(296 // ctas, keys // 64, 8))
+
+
+def latent_attention(ql, qr, cpages, rpages, m: SeqMeta, page_table, d: LatentDims, seq_lens=None, max_k=0,
+                     rows=None, out=None):
     """Absorbed form over pages: ql [T, H, Rp], qr [T, H, >= rot_dim] (strided views) -> mixtures of
-    latents [T, H, Rp].  ``seq_lens``: one row per sequence, length 0 marks padding."""
+    latents [T, H, Rp].  ``seq_lens``: one row per sequence, length 0 marks padding; ``max_k`` bounds
+    the keys of a sequence.  ``rows`` (int32): only these rows, into ``out``."""
     T, H = ql.shape[:2]
     page, Rp, RDp = cpages.shape[1], cpages.shape[-1], rpages.shape[-1]
     R, RD = d.kv_rank, d.rot_dim
     if ql.is_cuda:
-        out = torch.empty(T, H, Rp, dtype=ql.dtype, device=ql.device)
+        if out is None:
+            out = torch.empty(T, H, Rp, dtype=ql.dtype, device=ql.device)
+        if (rows is not None or m.one_token) and decode_fits(ql, cpages, rpages):
+            count = T if rows is None else rows.shape[0]
+            keys = max_k or page * page_table.shape[1]
+            keys = min(keys, d.window) if d.window > 0 else keys
+            N.call("us_latent_decode", N.ptr(ql), ql.stride(0), ql.stride(1), N.ptr(qr), qr.stride(0),
+                   qr.stride(1), N.ptr(cpages), Rp, N.ptr(rpages), RDp, N.ptr(out), out.stride(0),
+                   out.stride(1), N.ptr(rows), N.ptr(m.cu), N.ptr(m.positions), N.ptr(seq_lens),
+                   N.ptr(page_table), count, m.cu.shape[0] - 1, H, R, RD, page, page_table.shape[1], d.window,
+                   decode_splits(count, H, keys), d.scale, N.stream())
+            return out
+        assert rows is None
         N.call("us_latent_attention_rows", N.ptr(ql), ql.stride(0), ql.stride(1), N.ptr(qr), qr.stride(0),
                qr.stride(1), N.ptr(cpages), Rp, N.ptr(rpages), RDp, N.ptr(out), H * Rp, Rp, N.ptr(m.cu),
                N.ptr(m.positions), N.ptr(seq_lens), N.ptr(page_table), T, m.cu.shape[0] - 1, H, R, RD, page,

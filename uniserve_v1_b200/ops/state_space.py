@@ -21,6 +21,7 @@ P, I, L, F = N.P, N.I, N.L, N.F
 N.register_signatures({
     "us_short_conv": (I, [P, L, I, P, P, P, P, L, P, P, P, I, I, I, I, I, I, P]),
     "us_state_space_scan": (I, [P, L, P, L, I, P, P, P, P, P, L, P, P, P, I, I, I, I, I, I, I, P]),
+    "us_state_space_chunks": (I, [P, L, P, L, I, P, P, P, P, P, L, P, P, P, I, I, I, I, I, I, P]),
     "us_group_norm_gate": (I, [P, L, P, L, I, P, P, L, I, I, I, F, I, P]),
 })
 
@@ -41,11 +42,6 @@ class StateSpaceDims:
     @property
     def channels(self) -> int:          # of the convolution: x, B, C
         return self.inner + 2 * self.groups * self.state
-
-
-def tiles(m: SeqMeta, rows: int) -> int:
-    """Upper bound of the row tiles (16 rows of one sequence each) of a packed batch."""
-    return rows if m.one_token else rows // 16 + m.slots.shape[0]
 
 
 def short_conv(x, off, taps, bias, ring, m: SeqMeta):
@@ -76,6 +72,11 @@ def short_conv(x, off, taps, bias, ring, m: SeqMeta):
     return torch.nn.functional.silu(y).to(x.dtype)
 
 
+def chunks_fit(u, d: StateSpaceDims) -> bool:
+    """Whether prompts take the chunked form (products on the tensor cores)."""
+    return u.dtype == BF16 and d.vdim % 8 == 0 and d.state % 8 == 0 and d.state <= 128
+
+
 def state_space_scan(u, proj, off_dt, w, state, m: SeqMeta, d: StateSpaceDims):
     """The recurrence and its read-out.  ``u`` [T, channels]: convolved x | B | C; the step sizes
     stand at column ``off_dt`` of ``proj`` before their bias.  ``state`` [slots, H, N, V] FP32 is
@@ -85,6 +86,12 @@ def state_space_scan(u, proj, off_dt, w, state, m: SeqMeta, d: StateSpaceDims):
         assert state.is_contiguous() and state.dtype == torch.float32
         ld = (d.inner + 7) // 8 * 8
         y = torch.empty(T, ld, dtype=u.dtype, device=u.device)
+        if chunks_fit(u, d) and not m.one_token:
+            N.call("us_state_space_chunks", N.ptr(u), u.stride(0), N.ptr(proj), proj.stride(0), off_dt,
+                   N.ptr(w["dt_bias"]), N.ptr(w["A_log"]), N.ptr(w["D"]), N.ptr(state), N.ptr(y), ld,
+                   N.ptr(m.cu), N.ptr(m.slots), N.ptr(m.positions), m.slots.shape[0], T, H, V, S_, G,
+                   N.stream())
+            return y[:, :d.inner]
         N.call("us_state_space_scan", N.ptr(u), u.stride(0), N.ptr(proj), proj.stride(0), off_dt,
                N.ptr(w["dt_bias"]), N.ptr(w["A_log"]), N.ptr(w["D"]), N.ptr(state), N.ptr(y), ld,
                N.ptr(m.cu), N.ptr(m.slots), N.ptr(m.positions), m.slots.shape[0], T, H, V, S_, G,

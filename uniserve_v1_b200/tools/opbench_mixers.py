@@ -1,5 +1,6 @@
-"""Kernels of the vector-decay, head-mixing and table-routed layers beside the like kernels of
-the hybrid and Qwen3 decoders at equal sizes, each with its roofline fraction.
+"""Kernels of the vector-decay, head-mixing, table-routed, state-space and latent-attention layers
+beside the like kernels of the hybrid and Qwen3 decoders at equal sizes, each with its roofline
+fraction.
 
     python -m uniserve_v1_b200.tools.opbench_mixers [--only NAME,...] [--batch 64] [--rows 8192]
 
@@ -16,6 +17,8 @@ import torch
 
 from ..ops import functional as F
 from ..ops import gated_delta as GD
+from ..ops import latent as LA
+from ..ops import state_space as SS
 from ..ops import vector_delta as VD
 from .opbench import peaks, timeit
 
@@ -180,6 +183,54 @@ def main():
         case(f"qk_norm_rope_kv_{kind} (like)", lambda: F.qk_norm_rope_kv_(
             xr, nw[:D].contiguous(), nw[:D].contiguous(), pos, inv, slots, kc, vc, Hq, G, D),
             n * (2 * Hq * D + 4 * G * D) * 2.0)
+        # ---- state space: 64 heads x 64, state 128, 8 groups ----
+        d = SS.StateSpaceDims(64, 64, 128, 8, 8, 4)
+        Cs, inner = d.channels, d.inner
+        proj = rnd(n, inner + Cs + d.heads)
+        sw = {"conv": rnd(Cs, 4, dtype=torch.float32), "conv_b": rnd(Cs, dtype=torch.float32),
+              "dt_bias": rnd(d.heads, dtype=torch.float32) - 3.0, "A_log": rnd(d.heads, dtype=torch.float32),
+              "D": rnd(d.heads, dtype=torch.float32), "norm": rnd(inner, dtype=torch.float32),
+              "offs": (0, inner, inner + Cs), "o": torch.empty(8, inner, device=dev)}
+        ring = torch.zeros(B, 4, Cs, dtype=bf, device=dev)
+        spool = torch.zeros(B, d.heads, d.state, d.vdim, **f32)
+        sbytes = 2.0 * (B if kind == "decode" else 1) * d.heads * d.state * d.vdim * 4
+        u, yy = rnd(n, Cs), rnd(n, inner)
+        case(f"short_conv_{kind}", lambda: SS.short_conv(proj, inner, sw["conv"], sw["conv_b"], ring, m),
+             4.0 * n * Cs + (2 * B * 3 * Cs * 2.0 if kind == "decode" else 0))
+        case(f"state_space_scan_{kind}", lambda: SS.state_space_scan(u, proj, inner + Cs, sw, spool, m, d),
+             sbytes + n * (Cs + inner + d.heads) * 2.0)
+        case(f"group_norm_gate_{kind}", lambda: SS.group_norm_gate(yy, proj[:, :inner], sw["norm"], 8, 1e-6, inner),
+             n * inner * 6.0)
+        case(f"state_space_mixer_{kind}", lambda: SS.mixer(proj, sw, ring, spool, m, d, 1e-6),
+             sbytes + n * (2 * inner + Cs + d.heads) * 2.0)
+        # ---- rows between sublayers ----
+        nw32, mu = rnd(W, dtype=torch.float32), torch.rand(W, device=dev)
+        shift_pool = torch.zeros(B, W, **f32)
+        case(f"add_norm_rows_{kind}", lambda: F.add_norm_rows(y, res, nw32, F.NextRows(nw32), 1e-6, W),
+             n * W * (2 + 4 + 4 + 2.0))
+        case(f"add_norm_shift_rows_{kind}", lambda: F.add_norm_rows(
+            y, res, nw32, F.NextRows(nw32, mu, shift_pool, m), 1e-6, W), n * W * (2 + 4 + 4 + 2.0))
+        zf, pact = rnd(n, 8192), torch.tensor([0.4, 0.3, 0.1, 0.2], device=dev)
+        case(f"poly_norm_{kind}", lambda: F.poly_norm_(zf, pact, 8192, 1e-6), n * 8192 * 4.0)
+        # ---- latent attention: 32 heads of 128 + 64, latents of 512, window 1024 ----
+        ld = LA.LatentDims(32, 128, 64, 128, 512, 1536, 192 ** -0.5, 1024)
+        cpg, rpg = rnd(seqs * per + 1, page, 1, 512), rnd(seqs * per + 1, page, 1, 64)
+        lx, lq, lc = rnd(n, 1536 + 512 + 64), rnd(1536, dtype=torch.float32), rnd(512, dtype=torch.float32)
+        freq = LA.frequencies(64, 10000.0, dev)
+        case(f"latent_prep_{kind}", lambda: LA.latent_prep_(lx, (0, 1536, 2048), ld, lq, lc, freq, pos, slots, cpg,
+                                                            rpg, 1e-6), n * (2 * 1536 + 2 * 576) * 2.0)
+        q3 = rnd(n, 32, 192)
+        case(f"rotate_heads_{kind}", lambda: LA.rotate_heads_(q3, 128, pos, freq), n * 32 * 64 * 4.0)
+        wab, wuv = rnd(32, 512, 128), rnd(32, 128, 512)
+        ql, lat, att = rnd(n, 32, 512), rnd(n, 32, 512), torch.empty(n, 32, 128, dtype=bf, device=dev)
+        case(f"head_linear_absorb_{kind}", lambda: LA.head_linear(wab, q3, ql),
+             32 * 512 * 128 * 2.0 + n * 32 * 640 * 2.0, 2.0 * n * 32 * 512 * 128)
+        case(f"head_linear_values_{kind}", lambda: LA.head_linear(wuv, lat, att),
+             32 * 512 * 128 * 2.0 + n * 32 * 640 * 2.0, 2.0 * n * 32 * 512 * 128)
+        case(f"latent_attention_{kind}", lambda: LA.latent_attention(
+            ql, q3[:, :, 128:], cpg, rpg, m, pt, ld, seq_lens=sl if kind == "decode" else None, max_k=ctx),
+            2.0 * (B * 1024 if kind == "decode" else n) * 576 + n * 32 * (576 + 512) * 2.0,
+            (1024.0 * B if kind == "decode" else 1024.0 * n) * 32 * 2 * (576 + 512))
 
 
 def F_flash(q, k, v, cu, n):
