@@ -575,6 +575,58 @@ def test_latent_attention_alone(form, case):
     settled(dev)
 
 
+EXPANDED = [(4, 20, 12, 17, 36, 19), (2, 64, 64, 64, 64, 0), (3, 128, 64, 128, 512, 70), (5, 96, 40, 100, 128, 129),
+            (2, 128, 32, 64, 72, 300), (4, 64, 16, 128, 64, 1), (2, 136, 16, 32, 64, 40), (3, 40, 64, 96, 520, 128)]
+
+
+@pytest.mark.parametrize("form", FORMS)
+@pytest.mark.parametrize("case", EXPANDED, ids=str)
+def test_latent_attention_of_prompts_alone(form, case):
+    """Expanded and absorbed rows of one batch: whole prompts longer than two query tiles, portions
+    that start inside a page, a window or a key block, short ones and single rows between them; one
+    key stands out per probed query, at the edges of the window, of pages and of key blocks."""
+    H, D, RD, V, R, size = case
+    g = gen(H * R + D)
+    scale, page, dev, win = 0.11, 16, form[0], size or 10000
+    lens = [430, 37, 150]
+    d = LA.LatentDims(H, D, RD, V, R, 8, scale, size)
+    q = [rnd(g, T, H, D + RD, std=0.3) for T in lens]
+    c, kr = [rnd(g, T, R) for T in lens], [rnd(g, T, RD) for T in lens]
+    uk, uv = rnd(g, H, D, R, std=R ** -0.5), rnd(g, H, V, R, std=R ** -0.5)
+    uk, uv = as_typed(form, uk, uv)
+    c, kr = ([as_typed(form, t) for t in x] for x in (c, kr))
+    k = [torch.cat([torch.einsum("hdr,tr->thd", uk, a), b[:, None].expand(-1, H, -1)], -1) for a, b in zip(c, kr)]
+    T = lens[0]
+    for i, j in ((T - 1, T - win), (T - 2, T - 2 - win), (T - 3, 0), (300, 300 - win + 1), (301, 301 - win), (260, 128),
+                 (261, 127), (262, 256), (263, 255), (129, 128), (140, 15), (141, 16), (90, 90), (200, 199)):
+        if 0 <= j <= i:                             # query i points along key j
+            q[0][i] = k[0][j] / k[0][j].norm(dim=-1, keepdim=True) * 12.0 / (scale * k[0][j].norm(dim=-1, keepdim=True))
+    q = [as_typed(form, t) for t in q]
+    want = [P.windowed_attention(a, b, torch.einsum("hvr,tr->thv", uv, e), scale, win) for a, b, e in zip(q, k, c)]
+    (cp, rp), pt = paged([c, kr], page, dev, form[1], g)
+    Dp, RDp = LA.query_layout(d, form[1])
+    Rp, dv, ldo = cp.shape[-1], LA.value_layout(d), (H * V + 7) // 8 * 8
+    cp[..., R:], rp[..., RD:] = 0, 0
+    w = {"absorb": torch.zeros(H, Rp, (D + 7) // 8 * 8), "uv": torch.zeros(H, V, Rp)}
+    w["absorb"][:, :R, :D], w["uv"][..., :R] = uk.transpose(1, 2), uv
+    if LA.expands(d, form[1]):
+        kv = torch.zeros(H * (Dp + dv), Rp)
+        kv[:H * Dp].view(H, Dp, Rp)[:, :D, :R], kv[H * Dp:].view(H, dv, Rp)[:, :V, :R] = uk, uv
+        w["kv"] = kv
+    w = {n: to(form, t) for n, t in w.items()}
+    for spans in ([(0, 430), (0, 37), (0, 150)], [(300, 430), (36, 37), (0, 150)], [(129, 145), (5, 20), (149, 150)],
+                  [(100, 103), (0, 2), (20, 21)], [(255, 302), (0, 15), (1, 150)]):
+        rows = torch.cat([a[lo:hi] for a, (lo, hi) in zip(q, spans)])
+        m = seq_meta([hi - lo for lo, hi in spans], [lo for lo, _ in spans], [0, 1, 2], dev)
+        qq = torch.zeros(rows.shape[0], H, Dp + RDp)
+        qq[..., :D], qq[..., Dp:Dp + RD] = rows[..., :D], rows[..., D:]
+        out = LA.attend(to(form, qq), Dp, w, cp, rp, m, pt, d, ldo)
+        ref = torch.cat([a[lo:hi] for a, (lo, hi) in zip(want, spans)]).flatten(1)
+        close(out[:, :H * V], ref, form[1], f"spans {spans}", 1.5)
+        assert ldo == H * V or float(out[:, H * V:].float().abs().max()) == 0.0
+    settled(dev)
+
+
 @pytest.mark.parametrize("form", FORMS)
 @pytest.mark.parametrize("H,D,RD,turned,V,R,Q", [(5, 20, 12, 8, 28, 36, 44), (2, 64, 64, 64, 64, 512, 96), (3, 7, 6, 6, 9, 33, 17)])
 def test_latent_projections_norms_and_rotation_alone(form, H, D, RD, turned, V, R, Q):

@@ -47,7 +47,8 @@ GROUPS = {
                  "misc.cu", "sampler.cu", "row_ops.cu", "vector_delta.cu", "head_mix_attn.cu"),
                 ("block_manager.cpp",)),
     "zonopel": (("runtime.cu", "gemm_tc05.cu", "linear_decode.cu", "gemm_f32.cu", "misc.cu", "sampler.cu",
-                 "stream_rows.cu", "state_space.cu", "state_space_chunk.cu", "latent_attn.cu", "latent_decode.cu"),
+                 "stream_rows.cu", "state_space.cu", "state_space_chunk.cu", "latent_attn.cu", "latent_decode.cu",
+                 "latent_flash_tc05.cu"),
                 ("block_manager.cpp",)),
 }
 CXX_FLAGS = ["-O3", "-std=c++17", "-fPIC", "-fvisibility=hidden", "-pthread", "-Wall"]

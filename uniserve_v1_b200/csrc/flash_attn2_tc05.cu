@@ -26,10 +26,13 @@
 // same idea, the code is independent.
 #include <mutex>
 #include "include/us_common.cuh"
+#include "include/us_flash.cuh"
 #include "include/us_tc05.cuh"
 #include "include/us_tmap.h"
 
 namespace {
+
+using namespace flash;
 
 constexpr int kDMax = 128;  // head widths served: 128 and 64 (template parameter kD)
 constexpr int kBM = 128;   // query rows per tile (two tiles per CTA)
@@ -65,33 +68,6 @@ struct Flash2Args {
   int tail_follows; // the next launch is this one's tail and has no_wait set
 };
 
-__device__ __forceinline__ float ex2f(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-
-// Packed FP32 pairs (two lanes per instruction) and the three-input maximum: the
-// softmax warpgroups are bound by instruction issue, not by the special-function unit.
-__device__ __forceinline__ unsigned long long pack2(float a, float b) {
-  unsigned long long r;
-  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
-  return r;
-}
-__device__ __forceinline__ void unpack2(unsigned long long r, float& a, float& b) {
-  asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(r));
-}
-__device__ __forceinline__ unsigned long long fma2(unsigned long long a, unsigned long long b,
-                                                   unsigned long long c) {
-  unsigned long long d;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-  return d;
-}
-__device__ __forceinline__ unsigned long long add2(unsigned long long a, unsigned long long b) {
-  unsigned long long d;
-  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
-  return d;
-}
 __device__ __forceinline__ unsigned long long add2_rm(unsigned long long a, unsigned long long b) {
   unsigned long long d;
   asm("add.rm.ftz.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
@@ -120,65 +96,6 @@ __device__ __forceinline__ void ex2_poly2(float t0, float t1, float& p0, float& 
   p0 = __uint_as_float(__float_as_uint(q0) + (__float_as_uint(u0) << 23));
   p1 = __uint_as_float(__float_as_uint(q1) + (__float_as_uint(u1) << 23));
 }
-// tcgen05.mma with the shared-memory descriptors given as (low, high) words.  The thread that
-// issues the products is a single instruction stream: with 64 cycles of tensor work per
-// 128 x 128 x 16 product, a dozen dependent instructions of 64-bit descriptor arithmetic per
-// product make the issue the limit.  The high words are constants of the layout and the low
-// words (start address in 16-byte units) advance by compile-time offsets, so a product costs
-// one 32-bit add per operand.
-//
-// The whole issuing warp runs the loop and one elected lane executes each tcgen05 instruction:
-// addresses, descriptors and loop control are then the same in all lanes, which lets the
-// compiler keep them in the uniform datapath where the instruction takes its operands from
-// (a single lane inside a divergent branch computes them in vector registers and moves every
-// operand of every product across).
-__device__ __forceinline__ void umma_f16_words(uint32_t tmem_d, uint32_t a_lo, uint32_t a_hi,
-                                               uint32_t b_lo, uint32_t b_hi, uint32_t idesc,
-                                               uint32_t accumulate) {
-  asm volatile(
-      "{\n"
-      ".reg .pred p, q;\n"
-      ".reg .b64 da, db;\n"
-      "mov.b64 da, {%1, %2};\n"
-      "mov.b64 db, {%3, %4};\n"
-      "setp.ne.b32 p, %6, 0;\n"
-      "elect.sync _|q, 0xffffffff;\n"
-      "@q tcgen05.mma.cta_group::1.kind::f16 [%0], da, db, %5, p;\n"
-      "}\n" ::"r"(tmem_d),
-      "r"(a_lo), "r"(a_hi), "r"(b_lo), "r"(b_hi), "r"(idesc), "r"(accumulate)
-      : "memory");
-}
-__device__ __forceinline__ void umma_f16_ts_words(uint32_t tmem_d, uint32_t tmem_a, uint32_t b_lo,
-                                                  uint32_t b_hi, uint32_t idesc,
-                                                  uint32_t accumulate) {
-  asm volatile(
-      "{\n"
-      ".reg .pred p, q;\n"
-      ".reg .b64 db;\n"
-      "mov.b64 db, {%2, %3};\n"
-      "setp.ne.b32 p, %5, 0;\n"
-      "elect.sync _|q, 0xffffffff;\n"
-      "@q tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], db, %4, p;\n"
-      "}\n" ::"r"(tmem_d),
-      "r"(tmem_a), "r"(b_lo), "r"(b_hi), "r"(idesc), "r"(accumulate)
-      : "memory");
-}
-// tcgen05.commit by one elected lane of a converged warp.
-__device__ __forceinline__ void umma_commit_elect(uint64_t* bar) {
-  asm volatile(
-      "{\n"
-      ".reg .pred q;\n"
-      "elect.sync _|q, 0xffffffff;\n"
-      "@q tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];\n"
-      "}\n" ::"r"(tc::smem_u32(bar))
-      : "memory");
-}
-__device__ __forceinline__ float max3(float a, float b, float c) {
-  float d;
-  asm("max.f32 %0, %1, %2, %3;" : "=f"(d) : "f"(a), "f"(b), "f"(c));
-  return d;
-}
-
 // kEmu: which of every eight exponential pairs go to the polynomial (bit = pair slot).
 // kSplit: threads per query row.  1: a warpgroup per tile, a thread owns a whole row of S
 // (128 columns).  2: two warpgroups per tile, a thread owns half a row (64 columns); the two

@@ -58,18 +58,19 @@ __global__ void __launch_bounds__(kThreads, 2) latent_decode_kernel(const Decode
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int lrow = lane & 15, lhalf = lane >> 4, r0 = lane >> 2, cq = (lane & 3) * 2;
   const int split = blockIdx.x, h0 = blockIdx.y * HT, nh = min(HT, a.H - h0);
-  const long long t = a.rows ? a.rows[blockIdx.z] : (int)blockIdx.z;
+  const long long t = blockIdx.z;         // row of ql, qr and out
+  const int row = a.rows ? a.rows[t] : (int)t;                  // row of the packed batch
   int s = blockIdx.z;
   if (a.rows) {
     int lo = 0, hi = a.B - 1;
     while (lo < hi) {
       const int mid = (lo + hi + 1) >> 1;
-      if (a.cu[mid] <= (int)t) lo = mid; else hi = mid - 1;
+      if (a.cu[mid] <= row) lo = mid; else hi = mid - 1;
     }
     s = lo;
   }
   const bool live = !a.seq_lens || a.seq_lens[s] > 0;           // the same in the whole cluster
-  const int i = live ? a.pos[t] : -1;
+  const int i = live ? a.pos[row] : -1;
   const int first = a.window > 0 ? max(0, i - a.window + 1) : 0;
   const int n = i + 1 - first;
   const int per = ((n + a.splits - 1) / a.splits + kTile - 1) / kTile * kTile;
@@ -343,8 +344,8 @@ int launch_decode(const DecodeArgs& a, int rows, cudaStream_t stream) {
 
 }  // namespace
 
-// `count` single rows: row indices `rows` (of sequence cu[s] <= row < cu[s + 1]), or rows null: row i
-// is sequence i's only one.
+// `count` single rows: rows `rows` of the packed batch (sequence s has cu[s] .. cu[s + 1]), packed in ql, qr
+// and out; rows null: row i is sequence i's only one.
 US_API int us_latent_decode(const void* ql, long long ldql, int hsql, const void* qr, long long ldqr,
                             int hsqr, const void* cpages, int ldc, const void* rpages, int ldr,
                             void* out, long long ldo, int hso, const int* rows, const int* cu,

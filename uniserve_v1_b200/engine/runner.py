@@ -740,7 +740,8 @@ class CausalLmRunner:
             page_table = page_table.to(dev)
         meta = AttnMeta(kind="prefill", slots=d[2 * T:3 * T], cu_q=d[3 * T:3 * T + nq],
                         cu_k=d[3 * T + nq:3 * T + 2 * nq], max_q=max_q, max_k=max_k,
-                        context_lens=ctx, page_table=page_table, live=live, rows_real=T_real,
+                        context_lens=ctx, q_lens=[c.length for c in chunks], page_table=page_table,
+                        live=live, rows_real=T_real,
                         state_slots=d[3 * T + 2 * nq:], states=self.states)
         if page_table is not None and dev.type == "cuda" and not self.attends_pages:
             from ..ops.attention import context_tables

@@ -148,6 +148,7 @@ class AttnMeta:
     max_q: int = 0
     max_k: int = 0
     context_lens: Optional[list] = None         # per sequence keys already in the cache
+    q_lens: Optional[list] = None               # per sequence rows of this call
     logits_rows: Optional[torch.Tensor] = None  # rows whose logits are needed (int32)
     live: Optional[torch.Tensor] = None         # device word: rows that are real (padding after)
     rows_real: Optional[int] = None             # prefill padded to a capacity: rows before the padding

@@ -186,16 +186,22 @@ class ZonopelModel(LayeredDecoder):
         w["q_norm"], w["kv_norm"] = norm(p + "dq.norm", Q), norm(p + "dkv.norm", R)
         w["freq"] = LA.frequencies(L.rot_dims, L.rot_base, self.device)
         # queries head by head as [unrotated | rotated], each section padded
-        Dp, RDp, Rp = pad8(D), pad8(RD), pad8(R)
+        (Dp, RDp), Rp = LA.query_layout(s, self.dtype), pad8(R)
         q = need(p + "uq", H * (D + RD), Q).view(H, D + RD, Q)
         uq = torch.zeros(H, Dp + RDp, pad8(Q), dtype=self.dtype, device=self.device)
         uq[:, :D, :Q], uq[:, Dp:Dp + RD, :Q] = self._put(q[:, :D]), self._put(q[:, D:])
         w["uq"] = uq.view(H * (Dp + RDp), pad8(Q))
         uk, uv = need(p + "uk", H * D, R).view(H, D, R), need(p + "uv", H * V, R).view(H, V, R)
-        w["absorb"] = torch.zeros(H, Rp, Dp, dtype=self.dtype, device=self.device)
+        w["absorb"] = torch.zeros(H, Rp, pad8(D), dtype=self.dtype, device=self.device)
         w["absorb"][:, :R, :D] = self._put(uk).transpose(1, 2)
         w["uv"] = torch.zeros(H, V, Rp, dtype=self.dtype, device=self.device)
         w["uv"][:, :, :R] = self._put(uv)
+        if LA.expands(s, self.dtype) and self.device.type == "cuda":
+            dv = LA.value_layout(s)
+            kv = torch.zeros(H * (Dp + dv), Rp, dtype=self.dtype, device=self.device)
+            kv[:H * Dp].view(H, Dp, Rp)[:, :D, :R] = self._put(uk)
+            kv[H * Dp:].view(H, dv, Rp)[:, :V, :R] = self._put(uv)
+            w["kv"] = kv
         w["o"] = self._matrix(need(p + "o", W, H * V))
 
     def random_state(self, seed: int = 0) -> dict:
@@ -279,26 +285,21 @@ class ZonopelModel(LayeredDecoder):
     # ------------------------------------------------------------- forward --
     def _latent_attention(self, L: LayerSpec, w, x, m: SeqMeta, meta, caches):
         s, (cp, rp) = L.mixer, caches
-        T, H, Dp, RDp = x.shape[0], s.heads, pad8(s.dim), pad8(s.rot_dim)
+        T, H, (Dp, RDp) = x.shape[0], s.heads, LA.query_layout(s, self.dtype)
         proj = F.linear(x, w["proj"])
         LA.latent_prep_(proj, w["offs"], s, w["q_norm"], w["kv_norm"], w["freq"], m.positions, meta.slots,
                         cp, rp, self.cfg.eps)
         oq = w["offs"][0]
         q = F.linear(proj[:, oq:oq + pad8(s.q_rank)], w["uq"]).view(T, H, Dp + RDp)
         LA.rotate_heads_(q, Dp, m.positions, w["freq"])
-        ql = LA.head_linear(w["absorb"], q, torch.empty(T, H, cp.shape[-1], dtype=q.dtype, device=q.device))
-        lat = LA.latent_attention(ql, q[:, :, Dp:], cp, rp, m, meta.page_table, s, seq_lens=meta.seq_lens,
-                                  max_k=meta.max_k)
-        n, ldo = H * s.vdim, w["o"].shape[1]
-        att = (torch.empty if ldo == n else torch.zeros)(T, ldo, dtype=x.dtype, device=x.device)
-        LA.head_linear(w["uv"], lat, att[:, :n].unflatten(1, (H, s.vdim)))
+        att = LA.attend(q, Dp, w, cp, rp, m, meta.page_table, s, w["o"].shape[1], meta.seq_lens, meta.max_k)
         return F.linear(att, w["o"])
 
     def forward(self, input_ids, positions, meta, kv_caches) -> torch.Tensor:
         """Final-normed rows [T, Wp] of the packed batch ``meta`` (``cu_q``, ``state_slots``,
         ``page_table``, ``slots``); ``meta.states`` are the pools of ``new_state_pools``."""
         c, states = self.cfg, meta.states
-        m = SeqMeta(meta.cu_q, meta.state_slots, positions, meta.kind == "decode")
+        m = SeqMeta(meta.cu_q, meta.state_slots, positions, meta.kind == "decode", meta.context_lens, meta.q_lens)
         n = len(c.layers)
 
         def entry(i):                    # the input rows of layer i, or of the output projection

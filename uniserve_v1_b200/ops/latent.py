@@ -15,19 +15,26 @@ from dataclasses import dataclass
 
 import torch
 
+from . import functional as F
 from . import native as N
 from .vector_delta import BF16, SeqMeta
 
-P, I, L, F = N.P, N.I, N.L, N.F
+P, I, L = N.P, N.I, N.L
 N.register_signatures({
-    "us_latent_prep": (I, [P, L, I, I, I, I, I, I, P, P, P, I, P, P, P, I, P, I, I, F, I, P]),
+    "us_latent_prep": (I, [P, L, I, I, I, I, I, I, P, P, P, I, P, P, P, I, P, I, I, N.F, I, P]),
     "us_rotate_heads": (I, [P, L, I, I, I, P, I, P, I, I, P]),
     "us_head_linear": (I, [P, P, P, L, L, L, L, L, L, I, I, I, I, I, P]),
     "us_latent_attention_rows": (I, [P, L, I, P, L, I, P, I, P, I, P, L, I, P, P, P, P, I, I, I, I, I, I,
-                                     I, I, F, I, P]),
+                                     I, I, N.F, I, P]),
     "us_latent_decode": (I, [P, L, I, P, L, I, P, I, P, I, P, L, I, P, P, P, P, P, I, I, I, I, I, I, I, I, I,
-                             F, P]),
+                             N.F, P]),
+    "us_latent_gather": (I, [P, I, P, I, P, P, P, P, P, P, I, I, I, I, I, I, P]),
+    "us_latent_flash": (I, [P, L, P, L, P, P, L, P, P, I, I, I, I, I, I, I, I, I, N.F, P]),
 })
+
+# sequences that bring at least this many rows take the expanded form (an absorbed row costs a pass
+# over the latents in view, an expanded prompt their expansion once)
+EXPAND_ROWS = 16
 
 
 @dataclass(frozen=True)
@@ -122,17 +129,18 @@ def decode_splits(rows: int, heads: int, keys: int) -> int:
 
 
 def latent_attention(ql, qr, cpages, rpages, m: SeqMeta, page_table, d: LatentDims, seq_lens=None, max_k=0,
-                     rows=None, out=None):
+                     rows=None):
     """Absorbed form over pages: ql [T, H, Rp], qr [T, H, >= rot_dim] (strided views) -> mixtures of
     latents [T, H, Rp].  ``seq_lens``: one row per sequence, length 0 marks padding; ``max_k`` bounds
-    the keys of a sequence.  ``rows`` (int32): only these rows, into ``out``."""
+    the keys of a sequence.  ``rows`` (int32): the rows of the packed batch that ql and qr hold."""
     T, H = ql.shape[:2]
     page, Rp, RDp = cpages.shape[1], cpages.shape[-1], rpages.shape[-1]
     R, RD = d.kv_rank, d.rot_dim
     if ql.is_cuda:
-        if out is None:
-            out = torch.empty(T, H, Rp, dtype=ql.dtype, device=ql.device)
-        if (rows is not None or m.one_token) and decode_fits(ql, cpages, rpages):
+        out = torch.empty(T, H, Rp, dtype=ql.dtype, device=ql.device)
+        if decode_fits(ql, cpages, rpages):
+            if rows is None and not m.one_token:
+                rows = torch.arange(T, dtype=torch.int32, device=ql.device)
             count = T if rows is None else rows.shape[0]
             keys = max_k or page * page_table.shape[1]
             keys = min(keys, d.window) if d.window > 0 else keys
@@ -167,4 +175,69 @@ def latent_attention(ql, qr, cpages, rpages, m: SeqMeta, page_table, d: LatentDi
             see = see & (gap < d.window)
         p = sc.masked_fill(~see[None], float("-inf")).softmax(-1)
         out[lo:hi, :, :R] = torch.einsum("htn,nr->thr", p, c).to(out.dtype)
+    return out
+
+
+def expands(d: LatentDims, dtype) -> bool:
+    """Whether prompts take the expanded form."""
+    return dtype == BF16 and d.dim <= 128 and d.rot_dim <= 64 and d.vdim <= 128
+
+
+def query_layout(d: LatentDims, dtype):
+    """Columns (unrotated, rotated) a head's query takes: slabs of 64 where a flash kernel reads it."""
+    n = 64 if expands(d, dtype) else 8
+    return -(-d.dim // n) * n, -(-d.rot_dim // n) * n
+
+
+def value_layout(d: LatentDims) -> int:
+    """Columns a head's expanded value takes."""
+    return 64 if d.vdim <= 64 else 128
+
+
+def expanded_attention(q, w_kv, cpages, rpages, m: SeqMeta, page_table, d: LatentDims, out, least):
+    """Prompts: rows of the sequences that bring at least ``least`` rows, into ``out`` [T, >= H * vdim].
+    q [T, H, columns of ``query_layout``], ``w_kv`` the stacked expansion [H * slabs * 64 | H * dv, Rp]."""
+    T, H, W = q.shape
+    Rp, RDp, dev = cpages.shape[-1], rpages.shape[-1], q.device
+    starts, lengths = m.host()
+    seen = [n + (p if d.window <= 0 else min(p, d.window - 1)) for p, n in zip(starts, lengths) if n >= least]
+    Tk, B = sum(seen), m.cu.shape[0] - 1
+    c = torch.empty(Tk, Rp, dtype=q.dtype, device=dev)
+    r = torch.empty(Tk, 64, dtype=q.dtype, device=dev)
+    cu_k = torch.empty(B + 1, dtype=torch.int32, device=dev)
+    N.call("us_latent_gather", N.ptr(cpages), Rp, N.ptr(rpages), RDp, N.ptr(c), N.ptr(r), N.ptr(cu_k),
+           N.ptr(m.cu), N.ptr(m.positions), N.ptr(page_table), B, cpages.shape[1], page_table.shape[1],
+           d.window, least, Tk, N.stream())
+    kv = F.linear(c, w_kv)
+    N.call("us_latent_flash", N.ptr(q), q.stride(0), N.ptr(kv), kv.stride(0), N.ptr(r), N.ptr(out),
+           out.stride(0), N.ptr(m.cu), N.ptr(cu_k), B, T, Tk, H, W // 64 - 1, value_layout(d), d.vdim,
+           max(n for n in lengths if n >= least), d.window, d.scale, N.stream())
+
+
+def attend(q, off, w, cpages, rpages, m: SeqMeta, page_table, d: LatentDims, ldo, seq_lens=None, max_k=0):
+    """Attention of query rows q [T, H, n] (unrotated channels first, the turned ones at column
+    ``off``) over pages -> rows [T, ldo] of all heads' outputs (zero past H * vdim).  ``w``: 'absorb'
+    [H, Rp, dim], 'uv' [H, vdim, Rp] and, where ``expands``, 'kv'."""
+    T, H = q.shape[:2]
+    n = H * d.vdim
+    out = (torch.empty if ldo == n else torch.zeros)(T, ldo, dtype=q.dtype, device=q.device)
+
+    def absorbed(q, out, rows=None):
+        ql = torch.empty(q.shape[0], H, cpages.shape[-1], dtype=q.dtype, device=q.device)
+        head_linear(w["absorb"], q, ql)
+        lat = latent_attention(ql, q[:, :, off:], cpages, rpages, m, page_table, d, seq_lens, max_k, rows)
+        head_linear(w["uv"], lat, out[:, :n].unflatten(1, (H, d.vdim)))
+    if not (q.is_cuda and "kv" in w) or m.one_token:
+        absorbed(q, out)
+        return out
+    least = EXPAND_ROWS if decode_fits(q, cpages, rpages) else 1
+    short = m.short_rows(least)
+    if short is None or short.shape[0] < T:
+        expanded_attention(q, w["kv"], cpages, rpages, m, page_table, d, out, least)
+    if short is not None and short.shape[0] == T:
+        absorbed(q, out, short)
+    elif short is not None:
+        part = torch.zeros(short.shape[0], ldo, dtype=q.dtype, device=q.device)
+        absorbed(F.gather_rows(q.view(T, -1), short).view(-1, *q.shape[1:]), part, short)
+        out.index_copy_(0, short.long(), part)
     return out

@@ -12,6 +12,7 @@ from __future__ import annotations
 
 import math
 from dataclasses import dataclass
+from typing import Optional
 
 import torch
 
@@ -29,6 +30,29 @@ class SeqMeta:
     slots: torch.Tensor         # [B] int32 state slot of every sequence
     positions: torch.Tensor     # [T] int32
     one_token: bool             # every sequence brings exactly one row
+    starts: Optional[list] = None    # on the host: first position and number of rows of every
+    lengths: Optional[list] = None   # sequence (read back from the device when not given)
+    short: Optional[tuple] = None    # cache of ``short_rows``
+
+    def host(self):
+        if self.lengths is None:
+            cu, pos = self.cu.tolist(), self.positions.tolist()
+            self.lengths = [b - a for a, b in zip(cu, cu[1:])]
+            self.starts = [pos[a] if b > a else 0 for a, b in zip(cu, cu[1:])]
+        return self.starts, self.lengths
+
+    def short_rows(self, least: int):
+        """Rows of the sequences that bring fewer than ``least`` (int32 on the device), None if there
+        are none."""
+        if self.short is None or self.short[0] != least:
+            rows, at = [], 0
+            for n in self.host()[1]:
+                if n < least:
+                    rows.extend(range(at, at + n))
+                at += n
+            self.short = (least, torch.tensor(rows, dtype=torch.int32, pin_memory=self.cu.is_cuda)
+                          .to(self.cu.device, non_blocking=True) if rows else None)
+        return self.short[1]
 
 
 def _spans(m: SeqMeta):

@@ -18,6 +18,7 @@ import torch
 from ..ops import functional as F
 from ..ops import gated_delta as GD
 from ..ops import latent as LA
+from ..ops import native as N
 from ..ops import state_space as SS
 from ..ops import vector_delta as VD
 from .opbench import peaks, timeit
@@ -227,10 +228,25 @@ def main():
              32 * 512 * 128 * 2.0 + n * 32 * 640 * 2.0, 2.0 * n * 32 * 512 * 128)
         case(f"head_linear_values_{kind}", lambda: LA.head_linear(wuv, lat, att),
              32 * 512 * 128 * 2.0 + n * 32 * 640 * 2.0, 2.0 * n * 32 * 512 * 128)
-        case(f"latent_attention_{kind}", lambda: LA.latent_attention(
-            ql, q3[:, :, 128:], cpg, rpg, m, pt, ld, seq_lens=sl if kind == "decode" else None, max_k=ctx),
-            2.0 * (B * 1024 if kind == "decode" else n) * 576 + n * 32 * (576 + 512) * 2.0,
-            (1024.0 * B if kind == "decode" else 1024.0 * n) * 32 * 2 * (576 + 512))
+        if kind == "decode":
+            case("latent_attention_decode", lambda: LA.latent_attention(
+                ql, q3[:, :, 128:], cpg, rpg, m, pt, ld, seq_lens=sl, max_k=ctx),
+                2.0 * B * 1024 * 576 + n * 32 * (576 + 512) * 2.0, 1024.0 * B * 32 * 2 * (576 + 512))
+        else:
+            m.starts, m.lengths = [0], [n]
+            wl = {"absorb": wab, "uv": wuv, "kv": rnd(32 * 256, 512)}
+            for win in (1024, 0):
+                lw = LA.LatentDims(32, 128, 64, 128, 512, 1536, 192 ** -0.5, win)
+                pairs = sum(min(i + 1, win or n) for i in range(n))
+                case(f"latent_attention_prefill, window {win} (expansion and attention)",
+                     lambda: LA.attend(q3, 128, wl, cpg, rpg, m, pt, lw, 32 * 128), None,
+                     pairs * 32 * 2.0 * (192 + 128) + 2.0 * n * 512 * 32 * 256)
+                kvx, rx = rnd(n, 32 * 256), rnd(n, 64)
+                cuk = i32([0, n])
+                case(f"latent_flash_prefill, window {win}", lambda: N.call(
+                    "us_latent_flash", N.ptr(q3), 32 * 192, N.ptr(kvx), 32 * 256, N.ptr(rx), N.ptr(att), 32 * 128,
+                    N.ptr(m.cu), N.ptr(cuk), 1, n, n, 32, 2, 128, 128, n, win, 0.07, N.stream()), None,
+                    pairs * 32 * 2.0 * (192 + 128))
 
 
 def F_flash(q, k, v, cu, n):
