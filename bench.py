@@ -629,12 +629,12 @@ def qwen3_record(job: Job) -> dict:
     return rec
 
 
-# ------------------------------------------------------------------ Nepevik --
-def nepevik_record(job: Job) -> dict:
-    """Prefill and decode throughput of the Nepevik decoder at a production-like layer size
-    (random weights) through ``LLMEngine``, beside two existing models of equal size: the
-    Qwen3.5-style hybrid (gated delta net, dense-state engine) and Qwen3-MoE (attention in every
-    layer, the same paged engine).  One GPU.
+# ------------------------------------------------- decoders of unlike layers --
+def layered_record(job: Job, family: str) -> dict:
+    """Prefill and decode throughput of the Nepevik or Zonopel decoder at a production-like layer
+    size (random weights) through ``LLMEngine``, beside existing models of equal size: Nepevik beside
+    the Qwen3.5-style hybrid (gated delta net, dense-state engine) and Qwen3-MoE (attention in every
+    layer, the same paged engine), Zonopel beside Nepevik and Qwen3-MoE.  One GPU.
 
     ``value``: output tokens/s of the device-timed decode step of all concurrent requests (graph
     replays); ``sizes``: the same and the prompt throughput per (requests, prompt length)."""
@@ -645,6 +645,7 @@ def nepevik_record(job: Job) -> dict:
     from uniserve_v1_b200.models.nepevik import NepevikConfig, NepevikModel
     from uniserve_v1_b200.models.qwen3_5 import Qwen35Config, Qwen35MoeModel
     from uniserve_v1_b200.models.qwen3_moe import Qwen3MoeConfig, Qwen3MoeModel
+    from uniserve_v1_b200.models.zonopel import ZonopelConfig, ZonopelModel
     from uniserve_v1_b200.ops import native
 
     args, dev = job.args, job.dev
@@ -654,7 +655,8 @@ def nepevik_record(job: Job) -> dict:
     sizes = [(args.concurrency, args.prompt_len)] if args.concurrency and args.prompt_len \
         else [(64, 1024), (8, 4096), (1, 4096)]
     ncfg = NepevikConfig.bench(layers)
-    ncfg.vocab_size = vocab
+    zcfg = ZonopelConfig.bench(layers)
+    ncfg.vocab_size = zcfg.vocab_size = vocab
     hcfg = Qwen35Config(vocab_size=vocab, hidden_size=2048, num_hidden_layers=layers,
                         num_attention_heads=32, num_key_value_heads=4, head_dim=128,
                         linear_num_key_heads=16, linear_num_value_heads=32, num_experts=64,
@@ -719,22 +721,25 @@ def nepevik_record(job: Job) -> dict:
                                            max_num_batched_tokens=8192, enable_prefix_cache=False)
 
     out, clocks, launches, head = [], None, 0, None
-    for name, build_model, make, graphs in (
-            ("nepevik", lambda: NepevikModel(ncfg, dev).init_random(0), paged, True),
-            ("qwen3.5-style hybrid", lambda: Qwen35MoeModel(hcfg, dev).init_random(0, std=0.02),
-             lambda m: lambda n, length: DenseStateEngine(m, max_num_seqs=n, max_model_len=length + 128,
-                                                          prefill_chunk=8192, state_cache_entries=0), False),
-            ("qwen3-moe", lambda: Qwen3MoeModel(qcfg, dev).init_random(0), paged, True)):
-        if args.only_nepevik and name != "nepevik":
-            continue
+    models = {
+        "zonopel": (lambda: ZonopelModel(zcfg, dev).init_random(0), paged, True),
+        "nepevik": (lambda: NepevikModel(ncfg, dev).init_random(0), paged, True),
+        "qwen3.5-style hybrid": (lambda: Qwen35MoeModel(hcfg, dev).init_random(0, std=0.02),
+                                 lambda m: lambda n, length: DenseStateEngine(
+                                     m, max_num_seqs=n, max_model_len=length + 128, prefill_chunk=8192,
+                                     state_cache_entries=0), False),
+        "qwen3-moe": (lambda: Qwen3MoeModel(qcfg, dev).init_random(0), paged, True)}
+    beside = {"nepevik": ("qwen3.5-style hybrid", "qwen3-moe"), "zonopel": ("nepevik", "qwen3-moe")}
+    for name in (family,) + (() if args.alone else beside[family]):
+        build_model, make, graphs = models[name]
         model = build_model()
         for n, length in sizes:
             sampler = ClockSampler(job.local, period_ms=50)
-            if name == "nepevik" and head is None:
+            if name == family and head is None:
                 sampler.start()
             l0 = native.launch_count
             pre, ms, per_step, e2e, eng = measure(make(model), n, length, graphs)
-            if name == "nepevik" and head is None:
+            if name == family and head is None:
                 clocks, launches = sampler.stop(), native.launch_count - l0
                 head = (n, length, ms, e2e, per_step)
             native.raise_on_device_error()
@@ -749,11 +754,12 @@ def nepevik_record(job: Job) -> dict:
         del model
         release_device_memory()
     n, length, ms, e2e, per_step = head
-    return {"metric": "Nepevik output tokens/s", "value": n / ms * 1e3, "unit": "tokens/s", "n_gpus": 1,
+    title = family.capitalize()
+    return {"metric": f"{title} output tokens/s", "value": n / ms * 1e3, "unit": "tokens/s", "n_gpus": 1,
             "steps": K, "warmup": W, "ms_per_step": ms, "higher_is_better": True, "scaling": "strong",
             "vs_baseline": None, "dtype": "bf16",
             "data": "synthetic (uniform-random prompt ids, random-init weights)",
-            "config": {"model": "Nepevik, layer sizes of NepevikConfig.bench", "layers": layers, "hidden": 2048,
+            "config": {"model": f"{title}, layer sizes of {title}Config.bench", "layers": layers, "hidden": 2048,
                        "vocab": vocab, "global_batch": n, "seq_len": length, "parallelism": "tp1",
                        "step": "one decode step of all concurrent requests",
                        "l2": "inputs larger than L2 (weights and state read per step >> 126 MB)"},
@@ -763,12 +769,12 @@ def nepevik_record(job: Job) -> dict:
 
 def main() -> int:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--workload", default="all", choices=["all", "qwen3-moe", "fasth3", "nepevik"],
+    ap.add_argument("--workload", default="all", choices=["all", "qwen3-moe", "fasth3", "nepevik", "zonopel"],
                     help="all (default): the FastH3 clip latency as the headline with the "
-                         "Qwen3-MoE record nested; or one of the two alone; nepevik: that decoder's "
+                         "Qwen3-MoE record nested; or one of the two alone; nepevik, zonopel: that decoder's "
                          "throughput beside models of equal size (one GPU, not part of all)")
-    ap.add_argument("--only-nepevik", action="store_true",
-                    help="nepevik: without the models it is compared with")
+    ap.add_argument("--alone", "--only-nepevik", dest="alone", action="store_true",
+                    help="nepevik, zonopel: without the models it is compared with")
     ap.add_argument("--frames", type=int, default=0, help="fasth3: frame count (rule 17n + 5)")
     ap.add_argument("--mlp-fp8", action="store_true",
                     help="fasth3: feed-forward projections in FP8 (per-tensor weights, per-row "
@@ -824,8 +830,8 @@ def main() -> int:
             line["metric"] = "FastH3 8-step clip latency (s); Qwen3-MoE output tokens/s nested"
             line["qwen3_moe"] = q
             line["gpu_launches"] = line["gpu_launches"] + q.get("gpu_launches", 0)
-    if args.workload == "nepevik":
-        line = nepevik_record(job)
+    if args.workload in ("nepevik", "zonopel"):
+        line = layered_record(job, args.workload)
     if job.rank == 0 and line:
         print(json.dumps(line))
     job.mark("line printed")

@@ -110,15 +110,15 @@ class ZonopelConfig:
     def bench(cls, layers: int = 8) -> "ZonopelConfig":
         """Layer sizes of a mid-size production decoder: width 2048, 64 state-space heads of 64 with a
         state of 128, 32 latent-attention heads of 128 + 64 over latents of 512, feed-forward
-        8192; three state-space layers for every attention layer, the last one borrowing weights."""
+        4096; three state-space layers for every attention layer, the last one borrowing weights."""
         ss = SS.StateSpaceDims(64, 64, 128, 8, 8, 4)
         at = LA.LatentDims(32, 128, 64, 128, 512, 1536, 192 ** -0.5, 1024)
         out = []
         for i in range(layers):
             if i % 4 == 3:
-                out.append(LayerSpec("latent_attention", at, 8192, 64))
+                out.append(LayerSpec("latent_attention", at, 4096, 64))
             else:
-                out.append(LayerSpec("mamba2", ss, 8192, weights_of=i - 1 if i % 4 == 2 else None))
+                out.append(LayerSpec("mamba2", ss, 4096, weights_of=i - 1 if i % 4 == 2 else None))
         return cls(151936, 2048, 1e-6, 1.0, Bigram(65521, 31, 7), out)
 
     @classmethod
