@@ -113,15 +113,17 @@ __global__ void __launch_bounds__(256) stream_rows_kernel(const StreamRows a) {
     }
     if (t0 == t1) return;
   }
-  auto source = [&](int t, float4 (&v)[NV]) {
+  // raw operands of a row: the sublayer's output (or the embedding sum) and the residual
+  auto load = [&](int t, float4 (&v)[NV], float4 (&r)[NV]) {
     const long long base = (long long)t * W;
-    float ss = 0.f;
     if (a.y) {
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
         const int c = c0 + i * step;
-        v[i] = c < W ? ld4(a.y, base + c, a.bf16) : make_float4(0.f, 0.f, 0.f, 0.f);
-        ss += sq4(v[i]);
+        v[i] = r[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (c >= W) continue;
+        v[i] = ld4(a.y, base + c, a.bf16);
+        r[i] = *reinterpret_cast<const float4*>(a.residual + base + c);
       }
     } else {
       const int id = a.ids[t], r2 = a.rows2 ? a.rows2[t] : 0;
@@ -130,22 +132,24 @@ __global__ void __launch_bounds__(256) stream_rows_kernel(const StreamRows a) {
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
         const int c = c0 + i * step;
-        v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        v[i] = r[i] = make_float4(0.f, 0.f, 0.f, 0.f);
         if (ok && c < W) {
           const float4 e = ld4(a.table, (long long)id * W + c, a.bf16);
           v[i] = make_float4(e.x * a.scale, e.y * a.scale, e.z * a.scale, e.w * a.scale);
           if (a.rows2) v[i] = add4(v[i], ld4(a.table2, (long long)r2 * W + c, a.bf16));
         }
-        ss += sq4(v[i]);
       }
     }
+  };
+  auto source = [&](float4 (&v)[NV], const float4 (&r)[NV]) {     // v becomes the row of the stream
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) ss += sq4(v[i]);
     const float inv = 1.f / sqrtf(turn_sum(ss, buf, turn) * inv_n + a.eps);
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
       const int c = c0 + i * step;
-      if (c >= W) continue;
-      v[i] = mul4(v[i], *reinterpret_cast<const float4*>(a.w + c), inv);
-      if (a.y) v[i] = add4(v[i], *reinterpret_cast<const float4*>(a.residual + base + c));
+      if (c < W) v[i] = add4(r[i], mul4(v[i], *reinterpret_cast<const float4*>(a.w + c), inv));
     }
   };
   auto norm = [&](float4 (&v)[NV]) {
@@ -165,7 +169,9 @@ __global__ void __launch_bounds__(256) stream_rows_kernel(const StreamRows a) {
 #pragma unroll
     for (int i = 0; i < NV; ++i) before[i] = make_float4(0.f, 0.f, 0.f, 0.f);
     if (t0 > start) {
-      source(t0 - 1, before);
+      float4 r[NV];
+      load(t0 - 1, before, r);
+      source(before, r);
       norm(before);
     } else if (a.slots[s] >= 0) {
       kept = a.state + (long long)a.slots[s] * W;
@@ -176,9 +182,21 @@ __global__ void __launch_bounds__(256) stream_rows_kernel(const StreamRows a) {
       }
     }
   }
-  float4 v[NV];
+  constexpr bool kAhead = NV <= 4;  // the next row's loads run under this row's sums
+  float4 v[NV], r[NV], v1[kAhead ? NV : 1], r1[kAhead ? NV : 1];
+  if constexpr (kAhead) load(t0, v1, r1);
   for (int t = t0; t < t1; ++t) {
-    source(t, v);
+    if constexpr (kAhead) {
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        v[i] = v1[i];
+        r[i] = r1[i];
+      }
+      if (t + 1 < t1) load(t + 1, v1, r1);
+    } else {
+      load(t, v, r);
+    }
+    source(v, r);
     const long long base = (long long)t * W;
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
@@ -200,7 +218,8 @@ __global__ void __launch_bounds__(256) stream_rows_kernel(const StreamRows a) {
   }
   if (!kept) return;
   if (t1 < end) {
-    source(end - 1, v);
+    load(end - 1, v, r);
+    source(v, r);
     norm(v);
   }
 #pragma unroll
@@ -310,7 +329,7 @@ US_API int us_stream_rows(const int* ids, const int* rows2, const void* table, c
   US_REQUIRE(!mu || (state && cu && slots && pos && B >= 1 && (!one_token || B == T)));
   if (T == 0) return US_OK;
   StreamRows a{ids, rows2, table, table2, scale, vocab, n2, y, residual, w, residual_out, w_out, mu,
-               state, cu, slots, pos, x, B, T, W, width, bf16, one_token, eps, T >= 2048 ? 2 : 1, us_status_ptr()};
+               state, cu, slots, pos, x, B, T, W, width, bf16, one_token, eps, T >= 2048 ? 4 : 1, us_status_ptr()};
   const int grid = !mu ? us::ceil_div(T, a.rows) : one_token ? T : T / kRows + B;
   const dim3 block(block_threads(W));
   const int nv = us::ceil_div(W, 1024);
