@@ -1,5 +1,5 @@
 // Absorbed latent attention (see latent_attn.cu) for single query rows, bf16: every head of a row
-// reads the same keys, so a key tile [32 tokens][latent | rotated part] is fetched once for up to
+// reads the same keys, so a key tile [64 tokens][latent | rotated part] is fetched once for up to
 // 32 heads and serves as keys and, by its latent columns, as values.
 //
 // A CTA takes one split of a row's keys and 16 MT heads; the splits of a row are one thread-block
@@ -13,8 +13,8 @@
 
 namespace {
 
-constexpr int kThreads = 256;
-constexpr int kTile = 32;            // keys
+constexpr int kThreads = 512, kWarps = kThreads / 32;
+constexpr int kTile = 64;            // keys
 constexpr int kRot = 64;             // rotated channels, padded
 constexpr int kPRow = kTile * 2 + 16;
 constexpr int kSRow = kTile + 8;     // floats of a head's scores (rows apart hit other banks)
@@ -40,12 +40,12 @@ __device__ __forceinline__ float ex2(float x) {
 }
 
 template <int RP, int MT>
-__global__ void __launch_bounds__(kThreads, 2) latent_decode_kernel(const DecodeArgs a) {
+__global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const DecodeArgs a) {
   US_PDL_PROLOGUE();
   constexpr int PC = RP / 8 + kRot / 8;          // 16-byte pieces per key
   constexpr int NK = RP / 16 + kRot / 16;        // 16-channel steps of a score
   constexpr int KG = 8 / MT, NS = (NK + KG - 1) / KG;
-  constexpr int NT = RP / 64;                    // 8-column value tiles per warp
+  constexpr int NT = RP >= 128 ? RP / 128 : 1;   // 8-column value tiles per warp
   constexpr int HT = 16 * MT;
   constexpr uint32_t kKeyBytes = kTile * PC * 16;
   extern __shared__ __align__(1024) uint8_t sm[];
@@ -105,8 +105,10 @@ __global__ void __launch_bounds__(kThreads, 2) latent_decode_kernel(const Decode
   };
   fetch(where(k0), 0);
   long long ahead = where(k0 + kTile);
-  // queries: warp (m, g) keeps head tile m's fragments of channel steps g, g + KG, ...
-  const int wm = warp % MT, wg = warp / MT;
+  // queries: warp (m, g) keeps head tile m's fragments of channel steps g, g + KG, ... (two warps
+  // each, for half of a tile's keys)
+  const int wm = warp % MT, wg = (warp / MT) % KG, wk = (warp / 8) * 32;
+  const bool has_values = warp * NT * 8 < RP;
   uint32_t qf[NS][4];
 #pragma unroll
   for (int x = 0; x < NS; ++x) {
@@ -160,12 +162,12 @@ __global__ void __launch_bounds__(kThreads, 2) latent_decode_kernel(const Decode
 #pragma unroll
         for (int y = 0; y < 2; ++y) {
           uint32_t b[4];
-          us::ldsm4(b, kb + us::swz(y * 16 + lrow, 2 * st + lhalf, PC));
+          us::ldsm4(b, kb + us::swz(wk + y * 16 + lrow, 2 * st + lhalf, PC));
           us::mma16816(sc[2 * y], qf[x][0], qf[x][1], qf[x][2], qf[x][3], b[0], b[2]);
           us::mma16816(sc[2 * y + 1], qf[x][0], qf[x][1], qf[x][2], qf[x][3], b[1], b[3]);
         }
       }
-      float* p = part + (wg * HT + wm * 16 + r0) * kSRow + cq;
+      float* p = part + (wg * HT + wm * 16 + r0) * kSRow + wk + cq;
 #pragma unroll
       for (int x = 0; x < 4; ++x) {
         *reinterpret_cast<float2*>(p + x * 8) = make_float2(sc[x][0], sc[x][1]);
@@ -173,17 +175,22 @@ __global__ void __launch_bounds__(kThreads, 2) latent_decode_kernel(const Decode
       }
     }
     __syncthreads();
-    {                                     // lane: key, warp: every eighth head
-      constexpr int HW = HT / 8;
-      float v[HW], m[HW], m0[HW], l[HW];
+    {                                     // lane: two keys, warp: every sixteenth head
+      constexpr int HW = HT / kWarps;
+      float v[HW][2], m[HW], m0[HW], l[HW];
 #pragma unroll
       for (int x = 0; x < HW; ++x) {
-        const int h = warp + x * 8;
-        v[x] = 0.f;
+        const int h = warp + x * kWarps;
+        float2 q = make_float2(0.f, 0.f);
 #pragma unroll
-        for (int g = 0; g < KG; ++g) v[x] += part[(g * HT + h) * kSRow + lane];
-        v[x] = j0 + lane < k1 ? v[x] * a.scale_log2 : -INFINITY;
-        m[x] = v[x];
+        for (int g = 0; g < KG; ++g) {
+          const float2 e = *reinterpret_cast<const float2*>(part + (g * HT + h) * kSRow + lane * 2);
+          q.x += e.x;
+          q.y += e.y;
+        }
+        v[x][0] = j0 + lane * 2 < k1 ? q.x * a.scale_log2 : -INFINITY;
+        v[x][1] = j0 + lane * 2 + 1 < k1 ? q.y * a.scale_log2 : -INFINITY;
+        m[x] = fmaxf(v[x][0], v[x][1]);
         m0[x] = mx[h];
       }
 #pragma unroll
@@ -193,7 +200,9 @@ __global__ void __launch_bounds__(kThreads, 2) latent_decode_kernel(const Decode
 #pragma unroll
       for (int x = 0; x < HW; ++x) {
         m[x] = fmaxf(m[x], m0[x]);
-        v[x] = l[x] = ex2(v[x] - m[x]);
+        v[x][0] = ex2(v[x][0] - m[x]);
+        v[x][1] = ex2(v[x][1] - m[x]);
+        l[x] = v[x][0] + v[x][1];
       }
 #pragma unroll
       for (int o2 = 16; o2 > 0; o2 >>= 1)
@@ -201,9 +210,9 @@ __global__ void __launch_bounds__(kThreads, 2) latent_decode_kernel(const Decode
         for (int x = 0; x < HW; ++x) l[x] += __shfl_xor_sync(0xffffffffu, l[x], o2);
 #pragma unroll
       for (int x = 0; x < HW; ++x) {
-        const int h = warp + x * 8;
-        asm volatile("st.shared.b16 [%0], %1;" ::"r"(sp + h * kPRow + lane * 2),
-                     "h"(__bfloat16_as_ushort(us::f2bf(v[x]))) : "memory");
+        const int h = warp + x * kWarps;
+        asm volatile("st.shared.u32 [%0], %1;" ::"r"(sp + h * kPRow + lane * 4),
+                     "r"(us::pack_bf(v[x][0], v[x][1])) : "memory");
         if (lane == 0) {
           const float f = ex2(m0[x] - m[x]);
           fac[h] = f;
@@ -225,32 +234,38 @@ __global__ void __launch_bounds__(kThreads, 2) latent_decode_kernel(const Decode
         o[m][x][3] *= f1;
       }
     }
-    uint32_t p[MT][2][4];
+    if (!has_values) continue;
+    uint32_t p[MT][4][4];
 #pragma unroll
     for (int m = 0; m < MT; ++m)
 #pragma unroll
-      for (int k = 0; k < 2; ++k) us::ldsm4(p[m][k], sp + (m * 16 + lrow) * kPRow + (k * 16 + lhalf * 8) * 2);
-#pragma unroll
-    for (int x = 0; x < NT; ++x) {
-      uint32_t b[4];                      // 32 keys x 8 columns
-      us::ldsm4t(b, kb + us::swz(lane, warp * NT + x, PC));
-#pragma unroll
-      for (int m = 0; m < MT; ++m) {
-        us::mma16816(o[m][x], p[m][0][0], p[m][0][1], p[m][0][2], p[m][0][3], b[0], b[1]);
-        us::mma16816(o[m][x], p[m][1][0], p[m][1][1], p[m][1][2], p[m][1][3], b[2], b[3]);
-      }
-    }
-  }
-  __syncthreads();                        // the key tiles become the partial outputs
-  float* os = reinterpret_cast<float*>(sm);                      // [HT][RP]
-#pragma unroll
-  for (int m = 0; m < MT; ++m)
+      for (int k = 0; k < 4; ++k) us::ldsm4(p[m][k], sp + (m * 16 + lrow) * kPRow + (k * 16 + lhalf * 8) * 2);
 #pragma unroll
     for (int x = 0; x < NT; ++x)
 #pragma unroll
-      for (int e = 0; e < 2; ++e)
-        *reinterpret_cast<float2*>(os + (m * 16 + r0 + e * 8) * RP + (warp * NT + x) * 8 + cq) =
-            make_float2(o[m][x][e * 2], o[m][x][e * 2 + 1]);
+      for (int y = 0; y < 2; ++y) {
+        uint32_t b[4];                    // 32 keys x 8 columns
+        us::ldsm4t(b, kb + us::swz(y * 32 + lane, warp * NT + x, PC));
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+          us::mma16816(o[m][x], p[m][2 * y][0], p[m][2 * y][1], p[m][2 * y][2], p[m][2 * y][3], b[0], b[1]);
+          us::mma16816(o[m][x], p[m][2 * y + 1][0], p[m][2 * y + 1][1], p[m][2 * y + 1][2],
+                       p[m][2 * y + 1][3], b[2], b[3]);
+        }
+      }
+  }
+  __syncthreads();                        // the key tiles become the partial outputs
+  float* os = reinterpret_cast<float*>(sm);                      // [HT][RP]
+  if (has_values) {
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int x = 0; x < NT; ++x)
+#pragma unroll
+        for (int e = 0; e < 2; ++e)
+          *reinterpret_cast<float2*>(os + (m * 16 + r0 + e * 8) * RP + (warp * NT + x) * 8 + cq) =
+              make_float2(o[m][x][e * 2], o[m][x][e * 2 + 1]);
+  }
   __syncthreads();
   if (a.splits > 1) tc::cluster_sync();
   // every CTA of the cluster finishes a share of the heads' columns, adding the splits in order:

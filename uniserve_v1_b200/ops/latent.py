@@ -123,9 +123,9 @@ def decode_fits(ql, cpages, rpages) -> bool:
 
 
 def decode_splits(rows: int, heads: int, keys: int) -> int:
-    """Key splits per row: up to two CTAs per SM, at least 64 keys each."""
+    """Key splits per row: one CTA per SM, at least 64 keys each."""
     ctas = rows * -(-heads // (16 if heads <= 16 else 32))
-    return max(1, min(296 // ctas, keys // 64, 8))
+    return max(1, min(148 // ctas, keys // 64, 8))
 
 
 def latent_attention(ql, qr, cpages, rpages, m: SeqMeta, page_table, d: LatentDims, seq_lens=None, max_k=0,
