@@ -467,6 +467,38 @@ def test_state_space_mixer_alone(form, dims):
     settled(dev)
 
 
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16], ids=["f32", "bf16"])
+@pytest.mark.parametrize("dims", [(8, 64, 128, 2, 2, 4), (4, 32, 64, 4, 4, 1), (6, 128, 40, 3, 2, 3), (16, 24, 256, 2, 1, 5),
+                                  (8, 8, 33, 1, 1, 16), (4, 256, 64, 1, 8, 2)], ids=str)
+def test_one_launch_decode_step_equals_the_separate_kernels(dims, dtype):
+    """Tokens of several sequences at different positions, one of them fresh, one row padding: norm parts
+    of one head, of a cluster of heads, of more heads than a cluster holds, and of half a head."""
+    g, dev, eps, B = gen(sum(dims)), "cuda", 1e-4, 5
+    d, _, w = mixer_case(g, (dev, dtype), dims, 1)
+    assert SS.step_fits(d, d.inner)
+    oc = d.inner
+    odt = oc + (d.channels + 7) // 8 * 8
+    wd = {n: t.to(dev) for n, t in w.items()}
+    wd.update(offs=(0, oc, odt), o=torch.empty(8, d.inner, device=dev))
+    slots, starts = [2, 5, -1, 0, 3], [0, 7, 0, 1, 300]
+    ring = rnd(g, 6, d.taps, d.channels).to(dev, dtype) if d.taps > 1 else None
+    state = rnd(g, 6, d.heads, d.state, d.vdim).to(dev)
+    rings, states = [ring, ring.clone() if ring is not None else None], [state, state.clone()]
+    for step in range(3):
+        m = seq_meta([1] * B, [s + step for s in starts], slots, dev)
+        x = rnd(g, B, odt + (d.heads + 7) // 8 * 8).to(dev, dtype)
+        got = SS.mixer(x, wd, rings[0], states[0], m, d, eps)
+        u = SS.short_conv(x, oc, wd["conv"], wd["conv_b"], rings[1], m)
+        y = SS.state_space_scan(u, x, odt, wd, states[1], m, d)
+        want = SS.group_norm_gate(y, x[:, :d.inner], wd["norm"], d.norm_groups, eps, d.inner)
+        close(got[[0, 1, 3, 4]], want[[0, 1, 3, 4]], dtype, f"step {step}")
+        assert float(got[2].float().abs().max()) == 0.0
+    close(states[0].flatten(1), states[1].flatten(1), torch.float32, "states")
+    assert ring is None or torch.equal(*rings)
+    settled(dev)
+
+
 @pytest.mark.parametrize("form", FORMS)
 @pytest.mark.parametrize("dims", [MIXES[0], MIXES[3], MIXES[4], MIXES[6], MIXES[8]], ids=str)
 def test_recurrence_alone_is_exact_in_32_bit(form, dims):

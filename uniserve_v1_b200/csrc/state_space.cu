@@ -6,10 +6,12 @@
 //   us_short_conv          causal convolution + bias + silu of x | B | C, inputs kept in a ring
 //   us_state_space_scan    dt = softplus(raw + bias), the recurrence and its read-out
 //   us_group_norm_gate     y * silu(z), RMS norm over equal parts of the row, weight
+//   us_state_space_step    all of these for one token of every sequence in one launch
 //
 // A sequence whose first packed row stands at position 0 starts from a zero state whatever its
 // slot holds; a negative slot marks padding.
 #include "include/us_common.cuh"
+#include "include/us_tc05.cuh"
 
 namespace {
 
@@ -306,6 +308,154 @@ group_norm_gate_kernel(const void* __restrict__ y, long long ldy, const void* __
       st_any(out, (long long)blockIdx.x * ldo + c, bf16, 0.f);
 }
 
+// ------------------------------------------------------------- decode step --
+struct StepArgs {
+  const void* x;                // projection rows: z | x B C | dt at the three offsets
+  long long ldx;
+  int oz, oc, odt;
+  const float *taps, *bias;     // [C, K], [C]
+  void* ring;                   // [slots, K, C]
+  const float *dt_bias, *A_log, *D, *w;   // [H] x 3, [H * V]
+  float* state;                 // [slots, H, N, V]
+  void* out;                    // [B, ldo]
+  long long ldo;
+  const int *slots, *pos;
+  int H, V, N, G, K, bf16, heads;         // heads: of a norm part (the cluster), 0: no gate and norm
+  float eps;
+};
+
+constexpr int kStepThreads = 256;
+
+// One CTA per (head, sequence).  A thread keeps up to R rows of four state columns (VQ threads
+// span the columns); their loads are issued first, the convolution, the step size and the decay are
+// formed meanwhile.  B and C of a group are convolved by each of its heads and kept by the
+// first one (the entry that a token writes is none of those it reads).  The heads of a norm part are
+// one cluster that adds up their sums of squares.
+template <int VQ, int R>
+__global__ void __launch_bounds__(kStepThreads, R <= 8 ? 3 : 2) state_space_step_kernel(const StepArgs a) {
+  US_PDL_PROLOGUE();
+  constexpr int GR = kStepThreads / VQ;           // row groups
+  extern __shared__ __align__(16) float sm[];
+  float* u = sm;                                  // [V | N | N] convolved inputs
+  float* red = u + ((a.V + 2 * a.N + 3) & ~3);    // [GR][VQ * 4]
+  __shared__ float part[33], steps[2], total;
+  const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x;
+  const int g = h / (a.H / a.G), inner = a.H * a.V, C = inner + 2 * a.G * a.N;
+  const int slot = a.slots[b], p = a.pos[b];
+  const bool live = slot >= 0;
+  const int q = tid % VQ, gr = tid / VQ, v0 = q * 4;
+  float* Sg = a.state + ((long long)max(slot, 0) * a.H + h) * a.N * a.V;
+  float4 S[R];
+#pragma unroll
+  for (int j = 0; j < R; ++j) {
+    const int row = gr + j * GR;
+    S[j] = (live && p > 0 && row < a.N && v0 < a.V)
+               ? __ldcs(reinterpret_cast<const float4*>(Sg + (long long)row * a.V + v0))
+               : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  const bool mine = tid < a.V;                    // thread v < V finishes column v
+  const float z = live && mine && a.heads > 0
+                      ? ld_any(a.x, (long long)b * a.ldx + a.oz + (long long)h * a.V + tid, a.bf16) : 0.f;
+  if (live) {
+    const bool keeps = h % (a.H / a.G) == 0;      // this head writes its group's B and C inputs
+    for (int e = tid; e < a.V + 2 * a.N; e += kStepThreads) {
+      const int c = e < a.V ? h * a.V + e
+                            : inner + (e < a.V + a.N ? g * a.N + e - a.V : (a.G + g) * a.N + e - a.V - a.N);
+      const float now = ld_any(a.x, (long long)b * a.ldx + a.oc + c, a.bf16);
+      const float* w = a.taps + (long long)c * a.K;
+      float acc = fmaf(w[a.K - 1], now, a.bias[c]);
+      for (int k = 1; k < min(a.K, p + 1); ++k)
+        acc = fmaf(w[a.K - 1 - k], ld_any(a.ring, ((long long)slot * a.K + (p - k) % a.K) * C + c, a.bf16), acc);
+      if (a.K > 1 && (e < a.V || keeps))
+        st_any(a.ring, ((long long)slot * a.K + p % a.K) * C + c, a.bf16, now);
+      acc = silu_f(acc);
+      u[e] = a.bf16 ? us::bf2f(us::f2bf(acc)) : acc;
+    }
+    if (tid == kStepThreads - 1) {
+      const float dt = softplus_f(ld_any(a.x, (long long)b * a.ldx + a.odt + h, a.bf16) + a.dt_bias[h]);
+      steps[0] = dt;
+      steps[1] = decay_exp(-expf(a.A_log[h]) * dt);
+    }
+  }
+  __syncthreads();
+  float y = 0.f;
+  if (live) {
+    const float dt = steps[0], dec = steps[1];
+    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (v0 < a.V) {
+      const float4 x4 = make_float4(u[v0] * dt, u[v0 + 1] * dt, u[v0 + 2] * dt, u[v0 + 3] * dt);
+#pragma unroll
+      for (int j = 0; j < R; ++j) {
+        const int row = gr + j * GR;
+        if (row >= a.N) continue;
+        const float B = u[a.V + row], Cn = u[a.V + a.N + row];
+        S[j].x = fmaf(S[j].x, dec, B * x4.x);
+        S[j].y = fmaf(S[j].y, dec, B * x4.y);
+        S[j].z = fmaf(S[j].z, dec, B * x4.z);
+        S[j].w = fmaf(S[j].w, dec, B * x4.w);
+        __stcs(reinterpret_cast<float4*>(Sg + (long long)row * a.V + v0), S[j]);
+        o.x = fmaf(S[j].x, Cn, o.x);
+        o.y = fmaf(S[j].y, Cn, o.y);
+        o.z = fmaf(S[j].z, Cn, o.z);
+        o.w = fmaf(S[j].w, Cn, o.w);
+      }
+    }
+    *reinterpret_cast<float4*>(red + (gr * VQ + q) * 4) = o;
+  }
+  __syncthreads();
+  if (live && mine) {
+    for (int r = 0; r < GR; ++r) y += red[r * VQ * 4 + tid];
+    y = fmaf(a.D[h], u[tid], y);
+    if (a.bf16) y = us::bf2f(us::f2bf(y));
+  }
+  const long long at = (long long)b * a.ldo + (long long)h * a.V + tid;
+  if (a.heads == 0) {
+    if (mine) st_any(a.out, at, a.bf16, y);
+    return;
+  }
+  y *= silu_f(z);
+  float ss = us::block_sum(y * y, part);
+  if (a.heads > 1) {
+    if (tid == 0) total = ss;
+    tc::cluster_sync();
+    const uint32_t addr = (uint32_t)__cvta_generic_to_shared(&total);
+    ss = 0.f;
+    for (int r = 0; r < a.heads; ++r) ss += tc::ld_dsmem_f32(tc::map_to_cta(addr, r));
+  }
+  if (mine)
+    st_any(a.out, at, a.bf16,
+           live ? y * (1.f / sqrtf(ss / (float)(max(a.heads, 1) * a.V) + a.eps)) * a.w[h * a.V + tid] : 0.f);
+  if (a.heads > 1) tc::cluster_sync();            // nobody leaves while its sum may still be read
+}
+
+template <int VQ, int R>
+int launch_step_rows(const StepArgs& a, int B, cudaStream_t stream) {
+  const size_t smem = (((a.V + 2 * a.N + 3) & ~3) + kStepThreads * 4) * sizeof(float);
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3(a.H, B);
+  cfg.blockDim = dim3(kStepThreads);
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = stream;
+  cudaLaunchAttribute attr[2];
+  attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[0].val.programmaticStreamSerializationAllowed = us::pdl_enabled() ? 1 : 0;
+  attr[1].id = cudaLaunchAttributeClusterDimension;
+  attr[1].val.clusterDim.x = a.heads;
+  attr[1].val.clusterDim.y = 1;
+  attr[1].val.clusterDim.z = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = a.heads > 1 ? 2 : 1;
+  US_CUDA_CHECK(cudaLaunchKernelEx(&cfg, state_space_step_kernel<VQ, R>, a));
+  return US_OK;
+}
+
+template <int VQ>
+int launch_step(const StepArgs& a, int B, cudaStream_t stream) {
+  const int rows = us::ceil_div(a.N, kStepThreads / VQ);
+  return rows <= 4 ? launch_step_rows<VQ, 4>(a, B, stream)
+                   : rows <= 8 ? launch_step_rows<VQ, 8>(a, B, stream) : launch_step_rows<VQ, 16>(a, B, stream);
+}
+
 bool aligned(const void* p, int bytes) { return ((uintptr_t)p % bytes) == 0; }
 
 }  // namespace
@@ -389,4 +539,29 @@ US_API int us_group_norm_gate(const void* y, long long ldy, const void* z, long 
   }
 #undef US_GN
   return US_OK;
+}
+
+// One token of every sequence: convolution, recurrence, read-out and, with heads >= 1 (the heads of a
+// norm part, at most 8, dividing H), gate and norm.  V a multiple of 4, V <= 256, N <= 16 row groups.
+US_API int us_state_space_step(const void* x, long long ldx, int oz, int oc, int odt,
+                               const float* taps, const float* bias, void* ring,
+                               const float* dt_bias, const float* A_log, const float* D,
+                               const float* w, float* state, void* out, long long ldo,
+                               const int* slots, const int* pos, int B, int H, int V, int N, int G,
+                               int K, int bf16, int heads, float eps, void* stream_) {
+  US_REQUIRE(x && taps && bias && dt_bias && A_log && D && state && out && slots && pos);
+  US_REQUIRE(B >= 0 && H >= 1 && V >= 4 && N >= 1 && G >= 1 && H % G == 0 && K >= 1 && (K == 1 || ring) &&
+             (V % 4) == 0 && heads >= 0 && heads <= 8 && (heads == 0 || (H % heads == 0 && w)) && B <= 65535);
+  const int vq = V <= 32 ? 8 : V <= 64 ? 16 : V <= 128 ? 32 : 64;
+  if (V > 256 || us::ceil_div(N, kStepThreads / vq) > 16) return US_ERR_LIMIT;
+  if (B == 0) return US_OK;
+  StepArgs a{x, ldx, oz, oc, odt, taps, bias, ring, dt_bias, A_log, D, w, state, out, ldo, slots, pos,
+             H, V, N, G, K, bf16, heads, eps};
+  cudaStream_t stream = (cudaStream_t)stream_;
+  switch (vq) {
+    case 8: return launch_step<8>(a, B, stream);
+    case 16: return launch_step<16>(a, B, stream);
+    case 32: return launch_step<32>(a, B, stream);
+    default: return launch_step<64>(a, B, stream);
+  }
 }

@@ -22,6 +22,8 @@ N.register_signatures({
     "us_short_conv": (I, [P, L, I, P, P, P, P, L, P, P, P, I, I, I, I, I, I, P]),
     "us_state_space_scan": (I, [P, L, P, L, I, P, P, P, P, P, L, P, P, P, I, I, I, I, I, I, I, P]),
     "us_state_space_chunks": (I, [P, L, P, L, I, P, P, P, P, P, L, P, P, P, I, I, I, I, I, I, P]),
+    "us_state_space_step": (I, [P, L, I, I, I, P, P, P, P, P, P, P, P, P, L, P, P, I, I, I, I, I, I, I, I, F,
+                                P]),
     "us_group_norm_gate": (I, [P, L, P, L, I, P, P, L, I, I, I, F, I, P]),
 })
 
@@ -128,10 +130,29 @@ def group_norm_gate(y, z, w, groups, eps, ldo):
     return out
 
 
+def step_fits(d: StateSpaceDims, ldo: int) -> bool:
+    """Whether the one-launch decode step serves these sizes (else: the separate kernels)."""
+    threads = 8 if d.vdim <= 32 else 16 if d.vdim <= 64 else 32 if d.vdim <= 128 else 64
+    return d.vdim % 4 == 0 and d.vdim <= 256 and -(-d.state // (256 // threads)) <= 16 and ldo == d.inner
+
+
 def mixer(x, w, ring, state, m: SeqMeta, d: StateSpaceDims, eps):
     """Everything between the input projection's rows and the output projection's: ``x`` holds
     z | x B C | dt at the columns ``w['offs']``."""
     oz, oc, odt = w["offs"]
+    ldo = w["o"].shape[1]
+    if x.is_cuda and m.one_token and step_fits(d, ldo):
+        # gate and norm in the same launch where a norm part is one head, or where it is one cluster
+        # and the launch leaves SMs empty anyway (a cluster waits for its slowest head)
+        heads = d.heads // d.norm_groups if d.heads % d.norm_groups == 0 else 0
+        if heads > 8 or (heads > 1 and x.shape[0] * d.heads > 296):
+            heads = 0
+        y = torch.empty(x.shape[0], ldo, dtype=x.dtype, device=x.device)
+        N.call("us_state_space_step", N.ptr(x), x.stride(0), oz, oc, odt, N.ptr(w["conv"]), N.ptr(w["conv_b"]),
+               N.ptr(ring), N.ptr(w["dt_bias"]), N.ptr(w["A_log"]), N.ptr(w["D"]), N.ptr(w["norm"]),
+               N.ptr(state), N.ptr(y), ldo, N.ptr(m.slots), N.ptr(m.positions), x.shape[0], d.heads, d.vdim,
+               d.state, d.groups, d.taps, int(x.dtype == BF16), heads, eps, N.stream())
+        return y if heads else group_norm_gate(y, x[:, oz:oz + d.inner], w["norm"], d.norm_groups, eps, ldo)
     u = short_conv(x, oc, w["conv"], w["conv_b"], ring, m)
     y = state_space_scan(u, x, odt, w, state, m, d)
-    return group_norm_gate(y, x[:, oz:oz + d.inner], w["norm"], d.norm_groups, eps, w["o"].shape[1])
+    return group_norm_gate(y, x[:, oz:oz + d.inner], w["norm"], d.norm_groups, eps, ldo)
