@@ -35,6 +35,8 @@ struct DecodeArgs {
   long long ldq, ldo;
   int B, Hq, Hkv, max_pages, page_size, splits, window;
   float scale;
+  const float* sink;       // [Hq] or null: exp(sink) joins the softmax denominator
+  float out_scale;         // of the finished output
 };
 
 __device__ __forceinline__ void cp_async16(void* dst, const void* src) {
@@ -182,10 +184,12 @@ __global__ void __launch_bounds__(kThreads) paged_decode_kernel(const DecodeArgs
   for (int i = 0; i < kHpt; ++i) {
     const int g = grp + i * kGroups;
     if (g < G) {
-      const float l = Lsum[g];
-      const float inv = l > 0.f ? 1.f / l : 0.f;
       const int h = hk * G + g;
+      const float l = Lsum[g];
+      float inv = l > 0.f ? 1.f / l : 0.f;
       if (a.splits == 1) {
+        if (a.sink && l > 0.f) inv = 1.f / (l + __expf(a.sink[h] - Mmax[g]));
+        inv *= a.out_scale;
         __nv_bfloat162 o = __floats2bfloat162_rn(acc[i][0] * inv, acc[i][1] * inv);
         *reinterpret_cast<__nv_bfloat162*>(a.out + (long long)b * a.ldo + (long long)h * D +
                                            pair * 2) = o;
@@ -203,7 +207,8 @@ template <int D>
 __global__ void __launch_bounds__(D) merge_splits_kernel(const float* __restrict__ part_o,
                                                          const float* __restrict__ part_lse,
                                                          __nv_bfloat16* __restrict__ out,
-                                                         long long ldo, int Hq, int splits) {
+                                                         long long ldo, int Hq, int splits,
+                                                         const float* __restrict__ sink, float out_scale) {
   US_PDL_PROLOGUE();
   const int b = blockIdx.x, h = blockIdx.y, d = threadIdx.x;
   const long long base = ((long long)b * Hq + h) * splits;
@@ -216,8 +221,9 @@ __global__ void __launch_bounds__(D) merge_splits_kernel(const float* __restrict
       num += w * part_o[(base + s) * D + d];
       den += w;
     }
+    if (sink) den += __expf(sink[h] - m);
   }
-  out[(long long)b * ldo + (long long)h * D + d] = us::f2bf(den > 0.f ? num / den : 0.f);
+  out[(long long)b * ldo + (long long)h * D + d] = us::f2bf(den > 0.f ? out_scale * num / den : 0.f);
 }
 
 template <int D, int G>
@@ -228,7 +234,7 @@ int launch_decode(const DecodeArgs& a, cudaStream_t stream) {
   if (a.splits > 1) {
     dim3 g2(a.B, a.Hq);
     us::launch_pdl(merge_splits_kernel<D>, dim3(g2), dim3(D), 0, stream, a.part_o, a.part_lse, a.out, a.ldo, a.Hq,
-                                                 a.splits);
+                                                 a.splits, a.sink, a.out_scale);
     US_LAUNCH_CHECK();
   }
   return US_OK;
@@ -238,12 +244,12 @@ int launch_decode(const DecodeArgs& a, cudaStream_t stream) {
 
 extern "C" int us_merge_decode_splits(const float* part_o, const float* part_lse, void* out,
                                       long long ldo, int B, int Hq, int D, int splits,
-                                      void* stream) {
+                                      const float* sink, float out_scale, void* stream) {
   dim3 g2(B, Hq);
   if (D == 128)
-    us::launch_pdl(merge_splits_kernel<128>, dim3(g2), dim3(128), 0, (cudaStream_t)stream, part_o, part_lse, (__nv_bfloat16*)out, ldo, Hq, splits);
+    us::launch_pdl(merge_splits_kernel<128>, dim3(g2), dim3(128), 0, (cudaStream_t)stream, part_o, part_lse, (__nv_bfloat16*)out, ldo, Hq, splits, sink, out_scale);
   else if (D == 64)
-    us::launch_pdl(merge_splits_kernel<64>, dim3(g2), dim3(64), 0, (cudaStream_t)stream, part_o, part_lse, (__nv_bfloat16*)out, ldo, Hq, splits);
+    us::launch_pdl(merge_splits_kernel<64>, dim3(g2), dim3(64), 0, (cudaStream_t)stream, part_o, part_lse, (__nv_bfloat16*)out, ldo, Hq, splits, sink, out_scale);
   else
     return US_ERR_UNSUPPORTED;
   US_LAUNCH_CHECK();
@@ -255,11 +261,12 @@ US_API long long us_paged_decode_scratch_bytes(int B, int Hq, int D, int splits)
   return (long long)B * Hq * splits * (D + 1) * (long long)sizeof(float);
 }
 
-US_API int us_paged_decode_attention(const void* q, const void* kcache, const void* vcache,
-                                     const int* page_table, const int* seq_lens, void* out,
-                                     void* scratch, int B, int Hq, int Hkv, int D, int max_pages,
-                                     int page_size, int splits, int window, float scale,
-                                     long long ldq, long long ldo, void* stream_) {
+// sink [Hq] FP32 or null: a logit per head without key or value; out_scale multiplies the output.
+extern "C" int us_paged_decode_simt(const void* q, const void* kcache, const void* vcache,
+                                    const int* page_table, const int* seq_lens, void* out,
+                                    void* scratch, int B, int Hq, int Hkv, int D, int max_pages,
+                                    int page_size, int splits, int window, float scale, long long ldq,
+                                    long long ldo, const float* sink, float out_scale, void* stream_) {
   US_REQUIRE(q && kcache && vcache && page_table && seq_lens && out);
   US_REQUIRE(B >= 0 && Hkv >= 1 && Hq % Hkv == 0 && splits >= 1 && page_size >= 1);
   US_REQUIRE(splits == 1 || scratch != nullptr);
@@ -276,6 +283,7 @@ US_API int us_paged_decode_attention(const void* q, const void* kcache, const vo
   a.ldq = ldq; a.ldo = ldo;
   a.B = B; a.Hq = Hq; a.Hkv = Hkv; a.max_pages = max_pages; a.page_size = page_size;
   a.splits = splits; a.window = window; a.scale = scale;
+  a.sink = sink; a.out_scale = out_scale;
   cudaStream_t stream = (cudaStream_t)stream_;
   const int G = Hq / Hkv;
 #define US_DEC(DD, GG) \
@@ -284,6 +292,15 @@ US_API int us_paged_decode_attention(const void* q, const void* kcache, const vo
   US_DEC(64, 1) US_DEC(64, 2) US_DEC(64, 4) US_DEC(64, 8)
 #undef US_DEC
   return US_ERR_UNSUPPORTED;
+}
+
+US_API int us_paged_decode_attention(const void* q, const void* kcache, const void* vcache,
+                                     const int* page_table, const int* seq_lens, void* out,
+                                     void* scratch, int B, int Hq, int Hkv, int D, int max_pages,
+                                     int page_size, int splits, int window, float scale,
+                                     long long ldq, long long ldo, void* stream_) {
+  return us_paged_decode_simt(q, kcache, vcache, page_table, seq_lens, out, scratch, B, Hq, Hkv, D,
+                              max_pages, page_size, splits, window, scale, ldq, ldo, nullptr, 1.f, stream_);
 }
 
 // ---------------------------------------------------------------------------

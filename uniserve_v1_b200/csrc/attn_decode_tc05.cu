@@ -57,6 +57,8 @@ struct DecTcArgs {
   int B, Hq, Hkv, max_pages, page_size, splits, window;
   float scale_log2;
   unsigned int* status;
+  const float* sink;      // [Hq] or null: exp(sink) joins the softmax denominator
+  float out_scale;        // of the finished output
   const float* k_scale;   // FP8 pages: one scale per page and plane
   const float* v_scale;
 };
@@ -141,9 +143,11 @@ __device__ __forceinline__ void merge_if_last(const DecTcArgs& a, int b, int hk)
     }
   }
 #pragma unroll
-  for (int g = 0; g < G; ++g)
+  for (int g = 0; g < G; ++g) {
+    if (a.sink && den[g] > 0.f) den[g] += __expf(a.sink[hk * G + g] - m[g]);
     a.out[(long long)b * a.ldo + (long long)(hk * G + g) * kD + tid] =
-        us::f2bf(den[g] > 0.f ? acc[g] / den[g] : 0.f);
+        us::f2bf(den[g] > 0.f ? a.out_scale * acc[g] / den[g] : 0.f);
+  }
 }
 
 template <int G, bool FP8>
@@ -519,9 +523,11 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK,
 #pragma unroll
         for (int g = 0; g < G; ++g) {
           const float l = rbuf[g] + rbuf[kNPad + g] + rbuf[2 * kNPad + g] + rbuf[3 * kNPad + g];
-          const float inv = l > 0.f ? 1.f / l : 0.f;
           const int h = hk * G + g;
+          float inv = l > 0.f ? 1.f / l : 0.f;
           if (a.splits == 1) {
+            if (a.sink && l > 0.f) inv = 1.f / (l + ex2(a.sink[h] * 1.4426950408889634f - m_run[g]));
+            inv *= a.out_scale;
             a.out[(long long)b * a.ldo + (long long)h * kD + tid] = us::f2bf(o_acc[g] * inv);
           } else {
             const long long base = ((long long)b * a.Hq + h) * a.splits + split;
@@ -568,13 +574,18 @@ int launch_tc(const CUtensorMap& tmK, const CUtensorMap& tmV, const DecTcArgs& a
 
 extern "C" int us_merge_decode_splits(const float* part_o, const float* part_lse, void* out,
                                       long long ldo, int B, int Hq, int D, int splits,
-                                      void* stream);
+                                      const float* sink, float out_scale, void* stream);
+extern "C" int us_paged_decode_simt(const void* q, const void* kcache, const void* vcache,
+                                    const int* page_table, const int* seq_lens, void* out, void* scratch,
+                                    int B, int Hq, int Hkv, int D, int max_pages, int page_size,
+                                    int splits, int window, float scale, long long ldq, long long ldo,
+                                    const float* sink, float out_scale, void* stream);
 
 static int decode_tc(const void* q, const void* kcache, const void* vcache,
                      const float* k_scale, const float* v_scale, const int* page_table, const int* seq_lens, void* out, void* scratch,
                      int* counters, int B, int Hq, int Hkv, int D, int num_pages, int max_pages,
                      int page_size, int splits, int window, float scale, long long ldq,
-                     long long ldo, void* stream_) {
+                     long long ldo, const float* sink, float out_scale, void* stream_) {
   US_REQUIRE(q && kcache && vcache && page_table && seq_lens && out);
   US_REQUIRE(D == kD && Hkv >= 1 && Hq % Hkv == 0 && Hq / Hkv <= kNPad && splits >= 1);
   US_REQUIRE(page_size >= 8 && page_size <= 128 && (kTileKeys % page_size) == 0);
@@ -606,6 +617,8 @@ static int decode_tc(const void* q, const void* kcache, const void* vcache,
   a.splits = splits; a.window = window;
   a.scale_log2 = scale * 1.4426950408889634f;
   a.status = us_status_ptr();
+  a.sink = sink;
+  a.out_scale = out_scale;
   a.k_scale = k_scale;
   a.v_scale = v_scale;
   const int G = Hq / Hkv;
@@ -630,7 +643,7 @@ static int decode_tc(const void* q, const void* kcache, const void* vcache,
   }
   if (rc) return rc;
   if (splits > 1 && !counters)
-    return us_merge_decode_splits(a.part_o, a.part_lse, out, ldo, B, Hq, D, splits, stream_);
+    return us_merge_decode_splits(a.part_o, a.part_lse, out, ldo, B, Hq, D, splits, sink, out_scale, stream_);
   return US_OK;
 }
 
@@ -644,7 +657,7 @@ US_API int us_paged_decode_attention_tc(const void* q, const void* kcache, const
                                         void* stream_) {
   return decode_tc(q, kcache, vcache, nullptr, nullptr, page_table, seq_lens, out, scratch, nullptr,
                    B, Hq, Hkv, D, num_pages, max_pages, page_size, splits, window, scale, ldq, ldo,
-                   stream_);
+                   nullptr, 1.f, stream_);
 }
 
 // One launch: `counters` [B * Hkv] int32 must be zero before the first call and is left zero
@@ -660,7 +673,26 @@ US_API int us_paged_decode_attention_tc_merged(const void* q, const void* kcache
   US_REQUIRE((splits == 1 || counters != nullptr) && splits <= 32);
   return decode_tc(q, kcache, vcache, nullptr, nullptr, page_table, seq_lens, out, scratch,
                    counters, B, Hq, Hkv, D, num_pages, max_pages, page_size, splits, window, scale,
-                   ldq, ldo, stream_);
+                   ldq, ldo, nullptr, 1.f, stream_);
+}
+
+// Either kernel with a sink (a logit per head [Hq], FP32, without key or value; null: none) and a
+// factor on the output.  `counters` as above, or null: splits are merged by a second launch.
+US_API int us_paged_decode_attention_sink(const void* q, const void* kcache, const void* vcache,
+                                          const int* page_table, const int* seq_lens, void* out,
+                                          void* scratch, int* counters, int B, int Hq, int Hkv, int D,
+                                          int num_pages, int max_pages, int page_size, int splits,
+                                          int window, float scale, long long ldq, long long ldo,
+                                          const float* sink, float out_scale, void* stream_) {
+  US_REQUIRE(splits >= 1 && splits <= 32 && page_size >= 1);
+  if (D == kD && page_size >= 8 && page_size <= 128 && (kTileKeys % page_size) == 0 && Hkv >= 1 &&
+      Hq / Hkv <= kNPad)
+    return decode_tc(q, kcache, vcache, nullptr, nullptr, page_table, seq_lens, out, scratch, counters,
+                     B, Hq, Hkv, D, num_pages, max_pages, page_size, splits, window, scale, ldq, ldo,
+                     sink, out_scale, stream_);
+  return us_paged_decode_simt(q, kcache, vcache, page_table, seq_lens, out, scratch, B, Hq, Hkv, D,
+                              max_pages, page_size, splits, window, scale, ldq, ldo, sink, out_scale,
+                              stream_);
 }
 
 // E4M3 pages with one FP32 scale per page and plane (k_scale, v_scale [num_pages]); the
@@ -676,5 +708,5 @@ US_API int us_paged_decode_attention_fp8(const void* q, const void* kcache, cons
   US_REQUIRE(k_scale && v_scale && splits <= 32);
   return decode_tc(q, kcache, vcache, k_scale, v_scale, page_table, seq_lens, out, scratch,
                    counters, B, Hq, Hkv, D, num_pages, max_pages, page_size, splits, window, scale,
-                   ldq, ldo, stream_);
+                   ldq, ldo, nullptr, 1.f, stream_);
 }

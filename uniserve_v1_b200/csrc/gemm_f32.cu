@@ -75,7 +75,30 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const F32Args a) {
   }
 }
 
+// z [rows, 2 I]: first | second -> (clamp(first) + 1) g sigmoid(alpha g), g = min(second, limit)
+__global__ void __launch_bounds__(256)
+clamped_glu_kernel(const float* __restrict__ z, float* __restrict__ out, long long total, int I,
+                   float limit, float alpha) {
+  US_PDL_PROLOGUE();
+  const long long e = (long long)blockIdx.x * 256 + threadIdx.x;
+  if (e >= total) return;
+  const long long r = e / I;
+  const float* row = z + r * 2 * I + (e - r * I);
+  const float g = fminf(row[I], limit), u = fminf(fmaxf(row[0], -limit), limit);
+  out[e] = (u + 1.f) * (g / (1.f + expf(-alpha * g)));
+}
+
 }  // namespace
+
+US_API int us_clamped_glu_f32(const float* z, float* out, int rows, int I, float limit, float alpha,
+                              void* stream_) {
+  US_REQUIRE(z && out && rows >= 0 && I >= 1);
+  const long long total = (long long)rows * I;
+  if (total == 0) return US_OK;
+  US_CUDA_CHECK(us::launch_pdl(clamped_glu_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0,
+                               (cudaStream_t)stream_, z, out, total, I, limit, alpha));
+  return US_OK;
+}
 
 // Same operand conventions as us_gemm_wx; act: 0 none, 3 gelu (erf).
 US_API int us_gemm_f32(const float* W, const float* X, float* out, int G, int w_rows, int M, int K,

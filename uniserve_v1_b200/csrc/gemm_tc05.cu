@@ -775,6 +775,8 @@ gemm_wx_pair_kernel(const __grid_constant__ CUtensorMap tmA,
               } else if (act == 1) {
                 const float sg = us::bf2f(us::f2bf(silu_f(us::bf2f(us::f2bf(gate)))));
                 val = us::bf2f(us::f2bf(val)) * sg;
+              } else if (act == 4) {
+                val = clamped_glu_f(val, gate, args.glu_limit, args.glu_alpha);
               } else {
                 val = val * gelu_tanh_f(gate);
               }
@@ -1100,6 +1102,7 @@ struct PeerSpec {
   int rows_per_peer = 0;                 // gather: rows of the activation per rank
   int peer_rows = 0;                     // reduce-scatter: rows owned per rank
   int peer_slot = 0;
+  float glu_limit = 0.f, glu_alpha = 0.f;  // dual products with act 4
 };
 
 int gemm_impl(const void* W, const void* X, void* out, int G, int w_rows, int M, int K, int x_rows,
@@ -1217,6 +1220,8 @@ int gemm_impl(const void* W, const void* X, void* out, int G, int w_rows, int M,
   a.route_w = nullptr;
   a.route_per = 0;
   a.scale_first = 0;
+  a.glu_limit = ps.glu_limit;
+  a.glu_alpha = ps.glu_alpha;
   if (ps.route_map) {
     US_REQUIRE(ps.out_peers && ps.route_w && ps.route_per > 0 && ps.n_out_peers >= 1 &&
                ps.n_out_peers <= 8 && out_dtype == 0);
@@ -1330,6 +1335,21 @@ US_API int us_gemm_wx(const void* W, const void* X, void* out, int G, int w_rows
   return gemm_impl(W, X, out, G, w_rows, M, K, x_rows, ldw, ldx, ldo, dual, dual_offset, act,
                    out_dtype, bias, bias_dtype, row_scale, out_row_map, tile_group, tile_row0,
                    tile_rows, num_tiles, max_tiles, block_n, ps, (cudaStream_t)stream_);
+}
+
+// Gated product out = (clamp(first) + 1) g sigmoid(alpha g), g = min(second, limit), first clamped to
+// +-limit; dense, or grouped over a tile list.  bf16 out.
+US_API int us_gemm_wx_clamped(const void* W, const void* X, void* out, int G, int w_rows, int M, int K,
+                              int x_rows, long long ldw, long long ldx, long long ldo, int dual_offset,
+                              float limit, float alpha, const int* tile_group, const int* tile_row0,
+                              const int* tile_rows, const int* num_tiles, int max_tiles, int block_n,
+                              void* stream_) {
+  PeerSpec ps;
+  ps.glu_limit = limit;
+  ps.glu_alpha = alpha;
+  return gemm_impl(W, X, out, G, w_rows, M, K, x_rows, ldw, ldx, ldo, 1, dual_offset, 4, 0, nullptr, 0,
+                   nullptr, nullptr, tile_group, tile_row0, tile_rows, num_tiles, max_tiles, block_n, ps,
+                   (cudaStream_t)stream_);
 }
 
 // Dense GEMM whose output tiles are scattered into the peers' buffers from the

@@ -14,7 +14,8 @@ struct GemmArgs {
   int dual_offset;  // row offset of the second weight tile (dual epilogue)
   int stages;
   int early;        // dense: weight tiles of the first stages are fetched before the PDL wait
-  int act;          // dual: 0 = silu fused rounding, 1 = silu stepwise rounding, 2 = gelu-tanh
+  int act;          // dual: 0 = silu fused rounding, 1 = silu stepwise rounding, 2 = gelu-tanh,
+                    //       4 = clamped (glu_limit, glu_alpha)
                     // single: 0 = none, 3 = gelu (erf) of the biased value
   int out_dtype;    // 0 = bf16, 1 = fp32
   int bias_dtype;   // 0 = bf16, 1 = fp32
@@ -69,6 +70,7 @@ struct GemmArgs {
   // 1: the swapped epilogue writes rows bound for another GPU as whole 128-byte lines
   // (collected per warp in the staging area) instead of 32-byte pieces per thread.
   int remote_lines;
+  float glu_limit, glu_alpha;
 };
 
 struct BMaps {
@@ -83,6 +85,13 @@ __device__ __forceinline__ float silu_f(float x) { return x / (1.f + __expf(-x))
 __device__ __forceinline__ float gelu_tanh_f(float x) {
   const float k0 = 0.7978845608028654f, k1 = 0.044715f;
   return 0.5f * x * (1.f + tanhf(k0 * (x + k1 * x * x * x)));
+}
+
+// (clamp(u) + 1) g sigmoid(alpha g) with g cut off above `limit`, u on both sides
+__device__ __forceinline__ float clamped_glu_f(float u, float g, float limit, float alpha) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return (u + 1.f) * (g / (1.f + __expf(-alpha * g)));
 }
 
 __device__ __forceinline__ float gelu_erf_f(float x) {
@@ -115,6 +124,7 @@ struct Epilogue {
   // branches per value - 3,300 clocks per 16-row chunk, more than the mainloop.
   const int m0, ml, m, row0;
   const bool m_ok;
+  const float glu_limit, glu_alpha;
   float bias;
   char* tile_base;     // element (row0, m0) of the destination; null = per-row lookup
   long long row_bytes;
@@ -129,7 +139,8 @@ struct Epilogue {
   char* out;
   const GemmArgs& a;         // rare paths only (the peer table of the route push)
   __device__ __forceinline__ Epilogue(const GemmArgs& args, int group, int m0_, int ml_, int row0_)
-      : m0(m0_), ml(ml_), m(m0_ + ml_), row0(row0_), m_ok(m0_ + ml_ < args.M), bias(0.f),
+      : m0(m0_), ml(ml_), m(m0_ + ml_), row0(row0_), m_ok(m0_ + ml_ < args.M),
+        glu_limit(args.glu_limit), glu_alpha(args.glu_alpha), bias(0.f),
         tile_base(nullptr), row_bytes(0), esz(args.out_dtype == 0 ? 2 : 4), M(args.M),
         act(args.act), route_per(args.route_per), vec_store(args.vec_store), ldo(args.ldo),
         scale_rows(args.row_scale ? args.row_scale + row0_ : nullptr),
@@ -170,6 +181,8 @@ struct Epilogue {
       } else if (act == 1) {
         const float sg = us::bf2f(us::f2bf(silu_f(us::bf2f(us::f2bf(gate)))));
         val = us::bf2f(us::f2bf(val)) * sg;
+      } else if (act == 4) {
+        val = clamped_glu_f(val, gate, glu_limit, glu_alpha);
       } else {
         val = val * gelu_tanh_f(gate);
       }

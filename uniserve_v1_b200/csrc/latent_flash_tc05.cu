@@ -5,10 +5,12 @@
 //   us_latent_gather    the latents and rotated parts that a batch's prompts see, from their pages
 //                       into packed rows (sequence by sequence, oldest first)
 //   us_latent_flash     score = q_unrotated . k_head + q_rotated . k_shared, window, softmax, values
+//   us_window_flash     score = q . k, grouped heads, window, softmax with a sink, values
 //
 // The flash kernel is the two-tile scheme of flash_attn2_tc05.cu with unlike operands: a CTA owns 256
 // query rows of one (sequence, head) as tiles A and B; keys come in blocks of 128 as one or two
-// 64-channel slabs of the head's own keys and one slab of the rotated part that all heads share.
+// 64-channel slabs of the head's own keys and, in the latent form, one slab of the rotated part that
+// all heads share.
 // Where 192-wide keys leave no room for two value stages there is one; the block of values is then
 // fetched while the tensor pipe forms the next scores.  Blocks outside a tile's window are skipped.
 // Every wait is bounded.
@@ -91,19 +93,23 @@ struct FlashArgs {
   int V, window;
   float scale_log2;
   unsigned int* status;
+  int rep;                               // query heads per key / value head
+  const float* sink;                     // [H] or null: exp(sink) joins the softmax denominator
+  float out_scale;
 };
 
-// kN: 64-channel slabs of the head's own keys; kDV: value width; kVS: value stages.
-template <int kN, int kDV, int kVS>
+// kN: 64-channel slabs of the head's own keys; kR: slabs of the shared part (0 or 1); kDV: value
+// width; kVS: value stages.
+template <int kN, int kR, int kDV, int kVS>
 __global__ void __launch_bounds__(320, 1)
 latent_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                     const __grid_constant__ CUtensorMap tmR, const __grid_constant__ CUtensorMap tmV,
                     const FlashArgs a) {
   US_PDL_PROLOGUE();
-  constexpr int kS = kN + 1;                     // slabs of a query or key tile
+  constexpr int kS = kN + kR;                    // slabs of a query or key tile
   constexpr int kTile = kS * kSlab, kVTile = kDV / 64 * kSlab;
   const int q_pair = a.window > 0 ? (int)blockIdx.x : (int)gridDim.x - 1 - (int)blockIdx.x;
-  const int h = blockIdx.y, seq = blockIdx.z;
+  const int h = blockIdx.y, hk = h / a.rep, seq = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, tid = threadIdx.x;
   constexpr int kTmaWarp = 8, kMmaWarp = 9;
   const int q_start = a.cu_q[seq], q_len = a.cu_q[seq + 1] - q_start;
@@ -181,8 +187,8 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         tc::mbar_expect_tx(&k_full[st], kTile);
 #pragma unroll
         for (int p = 0; p < kN; ++p)
-          tc::tma_load_2d(sK + st * kTile + p * kSlab, &tmK, &k_full[st], (h * kN + p) * 64, row);
-        tc::tma_load_2d(sK + st * kTile + kN * kSlab, &tmR, &k_full[st], 0, row);
+          tc::tma_load_2d(sK + st * kTile + p * kSlab, &tmK, &k_full[st], (hk * kN + p) * 64, row);
+        if (kR) tc::tma_load_2d(sK + st * kTile + kN * kSlab, &tmR, &k_full[st], 0, row);
         return true;
       };
       auto load_v = [&](int j) {
@@ -191,7 +197,7 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         tc::mbar_expect_tx(&v_full[st], kVTile);
 #pragma unroll
         for (int p = 0; p < kDV / 64; ++p)
-          tc::tma_load_2d(sV + st * kVTile + p * kSlab, &tmV, &v_full[st], h * kDV + p * 64, row);
+          tc::tma_load_2d(sV + st * kVTile + p * kSlab, &tmV, &v_full[st], hk * kDV + p * 64, row);
         return true;
       };
       ok = load_k(0) && (nb < 2 || load_k(1));
@@ -358,7 +364,8 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     if (j1 > j0) {
       if (ok && tc::mbar_wait(&o_full[x], 0, abort_flag)) {
         tc::tc_fence_after_sync();
-        const float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
+        if (a.sink && l_sum > 0.f) l_sum += ex2f(a.sink[h] * 1.4426950408889634f - m_used);
+        const float inv = l_sum > 0.f ? a.out_scale / l_sum : 0.f;
         const bool row_ok = q_idx < q_len, wide = ((a.V | (int)a.ldo) & 7) == 0;
         __nv_bfloat16* orow = a.out + (long long)(q_start + q_idx) * a.ldo + (long long)h * a.V;
 #pragma unroll 1
@@ -394,18 +401,18 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   }
 }
 
-template <int kN, int kDV, int kVS>
+template <int kN, int kR, int kDV, int kVS>
 int launch_flash(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmR,
                  const CUtensorMap& tmV, const FlashArgs& a, dim3 grid, cudaStream_t stream) {
-  constexpr size_t smem = (size_t)4 * (kN + 1) * kSlab + (size_t)kVS * (kDV / 64) * kSlab + 17 * 8 + 1024;
+  constexpr size_t smem = (size_t)4 * (kN + kR) * kSlab + (size_t)kVS * (kDV / 64) * kSlab + 17 * 8 + 1024;
   static_assert(smem <= 227 * 1024, "shared memory of a CTA");
   static bool configured = false;
   if (!configured) {
-    US_CUDA_CHECK(cudaFuncSetAttribute(latent_flash_kernel<kN, kDV, kVS>,
+    US_CUDA_CHECK(cudaFuncSetAttribute(latent_flash_kernel<kN, kR, kDV, kVS>,
                                        cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     configured = true;
   }
-  US_CUDA_CHECK(us::launch_pdl(latent_flash_kernel<kN, kDV, kVS>, grid, dim3(320), smem, stream, tmQ,
+  US_CUDA_CHECK(us::launch_pdl(latent_flash_kernel<kN, kR, kDV, kVS>, grid, dim3(320), smem, stream, tmQ,
                                tmK, tmR, tmV, a));
   return US_OK;
 }
@@ -446,11 +453,39 @@ US_API int us_latent_flash(const void* q, long long ldq, const void* kv, long lo
   if (!rc) rc = us_tmap_2d(&tmR, r, US_TMAP_BF16, Tk, 64, 64, kBN, 64, US_SWZ_128);
   if (!rc) rc = us_tmap_2d(&tmV, v, US_TMAP_BF16, Tk, (uint64_t)H * dv, ldkv, kBN, 64, US_SWZ_128);
   if (rc) return rc;
-  FlashArgs a{cu_q, cu_k, (__nv_bfloat16*)out, ldo, V, window, scale * 1.4426950408889634f, us_status_ptr()};
+  FlashArgs a{cu_q, cu_k, (__nv_bfloat16*)out, ldo, V, window, scale * 1.4426950408889634f, us_status_ptr(), 1,
+              nullptr, 1.f};
   const dim3 grid((max_q + 2 * kBM - 1) / (2 * kBM), H, n_seqs);
   cudaStream_t stream = (cudaStream_t)stream_;
-  if (slabs == 1) return dv == 64 ? launch_flash<1, 64, 2>(tmQ, tmK, tmR, tmV, a, grid, stream)
-                                  : launch_flash<1, 128, 2>(tmQ, tmK, tmR, tmV, a, grid, stream);
-  return dv == 64 ? launch_flash<2, 64, 2>(tmQ, tmK, tmR, tmV, a, grid, stream)
-                  : launch_flash<2, 128, 1>(tmQ, tmK, tmR, tmV, a, grid, stream);
+  if (slabs == 1) return dv == 64 ? launch_flash<1, 1, 64, 2>(tmQ, tmK, tmR, tmV, a, grid, stream)
+                                  : launch_flash<1, 1, 128, 2>(tmQ, tmK, tmR, tmV, a, grid, stream);
+  return dv == 64 ? launch_flash<2, 1, 64, 2>(tmQ, tmK, tmR, tmV, a, grid, stream)
+                  : launch_flash<2, 1, 128, 1>(tmQ, tmK, tmR, tmV, a, grid, stream);
+}
+
+// q [Tq, H slabs 64] rows at ldq; k [Tk, G slabs 64] and v [Tk, G dv] rows at ldk, ldv, query head h reading
+// key / value head h / (H / G); V <= dv output columns per head at column h V of `out`; window 0: every
+// earlier key; sink [H] or null; out_scale multiplies the output.  Sequences without keys are left alone.
+US_API int us_window_flash(const void* q, long long ldq, const void* k, long long ldk, const void* v,
+                           long long ldv, void* out, long long ldo, const int* cu_q, const int* cu_k,
+                           int n_seqs, int Tq, int Tk, int H, int G, int slabs, int dv, int V, int max_q,
+                           int window, float scale, const float* sink, float out_scale, void* stream_) {
+  US_REQUIRE(q && k && v && out && cu_q && cu_k && n_seqs >= 1 && Tq >= 1 && Tk >= 1 && H >= 1 && G >= 1 &&
+             H % G == 0 && max_q >= 1 && V >= 1 && V <= dv);
+  US_REQUIRE((ldq % 8) == 0 && (ldk % 8) == 0 && (ldv % 8) == 0 && ((uintptr_t)q % 16) == 0 &&
+             ((uintptr_t)k % 16) == 0 && ((uintptr_t)v % 16) == 0 && ((uintptr_t)out % 16) == 0);
+  if (slabs < 1 || slabs > 2 || (dv != 64 && dv != 128)) return US_ERR_UNSUPPORTED;
+  CUtensorMap tmQ, tmK, tmV;
+  int rc = us_tmap_2d(&tmQ, q, US_TMAP_BF16, Tq, (uint64_t)H * slabs * 64, ldq, kBM, 64, US_SWZ_128);
+  if (!rc) rc = us_tmap_2d(&tmK, k, US_TMAP_BF16, Tk, (uint64_t)G * slabs * 64, ldk, kBN, 64, US_SWZ_128);
+  if (!rc) rc = us_tmap_2d(&tmV, v, US_TMAP_BF16, Tk, (uint64_t)G * dv, ldv, kBN, 64, US_SWZ_128);
+  if (rc) return rc;
+  FlashArgs a{cu_q, cu_k, (__nv_bfloat16*)out, ldo, V, window, scale * 1.4426950408889634f, us_status_ptr(),
+              H / G, sink, out_scale};
+  const dim3 grid((max_q + 2 * kBM - 1) / (2 * kBM), H, n_seqs);
+  cudaStream_t stream = (cudaStream_t)stream_;
+  if (slabs == 1) return dv == 64 ? launch_flash<1, 0, 64, 2>(tmQ, tmK, tmK, tmV, a, grid, stream)
+                                  : launch_flash<1, 0, 128, 2>(tmQ, tmK, tmK, tmV, a, grid, stream);
+  return dv == 64 ? launch_flash<2, 0, 64, 2>(tmQ, tmK, tmK, tmV, a, grid, stream)
+                  : launch_flash<2, 0, 128, 2>(tmQ, tmK, tmK, tmV, a, grid, stream);
 }

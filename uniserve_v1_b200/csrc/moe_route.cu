@@ -5,6 +5,8 @@
 //                  FLT_EPSILON) -> ids through an optional logical->physical map,
 //                  expert-load counters by logical id.  Rows at or past the
 //                  device word `live` route nowhere (id -1, weight 0).
+//                  With `correction` [E] the choice is by score + correction, the weights
+//                  are the uncorrected scores over their sum (+ 1e-20).
 //   moe_sort       counting sort of the (token, route) pairs by local expert;
 //                  emits the permutation both ways, the expert offsets and the
 //                  list of row tiles the grouped GEMM walks.
@@ -30,13 +32,14 @@ constexpr int kMaxExperts = 1024;
 constexpr int kMaxPerLane = kMaxExperts / 32;
 
 // Softmax, top-k and renormalisation of one token's router logits by one warp.
-template <int PER_LANE>
+template <int PER_LANE, bool CORR>
 __device__ __forceinline__ void topk_token(const float* __restrict__ logits,
                                            int* __restrict__ ids, float* __restrict__ weights,
                                            int t, int E, int top_k, int renorm,
                                            const int* __restrict__ live,
                                            const int* __restrict__ expert_map,
-                                           int* __restrict__ load) {
+                                           int* __restrict__ load,
+                                           const float* __restrict__ correction) {
   const int lane = threadIdx.x & 31;
   if (live && t >= *live) {
     for (int j = lane; j < top_k; j += 32) {
@@ -58,16 +61,30 @@ __device__ __forceinline__ void topk_token(const float* __restrict__ logits,
   float sum = 0.f;
 #pragma unroll
   for (int i = 0; i < PER_LANE; ++i) {
-    v[i] = (lane + 32 * i) < E ? __expf(v[i] - mx) : -1.f;
+    if (CORR)
+      v[i] = (lane + 32 * i) < E ? expf(v[i] - mx) : 0.f;
+    else
+      v[i] = (lane + 32 * i) < E ? __expf(v[i] - mx) : -1.f;
     if (v[i] > 0.f) sum += v[i];
   }
   sum = us::warp_sum(sum);
   const float inv = 1.f / sum;
+  // CORR: v holds the choice scores, s the scores that the weights are made of
+  constexpr float kGone = CORR ? -INFINITY : -1.f;
+  float s[CORR ? PER_LANE : 1];
+  if (CORR) {
+#pragma unroll
+    for (int i = 0; i < PER_LANE; ++i) {
+      const int e = lane + 32 * i;
+      s[CORR ? i : 0] = v[i] * inv;
+      v[i] = e < E ? s[CORR ? i : 0] + correction[e] : -INFINITY;
+    }
+  }
   float picked_sum = 0.f;
   float my_w = 0.f;
   int my_id = -1;
   for (int j = 0; j < top_k; ++j) {
-    float best = -1.f;
+    float best = kGone, score = 0.f;
     int best_e = 0x7fffffff;
 #pragma unroll
     for (int i = 0; i < PER_LANE; ++i) {
@@ -75,18 +92,21 @@ __device__ __forceinline__ void topk_token(const float* __restrict__ logits,
       if (v[i] > best) {  // ascending e inside a lane keeps the lower id on ties
         best = v[i];
         best_e = e;
+        if (CORR) score = s[CORR ? i : 0];
       }
     }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) {
       const float ob = __shfl_xor_sync(0xffffffffu, best, o);
       const int oe = __shfl_xor_sync(0xffffffffu, best_e, o);
+      const float os = CORR ? __shfl_xor_sync(0xffffffffu, score, o) : 0.f;
       if (ob > best || (ob == best && oe < best_e)) {
         best = ob;
         best_e = oe;
+        score = os;
       }
     }
-    const float p = best * inv;
+    const float p = CORR ? score : best * inv;
     picked_sum += p;
     if (lane == j) {
       my_w = p;
@@ -95,27 +115,27 @@ __device__ __forceinline__ void topk_token(const float* __restrict__ logits,
     if ((best_e & 31) == lane) {
 #pragma unroll
       for (int i = 0; i < PER_LANE; ++i)
-        if (i == (best_e >> 5)) v[i] = -1.f;
+        if (i == (best_e >> 5)) v[i] = kGone;
     }
   }
   if (lane < top_k) {
-    if (renorm) my_w = my_w / fmaxf(picked_sum, FLT_EPSILON);
+    if (renorm) my_w = CORR ? my_w / (picked_sum + 1e-20f) : my_w / fmaxf(picked_sum, FLT_EPSILON);
     if (load) atomicAdd(&load[my_id], 1);
     ids[(long long)t * top_k + lane] = expert_map ? expert_map[my_id] : my_id;
     weights[(long long)t * top_k + lane] = my_w;
   }
 }
 
-template <int PER_LANE>
+template <int PER_LANE, bool CORR>
 __global__ void __launch_bounds__(128)
 topk_softmax_kernel(const float* __restrict__ logits, int* __restrict__ ids,
                     float* __restrict__ weights, int T, int E, int top_k, int renorm,
                     const int* __restrict__ live, const int* __restrict__ expert_map,
-                    int* __restrict__ load) {
+                    int* __restrict__ load, const float* __restrict__ correction) {
   US_PDL_PROLOGUE();
   const int t = blockIdx.x * 4 + (threadIdx.x >> 5);
   if (t >= T) return;
-  topk_token<PER_LANE>(logits, ids, weights, t, E, top_k, renorm, live, expert_map, load);
+  topk_token<PER_LANE, CORR>(logits, ids, weights, t, E, top_k, renorm, live, expert_map, load, correction);
 }
 
 // One CTA sorts all routes.  Local experts are [e_lo, e_lo + E).
@@ -359,7 +379,7 @@ moe_sort_cluster_kernel(const int* __restrict__ ids, int R, int e_lo, int E, int
 
 // Routing and sorting in one launch (decode-size batches): the CTA's 32 warps take the
 // tokens in turn, then the whole CTA sorts the routes they wrote.
-template <int PER_LANE>
+template <int PER_LANE, bool CORR>
 __global__ void __launch_bounds__(1024)
 route_sort_kernel(const float* __restrict__ logits, int* __restrict__ ids,
                   float* __restrict__ weights, int T, int E_all, int top_k, int renorm,
@@ -367,10 +387,11 @@ route_sort_kernel(const float* __restrict__ logits, int* __restrict__ ids,
                   int* __restrict__ sorted_route, int* __restrict__ perm_of_route,
                   int* __restrict__ expert_offsets, int* __restrict__ tile_group,
                   int* __restrict__ tile_row0, int* __restrict__ tile_rows,
-                  int* __restrict__ num_tiles, unsigned int* status) {
+                  int* __restrict__ num_tiles, unsigned int* status,
+                  const float* __restrict__ correction) {
   US_PDL_PROLOGUE();
   for (int t = threadIdx.x >> 5; t < T; t += 32)
-    topk_token<PER_LANE>(logits, ids, weights, t, E_all, top_k, renorm, live, nullptr, nullptr);
+    topk_token<PER_LANE, CORR>(logits, ids, weights, t, E_all, top_k, renorm, live, nullptr, nullptr, correction);
   __syncthreads();   // the routes written above are read below by other threads of the CTA
   sort_routes(ids, T * top_k, e_lo, E, block_n, max_tiles, sorted_route, perm_of_route,
               expert_offsets, tile_group, tile_row0, tile_rows, num_tiles, status);
@@ -515,7 +536,7 @@ __device__ __forceinline__ bool grid_wait(const unsigned int* ctr, unsigned int 
 // `sync` holds three zero-initialised counters: [0] CTAs that routed their tokens, [1] set
 // by CTA 0 once the sort is written, [2] CTAs that passed the second wait (the last one
 // clears all three for the next launch).
-template <int PER_LANE>
+template <int PER_LANE, bool CORR>
 __global__ void __launch_bounds__(256)
 route_sort_gather_kernel(const float* __restrict__ logits, int* __restrict__ ids,
                          float* __restrict__ weights, int T, int E_all, int top_k, int renorm,
@@ -526,11 +547,11 @@ route_sort_gather_kernel(const float* __restrict__ logits, int* __restrict__ ids
                          int* __restrict__ tile_rows, int* __restrict__ num_tiles,
                          const __nv_bfloat16* __restrict__ x, int H,
                          __nv_bfloat16* __restrict__ xp, unsigned int* sync,
-                         unsigned int* status) {
+                         unsigned int* status, const float* __restrict__ correction) {
   US_PDL_PROLOGUE();
   const int warps = blockDim.x >> 5;
   for (int t = blockIdx.x * warps + (threadIdx.x >> 5); t < T; t += gridDim.x * warps)
-    topk_token<PER_LANE>(logits, ids, weights, t, E_all, top_k, renorm, live, nullptr, nullptr);
+    topk_token<PER_LANE, CORR>(logits, ids, weights, t, E_all, top_k, renorm, live, nullptr, nullptr, correction);
   __threadfence();
   __syncthreads();
   __shared__ int ok_s;
@@ -572,7 +593,7 @@ route_sort_gather_kernel(const float* __restrict__ logits, int* __restrict__ ids
 
 US_API int us_topk_softmax(const float* logits, int* ids, float* weights, int T, int E, int top_k,
                            int renorm, const int* live, const int* expert_map, int* load,
-                           void* stream_) {
+                           const float* correction, void* stream_) {
   US_REQUIRE(logits && ids && weights && T >= 0 && E >= 1 && E <= kMaxExperts && top_k >= 1 &&
              top_k <= 32 && top_k <= E);
   if (T == 0) return US_OK;
@@ -581,8 +602,8 @@ US_API int us_topk_softmax(const float* logits, int* ids, float* weights, int T,
   const int per = (E + 31) / 32;
 #define US_TOPK(P)                                                                          \
   if (per <= P) {                                                                           \
-    us::launch_pdl(topk_softmax_kernel<P>, dim3(blocks), dim3(128), 0, stream, logits, ids, weights, T, E, top_k,   \
-                                                       renorm, live, expert_map, load);     \
+    us::launch_pdl(correction ? topk_softmax_kernel<P, true> : topk_softmax_kernel<P, false>, dim3(blocks),        \
+                   dim3(128), 0, stream, logits, ids, weights, T, E, top_k, renorm, live, expert_map, load, correction);  \
     US_LAUNCH_CHECK();                                                                      \
     return US_OK;                                                                           \
   }
@@ -663,7 +684,7 @@ US_API int us_route_sort(const float* logits, int* ids, float* weights, int T, i
                          int top_k, int renorm, const int* live, int e_lo, int E, int block_n,
                          int max_tiles, int* sorted_route, int* perm_of_route,
                          int* expert_offsets, int* tile_group, int* tile_row0, int* tile_rows,
-                         int* num_tiles, void* stream_) {
+                         int* num_tiles, const float* correction, void* stream_) {
   US_REQUIRE(logits && ids && weights && T >= 1 && T <= 512 && E_all >= 1 &&
              E_all <= kMaxExperts && top_k >= 1 && top_k <= 32 && top_k <= E_all);
   US_REQUIRE(E >= 1 && E <= kMaxExperts && block_n >= 1 && max_tiles >= 1 && sorted_route &&
@@ -672,11 +693,12 @@ US_API int us_route_sort(const float* logits, int* ids, float* weights, int T, i
   const int per = (E_all + 31) / 32;
 #define US_RS_CASE(P)                                                                          \
   if (per <= P) {                                                                              \
-    US_CUDA_CHECK(us::launch_pdl(route_sort_kernel<P>, dim3(1), dim3(1024), 0, stream, logits, \
+    US_CUDA_CHECK(us::launch_pdl(correction ? route_sort_kernel<P, true> : route_sort_kernel<P, false>, \
+                                 dim3(1), dim3(1024), 0, stream, logits,                       \
                                  ids, weights, T, E_all, top_k, renorm, live, e_lo, E, block_n,\
                                  max_tiles, sorted_route, perm_of_route, expert_offsets,       \
                                  tile_group, tile_row0, tile_rows, num_tiles,                  \
-                                 us_status_ptr()));                                            \
+                                 us_status_ptr(), correction));                                \
     return US_OK;                                                                              \
   }
   US_RS_CASE(1)
@@ -710,7 +732,7 @@ US_API int us_route_sort_gather(const float* logits, int* ids, float* weights, i
                                 int block_n, int max_tiles, int* sorted_route,
                                 int* perm_of_route, int* expert_offsets, int* tile_group,
                                 int* tile_row0, int* tile_rows, int* num_tiles, const void* x,
-                                int H, void* xp, void* sync, void* stream_) {
+                                int H, void* xp, void* sync, const float* correction, void* stream_) {
   US_REQUIRE(logits && ids && weights && T >= 1 && T <= 512 && E_all >= 1 &&
              E_all <= kMaxExperts && top_k >= 1 && top_k <= 32 && top_k <= E_all);
   US_REQUIRE(E >= 1 && E <= kMaxExperts && block_n >= 1 && max_tiles >= 1 && sorted_route &&
@@ -723,12 +745,13 @@ US_API int us_route_sort_gather(const float* logits, int* ids, float* weights, i
   const int per = (E_all + 31) / 32;
 #define US_RSG_CASE(P)                                                                         \
   if (per <= P) {                                                                              \
-    US_CUDA_CHECK(us::launch_pdl(route_sort_gather_kernel<P>, dim3(ctas), dim3(256), 0, stream,\
+    US_CUDA_CHECK(us::launch_pdl(correction ? route_sort_gather_kernel<P, true> : route_sort_gather_kernel<P, false>, \
+                                 dim3(ctas), dim3(256), 0, stream,                             \
                                  logits, ids, weights, T, E_all, top_k, renorm, live, e_lo, E, \
                                  block_n, max_tiles, sorted_route, perm_of_route,              \
                                  expert_offsets, tile_group, tile_row0, tile_rows, num_tiles,  \
                                  (const __nv_bfloat16*)x, H, (__nv_bfloat16*)xp,               \
-                                 (unsigned int*)sync, us_status_ptr()));                       \
+                                 (unsigned int*)sync, us_status_ptr(), correction));           \
     return US_OK;                                                                              \
   }
   US_RSG_CASE(1)

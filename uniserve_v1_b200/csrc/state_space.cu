@@ -3,9 +3,15 @@
 //
 //   S <- exp(-exp(A_log) dt) S + dt B x^T,   y = S^T C + D x        S [N, V] FP32 per head
 //
+// or, with a fixed decay per head (linear attention: x, B, C are its values, keys and queries),
+//
+//   S <- decay S + B x^T,   y = S^T C
+//
 //   us_short_conv          causal convolution + bias + silu of x | B | C, inputs kept in a ring
+//                          (without taps: silu alone)
 //   us_state_space_scan    dt = softplus(raw + bias), the recurrence and its read-out
-//   us_group_norm_gate     y * silu(z), RMS norm over equal parts of the row, weight
+//   us_group_norm_gate     y * silu(z), RMS norm over equal parts of the row, weight; or norm and weight
+//                          first, then sigmoid(z)
 //   us_state_space_step    all of these for one token of every sequence in one launch
 //
 // A sequence whose first packed row stands at position 0 starts from a zero state whatever its
@@ -27,6 +33,7 @@ __device__ __forceinline__ float softplus_f(float x) {
   return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x)));
 }
 __device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
+__device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
 // e^x of a decay: hundreds of factors just below one multiply along a sequence, and a biased last
 // bit would add up; near zero the rounding of 1 + (e^x - 1) is the nearest one.
 __device__ __forceinline__ float decay_exp(float x) { return x > -0.5f ? 1.f + expm1f(x) : expf(x); }
@@ -70,7 +77,7 @@ struct ShortConv {
   const void* x;                // projection rows
   long long ldx;
   int off;
-  const float *taps, *bias;     // [C, K], [C]
+  const float *taps, *bias;     // [C, K], [C]; null: the input itself, no bias
   void* ring;                   // [slots, K, C]: input of position p in entry p % K
   void* y;                      // [T, ldy]
   long long ldy;
@@ -110,10 +117,10 @@ __global__ void __launch_bounds__(128) short_conv_kernel(const ShortConv a) {
   for (int j = 0; j < KT; ++j) {
     const int k = j - (KT - a.K);
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) w[j][e] = k >= 0 ? a.taps[(long long)(c + e) * a.K + k] : 0.f;
+    for (int e = 0; e < VEC; ++e) w[j][e] = k < 0 ? 0.f : a.taps ? a.taps[(long long)(c + e) * a.K + k] : 1.f;
   }
 #pragma unroll
-  for (int e = 0; e < VEC; ++e) b[e] = a.bias[c + e];
+  for (int e = 0; e < VEC; ++e) b[e] = a.bias ? a.bias[c + e] : 0.f;
 #pragma unroll
   for (int j = 1; j < KT; ++j) {                    // inputs of the rows before t0
     const int back = KT - j, src = t0 - back, p = p0 + src - start;
@@ -155,6 +162,7 @@ struct ScanArgs {
   const void* dt;               // raw step sizes, column h of rows at lddt
   long long lddt;
   const float *dt_bias, *A_log, *D;   // [H]
+  const double* log_decay;      // [H] or null; else no step sizes and no D
   float* state;                 // [slots, H, N, V]
   void* y;                      // [T, ldy]
   long long ldy;
@@ -187,7 +195,9 @@ __global__ void __launch_bounds__(128) scan_rows_kernel(const ScanArgs a) {
   }
   const bool fresh = a.pos[start] == 0, col_ok = col < a.V;
   float* Sg = a.state + ((long long)slot * a.H + h) * a.N * a.V;
-  const float A = expf(a.A_log[h]), D = a.D[h], bias = a.dt_bias[h];
+  const bool fixed = a.log_decay != nullptr;
+  const float A = fixed ? 0.f : expf(a.A_log[h]), D = fixed ? 0.f : a.D[h], bias = fixed ? 0.f : a.dt_bias[h];
+  const float decay = fixed ? (float)exp(a.log_decay[h]) : 0.f;
   const long long ob = (long long)a.H * a.V + (long long)g * a.N, oc = ob + (long long)a.G * a.N;
   float S[kPer];
 #pragma unroll
@@ -208,7 +218,12 @@ __global__ void __launch_bounds__(128) scan_rows_kernel(const ScanArgs a) {
       const int t = e / kCols, c = blockIdx.x * kCols + e % kCols;
       xs[t][e % kCols] = c < a.V ? ld_any(a.u, (long long)(start + c0 + t) * a.ldu + (long long)h * a.V + c, a.bf16) : 0.f;
     }
-    if (tid < n) {
+    if (fixed) {
+      if (tid < n) {
+        dts[tid] = 1.f;
+        dec[tid] = decay;
+      }
+    } else if (tid < n) {
       const float dt = softplus_f(ld_any(a.dt, (long long)(start + c0 + tid) * a.lddt + h, a.bf16) + bias);
       dts[tid] = dt;
       dec[tid] = decay_exp(-A * dt);
@@ -251,7 +266,8 @@ template <int NV, int VEC>
 __global__ void __launch_bounds__(256)
 group_norm_gate_kernel(const void* __restrict__ y, long long ldy, const void* __restrict__ z,
                        long long ldz, int groups, const float* __restrict__ w, void* __restrict__ out,
-                       long long ldo, int n, float eps, int bf16, int z_bf16) {
+                       long long ldo, int n, float eps, int bf16, int z_bf16,
+                       int after, long long padded) {
   US_PDL_PROLOGUE();
   __shared__ float part[8];
   const int len = n / groups, g = blockIdx.y, step = blockDim.x * VEC, c0 = threadIdx.x * VEC;
@@ -261,6 +277,7 @@ group_norm_gate_kernel(const void* __restrict__ y, long long ldy, const void* __
   auto gated = [&](int c, float (&v)[VEC]) {
     float gz[VEC];
     ld_vec<VEC>(v, y, yi + c, bf16);
+    if (after) return;
     ld_vec<VEC>(gz, z, zi + c, z_bf16);
 #pragma unroll
     for (int e = 0; e < VEC; ++e) v[e] *= silu_f(gz[e]);
@@ -268,6 +285,12 @@ group_norm_gate_kernel(const void* __restrict__ y, long long ldy, const void* __
   auto put = [&](int c, float (&v)[VEC], float inv) {
 #pragma unroll
     for (int e = 0; e < VEC; ++e) v[e] *= inv * w[g * len + c + e];
+    if (after) {
+      float gz[VEC];
+      ld_vec<VEC>(gz, z, zi + c, z_bf16);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) v[e] *= sigmoid_f(gz[e]);
+    }
     st_vec<VEC>(out, oi + c, bf16, v);
   };
   float held[NV > 0 ? NV : 1][VEC], ss = 0.f;
@@ -304,7 +327,7 @@ group_norm_gate_kernel(const void* __restrict__ y, long long ldy, const void* __
     }
   }
   if (g == groups - 1)
-    for (long long c = n + threadIdx.x; c < ldo; c += blockDim.x)
+    for (long long c = n + threadIdx.x; c < padded; c += blockDim.x)
       st_any(out, (long long)blockIdx.x * ldo + c, bf16, 0.f);
 }
 
@@ -313,14 +336,16 @@ struct StepArgs {
   const void* x;                // projection rows: z | x B C | dt at the three offsets
   long long ldx;
   int oz, oc, odt;
-  const float *taps, *bias;     // [C, K], [C]
+  const float *taps, *bias;     // [C, K], [C]; null: the input itself, no bias
   void* ring;                   // [slots, K, C]
   const float *dt_bias, *A_log, *D, *w;   // [H] x 3, [H * V]
+  const double* log_decay;      // [H] or null; else no step sizes and no D
   float* state;                 // [slots, H, N, V]
   void* out;                    // [B, ldo]
   long long ldo;
   const int *slots, *pos;
   int H, V, N, G, K, bf16, heads;         // heads: of a norm part (the cluster), 0: no gate and norm
+  int after;                    // gate: silu before the norm (0) or sigmoid after it (1)
   float eps;
 };
 
@@ -363,7 +388,7 @@ __global__ void __launch_bounds__(kStepThreads, R <= 8 ? 3 : 2) state_space_step
                             : inner + (e < a.V + a.N ? g * a.N + e - a.V : (a.G + g) * a.N + e - a.V - a.N);
       const float now = ld_any(a.x, (long long)b * a.ldx + a.oc + c, a.bf16);
       const float* w = a.taps + (long long)c * a.K;
-      float acc = fmaf(w[a.K - 1], now, a.bias[c]);
+      float acc = a.taps ? fmaf(w[a.K - 1], now, a.bias ? a.bias[c] : 0.f) : now;
       for (int k = 1; k < min(a.K, p + 1); ++k)
         acc = fmaf(w[a.K - 1 - k], ld_any(a.ring, ((long long)slot * a.K + (p - k) % a.K) * C + c, a.bf16), acc);
       if (a.K > 1 && (e < a.V || keeps))
@@ -371,7 +396,10 @@ __global__ void __launch_bounds__(kStepThreads, R <= 8 ? 3 : 2) state_space_step
       acc = silu_f(acc);
       u[e] = a.bf16 ? us::bf2f(us::f2bf(acc)) : acc;
     }
-    if (tid == kStepThreads - 1) {
+    if (tid == kStepThreads - 1 && a.log_decay) {
+      steps[0] = 1.f;
+      steps[1] = (float)exp(a.log_decay[h]);
+    } else if (tid == kStepThreads - 1) {
       const float dt = softplus_f(ld_any(a.x, (long long)b * a.ldx + a.odt + h, a.bf16) + a.dt_bias[h]);
       steps[0] = dt;
       steps[1] = decay_exp(-expf(a.A_log[h]) * dt);
@@ -405,7 +433,7 @@ __global__ void __launch_bounds__(kStepThreads, R <= 8 ? 3 : 2) state_space_step
   __syncthreads();
   if (live && mine) {
     for (int r = 0; r < GR; ++r) y += red[r * VQ * 4 + tid];
-    y = fmaf(a.D[h], u[tid], y);
+    if (!a.log_decay) y = fmaf(a.D[h], u[tid], y);
     if (a.bf16) y = us::bf2f(us::f2bf(y));
   }
   const long long at = (long long)b * a.ldo + (long long)h * a.V + tid;
@@ -413,7 +441,7 @@ __global__ void __launch_bounds__(kStepThreads, R <= 8 ? 3 : 2) state_space_step
     if (mine) st_any(a.out, at, a.bf16, y);
     return;
   }
-  y *= silu_f(z);
+  if (!a.after) y *= silu_f(z);
   float ss = us::block_sum(y * y, part);
   if (a.heads > 1) {
     if (tid == 0) total = ss;
@@ -422,9 +450,11 @@ __global__ void __launch_bounds__(kStepThreads, R <= 8 ? 3 : 2) state_space_step
     ss = 0.f;
     for (int r = 0; r < a.heads; ++r) ss += tc::ld_dsmem_f32(tc::map_to_cta(addr, r));
   }
-  if (mine)
+  if (mine) {
+    if (a.after) y *= sigmoid_f(z);
     st_any(a.out, at, a.bf16,
            live ? y * (1.f / sqrtf(ss / (float)(max(a.heads, 1) * a.V) + a.eps)) * a.w[h * a.V + tid] : 0.f);
+  }
   if (a.heads > 1) tc::cluster_sync();            // nobody leaves while its sum may still be read
 }
 
@@ -464,7 +494,7 @@ US_API int us_short_conv(const void* x, long long ldx, int off, const float* tap
                          void* ring, void* y, long long ldy, const int* cu, const int* slots,
                          const int* pos, int B, int T, int C, int K, int bf16, int one_token,
                          void* stream_) {
-  US_REQUIRE(x && taps && bias && y && cu && slots && pos && B >= 1 && T >= 0 && C >= 1 && K >= 1);
+  US_REQUIRE(x && y && cu && slots && pos && B >= 1 && T >= 0 && C >= 1 && K >= 1 && (taps || K == 1));
   US_REQUIRE((K == 1 || ring) && (!one_token || B == T));
   if (K > kMaxTaps) return US_ERR_LIMIT;
   if (T == 0) return US_OK;
@@ -490,15 +520,15 @@ US_API int us_short_conv(const void* x, long long ldx, int off, const float* tap
 
 US_API int us_state_space_scan(const void* u, long long ldu, const void* proj, long long ldp,
                                int off_dt, const float* dt_bias, const float* A_log, const float* D,
-                               float* state, void* y, long long ldy, const int* cu, const int* slots,
-                               const int* pos, int B, int T, int H, int V, int N, int G, int bf16,
-                               void* stream_) {
-  US_REQUIRE(u && proj && dt_bias && A_log && D && state && y && cu && slots && pos);
+                               const double* log_decay, float* state, void* y, long long ldy,
+                               const int* cu, const int* slots, const int* pos, int B, int T, int H,
+                               int V, int N, int G, int bf16, void* stream_) {
+  US_REQUIRE(u && (log_decay || (proj && dt_bias && A_log && D)) && state && y && cu && slots && pos);
   US_REQUIRE(B >= 1 && T >= 0 && H >= 1 && V >= 1 && N >= 1 && G >= 1 && H % G == 0);
   if (T == 0) return US_OK;
   const void* dt = bf16 ? (const void*)((const __nv_bfloat16*)proj + off_dt)
                         : (const void*)((const float*)proj + off_dt);
-  ScanArgs a{u, ldu, dt, ldp, dt_bias, A_log, D, state, y, ldy, cu, slots, pos, T, H, V, N, G, bf16};
+  ScanArgs a{u, ldu, dt, ldp, dt_bias, A_log, D, log_decay, state, y, ldy, cu, slots, pos, T, H, V, N, G, bf16};
   const dim3 grid(us::ceil_div(V, kCols), H, B);
 #define US_SCAN(NP)                                                                                \
   US_CUDA_CHECK(us::launch_pdl(scan_rows_kernel<NP>, grid, dim3(128), 0, (cudaStream_t)stream_, a))
@@ -512,10 +542,12 @@ US_API int us_state_space_scan(const void* u, long long ldu, const void* proj, l
   return US_OK;
 }
 
+// Columns n .. padded of an output row become zero.
 US_API int us_group_norm_gate(const void* y, long long ldy, const void* z, long long ldz, int groups,
-                              const float* w, void* out, long long ldo, int T, int n, int bf16,
-                              float eps, int z_bf16, void* stream_) {
-  US_REQUIRE(y && z && w && out && T >= 0 && n >= 1 && groups >= 1 && n % groups == 0 && ldo >= n);
+                              const float* w, void* out, long long ldo, int padded, int T, int n,
+                              int bf16, float eps, int z_bf16, int after, void* stream_) {
+  US_REQUIRE(y && z && w && out && T >= 0 && n >= 1 && groups >= 1 && n % groups == 0 && padded >= n &&
+             ldo >= padded);
   if (T == 0) return US_OK;
   const int len = n / groups, yb = bf16 ? 8 : 16, zb = z_bf16 ? 8 : 16;
   const bool vec = (len % 4) == 0 && (ldy % 4) == 0 && (ldz % 4) == 0 && (ldo % 4) == 0 &&
@@ -526,7 +558,7 @@ US_API int us_group_norm_gate(const void* y, long long ldy, const void* z, long 
 #define US_GN(NV, VEC)                                                                             \
   US_CUDA_CHECK(us::launch_pdl(group_norm_gate_kernel<NV, VEC>, grid, dim3(threads), 0,             \
                                (cudaStream_t)stream_, y, ldy, z, ldz, groups, w, out, ldo, n, eps,  \
-                               bf16, z_bf16))
+                               bf16, z_bf16, after, (long long)padded))
   if (vec) {
     if (nv <= 1) US_GN(1, 4);
     else if (nv <= 2) US_GN(2, 4);
@@ -546,17 +578,18 @@ US_API int us_group_norm_gate(const void* y, long long ldy, const void* z, long 
 US_API int us_state_space_step(const void* x, long long ldx, int oz, int oc, int odt,
                                const float* taps, const float* bias, void* ring,
                                const float* dt_bias, const float* A_log, const float* D,
-                               const float* w, float* state, void* out, long long ldo,
-                               const int* slots, const int* pos, int B, int H, int V, int N, int G,
-                               int K, int bf16, int heads, float eps, void* stream_) {
-  US_REQUIRE(x && taps && bias && dt_bias && A_log && D && state && out && slots && pos);
+                               const double* log_decay, const float* w, float* state, void* out,
+                               long long ldo, const int* slots, const int* pos, int B, int H, int V,
+                               int N, int G, int K, int bf16, int heads, int after, float eps,
+                               void* stream_) {
+  US_REQUIRE(x && (taps || K == 1) && (log_decay || (dt_bias && A_log && D)) && state && out && slots && pos);
   US_REQUIRE(B >= 0 && H >= 1 && V >= 4 && N >= 1 && G >= 1 && H % G == 0 && K >= 1 && (K == 1 || ring) &&
              (V % 4) == 0 && heads >= 0 && heads <= 8 && (heads == 0 || (H % heads == 0 && w)) && B <= 65535);
   const int vq = V <= 32 ? 8 : V <= 64 ? 16 : V <= 128 ? 32 : 64;
   if (V > 256 || us::ceil_div(N, kStepThreads / vq) > 16) return US_ERR_LIMIT;
   if (B == 0) return US_OK;
-  StepArgs a{x, ldx, oz, oc, odt, taps, bias, ring, dt_bias, A_log, D, w, state, out, ldo, slots, pos,
-             H, V, N, G, K, bf16, heads, eps};
+  StepArgs a{x, ldx, oz, oc, odt, taps, bias, ring, dt_bias, A_log, D, w, log_decay, state, out, ldo, slots, pos,
+             H, V, N, G, K, bf16, heads, after, eps};
   cudaStream_t stream = (cudaStream_t)stream_;
   switch (vq) {
     case 8: return launch_step<8>(a, B, stream);

@@ -5,6 +5,8 @@
 //   y_t  = e^{c_t} S^T C_t + sum_{s <= t} (C_t . B_s) e^{c_t - c_s} dt_s x_s + D x_t
 //   S'   = e^{c_63} S + sum_s B_s (e^{c_63 - c_s} dt_s x_s)^T
 //
+// A fixed decay per head is a_t = log decay, dt_t = 1, D = 0.
+//
 // The recurrence stays a 32-bit one: B, C and x are bf16 values and exact operands, and every FP32
 // operand (S, the decayed scores, the weighted x) enters as the sum of three bf16 values, which
 // holds all 24 bits; products accumulate in FP32 and S lives in FP32 accumulators across chunks.
@@ -30,6 +32,7 @@ struct ChunkArgs {
   const __nv_bfloat16* dt;          // raw step sizes, column h of rows at lddt
   long long lddt;
   const float *dt_bias, *A_log, *D;
+  const double* log_decay;          // [H] or null
   float* state;                     // [slots, H, N, V]
   __nv_bfloat16* y;
   long long ldy;
@@ -61,11 +64,14 @@ __device__ __forceinline__ void split3(float x, float y, uint32_t (&o)[3]) {
 }
 
 // One warp: exponents of the chunk whose raw step sizes its lanes hold (tokens 2 lane, 2 lane + 1).
+// With `fixed`, *fixed is every token's exponent.
 __device__ __forceinline__ void form_exponents(Exponents& x, float raw0, float raw1, int n, float A,
-                                               float bias) {
+                                               float bias, const double* fixed) {
   const int lane = threadIdx.x & 31, t = 2 * lane;
-  const float d0 = t < n ? softplus_f(raw0 + bias) : 0.f, d1 = t + 1 < n ? softplus_f(raw1 + bias) : 0.f;
-  const double a0 = -(double)(A * d0), a1 = -(double)(A * d1);
+  const float d0 = t >= n ? 0.f : fixed ? 1.f : softplus_f(raw0 + bias);
+  const float d1 = t + 1 >= n ? 0.f : fixed ? 1.f : softplus_f(raw1 + bias);
+  const double a0 = fixed ? (double)d0 * *fixed : -(double)(A * d0);
+  const double a1 = fixed ? (double)d1 * *fixed : -(double)(A * d1);
   double s = a0 + a1;
 #pragma unroll
   for (int o = 1; o < 32; o <<= 1) {
@@ -112,7 +118,8 @@ __global__ void __launch_bounds__(kThreads, 1) state_space_chunk_kernel(const Ch
   }
   const bool fresh = a.pos[start] == 0;
   float* Sg = a.state + ((long long)slot * a.H + h) * a.N * a.V;
-  const float A = expf(a.A_log[h]), bias = a.dt_bias[h], D = a.D[h];
+  const double* fixed = a.log_decay ? a.log_decay + h : nullptr;
+  const float A = fixed ? 0.f : expf(a.A_log[h]), bias = fixed ? 0.f : a.dt_bias[h], D = fixed ? 0.f : a.D[h];
   const __nv_bfloat16* xg = a.u + (long long)start * a.ldu + (long long)h * a.V + v0;
   const __nv_bfloat16* bg = a.u + (long long)start * a.ldu + (long long)a.H * a.V + (long long)g * a.N;
   const __nv_bfloat16* cg = bg + (long long)a.G * a.N;
@@ -143,6 +150,7 @@ __global__ void __launch_bounds__(kThreads, 1) state_space_chunk_kernel(const Ch
   const int chunks = (T + kQ - 1) / kQ;
   float raw0 = 0.f, raw1 = 0.f;
   auto fetch_steps = [&](int c) {                     // warp 0's lanes: two tokens each
+    if (fixed) return;
     const int t = c * kQ + 2 * lane;
     raw0 = t < T ? us::bf2f(a.dt[(long long)(start + t) * a.lddt + h]) : 0.f;
     raw1 = t + 1 < T ? us::bf2f(a.dt[(long long)(start + t + 1) * a.lddt + h]) : 0.f;
@@ -150,7 +158,7 @@ __global__ void __launch_bounds__(kThreads, 1) state_space_chunk_kernel(const Ch
   fetch(0, 0);
   if (warp == 0) {
     fetch_steps(0);
-    form_exponents(ex[0], raw0, raw1, min(kQ, T), A, bias);
+    form_exponents(ex[0], raw0, raw1, min(kQ, T), A, bias, fixed);
     if (chunks > 1) fetch_steps(1);
   }
   // state: warp (block m, part) holds rows 16 m .. and SN column tiles
@@ -206,7 +214,7 @@ __global__ void __launch_bounds__(kThreads, 1) state_space_chunk_kernel(const Ch
     __syncthreads();
     // the next chunk's exponents, while the other warps multiply
     if (warp == 0 && c + 1 < chunks) {
-      form_exponents(ex[buf ^ 1], raw0, raw1, min(kQ, T - (c + 1) * kQ), A, bias);
+      form_exponents(ex[buf ^ 1], raw0, raw1, min(kQ, T - (c + 1) * kQ), A, bias, fixed);
       if (c + 2 < chunks) fetch_steps(c + 2);
     }
     float acc[4][4];
@@ -357,16 +365,16 @@ int launch_chunk(const ChunkArgs& a, int B, cudaStream_t stream) {
 // Widths N <= 128 and V, every offset a multiple of 8.
 US_API int us_state_space_chunks(const void* u, long long ldu, const void* proj, long long ldp,
                                  int off_dt, const float* dt_bias, const float* A_log, const float* D,
-                                 float* state, void* y, long long ldy, const int* cu,
+                                 const double* log_decay, float* state, void* y, long long ldy, const int* cu,
                                  const int* slots, const int* pos, int B, int T, int H, int V, int N,
                                  int G, void* stream_) {
-  US_REQUIRE(u && proj && dt_bias && A_log && D && state && y && cu && slots && pos);
+  US_REQUIRE(u && (log_decay || (proj && dt_bias && A_log && D)) && state && y && cu && slots && pos);
   US_REQUIRE(B >= 1 && T >= 0 && H >= 1 && V >= 1 && N >= 1 && G >= 1 && H % G == 0);
   US_REQUIRE((V % 8) == 0 && (N % 8) == 0 && (ldu % 8) == 0 && (ldy % 2) == 0 && ((uintptr_t)u % 16) == 0 &&
              ((uintptr_t)y % 4) == 0);
   if (N > 128) return US_ERR_LIMIT;
   if (T == 0) return US_OK;
   ChunkArgs a{(const __nv_bfloat16*)u, ldu, (const __nv_bfloat16*)proj + off_dt, ldp, dt_bias, A_log, D,
-              state, (__nv_bfloat16*)y, ldy, cu, slots, pos, H, V, N, G};
+              log_decay, state, (__nv_bfloat16*)y, ldy, cu, slots, pos, H, V, N, G};
   return N <= 64 ? launch_chunk<64>(a, B, (cudaStream_t)stream_) : launch_chunk<128>(a, B, (cudaStream_t)stream_);
 }

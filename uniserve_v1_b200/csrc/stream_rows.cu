@@ -2,8 +2,12 @@
 //
 //   source   r(t) = rms(embed[id] * scale + table2[row]) * w              start of the stream
 //            r(t) = residual(t) + rms(y(t)) * w                           output norm and add
+//            r(t) = embed[id] * scale,  residual(t) + gain * y(t)         without w (plain form)
 //   output   h(t) = rms(r(t)) * w_out                                     input norm
 //            x(t) = h(t)   or   h(t) + (h(t - 1) - h(t)) * mu             token shift
+//
+// In the plain form y may also be a mixture of experts: sum_k weight_k * (row perm_k of the expert rows,
+// or row t of `ident` for an expert without tensors, perm_k < 0) + shared(t).
 //
 // with rms(v) = v / sqrt(mean(v^2) + eps).  r goes to a second residual buffer (the one that is
 // read stays as it is), because a shifted row needs its neighbour's h: a CTA takes up to kRows
@@ -69,7 +73,7 @@ struct StreamRows {
   int vocab, n2;
   const void* y;              // [T, W] sublayer output (null: start of the stream)
   const float* residual;      // [T, W]
-  const float* w;             // [W]
+  const float* w;             // [W], null: plain form
   float* residual_out;        // [T, W]
   const float* w_out;         // [W]
   const float* mu;            // [W] or null: no token shift
@@ -80,9 +84,16 @@ struct StreamRows {
   float eps;
   int rows;                   // rows per CTA without a shift
   unsigned int* status;
+  // plain form
+  float gain;
+  const void* y_perm;         // expert rows, or null: y
+  const int* perm;            // [T, top]
+  const float* route_w;       // [T, top]
+  int top;
+  const void *ident, *shared; // [T, W] or null
 };
 
-template <int NV>
+template <int NV, bool PLAIN>
 __global__ void __launch_bounds__(256) stream_rows_kernel(const StreamRows a) {
   US_PDL_PROLOGUE();
   __shared__ float buf[64];
@@ -116,7 +127,33 @@ __global__ void __launch_bounds__(256) stream_rows_kernel(const StreamRows a) {
   // raw operands of a row: the sublayer's output (or the embedding sum) and the residual
   auto load = [&](int t, float4 (&v)[NV], float4 (&r)[NV]) {
     const long long base = (long long)t * W;
-    if (a.y) {
+    if (PLAIN && a.y_perm) {
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int c = c0 + i * step;
+        v[i] = r[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (c >= W) continue;
+        if (a.shared) v[i] = ld4(a.shared, base + c, a.bf16);
+        r[i] = *reinterpret_cast<const float4*>(a.residual + base + c);
+      }
+      const long long k0 = (long long)t * a.top;
+#pragma unroll 4
+      for (int k = 0; k < a.top; ++k) {
+        const int p = a.perm[k0 + k];
+        const float wk = a.route_w[k0 + k];
+        if (p < 0 && !a.ident) continue;
+        const void* from = p < 0 ? a.ident : a.y_perm;
+        const long long row = (long long)(p < 0 ? t : p) * W;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+          const int c = c0 + i * step;
+          if (c >= W) continue;
+          const float4 e = ld4(from, row + c, a.bf16);
+          v[i] = make_float4(fmaf(wk, e.x, v[i].x), fmaf(wk, e.y, v[i].y), fmaf(wk, e.z, v[i].z),
+                             fmaf(wk, e.w, v[i].w));
+        }
+      }
+    } else if (a.y) {
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
         const int c = c0 + i * step;
@@ -142,6 +179,13 @@ __global__ void __launch_bounds__(256) stream_rows_kernel(const StreamRows a) {
     }
   };
   auto source = [&](float4 (&v)[NV], const float4 (&r)[NV]) {     // v becomes the row of the stream
+    if (PLAIN) {
+#pragma unroll
+      for (int i = 0; i < NV; ++i)
+        v[i] = make_float4(fmaf(a.gain, v[i].x, r[i].x), fmaf(a.gain, v[i].y, r[i].y),
+                           fmaf(a.gain, v[i].z, r[i].z), fmaf(a.gain, v[i].w, r[i].w));
+      return;
+    }
     float ss = 0.f;
 #pragma unroll
     for (int i = 0; i < NV; ++i) ss += sq4(v[i]);
@@ -316,6 +360,27 @@ int block_threads(int W) { return min(256, (W / 4 + 31) / 32 * 32); }
 
 }  // namespace
 
+namespace {
+
+template <bool PLAIN>
+int launch_stream(const StreamRows& a, cudaStream_t stream) {
+  const int grid = !a.mu ? us::ceil_div(a.T, a.rows) : a.one_token ? a.T : a.T / kRows + a.B;
+  const dim3 block(block_threads(a.W));
+  const int nv = us::ceil_div(a.W, 1024);
+#define US_STREAM(N) \
+  US_CUDA_CHECK(us::launch_pdl(stream_rows_kernel<N, PLAIN>, dim3(grid), block, 0, stream, a))
+  if (nv <= 1) US_STREAM(1);
+  else if (nv <= 2) US_STREAM(2);
+  else if (nv <= 4) US_STREAM(4);
+  else if (nv <= 8) US_STREAM(8);
+  else if (nv <= 16) US_STREAM(16);
+  else return US_ERR_LIMIT;
+#undef US_STREAM
+  return US_OK;
+}
+
+}  // namespace
+
 // Start of the stream (y null) or output norm and add, then the next sublayer's input rows.
 US_API int us_stream_rows(const int* ids, const int* rows2, const void* table, const void* table2,
                           float scale, int vocab, int n2, const void* y, const float* residual,
@@ -330,19 +395,24 @@ US_API int us_stream_rows(const int* ids, const int* rows2, const void* table, c
   if (T == 0) return US_OK;
   StreamRows a{ids, rows2, table, table2, scale, vocab, n2, y, residual, w, residual_out, w_out, mu,
                state, cu, slots, pos, x, B, T, W, width, bf16, one_token, eps, T >= 2048 ? 4 : 1, us_status_ptr()};
-  const int grid = !mu ? us::ceil_div(T, a.rows) : one_token ? T : T / kRows + B;
-  const dim3 block(block_threads(W));
-  const int nv = us::ceil_div(W, 1024);
-#define US_STREAM(N)                                                                              \
-  US_CUDA_CHECK(us::launch_pdl(stream_rows_kernel<N>, dim3(grid), block, 0, (cudaStream_t)stream_, a))
-  if (nv <= 1) US_STREAM(1);
-  else if (nv <= 2) US_STREAM(2);
-  else if (nv <= 4) US_STREAM(4);
-  else if (nv <= 8) US_STREAM(8);
-  else if (nv <= 16) US_STREAM(16);
-  else return US_ERR_LIMIT;
-#undef US_STREAM
-  return US_OK;
+  return launch_stream<false>(a, (cudaStream_t)stream_);
+}
+
+// The plain form: residual_out = table row * scale (ids given), or residual + gain * (y, or the mixture
+// of `top` expert rows per token); x = rms(residual_out) * w_out.
+US_API int us_plain_rows(const int* ids, const void* table, float scale, int vocab, const void* y,
+                         const void* y_perm, const int* perm, const float* route_w, int top,
+                         const void* ident, const void* shared, float gain, const float* residual,
+                         float* residual_out, const float* w_out, void* x, int T, int W, int width,
+                         int bf16, float eps, void* stream_) {
+  US_REQUIRE(residual_out && w_out && x && T >= 0 && W >= 8 && (W % 8) == 0 && width >= 1 && width <= W);
+  US_REQUIRE(y || y_perm ? residual && residual != residual_out : ids && table);
+  US_REQUIRE(!y_perm || (perm && route_w && top >= 1 && !y));
+  if (T == 0) return US_OK;
+  StreamRows a{ids, nullptr, table, nullptr, scale, vocab, 0, y, residual, nullptr, residual_out, w_out, nullptr,
+               nullptr, nullptr, nullptr, nullptr, x, 1, T, W, width, bf16, 0, eps, T >= 2048 ? 4 : 1, us_status_ptr(),
+               y || y_perm ? gain : 1.f, y_perm, perm, route_w, top, ident, shared};
+  return launch_stream<true>(a, (cudaStream_t)stream_);
 }
 
 US_API int us_bigram_rows(const int* ids, int* last, const int* cu, const int* slots, const int* pos,

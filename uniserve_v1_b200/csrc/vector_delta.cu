@@ -1,17 +1,19 @@
-// Recurrent mixers whose decay is a vector over the key channels of a head, for packed batches
-// of sequences with their state in slots of a pool:
+// Recurrent mixers with a delta rule, for packed batches of sequences with their state in slots of
+// a pool.  The decay is a vector over the key channels of a head, or one number per head:
 //
 //   channel rule   S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;       o = S^T q
+//   head rule      the same with a scalar g
 //   general rule   S <- diag(w) S - (a*n)(n^T S) + k v^T  (both read the old S);  o = S^T q
 //
-// with S [D, V] FP32 per (sequence, head).  Three kernels:
+// with S [D, V] FP32 per (sequence, head).  The kernels:
 //
 //   us_channel_delta_prep   short causal convolutions + silu of q, k, v, unit q and k, the decay
 //                           g = exp(-exp(A_log) softplus(low + dt_bias)) and beta = sigmoid(b)
+//   us_head_delta_prep      the same with the decay's argument a column per head of the projection
 //   us_general_delta_prep   decay w = exp(-c sigmoid(low + w0)), unit key n, removal a * n
 //   us_vector_delta_rule    the recurrence
-//   us_head_norm_gate       per-head RMS norm of o, weight, sigmoid gate
-//   us_{channel,general}_delta_step   all of these for one token of every sequence in one launch
+//   us_head_norm_gate       per-head RMS norm of o, weight, sigmoid or silu gate
+//   us_{channel,head,general}_delta_step   all of these for one token of every sequence in one launch
 //
 // The preparation is parallel over tokens, so the recurrence reads finished FP32 vectors and
 // does nothing but its multiply-adds.  A sequence whose first packed row stands at position 0
@@ -37,6 +39,10 @@ __device__ __forceinline__ void st_any(void* base, long long idx, int bf16, floa
   else reinterpret_cast<float*>(base)[idx] = v;
 }
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
+__device__ __forceinline__ float gate_f(float x, int silu) {
+  const float s = sigmoid_f(x);
+  return silu ? x * s : s;
+}
 __device__ __forceinline__ float softplus_f(float x) {
   return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x)));
 }
@@ -57,18 +63,21 @@ __device__ __forceinline__ int seq_of(const int* cu, int B, int t) {
 
 constexpr int kMaxTaps = 16;
 constexpr int kMaxDim = 256;      // key channels per head
-constexpr int kPrepTokens = 16;   // consecutive rows of one warp in the prefill form
+constexpr int kPrepTokens = 16;   // consecutive rows of one warp in the prefill form (<= 32)
+
+enum Rule : int { kChannel = 0, kGeneral = 1, kHead = 2 };
 
 struct ChannelPrep {
   const void* x;                // projection rows, element type = bf16 flag
   long long ldx;
   int off_q, off_k, off_v, off_b;
   const float *cq, *ck, *cv;    // taps [channels, K]
-  const float* low;             // [rows, H * D]
+  const float* low;             // [rows, H * D], or null: a decay per head from column off_a
   long long ldlow;
-  const float *A_log, *dt_bias; // [H], [H * D]
+  int off_a;
+  const float *A_log, *dt_bias; // [H], [H * D] (per head: [H])
   void* conv;                   // [slots, K, C], C = 2 Hk D + H V: input of position p in entry p % K
-  float *q, *k, *v, *g, *beta;  // [rows, Hk, D] x 2, [rows, H, V], [rows, H, D], [rows, H]
+  float *q, *k, *v, *g, *beta;  // [rows, Hk, D] x 2, [rows, H, V], [rows, H, D] or [rows, H], [rows, H]
   const int *cu, *slots, *pos;
   int B, rows, H, Hk, D, V, K, bf16, one_token;
 };
@@ -93,6 +102,14 @@ __global__ void __launch_bounds__(256) channel_prep_kernel(const ChannelPrep a) 
   if (unit >= 2 * a.Hk + a.H) {                       // decay and step size
     const int h = unit - 2 * a.Hk - a.H;
     const float A = expf(a.A_log[h]);
+    if (!a.low) {                                     // a lane per row
+      if (t0 + lane < t1) {
+        const long long row = t0 + lane, at = row * a.H + h;
+        a.g[at] = decay_exp(-A * softplus_f(ld_any(a.x, row * a.ldx + a.off_a + h, a.bf16) + a.dt_bias[h]));
+        a.beta[at] = sigmoid_f(ld_any(a.x, row * a.ldx + a.off_b + h, a.bf16));
+      }
+      return;
+    }
 #pragma unroll 2
     for (int t = t0; t < t1; ++t) {
       const float* lo = a.low + (long long)t * a.ldlow + (long long)h * a.D;
@@ -259,10 +276,10 @@ constexpr int kRuleBufs = 4;                         // chunks of vectors in sha
 
 struct RuleArgs {
   const float *q, *k, *v;         // [rows, Hk, D] x 2, [rows, H, V]
-  const float* g;                 // decay [rows, H, D]
+  const float* g;                 // decay [rows, H, D] (head rule: [rows, H])
   const float* n;                 // general: removal direction [rows, H, D]
   const float* p;                 // general: removal rate * direction [rows, H, D]
-  const float* beta;              // channel: [rows, H]
+  const float* beta;              // channel, head: [rows, H]
   float* state;                   // [slots, H, D, V]
   float* out;                     // [rows, H, V]
   const int *cu, *slots, *pos;
@@ -316,11 +333,12 @@ __device__ __forceinline__ void cp_async(float* dst, const float* src) {
   else asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(d), "l"(src) : "memory");
 }
 
-// A token in shared memory: kVecs vectors of DP floats (g, k, q and, general, n, p), then 32
-// columns of v and beta.
-template <int DP, bool GENERAL>
+// A token in shared memory: kVecs vectors of DP floats (g, k, q and, general, n, p; head: k, q), then
+// 32 columns of v, beta and, head, g.
+template <int DP, int RULE>
 struct Stage {
-  static constexpr int kVecs = GENERAL ? 5 : 3;
+  static constexpr int kVecs = RULE == kGeneral ? 5 : RULE == kHead ? 2 : 3;
+  static constexpr int kKey = RULE == kHead ? 0 : DP, kRead = kKey + DP;    // places of k and q
   static constexpr int kToken = kVecs * DP + kCols + 4;
   static constexpr int kChunk = 8;                    // tokens per chunk
   static constexpr int kFloats = kChunk * kToken;
@@ -329,22 +347,30 @@ struct Stage {
 // Asynchronous copies of tokens' vectors by the copying threads.  Widths that are multiples of
 // four move as 16-byte pieces: a thread owns the same pieces of every token and only advances its
 // pointers (address arithmetic per piece would cost as much as the recurrence).
-template <int DP, bool GENERAL>
+template <int DP, int RULE>
 struct Copier {
-  using St = Stage<DP, GENERAL>;
+  using St = Stage<DP, RULE>;
   static constexpr int kQ = DP / 4;
   static constexpr int kPieces = St::kVecs * kQ + kCols / 4;
   static constexpr int kMine = (kPieces + kRuleCopy - 1) / kRuleCopy;
   const float* src[kMine];
   int step[kMine], dst[kMine];          // floats per token, place in the token (-1: nothing)
-  const float* beta;
+  const float *beta, *decay;
   int tid, heads;
   bool quad;
+  static __device__ __forceinline__ bool shared_vec(int vec) {      // one per key head
+    return RULE == kHead || vec == 1 || vec == 2;
+  }
+  static __device__ __forceinline__ const float* source(const RuleArgs& a, int vec) {
+    if (RULE == kHead) return vec == 0 ? a.k : a.q;
+    return vec == 1 ? a.k : vec == 2 ? a.q : vec == 0 ? a.g : vec == 3 ? a.n : a.p;
+  }
   __device__ __forceinline__ void init(const RuleArgs& a, int tid_, long long row0, int h, int hk, int col0) {
     tid = tid_;
     heads = a.H;
     quad = (a.V & 3) == 0 && (a.D & 3) == 0;
-    beta = GENERAL ? nullptr : a.beta + row0 * a.H + h;
+    beta = RULE == kGeneral ? nullptr : a.beta + row0 * a.H + h;
+    decay = RULE == kHead ? a.g + row0 * a.H + h : nullptr;
 #pragma unroll
     for (int i = 0; i < kMine; ++i) {
       const int e = tid + i * kRuleCopy, vec = e / kQ, d = (e - vec * kQ) * 4;
@@ -353,10 +379,9 @@ struct Copier {
       step[i] = 0;
       if (e < St::kVecs * kQ) {
         if (d >= a.D) continue;
-        const bool shared = vec == 1 || vec == 2;
+        const bool shared = shared_vec(vec);
         const int heads_ = shared ? a.Hk : a.H, hh = shared ? hk : h;
-        src[i] = (vec == 1 ? a.k : vec == 2 ? a.q : vec == 0 ? a.g : vec == 3 ? a.n : a.p) +
-                 (row0 * heads_ + hh) * a.D + d;
+        src[i] = source(a, vec) + (row0 * heads_ + hh) * a.D + d;
         step[i] = heads_ * a.D;
         dst[i] = vec * DP + d;
       } else if (e < kPieces) {
@@ -379,9 +404,13 @@ struct Copier {
             cp_async<16>(buf + dst[i], src[i]);
             src[i] += step[i];
           }
-        if (!GENERAL && tid == 0) {
+        if (RULE != kGeneral && tid == 0) {
           cp_async<4>(buf + St::kVecs * DP + kCols, beta);
           beta += heads;
+        }
+        if (RULE == kHead && tid == 1) {
+          cp_async<4>(buf + St::kVecs * DP + kCols + 1, decay);
+          decay += heads;
         }
       }
     } else {
@@ -389,22 +418,23 @@ struct Copier {
         const long long row = row0 + t;
         for (int e = tid; e < St::kVecs * a.D; e += kRuleCopy) {
           const int vec = e / a.D, d = e - vec * a.D;
-          const bool shared = vec == 1 || vec == 2;
-          const float* from = vec == 1 ? a.k : vec == 2 ? a.q : vec == 0 ? a.g : vec == 3 ? a.n : a.p;
-          cp_async<4>(buf + vec * DP + d, from + (shared ? row * a.Hk + hk : row * a.H + h) * a.D + d);
+          cp_async<4>(buf + vec * DP + d,
+                      source(a, vec) + (shared_vec(vec) ? row * a.Hk + hk : row * a.H + h) * a.D + d);
         }
         for (int c = tid; c < kCols && col0 + c < a.V; c += kRuleCopy)
           cp_async<4>(buf + St::kVecs * DP + c, a.v + (row * a.H + h) * a.V + col0 + c);
-        if (!GENERAL && tid == 0) cp_async<4>(buf + St::kVecs * DP + kCols, a.beta + row * a.H + h);
+        if (RULE != kGeneral && tid == 0) cp_async<4>(buf + St::kVecs * DP + kCols, a.beta + row * a.H + h);
+        if (RULE == kHead && tid == 1) cp_async<4>(buf + St::kVecs * DP + kCols + 1, a.g + row * a.H + h);
       }
     }
   }
 };
 
-template <int DP, bool GENERAL>
+template <int DP, int RULE>
 __global__ void __launch_bounds__(kRuleThreads, DP > 128 ? 1 : 3) vector_delta_kernel(const RuleArgs a) {
   US_PDL_PROLOGUE();
-  using St = Stage<DP, GENERAL>;
+  using St = Stage<DP, RULE>;
+  constexpr bool GENERAL = RULE == kGeneral;
   constexpr int NG = DP / 32;                         // groups of four rows per lane
   extern __shared__ __align__(16) float sm[];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -426,7 +456,7 @@ __global__ void __launch_bounds__(kRuleThreads, DP > 128 ? 1 : 3) vector_delta_k
     __syncthreads();
   }
   if (tid >= kRuleCompute) {                          // the copying threads stay one chunk ahead
-    Copier<DP, GENERAL> cp;
+    Copier<DP, RULE> cp;
     cp.init(a, tid - kRuleCompute, start, h, hk, col0);
     const int chunks = (T + St::kChunk - 1) / St::kChunk;
     auto fetch = [&](int r) {                         // (an empty group past the end)
@@ -497,14 +527,16 @@ __global__ void __launch_bounds__(kRuleThreads, DP > 128 ? 1 : 3) vector_delta_k
         if (GENERAL) {
           lds_vec(m, base + 3 * DP + r0);
         } else {
-          f2 g[2];
-          lds_vec(m, base + DP + r0);
-          lds_vec(g, base + r0);
+          lds_vec(m, base + St::kKey + r0);
+          if (RULE == kChannel) {
+            f2 g[2];
+            lds_vec(g, base + r0);
 #pragma unroll
-          for (int e = 0; e < 2; ++e)
+            for (int e = 0; e < 2; ++e)
 #pragma unroll
-            for (int c = 0; c < 2; ++c)     // the key sees the decayed state
-              S[j * 2 + e][c] = mul2(S[j * 2 + e][c], g[e]);
+              for (int c = 0; c < 2; ++c)   // the key sees the decayed state
+                S[j * 2 + e][c] = mul2(S[j * 2 + e][c], g[e]);
+          }
         }
 #pragma unroll
         for (int e = 0; e < 2; ++e)
@@ -521,7 +553,8 @@ __global__ void __launch_bounds__(kRuleThreads, DP > 128 ? 1 : 3) vector_delta_k
       }
       pending = true;
       float c = seen;                               // general: n^T S of this lane's column
-      if (!GENERAL) c = vs[kCols] * (vs[cb + (up ? 1 : 0)] - seen);
+      const float dec = RULE == kHead ? vs[kCols + 1] : 1.f;
+      if (!GENERAL) c = vs[kCols] * (vs[cb + (up ? 1 : 0)] - (RULE == kHead ? dec * seen : seen));
       const float other = __shfl_xor_sync(0xffffffffu, c, 4);
       const float u0 = up ? other : c, u1 = up ? c : other;
       f2 uu[2], vv[2];
@@ -532,13 +565,14 @@ __global__ void __launch_bounds__(kRuleThreads, DP > 128 ? 1 : 3) vector_delta_k
       } else {
         uu[0] = pack2(u0, u0); uu[1] = pack2(u1, u1);
       }
+      const f2 dd = pack2(dec, dec);
       f2 oo[2][2] = {{0ull, 0ull}, {0ull, 0ull}};
 #pragma unroll
       for (int j = 0; j < NG; ++j) {
         const int r0 = (j * 8 + kq) * 4;
         f2 k[2], q[2], g[2], p[2];
-        lds_vec(k, base + DP + r0);
-        lds_vec(q, base + 2 * DP + r0);
+        lds_vec(k, base + St::kKey + r0);
+        lds_vec(q, base + St::kRead + r0);
         if (GENERAL) {
           lds_vec(g, base + r0);
           lds_vec(p, base + 4 * DP + r0);
@@ -549,6 +583,7 @@ __global__ void __launch_bounds__(kRuleThreads, DP > 128 ? 1 : 3) vector_delta_k
           for (int c = 0; c < 2; ++c) {
             f2& x = S[j * 2 + e][c];
             if (GENERAL) x = fma2(k[e], vv[c], fma2(p[e], uu[c], mul2(g[e], x)));
+            else if (RULE == kHead) x = fma2(k[e], uu[c], mul2(dd, x));
             else x = fma2(k[e], uu[c], x);
             oo[c][e] = fma2(x, q[e], oo[c][e]);
           }
@@ -579,12 +614,13 @@ __global__ void __launch_bounds__(kRuleThreads, DP > 128 ? 1 : 3) vector_delta_k
     }
 }
 
-// y = o / rms(o over V) * w * sigmoid(gate), one warp per (row, head); columns past H * V of
+// y = o / rms(o over V) * w * sigmoid(gate) (or silu), one warp per (row, head); columns past H * V of
 // the (padded) output row are zeroed by the last head's warp.
 __global__ void __launch_bounds__(256)
 head_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ w, int w_head_stride,
                       const void* __restrict__ gate, long long ldg, void* __restrict__ y,
-                      long long ldy, int rows, int H, int V, float eps, int bf16, int gate_bf16) {
+                      long long ldy, int rows, int H, int V, float eps, int bf16, int gate_bf16,
+                      int silu) {
   US_PDL_PROLOGUE();
   const long long r = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
@@ -597,7 +633,7 @@ head_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ w, 
   for (int c = lane; c < V; c += 32) {
     const float gv = ld_any(gate, (long long)t * ldg + h * V + c, gate_bf16);
     st_any(y, (long long)t * ldy + h * V + c, bf16,
-           x[c] * inv * w[h * w_head_stride + c] * sigmoid_f(gv));
+           x[c] * inv * w[h * w_head_stride + c] * gate_f(gv, silu));
   }
   if (h == H - 1)
     for (long long c = (long long)H * V + lane; c < ldy; c += 32)
@@ -612,7 +648,8 @@ struct StepArgs {
   const float *cq, *ck, *cv;      // channel: taps
   const float* low;               // [B, H * D]
   long long ldlow;
-  const float *A_log, *bias;      // channel: [H], dt_bias [H * D]; general: null, w0 [H * D]
+  int off_a;                      // head: column of the decay's argument
+  const float *A_log, *bias;      // channel: [H], dt_bias [H * D]; head: [H] x 2; general: null, w0 [H * D]
   const float* a_bias;            // general: [H * D]
   void* conv;                     // channel: ring [slots, K, C]
   float* state;                   // [slots, H, D, V]
@@ -623,7 +660,7 @@ struct StepArgs {
   void* y;                        // [B, ldy]
   long long ldy;
   const int *slots, *pos;
-  int H, Hk, D, V, K, bf16, gate_bf16;
+  int H, Hk, D, V, K, bf16, gate_bf16, silu;
   float eps, rate;
 };
 
@@ -634,13 +671,16 @@ constexpr int kStepThreads = 256;
 // owns one head of one sequence.  A thread holds R rows x 4 columns of S, a warp reading whole
 // rows; the state is on its way while the vectors are formed in shared memory.  LQ threads span
 // the value columns.  Sums over key channels meet in shared memory.
-template <int R, int LQ, bool GENERAL>
+template <int R, int LQ, int RULE>
 __global__ void __launch_bounds__(kStepThreads) vector_delta_step_kernel(const StepArgs a) {
   US_PDL_PROLOGUE();
+  constexpr bool GENERAL = RULE == kGeneral;
+  constexpr int kVecs = RULE == kHead ? 2 : 3;        // vectors of D formed before v
   constexpr int RG = kStepThreads / LQ;               // row groups
-  __shared__ float qs[kMaxDim], ks[kMaxDim], gs[kMaxDim], ps[GENERAL ? kMaxDim : 1], vs[LQ * 4];
+  __shared__ float qs[kMaxDim], ks[kMaxDim], gs[RULE == kHead ? 1 : kMaxDim], ps[GENERAL ? kMaxDim : 1],
+      vs[LQ * 4];
   __shared__ __align__(16) float red[RG][LQ * 4];
-  __shared__ float scal[4];
+  __shared__ float scal[5];                           // 1 / |q|, 1 / |k|, beta, (norm's second part), decay
   const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int slot = a.slots[b], H = a.H, D = a.D, V = a.V;
   if (slot < 0) {
@@ -660,10 +700,10 @@ __global__ void __launch_bounds__(kStepThreads) vector_delta_step_kernel(const S
   const long long xb = b * a.ldx;
   const int hk = h / (H / a.Hk);
   // ---- vectors ----
-  for (int e = tid; e < 3 * D + V; e += kStepThreads) {
-    const int what = e < D ? 0 : e < 2 * D ? 1 : e < 3 * D ? 2 : 3;       // q, k, decay, v
-    const int d = e - what * D;
-    if (what == 2) {
+  for (int e = tid; e < kVecs * D + V; e += kStepThreads) {
+    const int what = e < D ? 0 : e < 2 * D ? 1 : e < kVecs * D ? 2 : 3;   // q, k, decay, v
+    const int d = e - (what == 3 ? kVecs : what) * D;
+    if (RULE != kHead && what == 2) {
       const float lo = a.low[b * a.ldlow + h * D + d] + a.bias[h * D + d];
       if (GENERAL) {
         gs[d] = decay_exp(-a.rate * sigmoid_f(lo));
@@ -705,6 +745,8 @@ __global__ void __launch_bounds__(kStepThreads) vector_delta_step_kernel(const S
     if (lane == 0) scal[warp] = 1.f / sqrtf(ss + 1e-6f);
   } else if (!GENERAL && tid == 64) {
     scal[2] = sigmoid_f(ld_any(a.x, xb + a.off_b + h, a.bf16));
+    if (RULE == kHead)
+      scal[4] = decay_exp(-expf(a.A_log[h]) * softplus_f(ld_any(a.x, xb + a.off_a + h, a.bf16) + a.bias[h]));
   }
   __syncthreads();
   const float kinv = scal[1];
@@ -716,7 +758,7 @@ __global__ void __launch_bounds__(kStepThreads) vector_delta_step_kernel(const S
     if (row >= D) break;
     const float k = ks[row] * kinv;
     if (!GENERAL) {
-      const float g = gs[row];
+      const float g = RULE == kHead ? scal[4] : gs[row];
       S[i].x *= g; S[i].y *= g; S[i].z *= g; S[i].w *= g;
     }
     acc.x = fmaf(S[i].x, k, acc.x); acc.y = fmaf(S[i].y, k, acc.y);
@@ -781,43 +823,66 @@ __global__ void __launch_bounds__(kStepThreads) vector_delta_step_kernel(const S
   for (int i = 0; i < 4; ++i) {
     const int c = h * V + cq4 + i;
     st_any(a.y, b * a.ldy + c, a.bf16,
-           r[i] * inv * a.nw[h * a.nw_head_stride + cq4 + i] * sigmoid_f(ld_any(a.gate, b * a.ldg + c, a.gate_bf16)));
+           r[i] * inv * a.nw[h * a.nw_head_stride + cq4 + i] * gate_f(ld_any(a.gate, b * a.ldg + c, a.gate_bf16), a.silu));
   }
 }
 
-template <int LQ, bool GENERAL>
+template <int LQ, int RULE>
 int launch_step(const StepArgs& a, int B, cudaStream_t stream) {
   const int rows = (a.D + kStepThreads / LQ - 1) / (kStepThreads / LQ);
   const dim3 grid(a.H, B), block(kStepThreads);
-  if (rows <= 4) US_CUDA_CHECK(us::launch_pdl(vector_delta_step_kernel<4, LQ, GENERAL>, grid, block, 0, stream, a));
-  else if (rows <= 8) US_CUDA_CHECK(us::launch_pdl(vector_delta_step_kernel<8, LQ, GENERAL>, grid, block, 0, stream, a));
-  else if (rows <= 16) US_CUDA_CHECK(us::launch_pdl(vector_delta_step_kernel<16, LQ, GENERAL>, grid, block, 0, stream, a));
+  if (rows <= 4) US_CUDA_CHECK(us::launch_pdl(vector_delta_step_kernel<4, LQ, RULE>, grid, block, 0, stream, a));
+  else if (rows <= 8) US_CUDA_CHECK(us::launch_pdl(vector_delta_step_kernel<8, LQ, RULE>, grid, block, 0, stream, a));
+  else if (rows <= 16) US_CUDA_CHECK(us::launch_pdl(vector_delta_step_kernel<16, LQ, RULE>, grid, block, 0, stream, a));
   else return US_ERR_UNSUPPORTED;
   return US_OK;
 }
 
-template <bool GENERAL>
+template <int RULE>
 int step_impl(const StepArgs& a, int B, cudaStream_t stream) {
-  US_REQUIRE(a.x && a.low && a.bias && a.state && a.nw && a.gate && a.y && a.slots && a.pos && B >= 1 &&
+  US_REQUIRE(a.x && (a.low || RULE == kHead) && a.bias && a.state && a.nw && a.gate && a.y && a.slots && a.pos && B >= 1 &&
              B <= 65535 && a.H >= 1 && a.ldy == (long long)a.H * a.V && ((uintptr_t)a.state % 16) == 0);
   if (a.D < 1 || a.D > kMaxDim || (a.V & 3) || a.V > 256) return US_ERR_UNSUPPORTED;
-  if (a.V <= 64) return launch_step<16, GENERAL>(a, B, stream);
-  if (a.V <= 128) return launch_step<32, GENERAL>(a, B, stream);
-  return launch_step<64, GENERAL>(a, B, stream);
+  if (a.V <= 64) return launch_step<16, RULE>(a, B, stream);
+  if (a.V <= 128) return launch_step<32, RULE>(a, B, stream);
+  return launch_step<64, RULE>(a, B, stream);
 }
 
-template <int DP, bool GENERAL>
+template <int DP, int RULE>
 int launch_rule(const RuleArgs& a, int B, cudaStream_t stream) {
-  constexpr size_t smem = kRuleBufs * Stage<DP, GENERAL>::kFloats * sizeof(float);
+  constexpr size_t smem = kRuleBufs * Stage<DP, RULE>::kFloats * sizeof(float);
   static bool configured = false;
   if (!configured && smem > 48 * 1024) {
-    US_CUDA_CHECK(cudaFuncSetAttribute(vector_delta_kernel<DP, GENERAL>,
+    US_CUDA_CHECK(cudaFuncSetAttribute(vector_delta_kernel<DP, RULE>,
                                        cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
   }
   configured = true;
-  US_CUDA_CHECK(us::launch_pdl(vector_delta_kernel<DP, GENERAL>,
+  US_CUDA_CHECK(us::launch_pdl(vector_delta_kernel<DP, RULE>,
                                dim3((a.V + kCols - 1) / kCols, a.H, B), dim3(kRuleThreads), smem,
                                stream, a));
+  return US_OK;
+}
+
+int prep_impl(const ChannelPrep& a, cudaStream_t stream) {
+  US_REQUIRE(a.x && a.cq && a.ck && a.cv && a.A_log && a.dt_bias && a.q && a.k && a.v && a.g && a.beta && a.cu &&
+             a.slots && a.pos && a.B >= 1 && a.rows >= 1 && a.H >= 1 && a.Hk >= 1 && a.H % a.Hk == 0);
+  US_REQUIRE(a.K == 1 || a.conv);
+  US_REQUIRE(!a.one_token || a.rows == a.B);
+  if (a.K < 1 || a.K > kMaxTaps || a.D < 1 || a.D > kMaxDim || a.V < 1 || a.V > kMaxDim)
+    return US_ERR_UNSUPPORTED;
+  const int per = a.one_token ? 1 : kPrepTokens;
+  const int units = 2 * a.Hk + 2 * a.H;
+  const dim3 grid((a.rows + per - 1) / per, (units + 7) / 8);
+  const int widest = a.D > a.V ? a.D : a.V;
+#define US_PREP(KT)                                                                               \
+  if (widest <= 64) US_CUDA_CHECK(us::launch_pdl(channel_prep_kernel<KT, 2>, grid, dim3(256), 0, stream, a));       \
+  else if (widest <= 128) US_CUDA_CHECK(us::launch_pdl(channel_prep_kernel<KT, 4>, grid, dim3(256), 0, stream, a)); \
+  else US_CUDA_CHECK(us::launch_pdl(channel_prep_kernel<KT, 8>, grid, dim3(256), 0, stream, a));
+  if (a.K <= 4) { US_PREP(4) } else if (a.K <= 8) { US_PREP(8) } else { US_PREP(16) }
+#undef US_PREP
+  if (!a.one_token && a.K > 1)
+    US_CUDA_CHECK(us::launch_pdl(conv_ring_kernel, dim3((2 * a.Hk * a.D + a.H * a.V + 255) / 256, a.B),
+                                 dim3(256), 0, stream, a));
   return US_OK;
 }
 
@@ -832,29 +897,23 @@ US_API int us_channel_delta_prep(const void* x, long long ldx, int off_q, int of
                                  float* g, float* beta, const int* cu, const int* slots,
                                  const int* pos, int B, int rows, int H, int Hk, int D, int V, int K,
                                  int bf16, int one_token, void* stream_) {
-  US_REQUIRE(x && cq && ck && cv && low && A_log && dt_bias && q && k && v && g && beta && cu &&
-             slots && pos && B >= 1 && rows >= 1 && H >= 1 && Hk >= 1 && H % Hk == 0);
-  US_REQUIRE(K == 1 || conv);
-  US_REQUIRE(!one_token || rows == B);
-  if (K < 1 || K > kMaxTaps || D < 1 || D > kMaxDim || V < 1 || V > kMaxDim)
-    return US_ERR_UNSUPPORTED;
-  ChannelPrep a{x, ldx, off_q, off_k, off_v, off_b, cq, ck, cv, low, ldlow, A_log, dt_bias, conv,
+  US_REQUIRE(low);
+  ChannelPrep a{x, ldx, off_q, off_k, off_v, off_b, cq, ck, cv, low, ldlow, 0, A_log, dt_bias, conv,
                 q, k, v, g, beta, cu, slots, pos, B, rows, H, Hk, D, V, K, bf16, one_token};
-  cudaStream_t stream = (cudaStream_t)stream_;
-  const int per = one_token ? 1 : kPrepTokens;
-  const int units = 2 * Hk + 2 * H;
-  const dim3 grid((rows + per - 1) / per, (units + 7) / 8);
-  const int widest = D > V ? D : V;
-#define US_PREP(KT)                                                                               \
-  if (widest <= 64) US_CUDA_CHECK(us::launch_pdl(channel_prep_kernel<KT, 2>, grid, dim3(256), 0, stream, a));       \
-  else if (widest <= 128) US_CUDA_CHECK(us::launch_pdl(channel_prep_kernel<KT, 4>, grid, dim3(256), 0, stream, a)); \
-  else US_CUDA_CHECK(us::launch_pdl(channel_prep_kernel<KT, 8>, grid, dim3(256), 0, stream, a));
-  if (K <= 4) { US_PREP(4) } else if (K <= 8) { US_PREP(8) } else { US_PREP(16) }
-#undef US_PREP
-  if (!one_token && K > 1)
-    US_CUDA_CHECK(us::launch_pdl(conv_ring_kernel, dim3((2 * Hk * D + H * V + 255) / 256, B),
-                                 dim3(256), 0, stream, a));
-  return US_OK;
+  return prep_impl(a, (cudaStream_t)stream_);
+}
+
+// The same for a decay per head: its argument stands at column off_a + h of the projection rows,
+// dt_bias is [H] and g [rows, H].
+US_API int us_head_delta_prep(const void* x, long long ldx, int off_q, int off_k, int off_v, int off_b,
+                              int off_a, const float* cq, const float* ck, const float* cv,
+                              const float* A_log, const float* dt_bias, void* conv, float* q, float* k,
+                              float* v, float* g, float* beta, const int* cu, const int* slots,
+                              const int* pos, int B, int rows, int H, int Hk, int D, int V, int K,
+                              int bf16, int one_token, void* stream_) {
+  ChannelPrep a{x, ldx, off_q, off_k, off_v, off_b, cq, ck, cv, nullptr, 0, off_a, A_log, dt_bias, conv,
+                q, k, v, g, beta, cu, slots, pos, B, rows, H, Hk, D, V, K, bf16, one_token};
+  return prep_impl(a, (cudaStream_t)stream_);
 }
 
 // out: six [rows, H, D] arrays one behind another: decay, unit key, removal, key, read-out, value.
@@ -872,21 +931,23 @@ US_API int us_general_delta_prep(const void* x, long long ldx, int off_r, int of
   return US_OK;
 }
 
-// general = 0: the channel rule (g, beta); 1: the general rule (g, n, p).  q and k heads serve
-// H / Hk value heads each; all vectors dense FP32.
-US_API int us_vector_delta_rule(int general, const float* q, const float* k, const float* v,
+// rule = 0: the channel rule (g, beta); 1: the general rule (g, n, p); 2: the head rule (g per head,
+// beta).  q and k heads serve H / Hk value heads each; all vectors dense FP32.
+US_API int us_vector_delta_rule(int rule, const float* q, const float* k, const float* v,
                                 const float* g, const float* n, const float* p, const float* beta,
                                 float* state, float* out, const int* cu, const int* slots,
                                 const int* pos, int B, int H, int Hk, int D, int V, void* stream_) {
   US_REQUIRE(q && k && v && g && state && out && cu && slots && pos && B >= 1 && B <= 65535);
-  US_REQUIRE(general ? (n && p) : (beta != nullptr));
+  US_REQUIRE(rule >= kChannel && rule <= kHead && (rule == kGeneral ? (n && p) : (beta != nullptr)));
   US_REQUIRE(H >= 1 && Hk >= 1 && H % Hk == 0 && H <= 65535 && D >= 1 && V >= 1);
-  US_REQUIRE((D & 3) || (V & 3) || (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)g | (uintptr_t)n |
-               (uintptr_t)p | (uintptr_t)state) % 16) == 0);
+  US_REQUIRE((D & 3) || (V & 3) || (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (rule == kHead ? 0 : (uintptr_t)g) |
+               (uintptr_t)n | (uintptr_t)p | (uintptr_t)state) % 16) == 0);
   RuleArgs a{q, k, v, g, n, p, beta, state, out, cu, slots, pos, H, Hk, D, V};
   cudaStream_t stream = (cudaStream_t)stream_;
 #define US_VD(DP) \
-  if (D <= DP) return general ? launch_rule<DP, true>(a, B, stream) : launch_rule<DP, false>(a, B, stream);
+  if (D <= DP) return rule == kGeneral ? launch_rule<DP, kGeneral>(a, B, stream)                       \
+                      : rule == kHead  ? launch_rule<DP, kHead>(a, B, stream)                          \
+                                       : launch_rule<DP, kChannel>(a, B, stream);
   US_VD(32) US_VD(64) US_VD(128) US_VD(256)
 #undef US_VD
   return US_ERR_UNSUPPORTED;
@@ -894,12 +955,12 @@ US_API int us_vector_delta_rule(int general, const float* q, const float* k, con
 
 US_API int us_head_norm_gate(const float* o, const float* w, int w_head_stride, const void* gate,
                              long long ldg, void* y, long long ldy, int rows, int H, int V,
-                             float eps, int bf16, int gate_bf16, void* stream_) {
+                             float eps, int bf16, int gate_bf16, int silu, void* stream_) {
   US_REQUIRE(o && w && gate && y && rows >= 1 && H >= 1 && V >= 1 && ldy >= (long long)H * V);
   const long long warps = (long long)rows * H;
   US_CUDA_CHECK(us::launch_pdl(head_norm_gate_kernel, dim3((unsigned)((warps + 7) / 8)), dim3(256),
                                0, (cudaStream_t)stream_, o, w, w_head_stride, gate, ldg, y, ldy, rows,
-                               H, V, eps, bf16, gate_bf16));
+                               H, V, eps, bf16, gate_bf16, silu));
   return US_OK;
 }
 
@@ -916,10 +977,26 @@ US_API int us_channel_delta_step(const void* x, long long ldx, int off_q, int of
                                  void* stream_) {
   US_REQUIRE(cq && ck && cv && A_log && Hk >= 1 && H % Hk == 0 && K >= 1 && (K == 1 || conv));
   if (K > kMaxTaps) return US_ERR_UNSUPPORTED;
-  StepArgs a{x, ldx, off_q, off_k, off_v, off_b, cq, ck, cv, low, ldlow, A_log, dt_bias, nullptr, conv,
+  StepArgs a{x, ldx, off_q, off_k, off_v, off_b, cq, ck, cv, low, ldlow, 0, A_log, dt_bias, nullptr, conv,
              state, nw, nw_head_stride, gate, ldg, y, ldy, slots, pos, H, Hk, D, V, K, bf16, gate_bf16,
-             eps, 0.f};
-  return step_impl<false>(a, B, (cudaStream_t)stream_);
+             0, eps, 0.f};
+  return step_impl<kChannel>(a, B, (cudaStream_t)stream_);
+}
+
+// silu: the gate's activation (0: sigmoid).
+US_API int us_head_delta_step(const void* x, long long ldx, int off_q, int off_k, int off_v, int off_b,
+                              int off_a, const float* cq, const float* ck, const float* cv,
+                              const float* A_log, const float* dt_bias, void* conv, float* state,
+                              const float* nw, int nw_head_stride, const void* gate, long long ldg,
+                              void* y, long long ldy, const int* slots, const int* pos, int B, int H,
+                              int Hk, int D, int V, int K, float eps, int bf16, int gate_bf16, int silu,
+                              void* stream_) {
+  US_REQUIRE(cq && ck && cv && A_log && Hk >= 1 && H % Hk == 0 && K >= 1 && (K == 1 || conv));
+  if (K > kMaxTaps) return US_ERR_UNSUPPORTED;
+  StepArgs a{x, ldx, off_q, off_k, off_v, off_b, cq, ck, cv, nullptr, 0, off_a, A_log, dt_bias, nullptr, conv,
+             state, nw, nw_head_stride, gate, ldg, y, ldy, slots, pos, H, Hk, D, V, K, bf16, gate_bf16,
+             silu, eps, 0.f};
+  return step_impl<kHead>(a, B, (cudaStream_t)stream_);
 }
 
 US_API int us_general_delta_step(const void* x, long long ldx, int off_r, int off_k, int off_v,
@@ -929,8 +1006,8 @@ US_API int us_general_delta_step(const void* x, long long ldx, int off_r, int of
                                  long long ldy, const int* slots, const int* pos, int B, int H, int D,
                                  float rate, float eps, int bf16, int gate_bf16, void* stream_) {
   US_REQUIRE(a_bias);
-  StepArgs a{x, ldx, off_r, off_k, off_v, off_a, nullptr, nullptr, nullptr, low, ldlow, nullptr, w0,
+  StepArgs a{x, ldx, off_r, off_k, off_v, off_a, nullptr, nullptr, nullptr, low, ldlow, 0, nullptr, w0,
              a_bias, nullptr, state, nw, nw_head_stride, gate, ldg, y, ldy, slots, pos, H, H, D, D, 1,
-             bf16, gate_bf16, eps, rate};
-  return step_impl<true>(a, B, (cudaStream_t)stream_);
+             bf16, gate_bf16, 0, eps, rate};
+  return step_impl<kGeneral>(a, B, (cudaStream_t)stream_);
 }

@@ -86,9 +86,11 @@ class LayeredDecoder:
         return F.linear(hidden_rows, self.lm_head, out_dtype=torch.float32)
 
     def weight_bytes(self) -> int:
-        seen = {}
-        for w in [vars(self)] + self.layers:
-            for t in w.values():
+        seen, todo = {}, [vars(self)] + self.layers
+        while todo:
+            for t in todo.pop().values():
                 if torch.is_tensor(t):
                     seen[(t.data_ptr(), t.numel())] = t.numel() * t.element_size()
+                elif isinstance(t, dict):
+                    todo.append(t)
         return sum(seen.values())

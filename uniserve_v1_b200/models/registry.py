@@ -67,12 +67,31 @@ def _zonopel_model(cfg, device, dtype, ctx=None):
     return ZonopelModel(cfg, device, dtype)
 
 
+def _tadinex_config(d):
+    from .tadinex import TadinexConfig
+    return TadinexConfig.from_json(d)
+
+
+def _tadinex_named(name):
+    from .tadinex import TadinexConfig
+    return TadinexConfig.tiny() if name == "tiny" else TadinexConfig.bench()
+
+
+def _tadinex_model(cfg, device, dtype, ctx=None):
+    from .tadinex import TadinexModel
+    if ctx is not None and ctx.world_size > 1:
+        raise ValueError("this family is served on one GPU")
+    return TadinexModel(cfg, device, dtype)
+
+
 PAGED_DECODERS = {
     "qwen3_moe": PagedDecoder(_qwen3_config, _qwen3_named, _qwen3_model, (torch.bfloat16,)),
     "nepevik": PagedDecoder(_nepevik_config, _nepevik_named, _nepevik_model,
                             (torch.bfloat16, torch.float32), "nepevik"),
     "zonopel": PagedDecoder(_zonopel_config, _zonopel_named, _zonopel_model,
                             (torch.bfloat16, torch.float32), "zonopel"),
+    "tadinex": PagedDecoder(_tadinex_config, _tadinex_named, _tadinex_model,
+                            (torch.bfloat16, torch.float32), "tadinex"),
 }
 
 

@@ -359,6 +359,33 @@ def linear(x, w, bias=None, out_dtype=None, out=None, block_n=None, act=None):
 _ACT = {"silu": 0, "silu_stepwise": 1, "gelu_tanh": 2}
 
 
+def clamped_linear(x, w, limit, alpha, out=None, tiles=None, block_n=None, live=0):
+    """(clamp(first, -limit, limit) + 1) g sigmoid(alpha g) with g = min(second, limit), as [rows, I]: w
+    [2 * I, K] (or [E, 2 * I, K] with ``tiles``, an expert tile list) stacks the `first` rows, then the
+    `second` ones.  bf16: in the product's epilogue."""
+    if not _cuda(x):
+        return R.clamped_linear(x, w, limit, alpha)
+    rows, K = x.shape
+    I2 = w.shape[-2]
+    I_, E = I2 // 2, w.shape[0] if w.dim() == 3 else 1
+    if out is None:
+        out = torch.empty(rows, I_, dtype=x.dtype, device=x.device)
+    if rows == 0:
+        return out
+    tile_args = tiles or (None, None, None, None, 0)
+    if x.dtype == torch.float32:
+        z = torch.empty(rows, I2, dtype=torch.float32, device=x.device)
+        N.call("us_gemm_f32", N.ptr(w), N.ptr(x), N.ptr(z), E, I2, I2, K, rows, K, x.stride(0), I2, 0, None,
+               *tile_args, N.stream())
+        N.call("us_clamped_glu_f32", N.ptr(z), N.ptr(out), rows, I_, limit, alpha, N.stream())
+        return out
+    if live:
+        N.kernels().us_gemm_wx_hint(live * ((I_ + 127) // 128))
+    N.call("us_gemm_wx_clamped", N.ptr(w), N.ptr(x), N.ptr(out), E, I2, I_, K, rows, K, x.stride(0), I_, I_,
+           limit, alpha, *tile_args, block_n or _block_n(rows, True), N.stream())
+    return out
+
+
 def linear_gated(x, w, act="silu", stepwise=False, out=None, block_n=None):
     """w [2*I, K] stacks the `first` rows then the `second` (gate) rows;
     returns first * act(second) as [rows, I] bf16, fused in the GEMM epilogue."""
@@ -391,7 +418,7 @@ def topk_softmax(logits, top_k, renorm=True, live=None, expert_map=None, load=No
         ids = torch.empty(T, top_k, dtype=torch.int32, device=logits.device)
         weights = torch.empty(T, top_k, dtype=torch.float32, device=logits.device)
     N.call("us_topk_softmax", N.ptr(logits), N.ptr(ids), N.ptr(weights), T, E, top_k,
-           int(renorm), N.ptr(live), N.ptr(expert_map), N.ptr(load), N.stream())
+           int(renorm), N.ptr(live), N.ptr(expert_map), N.ptr(load), None, N.stream())
     return ids, weights
 
 
@@ -460,7 +487,7 @@ def route_and_sort(logits, top_k, renorm, ws, e_lo, E_local):
     N.call("us_route_sort", N.ptr(logits), N.ptr(ids), N.ptr(weights), T, E_all, top_k,
            int(renorm), None, e_lo, E_local, ws.block_n, ws.max_tiles, N.ptr(ws.sorted_route),
            N.ptr(ws.perm_of_route), N.ptr(ws.expert_offsets), N.ptr(ws.tile_group),
-           N.ptr(ws.tile_row0), N.ptr(ws.tile_rows), N.ptr(ws.num_tiles), N.stream())
+           N.ptr(ws.tile_row0), N.ptr(ws.tile_rows), N.ptr(ws.num_tiles), None, N.stream())
     return ids, weights
 
 
@@ -474,7 +501,7 @@ def route_sort_gather(logits, x, top_k, renorm, ws, e_lo, E_local, live=None):
            int(renorm), N.ptr(live), e_lo, E_local, ws.block_n, ws.max_tiles,
            N.ptr(ws.sorted_route), N.ptr(ws.perm_of_route), N.ptr(ws.expert_offsets),
            N.ptr(ws.tile_group), N.ptr(ws.tile_row0), N.ptr(ws.tile_rows), N.ptr(ws.num_tiles),
-           N.ptr(x), x.shape[1], N.ptr(ws.xp), N.ptr(ws.sync), N.stream())
+           N.ptr(x), x.shape[1], N.ptr(ws.xp), N.ptr(ws.sync), None, N.stream())
     return ids, weights
 
 
@@ -543,8 +570,8 @@ def moe_experts(x, ids, weights, w13, w2, e_lo=0, act="silu", stepwise=False, ws
 
 
 @dataclass
-class TableRoutes:
-    """Routes of one layer chosen by token id: the sorted route list and the expert tile list."""
+class Routes:
+    """Routes of one layer: the sorted route list and the expert tile list."""
     ids: torch.Tensor             # [T, top] expert of every route
     sorted_route: torch.Tensor
     perm: torch.Tensor            # [T, top] permuted row of every route
@@ -556,22 +583,63 @@ class TableRoutes:
     block_n: int
     max_tiles: int
     live_tiles: int
+    weights: Optional[torch.Tensor] = None      # [T, top] FP32 (routes chosen by scores)
+    xp: Optional[torch.Tensor] = None           # the routed rows in sorted order, once gathered
+
+    @property
+    def tiles(self):
+        return (N.ptr(self.tile_group), N.ptr(self.tile_row0), N.ptr(self.tile_rows),
+                N.ptr(self.num_tiles), self.max_tiles)
+
+
+def _route_tiles(R_, E, E_total):
+    """(rows per tile, most tiles, expected live tiles) of R_ routes over E_total experts, E of them here."""
+    avg = max(1, R_ // E_total)
+    block_n = 16 if avg <= 16 else 32 if avg <= 32 else 64 if avg <= 64 else 128
+    if avg >= MOE_PAIR_MIN_ROWS:
+        block_n = 256
+    return block_n, min(R_, E) + R_ // block_n + 1, MoeWorkspace._expected_tiles(R_, E, E_total, block_n)
+
+
+def scored_routes(logits, correction, top, E, x, sync):
+    """Softmax scores over all experts, the ``top`` of score + ``correction`` chosen, weighted by their
+    scores over the scores' sum.  ``logits`` [T, n] FP32; experts at or past ``E`` have no tensors: their
+    routes are not sorted and stand as negative rows in ``perm``.  ``sync``: four int32 zeros that calls of
+    one stream share.  Up to 512 rows of ``x`` are routed, sorted and gathered in one launch."""
+    if not _cuda(logits):
+        return R.scored_routes(logits, correction, top, E)
+    T, E_all = logits.shape
+    dev, st = logits.device, N.stream()
+    assert logits.dtype == torch.float32 and logits.is_contiguous()
+    R_ = T * top
+    block_n, max_tiles, live = _route_tiles(R_, E, E_all)
+    buf = torch.empty(3 * R_ + E + 1 + 3 * max_tiles + 1, dtype=torch.int32, device=dev)
+    ids, srt, perm, offs, tg, t0, tr, nt = buf.split([R_, R_, R_, E + 1, max_tiles, max_tiles, max_tiles, 1])
+    weights = torch.empty(T, top, dtype=torch.float32, device=dev)
+    r = Routes(ids.view(T, top), srt, perm.view(T, top), offs, tg, t0, tr, nt, block_n, max_tiles, live, weights)
+    sort = (E, block_n, max_tiles, N.ptr(srt), N.ptr(perm), N.ptr(offs), N.ptr(tg), N.ptr(t0), N.ptr(tr), N.ptr(nt))
+    if T <= 512:
+        r.xp = torch.empty(R_, x.shape[1], dtype=x.dtype, device=dev)
+        wide = 1 if x.dtype == BF16 else 2          # the gather moves 16-bit units
+        N.call("us_route_sort_gather", N.ptr(logits), N.ptr(ids), N.ptr(weights), T, E_all, top, 1, None, 0, *sort,
+               N.ptr(x), x.shape[1] * wide, N.ptr(r.xp), N.ptr(sync), N.ptr(correction), st)
+    else:
+        N.call("us_topk_softmax", N.ptr(logits), N.ptr(ids), N.ptr(weights), T, E_all, top, 1, None, None, None,
+               N.ptr(correction), st)
+        N.call("us_moe_sort", N.ptr(ids), R_, 0, *sort, st)
+    return r
 
 
 def table_routes(tokens, tables, E):
     """``tables`` [layers, vocab, top] (int32): the experts of every token id, layer by layer.
     Routes and their sort of all layers in one launch (they depend on the token ids only);
-    returns a ``TableRoutes`` per layer."""
+    returns a ``Routes`` per layer."""
     Ln, V, top = tables.shape
     T = tokens.shape[0]
     if not _cuda(tokens):
         return [R.table_routes(tokens, tables[i]) for i in range(Ln)]
     R_ = T * top
-    avg = max(1, R_ // E)
-    block_n = 16 if avg <= 16 else 32 if avg <= 32 else 64 if avg <= 64 else 128
-    if avg >= MOE_PAIR_MIN_ROWS:
-        block_n = 256
-    max_tiles = min(R_, E) + R_ // block_n + 1
+    block_n, max_tiles, live = _route_tiles(R_, E, E)
     widths = (R_, R_, R_, E + 1, max_tiles, max_tiles, max_tiles, 1)
     buf = torch.empty(Ln * sum(widths), dtype=torch.int32, device=tokens.device)
     parts, off = [], 0
@@ -580,32 +648,35 @@ def table_routes(tokens, tables, E):
         off += Ln * w
     N.call("us_table_route_sort", N.ptr(tokens), N.ptr(tables), Ln, T, top, V, E, block_n, max_tiles,
            *[N.ptr(p) for p in parts], N.stream())
-    live = MoeWorkspace._expected_tiles(R_, E, E, block_n)
-    return [TableRoutes(parts[0][i].view(T, top), parts[1][i], parts[2][i].view(T, top), parts[3][i],
-                        parts[4][i], parts[5][i], parts[6][i], parts[7][i], block_n, max_tiles, live)
+    return [Routes(parts[0][i].view(T, top), parts[1][i], parts[2][i].view(T, top), parts[3][i],
+                   parts[4][i], parts[5][i], parts[6][i], parts[7][i], block_n, max_tiles, live)
             for i in range(Ln)]
 
 
-def routed_mlp(x, routes, w_up, w_down, act="gelu_erf"):
-    """Ungated experts W_down act(W_up x) over sorted routes: gather, two grouped products with
-    the activation in the first one's epilogue.  w_up [E, I, H], w_down [E, H, I].  Returns the
-    expert rows in permuted order; ``routes.perm`` says where a token's are."""
+def routed_mlp(x, routes, w_up, w_down, act="gelu_erf", clamped=None):
+    """Experts W_down act(W_up x) over sorted routes: gather, two grouped products with the activation in
+    the first one's epilogue.  w_up [E, I, H], w_down [E, H, I]; with ``clamped`` = (limit, alpha) the
+    experts are gated (``clamped_linear``) and w_up is [E, 2 * I, H].  Returns the expert rows in permuted
+    order; ``routes.perm`` says where a token's are."""
     if not _cuda(x):
-        return R.routed_mlp(x, routes, w_up, w_down)
+        return R.routed_mlp(x, routes, w_up, w_down, clamped)
     T, H = x.shape
-    E, I_, _ = w_up.shape
+    E, _, I_ = w_down.shape
     top = routes.perm.shape[1]
     R_ = T * top
     dev, st, code = x.device, N.stream(), _ACT1[act]
-    xp = torch.empty(R_, H, dtype=x.dtype, device=dev)
+    xp = routes.xp
     h = torch.empty(R_, I_, dtype=x.dtype, device=dev)
     y = torch.empty(R_, H, dtype=x.dtype, device=dev)
     wide = 1 if x.dtype == BF16 else 2          # the gather moves 16-bit units
-    N.call("us_moe_gather", N.ptr(x), N.ptr(routes.sorted_route), N.ptr(routes.expert_offsets[E:]),
-           R_, top, H * wide, N.ptr(xp), st)
-    tiles = (N.ptr(routes.tile_group), N.ptr(routes.tile_row0), N.ptr(routes.tile_rows),
-             N.ptr(routes.num_tiles), routes.max_tiles)
-    for w, a, o, M, K, c in ((w_up, xp, h, I_, H, code), (w_down, h, y, H, I_, 0)):
+    if xp is None:
+        xp = torch.empty(R_, H, dtype=x.dtype, device=dev)
+        N.call("us_moe_gather", N.ptr(x), N.ptr(routes.sorted_route), N.ptr(routes.expert_offsets[E:]),
+               R_, top, H * wide, N.ptr(xp), st)
+    tiles = routes.tiles
+    if clamped:
+        clamped_linear(xp, w_up, *clamped, out=h, tiles=tiles, block_n=routes.block_n, live=routes.live_tiles)
+    for w, a, o, M, K, c in ((w_up, xp, h, I_, H, code), (w_down, h, y, H, I_, 0))[int(clamped is not None):]:
         if x.dtype == torch.float32:
             N.call("us_gemm_f32", N.ptr(w), N.ptr(a), N.ptr(o), E, M, M, K, R_, K, K, M, c, None,
                    *tiles, st)
@@ -676,6 +747,51 @@ def _stream_rows(embed, y, residual, w, nxt, eps, width, dtype, T, W):
            m.slots.shape[0] if shift else 1, T, W, width, int(dtype == BF16),
            int(shift and m.one_token), eps, N.stream())
     return res, x
+
+
+@dataclass
+class Mixture:
+    """A sublayer's output as a weighted sum of routed expert rows; routes without a row (experts without
+    tensors) take the sublayer's own input ``ident`` instead."""
+    rows: torch.Tensor                      # expert rows (``routed_mlp``)
+    routes: Routes
+    ident: Optional[torch.Tensor] = None
+    shared: Optional[torch.Tensor] = None   # added without a weight
+
+
+def _plain_rows(ids, table, scale, y, residual, gain, nxt, eps, width, dtype, T, W):
+    dev = nxt.weight.device
+    res = torch.empty(T, W, dtype=torch.float32, device=dev)
+    x = torch.empty(T, W, dtype=dtype, device=dev)
+    mix = y if isinstance(y, Mixture) else None
+    r = mix.routes if mix else None
+    N.call("us_plain_rows", N.ptr(ids), N.ptr(table), scale, table.shape[0] if table is not None else 0,
+           None if mix else N.ptr(y), N.ptr(mix.rows) if mix else None, N.ptr(r.perm) if mix else None,
+           N.ptr(r.weights) if mix else None, r.perm.shape[1] if mix else 0, N.ptr(mix.ident) if mix else None,
+           N.ptr(mix.shared) if mix else None, gain, N.ptr(residual), N.ptr(res), N.ptr(nxt.weight), N.ptr(x),
+           T, W, width, int(dtype == BF16), eps, N.stream())
+    return res, x
+
+
+def embed_plain_rows(ids, table, scale, nxt: NextRows, eps, width):
+    """Start of a stream without an embedding norm: table row * scale in FP32, and the next sublayer's
+    rows in the table's type."""
+    if not _cuda(table):
+        return R.plain_rows(table[ids.long()].float() * scale, None, 1.0, nxt, eps, width, table.dtype)
+    return _plain_rows(ids, table, scale, None, None, 1.0, nxt, eps, width, table.dtype, ids.shape[0], table.shape[1])
+
+
+def add_plain_rows(y, residual, gain, nxt: NextRows, eps, width):
+    """(residual + gain * y, the next sublayer's rows in y's type); ``y``: rows or a ``Mixture``.  The
+    residual handed in stays as it is."""
+    if isinstance(y, Mixture):
+        if not _cuda(y.rows):
+            return R.plain_rows(R.mixture(y), residual, gain, nxt, eps, width, y.rows.dtype)
+        return _plain_rows(None, None, 0.0, y, residual, gain, nxt, eps, width, y.rows.dtype, *residual.shape)
+    if not _cuda(y):
+        return R.plain_rows(y.float(), residual, gain, nxt, eps, width, y.dtype)
+    assert y.is_contiguous() and y.shape == residual.shape
+    return _plain_rows(None, None, 0.0, y, residual, gain, nxt, eps, width, y.dtype, *y.shape)
 
 
 def embed_norm_rows(ids, table, scale, w, nxt: NextRows, eps, width, second=None):

@@ -49,10 +49,17 @@ _SIGNATURES = {
                                   I, I, I, I, I, I, F, I, I, P]),
     "us_general_delta_step": (I, [P, L, I, I, I, I, P, L, P, P, P, P, I, P, L, P, L, P, P, I, I, I, F,
                                   F, I, I, P]),
-    "us_head_norm_gate": (I, [P, P, I, P, L, P, L, I, I, I, F, I, I, P]),
+    "us_head_delta_prep": (I, [P, L, I, I, I, I, I, P, P, P, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I,
+                               I, I, I, I, I, P]),
+    "us_head_delta_step": (I, [P, L, I, I, I, I, I, P, P, P, P, P, P, P, P, I, P, L, P, L, P, P, I, I, I,
+                               I, I, I, F, I, I, I, P]),
+    "us_head_norm_gate": (I, [P, P, I, P, L, P, L, I, I, I, F, I, I, I, P]),
     "us_embed_rows": (I, [P, P, P, P, I, I, I, I, P]),
     "us_output_norm_add": (I, [P, P, P, F, I, P, P, P, P, F, F, I, I, I, I, F, I, P]),
     "us_stream_rows": (I, [P, P, P, P, F, I, I, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, P]),
+    "us_plain_rows": (I, [P, P, F, I, P, P, P, P, I, P, P, F, P, P, P, P, I, I, I, I, F, P]),
+    "us_gemm_wx_clamped": (I, [P, P, P, I, I, I, I, I, L, L, L, I, F, F, P, P, P, P, I, I, P]),
+    "us_clamped_glu_f32": (I, [P, P, I, I, F, F, P]),
     "us_bigram_rows": (I, [P, P, P, P, P, P, I, I, I, L, L, I, P]),
     "us_poly_norm": (I, [P, L, P, P, L, I, I, I, F, I, P]),
     "us_row_norm_kv": (I, [P, L, I, I, I, I, I, I, P, P, P, P, P, I, F, I, P]),
@@ -89,10 +96,10 @@ _SIGNATURES = {
                                             L, L, P]),
     "us_unpermute_add_rmsnorm": (I, [P, P, P, I, I, I, P, P, P, F, I, P]),
     "us_route_sort_gather": (I, [P, P, P, I, I, I, I, P, I, I, I, I, P, P, P, P, P, P, P, P, I, P,
-                                 P, P]),
-    "us_topk_softmax": (I, [P, P, P, I, I, I, I, P, P, P, P]),
+                                 P, P, P]),
+    "us_topk_softmax": (I, [P, P, P, I, I, I, I, P, P, P, P, P]),
     "us_moe_sort": (I, [P, I, I, I, I, I, P, P, P, P, P, P, P, P]),
-    "us_route_sort": (I, [P, P, P, I, I, I, I, P, I, I, I, I, P, P, P, P, P, P, P, P]),
+    "us_route_sort": (I, [P, P, P, I, I, I, I, P, I, I, I, I, P, P, P, P, P, P, P, P, P]),
     "us_moe_gather": (I, [P, P, P, I, I, I, P, P]),
     "us_moe_unpermute": (I, [P, P, P, I, I, I, P, P]),
     "us_argmax": (I, [P, I, I, L, P, P]),

@@ -414,15 +414,63 @@ def table_routes(tokens, table):
     return table[tokens.long()].long()
 
 
-def routed_mlp(x, routes, w_up, w_down):
-    """Expert rows in route order (row t * top + k belongs to token t's k-th expert)."""
+def clamped_linear(x, w, limit, alpha):
+    """w stacks [first; second] rows: (clamp(first) + 1) g sigmoid(alpha g), g = min(second, limit)."""
+    z = x.float() @ w.float().t()
+    half = w.shape[0] // 2
+    g = z[:, half:].clamp(max=limit)
+    return ((z[:, :half].clamp(-limit, limit) + 1) * g * torch.sigmoid(alpha * g)).to(x.dtype)
+
+
+class ScoredRoutes:
+    """The CPU form of routes chosen by scores; experts at or past ``experts`` have no tensors."""
+
+    def __init__(self, ids, weights, experts):
+        self.ids, self.weights, self.experts = ids, weights, experts
+
+
+def scored_routes(logits, correction, top, experts):
+    s = logits.float().softmax(-1)
+    ids = torch.sort(s + correction, dim=-1, descending=True, stable=True).indices[:, :top]
+    w = s.gather(1, ids)
+    return ScoredRoutes(ids, w / (w.sum(-1, keepdim=True) + 1e-20), experts)
+
+
+def mixture(m):
+    """FP32 rows of an ``ops.functional.Mixture``; expert rows stand in route order."""
+    ids, w = m.routes.ids, m.routes.weights
+    T, top = ids.shape
+    y = m.rows.float().view(T, top, -1)
+    if m.ident is not None:         # rows of experts without tensors are zero
+        own = (ids >= m.routes.experts)[..., None]
+        y = torch.where(own, m.ident.float()[:, None], y)
+    y = (w[..., None] * y).sum(1)
+    return y if m.shared is None else y + m.shared.float()
+
+
+def plain_rows(source, residual, gain, nxt, eps, width, dtype):
+    """(residual + gain * source, its norm times the next weight in ``dtype``)."""
+    r = source * gain if residual is None else residual + gain * source
+    return r, (_rms(r, width, eps) * nxt.weight).to(dtype)
+
+
+def routed_mlp(x, routes, w_up, w_down, clamped=None):
+    """Expert rows in route order (row t * top + k belongs to token t's k-th expert; zero for experts
+    past the last one with tensors)."""
+    if isinstance(routes, ScoredRoutes):
+        routes = routes.ids
     T, top = routes.shape
     y = torch.zeros(T * top, w_down.shape[1], dtype=x.dtype)
     flat = routes.reshape(-1)
     tok = torch.arange(T).repeat_interleave(top)
     for e in flat.unique().tolist():
+        if e >= w_down.shape[0]:
+            continue
         sel = (flat == e).nonzero(as_tuple=True)[0]
-        h = gelu_erf(linear(x[tok[sel]], w_up[e], None, torch.float32)).to(x.dtype)
+        if clamped:
+            h = clamped_linear(x[tok[sel]], w_up[e], *clamped)
+        else:
+            h = gelu_erf(linear(x[tok[sel]], w_up[e], None, torch.float32)).to(x.dtype)
         y[sel] = linear(h, w_down[e], None, x.dtype)
     return y
 

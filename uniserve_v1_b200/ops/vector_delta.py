@@ -1,6 +1,8 @@
-"""Recurrent mixers whose decay is a vector over the key channels of a head.
+"""Recurrent mixers with a delta rule, the decay a vector over the key channels of a head or one number
+per head.
 
     channel rule:  S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;   o = S^T q
+    head rule:     the same with a scalar g
     general rule:  S <- diag(w) S - (a n)(n^T S) + k v^T (both on the old S); o = S^T q
 
 Batches are packed: rows of sequence s are cu[s] .. cu[s + 1], its state lives in slot
@@ -33,6 +35,7 @@ class SeqMeta:
     starts: Optional[list] = None    # on the host: first position and number of rows of every
     lengths: Optional[list] = None   # sequence (read back from the device when not given)
     short: Optional[tuple] = None    # cache of ``short_rows``
+    short_of: Optional[tuple] = None  # cache of ``short_sequences``
 
     def host(self):
         if self.lengths is None:
@@ -54,6 +57,18 @@ class SeqMeta:
                           .to(self.cu.device, non_blocking=True) if rows else None)
         return self.short[1]
 
+    def short_sequences(self, least: int):
+        """Beside ``short_rows``: (sequence, number of keys up to the row itself) of every such row, int32."""
+        if self.short_of is None or self.short_of[0] != least:
+            of, keys = [], []
+            for s, (p, n) in enumerate(zip(*self.host())):
+                if n < least:
+                    of.extend([s] * n)
+                    keys.extend(range(p + 1, p + n + 1))
+            both = torch.tensor([of, keys], dtype=torch.int32, pin_memory=self.cu.is_cuda)
+            self.short_of = (least, both.to(self.cu.device, non_blocking=True))
+        return self.short_of[1]
+
 
 def _spans(m: SeqMeta):
     cu, slots = m.cu.tolist(), m.slots.tolist()
@@ -71,14 +86,22 @@ def channel_prep(x, offs, low, w, conv, m: SeqMeta, H, Hk, D, V):
     low-rank rows ``low`` [T, H * D] (FP32) to what the rule reads: unit q (scaled) and k
     [T, Hk, D], v [T, H, V], decay g [T, H, D], beta [T, H], all FP32.  ``conv`` [slots, K, C]
     holds the last inputs of the short convolutions, the input of position p in entry p % K, and
-    is advanced."""
-    oq, ok, ov, ob = offs
+    is advanced.  ``low`` None: a decay per head, g [T, H], its argument at the fifth column of ``offs``."""
+    oq, ok, ov, ob = offs[:4]
     T, K, dev = x.shape[0], w["conv_q"].shape[1], x.device
     if x.is_cuda:
         f = dict(dtype=torch.float32, device=dev)
         q, k = torch.empty(T, Hk, D, **f), torch.empty(T, Hk, D, **f)
-        v, g = torch.empty(T, H, V, **f), torch.empty(T, H, D, **f)
-        beta = torch.empty(T, H, **f)
+        v, beta = torch.empty(T, H, V, **f), torch.empty(T, H, **f)
+        if low is None:
+            g = torch.empty(T, H, **f)
+            N.call("us_head_delta_prep", N.ptr(x), x.stride(0), *offs, N.ptr(w["conv_q"]), N.ptr(w["conv_k"]),
+                   N.ptr(w["conv_v"]), N.ptr(w["A_log"]), N.ptr(w["dt_bias"]), N.ptr(conv), N.ptr(q), N.ptr(k),
+                   N.ptr(v), N.ptr(g), N.ptr(beta), N.ptr(m.cu), N.ptr(m.slots), N.ptr(m.positions),
+                   m.slots.shape[0], T, H, Hk, D, V, K, int(x.dtype == BF16), int(m.one_token), N.stream(),
+                   launches=1 if m.one_token or K == 1 else 2)
+            return q, k, v, g, beta
+        g = torch.empty(T, H, D, **f)
         N.call("us_channel_delta_prep", N.ptr(x), x.stride(0), oq, ok, ov, ob, N.ptr(w["conv_q"]),
                N.ptr(w["conv_k"]), N.ptr(w["conv_v"]), N.ptr(low), low.stride(0), N.ptr(w["A_log"]),
                N.ptr(w["dt_bias"]), N.ptr(conv), N.ptr(q), N.ptr(k), N.ptr(v), N.ptr(g),
@@ -102,8 +125,11 @@ def channel_prep(x, offs, low, w, conv, m: SeqMeta, H, Hk, D, V):
     y = torch.nn.functional.silu(y)
     q = _unit(y[:, :nq].view(T, Hk, D)) * D ** -0.5
     k = _unit(y[:, nq:2 * nq].view(T, Hk, D))
-    g = torch.exp(-w["A_log"].exp()[None, :, None] *
-                  torch.nn.functional.softplus(low + w["dt_bias"]).view(T, H, D))
+    if low is None:
+        g = torch.exp(-w["A_log"].exp() * torch.nn.functional.softplus(x[:, offs[4]:offs[4] + H].float() + w["dt_bias"]))
+    else:
+        g = torch.exp(-w["A_log"].exp()[None, :, None] *
+                      torch.nn.functional.softplus(low + w["dt_bias"]).view(T, H, D))
     return q, k, y[:, 2 * nq:].view(T, H, V), g, torch.sigmoid(x[:, ob:ob + H].float())
 
 
@@ -127,20 +153,22 @@ def general_prep(x, offs, low, w, H, D):
 
 def vector_delta_rule(q, k, v, g, state, m: SeqMeta, beta=None, n=None, p=None):
     """The recurrence.  q, k [T, Hk, D], v [T, H, V], g / n / p [T, H, D] and beta [T, H] are dense
-    FP32; ``beta`` selects the channel rule, ``n`` and ``p`` the general one.  ``state``
-    [slots, H, D, V] FP32 is updated in place.  Returns o [T, H, V] FP32."""
-    T, H, D = g.shape
-    Hk, V = q.shape[1], v.shape[2]
+    FP32; ``beta`` selects the channel rule (with g [T, H] the head rule), ``n`` and ``p`` the general
+    one.  ``state`` [slots, H, D, V] FP32 is updated in place.  Returns o [T, H, V] FP32."""
+    T, H, V = v.shape
+    Hk, D = q.shape[1:]
     general = beta is None
     if q.is_cuda:
         for t in (q, k, v, g, state):
             assert t.dtype == torch.float32 and t.is_contiguous()
         out = torch.empty(T, H, V, dtype=torch.float32, device=q.device)
-        N.call("us_vector_delta_rule", int(general), N.ptr(q), N.ptr(k), N.ptr(v), N.ptr(g), N.ptr(n),
+        N.call("us_vector_delta_rule", 1 if general else 2 if g.dim() == 2 else 0, N.ptr(q), N.ptr(k), N.ptr(v), N.ptr(g), N.ptr(n),
                N.ptr(p), N.ptr(beta), N.ptr(state), N.ptr(out), N.ptr(m.cu), N.ptr(m.slots),
                N.ptr(m.positions), m.slots.shape[0], H, Hk, D, V, N.stream())
         return out
     q, k = (t.repeat_interleave(H // Hk, 1) for t in (q, k))
+    if g.dim() == 2:
+        g = g[:, :, None].expand(T, H, D)
     out = torch.zeros(T, H, V)
     for lo, hi, slot, fresh in _spans(m):
         S = torch.zeros_like(state[slot]) if fresh else state[slot]
@@ -158,20 +186,23 @@ def vector_delta_rule(q, k, v, g, state, m: SeqMeta, beta=None, n=None, p=None):
     return out
 
 
-def head_norm_gate(o, w, gate, eps, ldo, dtype):
+def head_norm_gate(o, w, gate, eps, ldo, dtype, act="sigmoid"):
     """o [T, H, V] divided by its root mean square per head, times ``w`` ([V] shared by the
-    heads or [H * V]) and sigmoid(gate [T, H * V]); rows ``ldo`` wide (zero past H * V)."""
+    heads or [H * V]) and act(gate [T, H * V]); rows ``ldo`` wide (zero past H * V).  ``act``: sigmoid
+    or silu."""
     T, H, V = o.shape
     if o.is_cuda:
         y = torch.empty(T, ldo, dtype=dtype, device=o.device)
         N.call("us_head_norm_gate", N.ptr(o), N.ptr(w), 0 if w.numel() == V else V, N.ptr(gate),
                gate.stride(0), N.ptr(y), ldo, T, H, V, eps, int(dtype == BF16),
-               int(gate.dtype == BF16), N.stream())
+               int(gate.dtype == BF16), int(act == "silu"), N.stream())
         return y
     y = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps)
     y = y * (w if w.numel() == V else w.view(H, V))
     out = torch.zeros(T, ldo, dtype=dtype)
-    out[:, :H * V] = (y.reshape(T, H * V) * torch.sigmoid(gate.float())).to(dtype)
+    gate = gate.float()
+    gate = torch.sigmoid(gate) * (gate if act == "silu" else 1.0)
+    out[:, :H * V] = (y.reshape(T, H * V) * gate).to(dtype)
     return out
 
 
@@ -192,6 +223,18 @@ def channel_step(x, offs, low, w, conv, state, gate, m: SeqMeta, H, Hk, D, V, ep
            0 if w["norm"].numel() == V else V, N.ptr(gate), gate.stride(0), N.ptr(y), H * V,
            N.ptr(m.slots), N.ptr(m.positions), B, H, Hk, D, V, w["conv_q"].shape[1], eps,
            int(x.dtype == BF16), int(gate.dtype == BF16), N.stream())
+    return y
+
+
+def head_step(x, offs, w, conv, state, gate, m: SeqMeta, H, Hk, D, V, eps, act="sigmoid"):
+    """``channel_step`` of the head rule: q, k, v, step size and decay argument at the columns ``offs``."""
+    B = x.shape[0]
+    y = torch.empty(B, H * V, dtype=x.dtype, device=x.device)
+    N.call("us_head_delta_step", N.ptr(x), x.stride(0), *offs, N.ptr(w["conv_q"]), N.ptr(w["conv_k"]),
+           N.ptr(w["conv_v"]), N.ptr(w["A_log"]), N.ptr(w["dt_bias"]), N.ptr(conv), N.ptr(state),
+           N.ptr(w["norm"]), 0 if w["norm"].numel() == V else V, N.ptr(gate), gate.stride(0), N.ptr(y), H * V,
+           N.ptr(m.slots), N.ptr(m.positions), B, H, Hk, D, V, w["conv_q"].shape[1], eps,
+           int(x.dtype == BF16), int(gate.dtype == BF16), int(act == "silu"), N.stream())
     return y
 
 
