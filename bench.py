@@ -631,10 +631,10 @@ def qwen3_record(job: Job) -> dict:
 
 # ------------------------------------------------- decoders of unlike layers --
 def layered_record(job: Job, family: str) -> dict:
-    """Prefill and decode throughput of the Nepevik or Zonopel decoder at a production-like layer
+    """Prefill and decode throughput of the Nepevik, Zonopel or Tadinex decoder at a production-like layer
     size (random weights) through ``LLMEngine``, beside existing models of equal size: Nepevik beside
     the Qwen3.5-style hybrid (gated delta net, dense-state engine) and Qwen3-MoE (attention in every
-    layer, the same paged engine), Zonopel beside Nepevik and Qwen3-MoE.  One GPU.
+    layer, the same paged engine), Zonopel and Tadinex beside Nepevik and Qwen3-MoE.  One GPU.
 
     ``value``: output tokens/s of the device-timed decode step of all concurrent requests (graph
     replays); ``sizes``: the same and the prompt throughput per (requests, prompt length)."""
@@ -645,6 +645,7 @@ def layered_record(job: Job, family: str) -> dict:
     from uniserve_v1_b200.models.nepevik import NepevikConfig, NepevikModel
     from uniserve_v1_b200.models.qwen3_5 import Qwen35Config, Qwen35MoeModel
     from uniserve_v1_b200.models.qwen3_moe import Qwen3MoeConfig, Qwen3MoeModel
+    from uniserve_v1_b200.models.tadinex import TadinexConfig, TadinexModel
     from uniserve_v1_b200.models.zonopel import ZonopelConfig, ZonopelModel
     from uniserve_v1_b200.ops import native
 
@@ -656,7 +657,8 @@ def layered_record(job: Job, family: str) -> dict:
         else [(64, 1024), (8, 4096), (1, 4096)]
     ncfg = NepevikConfig.bench(layers)
     zcfg = ZonopelConfig.bench(layers)
-    ncfg.vocab_size = zcfg.vocab_size = vocab
+    tcfg = TadinexConfig.bench(layers)
+    ncfg.vocab_size = zcfg.vocab_size = tcfg.vocab_size = vocab
     hcfg = Qwen35Config(vocab_size=vocab, hidden_size=2048, num_hidden_layers=layers,
                         num_attention_heads=32, num_key_value_heads=4, head_dim=128,
                         linear_num_key_heads=16, linear_num_value_heads=32, num_experts=64,
@@ -722,6 +724,7 @@ def layered_record(job: Job, family: str) -> dict:
 
     out, clocks, launches, head = [], None, 0, None
     models = {
+        "tadinex": (lambda: TadinexModel(tcfg, dev).init_random(0), paged, True),
         "zonopel": (lambda: ZonopelModel(zcfg, dev).init_random(0), paged, True),
         "nepevik": (lambda: NepevikModel(ncfg, dev).init_random(0), paged, True),
         "qwen3.5-style hybrid": (lambda: Qwen35MoeModel(hcfg, dev).init_random(0, std=0.02),
@@ -729,7 +732,8 @@ def layered_record(job: Job, family: str) -> dict:
                                      m, max_num_seqs=n, max_model_len=length + 128, prefill_chunk=8192,
                                      state_cache_entries=0), False),
         "qwen3-moe": (lambda: Qwen3MoeModel(qcfg, dev).init_random(0), paged, True)}
-    beside = {"nepevik": ("qwen3.5-style hybrid", "qwen3-moe"), "zonopel": ("nepevik", "qwen3-moe")}
+    beside = {"nepevik": ("qwen3.5-style hybrid", "qwen3-moe"), "zonopel": ("nepevik", "qwen3-moe"),
+              "tadinex": ("nepevik", "qwen3-moe")}
     for name in (family,) + (() if args.alone else beside[family]):
         build_model, make, graphs = models[name]
         model = build_model()
@@ -769,12 +773,12 @@ def layered_record(job: Job, family: str) -> dict:
 
 def main() -> int:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--workload", default="all", choices=["all", "qwen3-moe", "fasth3", "nepevik", "zonopel"],
+    ap.add_argument("--workload", default="all", choices=["all", "qwen3-moe", "fasth3", "nepevik", "zonopel", "tadinex"],
                     help="all (default): the FastH3 clip latency as the headline with the "
-                         "Qwen3-MoE record nested; or one of the two alone; nepevik, zonopel: that decoder's "
+                         "Qwen3-MoE record nested; or one of the two alone; nepevik, zonopel, tadinex: that decoder's "
                          "throughput beside models of equal size (one GPU, not part of all)")
     ap.add_argument("--alone", "--only-nepevik", dest="alone", action="store_true",
-                    help="nepevik, zonopel: without the models it is compared with")
+                    help="nepevik, zonopel, tadinex: without the models it is compared with")
     ap.add_argument("--frames", type=int, default=0, help="fasth3: frame count (rule 17n + 5)")
     ap.add_argument("--mlp-fp8", action="store_true",
                     help="fasth3: feed-forward projections in FP8 (per-tensor weights, per-row "
@@ -830,7 +834,7 @@ def main() -> int:
             line["metric"] = "FastH3 8-step clip latency (s); Qwen3-MoE output tokens/s nested"
             line["qwen3_moe"] = q
             line["gpu_launches"] = line["gpu_launches"] + q.get("gpu_launches", 0)
-    if args.workload in ("nepevik", "zonopel"):
+    if args.workload in ("nepevik", "zonopel", "tadinex"):
         line = layered_record(job, args.workload)
     if job.rank == 0 and line:
         print(json.dumps(line))

@@ -21,6 +21,9 @@
 // thread-block cluster (grid = M / 16 x S).  CTA s takes the K iterations s, s + S, ...;
 // the partial sums meet in the first CTA through distributed shared memory, in a fixed
 // order (the result does not depend on timing).
+//
+// The gated form pairs 8 features of the first half of the weight rows with 8 of the second: the two
+// feature groups of a CTA meet in its epilogue.
 #include "include/us_common.cuh"
 #include "include/us_tc05.cuh"
 
@@ -56,13 +59,29 @@ __device__ __forceinline__ float gelu_erf(float x) {
   return 0.5f * x * (1.f + erff(x * 0.70710678118654752f));
 }
 
+// (clamp(u) + 1) g sigmoid(alpha g) with g cut off above `limit`, u on both sides
+__device__ __forceinline__ float clamped_glu(float u, float g, float limit, float alpha) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return (u + 1.f) * (g / (1.f + __expf(-alpha * g)));
+}
+
+enum Form : int { kPlain = 0, kGelu = 1, kClamped = 2 };
+
+struct Glu {
+  int second;             // weight row of the first feature of the second half
+  float limit, alpha;
+};
+
 // MT = 16-row tiles of the activation (rows <= 16 * MT).
-template <int MT, bool GELU>
+template <int MT, int FORM>
 __global__ void __launch_bounds__(256)
 linear_decode_kernel(const __nv_bfloat16* __restrict__ W, const __nv_bfloat16* __restrict__ X,
                      void* __restrict__ out, const void* __restrict__ bias, int rows, int M, int K,
                      long long ldw, long long ldx, long long ldo, int out_f32, int bias_f32,
-                     int ksplit) {
+                     int ksplit, const Glu glu) {
+  constexpr bool GELU = FORM == kGelu, GATED = FORM == kClamped;
+  constexpr int kOut = GATED ? kFeat / 2 : kFeat;       // output features per CTA
   // Weights are never written by a kernel: the first loads go out before the wait on the
   // kernels that produce the activation.
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
@@ -75,9 +94,9 @@ linear_decode_kernel(const __nv_bfloat16* __restrict__ W, const __nv_bfloat16* _
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int ng = warp & 1, ks = warp >> 1;              // feature group, K slice
   const int n = lane >> 2, kq = lane & 3;
-  const int feat = blockIdx.x * kFeat + ng * 8 + n;
+  const int feat = blockIdx.x * kOut + (GATED ? n : ng * 8 + n);
   const bool feat_ok = feat < M;
-  const __nv_bfloat16* wrow = W + (long long)(feat_ok ? feat : 0) * ldw;
+  const __nv_bfloat16* wrow = W + (long long)(feat_ok ? feat + (GATED && ng ? glu.second : 0) : 0) * ldw;
   // this CTA's K iterations: every ksplit-th one starting at its cluster rank
   const int kr = ksplit > 1 ? (int)tc::cluster_ctarank() : 0;
   const int all_iters = K / kIterK;
@@ -175,13 +194,18 @@ linear_decode_kernel(const __nv_bfloat16* __restrict__ W, const __nv_bfloat16* _
     }
     tc::cluster_sync();
     if (kr == 0) {
-      for (int e = threadIdx.x; e < 16 * MT * kFeat; e += 256) {
-        const int r = e / kFeat, f = e - r * kFeat;
-        const int col = blockIdx.x * kFeat + f;
-        if (r >= rows || col >= M) continue;
+      auto whole = [&](int r, int f) {
         const uint32_t local = (uint32_t)__cvta_generic_to_shared(&red[0][f >> 3][r][f & 7]);
         float v = red[0][f >> 3][r][f & 7];
         for (int p = 1; p < ksplit; ++p) v += tc::ld_dsmem_f32(tc::map_to_cta(local, (uint32_t)p));
+        return v;
+      };
+      for (int e = threadIdx.x; e < 16 * MT * kOut; e += 256) {
+        const int r = e / kOut, f = e - r * kOut;
+        const int col = blockIdx.x * kOut + f;
+        if (r >= rows || col >= M) continue;
+        float v = whole(r, f);
+        if (GATED) v = clamped_glu(v, whole(r, f + 8), glu.limit, glu.alpha);
         if (bias)
           v += bias_f32 ? reinterpret_cast<const float*>(bias)[col]
                         : us::bf2f(reinterpret_cast<const __nv_bfloat16*>(bias)[col]);
@@ -195,13 +219,18 @@ linear_decode_kernel(const __nv_bfloat16* __restrict__ W, const __nv_bfloat16* _
     tc::cluster_sync();           // nobody leaves while its sums may still be read
     return;
   }
-  for (int e = threadIdx.x; e < 16 * MT * kFeat; e += 256) {
-    const int r = e / kFeat, f = e - r * kFeat;
-    const int col = blockIdx.x * kFeat + f;
-    if (r >= rows || col >= M) continue;
+  auto sliced = [&](int r, int f) {
     float v = 0.f;
 #pragma unroll
     for (int s = 0; s < kSlices; ++s) v += red[s][f >> 3][r][f & 7];
+    return v;
+  };
+  for (int e = threadIdx.x; e < 16 * MT * kOut; e += 256) {
+    const int r = e / kOut, f = e - r * kOut;
+    const int col = blockIdx.x * kOut + f;
+    if (r >= rows || col >= M) continue;
+    float v = sliced(r, f);
+    if (GATED) v = clamped_glu(v, sliced(r, f + 8), glu.limit, glu.alpha);
     if (bias)
       v += bias_f32 ? reinterpret_cast<const float*>(bias)[col]
                     : us::bf2f(reinterpret_cast<const __nv_bfloat16*>(bias)[col]);
@@ -213,27 +242,22 @@ linear_decode_kernel(const __nv_bfloat16* __restrict__ W, const __nv_bfloat16* _
   }
 }
 
-}  // namespace
-
-// act: 0 none, 3 gelu (erf) of the biased value.  rows <= 64, K a multiple of 256, 16-byte aligned rows of W and X.  Returns
-// US_ERR_UNSUPPORTED for other shapes (the caller then takes the tcgen05 kernel).
-US_API int us_linear_decode(const void* W, const void* X, void* out, const void* bias, int rows,
-                            int M, int K, long long ldw, long long ldx, long long ldo,
-                            int out_f32, int bias_f32, int act, void* stream_) {
-  US_REQUIRE(W && X && out && rows >= 1 && M >= 1 && K >= 1);
+int run(int form, const void* W, const void* X, void* out, const void* bias, int rows, int M, int K,
+        long long ldw, long long ldx, long long ldo, int out_f32, int bias_f32, const Glu& glu,
+        cudaStream_t stream) {
   if (rows > 64 || (K % kIterK) != 0 || (ldw % 8) != 0 || (ldx % 8) != 0 ||
       ((uintptr_t)W % 16) != 0 || ((uintptr_t)X % 16) != 0)
     return US_ERR_UNSUPPORTED;
-  cudaStream_t stream = (cudaStream_t)stream_;
-  const dim3 grid((M + kFeat - 1) / kFeat), block(256);
+  const int per = form == kClamped ? kFeat / 2 : kFeat;
+  const dim3 grid((M + per - 1) / per), block(256);
   const __nv_bfloat16* w = (const __nv_bfloat16*)W;
   const __nv_bfloat16* x = (const __nv_bfloat16*)X;
   static bool configured = false;
   if (!configured) {
-    for (auto k : {linear_decode_kernel<4, false>, linear_decode_kernel<4, true>})
+    for (auto k : {linear_decode_kernel<4, kPlain>, linear_decode_kernel<4, kGelu>, linear_decode_kernel<4, kClamped>})
       US_CUDA_CHECK(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          4 * kStages * 8192));
-    for (auto k : {linear_decode_kernel<2, false>, linear_decode_kernel<2, true>})
+    for (auto k : {linear_decode_kernel<2, kPlain>, linear_decode_kernel<2, kGelu>, linear_decode_kernel<2, kClamped>})
       US_CUDA_CHECK(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          2 * kStages * 8192));
     configured = true;
@@ -271,16 +295,38 @@ US_API int us_linear_decode(const void* W, const void* X, void* out, const void*
     cfg.attrs = attr;
     cfg.numAttrs = ksplit > 1 ? 2 : 1;
     return cudaLaunchKernelEx(&cfg, kernel, w, x, out, bias, rows, M, K, ldw, ldx, ldo, out_f32,
-                              bias_f32, ksplit);
+                              bias_f32, ksplit, glu);
   };
   // kStages buffers x (16 MT) rows x 512 bytes
-  US_REQUIRE(act == 0 || act == 3);
-  const bool gelu = act == 3;
-  if (rows <= 16)
-    US_CUDA_CHECK(launch(gelu ? linear_decode_kernel<1, true> : linear_decode_kernel<1, false>, kStages * 8192));
-  else if (rows <= 32)
-    US_CUDA_CHECK(launch(gelu ? linear_decode_kernel<2, true> : linear_decode_kernel<2, false>, 2 * kStages * 8192));
-  else
-    US_CUDA_CHECK(launch(gelu ? linear_decode_kernel<4, true> : linear_decode_kernel<4, false>, 4 * kStages * 8192));
+#define US_LD(MT)                                                                                \
+  US_CUDA_CHECK(form == kClamped ? launch(linear_decode_kernel<MT, kClamped>, MT * kStages * 8192) \
+                : form == kGelu  ? launch(linear_decode_kernel<MT, kGelu>, MT * kStages * 8192)    \
+                                 : launch(linear_decode_kernel<MT, kPlain>, MT * kStages * 8192))
+  if (rows <= 16) US_LD(1);
+  else if (rows <= 32) US_LD(2);
+  else US_LD(4);
+#undef US_LD
   return US_OK;
+}
+
+}  // namespace
+
+// act: 0 none, 3 gelu (erf) of the biased value.  rows <= 64, K a multiple of 256, 16-byte aligned rows of W and X.  Returns
+// US_ERR_UNSUPPORTED for other shapes (the caller then takes the tcgen05 kernel).
+US_API int us_linear_decode(const void* W, const void* X, void* out, const void* bias, int rows,
+                            int M, int K, long long ldw, long long ldx, long long ldo,
+                            int out_f32, int bias_f32, int act, void* stream_) {
+  US_REQUIRE(W && X && out && rows >= 1 && M >= 1 && K >= 1 && (act == 0 || act == 3));
+  return run(act == 3 ? kGelu : kPlain, W, X, out, bias, rows, M, K, ldw, ldx, ldo, out_f32, bias_f32,
+             Glu{0, 0.f, 0.f}, (cudaStream_t)stream_);
+}
+
+// Gated: out[rows, I] = (clamp(first) + 1) g sigmoid(alpha g), g = min(second, limit); W [2 I, K] holds the
+// rows of `first`, then those of `second`.  Same shapes otherwise; bf16 out.
+US_API int us_linear_decode_clamped(const void* W, const void* X, void* out, int rows, int I, int K,
+                                    long long ldw, long long ldx, long long ldo, float limit,
+                                    float alpha, void* stream_) {
+  US_REQUIRE(W && X && out && rows >= 1 && I >= 1 && K >= 1);
+  return run(kClamped, W, X, out, nullptr, rows, I, K, ldw, ldx, ldo, 0, 0, Glu{I, limit, alpha},
+             (cudaStream_t)stream_);
 }

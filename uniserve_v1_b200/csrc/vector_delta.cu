@@ -2,7 +2,7 @@
 // a pool.  The decay is a vector over the key channels of a head, or one number per head:
 //
 //   channel rule   S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;       o = S^T q
-//   head rule      the same with a scalar g
+//   head rule      the same with a scalar g (the recurrence itself: head_delta.cu)
 //   general rule   S <- diag(w) S - (a*n)(n^T S) + k v^T  (both read the old S);  o = S^T q
 //
 // with S [D, V] FP32 per (sequence, head).  The kernels:
@@ -27,8 +27,11 @@
 // is what a long prompt costs.  The vectors of the next chunks of 8 tokens are on their way into
 // a ring in shared memory meanwhile (four warps multiply, one fetches).  The state crosses HBM once per call.
 #include "include/us_common.cuh"
+#include "include/us_f32x2.cuh"
 
 namespace {
+
+using namespace us::f32x2;        // two rows of one state column per instruction
 
 __device__ __forceinline__ float ld_any(const void* base, long long idx, int bf16) {
   return bf16 ? us::bf2f(reinterpret_cast<const __nv_bfloat16*>(base)[idx])
@@ -276,10 +279,10 @@ constexpr int kRuleBufs = 4;                         // chunks of vectors in sha
 
 struct RuleArgs {
   const float *q, *k, *v;         // [rows, Hk, D] x 2, [rows, H, V]
-  const float* g;                 // decay [rows, H, D] (head rule: [rows, H])
+  const float* g;                 // decay [rows, H, D]
   const float* n;                 // general: removal direction [rows, H, D]
   const float* p;                 // general: removal rate * direction [rows, H, D]
-  const float* beta;              // channel, head: [rows, H]
+  const float* beta;              // channel: [rows, H]
   float* state;                   // [slots, H, D, V]
   float* out;                     // [rows, H, V]
   const int *cu, *slots, *pos;
@@ -295,37 +298,6 @@ __device__ __forceinline__ float fold8(float c0, float c1, bool up) {
   return s;
 }
 
-// Packed FP32 pairs (two rows of one state column per instruction).
-typedef unsigned long long f2;
-__device__ __forceinline__ f2 pack2(float a, float b) {
-  f2 r;
-  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
-  return r;
-}
-__device__ __forceinline__ float lo2(f2 r) { return __uint_as_float((uint32_t)r); }
-__device__ __forceinline__ float hi2(f2 r) { return __uint_as_float((uint32_t)(r >> 32)); }
-__device__ __forceinline__ f2 fma2(f2 a, f2 b, f2 c) {
-  f2 d;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-  return d;
-}
-__device__ __forceinline__ f2 mul2(f2 a, f2 b) {
-  f2 d;
-  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
-  return d;
-}
-__device__ __forceinline__ f2 add2(f2 a, f2 b) {
-  f2 d;
-  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
-  return d;
-}
-// four consecutive floats as two pairs
-__device__ __forceinline__ void lds_vec(f2 (&o)[2], const float* p) {
-  const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(p);
-  o[0] = v.x;
-  o[1] = v.y;
-}
-
 template <int BYTES>
 __device__ __forceinline__ void cp_async(float* dst, const float* src) {
   const uint32_t d = (uint32_t)__cvta_generic_to_shared(dst);
@@ -333,12 +305,11 @@ __device__ __forceinline__ void cp_async(float* dst, const float* src) {
   else asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(d), "l"(src) : "memory");
 }
 
-// A token in shared memory: kVecs vectors of DP floats (g, k, q and, general, n, p; head: k, q), then
-// 32 columns of v, beta and, head, g.
-template <int DP, int RULE>
+// A token in shared memory: kVecs vectors of DP floats (g, k, q and, general, n, p), then 32
+// columns of v and beta.
+template <int DP, bool GENERAL>
 struct Stage {
-  static constexpr int kVecs = RULE == kGeneral ? 5 : RULE == kHead ? 2 : 3;
-  static constexpr int kKey = RULE == kHead ? 0 : DP, kRead = kKey + DP;    // places of k and q
+  static constexpr int kVecs = GENERAL ? 5 : 3;
   static constexpr int kToken = kVecs * DP + kCols + 4;
   static constexpr int kChunk = 8;                    // tokens per chunk
   static constexpr int kFloats = kChunk * kToken;
@@ -347,30 +318,22 @@ struct Stage {
 // Asynchronous copies of tokens' vectors by the copying threads.  Widths that are multiples of
 // four move as 16-byte pieces: a thread owns the same pieces of every token and only advances its
 // pointers (address arithmetic per piece would cost as much as the recurrence).
-template <int DP, int RULE>
+template <int DP, bool GENERAL>
 struct Copier {
-  using St = Stage<DP, RULE>;
+  using St = Stage<DP, GENERAL>;
   static constexpr int kQ = DP / 4;
   static constexpr int kPieces = St::kVecs * kQ + kCols / 4;
   static constexpr int kMine = (kPieces + kRuleCopy - 1) / kRuleCopy;
   const float* src[kMine];
   int step[kMine], dst[kMine];          // floats per token, place in the token (-1: nothing)
-  const float *beta, *decay;
+  const float* beta;
   int tid, heads;
   bool quad;
-  static __device__ __forceinline__ bool shared_vec(int vec) {      // one per key head
-    return RULE == kHead || vec == 1 || vec == 2;
-  }
-  static __device__ __forceinline__ const float* source(const RuleArgs& a, int vec) {
-    if (RULE == kHead) return vec == 0 ? a.k : a.q;
-    return vec == 1 ? a.k : vec == 2 ? a.q : vec == 0 ? a.g : vec == 3 ? a.n : a.p;
-  }
   __device__ __forceinline__ void init(const RuleArgs& a, int tid_, long long row0, int h, int hk, int col0) {
     tid = tid_;
     heads = a.H;
     quad = (a.V & 3) == 0 && (a.D & 3) == 0;
-    beta = RULE == kGeneral ? nullptr : a.beta + row0 * a.H + h;
-    decay = RULE == kHead ? a.g + row0 * a.H + h : nullptr;
+    beta = GENERAL ? nullptr : a.beta + row0 * a.H + h;
 #pragma unroll
     for (int i = 0; i < kMine; ++i) {
       const int e = tid + i * kRuleCopy, vec = e / kQ, d = (e - vec * kQ) * 4;
@@ -379,9 +342,10 @@ struct Copier {
       step[i] = 0;
       if (e < St::kVecs * kQ) {
         if (d >= a.D) continue;
-        const bool shared = shared_vec(vec);
+        const bool shared = vec == 1 || vec == 2;
         const int heads_ = shared ? a.Hk : a.H, hh = shared ? hk : h;
-        src[i] = source(a, vec) + (row0 * heads_ + hh) * a.D + d;
+        src[i] = (vec == 1 ? a.k : vec == 2 ? a.q : vec == 0 ? a.g : vec == 3 ? a.n : a.p) +
+                 (row0 * heads_ + hh) * a.D + d;
         step[i] = heads_ * a.D;
         dst[i] = vec * DP + d;
       } else if (e < kPieces) {
@@ -404,13 +368,9 @@ struct Copier {
             cp_async<16>(buf + dst[i], src[i]);
             src[i] += step[i];
           }
-        if (RULE != kGeneral && tid == 0) {
+        if (!GENERAL && tid == 0) {
           cp_async<4>(buf + St::kVecs * DP + kCols, beta);
           beta += heads;
-        }
-        if (RULE == kHead && tid == 1) {
-          cp_async<4>(buf + St::kVecs * DP + kCols + 1, decay);
-          decay += heads;
         }
       }
     } else {
@@ -418,23 +378,22 @@ struct Copier {
         const long long row = row0 + t;
         for (int e = tid; e < St::kVecs * a.D; e += kRuleCopy) {
           const int vec = e / a.D, d = e - vec * a.D;
-          cp_async<4>(buf + vec * DP + d,
-                      source(a, vec) + (shared_vec(vec) ? row * a.Hk + hk : row * a.H + h) * a.D + d);
+          const bool shared = vec == 1 || vec == 2;
+          const float* from = vec == 1 ? a.k : vec == 2 ? a.q : vec == 0 ? a.g : vec == 3 ? a.n : a.p;
+          cp_async<4>(buf + vec * DP + d, from + (shared ? row * a.Hk + hk : row * a.H + h) * a.D + d);
         }
         for (int c = tid; c < kCols && col0 + c < a.V; c += kRuleCopy)
           cp_async<4>(buf + St::kVecs * DP + c, a.v + (row * a.H + h) * a.V + col0 + c);
-        if (RULE != kGeneral && tid == 0) cp_async<4>(buf + St::kVecs * DP + kCols, a.beta + row * a.H + h);
-        if (RULE == kHead && tid == 1) cp_async<4>(buf + St::kVecs * DP + kCols + 1, a.g + row * a.H + h);
+        if (!GENERAL && tid == 0) cp_async<4>(buf + St::kVecs * DP + kCols, a.beta + row * a.H + h);
       }
     }
   }
 };
 
-template <int DP, int RULE>
+template <int DP, bool GENERAL>
 __global__ void __launch_bounds__(kRuleThreads, DP > 128 ? 1 : 3) vector_delta_kernel(const RuleArgs a) {
   US_PDL_PROLOGUE();
-  using St = Stage<DP, RULE>;
-  constexpr bool GENERAL = RULE == kGeneral;
+  using St = Stage<DP, GENERAL>;
   constexpr int NG = DP / 32;                         // groups of four rows per lane
   extern __shared__ __align__(16) float sm[];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -456,7 +415,7 @@ __global__ void __launch_bounds__(kRuleThreads, DP > 128 ? 1 : 3) vector_delta_k
     __syncthreads();
   }
   if (tid >= kRuleCompute) {                          // the copying threads stay one chunk ahead
-    Copier<DP, RULE> cp;
+    Copier<DP, GENERAL> cp;
     cp.init(a, tid - kRuleCompute, start, h, hk, col0);
     const int chunks = (T + St::kChunk - 1) / St::kChunk;
     auto fetch = [&](int r) {                         // (an empty group past the end)
@@ -527,16 +486,14 @@ __global__ void __launch_bounds__(kRuleThreads, DP > 128 ? 1 : 3) vector_delta_k
         if (GENERAL) {
           lds_vec(m, base + 3 * DP + r0);
         } else {
-          lds_vec(m, base + St::kKey + r0);
-          if (RULE == kChannel) {
-            f2 g[2];
-            lds_vec(g, base + r0);
+          f2 g[2];
+          lds_vec(m, base + DP + r0);
+          lds_vec(g, base + r0);
 #pragma unroll
-            for (int e = 0; e < 2; ++e)
+          for (int e = 0; e < 2; ++e)
 #pragma unroll
-              for (int c = 0; c < 2; ++c)   // the key sees the decayed state
-                S[j * 2 + e][c] = mul2(S[j * 2 + e][c], g[e]);
-          }
+            for (int c = 0; c < 2; ++c)     // the key sees the decayed state
+              S[j * 2 + e][c] = mul2(S[j * 2 + e][c], g[e]);
         }
 #pragma unroll
         for (int e = 0; e < 2; ++e)
@@ -553,8 +510,7 @@ __global__ void __launch_bounds__(kRuleThreads, DP > 128 ? 1 : 3) vector_delta_k
       }
       pending = true;
       float c = seen;                               // general: n^T S of this lane's column
-      const float dec = RULE == kHead ? vs[kCols + 1] : 1.f;
-      if (!GENERAL) c = vs[kCols] * (vs[cb + (up ? 1 : 0)] - (RULE == kHead ? dec * seen : seen));
+      if (!GENERAL) c = vs[kCols] * (vs[cb + (up ? 1 : 0)] - seen);
       const float other = __shfl_xor_sync(0xffffffffu, c, 4);
       const float u0 = up ? other : c, u1 = up ? c : other;
       f2 uu[2], vv[2];
@@ -565,14 +521,13 @@ __global__ void __launch_bounds__(kRuleThreads, DP > 128 ? 1 : 3) vector_delta_k
       } else {
         uu[0] = pack2(u0, u0); uu[1] = pack2(u1, u1);
       }
-      const f2 dd = pack2(dec, dec);
       f2 oo[2][2] = {{0ull, 0ull}, {0ull, 0ull}};
 #pragma unroll
       for (int j = 0; j < NG; ++j) {
         const int r0 = (j * 8 + kq) * 4;
         f2 k[2], q[2], g[2], p[2];
-        lds_vec(k, base + St::kKey + r0);
-        lds_vec(q, base + St::kRead + r0);
+        lds_vec(k, base + DP + r0);
+        lds_vec(q, base + 2 * DP + r0);
         if (GENERAL) {
           lds_vec(g, base + r0);
           lds_vec(p, base + 4 * DP + r0);
@@ -583,7 +538,6 @@ __global__ void __launch_bounds__(kRuleThreads, DP > 128 ? 1 : 3) vector_delta_k
           for (int c = 0; c < 2; ++c) {
             f2& x = S[j * 2 + e][c];
             if (GENERAL) x = fma2(k[e], vv[c], fma2(p[e], uu[c], mul2(g[e], x)));
-            else if (RULE == kHead) x = fma2(k[e], uu[c], mul2(dd, x));
             else x = fma2(k[e], uu[c], x);
             oo[c][e] = fma2(x, q[e], oo[c][e]);
           }
@@ -848,16 +802,16 @@ int step_impl(const StepArgs& a, int B, cudaStream_t stream) {
   return launch_step<64, RULE>(a, B, stream);
 }
 
-template <int DP, int RULE>
+template <int DP, bool GENERAL>
 int launch_rule(const RuleArgs& a, int B, cudaStream_t stream) {
-  constexpr size_t smem = kRuleBufs * Stage<DP, RULE>::kFloats * sizeof(float);
+  constexpr size_t smem = kRuleBufs * Stage<DP, GENERAL>::kFloats * sizeof(float);
   static bool configured = false;
   if (!configured && smem > 48 * 1024) {
-    US_CUDA_CHECK(cudaFuncSetAttribute(vector_delta_kernel<DP, RULE>,
+    US_CUDA_CHECK(cudaFuncSetAttribute(vector_delta_kernel<DP, GENERAL>,
                                        cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
   }
   configured = true;
-  US_CUDA_CHECK(us::launch_pdl(vector_delta_kernel<DP, RULE>,
+  US_CUDA_CHECK(us::launch_pdl(vector_delta_kernel<DP, GENERAL>,
                                dim3((a.V + kCols - 1) / kCols, a.H, B), dim3(kRuleThreads), smem,
                                stream, a));
   return US_OK;
@@ -931,23 +885,21 @@ US_API int us_general_delta_prep(const void* x, long long ldx, int off_r, int of
   return US_OK;
 }
 
-// rule = 0: the channel rule (g, beta); 1: the general rule (g, n, p); 2: the head rule (g per head,
-// beta).  q and k heads serve H / Hk value heads each; all vectors dense FP32.
-US_API int us_vector_delta_rule(int rule, const float* q, const float* k, const float* v,
+// general = 0: the channel rule (g, beta); 1: the general rule (g, n, p).  q and k heads serve
+// H / Hk value heads each; all vectors dense FP32.
+US_API int us_vector_delta_rule(int general, const float* q, const float* k, const float* v,
                                 const float* g, const float* n, const float* p, const float* beta,
                                 float* state, float* out, const int* cu, const int* slots,
                                 const int* pos, int B, int H, int Hk, int D, int V, void* stream_) {
   US_REQUIRE(q && k && v && g && state && out && cu && slots && pos && B >= 1 && B <= 65535);
-  US_REQUIRE(rule >= kChannel && rule <= kHead && (rule == kGeneral ? (n && p) : (beta != nullptr)));
+  US_REQUIRE(general ? (n && p) : (beta != nullptr));
   US_REQUIRE(H >= 1 && Hk >= 1 && H % Hk == 0 && H <= 65535 && D >= 1 && V >= 1);
-  US_REQUIRE((D & 3) || (V & 3) || (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (rule == kHead ? 0 : (uintptr_t)g) |
-               (uintptr_t)n | (uintptr_t)p | (uintptr_t)state) % 16) == 0);
+  US_REQUIRE((D & 3) || (V & 3) || (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)g | (uintptr_t)n |
+               (uintptr_t)p | (uintptr_t)state) % 16) == 0);
   RuleArgs a{q, k, v, g, n, p, beta, state, out, cu, slots, pos, H, Hk, D, V};
   cudaStream_t stream = (cudaStream_t)stream_;
 #define US_VD(DP) \
-  if (D <= DP) return rule == kGeneral ? launch_rule<DP, kGeneral>(a, B, stream)                       \
-                      : rule == kHead  ? launch_rule<DP, kHead>(a, B, stream)                          \
-                                       : launch_rule<DP, kChannel>(a, B, stream);
+  if (D <= DP) return general ? launch_rule<DP, true>(a, B, stream) : launch_rule<DP, false>(a, B, stream);
   US_VD(32) US_VD(64) US_VD(128) US_VD(256)
 #undef US_VD
   return US_ERR_UNSUPPORTED;

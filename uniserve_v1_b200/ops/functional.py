@@ -379,6 +379,11 @@ def clamped_linear(x, w, limit, alpha, out=None, tiles=None, block_n=None, live=
                *tile_args, N.stream())
         N.call("us_clamped_glu_f32", N.ptr(z), N.ptr(out), rows, I_, limit, alpha, N.stream())
         return out
+    if LINEAR_DECODE and tiles is None and rows <= 64 and K % 256 == 0 and I2 * K <= LINEAR_DECODE_MAX and \
+            x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0:
+        N.call("us_linear_decode_clamped", N.ptr(w), N.ptr(x), N.ptr(out), rows, I_, K, K, x.stride(0), I_, limit, alpha,
+               N.stream())
+        return out
     if live:
         N.kernels().us_gemm_wx_hint(live * ((I_ + 127) // 128))
     N.call("us_gemm_wx_clamped", N.ptr(w), N.ptr(x), N.ptr(out), E, I2, I_, K, rows, K, x.stride(0), I_, I_,

@@ -40,6 +40,7 @@ _SIGNATURES = {
     "us_gemm_wx": (I, [P, P, P, I, I, I, I, I, L, L, L, I, I, I, I, P, I, P, P, P, P, P, P, I, I, P]),
     "us_gemm_wx_hint": (I, [I]),
     "us_linear_decode": (I, [P, P, P, P, I, I, I, L, L, L, I, I, I, P]),
+    "us_linear_decode_clamped": (I, [P, P, P, I, I, I, L, L, L, F, F, P]),
     "us_gemm_f32": (I, [P, P, P, I, I, I, I, I, L, L, L, I, P, P, P, P, P, I, P]),
     "us_channel_delta_prep": (I, [P, L, I, I, I, I, P, P, P, P, L, P, P, P, P, P, P, P, P, P, P, P,
                                   I, I, I, I, I, I, I, I, I, P]),
@@ -51,6 +52,8 @@ _SIGNATURES = {
                                   F, I, I, P]),
     "us_head_delta_prep": (I, [P, L, I, I, I, I, I, P, P, P, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I,
                                I, I, I, I, I, P]),
+    "us_head_delta_coef_floats": (L, [I, I, I]),
+    "us_head_delta_rule": (I, [P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, P]),
     "us_head_delta_step": (I, [P, L, I, I, I, I, I, P, P, P, P, P, P, P, P, I, P, L, P, L, P, P, I, I, I,
                                I, I, I, F, I, I, I, P]),
     "us_head_norm_gate": (I, [P, P, I, P, L, P, L, I, I, I, F, I, I, I, P]),

@@ -8,7 +8,7 @@ per head.
 Batches are packed: rows of sequence s are cu[s] .. cu[s + 1], its state lives in slot
 ``slots[s]`` of a pool and is updated in place; a sequence whose first row stands at position 0
 starts from zero whatever the slot holds, a negative slot marks padding.  On a GPU the entry
-points run ``csrc/vector_delta.cu``; on the CPU the same recurrences run step by step in FP32.
+points run ``csrc/vector_delta.cu`` (the head rule's recurrence: ``csrc/head_delta.cu``); on the CPU the same recurrences run step by step in FP32.
 """
 from __future__ import annotations
 
@@ -162,7 +162,14 @@ def vector_delta_rule(q, k, v, g, state, m: SeqMeta, beta=None, n=None, p=None):
         for t in (q, k, v, g, state):
             assert t.dtype == torch.float32 and t.is_contiguous()
         out = torch.empty(T, H, V, dtype=torch.float32, device=q.device)
-        N.call("us_vector_delta_rule", 1 if general else 2 if g.dim() == 2 else 0, N.ptr(q), N.ptr(k), N.ptr(v), N.ptr(g), N.ptr(n),
+        if g.dim() == 2:
+            coef = torch.empty(N.kernels().us_head_delta_coef_floats(T, m.slots.shape[0], H), dtype=torch.float32,
+                               device=q.device)
+            N.call("us_head_delta_rule", N.ptr(q), N.ptr(k), N.ptr(v), N.ptr(g), N.ptr(beta), N.ptr(coef), N.ptr(state),
+                   N.ptr(out), N.ptr(m.cu), N.ptr(m.slots), N.ptr(m.positions), m.slots.shape[0], T, H, Hk, D, V,
+                   N.stream(), launches=2)
+            return out
+        N.call("us_vector_delta_rule", int(general), N.ptr(q), N.ptr(k), N.ptr(v), N.ptr(g), N.ptr(n),
                N.ptr(p), N.ptr(beta), N.ptr(state), N.ptr(out), N.ptr(m.cu), N.ptr(m.slots),
                N.ptr(m.positions), m.slots.shape[0], H, Hk, D, V, N.stream())
         return out

@@ -1,5 +1,5 @@
-"""Kernels of the vector-decay, head-mixing, table-routed, state-space and latent-attention layers
-beside the like kernels of the hybrid and Qwen3 decoders at equal sizes, each with its roofline
+"""Kernels of the delta-rule, head-mixing, table- and score-routed, state-space, linear-attention, latent-
+and windowed-attention layers beside the like kernels of the hybrid and Qwen3 decoders at equal sizes, each with its roofline
 fraction.
 
     python -m uniserve_v1_b200.tools.opbench_mixers [--only NAME,...] [--batch 64] [--rows 8192]
@@ -21,6 +21,7 @@ from ..ops import latent as LA
 from ..ops import native as N
 from ..ops import state_space as SS
 from ..ops import vector_delta as VD
+from ..ops import window as WA
 from .opbench import peaks, timeit
 
 
@@ -99,6 +100,14 @@ def main():
         conv = torch.zeros(B, K, C, dtype=bf, device=dev)
         case(f"channel_prep_{kind}", lambda: VD.channel_prep(x, (0, Hk * D, 2 * Hk * D, C), low, w, conv, m, H, Hk, D, V),
              n * (2.0 * C + 4 * H * D) + vec - n * H * V * 4.0 + (2 * B * (K - 1) * C * 2.0 if kind == "decode" else 0))
+        # one decay per head
+        gh = torch.rand(n, H, device=dev) * 0.1 + 0.9
+        vech = 4.0 * n * (2 * Hk * D + 2 * H * V + 2 * H)
+        case(f"head_rule_{kind}", lambda: VD.vector_delta_rule(q, k, v, gh, pool, m, beta=beta), state + vech)
+        wh = dict(w, dt_bias=rnd(H, dtype=torch.float32))
+        case(f"head_prep_{kind}", lambda: VD.channel_prep(x, (0, Hk * D, 2 * Hk * D, C, C + 32), None, wh, conv, m, H, Hk, D,
+                                                          V),
+             n * 2.0 * C + vech - n * H * V * 4.0 + (2 * B * (K - 1) * C * 2.0 if kind == "decode" else 0))
         xc, conv3 = rnd(n, C), torch.zeros(B, K - 1, C, dtype=bf, device=dev)
         wc = rnd(C, K, dtype=torch.float32)
         case(f"causal_conv1d_{kind} (like)", lambda: GD.causal_conv1d(xc, wc, conv3, cu=m.cu, slots=m.slots),
@@ -113,6 +122,10 @@ def main():
             case("channel_step_decode", lambda: VD.channel_step(x, (0, Hk * D, 2 * Hk * D, C), low, w, conv, pool,
                                                                 gate, m, H, Hk, D, V, 1e-6),
                  state + n * (2.0 * C * (K + 1) + 4 * H * D + 4 * H * V))
+            wh.update(norm=hw)
+            case("head_step_decode", lambda: VD.head_step(x, (0, Hk * D, 2 * Hk * D, C, C + 32), wh, conv, pool, gate, m,
+                                                          H, Hk, D, V, 1e-6, "silu"),
+                 state + n * (2.0 * C * (K + 1) + 4 * H * V))
             w2 = dict(w, norm=rnd(H * D2, dtype=torch.float32))
             case("general_step_decode", lambda: VD.general_step(xg, (0, H * D2, 2 * H * D2, 4 * H * D2), lowg, w2,
                                                                 pool2, xg[:, 3 * H * D2:4 * H * D2], m, H, D2, 1e-6),
@@ -148,6 +161,35 @@ def main():
         ids = routes.ids.contiguous()
         case(f"moe_experts_{kind} (like)", lambda: F.moe_experts(y, ids, wts, w13, down, ws=ws, defer_unpermute=True),
              1.5 * wb + n * top * (2 * W + I) * 2.0, 6.0 * n * top * I * W)
+        # routes by scores: 64 experts and 4 identities
+        logits, corr = rnd(n, E + 4, dtype=torch.float32), rnd(E + 4, dtype=torch.float32) * 0.02
+        sync = torch.zeros(4, dtype=torch.int32, device=dev)
+        case(f"scored_routes_{kind}", lambda: F.scored_routes(logits, corr, top, E, y, sync))
+        l64 = logits[:, :E].contiguous()
+
+        def like_routes():
+            if n <= 512:
+                return F.route_sort_gather(l64, y, top, True, ws, 0, E)
+            i4, _ = F.topk_softmax(l64, top, True)
+            N.call("us_moe_sort", N.ptr(i4), n * top, 0, E, ws.block_n, ws.max_tiles, N.ptr(ws.sorted_route),
+                   N.ptr(ws.perm_of_route), N.ptr(ws.expert_offsets), N.ptr(ws.tile_group), N.ptr(ws.tile_row0),
+                   N.ptr(ws.tile_rows), N.ptr(ws.num_tiles), N.stream())
+        case(f"topk_sort_{kind} (like)", like_routes)
+        sr = F.scored_routes(logits, corr, top, E, y, sync)
+        share = float((sr.perm >= 0).float().mean())        # routes that reach an expert with tensors
+        sr.xp = None
+        case(f"clamped_experts_{kind}", lambda: F.routed_mlp(y, sr, w13, down, clamped=(7.0, 1.702)),
+             1.5 * wb + share * n * top * (2 * W + I) * 2.0, 6.0 * share * n * top * I * W)
+        s13 = rnd(2 * 1024, W)
+        case(f"clamped_linear_{kind}", lambda: F.clamped_linear(y, s13, 7.0, 1.702), 2.0 * (2048 * W + n * (W + 1024)),
+             4.0 * n * 1024 * W)
+        case(f"linear_gated_{kind} (like)", lambda: F.linear_gated(y, s13), 2.0 * (2048 * W + n * (W + 1024)),
+             4.0 * n * 1024 * W)
+        pw = F.NextRows(rnd(W, dtype=torch.float32))
+        case(f"add_plain_rows_{kind}", lambda: F.add_plain_rows(y, res, 0.7, pw, 1e-6, W), n * W * (2 + 4 + 4 + 2.0))
+        mix = F.Mixture(rows, F.Routes(*[None] * 2, perm, *[None] * 5, 0, 0, 0, wts), y, shared)
+        case(f"add_plain_rows_mixture_{kind}", lambda: F.add_plain_rows(mix, res, 0.7, pw, 1e-6, W),
+             n * W * (2 * top + 2 + 4 + 4 + 2.0))
         # ---- attention over pages: window 1024 + 4 first keys ----
         Hq, G, page, size, keep = 32, 4, 16, 1024, 4
         ctx = 2048 if kind == "decode" else n
@@ -184,6 +226,45 @@ def main():
         case(f"qk_norm_rope_kv_{kind} (like)", lambda: F.qk_norm_rope_kv_(
             xr, nw[:D].contiguous(), nw[:D].contiguous(), pos, inv, slots, kc, vc, Hq, G, D),
             n * (2 * Hq * D + 4 * G * D) * 2.0)
+        # ---- attention with norms per head, partial rotation, window 1024 and a sink ----
+        wd = WA.WindowDims(Hq, G, D, V, 0.088, 1024)
+        wfreq, mag = WA.rotary(64, 1e6, (4.0, 32768, 32.0, 1.0), dev)
+        hq, hk = rnd(D, dtype=torch.float32), rnd(D, dtype=torch.float32)
+        sink, out_a = rnd(Hq, dtype=torch.float32), torch.empty(n, Hq * V, dtype=bf, device=dev)
+        case(f"window_prep_{kind}", lambda: WA.prep(xr, (0, Hq * D, Hq * D), wd, hq, hk, wfreq, mag, pos, slots, kc, vc, 1e-6),
+             n * (2 * Hq * D + 3 * G * D) * 2.0)
+        q4, ctr = q2.view(n, Hq, D), torch.zeros(4096, dtype=torch.int32, device=dev)
+        if kind == "decode":
+            case("window_attention_decode", lambda: WA.attend(q4, kc, vc, m, pt, sink, wd, out_a, 1.0, sl, ctx, ctr),
+                 2.0 * B * 1024 * G * (D + V))
+        else:
+            m.starts, m.lengths = [0], [n]
+            for win in (1024, 0):
+                wd2 = WA.WindowDims(Hq, G, D, V, 0.088, win)
+                pairs = sum(min(i + 1, win or n) for i in range(n))
+                case(f"window_attention_prefill, window {win} (gather and attention)", lambda: WA.attend(
+                    q4, kc, vc, m, pt, sink, wd2, out_a, 1.0, None, n, ctr), None, pairs * Hq * 2.0 * (D + V))
+                cuk = i32([0, n])
+                kx, vx = rnd(n, G * D), rnd(n, G * V)
+                case(f"window_flash_prefill, window {win}", lambda: N.call(
+                    "us_window_flash", N.ptr(q4), Hq * D, N.ptr(kx), G * D, N.ptr(vx), G * V, N.ptr(out_a), Hq * V,
+                    N.ptr(m.cu), N.ptr(cuk), 1, n, n, Hq, G, 2, 128, 128, n, win, 0.088, N.ptr(sink), 1.0, N.stream()),
+                    None, pairs * Hq * 2.0 * (D + V))
+        # ---- linear attention: 16 heads x 128 x 128 with a fixed decay ----
+        fd = SS.fixed_decay_dims(16, 128, 128)
+        fw = {"offs": (0, fd.inner, None), "norm": rnd(fd.inner, dtype=torch.float32),
+              "log_decay": SS.log_decays([1.0 - 2.0 ** -(3 + h / 2) for h in range(16)], dev)}
+        fproj, fu, fy = rnd(n, fd.inner + fd.channels), rnd(n, fd.channels), rnd(n, fd.inner)
+        fpool, fout = torch.zeros(B, 16, 128, 128, **f32), torch.empty(n, fd.inner, dtype=bf, device=dev)
+        fbytes = 2.0 * (B if kind == "decode" else 1) * 16 * 128 * 128 * 4
+        case(f"fixed_decay_scan_{kind}", lambda: SS.state_space_scan(fu, None, None, fw, fpool, m, fd),
+             fbytes + n * (fd.channels + fd.inner) * 2.0)
+        case(f"fixed_decay_silu_{kind}", lambda: SS.short_conv(fproj, fd.inner, None, None, None, m, fd.channels),
+             4.0 * n * fd.channels)
+        case(f"group_norm_sigmoid_{kind}", lambda: SS.group_norm_gate(fy, fproj[:, :fd.inner], fw["norm"], 1, 1e-6, fd.inner,
+                                                                      True), n * fd.inner * 6.0)
+        case(f"fixed_decay_mixer_{kind}", lambda: SS.mixer(fproj, fw, None, fpool, m, fd, 1e-6, fout),
+             fbytes + n * (2 * fd.inner + fd.channels) * 2.0)
         # ---- state space: 64 heads x 64, state 128, 8 groups ----
         d = SS.StateSpaceDims(64, 64, 128, 8, 8, 4)
         Cs, inner = d.channels, d.inner
