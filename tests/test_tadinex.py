@@ -874,6 +874,52 @@ def test_checkpoint_is_served_through_the_registry(tmp_path):
     assert len(out[0]) == 5
 
 
+def test_serve_command_answers_chat_requests(tmp_path):
+    """`serve` on a package that names a checkpoint of the family: the command line picks the model by the
+    checkpoint's architecture; greedy and seeded sampled answers repeat."""
+    import os
+    import socket
+    import time
+    import urllib.request
+    from uniserve_v1_b200.checkpoint.safetensors_io import save_file
+    c = dict(copy.deepcopy(CONFIGS["odd"]), vocab=300)
+    (tmp_path / "m").mkdir()
+    (tmp_path / "m" / "config.json").write_text(json.dumps(c))
+    save_file(weights(c, 2), tmp_path / "m" / "model.safetensors")
+    with socket.socket() as sock:
+        sock.bind(("127.0.0.1", 0))
+        port = sock.getsockname()[1]
+    (tmp_path / "config.toml").write_text(
+        f'model_dir = "{tmp_path / "m"}"\nserved_model_name = "tad"\nmax_model_len = 256\n'
+        f'[admin_config]\nhost = "127.0.0.1"\nport = {port}\n')
+    proc = subprocess.Popen([sys.executable, "-m", "uniserve_v1_b200", "serve", str(tmp_path)], cwd=ROOT,
+                            env=dict(os.environ, UNISERVE_CPU_RANKS="1"))
+    base = f"http://127.0.0.1:{port}"
+
+    def chat(**kw):
+        body = json.dumps(dict({"model": "tad", "max_tokens": 6, "temperature": 0, "ignore_eos": True,
+                                "messages": [{"role": "user", "content": "hello"}]}, **kw)).encode()
+        req = urllib.request.Request(base + "/v1/chat/completions", data=body,
+                                     headers={"Content-Type": "application/json"})
+        with urllib.request.urlopen(req, timeout=60) as r:
+            return json.loads(r.read())
+    try:
+        for _ in range(240):
+            try:
+                urllib.request.urlopen(base + "/health", timeout=5).close()
+                break
+            except Exception:
+                assert proc.poll() is None, "server ended"
+                time.sleep(0.25)
+        for kw in ({}, {"temperature": 0.8, "top_p": 0.9, "seed": 5}):
+            a, b = chat(**kw), chat(**kw)
+            assert a["choices"][0]["message"] == b["choices"][0]["message"]
+            assert a["usage"]["completion_tokens"] == 6
+    finally:
+        proc.terminate()
+        proc.wait(timeout=30)
+
+
 def test_engine_limits_of_recurrent_models():
     """State bytes are accounted; sleep frees the state pools and wake brings empty ones."""
     c, w, model = build("odd", ("cpu", torch.float32))
