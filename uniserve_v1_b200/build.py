@@ -54,6 +54,10 @@ GROUPS = {
                  "sampler.cu", "stream_rows.cu", "vector_delta.cu", "head_delta.cu", "state_space.cu",
                  "state_space_chunk.cu", "window_attn.cu", "latent_flash_tc05.cu", "attn_decode.cu", "attn_decode_tc05.cu"),
                 ("block_manager.cpp",)),
+    "nopuzen": (("runtime.cu", "gemm_tc05.cu", "linear_decode.cu", "gemm_f32.cu", "moe_route.cu", "misc.cu",
+                 "sampler.cu", "stream_rows.cu", "latent_attn.cu", "latent_decode.cu", "latent_flash_tc05.cu",
+                 "window_attn.cu", "sigmoid_decode.cu"),
+                ("block_manager.cpp",)),
 }
 CXX_FLAGS = ["-O3", "-std=c++17", "-fPIC", "-fvisibility=hidden", "-pthread", "-Wall"]
 

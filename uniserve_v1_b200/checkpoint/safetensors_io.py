@@ -181,7 +181,7 @@ FAMILIES = {
     "Qwen4ExpForConditionalGeneration": "qwen4_exp", "Qwen4ExpForCausalLM": "qwen4_exp",
     "MiniMaxH3Pipeline": "minimax_h3", "FastH3Pipeline": "minimax_h3",
     "MiniMaxH3Transformer3DModel": "minimax_h3",
-    "Nepevik": "nepevik", "Zonopel": "zonopel", "Tadinex": "tadinex",
+    "Nepevik": "nepevik", "Zonopel": "zonopel", "Tadinex": "tadinex", "Nopuzen": "nopuzen",
 }
 
 

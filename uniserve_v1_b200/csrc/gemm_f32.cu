@@ -14,9 +14,15 @@ struct F32Args {
   long long ldw, ldx, ldo;
   int w_rows, M, K, rows, act;
   const int *tile_group, *tile_row0, *tile_rows, *num_tiles;
+  float act_a, act_b;
 };
 
-__device__ __forceinline__ float act_f(float x, int act) {
+__device__ __forceinline__ float act_f(float x, int act, float a, float b) {
+  if (act == 5) {
+    x = fmaxf(x, 0.f);
+    return x * x;
+  }
+  if (act == 6) return fmaf(x > 0.f ? a * x : b, x > 0.f ? x : expm1f(x) - x, 0.5f * x);
   return act == 3 ? 0.5f * x * (1.f + erff(x * 0.70710678118654752f)) : x;
 }
 
@@ -69,7 +75,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const F32Args a) {
       for (int j = 0; j < 4; ++j) {
         const int m = m0 + tx * 4 + j;
         if (m >= a.M) continue;
-        a.out[(long long)r * a.ldo + m] = act_f(acc[i][j] + (a.bias ? a.bias[m] : 0.f), a.act);
+        a.out[(long long)r * a.ldo + m] = act_f(acc[i][j] + (a.bias ? a.bias[m] : 0.f), a.act, a.act_a, a.act_b);
       }
     }
   }
@@ -100,18 +106,20 @@ US_API int us_clamped_glu_f32(const float* z, float* out, int rows, int I, float
   return US_OK;
 }
 
-// Same operand conventions as us_gemm_wx; act: 0 none, 3 gelu (erf).
+// Same operand conventions as us_gemm_wx; act: 0 none, 3 gelu (erf), 5 square of relu, 6 xIELU (act_a,
+// act_b).
 US_API int us_gemm_f32(const float* W, const float* X, float* out, int G, int w_rows, int M, int K,
                        int x_rows, long long ldw, long long ldx, long long ldo, int act,
-                       const float* bias, const int* tile_group, const int* tile_row0,
+                       float act_a, float act_b, const float* bias, const int* tile_group, const int* tile_row0,
                        const int* tile_rows, const int* num_tiles, int max_tiles, void* stream_) {
-  US_REQUIRE(W && X && out && G >= 1 && M >= 1 && K >= 1 && x_rows >= 0 && (act == 0 || act == 3));
+  US_REQUIRE(W && X && out && G >= 1 && M >= 1 && K >= 1 && x_rows >= 0 &&
+             (act == 0 || act == 3 || act == 5 || act == 6));
   US_REQUIRE(!num_tiles || (tile_group && tile_row0 && tile_rows && max_tiles >= 1 && !bias));
   if (x_rows == 0) return US_OK;
   const int tiles = num_tiles ? max_tiles : (x_rows + kT - 1) / kT;
   US_REQUIRE(tiles <= 65535);
   F32Args a{W, X, bias, out, ldw, ldx, ldo, w_rows, M, K, x_rows, act, tile_group, tile_row0,
-            tile_rows, num_tiles};
+            tile_rows, num_tiles, act_a, act_b};
   US_CUDA_CHECK(us::launch_pdl(gemm_f32_kernel, dim3((M + kT - 1) / kT, tiles), dim3(256), 0,
                                (cudaStream_t)stream_, a));
   return US_OK;

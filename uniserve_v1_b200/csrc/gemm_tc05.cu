@@ -23,7 +23,7 @@
 
 namespace {
 
-template <int BN, bool DUAL, bool GELU>
+template <int BN, bool DUAL, bool ACT>
 __global__ void __launch_bounds__(192)
 gemm_wx_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ BMaps tmBs,
                const GemmArgs args) {
@@ -194,7 +194,7 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
         }
       } else {
         // The pipeline stages are idle: their first 16 KiB stage the stores.
-        Epilogue<DUAL, GELU> epi(args, group, m_tile * kBlockM, ml, row0);
+        Epilogue<DUAL, ACT> epi(args, group, m_tile * kBlockM, ml, row0);
         int chunk = 0;
 #pragma unroll 1
         for (int c = 0; c < BN; c += 16, ++chunk) {
@@ -218,7 +218,7 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
       const int q = warp & 3;
       const int ml = q * 32 + lane;
       const uint32_t my_rank = tc::cluster_ctarank();
-      Epilogue<false, GELU> epi(args, group, m_tile * kBlockM, ml, row0);
+      Epilogue<false, ACT> epi(args, group, m_tile * kBlockM, ml, row0);
       const uint32_t local = tc::smem_u32(smem) + (uint32_t)ml * 4u;
       for (int r = (int)my_rank; r < nrows; r += args.splits) {
         float acc = 0.f;
@@ -469,7 +469,7 @@ __device__ __forceinline__ void swapped_tile(int t, int m_pairs, int n_tiles, in
 // per CTA) and every epilogue thread owns one activation row, whose features it
 // stores from registers as 32-byte pieces - no staging tile, and every destination
 // (plain, row-mapped, a peer's buffer by feature block or by row interval, the
-// token owner's combine buffer) is one pointer per thread.  SWAP = 2 (dense; 3: with gelu): the
+// token owner's combine buffer) is one pointer per thread.  SWAP = 2 (dense; 3: with an activation): the
 // other side is 256 weight rows, 128 per CTA.  SWAP = 1 (gated): 128 value rows in
 // the even CTA and the matching 128 gate rows in the odd CTA, so one N = 256
 // instruction produces both halves and a thread finds value j in column j and its
@@ -721,6 +721,7 @@ gemm_wx_pair_kernel(const __grid_constant__ CUtensorMap tmA,
                                     : xrow < args.rows;
         const int f0 = nt * kFeat;
         const int act = args.act;
+        const float act_a = args.act_a, act_b = args.act_b;
         const int esz = args.out_dtype == 0 ? 2 : 4;
         const int M = args.M;
         const bool vec = args.vec_store != 0;
@@ -791,7 +792,7 @@ gemm_wx_pair_kernel(const __grid_constant__ CUtensorMap tmA,
           }
           if (SWAP == 3) {
 #pragma unroll
-            for (int j = 0; j < 16; ++j) x[j] = gelu_erf_f(x[j]);
+            for (int j = 0; j < 16; ++j) x[j] = act_single_f(x[j], act, act_a, act_b);
           }
           if (lines) {
             const int ch = (c & 63) >> 3;     // first of this piece's two 16-byte chunks
@@ -972,7 +973,7 @@ int launch_persist(const CUtensorMap& tmA, const BMaps& tmB, GemmArgs a, int til
 // Live CTAs expected of the next grouped launch of this thread (us_gemm_wx_hint); 0 = none.
 thread_local int g_cta_hint = 0;
 
-template <int BN, bool DUAL, bool GELU = false>
+template <int BN, bool DUAL, bool ACT = false>
 int launch(const CUtensorMap& tmA, const BMaps& tmB, GemmArgs a, int m_tiles, int n_tiles,
            cudaStream_t stream) {
   constexpr int kBTile = BN * kBlockK * 2;
@@ -1040,7 +1041,7 @@ int launch(const CUtensorMap& tmA, const BMaps& tmB, GemmArgs a, int m_tiles, in
   const size_t smem = (size_t)stages * kStageBytes + (2 * stages + 1) * 8 + 16 + 1024;
   static bool configured = false;
   if (!configured) {
-    US_CUDA_CHECK(cudaFuncSetAttribute(gemm_wx_kernel<BN, DUAL, GELU>,
+    US_CUDA_CHECK(cudaFuncSetAttribute(gemm_wx_kernel<BN, DUAL, ACT>,
                                        cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
     configured = true;
   }
@@ -1061,7 +1062,7 @@ int launch(const CUtensorMap& tmA, const BMaps& tmB, GemmArgs a, int m_tiles, in
   attr[1].val.programmaticStreamSerializationAllowed = us::pdl_enabled() ? 1 : 0;
   cfg.attrs = attr;
   cfg.numAttrs = 2;
-  US_CUDA_CHECK(cudaLaunchKernelEx(&cfg, gemm_wx_kernel<BN, DUAL, GELU>, tmA, tmB, a));
+  US_CUDA_CHECK(cudaLaunchKernelEx(&cfg, gemm_wx_kernel<BN, DUAL, ACT>, tmA, tmB, a));
   return US_OK;
 }
 
@@ -1103,6 +1104,7 @@ struct PeerSpec {
   int peer_rows = 0;                     // reduce-scatter: rows owned per rank
   int peer_slot = 0;
   float glu_limit = 0.f, glu_alpha = 0.f;  // dual products with act 4
+  float act_a = 0.f, act_b = 0.f;          // single products with act 6
 };
 
 int gemm_impl(const void* W, const void* X, void* out, int G, int w_rows, int M, int K, int x_rows,
@@ -1119,9 +1121,9 @@ int gemm_impl(const void* W, const void* X, void* out, int G, int w_rows, int M,
   if (num_tiles) US_REQUIRE(tile_group && tile_row0 && tile_rows && max_tiles >= 1);
 
   // Dense problems of more than one wave run on CTA pairs (US_GEMM_PAIR=0: single CTAs).
-  const bool gelu = !dual && act == 3;    // single-CTA and swapped kernels only
-  US_REQUIRE(dual || act == 0 || gelu);
-  const bool pair = pair_enabled() && (!gelu || pair_mode() == 1) && num_tiles == nullptr && G == 1 && !ps.x_peers &&
+  const bool with_act = !dual && act != 0;   // single-CTA and swapped kernels only
+  US_REQUIRE(dual || act == 0 || act == 3 || act == 5 || act == 6);
+  const bool pair = pair_enabled() && (!with_act || pair_mode() == 1) && num_tiles == nullptr && G == 1 && !ps.x_peers &&
                     (K % kBlockK) == 0 &&
                     (dual ? block_n == 128 : block_n == 256) &&
                     (long long)((M + kBlockM - 1) / kBlockM) * ((x_rows + block_n - 1) / block_n) >
@@ -1222,6 +1224,8 @@ int gemm_impl(const void* W, const void* X, void* out, int G, int w_rows, int M,
   a.scale_first = 0;
   a.glu_limit = ps.glu_limit;
   a.glu_alpha = ps.glu_alpha;
+  a.act_a = ps.act_a;
+  a.act_b = ps.act_b;
   if (ps.route_map) {
     US_REQUIRE(ps.out_peers && ps.route_w && ps.route_per > 0 && ps.n_out_peers >= 1 &&
                ps.n_out_peers <= 8 && out_dtype == 0);
@@ -1279,7 +1283,7 @@ int gemm_impl(const void* W, const void* X, void* out, int G, int w_rows, int M,
     const int x_pairs = gpair ? max_tiles : ((x_rows + kBlockM - 1) / kBlockM + 1) / 2;
     if (dual)
       return launch_pair<256, false, false, 1>(tmA, tmB, a, x_pairs * ((M + 127) / 128), stream);
-    if (gelu) return launch_pair<256, false, false, 3>(tmA, tmB, a, x_pairs * ((M + 255) / 256), stream);
+    if (with_act) return launch_pair<256, false, false, 3>(tmA, tmB, a, x_pairs * ((M + 255) / 256), stream);
     return launch_pair<256, false, false, 2>(tmA, tmB, a, x_pairs * ((M + 255) / 256), stream);
   }
   if (pair) {
@@ -1287,7 +1291,7 @@ int gemm_impl(const void* W, const void* X, void* out, int G, int w_rows, int M,
     if (dual) return launch_pair<128, true>(tmA, tmB, a, pair_tiles, stream);
     return launch_pair<256, false>(tmA, tmB, a, pair_tiles, stream);
   }
-  if (!no_persist && !gelu && num_tiles == nullptr && G == 1 && m_tiles * n_tiles > 148 &&
+  if (!no_persist && !with_act && num_tiles == nullptr && G == 1 && m_tiles * n_tiles > 148 &&
       (dual ? block_n == 128 : (block_n == 128 || block_n == 256))) {
     const int tiles = m_tiles * n_tiles;
     if (dual) return launch_persist<128, true>(tmA, tmB, a, tiles, stream);
@@ -1297,7 +1301,7 @@ int gemm_impl(const void* W, const void* X, void* out, int G, int w_rows, int M,
 #define US_GEMM_CASE(BN)                                                              \
   case BN:                                                                            \
     return dual   ? launch<BN, true>(tmA, tmB, a, m_tiles, n_tiles, stream)             \
-           : gelu ? launch<BN, false, true>(tmA, tmB, a, m_tiles, n_tiles, stream)      \
+           : with_act ? launch<BN, false, true>(tmA, tmB, a, m_tiles, n_tiles, stream)      \
                   : launch<BN, false>(tmA, tmB, a, m_tiles, n_tiles, stream);
   switch (block_n) {
     US_GEMM_CASE(16)
@@ -1335,6 +1339,19 @@ US_API int us_gemm_wx(const void* W, const void* X, void* out, int G, int w_rows
   return gemm_impl(W, X, out, G, w_rows, M, K, x_rows, ldw, ldx, ldo, dual, dual_offset, act,
                    out_dtype, bias, bias_dtype, row_scale, out_row_map, tile_group, tile_row0,
                    tile_rows, num_tiles, max_tiles, block_n, ps, (cudaStream_t)stream_);
+}
+
+// Single product with an activation of two constants; dense, or grouped over a tile list.  bf16 out.
+US_API int us_gemm_wx_act(const void* W, const void* X, void* out, int G, int w_rows, int M, int K,
+                          int x_rows, long long ldw, long long ldx, long long ldo, int act, float act_a,
+                          float act_b, const int* tile_group, const int* tile_row0,
+                          const int* tile_rows, const int* num_tiles, int max_tiles, int block_n,
+                          void* stream_) {
+  PeerSpec ps;
+  ps.act_a = act_a;
+  ps.act_b = act_b;
+  return gemm_impl(W, X, out, G, w_rows, M, K, x_rows, ldw, ldx, ldo, 0, 0, act, 0, nullptr, 0, nullptr, nullptr,
+                   tile_group, tile_row0, tile_rows, num_tiles, max_tiles, block_n, ps, (cudaStream_t)stream_);
 }
 
 // Gated product out = (clamp(first) + 1) g sigmoid(alpha g), g = min(second, limit), first clamped to

@@ -33,6 +33,11 @@ __device__ __forceinline__ unsigned long long add2(unsigned long long a, unsigne
   asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
   return d;
 }
+__device__ __forceinline__ unsigned long long mul2(unsigned long long a, unsigned long long b) {
+  unsigned long long d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
 // tcgen05.mma with the shared-memory descriptors given as (low, high) words.  The thread that
 // issues the products is a single instruction stream: with 64 cycles of tensor work per
 // 128 x 128 x 16 product, a dozen dependent instructions of 64-bit descriptor arithmetic per

@@ -16,7 +16,8 @@ struct GemmArgs {
   int early;        // dense: weight tiles of the first stages are fetched before the PDL wait
   int act;          // dual: 0 = silu fused rounding, 1 = silu stepwise rounding, 2 = gelu-tanh,
                     //       4 = clamped (glu_limit, glu_alpha)
-                    // single: 0 = none, 3 = gelu (erf) of the biased value
+                    // single: 0 = none; of the biased value 3 = gelu (erf), 5 = square of relu,
+                    //       6 = xIELU (act_a, act_b)
   int out_dtype;    // 0 = bf16, 1 = fp32
   int bias_dtype;   // 0 = bf16, 1 = fp32
   long long ldo;
@@ -71,6 +72,7 @@ struct GemmArgs {
   // (collected per warp in the staging area) instead of 32-byte pieces per thread.
   int remote_lines;
   float glu_limit, glu_alpha;
+  float act_a, act_b;
 };
 
 struct BMaps {
@@ -98,6 +100,20 @@ __device__ __forceinline__ float gelu_erf_f(float x) {
   return 0.5f * x * (1.f + erff(x * 0.70710678118654752f));
 }
 
+// a x^2 + x / 2 above zero, b (e^x - 1 - x) + x / 2 below
+__device__ __forceinline__ float xielu_f(float x, float a, float b) {
+  return fmaf(x > 0.f ? a * x : b, x > 0.f ? x : __expf(x) - 1.f - x, 0.5f * x);
+}
+
+// activations of a single product (`act` of GemmArgs)
+__device__ __forceinline__ float act_single_f(float x, int act, float a, float b) {
+  if (act == 5) {
+    x = fmaxf(x, 0.f);
+    return x * x;
+  }
+  return act == 6 ? xielu_f(x, a, b) : gelu_erf_f(x);
+}
+
 template <int BN>
 constexpr int tmem_cols(bool dual) {
   int need = dual ? 2 * BN : BN;
@@ -114,9 +130,9 @@ constexpr int kEpiStageBytes = 16 * 1024;   // two staging tiles of 16 rows x 12
 // so that every row leaves as contiguous 16-byte pieces (256 B per row for bf16)
 // whatever the destination: the plain output, a row-mapped output, a peer's buffer
 // (scatter by feature, reduce-scatter by row) or the token owner's combine buffer.
-// GELU: gelu (erf) of the biased value, a form of its own so that the other products' epilogues
-// do not carry its code.
-template <bool DUAL, bool GELU = false>
+// ACT: an activation of the biased value (act_single_f), a form of its own so that the other products'
+// epilogues do not carry its code.
+template <bool DUAL, bool ACT = false>
 struct Epilogue {
   // Everything the per-element code needs is copied out of the argument block
   // once: the block lives in parameter memory, and reading it per element (after
@@ -124,7 +140,7 @@ struct Epilogue {
   // branches per value - 3,300 clocks per 16-row chunk, more than the mainloop.
   const int m0, ml, m, row0;
   const bool m_ok;
-  const float glu_limit, glu_alpha;
+  const float glu_limit, glu_alpha, act_a, act_b;
   float bias;
   char* tile_base;     // element (row0, m0) of the destination; null = per-row lookup
   long long row_bytes;
@@ -140,7 +156,7 @@ struct Epilogue {
   const GemmArgs& a;         // rare paths only (the peer table of the route push)
   __device__ __forceinline__ Epilogue(const GemmArgs& args, int group, int m0_, int ml_, int row0_)
       : m0(m0_), ml(ml_), m(m0_ + ml_), row0(row0_), m_ok(m0_ + ml_ < args.M),
-        glu_limit(args.glu_limit), glu_alpha(args.glu_alpha), bias(0.f),
+        glu_limit(args.glu_limit), glu_alpha(args.glu_alpha), act_a(args.act_a), act_b(args.act_b), bias(0.f),
         tile_base(nullptr), row_bytes(0), esz(args.out_dtype == 0 ? 2 : 4), M(args.M),
         act(args.act), route_per(args.route_per), vec_store(args.vec_store), ldo(args.ldo),
         scale_rows(args.row_scale ? args.row_scale + row0_ : nullptr),
@@ -188,7 +204,7 @@ struct Epilogue {
       }
     }
     val += bias;
-    if (GELU) val = gelu_erf_f(val);
+    if (ACT) val = act_single_f(val, act, act_a, act_b);
     if (route_rows != nullptr) return val * route_w[route_rows[r]];
     if (scale_rows != nullptr && !scale_first) val *= scale_rows[r];
     return val;
@@ -231,7 +247,7 @@ struct Epilogue {
     }
     const uint32_t buf = tc::smem_u32(stage) + (uint32_t)(chunk & 1) * (kEpiStageBytes / 2);
     // fast path: nothing per row but the gated activation and the bias
-    const bool plain = scale_rows == nullptr && route_rows == nullptr && !GELU;
+    const bool plain = scale_rows == nullptr && route_rows == nullptr && !ACT;
     if (esz == 2) {
 #pragma unroll
       for (int j = 0; j < 16; ++j) {

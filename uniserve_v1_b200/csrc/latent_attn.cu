@@ -7,10 +7,11 @@
 //
 //   us_latent_prep              norms of the query and key latents, rotation of the key part, pages
 //   us_rotate_heads             rotation of the queries' rotated parts, in place
-//   us_head_linear              a product per head: out[t, h] = W_h x[t, h]
+//   us_head_linear              a product per head: out[t, h] = W_h x[t, h], also times sigmoid(gate[t, h])
 //   us_latent_attention_rows    any sizes, bf16 or FP32: one CTA per (query row, up to 16 heads)
 //
-// Channel 2i turns with channel 2i + 1.  The angle is formed and reduced to a fraction of a turn in
+// Channel 2i turns with channel 2i + 1 or, in halves, i with i + pairs; cosine and sine carry a factor.
+// The angle is formed and reduced to a fraction of a turn in
 // FP64, so far positions lose nothing before the FP32 sine and cosine.
 #include "include/us_common.cuh"
 #include "include/us_mma.cuh"
@@ -53,6 +54,8 @@ struct LatentPrep {
   int ldc, ldr;
   float eps;
   int bf16;
+  float mag;
+  int halves;
 };
 
 __global__ void __launch_bounds__(kPrepThreads) latent_prep_kernel(const LatentPrep a) {
@@ -87,26 +90,26 @@ __global__ void __launch_bounds__(kPrepThreads) latent_prep_kernel(const LatentP
   for (int c = tid; c < a.nc; c += kPrepThreads)
     st1(a.cpages, slot * a.ldc + c, a.bf16, ld1(a.x, base + a.off_c + c, a.bf16) * ic * a.wc[c]);
   const int pos = a.pos[t];
-  for (int i = tid; i < (a.nr + 1) / 2; i += kPrepThreads) {
-    float u = ld1(a.x, base + a.off_r + 2 * i, a.bf16);
-    float v = 2 * i + 1 < a.nr ? ld1(a.x, base + a.off_r + 2 * i + 1, a.bf16) : 0.f;
-    if (i < a.pairs) {
-      float c, s;
-      turn(pos, a.freq[i], c, s);
-      const float u1 = u * c - v * s;
-      v = v * c + u * s;
-      u = u1;
-    }
-    st1(a.rpages, slot * a.ldr + 2 * i, a.bf16, u);
-    if (2 * i + 1 < a.nr) st1(a.rpages, slot * a.ldr + 2 * i + 1, a.bf16, v);
+  const long long from = base + a.off_r, to = slot * a.ldr;
+  for (int i = tid; i < a.pairs; i += kPrepThreads) {
+    const int p = a.halves ? i : 2 * i, q = a.halves ? i + a.pairs : 2 * i + 1;
+    const float u = ld1(a.x, from + p, a.bf16), v = ld1(a.x, from + q, a.bf16);
+    float c, s;
+    turn(pos, a.freq[i], c, s);
+    c *= a.mag;
+    s *= a.mag;
+    st1(a.rpages, to + p, a.bf16, u * c - v * s);
+    st1(a.rpages, to + q, a.bf16, v * c + u * s);
   }
+  for (int i = 2 * a.pairs + tid; i < a.nr; i += kPrepThreads)
+    st1(a.rpages, to + i, a.bf16, ld1(a.x, from + i, a.bf16));
 }
 
 // x [T, ldx]: head h's pairs start at column off + h * hs.  A thread per (pair, group of heads).
 __global__ void __launch_bounds__(256)
 rotate_heads_kernel(void* __restrict__ x, long long ldx, int off, int hs, int H,
                     const double* __restrict__ freq, int pairs, const int* __restrict__ pos,
-                    long long total, int bf16) {
+                    long long total, int bf16, float mag, int halves) {
   US_PDL_PROLOGUE();
   const long long e = (long long)blockIdx.x * 256 + threadIdx.x;
   if (e >= total) return;
@@ -117,11 +120,14 @@ rotate_heads_kernel(void* __restrict__ x, long long ldx, int off, int hs, int H,
   const long long t = r / groups;
   float c, s;
   turn(pos[t], freq[i], c, s);
+  c *= mag;
+  s *= mag;
+  const int p = halves ? i : 2 * i, gap = halves ? pairs : 1;
   for (int h = h0; h < min(H, h0 + 4); ++h) {
-    const long long at = t * ldx + off + (long long)h * hs + 2 * i;
-    const float u = ld1(x, at, bf16), v = ld1(x, at + 1, bf16);
+    const long long at = t * ldx + off + (long long)h * hs + p;
+    const float u = ld1(x, at, bf16), v = ld1(x, at + gap, bf16);
     st1(x, at, bf16, u * c - v * s);
-    st1(x, at + 1, bf16, v * c + u * s);
+    st1(x, at + gap, bf16, v * c + u * s);
   }
 }
 
@@ -131,7 +137,16 @@ struct HeadLinear {
   void* out;
   long long hsw, ldw, ldx, hsx, ldo, hso;
   int H, M, K, rows;
+  const void* gate;           // or null: feature m of head h at column h M + m, rows at ldg
+  long long ldg;
+  const int* gate_rows;       // row of `gate` for every row of X, or null: the same
 };
+
+__device__ __forceinline__ float gated(const HeadLinear& a, float v, int h, int r, int m, int bf16) {
+  if (!a.gate) return v;
+  const long long row = a.gate_rows ? a.gate_rows[r] : r;
+  return v / (1.f + expf(-ld1(a.gate, row * a.ldg + (long long)h * a.M + m, bf16)));
+}
 
 __global__ void __launch_bounds__(256) head_linear_f32_kernel(const HeadLinear a) {
   US_PDL_PROLOGUE();
@@ -164,7 +179,8 @@ __global__ void __launch_bounds__(256) head_linear_f32_kernel(const HeadLinear a
 #pragma unroll
     for (int j = 0; j < 4; ++j)
       if (r0 + ty * 4 + i < a.rows && m0 + tx * 4 + j < a.M)
-        out[(long long)(r0 + ty * 4 + i) * a.ldo + m0 + tx * 4 + j] = acc[i][j];
+        out[(long long)(r0 + ty * 4 + i) * a.ldo + m0 + tx * 4 + j] =
+            gated(a, acc[i][j], h, r0 + ty * 4 + i, m0 + tx * 4 + j, 0);
 }
 
 // 64 rows x 64 features of one head; a warp takes 16 rows.  K in steps of 64, the next step's
@@ -218,11 +234,13 @@ __global__ void __launch_bounds__(128) head_linear_kernel(const HeadLinear a) {
       const int r = r0 + warp * 16 + (lane >> 2) + e * 8, m = m0 + n * 8 + (lane & 3) * 2;
       if (r >= a.rows || m >= a.M) continue;
       __nv_bfloat16* o = out + (long long)r * a.ldo + m;
-      if (pairs && m + 1 < a.M) {
-        *reinterpret_cast<__nv_bfloat162*>(o) = __floats2bfloat162_rn(acc[n][e * 2], acc[n][e * 2 + 1]);
+      const bool both = m + 1 < a.M;
+      const float v0 = gated(a, acc[n][e * 2], h, r, m, 1), v1 = both ? gated(a, acc[n][e * 2 + 1], h, r, m + 1, 1) : 0.f;
+      if (pairs && both) {
+        *reinterpret_cast<__nv_bfloat162*>(o) = __floats2bfloat162_rn(v0, v1);
       } else {
-        o[0] = us::f2bf(acc[n][e * 2]);
-        if (m + 1 < a.M) o[1] = us::f2bf(acc[n][e * 2 + 1]);
+        o[0] = us::f2bf(v0);
+        if (both) o[1] = us::f2bf(v1);
       }
     }
 }
@@ -321,33 +339,37 @@ __global__ void __launch_bounds__(kRowThreads) latent_rows_kernel(const LatentAt
 US_API int us_latent_prep(void* x, long long ldx, int off_q, int off_c, int off_r, int nq, int nc,
                           int nr, const float* wq, const float* wc, const double* freq, int pairs,
                           const int* pos, const int* slots, void* cpages, int ldc, void* rpages,
-                          int ldr, int T, float eps, int bf16, void* stream_) {
+                          int ldr, int T, float eps, float mag, int halves, int bf16, void* stream_) {
   US_REQUIRE(x && wq && wc && pos && slots && cpages && rpages && T >= 0 && nq >= 1 && nc >= 1 &&
              nr >= 0 && ldc >= nc && ldr >= nr && 2 * pairs <= nr && (pairs == 0 || freq));
   if (T == 0) return US_OK;
   LatentPrep a{x, ldx, off_q, off_c, off_r, nq, nc, nr, pairs, wq, wc, freq, pos, slots, cpages,
-               rpages, ldc, ldr, eps, bf16};
+               rpages, ldc, ldr, eps, bf16, mag, halves};
   US_CUDA_CHECK(us::launch_pdl(latent_prep_kernel, dim3(T), dim3(kPrepThreads), 0,
                                (cudaStream_t)stream_, a));
   return US_OK;
 }
 
 US_API int us_rotate_heads(void* x, long long ldx, int off, int hs, int H, const double* freq,
-                           int pairs, const int* pos, int T, int bf16, void* stream_) {
+                           int pairs, const int* pos, int T, float mag, int halves, int bf16,
+                           void* stream_) {
   US_REQUIRE(x && freq && pos && T >= 0 && H >= 1 && pairs >= 1);
   const long long total = (long long)T * ((H + 3) / 4) * pairs;
   if (total == 0) return US_OK;
   US_CUDA_CHECK(us::launch_pdl(rotate_heads_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0,
-                               (cudaStream_t)stream_, x, ldx, off, hs, H, freq, pairs, pos, total, bf16));
+                               (cudaStream_t)stream_, x, ldx, off, hs, H, freq, pairs, pos, total, bf16, mag, halves));
   return US_OK;
 }
 
+// gate (or null) [.., H M] rows at ldg: the result times its sigmoid; gate_rows (or null): its row for every
+// row of X.
 US_API int us_head_linear(const void* W, const void* X, void* out, long long hsw, long long ldw,
                           long long ldx, long long hsx, long long ldo, long long hso, int H, int M,
-                          int K, int rows, int bf16, void* stream_) {
+                          int K, int rows, const void* gate, long long ldg, const int* gate_rows,
+                          int bf16, void* stream_) {
   US_REQUIRE(W && X && out && H >= 1 && M >= 1 && K >= 1 && rows >= 0 && H <= 65535);
   if (rows == 0) return US_OK;
-  HeadLinear a{W, X, out, hsw, ldw, ldx, hsx, ldo, hso, H, M, K, rows};
+  HeadLinear a{W, X, out, hsw, ldw, ldx, hsx, ldo, hso, H, M, K, rows, gate, ldg, gate_rows};
   const dim3 grid(us::ceil_div(M, 64), us::ceil_div(rows, 64), H);
   if (bf16) {
     US_REQUIRE((K % 8) == 0 && (ldw % 8) == 0 && (hsw % 8) == 0 && (ldx % 8) == 0 && (hsx % 8) == 0 &&

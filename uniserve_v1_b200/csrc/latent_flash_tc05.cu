@@ -6,6 +6,7 @@
 //                       into packed rows (sequence by sequence, oldest first)
 //   us_latent_flash     score = q_unrotated . k_head + q_rotated . k_shared, window, softmax, values
 //   us_window_flash     score = q . k, grouped heads, window, softmax with a sink, values
+//   us_sigmoid_flash    the same with a key's weight the sigmoid of its capped and shifted score (no softmax)
 //
 // The flash kernel is the two-tile scheme of flash_attn2_tc05.cu with unlike operands: a CTA owns 256
 // query rows of one (sequence, head) as tiles A and B; keys come in blocks of 128 as one or two
@@ -13,7 +14,8 @@
 // all heads share.
 // Where 192-wide keys leave no room for two value stages there is one; the block of values is then
 // fetched while the tensor pipe forms the next scores.  Blocks outside a tile's window are skipped.
-// Every wait is bounded.
+// Without a softmax there is neither a maximum nor a sum: weights go straight into the value product, whose
+// accumulator is never rescaled.  Every wait is bounded.
 #include "include/us_common.cuh"
 #include "include/us_flash.cuh"
 #include "include/us_mma.cuh"
@@ -96,11 +98,32 @@ struct FlashArgs {
   int rep;                               // query heads per key / value head
   const float* sink;                     // [H] or null: exp(sink) joins the softmax denominator
   float out_scale;
+  // or null: the output times the sigmoid of column h * gate_cols + (column of the head) % gate_cols of
+  // the row (gate_cols 1: a logit per head, V: one per column)
+  const __nv_bfloat16* gate;
+  long long ldg;
+  int gate_cols;
+  // sigmoid form: z = score * scale * temp / cap, weight = sigmoid(cap * tanh(z) + shift)
+  const float *temp, *shift;             // [H]
+  float scale, cap;
 };
 
+__device__ __forceinline__ float rcpf(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+// tanh(z) / z as a polynomial in u = z^2, u <= 1/4 (least maximum error, 1.3e-8)
+constexpr float kTanhMost = 0.5f;
+constexpr float kT1 = -0.33333075046539307f, kT2 = 0.13324907422065735f, kT3 = -0.05299423262476921f,
+                kT4 = 0.017151299864053726f;
+
+__device__ __forceinline__ float sigmoid_of(__nv_bfloat16 x) { return 1.f / (1.f + __expf(-us::bf2f(x))); }
+
 // kN: 64-channel slabs of the head's own keys; kR: slabs of the shared part (0 or 1); kDV: value
-// width; kVS: value stages.
-template <int kN, int kR, int kDV, int kVS>
+// width; kVS: value stages; kSig: sigmoid weights.
+template <int kN, int kR, int kDV, int kVS, bool kSig>
 __global__ void __launch_bounds__(320, 1)
 latent_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                     const __grid_constant__ CUtensorMap tmR, const __grid_constant__ CUtensorMap tmV,
@@ -287,6 +310,8 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     const int q_idx = q0 + x * kBM + r;
     const int j0 = x ? jb[1] : jb[0], j1 = x ? je[1] : je[0];
     float m_used = -INFINITY, l_sum = 0.f;
+    const float f_z = kSig ? a.scale * a.temp[h] / a.cap : 0.f;
+    const float f_cap = -a.cap * 1.4426950408889634f, f_shift = kSig ? -a.shift[h] * 1.4426950408889634f : 0.f;
     bool ok = true;
     for (int j = j0; j < j1; ++j) {
       ok = __all_sync(0xffffffffu, tc::mbar_wait(&s_full[x], (uint32_t)(j - j0) & 1u, abort_flag));
@@ -301,6 +326,60 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       for (int c = 0; c < 4; ++c)
         tc::tmem_ld32(s_tmem + 32 * c, *reinterpret_cast<uint32_t(*)[32]>(v + 32 * c));
       tc::tmem_ld_wait();
+      if constexpr (kSig) {
+        uint32_t pk[kBN / 2];
+        float tops[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+        for (int i = 0; i < 32; ++i)
+#pragma unroll
+          for (int c = 0; c < 4; ++c) tops[c] = fmaxf(tops[c], fabsf(__uint_as_float(v[32 * c + i])));
+        const float top = fmaxf(fmaxf(tops[0], tops[1]), fmaxf(tops[2], tops[3]));
+        const unsigned long long f2 = pack2(f_z, f_z), sh2 = pack2(f_shift, f_shift), one2 = pack2(1.f, 1.f);
+        // two exponents (base 2) of the negated argument -> two weights with one reciprocal
+        auto weigh = [&](float x0, float x1, int at) {
+          const float u0 = ex2f(fminf(x0, 60.f)), u1 = ex2f(fminf(x1, 60.f));
+          float a0, a1;
+          unpack2(add2(pack2(u0, u1), one2), a0, a1);
+          const float r = rcpf(a0 * a1);
+          pk[at] = us::pack_bf(r * a1, r * a0);
+        };
+        if (__all_sync(0xffffffffu, top * fabsf(f_z) <= kTanhMost)) {
+          const unsigned long long c2 = pack2(f_cap, f_cap);
+#pragma unroll
+          for (int i = 0; i < kBN; i += 2) {
+            const unsigned long long z = mul2(pack2(__uint_as_float(v[i]), __uint_as_float(v[i + 1])), f2);
+            const unsigned long long u = mul2(z, z);
+            unsigned long long p = fma2(pack2(kT4, kT4), u, pack2(kT3, kT3));
+            p = fma2(fma2(p, u, pack2(kT2, kT2)), u, pack2(kT1, kT1));
+            p = fma2(p, u, one2);
+            float x0, x1;
+            unpack2(fma2(mul2(z, c2), p, sh2), x0, x1);
+            weigh(x0, x1, i >> 1);
+          }
+        } else {
+          const float f_e = 2.8853900817779268f * f_z;       // e^{2 z} = 2^{score f_e}
+#pragma unroll
+          for (int i = 0; i < kBN; i += 2) {                  // tanh(z) = 1 - 2 / (e^{2 z} + 1)
+            const float t0 = fmaf(-2.f, rcpf(ex2f(__uint_as_float(v[i]) * f_e) + 1.f), 1.f);
+            const float t1 = fmaf(-2.f, rcpf(ex2f(__uint_as_float(v[i + 1]) * f_e) + 1.f), 1.f);
+            weigh(fmaf(t0, f_cap, f_shift), fmaf(t1, f_cap, f_shift), i >> 1);
+          }
+        }
+        if (lim < kBN || low > 0) {
+#pragma unroll
+          for (int i = 0; i < kBN; i += 2) {
+            if (i >= lim || i < low) pk[i >> 1] &= 0xffff0000u;
+            if (i + 1 >= lim || i + 1 < low) pk[i >> 1] &= 0x0000ffffu;
+          }
+        }
+#pragma unroll
+        for (int c = 0; c < 2; ++c)
+          tc::tmem_st32(s_tmem + 32 * c, *reinterpret_cast<const uint32_t(*)[32]>(pk + 32 * c));
+        tc::tmem_st_wait();
+        tc::tc_fence_before_sync();
+        tc::mbar_arrive(&p_full[x]);
+        continue;
+      }
       if (lim < kBN || low > 0) {
 #pragma unroll
         for (int i = 0; i < kBN; ++i)
@@ -365,9 +444,17 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       if (ok && tc::mbar_wait(&o_full[x], 0, abort_flag)) {
         tc::tc_fence_after_sync();
         if (a.sink && l_sum > 0.f) l_sum += ex2f(a.sink[h] * 1.4426950408889634f - m_used);
-        const float inv = l_sum > 0.f ? a.out_scale / l_sum : 0.f;
+        float inv = kSig ? a.out_scale : l_sum > 0.f ? a.out_scale / l_sum : 0.f;
         const bool row_ok = q_idx < q_len, wide = ((a.V | (int)a.ldo) & 7) == 0;
         __nv_bfloat16* orow = a.out + (long long)(q_start + q_idx) * a.ldo + (long long)h * a.V;
+        const __nv_bfloat16* grow = nullptr;     // gate of every column
+        if (a.gate && row_ok) {
+          grow = a.gate + (long long)(q_start + q_idx) * a.ldg + (long long)h * a.gate_cols;
+          if (a.gate_cols == 1) {
+            inv *= sigmoid_of(*grow);
+            grow = nullptr;
+          }
+        }
 #pragma unroll 1
         for (int c = 0; c < kDV; c += 32) {
           uint32_t w[32];
@@ -378,7 +465,11 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
           for (int q4 = 0; q4 < 4; ++q4) {
             us::Pack16 o;
 #pragma unroll
-            for (int i = 0; i < 8; ++i) o.b[i] = us::f2bf(__uint_as_float(w[q4 * 8 + i]) * inv);
+            for (int i = 0; i < 8; ++i) {
+              float f = __uint_as_float(w[q4 * 8 + i]) * inv;
+              if (grow && c + q4 * 8 + i < a.V) f *= sigmoid_of(grow[c + q4 * 8 + i]);
+              o.b[i] = us::f2bf(f);
+            }
             if (wide) {
               if (c + q4 * 8 < a.V) *reinterpret_cast<uint4*>(orow + c + q4 * 8) = o.u;
             } else {
@@ -401,18 +492,18 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   }
 }
 
-template <int kN, int kR, int kDV, int kVS>
+template <int kN, int kR, int kDV, int kVS, bool kSig = false>
 int launch_flash(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmR,
                  const CUtensorMap& tmV, const FlashArgs& a, dim3 grid, cudaStream_t stream) {
   constexpr size_t smem = (size_t)4 * (kN + kR) * kSlab + (size_t)kVS * (kDV / 64) * kSlab + 17 * 8 + 1024;
   static_assert(smem <= 227 * 1024, "shared memory of a CTA");
   static bool configured = false;
   if (!configured) {
-    US_CUDA_CHECK(cudaFuncSetAttribute(latent_flash_kernel<kN, kR, kDV, kVS>,
+    US_CUDA_CHECK(cudaFuncSetAttribute(latent_flash_kernel<kN, kR, kDV, kVS, kSig>,
                                        cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     configured = true;
   }
-  US_CUDA_CHECK(us::launch_pdl(latent_flash_kernel<kN, kR, kDV, kVS>, grid, dim3(320), smem, stream, tmQ,
+  US_CUDA_CHECK(us::launch_pdl(latent_flash_kernel<kN, kR, kDV, kVS, kSig>, grid, dim3(320), smem, stream, tmQ,
                                tmK, tmR, tmV, a));
   return US_OK;
 }
@@ -436,11 +527,11 @@ US_API int us_latent_gather(const void* cpages, int ldc, const void* rpages, int
 
 // q [Tq, H (slabs + 1) 64] rows at ldq: per head its unrotated channels in `slabs` slabs of 64, then the
 // rotated ones; kv [Tk, H slabs 64 | H dv] rows at ldkv; r [Tk, 64]; V <= dv output columns per head.
-// Sequences without keys (cu_k) are left alone.
+// gate [Tq, H V] rows at ldg, or null: the output times its sigmoid.  Sequences without keys (cu_k) are left alone.
 US_API int us_latent_flash(const void* q, long long ldq, const void* kv, long long ldkv, const void* r,
                            void* out, long long ldo, const int* cu_q, const int* cu_k, int n_seqs,
                            int Tq, int Tk, int H, int slabs, int dv, int V, int max_q, int window,
-                           float scale, void* stream_) {
+                           float scale, const void* gate, long long ldg, void* stream_) {
   US_REQUIRE(q && kv && r && out && cu_q && cu_k && n_seqs >= 1 && Tq >= 1 && Tk >= 1 && H >= 1 &&
              max_q >= 1 && V >= 1 && V <= dv);
   US_REQUIRE((ldq % 8) == 0 && (ldkv % 8) == 0 && ((uintptr_t)q % 16) == 0 && ((uintptr_t)kv % 16) == 0 &&
@@ -454,7 +545,7 @@ US_API int us_latent_flash(const void* q, long long ldq, const void* kv, long lo
   if (!rc) rc = us_tmap_2d(&tmV, v, US_TMAP_BF16, Tk, (uint64_t)H * dv, ldkv, kBN, 64, US_SWZ_128);
   if (rc) return rc;
   FlashArgs a{cu_q, cu_k, (__nv_bfloat16*)out, ldo, V, window, scale * 1.4426950408889634f, us_status_ptr(), 1,
-              nullptr, 1.f};
+              nullptr, 1.f, (const __nv_bfloat16*)gate, ldg, V};
   const dim3 grid((max_q + 2 * kBM - 1) / (2 * kBM), H, n_seqs);
   cudaStream_t stream = (cudaStream_t)stream_;
   if (slabs == 1) return dv == 64 ? launch_flash<1, 1, 64, 2>(tmQ, tmK, tmR, tmV, a, grid, stream)
@@ -463,29 +554,59 @@ US_API int us_latent_flash(const void* q, long long ldq, const void* kv, long lo
                   : launch_flash<2, 1, 128, 1>(tmQ, tmK, tmR, tmV, a, grid, stream);
 }
 
-// q [Tq, H slabs 64] rows at ldq; k [Tk, G slabs 64] and v [Tk, G dv] rows at ldk, ldv, query head h reading
-// key / value head h / (H / G); V <= dv output columns per head at column h V of `out`; window 0: every
-// earlier key; sink [H] or null; out_scale multiplies the output.  Sequences without keys are left alone.
-US_API int us_window_flash(const void* q, long long ldq, const void* k, long long ldk, const void* v,
-                           long long ldv, void* out, long long ldo, const int* cu_q, const int* cu_k,
-                           int n_seqs, int Tq, int Tk, int H, int G, int slabs, int dv, int V, int max_q,
-                           int window, float scale, const float* sink, float out_scale, void* stream_) {
-  US_REQUIRE(q && k && v && out && cu_q && cu_k && n_seqs >= 1 && Tq >= 1 && Tk >= 1 && H >= 1 && G >= 1 &&
-             H % G == 0 && max_q >= 1 && V >= 1 && V <= dv);
+namespace {
+
+template <bool kSig>
+int grouped_flash(FlashArgs a, const void* q, long long ldq, const void* k, long long ldk, const void* v,
+                  long long ldv, int n_seqs, int Tq, int Tk, int H, int G, int slabs, int dv, int max_q,
+                  cudaStream_t stream) {
+  US_REQUIRE(q && k && v && a.out && a.cu_q && a.cu_k && n_seqs >= 1 && Tq >= 1 && Tk >= 1 && H >= 1 && G >= 1 &&
+             H % G == 0 && max_q >= 1 && a.V >= 1 && a.V <= dv);
   US_REQUIRE((ldq % 8) == 0 && (ldk % 8) == 0 && (ldv % 8) == 0 && ((uintptr_t)q % 16) == 0 &&
-             ((uintptr_t)k % 16) == 0 && ((uintptr_t)v % 16) == 0 && ((uintptr_t)out % 16) == 0);
+             ((uintptr_t)k % 16) == 0 && ((uintptr_t)v % 16) == 0 && ((uintptr_t)a.out % 16) == 0);
   if (slabs < 1 || slabs > 2 || (dv != 64 && dv != 128)) return US_ERR_UNSUPPORTED;
   CUtensorMap tmQ, tmK, tmV;
   int rc = us_tmap_2d(&tmQ, q, US_TMAP_BF16, Tq, (uint64_t)H * slabs * 64, ldq, kBM, 64, US_SWZ_128);
   if (!rc) rc = us_tmap_2d(&tmK, k, US_TMAP_BF16, Tk, (uint64_t)G * slabs * 64, ldk, kBN, 64, US_SWZ_128);
   if (!rc) rc = us_tmap_2d(&tmV, v, US_TMAP_BF16, Tk, (uint64_t)G * dv, ldv, kBN, 64, US_SWZ_128);
   if (rc) return rc;
-  FlashArgs a{cu_q, cu_k, (__nv_bfloat16*)out, ldo, V, window, scale * 1.4426950408889634f, us_status_ptr(),
-              H / G, sink, out_scale};
+  a.status = us_status_ptr();
+  a.rep = H / G;
   const dim3 grid((max_q + 2 * kBM - 1) / (2 * kBM), H, n_seqs);
-  cudaStream_t stream = (cudaStream_t)stream_;
-  if (slabs == 1) return dv == 64 ? launch_flash<1, 0, 64, 2>(tmQ, tmK, tmK, tmV, a, grid, stream)
-                                  : launch_flash<1, 0, 128, 2>(tmQ, tmK, tmK, tmV, a, grid, stream);
-  return dv == 64 ? launch_flash<2, 0, 64, 2>(tmQ, tmK, tmK, tmV, a, grid, stream)
-                  : launch_flash<2, 0, 128, 2>(tmQ, tmK, tmK, tmV, a, grid, stream);
+  if (slabs == 1) return dv == 64 ? launch_flash<1, 0, 64, 2, kSig>(tmQ, tmK, tmK, tmV, a, grid, stream)
+                                  : launch_flash<1, 0, 128, 2, kSig>(tmQ, tmK, tmK, tmV, a, grid, stream);
+  return dv == 64 ? launch_flash<2, 0, 64, 2, kSig>(tmQ, tmK, tmK, tmV, a, grid, stream)
+                  : launch_flash<2, 0, 128, 2, kSig>(tmQ, tmK, tmK, tmV, a, grid, stream);
+}
+
+}  // namespace
+
+// q [Tq, H slabs 64] rows at ldq; k [Tk, G slabs 64] and v [Tk, G dv] rows at ldk, ldv, query head h reading
+// key / value head h / (H / G); V <= dv output columns per head at column h V of `out`; window 0: every
+// earlier key; sink [H] or null; out_scale multiplies the output, gate [Tq, H] (rows at ldg, or null) by its
+// sigmoid.  Sequences without keys are left alone.
+US_API int us_window_flash(const void* q, long long ldq, const void* k, long long ldk, const void* v,
+                           long long ldv, void* out, long long ldo, const int* cu_q, const int* cu_k,
+                           int n_seqs, int Tq, int Tk, int H, int G, int slabs, int dv, int V, int max_q,
+                           int window, float scale, const float* sink, float out_scale, const void* gate,
+                           long long ldg, void* stream_) {
+  FlashArgs a{cu_q, cu_k, (__nv_bfloat16*)out, ldo, V, window, scale * 1.4426950408889634f, nullptr, 1, sink,
+              out_scale, (const __nv_bfloat16*)gate, ldg, 1};
+  return grouped_flash<false>(a, q, ldq, k, ldk, v, ldv, n_seqs, Tq, Tk, H, G, slabs, dv, max_q,
+                              (cudaStream_t)stream_);
+}
+
+// The same with weight sigmoid(cap tanh(scale temp_h (q . k) / cap) + shift_h) for a visible key (cap 0: the
+// score as it is); temp and shift [H].
+US_API int us_sigmoid_flash(const void* q, long long ldq, const void* k, long long ldk, const void* v,
+                            long long ldv, void* out, long long ldo, const int* cu_q, const int* cu_k,
+                            int n_seqs, int Tq, int Tk, int H, int G, int slabs, int dv, int V, int max_q,
+                            int window, float scale, const float* temp, const float* shift, float cap,
+                            float out_scale, const void* gate, long long ldg, void* stream_) {
+  US_REQUIRE(temp && shift && cap >= 0.f);
+  // an enormous cap: z is tiny, its tanh z itself, and cap * z the score
+  FlashArgs a{cu_q, cu_k, (__nv_bfloat16*)out, ldo, V, window, 0.f, nullptr, 1, nullptr, out_scale,
+              (const __nv_bfloat16*)gate, ldg, 1, temp, shift, scale, cap > 0.f ? cap : 1e12f};
+  return grouped_flash<true>(a, q, ldq, k, ldk, v, ldv, n_seqs, Tq, Tk, H, G, slabs, dv, max_q,
+                             (cudaStream_t)stream_);
 }

@@ -59,6 +59,16 @@ __device__ __forceinline__ float gelu_erf(float x) {
   return 0.5f * x * (1.f + erff(x * 0.70710678118654752f));
 }
 
+// 3: gelu (erf), 5: square of relu, 6: a x^2 + x / 2 above zero, b (e^x - 1 - x) + x / 2 below
+__device__ __forceinline__ float act_single(float x, int act, float a, float b) {
+  if (act == 5) {
+    x = fmaxf(x, 0.f);
+    return x * x;
+  }
+  if (act == 6) return fmaf(x > 0.f ? a * x : b, x > 0.f ? x : __expf(x) - 1.f - x, 0.5f * x);
+  return gelu_erf(x);
+}
+
 // (clamp(u) + 1) g sigmoid(alpha g) with g cut off above `limit`, u on both sides
 __device__ __forceinline__ float clamped_glu(float u, float g, float limit, float alpha) {
   g = fminf(g, limit);
@@ -66,11 +76,13 @@ __device__ __forceinline__ float clamped_glu(float u, float g, float limit, floa
   return (u + 1.f) * (g / (1.f + __expf(-alpha * g)));
 }
 
-enum Form : int { kPlain = 0, kGelu = 1, kClamped = 2 };
+enum Form : int { kPlain = 0, kAct = 1, kClamped = 2 };
 
 struct Glu {
   int second;             // weight row of the first feature of the second half
   float limit, alpha;
+  int act;                // kAct: which one, and its constants
+  float a, b;
 };
 
 // MT = 16-row tiles of the activation (rows <= 16 * MT).
@@ -80,7 +92,7 @@ linear_decode_kernel(const __nv_bfloat16* __restrict__ W, const __nv_bfloat16* _
                      void* __restrict__ out, const void* __restrict__ bias, int rows, int M, int K,
                      long long ldw, long long ldx, long long ldo, int out_f32, int bias_f32,
                      int ksplit, const Glu glu) {
-  constexpr bool GELU = FORM == kGelu, GATED = FORM == kClamped;
+  constexpr bool ACT = FORM == kAct, GATED = FORM == kClamped;
   constexpr int kOut = GATED ? kFeat / 2 : kFeat;       // output features per CTA
   // Weights are never written by a kernel: the first loads go out before the wait on the
   // kernels that produce the activation.
@@ -209,7 +221,7 @@ linear_decode_kernel(const __nv_bfloat16* __restrict__ W, const __nv_bfloat16* _
         if (bias)
           v += bias_f32 ? reinterpret_cast<const float*>(bias)[col]
                         : us::bf2f(reinterpret_cast<const __nv_bfloat16*>(bias)[col]);
-        if (GELU) v = gelu_erf(v);
+        if (ACT) v = act_single(v, glu.act, glu.a, glu.b);
         if (out_f32)
           reinterpret_cast<float*>(out)[(long long)r * ldo + col] = v;
         else
@@ -234,7 +246,7 @@ linear_decode_kernel(const __nv_bfloat16* __restrict__ W, const __nv_bfloat16* _
     if (bias)
       v += bias_f32 ? reinterpret_cast<const float*>(bias)[col]
                     : us::bf2f(reinterpret_cast<const __nv_bfloat16*>(bias)[col]);
-    if (GELU) v = gelu_erf(v);
+    if (ACT) v = act_single(v, glu.act, glu.a, glu.b);
     if (out_f32)
       reinterpret_cast<float*>(out)[(long long)r * ldo + col] = v;
     else
@@ -254,10 +266,10 @@ int run(int form, const void* W, const void* X, void* out, const void* bias, int
   const __nv_bfloat16* x = (const __nv_bfloat16*)X;
   static bool configured = false;
   if (!configured) {
-    for (auto k : {linear_decode_kernel<4, kPlain>, linear_decode_kernel<4, kGelu>, linear_decode_kernel<4, kClamped>})
+    for (auto k : {linear_decode_kernel<4, kPlain>, linear_decode_kernel<4, kAct>, linear_decode_kernel<4, kClamped>})
       US_CUDA_CHECK(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          4 * kStages * 8192));
-    for (auto k : {linear_decode_kernel<2, kPlain>, linear_decode_kernel<2, kGelu>, linear_decode_kernel<2, kClamped>})
+    for (auto k : {linear_decode_kernel<2, kPlain>, linear_decode_kernel<2, kAct>, linear_decode_kernel<2, kClamped>})
       US_CUDA_CHECK(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          2 * kStages * 8192));
     configured = true;
@@ -300,7 +312,7 @@ int run(int form, const void* W, const void* X, void* out, const void* bias, int
   // kStages buffers x (16 MT) rows x 512 bytes
 #define US_LD(MT)                                                                                \
   US_CUDA_CHECK(form == kClamped ? launch(linear_decode_kernel<MT, kClamped>, MT * kStages * 8192) \
-                : form == kGelu  ? launch(linear_decode_kernel<MT, kGelu>, MT * kStages * 8192)    \
+                : form == kAct  ? launch(linear_decode_kernel<MT, kAct>, MT * kStages * 8192)    \
                                  : launch(linear_decode_kernel<MT, kPlain>, MT * kStages * 8192))
   if (rows <= 16) US_LD(1);
   else if (rows <= 32) US_LD(2);
@@ -311,14 +323,15 @@ int run(int form, const void* W, const void* X, void* out, const void* bias, int
 
 }  // namespace
 
-// act: 0 none, 3 gelu (erf) of the biased value.  rows <= 64, K a multiple of 256, 16-byte aligned rows of W and X.  Returns
+// act, of the biased value: 0 none, 3 gelu (erf), 5 square of relu, 6 xIELU (act_a, act_b).  rows <= 64, K a multiple of 256, 16-byte aligned rows of W and X.  Returns
 // US_ERR_UNSUPPORTED for other shapes (the caller then takes the tcgen05 kernel).
 US_API int us_linear_decode(const void* W, const void* X, void* out, const void* bias, int rows,
                             int M, int K, long long ldw, long long ldx, long long ldo,
-                            int out_f32, int bias_f32, int act, void* stream_) {
-  US_REQUIRE(W && X && out && rows >= 1 && M >= 1 && K >= 1 && (act == 0 || act == 3));
-  return run(act == 3 ? kGelu : kPlain, W, X, out, bias, rows, M, K, ldw, ldx, ldo, out_f32, bias_f32,
-             Glu{0, 0.f, 0.f}, (cudaStream_t)stream_);
+                            int out_f32, int bias_f32, int act, float act_a, float act_b,
+                            void* stream_) {
+  US_REQUIRE(W && X && out && rows >= 1 && M >= 1 && K >= 1 && (act == 0 || act == 3 || act == 5 || act == 6));
+  return run(act ? kAct : kPlain, W, X, out, bias, rows, M, K, ldw, ldx, ldo, out_f32, bias_f32,
+             Glu{0, 0.f, 0.f, act, act_a, act_b}, (cudaStream_t)stream_);
 }
 
 // Gated: out[rows, I] = (clamp(first) + 1) g sigmoid(alpha g), g = min(second, limit); W [2 I, K] holds the
@@ -327,6 +340,6 @@ US_API int us_linear_decode_clamped(const void* W, const void* X, void* out, int
                                     long long ldw, long long ldx, long long ldo, float limit,
                                     float alpha, void* stream_) {
   US_REQUIRE(W && X && out && rows >= 1 && I >= 1 && K >= 1);
-  return run(kClamped, W, X, out, nullptr, rows, I, K, ldw, ldx, ldo, 0, 0, Glu{I, limit, alpha},
+  return run(kClamped, W, X, out, nullptr, rows, I, K, ldw, ldx, ldo, 0, 0, Glu{I, limit, alpha, 0, 0.f, 0.f},
              (cudaStream_t)stream_);
 }

@@ -7,6 +7,9 @@
 //                  device word `live` route nowhere (id -1, weight 0).
 //                  With `correction` [E] the choice is by score + correction, the weights
 //                  are the uncorrected scores over their sum (+ 1e-20).
+//                  Grouped form: experts stand in groups of neighbours, a group scores
+//                  what its best expert does, only experts of the best groups are
+//                  chosen; the weights are the scores times a factor.
 //   moe_sort       counting sort of the (token, route) pairs by local expert;
 //                  emits the permutation both ways, the expert offsets and the
 //                  list of row tiles the grouped GEMM walks.
@@ -31,15 +34,48 @@ namespace {
 constexpr int kMaxExperts = 1024;
 constexpr int kMaxPerLane = kMaxExperts / 32;
 
+enum RouteForm : int { kByScore = 0, kCorrected = 1, kGrouped = 2 };
+
+struct RouteRule {
+  const float* correction;    // [E], kCorrected
+  int ld;                     // floats between two tokens' logits
+  int group, keep;            // kGrouped: experts per group, groups that stay
+  float scale;                // kGrouped: of the weights
+};
+
+// Expert of the largest value (the lower id on ties) over a warp's registers.
+template <int PER_LANE>
+__device__ __forceinline__ int best_expert(const float (&v)[PER_LANE], float gone) {
+  const int lane = threadIdx.x & 31;
+  float best = gone;
+  int best_e = 0x7fffffff;
+#pragma unroll
+  for (int i = 0; i < PER_LANE; ++i)
+    if (v[i] > best) {
+      best = v[i];
+      best_e = lane + 32 * i;
+    }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+    const int oe = __shfl_xor_sync(0xffffffffu, best_e, o);
+    if (ob > best || (ob == best && oe < best_e)) {
+      best = ob;
+      best_e = oe;
+    }
+  }
+  return best_e;
+}
+
 // Softmax, top-k and renormalisation of one token's router logits by one warp.
-template <int PER_LANE, bool CORR>
+template <int PER_LANE, int FORM>
 __device__ __forceinline__ void topk_token(const float* __restrict__ logits,
                                            int* __restrict__ ids, float* __restrict__ weights,
                                            int t, int E, int top_k, int renorm,
                                            const int* __restrict__ live,
                                            const int* __restrict__ expert_map,
-                                           int* __restrict__ load,
-                                           const float* __restrict__ correction) {
+                                           int* __restrict__ load, const RouteRule& rule) {
+  constexpr bool CORR = FORM == kCorrected;
   const int lane = threadIdx.x & 31;
   if (live && t >= *live) {
     for (int j = lane; j < top_k; j += 32) {
@@ -48,7 +84,7 @@ __device__ __forceinline__ void topk_token(const float* __restrict__ logits,
     }
     return;
   }
-  const float* row = logits + (long long)t * E;
+  const float* row = logits + (long long)t * rule.ld;
   float v[PER_LANE];
   float mx = -INFINITY;
 #pragma unroll
@@ -63,6 +99,8 @@ __device__ __forceinline__ void topk_token(const float* __restrict__ logits,
   for (int i = 0; i < PER_LANE; ++i) {
     if (CORR)
       v[i] = (lane + 32 * i) < E ? expf(v[i] - mx) : 0.f;
+    else if (FORM == kGrouped)
+      v[i] = (lane + 32 * i) < E ? expf(v[i] - mx) : -1.f;
     else
       v[i] = (lane + 32 * i) < E ? __expf(v[i] - mx) : -1.f;
     if (v[i] > 0.f) sum += v[i];
@@ -77,8 +115,26 @@ __device__ __forceinline__ void topk_token(const float* __restrict__ logits,
     for (int i = 0; i < PER_LANE; ++i) {
       const int e = lane + 32 * i;
       s[CORR ? i : 0] = v[i] * inv;
-      v[i] = e < E ? s[CORR ? i : 0] + correction[e] : -INFINITY;
+      v[i] = e < E ? s[CORR ? i : 0] + rule.correction[e] : -INFINITY;
     }
+  }
+  if (FORM == kGrouped && rule.group * rule.keep < E) {
+    float u[PER_LANE];
+    unsigned int stays = 0;
+#pragma unroll
+    for (int i = 0; i < PER_LANE; ++i) u[i] = v[i];
+    for (int k = 0; k < rule.keep; ++k) {        // the best expert left names the next group
+      const int g = best_expert<PER_LANE>(u, kGone) / rule.group;
+#pragma unroll
+      for (int i = 0; i < PER_LANE; ++i)
+        if ((lane + 32 * i) / rule.group == g) {
+          u[i] = kGone;
+          stays |= 1u << i;
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < PER_LANE; ++i)
+      if (!((stays >> i) & 1u)) v[i] = kGone;
   }
   float picked_sum = 0.f;
   float my_w = 0.f;
@@ -119,23 +175,24 @@ __device__ __forceinline__ void topk_token(const float* __restrict__ logits,
     }
   }
   if (lane < top_k) {
-    if (renorm) my_w = CORR ? my_w / (picked_sum + 1e-20f) : my_w / fmaxf(picked_sum, FLT_EPSILON);
+    if (FORM == kGrouped) my_w *= rule.scale;
+    else if (renorm) my_w = CORR ? my_w / (picked_sum + 1e-20f) : my_w / fmaxf(picked_sum, FLT_EPSILON);
     if (load) atomicAdd(&load[my_id], 1);
     ids[(long long)t * top_k + lane] = expert_map ? expert_map[my_id] : my_id;
     weights[(long long)t * top_k + lane] = my_w;
   }
 }
 
-template <int PER_LANE, bool CORR>
+template <int PER_LANE, int FORM>
 __global__ void __launch_bounds__(128)
 topk_softmax_kernel(const float* __restrict__ logits, int* __restrict__ ids,
                     float* __restrict__ weights, int T, int E, int top_k, int renorm,
                     const int* __restrict__ live, const int* __restrict__ expert_map,
-                    int* __restrict__ load, const float* __restrict__ correction) {
+                    int* __restrict__ load, const RouteRule rule) {
   US_PDL_PROLOGUE();
   const int t = blockIdx.x * 4 + (threadIdx.x >> 5);
   if (t >= T) return;
-  topk_token<PER_LANE, CORR>(logits, ids, weights, t, E, top_k, renorm, live, expert_map, load, correction);
+  topk_token<PER_LANE, FORM>(logits, ids, weights, t, E, top_k, renorm, live, expert_map, load, rule);
 }
 
 // One CTA sorts all routes.  Local experts are [e_lo, e_lo + E).
@@ -379,7 +436,7 @@ moe_sort_cluster_kernel(const int* __restrict__ ids, int R, int e_lo, int E, int
 
 // Routing and sorting in one launch (decode-size batches): the CTA's 32 warps take the
 // tokens in turn, then the whole CTA sorts the routes they wrote.
-template <int PER_LANE, bool CORR>
+template <int PER_LANE, int FORM>
 __global__ void __launch_bounds__(1024)
 route_sort_kernel(const float* __restrict__ logits, int* __restrict__ ids,
                   float* __restrict__ weights, int T, int E_all, int top_k, int renorm,
@@ -388,10 +445,10 @@ route_sort_kernel(const float* __restrict__ logits, int* __restrict__ ids,
                   int* __restrict__ expert_offsets, int* __restrict__ tile_group,
                   int* __restrict__ tile_row0, int* __restrict__ tile_rows,
                   int* __restrict__ num_tiles, unsigned int* status,
-                  const float* __restrict__ correction) {
+                  const RouteRule rule) {
   US_PDL_PROLOGUE();
   for (int t = threadIdx.x >> 5; t < T; t += 32)
-    topk_token<PER_LANE, CORR>(logits, ids, weights, t, E_all, top_k, renorm, live, nullptr, nullptr, correction);
+    topk_token<PER_LANE, FORM>(logits, ids, weights, t, E_all, top_k, renorm, live, nullptr, nullptr, rule);
   __syncthreads();   // the routes written above are read below by other threads of the CTA
   sort_routes(ids, T * top_k, e_lo, E, block_n, max_tiles, sorted_route, perm_of_route,
               expert_offsets, tile_group, tile_row0, tile_rows, num_tiles, status);
@@ -536,7 +593,7 @@ __device__ __forceinline__ bool grid_wait(const unsigned int* ctr, unsigned int 
 // `sync` holds three zero-initialised counters: [0] CTAs that routed their tokens, [1] set
 // by CTA 0 once the sort is written, [2] CTAs that passed the second wait (the last one
 // clears all three for the next launch).
-template <int PER_LANE, bool CORR>
+template <int PER_LANE, int FORM>
 __global__ void __launch_bounds__(256)
 route_sort_gather_kernel(const float* __restrict__ logits, int* __restrict__ ids,
                          float* __restrict__ weights, int T, int E_all, int top_k, int renorm,
@@ -547,11 +604,11 @@ route_sort_gather_kernel(const float* __restrict__ logits, int* __restrict__ ids
                          int* __restrict__ tile_rows, int* __restrict__ num_tiles,
                          const __nv_bfloat16* __restrict__ x, int H,
                          __nv_bfloat16* __restrict__ xp, unsigned int* sync,
-                         unsigned int* status, const float* __restrict__ correction) {
+                         unsigned int* status, const RouteRule rule) {
   US_PDL_PROLOGUE();
   const int warps = blockDim.x >> 5;
   for (int t = blockIdx.x * warps + (threadIdx.x >> 5); t < T; t += gridDim.x * warps)
-    topk_token<PER_LANE, CORR>(logits, ids, weights, t, E_all, top_k, renorm, live, nullptr, nullptr, correction);
+    topk_token<PER_LANE, FORM>(logits, ids, weights, t, E_all, top_k, renorm, live, nullptr, nullptr, rule);
   __threadfence();
   __syncthreads();
   __shared__ int ok_s;
@@ -591,25 +648,51 @@ route_sort_gather_kernel(const float* __restrict__ logits, int* __restrict__ ids
 
 }  // namespace
 
-US_API int us_topk_softmax(const float* logits, int* ids, float* weights, int T, int E, int top_k,
-                           int renorm, const int* live, const int* expert_map, int* load,
-                           const float* correction, void* stream_) {
+namespace {
+
+int topk(int form, const RouteRule& rule, const float* logits, int* ids, float* weights, int T, int E,
+         int top_k, int renorm, const int* live, const int* expert_map, int* load, cudaStream_t stream) {
   US_REQUIRE(logits && ids && weights && T >= 0 && E >= 1 && E <= kMaxExperts && top_k >= 1 &&
              top_k <= 32 && top_k <= E);
   if (T == 0) return US_OK;
-  cudaStream_t stream = (cudaStream_t)stream_;
   const int blocks = (T + 3) / 4;
   const int per = (E + 31) / 32;
 #define US_TOPK(P)                                                                          \
   if (per <= P) {                                                                           \
-    us::launch_pdl(correction ? topk_softmax_kernel<P, true> : topk_softmax_kernel<P, false>, dim3(blocks),        \
-                   dim3(128), 0, stream, logits, ids, weights, T, E, top_k, renorm, live, expert_map, load, correction);  \
-    US_LAUNCH_CHECK();                                                                      \
+    auto k = form == kCorrected ? topk_softmax_kernel<P, kCorrected>                        \
+             : form == kGrouped ? topk_softmax_kernel<P, kGrouped>                          \
+                                : topk_softmax_kernel<P, kByScore>;                         \
+    US_CUDA_CHECK(us::launch_pdl(k, dim3(blocks), dim3(128), 0, stream, logits, ids, weights, T, E, top_k, \
+                                 renorm, live, expert_map, load, rule));                    \
     return US_OK;                                                                           \
   }
   US_TOPK(1) US_TOPK(2) US_TOPK(4) US_TOPK(8) US_TOPK(16) US_TOPK(32)
 #undef US_TOPK
   return US_ERR_UNSUPPORTED;
+}
+
+RouteRule by_score(const float* correction, int E) { return RouteRule{correction, E, 0, 0, 1.f}; }
+
+bool groups_ok(int E, int ld, int top_k, int group, int keep) {
+  return ld >= E && group >= 1 && E % group == 0 && keep >= 1 && keep <= E / group && top_k <= group * keep;
+}
+
+}  // namespace
+
+US_API int us_topk_softmax(const float* logits, int* ids, float* weights, int T, int E, int top_k,
+                           int renorm, const int* live, const int* expert_map, int* load,
+                           const float* correction, void* stream_) {
+  return topk(correction ? kCorrected : kByScore, by_score(correction, E), logits, ids, weights, T, E, top_k, renorm,
+              live, expert_map, load, (cudaStream_t)stream_);
+}
+
+// Scores over all E experts (logits of a token at ld floats from the last one's), experts in groups of
+// `group` neighbours of which the `keep` best stay, weights = scores * scale.
+US_API int us_grouped_topk(const float* logits, int ld, int* ids, float* weights, int T, int E, int top_k,
+                           int group, int keep, float scale, void* stream_) {
+  US_REQUIRE(groups_ok(E, ld, top_k, group, keep));
+  return topk(kGrouped, RouteRule{nullptr, ld, group, keep, scale}, logits, ids, weights, T, E, top_k, 0, nullptr,
+              nullptr, nullptr, (cudaStream_t)stream_);
 }
 
 US_API int us_moe_sort(const int* ids, int R, int e_lo, int E, int block_n, int max_tiles,
@@ -693,12 +776,12 @@ US_API int us_route_sort(const float* logits, int* ids, float* weights, int T, i
   const int per = (E_all + 31) / 32;
 #define US_RS_CASE(P)                                                                          \
   if (per <= P) {                                                                              \
-    US_CUDA_CHECK(us::launch_pdl(correction ? route_sort_kernel<P, true> : route_sort_kernel<P, false>, \
+    US_CUDA_CHECK(us::launch_pdl(correction ? route_sort_kernel<P, kCorrected> : route_sort_kernel<P, kByScore>, \
                                  dim3(1), dim3(1024), 0, stream, logits,                       \
                                  ids, weights, T, E_all, top_k, renorm, live, e_lo, E, block_n,\
                                  max_tiles, sorted_route, perm_of_route, expert_offsets,       \
                                  tile_group, tile_row0, tile_rows, num_tiles,                  \
-                                 us_status_ptr(), correction));                                \
+                                 us_status_ptr(), by_score(correction, E_all)));               \
     return US_OK;                                                                              \
   }
   US_RS_CASE(1)
@@ -725,33 +808,33 @@ US_API int us_unpermute_add_rmsnorm(const void* y_perm, const int* perm, const f
   return US_OK;
 }
 
-// topk_softmax + moe_sort + moe_gather in one launch, for batches of at most 512 tokens.
-// `sync`: three zero-initialised uint32 counters owned by the caller's workspace.
-US_API int us_route_sort_gather(const float* logits, int* ids, float* weights, int T, int E_all,
-                                int top_k, int renorm, const int* live, int e_lo, int E,
-                                int block_n, int max_tiles, int* sorted_route,
-                                int* perm_of_route, int* expert_offsets, int* tile_group,
-                                int* tile_row0, int* tile_rows, int* num_tiles, const void* x,
-                                int H, void* xp, void* sync, const float* correction, void* stream_) {
+namespace {
+
+int route_sort_gather(int form, const RouteRule& rule, const float* logits, int* ids, float* weights,
+                      int T, int E_all, int top_k, int renorm, const int* live, int e_lo, int E,
+                      int block_n, int max_tiles, int* sorted_route, int* perm_of_route,
+                      int* expert_offsets, int* tile_group, int* tile_row0, int* tile_rows,
+                      int* num_tiles, const void* x, int H, void* xp, void* sync, cudaStream_t stream) {
   US_REQUIRE(logits && ids && weights && T >= 1 && T <= 512 && E_all >= 1 &&
              E_all <= kMaxExperts && top_k >= 1 && top_k <= 32 && top_k <= E_all);
   US_REQUIRE(E >= 1 && E <= kMaxExperts && block_n >= 1 && max_tiles >= 1 && sorted_route &&
              perm_of_route && expert_offsets && tile_group && tile_row0 && tile_rows && num_tiles);
   US_REQUIRE(x && xp && sync && (H % 8) == 0);
-  cudaStream_t stream = (cudaStream_t)stream_;
   int ctas = (T * top_k + 3) / 4;
   if (ctas < 8) ctas = 8;
   if (ctas > 128) ctas = 128;
   const int per = (E_all + 31) / 32;
 #define US_RSG_CASE(P)                                                                         \
   if (per <= P) {                                                                              \
-    US_CUDA_CHECK(us::launch_pdl(correction ? route_sort_gather_kernel<P, true> : route_sort_gather_kernel<P, false>, \
-                                 dim3(ctas), dim3(256), 0, stream,                             \
+    auto k = form == kCorrected ? route_sort_gather_kernel<P, kCorrected>                      \
+             : form == kGrouped ? route_sort_gather_kernel<P, kGrouped>                        \
+                                : route_sort_gather_kernel<P, kByScore>;                       \
+    US_CUDA_CHECK(us::launch_pdl(k, dim3(ctas), dim3(256), 0, stream,                          \
                                  logits, ids, weights, T, E_all, top_k, renorm, live, e_lo, E, \
                                  block_n, max_tiles, sorted_route, perm_of_route,              \
                                  expert_offsets, tile_group, tile_row0, tile_rows, num_tiles,  \
                                  (const __nv_bfloat16*)x, H, (__nv_bfloat16*)xp,               \
-                                 (unsigned int*)sync, us_status_ptr(), correction));           \
+                                 (unsigned int*)sync, us_status_ptr(), rule));                 \
     return US_OK;                                                                              \
   }
   US_RSG_CASE(1)
@@ -762,4 +845,33 @@ US_API int us_route_sort_gather(const float* logits, int* ids, float* weights, i
   US_RSG_CASE(32)
 #undef US_RSG_CASE
   return US_ERR_ARG;
+}
+
+}  // namespace
+
+// topk_softmax + moe_sort + moe_gather in one launch, for batches of at most 512 tokens.
+// `sync`: three zero-initialised uint32 counters owned by the caller's workspace.
+US_API int us_route_sort_gather(const float* logits, int* ids, float* weights, int T, int E_all,
+                                int top_k, int renorm, const int* live, int e_lo, int E,
+                                int block_n, int max_tiles, int* sorted_route,
+                                int* perm_of_route, int* expert_offsets, int* tile_group,
+                                int* tile_row0, int* tile_rows, int* num_tiles, const void* x,
+                                int H, void* xp, void* sync, const float* correction, void* stream_) {
+  return route_sort_gather(correction ? kCorrected : kByScore, by_score(correction, E_all), logits, ids, weights, T,
+                           E_all, top_k, renorm, live, e_lo, E, block_n, max_tiles, sorted_route, perm_of_route,
+                           expert_offsets, tile_group, tile_row0, tile_rows, num_tiles, x, H, xp, sync,
+                           (cudaStream_t)stream_);
+}
+
+// The same by us_grouped_topk's rule; every expert has tensors.
+US_API int us_grouped_route_sort_gather(const float* logits, int ld, int* ids, float* weights, int T, int E,
+                                        int top_k, int group, int keep, float scale, int block_n,
+                                        int max_tiles, int* sorted_route, int* perm_of_route,
+                                        int* expert_offsets, int* tile_group, int* tile_row0,
+                                        int* tile_rows, int* num_tiles, const void* x, int H, void* xp,
+                                        void* sync, void* stream_) {
+  US_REQUIRE(groups_ok(E, ld, top_k, group, keep));
+  return route_sort_gather(kGrouped, RouteRule{nullptr, ld, group, keep, scale}, logits, ids, weights, T, E, top_k, 0,
+                           nullptr, 0, E, block_n, max_tiles, sorted_route, perm_of_route, expert_offsets, tile_group,
+                           tile_row0, tile_rows, num_tiles, x, H, xp, sync, (cudaStream_t)stream_);
 }

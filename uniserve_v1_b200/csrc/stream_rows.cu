@@ -3,13 +3,16 @@
 //   source   r(t) = rms(embed[id] * scale + table2[row]) * w              start of the stream
 //            r(t) = residual(t) + rms(y(t)) * w                           output norm and add
 //            r(t) = embed[id] * scale,  residual(t) + gain * y(t)         without w (plain form)
+//            r(t) = embed[id] * scale,  residual(t) + ln(y(t)) * w + b    layer form
 //   output   h(t) = rms(r(t)) * w_out                                     input norm
+//            h(t) = r(t)   or   ln(r(t)) * w_out + b_out                  layer form
 //            x(t) = h(t)   or   h(t) + (h(t - 1) - h(t)) * mu             token shift
 //
-// In the plain form y may also be a mixture of experts: sum_k weight_k * (row perm_k of the expert rows,
-// or row t of `ident` for an expert without tensors, perm_k < 0) + shared(t).
+// In the plain and the layer form y may also be a mixture of experts: sum_k weight_k * (row perm_k of the
+// expert rows, or row t of `ident` for an expert without tensors, perm_k < 0) + shared(t), the last one
+// times sigmoid(shared_gate(t)) in the layer form.
 //
-// with rms(v) = v / sqrt(mean(v^2) + eps).  r goes to a second residual buffer (the one that is
+// with rms(v) = v / sqrt(mean(v^2) + eps) and ln(v) = (v - mean(v)) / sqrt(mean((v - mean(v))^2) + eps).  r goes to a second residual buffer (the one that is
 // read stays as it is), because a shifted row needs its neighbour's h: a CTA takes up to kRows
 // consecutive rows of one sequence and forms the row before its first one itself.  The h before a
 // sequence's first row of the batch comes from the state slot; the CTA that reads it also forms
@@ -91,9 +94,15 @@ struct StreamRows {
   const float* route_w;       // [T, top]
   int top;
   const void *ident, *shared; // [T, W] or null
+  // layer form
+  const float *b, *b_out;     // [W]
+  const float* shared_gate;   // logit of row t at t * ld_gate, or null: the shared rows as they are
+  long long ld_gate;
 };
 
-template <int NV, bool PLAIN>
+enum Form : int { kOutNorm = 0, kPlain = 1, kLayer = 2 };
+
+template <int NV, int FORM>
 __global__ void __launch_bounds__(256) stream_rows_kernel(const StreamRows a) {
   US_PDL_PROLOGUE();
   __shared__ float buf[64];
@@ -127,13 +136,15 @@ __global__ void __launch_bounds__(256) stream_rows_kernel(const StreamRows a) {
   // raw operands of a row: the sublayer's output (or the embedding sum) and the residual
   auto load = [&](int t, float4 (&v)[NV], float4 (&r)[NV]) {
     const long long base = (long long)t * W;
-    if (PLAIN && a.y_perm) {
+    if (FORM != kOutNorm && a.y_perm) {
+      const float sg = FORM == kLayer && a.shared_gate ? 1.f / (1.f + expf(-a.shared_gate[t * a.ld_gate])) : 1.f;
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
         const int c = c0 + i * step;
         v[i] = r[i] = make_float4(0.f, 0.f, 0.f, 0.f);
         if (c >= W) continue;
         if (a.shared) v[i] = ld4(a.shared, base + c, a.bf16);
+        if (FORM == kLayer) v[i] = make_float4(v[i].x * sg, v[i].y * sg, v[i].z * sg, v[i].w * sg);
         r[i] = *reinterpret_cast<const float4*>(a.residual + base + c);
       }
       const long long k0 = (long long)t * a.top;
@@ -178,8 +189,36 @@ __global__ void __launch_bounds__(256) stream_rows_kernel(const StreamRows a) {
       }
     }
   };
+  auto layer = [&](float4 (&v)[NV], const float* w, const float* b) {
+    float sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) sum += v[i].x + v[i].y + v[i].z + v[i].w;      // columns past `width` are zero
+    const float mean = turn_sum(sum, buf, turn) * inv_n;
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = c0 + i * step;
+      v[i] = make_float4(c < a.width ? v[i].x - mean : 0.f, c + 1 < a.width ? v[i].y - mean : 0.f,
+                         c + 2 < a.width ? v[i].z - mean : 0.f, c + 3 < a.width ? v[i].w - mean : 0.f);
+      ss += sq4(v[i]);
+    }
+    const float inv = 1.f / sqrtf(turn_sum(ss, buf, turn) * inv_n + a.eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = c0 + i * step;
+      if (c < W)
+        v[i] = add4(mul4(v[i], *reinterpret_cast<const float4*>(w + c), inv), *reinterpret_cast<const float4*>(b + c));
+    }
+  };
   auto source = [&](float4 (&v)[NV], const float4 (&r)[NV]) {     // v becomes the row of the stream
-    if (PLAIN) {
+    if (FORM == kLayer) {
+      if (!a.residual) return;                   // start of the stream
+      layer(v, a.w, a.b);
+#pragma unroll
+      for (int i = 0; i < NV; ++i) v[i] = add4(r[i], v[i]);
+      return;
+    }
+    if (FORM == kPlain) {
 #pragma unroll
       for (int i = 0; i < NV; ++i)
         v[i] = make_float4(fmaf(a.gain, v[i].x, r[i].x), fmaf(a.gain, v[i].y, r[i].y),
@@ -197,6 +236,10 @@ __global__ void __launch_bounds__(256) stream_rows_kernel(const StreamRows a) {
     }
   };
   auto norm = [&](float4 (&v)[NV]) {
+    if (FORM == kLayer) {
+      if (a.w_out) layer(v, a.w_out, a.b_out);
+      return;
+    }
     float ss = 0.f;
 #pragma unroll
     for (int i = 0; i < NV; ++i) ss += sq4(v[i]);
@@ -362,13 +405,13 @@ int block_threads(int W) { return min(256, (W / 4 + 31) / 32 * 32); }
 
 namespace {
 
-template <bool PLAIN>
+template <int FORM>
 int launch_stream(const StreamRows& a, cudaStream_t stream) {
   const int grid = !a.mu ? us::ceil_div(a.T, a.rows) : a.one_token ? a.T : a.T / kRows + a.B;
   const dim3 block(block_threads(a.W));
   const int nv = us::ceil_div(a.W, 1024);
 #define US_STREAM(N) \
-  US_CUDA_CHECK(us::launch_pdl(stream_rows_kernel<N, PLAIN>, dim3(grid), block, 0, stream, a))
+  US_CUDA_CHECK(us::launch_pdl(stream_rows_kernel<N, FORM>, dim3(grid), block, 0, stream, a))
   if (nv <= 1) US_STREAM(1);
   else if (nv <= 2) US_STREAM(2);
   else if (nv <= 4) US_STREAM(4);
@@ -395,7 +438,7 @@ US_API int us_stream_rows(const int* ids, const int* rows2, const void* table, c
   if (T == 0) return US_OK;
   StreamRows a{ids, rows2, table, table2, scale, vocab, n2, y, residual, w, residual_out, w_out, mu,
                state, cu, slots, pos, x, B, T, W, width, bf16, one_token, eps, T >= 2048 ? 4 : 1, us_status_ptr()};
-  return launch_stream<false>(a, (cudaStream_t)stream_);
+  return launch_stream<kOutNorm>(a, (cudaStream_t)stream_);
 }
 
 // The plain form: residual_out = table row * scale (ids given), or residual + gain * (y, or the mixture
@@ -412,7 +455,26 @@ US_API int us_plain_rows(const int* ids, const void* table, float scale, int voc
   StreamRows a{ids, nullptr, table, nullptr, scale, vocab, 0, y, residual, nullptr, residual_out, w_out, nullptr,
                nullptr, nullptr, nullptr, nullptr, x, 1, T, W, width, bf16, 0, eps, T >= 2048 ? 4 : 1, us_status_ptr(),
                y || y_perm ? gain : 1.f, y_perm, perm, route_w, top, ident, shared};
-  return launch_stream<true>(a, (cudaStream_t)stream_);
+  return launch_stream<kPlain>(a, (cudaStream_t)stream_);
+}
+
+// The layer form: residual_out = table row * scale (ids given), or residual + ln(y, or a mixture of `top`
+// expert rows per token and a shared row) * w + b; x = residual_out, or with w_out its layer norm.
+US_API int us_layer_rows(const int* ids, const void* table, float scale, int vocab, const void* y,
+                         const void* y_perm, const int* perm, const float* route_w, int top,
+                         const void* shared, const float* shared_gate, long long ld_gate,
+                         const float* residual, const float* w, const float* b, float* residual_out,
+                         const float* w_out, const float* b_out, void* x, int T, int W, int width,
+                         int bf16, float eps, void* stream_) {
+  US_REQUIRE(residual_out && x && T >= 0 && W >= 8 && (W % 8) == 0 && width >= 1 && width <= W);
+  US_REQUIRE(y || y_perm ? residual && residual != residual_out && w && b : ids && table && !residual);
+  US_REQUIRE(!y_perm || (perm && route_w && top >= 1 && !y));
+  US_REQUIRE(!w_out || b_out);
+  if (T == 0) return US_OK;
+  StreamRows a{ids, nullptr, table, nullptr, scale, vocab, 0, y, residual, w, residual_out, w_out, nullptr,
+               nullptr, nullptr, nullptr, nullptr, x, 1, T, W, width, bf16, 0, eps, T >= 2048 ? 4 : 1, us_status_ptr(),
+               1.f, y_perm, perm, route_w, top, nullptr, shared, b, b_out, shared_gate, ld_gate};
+  return launch_stream<kLayer>(a, (cudaStream_t)stream_);
 }
 
 US_API int us_bigram_rows(const int* ids, int* last, const int* cu, const int* slots, const int* pos,

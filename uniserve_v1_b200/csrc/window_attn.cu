@@ -4,13 +4,17 @@
 //   s_h(i, j) = scale q_h(i) . k_g(j),   j <= i, i - j < window (0: no limit),   g = h / (H / G)
 //   o_h(i)    = sum_j e^{s_h(i, j)} v_g(j) / (sum_j e^{s_h(i, j)} + e^{sink_h})
 //
+// or, with weights that do not depend on the other keys (a temperature and a shift per head, capped scores),
+//
+//   w_h(i, j) = sigmoid(cap tanh(temp_h s_h(i, j) / cap) + shift_h),   o_h(i) = sum_j w_h(i, j) v_g(j)
+//
 //   us_window_prep             RMS norm over each head, rotation of its first channels, q into rows of
 //                              their own, k and v into pages
 //   us_window_gather           the keys and values that a batch's prompts see, from pages into packed rows
 //   us_window_attention_rows   any sizes, bf16 or FP32: one CTA per (query row, key head)
 //
-// (prompts: us_window_flash; single rows: us_paged_decode_attention_sink).  Channel i turns with channel
-// i + n, n the number of pairs.  The angle is formed and reduced to a fraction of a turn in FP64, so
+// (prompts: us_window_flash; single rows: us_paged_decode_attention_sink, us_sigmoid_decode).  Channel i
+// turns with channel i + n, n the number of pairs, or 2i with 2i + 1 (neighbours).  The angle is formed and reduced to a fraction of a turn in FP64, so
 // far positions lose nothing before the FP32 sine and cosine.
 #include "include/us_common.cuh"
 
@@ -75,6 +79,7 @@ struct Prep {
   void *kp, *vp;                // pages [n, page, G, D], [n, page, G, V]
   int T, bf16;
   float eps;
+  int neighbours;
 };
 
 // A warp takes up to kPrepHeads heads of one token, whose sines and cosines it forms once.  A lane holds
@@ -142,12 +147,22 @@ __global__ void __launch_bounds__(kPrepWarps * 32) window_prep_kernel(const Prep
       float lo[VEC], hi[VEC];
 #pragma unroll
       for (int e = 0; e < VEC; ++e) {
-        const float x = sm[p + e], y = sm[p + n + e];
+        const float x = a.neighbours ? sm[2 * (p + e)] : sm[p + e];
+        const float y = a.neighbours ? sm[2 * (p + e) + 1] : sm[p + n + e];
         lo[e] = x * cs[i][e] - y * sn[i][e];
         hi[e] = y * cs[i][e] + x * sn[i][e];
       }
-      stv<VEC>(dst, to + p, a.bf16, lo);
-      stv<VEC>(dst, to + p + n, a.bf16, hi);
+      if (!a.neighbours) {
+        stv<VEC>(dst, to + p, a.bf16, lo);
+        stv<VEC>(dst, to + p + n, a.bf16, hi);
+      } else if constexpr (VEC == 2) {
+        const float first[VEC] = {lo[0], hi[0]}, second[VEC] = {lo[VEC - 1], hi[VEC - 1]};
+        stv<VEC>(dst, to + 2 * p, a.bf16, first);
+        stv<VEC>(dst, to + 2 * p + 2, a.bf16, second);
+      } else {
+        st1(dst, to + 2 * p, a.bf16, lo[0]);
+        st1(dst, to + 2 * p + 1, a.bf16, hi[0]);
+      }
     }
     if (is_q) {
       for (int d = a.D + lane; d < a.Dq; d += 32) st1(dst, to + d, a.bf16, 0.f);
@@ -255,6 +270,10 @@ struct RowAttn {
   const float* sink;          // [H] or null
   int B, H, G, D, V, page, max_pages, window, bf16, per;
   float scale, out_scale;
+  const float *temp, *shift;  // [H]: sigmoid weights, or null: softmax
+  float cap;                  // 0: none
+  const void* gate;           // head h's output times sigmoid(gate[t * ldg + h]), or null
+  long long ldg;
 };
 
 constexpr int kRowThreads = 256;
@@ -306,7 +325,17 @@ __global__ void __launch_bounds__(kRowThreads) window_rows_kernel(const RowAttn 
     }
     __syncthreads();
     for (int h = warp; h < nh; h += kRowThreads / 32) {
-      const float sc = ps[h * kRowKeys + lane];
+      float sc = ps[h * kRowKeys + lane];
+      if (a.shift) {
+        if (lane < nj) {
+          sc *= a.temp[h0 + h];
+          if (a.cap > 0.f) sc = a.cap * tanhf(sc / a.cap);
+          sc = 1.f / (1.f + expf(-(sc + a.shift[h0 + h])));
+        }
+        ps[h * kRowKeys + lane] = lane < nj ? sc : 0.f;
+        if (lane == 0) fac[h] = 1.f;
+        continue;
+      }
       const float m0 = mx[h], m = fmaxf(m0, us::warp_max(sc));
       const float p = lane < nj ? expf(sc - m) : 0.f;
       const float add = us::warp_sum(p);
@@ -329,8 +358,10 @@ __global__ void __launch_bounds__(kRowThreads) window_rows_kernel(const RowAttn 
   __syncthreads();
   for (int e = tid; e < nh * V; e += kRowThreads) {
     const int h = e / V, c = e - h * V;
-    const float den = live ? sum[h] + (a.sink ? expf(a.sink[h0 + h] - mx[h]) : 0.f) : 1.f;
-    st1(a.out, t * a.ldo + (long long)(h0 + h) * V + c, a.bf16, live ? a.out_scale * os[e] / den : 0.f);
+    const float den = live && !a.shift ? sum[h] + (a.sink ? expf(a.sink[h0 + h] - mx[h]) : 0.f) : 1.f;
+    float o = live ? a.out_scale * os[e] / den : 0.f;
+    if (a.gate) o /= 1.f + expf(-ld1(a.gate, t * a.ldg + h0 + h, a.bf16));
+    st1(a.out, t * a.ldo + (long long)(h0 + h) * V + c, a.bf16, o);
   }
 }
 
@@ -343,12 +374,12 @@ bool even(long long a, long long b, long long c, long long d) { return ((a | b |
 US_API int us_window_prep(const void* x, long long ldx, int off_q, int off_k, int off_v, int H, int G,
                           int D, int V, const float* wq, const float* wk, const double* freq, int pairs,
                           float mag, const int* pos, const int* slots, void* q, int Dq, void* kpages,
-                          void* vpages, int T, float eps, int bf16, void* stream_) {
+                          void* vpages, int T, float eps, int neighbours, int bf16, void* stream_) {
   US_REQUIRE(x && wq && wk && pos && slots && q && kpages && vpages && T >= 0 && H >= 1 && G >= 1 &&
              D >= 1 && V >= 1 && Dq >= D && 2 * pairs <= D && (pairs == 0 || freq));
   if (T == 0) return US_OK;
   Prep a{x, ldx, off_q, off_k, off_v, H, G, D, V, pairs, wq, wk, freq, mag, pos, slots, q, Dq, kpages, vpages,
-         T, bf16, eps};
+         T, bf16, eps, neighbours};
   const bool two = even(ldx, off_q, off_k, off_v) && even(D, V, pairs, Dq) && ((uintptr_t)x % 4) == 0;
   return two ? launch_prep<2>(a, (cudaStream_t)stream_) : launch_prep<1>(a, (cudaStream_t)stream_);
 }
@@ -371,15 +402,17 @@ US_API int us_window_gather(const void* kpages, const void* vpages, int G, int D
 }
 
 // Attention of T rows (rows of sequence s at cu[s] .. cu[s + 1], keys up to a row's own position).  seq_lens
-// [B] or null: length 0 marks padding, whose rows become zero.
+// [B] or null: length 0 marks padding, whose rows become zero.  temp and shift [H] (both or none): sigmoid
+// weights with scores capped at `cap` (0: not).  gate (or null): a logit per row and head.
 US_API int us_window_attention_rows(const void* q, long long ldq, int hsq, const void* kpages,
                                     const void* vpages, void* out, long long ldo, const int* cu,
                                     const int* pos, const int* seq_lens, const int* page_table,
                                     const float* sink, int T, int B, int H, int G, int D, int V, int page,
-                                    int max_pages, int window, float scale, float out_scale, int bf16,
-                                    void* stream_) {
+                                    int max_pages, int window, float scale, float out_scale,
+                                    const float* temp, const float* shift, float cap, const void* gate,
+                                    long long ldg, int bf16, void* stream_) {
   US_REQUIRE(q && kpages && vpages && out && cu && pos && page_table && T >= 0 && B >= 1 && H >= 1 &&
-             G >= 1 && H % G == 0 && D >= 1 && V >= 1 && page >= 1 && ldo >= (long long)H * V);
+             G >= 1 && H % G == 0 && D >= 1 && V >= 1 && page >= 1 && ldo >= (long long)H * V && !temp == !shift);
   if (T == 0) return US_OK;
   constexpr size_t kMost = 220 * 1024;
   auto bytes = [&](int per) {
@@ -391,7 +424,7 @@ US_API int us_window_attention_rows(const void* q, long long ldq, int hsq, const
   const int parts = us::ceil_div(rep, per);
   if (bytes(per) > kMost || (long long)G * parts > 65535) return US_ERR_LIMIT;
   RowAttn a{q, ldq, hsq, kpages, vpages, out, ldo, cu, pos, seq_lens, page_table, sink, B, H, G, D, V, page,
-            max_pages, window, bf16, per, scale, out_scale};
+            max_pages, window, bf16, per, scale, out_scale, temp, shift, cap, gate, ldg};
   static bool configured = false;
   if (!configured) {
     US_CUDA_CHECK(cudaFuncSetAttribute(window_rows_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kMost));

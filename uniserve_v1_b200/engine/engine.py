@@ -115,7 +115,7 @@ class LLMEngine:
         self.model = model
         self.device = model.device
         self.recurrent = bool(getattr(model, "recurrent_state", False))
-        if self.recurrent and kv_dtype not in (None, "auto", "bf16", "bfloat16"):
+        if getattr(model, "attends_pages", False) and kv_dtype not in (None, "auto", "bf16", "bfloat16"):
             raise ValueError(f"kv cache dtype {kv_dtype!r} is not served for this model")
         if kv_dtype in ("fp8", "fp8_e4m3", "e4m3"):
             model.kv_dtype = "fp8"       # E4M3 pages, one FP32 scale per page and plane

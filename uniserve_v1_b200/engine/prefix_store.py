@@ -27,7 +27,7 @@ from typing import Optional
 import numpy as np
 import torch
 
-MAGIC = b"USPC\x01"
+MAGIC = b"USPC\x02"
 _DTYPES = {str(d): d for d in (torch.bfloat16, torch.float16, torch.float32, torch.uint8)}
 
 
@@ -40,7 +40,7 @@ def _describe(engine) -> dict:
     runner = engine.runner
     layers = []
     for i, (k, v) in _layers(runner):
-        layers.append({"layer": i, "shape": list(k.shape[1:]), "dtype": str(k.dtype),
+        layers.append({"layer": i, "shapes": [list(k.shape[1:]), list(v.shape[1:])], "dtype": str(k.dtype),
                        "scaled": getattr(k, "page_scale", None) is not None})
     return {"identity": engine.blocks.identity, "page_size": engine.blocks.page_size,
             "layers": layers}
@@ -49,10 +49,8 @@ def _describe(engine) -> dict:
 def _page_bytes(desc: dict) -> int:
     total = 0
     for lay in desc["layers"]:
-        n = 1
-        for x in lay["shape"]:
-            n *= x
-        total += 2 * n * _DTYPES[lay["dtype"]].itemsize + (8 if lay["scaled"] else 0)
+        n = sum(int(np.prod(shape)) for shape in lay["shapes"])
+        total += n * _DTYPES[lay["dtype"]].itemsize + (8 if lay["scaled"] else 0)
     return total
 
 
@@ -127,10 +125,9 @@ def load_prefix_cache(engine, path: str, remove: bool = True) -> dict:
     first = n - take                                    # the newest pages are at the end
     idx = torch.as_tensor(pages, dtype=torch.long, device=runner.device)
     for _, pair in _layers(runner):
-        shape = list(pair[0].shape[1:])
-        numel = int(np.prod(shape))
         for plane in pair:
-            nbytes = n * numel * plane.element_size()
+            shape = list(plane.shape[1:])
+            nbytes = n * int(np.prod(shape)) * plane.element_size()
             raw = torch.frombuffer(bytearray(data[off:off + nbytes]), dtype=torch.uint8)
             off += nbytes
             sel = raw.view(plane.dtype).view(n, *shape)[first:]

@@ -391,9 +391,7 @@ class CausalLmRunner:
             if kc is None:
                 self.host_kv.append((None, None))
                 continue
-            shape = (slots,) + tuple(kc.shape[1:])
-            hk = torch.zeros(shape, dtype=kc.dtype)
-            hv = torch.zeros(shape, dtype=vc.dtype)
+            hk, hv = (torch.zeros((slots,) + tuple(t.shape[1:]), dtype=t.dtype) for t in (kc, vc))
             if self.device.type == "cuda":
                 hk, hv = hk.pin_memory(), hv.pin_memory()
             if getattr(kc, "page_scale", None) is not None:      # E4M3 pages travel with scales
@@ -419,8 +417,8 @@ class CausalLmRunner:
                 if getattr(kc, "page_scale", None) is not None:
                     hk.page_scale[slots] = kc.page_scale.index_select(0, pages).to("cpu")
                     hv.page_scale[slots] = vc.page_scale.index_select(0, pages).to("cpu")
-            self.d2h_bytes += sum(2 * len(offloads) * kc[0].numel() * kc.element_size()
-                                  for kc, _ in self.kv_caches if kc is not None)
+            self.d2h_bytes += sum(len(offloads) * t[0].numel() * t.element_size()
+                                  for pair in self.kv_caches for t in pair if t is not None)
         if fetches:
             slots = torch.tensor([s for s, _ in fetches], dtype=torch.long)
             pages = torch.tensor([p for _, p in fetches], dtype=torch.long, device=dev)
@@ -432,8 +430,8 @@ class CausalLmRunner:
                 if getattr(kc, "page_scale", None) is not None:
                     kc.page_scale.index_copy_(0, pages, hk.page_scale[slots].to(dev))
                     vc.page_scale.index_copy_(0, pages, hv.page_scale[slots].to(dev))
-            self.h2d_bytes += sum(2 * len(fetches) * kc[0].numel() * kc.element_size()
-                                  for kc, _ in self.kv_caches if kc is not None)
+            self.h2d_bytes += sum(len(fetches) * t[0].numel() * t.element_size()
+                                  for pair in self.kv_caches for t in pair if t is not None)
 
     def release_graphs(self) -> None:
         """Drops every captured graph (do this before tearing down a process

@@ -1,5 +1,5 @@
 """What decoders made of a list of unlike layers share: padded and stacked weights, random
-checkpoints, the output projection.
+checkpoints, latent attention, the output projection.
 
 Projections that read the same rows are stacked into one product; stacked sections and row
 widths are padded with zeros to multiples of 8 so that every operand row starts on a 16-byte
@@ -11,6 +11,7 @@ from typing import Optional
 import torch
 
 from ..ops import functional as F
+from ..ops import latent as LA
 
 
 def pad8(n: int) -> int:
@@ -81,6 +82,50 @@ class LayeredDecoder:
         class _Dict:
             get = staticmethod(state.__getitem__)
         return self.load_state(_Dict())
+
+    # ----------------------------------------------------- latent attention --
+    def _load_latent(self, w, p, s: LA.LatentDims, need, gate=False):
+        """Tensors ``p`` + dq, dkv, uq, uk, uv, o, their norms and, with ``gate``, g (a logit per output
+        column) into ``w``; the caller adds 'freq' and, where they are not 1 and neighbours, 'mag' and
+        'halves'."""
+        H, D, RD, V, R, Q = s.heads, s.dim, s.rot_dim, s.vdim, s.kv_rank, s.q_rank
+        W = self.cfg.hidden_size
+        t = need(p + "dkv", R + RD, W)
+        w["proj"], w["offs"] = self._stack([need(p + "dq", Q, W), t[:R], t[R:]] +
+                                           ([need(p + "g", H * V, W)] if gate else []))
+        w["q_norm"], w["kv_norm"] = self._vector(need(p + "dq.norm", Q)), self._vector(need(p + "dkv.norm", R))
+        # queries head by head as [unrotated | rotated], each section padded
+        (Dp, RDp), Rp = LA.query_layout(s, self.dtype), pad8(R)
+        q = need(p + "uq", H * (D + RD), Q).view(H, D + RD, Q)
+        uq = torch.zeros(H, Dp + RDp, pad8(Q), dtype=self.dtype, device=self.device)
+        uq[:, :D, :Q], uq[:, Dp:Dp + RD, :Q] = self._put(q[:, :D]), self._put(q[:, D:])
+        w["uq"] = uq.view(H * (Dp + RDp), pad8(Q))
+        uk, uv = need(p + "uk", H * D, R).view(H, D, R), need(p + "uv", H * V, R).view(H, V, R)
+        w["absorb"] = torch.zeros(H, Rp, pad8(D), dtype=self.dtype, device=self.device)
+        w["absorb"][:, :R, :D] = self._put(uk).transpose(1, 2)
+        w["uv"] = torch.zeros(H, V, Rp, dtype=self.dtype, device=self.device)
+        w["uv"][:, :, :R] = self._put(uv)
+        if LA.expands(s, self.dtype) and self.device.type == "cuda":
+            dv = LA.value_layout(s)
+            kv = torch.zeros(H * (Dp + dv), Rp, dtype=self.dtype, device=self.device)
+            kv[:H * Dp].view(H, Dp, Rp)[:, :D, :R] = self._put(uk)
+            kv[H * Dp:].view(H, dv, Rp)[:, :V, :R] = self._put(uv)
+            w["kv"] = kv
+        w["o"] = self._matrix(need(p + "o", W, H * V))
+
+    def _latent_attention(self, s: LA.LatentDims, w, x, m, meta, caches):
+        cp, rp = caches
+        T, H, (Dp, RDp) = x.shape[0], s.heads, LA.query_layout(s, self.dtype)
+        turn = (w.get("mag", 1.0), w.get("halves", False))
+        proj = F.linear(x, w["proj"])
+        LA.latent_prep_(proj, w["offs"][:3], s, w["q_norm"], w["kv_norm"], w["freq"], m.positions, meta.slots,
+                        cp, rp, self.cfg.eps, *turn)
+        oq = w["offs"][0]
+        q = F.linear(proj[:, oq:oq + pad8(s.q_rank)], w["uq"]).view(T, H, Dp + RDp)
+        LA.rotate_heads_(q, Dp, m.positions, w["freq"], *turn)
+        gate = proj[:, w["offs"][3]:w["offs"][3] + H * s.vdim] if len(w["offs"]) > 3 else None
+        att = LA.attend(q, Dp, w, cp, rp, m, meta.page_table, s, w["o"].shape[1], meta.seq_lens, meta.max_k, gate)
+        return F.linear(att, w["o"])
 
     def logits(self, hidden_rows: torch.Tensor) -> torch.Tensor:
         return F.linear(hidden_rows, self.lm_head, out_dtype=torch.float32)

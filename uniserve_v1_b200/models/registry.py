@@ -84,6 +84,23 @@ def _tadinex_model(cfg, device, dtype, ctx=None):
     return TadinexModel(cfg, device, dtype)
 
 
+def _nopuzen_config(d):
+    from .nopuzen import NopuzenConfig
+    return NopuzenConfig.from_json(d)
+
+
+def _nopuzen_named(name):
+    from .nopuzen import NopuzenConfig
+    return NopuzenConfig.tiny() if name == "tiny" else NopuzenConfig.bench()
+
+
+def _nopuzen_model(cfg, device, dtype, ctx=None):
+    from .nopuzen import NopuzenModel
+    if ctx is not None and ctx.world_size > 1:
+        raise ValueError("this family is served on one GPU")
+    return NopuzenModel(cfg, device, dtype)
+
+
 PAGED_DECODERS = {
     "qwen3_moe": PagedDecoder(_qwen3_config, _qwen3_named, _qwen3_model, (torch.bfloat16,)),
     "nepevik": PagedDecoder(_nepevik_config, _nepevik_named, _nepevik_model,
@@ -92,6 +109,8 @@ PAGED_DECODERS = {
                             (torch.bfloat16, torch.float32), "zonopel"),
     "tadinex": PagedDecoder(_tadinex_config, _tadinex_named, _tadinex_model,
                             (torch.bfloat16, torch.float32), "tadinex"),
+    "nopuzen": PagedDecoder(_nopuzen_config, _nopuzen_named, _nopuzen_model,
+                            (torch.bfloat16, torch.float32), "nopuzen"),
 }
 
 

@@ -166,7 +166,8 @@ class ZonopelModel(LayeredDecoder):
                 w["norm"] = norm(p + "norm", s.inner)
                 w["o"] = self._matrix(need(p + "o", W, s.inner))
             else:
-                self._load_latent(w, p, L, need, norm)
+                self._load_latent(w, p, s, need)
+                w["freq"] = LA.frequencies(L.rot_dims, L.rot_base, self.device)
             if L.ff:
                 m = f"l{i}.mlp."
                 w["norm2"], w["norm2b"] = norm(f"l{i}.norm2"), norm(f"l{i}.norm2b")
@@ -176,33 +177,6 @@ class ZonopelModel(LayeredDecoder):
             own[i] = w
         self.layers = [own[i if L.weights_of is None else L.weights_of] for i, L in enumerate(c.layers)]
         return self
-
-    def _load_latent(self, w, p, L: LayerSpec, need, norm):
-        s = L.mixer
-        H, D, RD, V, R, Q = s.heads, s.dim, s.rot_dim, s.vdim, s.kv_rank, s.q_rank
-        W = self.cfg.hidden_size
-        t = need(p + "dkv", R + RD, W)
-        w["proj"], w["offs"] = self._stack([need(p + "dq", Q, W), t[:R], t[R:]])
-        w["q_norm"], w["kv_norm"] = norm(p + "dq.norm", Q), norm(p + "dkv.norm", R)
-        w["freq"] = LA.frequencies(L.rot_dims, L.rot_base, self.device)
-        # queries head by head as [unrotated | rotated], each section padded
-        (Dp, RDp), Rp = LA.query_layout(s, self.dtype), pad8(R)
-        q = need(p + "uq", H * (D + RD), Q).view(H, D + RD, Q)
-        uq = torch.zeros(H, Dp + RDp, pad8(Q), dtype=self.dtype, device=self.device)
-        uq[:, :D, :Q], uq[:, Dp:Dp + RD, :Q] = self._put(q[:, :D]), self._put(q[:, D:])
-        w["uq"] = uq.view(H * (Dp + RDp), pad8(Q))
-        uk, uv = need(p + "uk", H * D, R).view(H, D, R), need(p + "uv", H * V, R).view(H, V, R)
-        w["absorb"] = torch.zeros(H, Rp, pad8(D), dtype=self.dtype, device=self.device)
-        w["absorb"][:, :R, :D] = self._put(uk).transpose(1, 2)
-        w["uv"] = torch.zeros(H, V, Rp, dtype=self.dtype, device=self.device)
-        w["uv"][:, :, :R] = self._put(uv)
-        if LA.expands(s, self.dtype) and self.device.type == "cuda":
-            dv = LA.value_layout(s)
-            kv = torch.zeros(H * (Dp + dv), Rp, dtype=self.dtype, device=self.device)
-            kv[:H * Dp].view(H, Dp, Rp)[:, :D, :R] = self._put(uk)
-            kv[H * Dp:].view(H, dv, Rp)[:, :V, :R] = self._put(uv)
-            w["kv"] = kv
-        w["o"] = self._matrix(need(p + "o", W, H * V))
 
     def random_state(self, seed: int = 0) -> dict:
         """A checkpoint's tensors drawn at random: {name: tensor} with the names ``load_state`` reads."""
@@ -283,18 +257,6 @@ class ZonopelModel(LayeredDecoder):
         return n
 
     # ------------------------------------------------------------- forward --
-    def _latent_attention(self, L: LayerSpec, w, x, m: SeqMeta, meta, caches):
-        s, (cp, rp) = L.mixer, caches
-        T, H, (Dp, RDp) = x.shape[0], s.heads, LA.query_layout(s, self.dtype)
-        proj = F.linear(x, w["proj"])
-        LA.latent_prep_(proj, w["offs"], s, w["q_norm"], w["kv_norm"], w["freq"], m.positions, meta.slots,
-                        cp, rp, self.cfg.eps)
-        oq = w["offs"][0]
-        q = F.linear(proj[:, oq:oq + pad8(s.q_rank)], w["uq"]).view(T, H, Dp + RDp)
-        LA.rotate_heads_(q, Dp, m.positions, w["freq"])
-        att = LA.attend(q, Dp, w, cp, rp, m, meta.page_table, s, w["o"].shape[1], meta.seq_lens, meta.max_k)
-        return F.linear(att, w["o"])
-
     def forward(self, input_ids, positions, meta, kv_caches) -> torch.Tensor:
         """Final-normed rows [T, Wp] of the packed batch ``meta`` (``cu_q``, ``state_slots``,
         ``page_table``, ``slots``); ``meta.states`` are the pools of ``new_state_pools``."""
@@ -318,7 +280,7 @@ class ZonopelModel(LayeredDecoder):
                 y = SS.mixer(F.linear(x, w["proj"]), w, states[i][1], states[i][2], m, L.mixer, c.eps)
                 y = F.linear(y, w["o"])
             else:
-                y = self._latent_attention(L, w, x, m, meta, kv_caches[i])
+                y = self._latent_attention(L.mixer, w, x, m, meta, kv_caches[i])
             nxt = F.NextRows(w["norm2"]) if L.ff else entry(i + 1)
             res, x = F.add_norm_rows(y, res, w["norm1b"], nxt, c.eps, c.hidden_size)
             if L.ff:

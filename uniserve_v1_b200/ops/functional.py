@@ -302,17 +302,18 @@ def _block_n(rows: int, dual: bool) -> int:
     return 128 if dual else 256
 
 
-_ACT1 = {None: 0, "gelu_erf": 3}       # activations of a single (ungated) product
+_ACT1 = {None: 0, "gelu_erf": 3, "relu2": 5, "xielu": 6}       # activations of a single (ungated) product
 
 
-def linear(x, w, bias=None, out_dtype=None, out=None, block_n=None, act=None):
+def linear(x, w, bias=None, out_dtype=None, out=None, block_n=None, act=None, act_ab=(0.0, 0.0)):
     """y[rows, M] = act(x[rows, K] @ w[M, K]^T (+ bias)).  bf16 operands, FP32
     accumulation in tensor memory, output bf16 or fp32; FP32 operands run in true 32-bit.
-    ``act``: None or "gelu_erf"."""
+    ``act``: None, "gelu_erf", "relu2" (square of relu) or "xielu" (with ``act_ab`` = (a, b): a z^2 + z / 2
+    above zero, b (e^z - 1 - z) + z / 2 below)."""
     out_dtype = out_dtype or x.dtype
     if not _cuda(x):
         y = R.linear(x, w, bias, torch.float32 if act else out_dtype)
-        return R.gelu_erf(y).to(out_dtype) if act else y
+        return R.activation(y, act, act_ab).to(out_dtype) if act else y
     acode = _ACT1[act]
     if x.dtype == torch.float32:
         assert w.dtype == torch.float32 and w.stride(1) == 1 and out_dtype == torch.float32
@@ -320,7 +321,7 @@ def linear(x, w, bias=None, out_dtype=None, out=None, block_n=None, act=None):
         if out is None:
             out = torch.empty(x2.shape[0], w.shape[0], dtype=torch.float32, device=x.device)
         N.call("us_gemm_f32", N.ptr(w), N.ptr(x2), N.ptr(out), 1, w.shape[0], w.shape[0],
-               x2.shape[1], x2.shape[0], w.stride(0), x2.stride(0), out.stride(0), acode,
+               x2.shape[1], x2.shape[0], w.stride(0), x2.stride(0), out.stride(0), acode, *act_ab,
                N.ptr(bias), None, None, None, None, 0, N.stream())
         return out.view(*x.shape[:-1], w.shape[0])
     assert x.dtype == BF16 and w.dtype == BF16
@@ -346,9 +347,14 @@ def linear(x, w, bias=None, out_dtype=None, out=None, block_n=None, act=None):
         # decode-size projection: weight-streaming kernel (latency-bound shape)
         N.call("us_linear_decode", N.ptr(w), N.ptr(x2), N.ptr(out), N.ptr(bias), rows, M, K,
                w.stride(0), x2.stride(0), out.stride(0), int(out.dtype == torch.float32),
-               0 if (bias is None or bias.dtype == BF16) else 1, acode, N.stream())
+               0 if (bias is None or bias.dtype == BF16) else 1, acode, *act_ab, N.stream())
         return out.view(*x.shape[:-1], M)
     bn = block_n or _block_n(rows, False)
+    if acode == 6:
+        assert bias is None and out.dtype == BF16
+        N.call("us_gemm_wx_act", N.ptr(w), N.ptr(x2), N.ptr(out), 1, M, M, K, rows, w.stride(0), x2.stride(0),
+               out.stride(0), acode, *act_ab, None, None, None, None, 0, bn, N.stream())
+        return out.view(*x.shape[:-1], M)
     N.call("us_gemm_wx", N.ptr(w), N.ptr(x2), N.ptr(out), 1, M, M, K, rows, w.stride(0),
            x2.stride(0), out.stride(0), 0, 0, acode, 0 if out.dtype == BF16 else 1, N.ptr(bias),
            0 if (bias is None or bias.dtype == BF16) else 1, None, None, None, None, None, None,
@@ -375,7 +381,7 @@ def clamped_linear(x, w, limit, alpha, out=None, tiles=None, block_n=None, live=
     tile_args = tiles or (None, None, None, None, 0)
     if x.dtype == torch.float32:
         z = torch.empty(rows, I2, dtype=torch.float32, device=x.device)
-        N.call("us_gemm_f32", N.ptr(w), N.ptr(x), N.ptr(z), E, I2, I2, K, rows, K, x.stride(0), I2, 0, None,
+        N.call("us_gemm_f32", N.ptr(w), N.ptr(x), N.ptr(z), E, I2, I2, K, rows, K, x.stride(0), I2, 0, 0.0, 0.0, None,
                *tile_args, N.stream())
         N.call("us_clamped_glu_f32", N.ptr(z), N.ptr(out), rows, I_, limit, alpha, N.stream())
         return out
@@ -606,6 +612,44 @@ def _route_tiles(R_, E, E_total):
     return block_n, min(R_, E) + R_ // block_n + 1, MoeWorkspace._expected_tiles(R_, E, E_total, block_n)
 
 
+def _route(logits, top, E, E_all, x, gather, pick):
+    """Routes of ``logits``: ``gather(ids, weights, sort, xp)`` in one launch up to 512 rows of ``x``, above
+    ``pick(ids, weights)`` and a sort."""
+    T, dev, R_ = logits.shape[0], logits.device, logits.shape[0] * top
+    block_n, max_tiles, live = _route_tiles(R_, E, E_all)
+    buf = torch.empty(3 * R_ + E + 1 + 3 * max_tiles + 1, dtype=torch.int32, device=dev)
+    ids, srt, perm, offs, tg, t0, tr, nt = buf.split([R_, R_, R_, E + 1, max_tiles, max_tiles, max_tiles, 1])
+    weights = torch.empty(T, top, dtype=torch.float32, device=dev)
+    r = Routes(ids.view(T, top), srt, perm.view(T, top), offs, tg, t0, tr, nt, block_n, max_tiles, live, weights)
+    sort = (block_n, max_tiles, N.ptr(srt), N.ptr(perm), N.ptr(offs), N.ptr(tg), N.ptr(t0), N.ptr(tr), N.ptr(nt))
+    if T <= 512:
+        r.xp = torch.empty(R_, x.shape[1], dtype=x.dtype, device=dev)
+        wide = 1 if x.dtype == BF16 else 2          # the gather moves 16-bit units
+        gather(N.ptr(ids), N.ptr(weights), sort, (N.ptr(x), x.shape[1] * wide, N.ptr(r.xp)))
+    else:
+        pick(N.ptr(ids), N.ptr(weights))
+        N.call("us_moe_sort", N.ptr(ids), R_, 0, E, *sort, N.stream())
+    return r
+
+
+def grouped_routes(logits, E, top, groups, scale, x, sync):
+    """Softmax scores over the first E columns of ``logits`` [T, >= E] (FP32, any row stride), the ``top``
+    best chosen, weighted by their scores times ``scale``.  ``groups``: None or (count, keep): experts stand
+    in ``count`` equal groups of neighbours, and only those of the ``keep`` groups with the best experts can
+    be chosen.  ``sync``: four int32 zeros that calls of one stream share."""
+    count, keep = groups or (1, 1)
+    if not _cuda(logits):
+        return R.grouped_routes(logits[:, :E], top, count, keep, scale)
+    assert logits.dtype == torch.float32 and logits.stride(1) == 1
+    T, ld, per, st = logits.shape[0], logits.stride(0), E // count, N.stream()
+    return _route(
+        logits, top, E, E, x,
+        lambda ids, weights, sort, rows: N.call("us_grouped_route_sort_gather", N.ptr(logits), ld, ids, weights, T, E,
+                                                top, per, keep, scale, *sort, *rows, N.ptr(sync), st),
+        lambda ids, weights: N.call("us_grouped_topk", N.ptr(logits), ld, ids, weights, T, E, top, per, keep, scale,
+                                    st))
+
+
 def scored_routes(logits, correction, top, E, x, sync):
     """Softmax scores over all experts, the ``top`` of score + ``correction`` chosen, weighted by their
     scores over the scores' sum.  ``logits`` [T, n] FP32; experts at or past ``E`` have no tensors: their
@@ -614,25 +658,14 @@ def scored_routes(logits, correction, top, E, x, sync):
     if not _cuda(logits):
         return R.scored_routes(logits, correction, top, E)
     T, E_all = logits.shape
-    dev, st = logits.device, N.stream()
+    st = N.stream()
     assert logits.dtype == torch.float32 and logits.is_contiguous()
-    R_ = T * top
-    block_n, max_tiles, live = _route_tiles(R_, E, E_all)
-    buf = torch.empty(3 * R_ + E + 1 + 3 * max_tiles + 1, dtype=torch.int32, device=dev)
-    ids, srt, perm, offs, tg, t0, tr, nt = buf.split([R_, R_, R_, E + 1, max_tiles, max_tiles, max_tiles, 1])
-    weights = torch.empty(T, top, dtype=torch.float32, device=dev)
-    r = Routes(ids.view(T, top), srt, perm.view(T, top), offs, tg, t0, tr, nt, block_n, max_tiles, live, weights)
-    sort = (E, block_n, max_tiles, N.ptr(srt), N.ptr(perm), N.ptr(offs), N.ptr(tg), N.ptr(t0), N.ptr(tr), N.ptr(nt))
-    if T <= 512:
-        r.xp = torch.empty(R_, x.shape[1], dtype=x.dtype, device=dev)
-        wide = 1 if x.dtype == BF16 else 2          # the gather moves 16-bit units
-        N.call("us_route_sort_gather", N.ptr(logits), N.ptr(ids), N.ptr(weights), T, E_all, top, 1, None, 0, *sort,
-               N.ptr(x), x.shape[1] * wide, N.ptr(r.xp), N.ptr(sync), N.ptr(correction), st)
-    else:
-        N.call("us_topk_softmax", N.ptr(logits), N.ptr(ids), N.ptr(weights), T, E_all, top, 1, None, None, None,
-               N.ptr(correction), st)
-        N.call("us_moe_sort", N.ptr(ids), R_, 0, *sort, st)
-    return r
+    return _route(
+        logits, top, E, E_all, x,
+        lambda ids, weights, sort, rows: N.call("us_route_sort_gather", N.ptr(logits), ids, weights, T, E_all, top, 1,
+                                                None, 0, E, *sort, *rows, N.ptr(sync), N.ptr(correction), st),
+        lambda ids, weights: N.call("us_topk_softmax", N.ptr(logits), ids, weights, T, E_all, top, 1, None, None, None,
+                                    N.ptr(correction), st))
 
 
 def table_routes(tokens, tables, E):
@@ -660,11 +693,11 @@ def table_routes(tokens, tables, E):
 
 def routed_mlp(x, routes, w_up, w_down, act="gelu_erf", clamped=None):
     """Experts W_down act(W_up x) over sorted routes: gather, two grouped products with the activation in
-    the first one's epilogue.  w_up [E, I, H], w_down [E, H, I]; with ``clamped`` = (limit, alpha) the
+    the first one's epilogue ("gelu_erf" or "relu2").  w_up [E, I, H], w_down [E, H, I]; with ``clamped`` = (limit, alpha) the
     experts are gated (``clamped_linear``) and w_up is [E, 2 * I, H].  Returns the expert rows in permuted
     order; ``routes.perm`` says where a token's are."""
     if not _cuda(x):
-        return R.routed_mlp(x, routes, w_up, w_down, clamped)
+        return R.routed_mlp(x, routes, w_up, w_down, clamped, act)
     T, H = x.shape
     E, _, I_ = w_down.shape
     top = routes.perm.shape[1]
@@ -683,7 +716,7 @@ def routed_mlp(x, routes, w_up, w_down, act="gelu_erf", clamped=None):
         clamped_linear(xp, w_up, *clamped, out=h, tiles=tiles, block_n=routes.block_n, live=routes.live_tiles)
     for w, a, o, M, K, c in ((w_up, xp, h, I_, H, code), (w_down, h, y, H, I_, 0))[int(clamped is not None):]:
         if x.dtype == torch.float32:
-            N.call("us_gemm_f32", N.ptr(w), N.ptr(a), N.ptr(o), E, M, M, K, R_, K, K, M, c, None,
+            N.call("us_gemm_f32", N.ptr(w), N.ptr(a), N.ptr(o), E, M, M, K, R_, K, K, M, c, 0.0, 0.0, None,
                    *tiles, st)
             continue
         if routes.live_tiles:
@@ -733,10 +766,11 @@ class NextRows:
     """What follows a residual row: the next sublayer's input norm and, with ``shift``, the token
     shift h + (h' - h) * shift, h' being the row before (``state`` [slots, W] FP32 keeps the last
     one of every sequence of the packed batch ``meta``)."""
-    weight: torch.Tensor
+    weight: Optional[torch.Tensor]          # None (layer form only): the residual row as it is
     shift: Optional[torch.Tensor] = None
     state: Optional[torch.Tensor] = None
     meta: object = None
+    bias: Optional[torch.Tensor] = None     # layer form: beside ``weight``
 
 
 def _stream_rows(embed, y, residual, w, nxt, eps, width, dtype, T, W):
@@ -762,6 +796,8 @@ class Mixture:
     routes: Routes
     ident: Optional[torch.Tensor] = None
     shared: Optional[torch.Tensor] = None   # added without a weight
+    shared_gate: Optional[torch.Tensor] = None      # layer form: [T] FP32 logits (a strided view), whose
+                                                    # sigmoid multiplies ``shared``
 
 
 def _plain_rows(ids, table, scale, y, residual, gain, nxt, eps, width, dtype, T, W):
@@ -797,6 +833,41 @@ def add_plain_rows(y, residual, gain, nxt: NextRows, eps, width):
         return R.plain_rows(y.float(), residual, gain, nxt, eps, width, y.dtype)
     assert y.is_contiguous() and y.shape == residual.shape
     return _plain_rows(None, None, 0.0, y, residual, gain, nxt, eps, width, y.dtype, *y.shape)
+
+
+def _layer_rows(ids, table, scale, y, residual, w, b, nxt, eps, width, dtype, T, W):
+    dev = (residual if table is None else table).device
+    res = torch.empty(T, W, dtype=torch.float32, device=dev)
+    x = torch.empty(T, W, dtype=dtype, device=dev)
+    mix = y if isinstance(y, Mixture) else None
+    r = mix.routes if mix else None
+    gate = mix.shared_gate if mix else None
+    N.call("us_layer_rows", N.ptr(ids), N.ptr(table), scale, table.shape[0] if table is not None else 0,
+           None if mix else N.ptr(y), N.ptr(mix.rows) if mix else None, N.ptr(r.perm) if mix else None,
+           N.ptr(r.weights) if mix else None, r.perm.shape[1] if mix else 0, N.ptr(mix.shared) if mix else None,
+           N.ptr(gate), gate.stride(0) if gate is not None else 0, N.ptr(residual), N.ptr(w), N.ptr(b), N.ptr(res),
+           N.ptr(nxt.weight), N.ptr(nxt.bias), N.ptr(x), T, W, width, int(dtype == BF16), eps, N.stream())
+    return res, x
+
+
+def embed_layer_rows(ids, table, nxt: NextRows, eps, width):
+    """Start of a stream whose sublayers read it as it is: table rows in FP32, and the next sublayer's rows
+    in the table's type."""
+    if not _cuda(table):
+        return R.layer_rows(table[ids.long()].float(), None, None, None, nxt, eps, width, table.dtype)
+    return _layer_rows(ids, table, 1.0, None, None, None, None, nxt, eps, width, table.dtype, ids.shape[0],
+                       table.shape[1])
+
+
+def add_layer_rows(y, residual, w, b, nxt: NextRows, eps, width):
+    """(residual + layer norm of y with weight ``w`` and bias ``b``, the next sublayer's rows in y's type);
+    ``y``: rows or a ``Mixture``.  The residual handed in stays as it is."""
+    src = y.rows if isinstance(y, Mixture) else y
+    if not _cuda(src):
+        return R.layer_rows(R.mixture(y) if isinstance(y, Mixture) else y.float(), residual, w, b, nxt, eps, width,
+                            src.dtype)
+    assert src.is_contiguous() and (isinstance(y, Mixture) or y.shape == residual.shape)
+    return _layer_rows(None, None, 1.0, y, residual, w, b, nxt, eps, width, src.dtype, *residual.shape)
 
 
 def embed_norm_rows(ids, table, scale, w, nxt: NextRows, eps, width, second=None):

@@ -7,6 +7,9 @@ by all heads; a head's unrotated keys and its values are linear images of c.
 *Absorbed form*: q W_uk is formed once per query, so attention runs over the latents alone, as
 with one key head of width rank + rot_dim whose values are its first ``rank`` columns.
 
+Rotated channels are paired with their neighbour (2i, 2i + 1) or, in halves, i with i + pairs, cosine and
+sine times ``mag``.  The output may carry a gate: head columns times sigmoid of a logit each.
+
 Pages hold ``[page, 1, rank]`` latents and ``[page, 1, rot_dim]`` rotated parts (each padded to a
 multiple of 8).  On a GPU the entry points run ``csrc/latent_attn.cu``, on the CPU FP32 formulas."""
 from __future__ import annotations
@@ -21,15 +24,15 @@ from .vector_delta import BF16, SeqMeta
 
 P, I, L = N.P, N.I, N.L
 N.register_signatures({
-    "us_latent_prep": (I, [P, L, I, I, I, I, I, I, P, P, P, I, P, P, P, I, P, I, I, N.F, I, P]),
-    "us_rotate_heads": (I, [P, L, I, I, I, P, I, P, I, I, P]),
-    "us_head_linear": (I, [P, P, P, L, L, L, L, L, L, I, I, I, I, I, P]),
+    "us_latent_prep": (I, [P, L, I, I, I, I, I, I, P, P, P, I, P, P, P, I, P, I, I, N.F, N.F, I, I, P]),
+    "us_rotate_heads": (I, [P, L, I, I, I, P, I, P, I, N.F, I, I, P]),
+    "us_head_linear": (I, [P, P, P, L, L, L, L, L, L, I, I, I, I, P, L, P, I, P]),
     "us_latent_attention_rows": (I, [P, L, I, P, L, I, P, I, P, I, P, L, I, P, P, P, P, I, I, I, I, I, I,
                                      I, I, N.F, I, P]),
     "us_latent_decode": (I, [P, L, I, P, L, I, P, I, P, I, P, L, I, P, P, P, P, P, I, I, I, I, I, I, I, I, I,
                              N.F, P]),
     "us_latent_gather": (I, [P, I, P, I, P, P, P, P, P, P, I, I, I, I, I, I, P]),
-    "us_latent_flash": (I, [P, L, P, L, P, P, L, P, P, I, I, I, I, I, I, I, I, I, N.F, P]),
+    "us_latent_flash": (I, [P, L, P, L, P, P, L, P, P, I, I, I, I, I, I, I, I, I, N.F, P, L, P]),
 })
 
 # sequences that bring at least this many rows take the expanded form (an absorbed row costs a pass
@@ -56,16 +59,17 @@ def frequencies(dims: int, base: float, device) -> torch.Tensor:
     return (float(base) ** (-2.0 * i / dims)).to(device)
 
 
-def _turned(x, positions, freq):
-    """Channel 2i turned with channel 2i + 1 of the last axis (x [T, ..., n] FP32)."""
+def _turned(x, positions, freq, mag=1.0, halves=False):
+    """The channel pairs of the last axis turned (x [T, ..., n] FP32)."""
     n = freq.shape[0]
     a = positions.double()[:, None] * freq[None]
-    c, s = torch.cos(a).float(), torch.sin(a).float()
+    c, s = (torch.cos(a) * mag).float(), (torch.sin(a) * mag).float()
     while c.dim() < x.dim():
         c, s = c[:, None], s[:, None]
-    u, v = x[..., 0:2 * n:2], x[..., 1:2 * n:2]
+    first, second = (slice(0, n), slice(n, 2 * n)) if halves else (slice(0, 2 * n, 2), slice(1, 2 * n, 2))
+    u, v = x[..., first], x[..., second]
     out = x.clone()
-    out[..., 0:2 * n:2], out[..., 1:2 * n:2] = u * c - v * s, v * c + u * s
+    out[..., first], out[..., second] = u * c - v * s, v * c + u * s
     return out
 
 
@@ -73,7 +77,7 @@ def _rms(x, w, eps):
     return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w
 
 
-def latent_prep_(x, offs, d: LatentDims, wq, wc, freq, positions, slots, cpages, rpages, eps):
+def latent_prep_(x, offs, d: LatentDims, wq, wc, freq, positions, slots, cpages, rpages, eps, mag=1.0, halves=False):
     """``x`` holds the query latent, the key latent and the rotated key part at columns ``offs``.
     Norms the query latent in place; the normed key latent and the turned part go to the cache
     rows ``slots`` (negative: not written)."""
@@ -82,38 +86,43 @@ def latent_prep_(x, offs, d: LatentDims, wq, wc, freq, positions, slots, cpages,
     if x.is_cuda:
         N.call("us_latent_prep", N.ptr(x), x.stride(0), oq, oc, orr, d.q_rank, d.kv_rank, d.rot_dim,
                N.ptr(wq), N.ptr(wc), N.ptr(freq), freq.shape[0], N.ptr(positions), N.ptr(slots),
-               N.ptr(cpages), nc, N.ptr(rpages), nr, x.shape[0], eps, int(x.dtype == BF16), N.stream())
+               N.ptr(cpages), nc, N.ptr(rpages), nr, x.shape[0], eps, mag, int(halves), int(x.dtype == BF16), N.stream())
         return
     x[:, oq:oq + d.q_rank] = _rms(x[:, oq:oq + d.q_rank].float(), wq, eps).to(x.dtype)
     c = _rms(x[:, oc:oc + d.kv_rank].float(), wc, eps).to(x.dtype)
-    r = _turned(x[:, orr:orr + d.rot_dim].float(), positions, freq).to(x.dtype)
+    r = _turned(x[:, orr:orr + d.rot_dim].float(), positions, freq, mag, halves).to(x.dtype)
     sel = slots >= 0
     at = slots[sel].long()
     cpages.view(-1, nc)[at, :d.kv_rank] = c[sel]
     rpages.view(-1, nr)[at, :d.rot_dim] = r[sel]
 
 
-def rotate_heads_(x, off, positions, freq):
+def rotate_heads_(x, off, positions, freq, mag=1.0, halves=False):
     """Turns the channel pairs that start at channel ``off`` of every head of x [T, H, n] in place."""
     T, H, n = x.shape
     if x.is_cuda:
         N.call("us_rotate_heads", N.ptr(x), x.stride(0), off, x.stride(1), H, N.ptr(freq), freq.shape[0],
-               N.ptr(positions), T, int(x.dtype == BF16), N.stream())
+               N.ptr(positions), T, mag, int(halves), int(x.dtype == BF16), N.stream())
         return
-    x[..., off:] = _turned(x[..., off:].float(), positions, freq).to(x.dtype)
+    x[..., off:] = _turned(x[..., off:].float(), positions, freq, mag, halves).to(x.dtype)
 
 
-def head_linear(w, x, out):
+def head_linear(w, x, out, gate=None, gate_rows=None):
     """out[t, h, :M] = w[h] x[t, h, :K]: w [H, M, K] contiguous, x [T, H, >= K] and out [T, H, >= M] with any
-    row and head strides (bf16: multiples of 8 for x)."""
+    row and head strides (bf16: multiples of 8 for x).  ``gate`` [.., H * M] (any row stride): the result
+    times its sigmoid, row ``gate_rows[t]`` (int32) of it, or row t."""
     H, M, K = w.shape
     if x.is_cuda:
         N.call("us_head_linear", N.ptr(w), N.ptr(x), N.ptr(out), M * K, K, x.stride(0), x.stride(1),
-               out.stride(0), out.stride(1), H, min(M, out.shape[2]), K, x.shape[0], int(x.dtype == BF16),
-               N.stream())
+               out.stride(0), out.stride(1), H, min(M, out.shape[2]), K, x.shape[0], N.ptr(gate),
+               gate.stride(0) if gate is not None else 0, N.ptr(gate_rows), int(x.dtype == BF16), N.stream())
         return out
     M = min(M, out.shape[2])
-    out[..., :M] = torch.einsum("hmk,thk->thm", w[:, :M].float(), x[..., :K].float()).to(out.dtype)
+    y = torch.einsum("hmk,thk->thm", w[:, :M].float(), x[..., :K].float())
+    if gate is not None:
+        g = gate if gate_rows is None else gate[gate_rows.long()]
+        y = y * torch.sigmoid(g.float()).view(-1, H, M)
+    out[..., :M] = y.to(out.dtype)
     return out
 
 
@@ -194,7 +203,7 @@ def value_layout(d: LatentDims) -> int:
     return 64 if d.vdim <= 64 else 128
 
 
-def expanded_attention(q, w_kv, cpages, rpages, m: SeqMeta, page_table, d: LatentDims, out, least):
+def expanded_attention(q, w_kv, cpages, rpages, m: SeqMeta, page_table, d: LatentDims, out, least, gate=None):
     """Prompts: rows of the sequences that bring at least ``least`` rows, into ``out`` [T, >= H * vdim].
     q [T, H, columns of ``query_layout``], ``w_kv`` the stacked expansion [H * slabs * 64 | H * dv, Rp]."""
     T, H, W = q.shape
@@ -211,33 +220,35 @@ def expanded_attention(q, w_kv, cpages, rpages, m: SeqMeta, page_table, d: Laten
     kv = F.linear(c, w_kv)
     N.call("us_latent_flash", N.ptr(q), q.stride(0), N.ptr(kv), kv.stride(0), N.ptr(r), N.ptr(out),
            out.stride(0), N.ptr(m.cu), N.ptr(cu_k), B, T, Tk, H, W // 64 - 1, value_layout(d), d.vdim,
-           max(n for n in lengths if n >= least), d.window, d.scale, N.stream())
+           max(n for n in lengths if n >= least), d.window, d.scale, N.ptr(gate),
+           gate.stride(0) if gate is not None else 0, N.stream())
 
 
-def attend(q, off, w, cpages, rpages, m: SeqMeta, page_table, d: LatentDims, ldo, seq_lens=None, max_k=0):
+def attend(q, off, w, cpages, rpages, m: SeqMeta, page_table, d: LatentDims, ldo, seq_lens=None, max_k=0, gate=None):
     """Attention of query rows q [T, H, n] (unrotated channels first, the turned ones at column
     ``off``) over pages -> rows [T, ldo] of all heads' outputs (zero past H * vdim).  ``w``: 'absorb'
-    [H, Rp, dim], 'uv' [H, vdim, Rp] and, where ``expands``, 'kv'."""
+    [H, Rp, dim], 'uv' [H, vdim, Rp] and, where ``expands``, 'kv'.  ``gate`` [T, H * vdim] (a view of any
+    row stride): the outputs times its sigmoid."""
     T, H = q.shape[:2]
     n = H * d.vdim
     out = (torch.empty if ldo == n else torch.zeros)(T, ldo, dtype=q.dtype, device=q.device)
 
-    def absorbed(q, out, rows=None):
+    def absorbed(q, out, rows=None, gate_rows=None):
         ql = torch.empty(q.shape[0], H, cpages.shape[-1], dtype=q.dtype, device=q.device)
         head_linear(w["absorb"], q, ql)
         lat = latent_attention(ql, q[:, :, off:], cpages, rpages, m, page_table, d, seq_lens, max_k, rows)
-        head_linear(w["uv"], lat, out[:, :n].unflatten(1, (H, d.vdim)))
+        head_linear(w["uv"], lat, out[:, :n].unflatten(1, (H, d.vdim)), gate, gate_rows)
     if not (q.is_cuda and "kv" in w) or m.one_token:
         absorbed(q, out)
         return out
     least = EXPAND_ROWS if decode_fits(q, cpages, rpages) else 1
     short = m.short_rows(least)
     if short is None or short.shape[0] < T:
-        expanded_attention(q, w["kv"], cpages, rpages, m, page_table, d, out, least)
+        expanded_attention(q, w["kv"], cpages, rpages, m, page_table, d, out, least, gate)
     if short is not None and short.shape[0] == T:
         absorbed(q, out, short)
     elif short is not None:
         part = torch.zeros(short.shape[0], ldo, dtype=q.dtype, device=q.device)
-        absorbed(F.gather_rows(q.view(T, -1), short).view(-1, *q.shape[1:]), part, short)
+        absorbed(F.gather_rows(q.view(T, -1), short).view(-1, *q.shape[1:]), part, short, short)
         out.index_copy_(0, short.long(), part)
     return out

@@ -39,9 +39,10 @@ _SIGNATURES = {
     "us_device_info": (I, [P, P, P, P]),
     "us_gemm_wx": (I, [P, P, P, I, I, I, I, I, L, L, L, I, I, I, I, P, I, P, P, P, P, P, P, I, I, P]),
     "us_gemm_wx_hint": (I, [I]),
-    "us_linear_decode": (I, [P, P, P, P, I, I, I, L, L, L, I, I, I, P]),
+    "us_linear_decode": (I, [P, P, P, P, I, I, I, L, L, L, I, I, I, F, F, P]),
+    "us_gemm_wx_act": (I, [P, P, P, I, I, I, I, I, L, L, L, I, F, F, P, P, P, P, I, I, P]),
     "us_linear_decode_clamped": (I, [P, P, P, I, I, I, L, L, L, F, F, P]),
-    "us_gemm_f32": (I, [P, P, P, I, I, I, I, I, L, L, L, I, P, P, P, P, P, I, P]),
+    "us_gemm_f32": (I, [P, P, P, I, I, I, I, I, L, L, L, I, F, F, P, P, P, P, P, I, P]),
     "us_channel_delta_prep": (I, [P, L, I, I, I, I, P, P, P, P, L, P, P, P, P, P, P, P, P, P, P, P,
                                   I, I, I, I, I, I, I, I, I, P]),
     "us_general_delta_prep": (I, [P, L, I, I, I, I, P, L, P, P, P, I, I, I, F, I, P]),
@@ -61,6 +62,9 @@ _SIGNATURES = {
     "us_output_norm_add": (I, [P, P, P, F, I, P, P, P, P, F, F, I, I, I, I, F, I, P]),
     "us_stream_rows": (I, [P, P, P, P, F, I, I, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, P]),
     "us_plain_rows": (I, [P, P, F, I, P, P, P, P, I, P, P, F, P, P, P, P, I, I, I, I, F, P]),
+    "us_layer_rows": (I, [P, P, F, I, P, P, P, P, I, P, P, L, P, P, P, P, P, P, P, I, I, I, I, F, P]),
+    "us_grouped_topk": (I, [P, I, P, P, I, I, I, I, I, F, P]),
+    "us_grouped_route_sort_gather": (I, [P, I, P, P, I, I, I, I, I, F, I, I, P, P, P, P, P, P, P, P, I, P, P, P]),
     "us_gemm_wx_clamped": (I, [P, P, P, I, I, I, I, I, L, L, L, I, F, F, P, P, P, P, I, I, P]),
     "us_clamped_glu_f32": (I, [P, P, I, I, F, F, P]),
     "us_bigram_rows": (I, [P, P, P, P, P, P, I, I, I, L, L, I, P]),

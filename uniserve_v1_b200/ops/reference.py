@@ -409,6 +409,16 @@ def gelu_erf(x):
     return torch.nn.functional.gelu(x.float())
 
 
+def activation(z, act, ab=(0.0, 0.0)):
+    z = z.float()
+    if act == "relu2":
+        return z.clamp_min(0) ** 2
+    if act == "xielu":
+        a, b = ab
+        return torch.where(z > 0, a * z * z, b * (torch.expm1(z.clamp(max=0)) - z)) + 0.5 * z
+    return gelu_erf(z)
+
+
 def table_routes(tokens, table):
     """Experts of every token [T, top] (the CPU form of a layer's routes)."""
     return table[tokens.long()].long()
@@ -436,6 +446,16 @@ def scored_routes(logits, correction, top, experts):
     return ScoredRoutes(ids, w / (w.sum(-1, keepdim=True) + 1e-20), experts)
 
 
+def grouped_routes(logits, top, count, keep, scale):
+    s = logits.float().softmax(-1)
+    T, n = s.shape
+    best = s.view(T, count, -1).amax(-1)
+    kept = torch.sort(best, dim=-1, descending=True, stable=True).indices[:, :keep]
+    stays = torch.zeros(T, count, dtype=torch.bool).scatter_(1, kept, True).repeat_interleave(n // count, 1)
+    ids = torch.sort(s.masked_fill(~stays, -1.0), dim=-1, descending=True, stable=True).indices[:, :top]
+    return ScoredRoutes(ids, s.gather(1, ids) * scale, n)
+
+
 def mixture(m):
     """FP32 rows of an ``ops.functional.Mixture``; expert rows stand in route order."""
     ids, w = m.routes.ids, m.routes.weights
@@ -445,7 +465,23 @@ def mixture(m):
         own = (ids >= m.routes.experts)[..., None]
         y = torch.where(own, m.ident.float()[:, None], y)
     y = (w[..., None] * y).sum(1)
-    return y if m.shared is None else y + m.shared.float()
+    if m.shared is None:
+        return y
+    gate = 1.0 if m.shared_gate is None else torch.sigmoid(m.shared_gate)[:, None]
+    return y + gate * m.shared.float()
+
+
+def _layer_norm(x, w, b, eps, width):
+    inside = torch.arange(x.shape[1]) < width
+    d = (x - x.sum(-1, keepdim=True) / width) * inside
+    return d * torch.rsqrt(d.pow(2).sum(-1, keepdim=True) / width + eps) * w + b
+
+
+def layer_rows(source, residual, w, b, nxt, eps, width, dtype):
+    """(residual + layer norm of source, or source itself; the next rows in ``dtype``)."""
+    r = source if residual is None else residual + _layer_norm(source, w, b, eps, width)
+    x = r if nxt.weight is None else _layer_norm(r, nxt.weight, nxt.bias, eps, width)
+    return r, x.to(dtype, copy=True)
 
 
 def plain_rows(source, residual, gain, nxt, eps, width, dtype):
@@ -454,7 +490,7 @@ def plain_rows(source, residual, gain, nxt, eps, width, dtype):
     return r, (_rms(r, width, eps) * nxt.weight).to(dtype)
 
 
-def routed_mlp(x, routes, w_up, w_down, clamped=None):
+def routed_mlp(x, routes, w_up, w_down, clamped=None, act="gelu_erf"):
     """Expert rows in route order (row t * top + k belongs to token t's k-th expert; zero for experts
     past the last one with tensors)."""
     if isinstance(routes, ScoredRoutes):
@@ -470,7 +506,7 @@ def routed_mlp(x, routes, w_up, w_down, clamped=None):
         if clamped:
             h = clamped_linear(x[tok[sel]], w_up[e], *clamped)
         else:
-            h = gelu_erf(linear(x[tok[sel]], w_up[e], None, torch.float32)).to(x.dtype)
+            h = activation(linear(x[tok[sel]], w_up[e], None, torch.float32), act).to(x.dtype)
         y[sel] = linear(h, w_down[e], None, x.dtype)
     return y
 
