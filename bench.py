@@ -631,10 +631,11 @@ def qwen3_record(job: Job) -> dict:
 
 # ------------------------------------------------- decoders of unlike layers --
 def layered_record(job: Job, family: str) -> dict:
-    """Prefill and decode throughput of the Nepevik, Zonopel or Tadinex decoder at a production-like layer
+    """Prefill and decode throughput of the Nepevik, Zonopel, Tadinex or Nopuzen decoder at a production-like layer
     size (random weights) through ``LLMEngine``, beside existing models of equal size: Nepevik beside
     the Qwen3.5-style hybrid (gated delta net, dense-state engine) and Qwen3-MoE (attention in every
-    layer, the same paged engine), Zonopel and Tadinex beside Nepevik and Qwen3-MoE.  One GPU.
+    layer, the same paged engine), Zonopel and Tadinex beside Nepevik and Qwen3-MoE, Nopuzen beside Zonopel
+    (latent attention), Tadinex (experts, shared expert) and Qwen3-MoE.  One GPU.
 
     ``value``: output tokens/s of the device-timed decode step of all concurrent requests (graph
     replays); ``sizes``: the same and the prompt throughput per (requests, prompt length)."""
@@ -643,6 +644,7 @@ def layered_record(job: Job, family: str) -> dict:
     from uniserve_v1_b200.engine.engine import LLMEngine
     from uniserve_v1_b200.engine.types import SamplingParams
     from uniserve_v1_b200.models.nepevik import NepevikConfig, NepevikModel
+    from uniserve_v1_b200.models.nopuzen import NopuzenConfig, NopuzenModel
     from uniserve_v1_b200.models.qwen3_5 import Qwen35Config, Qwen35MoeModel
     from uniserve_v1_b200.models.qwen3_moe import Qwen3MoeConfig, Qwen3MoeModel
     from uniserve_v1_b200.models.tadinex import TadinexConfig, TadinexModel
@@ -658,7 +660,8 @@ def layered_record(job: Job, family: str) -> dict:
     ncfg = NepevikConfig.bench(layers)
     zcfg = ZonopelConfig.bench(layers)
     tcfg = TadinexConfig.bench(layers)
-    ncfg.vocab_size = zcfg.vocab_size = tcfg.vocab_size = vocab
+    pcfg = NopuzenConfig.bench(layers)
+    ncfg.vocab_size = zcfg.vocab_size = tcfg.vocab_size = pcfg.vocab_size = vocab
     hcfg = Qwen35Config(vocab_size=vocab, hidden_size=2048, num_hidden_layers=layers,
                         num_attention_heads=32, num_key_value_heads=4, head_dim=128,
                         linear_num_key_heads=16, linear_num_value_heads=32, num_experts=64,
@@ -724,6 +727,7 @@ def layered_record(job: Job, family: str) -> dict:
 
     out, clocks, launches, head = [], None, 0, None
     models = {
+        "nopuzen": (lambda: NopuzenModel(pcfg, dev).init_random(0), paged, True),
         "tadinex": (lambda: TadinexModel(tcfg, dev).init_random(0), paged, True),
         "zonopel": (lambda: ZonopelModel(zcfg, dev).init_random(0), paged, True),
         "nepevik": (lambda: NepevikModel(ncfg, dev).init_random(0), paged, True),
@@ -733,7 +737,7 @@ def layered_record(job: Job, family: str) -> dict:
                                      state_cache_entries=0), False),
         "qwen3-moe": (lambda: Qwen3MoeModel(qcfg, dev).init_random(0), paged, True)}
     beside = {"nepevik": ("qwen3.5-style hybrid", "qwen3-moe"), "zonopel": ("nepevik", "qwen3-moe"),
-              "tadinex": ("nepevik", "qwen3-moe")}
+              "tadinex": ("nepevik", "qwen3-moe"), "nopuzen": ("zonopel", "tadinex", "qwen3-moe")}
     for name in (family,) + (() if args.alone else beside[family]):
         build_model, make, graphs = models[name]
         model = build_model()
@@ -773,12 +777,12 @@ def layered_record(job: Job, family: str) -> dict:
 
 def main() -> int:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--workload", default="all", choices=["all", "qwen3-moe", "fasth3", "nepevik", "zonopel", "tadinex"],
+    ap.add_argument("--workload", default="all", choices=["all", "qwen3-moe", "fasth3", "nepevik", "zonopel", "tadinex", "nopuzen"],
                     help="all (default): the FastH3 clip latency as the headline with the "
-                         "Qwen3-MoE record nested; or one of the two alone; nepevik, zonopel, tadinex: that decoder's "
+                         "Qwen3-MoE record nested; or one of the two alone; nepevik, zonopel, tadinex, nopuzen: that decoder's "
                          "throughput beside models of equal size (one GPU, not part of all)")
     ap.add_argument("--alone", "--only-nepevik", dest="alone", action="store_true",
-                    help="nepevik, zonopel, tadinex: without the models it is compared with")
+                    help="nepevik, zonopel, tadinex, nopuzen: without the models it is compared with")
     ap.add_argument("--frames", type=int, default=0, help="fasth3: frame count (rule 17n + 5)")
     ap.add_argument("--mlp-fp8", action="store_true",
                     help="fasth3: feed-forward projections in FP8 (per-tensor weights, per-row "
@@ -834,7 +838,7 @@ def main() -> int:
             line["metric"] = "FastH3 8-step clip latency (s); Qwen3-MoE output tokens/s nested"
             line["qwen3_moe"] = q
             line["gpu_launches"] = line["gpu_launches"] + q.get("gpu_launches", 0)
-    if args.workload in ("nepevik", "zonopel", "tadinex"):
+    if args.workload in ("nepevik", "zonopel", "tadinex", "nopuzen"):
         line = layered_record(job, args.workload)
     if job.rank == 0 and line:
         print(json.dumps(line))

@@ -67,7 +67,7 @@ class LayerSpec:
 
 def _rotation(i, m, most) -> Rotation:
     r = m.get("rot") or {}
-    rot = Rotation(int(r.get("dims") or 0), float(r.get("base", 10000.0)))
+    rot = Rotation(int(r.get("dims", most)) if r else 0, float(r.get("base", 10000.0)))
     if rot.dims % 2 or rot.dims > most:
         raise ValueError(f"layer {i}: {rot.dims} turned channels of {most}")
     if r.get("scaling"):
@@ -133,10 +133,10 @@ class NopuzenConfig:
     def bench(cls, layers: int = 8) -> "NopuzenConfig":
         """Layer sizes of a mid-size production decoder: width 2048, 32 latent-attention heads of 128 + 64
         over latents of 512, sigmoid attention with 32 / 4 heads of 128, 64 experts of 768 in eight groups
-        of which four stay, four per token; one attention layer and one dense feed-forward in four."""
+        of which three stay, four per token; one attention layer and one dense feed-forward in four."""
         at = WA.WindowDims(32, 4, 128, 128, 128 ** -0.5, 0)
         la = LA.LatentDims(32, 128, 64, 128, 512, 1536, 192 ** -0.5, 0)
-        moe = ExpertsSpec(64, 4, 768, 2.5, (8, 4), 1024)
+        moe = ExpertsSpec(64, 4, 768, 2.5, (8, 3), 1024)
         yarn = Rotation(64, 1e5, (8.0, 4096.0, 32.0, 1.0))
         return cls(151936, 2048, 1e-6, [
             LayerSpec("attention", at, Rotation(64, 1e6), 30.0, ff=6144) if i % 4 == 0 else

@@ -1,5 +1,5 @@
-"""Kernels of the delta-rule, head-mixing, table- and score-routed, state-space, linear-attention, latent-
-and windowed-attention layers beside the like kernels of the hybrid and Qwen3 decoders at equal sizes, each with its roofline
+"""Kernels of the delta-rule, head-mixing, table- and score-routed, state-space, linear-attention, latent-,
+windowed- and sigmoid-attention layers beside the like kernels of the hybrid and Qwen3 decoders at equal sizes, each with its roofline
 fraction.
 
     python -m uniserve_v1_b200.tools.opbench_mixers [--only NAME,...] [--batch 64] [--rows 8192]
@@ -185,6 +185,18 @@ def main():
              4.0 * n * 1024 * W)
         case(f"linear_gated_{kind} (like)", lambda: F.linear_gated(y, s13), 2.0 * (2048 * W + n * (W + 1024)),
              4.0 * n * 1024 * W)
+        # ungated experts by groups, ungated products with their activations in the epilogue
+        case(f"grouped_routes_{kind}", lambda: F.grouped_routes(logits, E, top, (8, 3), 2.5, y, sync))
+        gr = F.grouped_routes(logits, E, top, (8, 3), 2.5, y, sync)
+        gr.xp = None
+        case(f"square_relu_experts_{kind}", lambda: F.routed_mlp(y, gr, up, down, act="relu2"),
+             wb + n * top * (2 * W + I) * 2.0, 4.0 * n * top * I * W)
+        case(f"square_relu_linear_{kind}", lambda: F.linear(y, s13[:1024], act="relu2"), 2.0 * (1024 * W + n * (W + 1024)),
+             2.0 * n * 1024 * W)
+        wup = rnd(6144, W)
+        case(f"xielu_linear_{kind}", lambda: F.linear(y, wup, act="xielu", act_ab=(0.3, 0.8)),
+             2.0 * (6144 * W + n * (W + 6144)), 2.0 * n * 6144 * W)
+        case(f"linear_{kind} (like)", lambda: F.linear(y, wup), 2.0 * (6144 * W + n * (W + 6144)), 2.0 * n * 6144 * W)
         pw = F.NextRows(rnd(W, dtype=torch.float32))
         case(f"add_plain_rows_{kind}", lambda: F.add_plain_rows(y, res, 0.7, pw, 1e-6, W), n * W * (2 + 4 + 4 + 2.0))
         mix = F.Mixture(rows, F.Routes(*[None] * 2, perm, *[None] * 5, 0, 0, 0, wts), y, shared)
@@ -248,8 +260,26 @@ def main():
                 kx, vx = rnd(n, G * D), rnd(n, G * V)
                 case(f"window_flash_prefill, window {win}", lambda: N.call(
                     "us_window_flash", N.ptr(q4), Hq * D, N.ptr(kx), G * D, N.ptr(vx), G * V, N.ptr(out_a), Hq * V,
-                    N.ptr(m.cu), N.ptr(cuk), 1, n, n, Hq, G, 2, 128, 128, n, win, 0.088, N.ptr(sink), 1.0, N.stream()),
-                    None, pairs * Hq * 2.0 * (D + V))
+                    N.ptr(m.cu), N.ptr(cuk), 1, n, n, Hq, G, 2, 128, 128, n, win, 0.088, N.ptr(sink), 1.0, None, 0,
+                    N.stream()), None, pairs * Hq * 2.0 * (D + V))
+        # ---- attention without a softmax, every earlier key, a gate per head ----
+        sd = WA.WindowDims(Hq, G, D, V, 0.088, 0)
+        sig = WA.SigmoidScores(torch.ones(Hq, device=dev), torch.full((Hq,), -6.0, device=dev), 30.0)
+        sgate = rnd(n, Hq)
+        case(f"sigmoid_prep_{kind}", lambda: WA.prep(xr, (0, Hq * D, (Hq + G) * D), sd, hq, hk, wfreq, 1.0, pos, slots, kc, vc,
+                                                     1e-6, neighbours=True), n * (2 * Hq * D + 4 * G * D) * 2.0)
+        if kind == "decode":
+            case("sigmoid_attention_decode", lambda: WA.attend(q4, kc, vc, m, pt, None, sd, out_a, 1.0, sl, ctx, sig=sig,
+                                                               gate=sgate), 2.0 * B * 2001 * G * (D + V))
+        else:
+            pairs = n * (n + 1) / 2
+            case("sigmoid_attention_prefill (gather and attention)", lambda: WA.attend(
+                q4, kc, vc, m, pt, None, sd, out_a, 1.0, None, n, sig=sig, gate=sgate), None, pairs * Hq * 2.0 * (D + V))
+            for what, qs in (("", q4), (", scores deep in the cap", q4 * 30.0)):
+                case(f"sigmoid_flash_prefill{what}", lambda: N.call(
+                    "us_sigmoid_flash", N.ptr(qs), Hq * D, N.ptr(kx), G * D, N.ptr(vx), G * V, N.ptr(out_a), Hq * V,
+                    N.ptr(m.cu), N.ptr(cuk), 1, n, n, Hq, G, 2, 128, 128, n, 0, 0.088, N.ptr(sig.temp), N.ptr(sig.shift),
+                    30.0, 1.0, N.ptr(sgate), Hq, N.stream()), None, pairs * Hq * 2.0 * (D + V))
         # ---- linear attention: 16 heads x 128 x 128 with a fixed decay ----
         fd = SS.fixed_decay_dims(16, 128, 128)
         fw = {"offs": (0, fd.inner, None), "norm": rnd(fd.inner, dtype=torch.float32),
@@ -294,6 +324,12 @@ def main():
             y, res, nw32, F.NextRows(nw32, mu, shift_pool, m), 1e-6, W), n * W * (2 + 4 + 4 + 2.0))
         zf, pact = rnd(n, 8192), torch.tensor([0.4, 0.3, 0.1, 0.2], device=dev)
         case(f"poly_norm_{kind}", lambda: F.poly_norm_(zf, pact, 8192, 1e-6), n * 8192 * 4.0)
+        nb32 = rnd(W, dtype=torch.float32)
+        case(f"add_layer_rows_{kind}", lambda: F.add_layer_rows(y, res, nw32, nb32, F.NextRows(None), 1e-6, W),
+             n * W * (2 + 4 + 4 + 2.0))
+        lmix = F.Mixture(rows, F.Routes(*[None] * 2, perm, *[None] * 5, 0, 0, 0, wts), None, shared, logits[:, E])
+        case(f"add_layer_rows_mixture_{kind}", lambda: F.add_layer_rows(lmix, res, nw32, nb32, F.NextRows(None), 1e-6, W),
+             n * W * (2 * top + 2 + 4 + 4 + 2.0))
         # ---- latent attention: 32 heads of 128 + 64, latents of 512, window 1024 ----
         ld = LA.LatentDims(32, 128, 64, 128, 512, 1536, 192 ** -0.5, 1024)
         cpg, rpg = rnd(seqs * per + 1, page, 1, 512), rnd(seqs * per + 1, page, 1, 64)
@@ -309,7 +345,17 @@ def main():
              32 * 512 * 128 * 2.0 + n * 32 * 640 * 2.0, 2.0 * n * 32 * 512 * 128)
         case(f"head_linear_values_{kind}", lambda: LA.head_linear(wuv, lat, att),
              32 * 512 * 128 * 2.0 + n * 32 * 640 * 2.0, 2.0 * n * 32 * 512 * 128)
+        lgate = rnd(n, 32 * 128)
+        case(f"head_linear_values_gated_{kind}", lambda: LA.head_linear(wuv, lat, att, lgate),
+             32 * 512 * 128 * 2.0 + n * 32 * 768 * 2.0, 2.0 * n * 32 * 512 * 128)
+        case(f"latent_prep_halves_{kind}", lambda: LA.latent_prep_(lx, (0, 1536, 2048), ld, lq, lc, freq, pos, slots, cpg,
+                                                                   rpg, 1e-6, 1.2, True), n * (2 * 1536 + 2 * 576) * 2.0)
+        case(f"rotate_heads_halves_{kind}", lambda: LA.rotate_heads_(q3, 128, pos, freq, 1.2, True), n * 32 * 64 * 4.0)
         if kind == "decode":
+            le = LA.LatentDims(32, 128, 64, 128, 512, 1536, 192 ** -0.5, 0)
+            case("latent_attention_decode, no window", lambda: LA.latent_attention(
+                ql, q3[:, :, 128:], cpg, rpg, m, pt, le, seq_lens=sl, max_k=ctx),
+                2.0 * B * 2001 * 576 + n * 32 * (576 + 512) * 2.0, 2001.0 * B * 32 * 2 * (576 + 512))
             case("latent_attention_decode", lambda: LA.latent_attention(
                 ql, q3[:, :, 128:], cpg, rpg, m, pt, ld, seq_lens=sl, max_k=ctx),
                 2.0 * B * 1024 * 576 + n * 32 * (576 + 512) * 2.0, 1024.0 * B * 32 * 2 * (576 + 512))
@@ -322,12 +368,21 @@ def main():
                 case(f"latent_attention_prefill, window {win} (expansion and attention)",
                      lambda: LA.attend(q3, 128, wl, cpg, rpg, m, pt, lw, 32 * 128), None,
                      pairs * 32 * 2.0 * (192 + 128) + 2.0 * n * 512 * 32 * 256)
+                if not win:
+                    case("latent_attention_prefill, gated (expansion and attention)",
+                         lambda: LA.attend(q3, 128, wl, cpg, rpg, m, pt, lw, 32 * 128, gate=lgate), None,
+                         pairs * 32 * 2.0 * (192 + 128) + 2.0 * n * 512 * 32 * 256)
                 kvx, rx = rnd(n, 32 * 256), rnd(n, 64)
                 cuk = i32([0, n])
                 case(f"latent_flash_prefill, window {win}", lambda: N.call(
                     "us_latent_flash", N.ptr(q3), 32 * 192, N.ptr(kvx), 32 * 256, N.ptr(rx), N.ptr(att), 32 * 128,
-                    N.ptr(m.cu), N.ptr(cuk), 1, n, n, 32, 2, 128, 128, n, win, 0.07, N.stream()), None,
+                    N.ptr(m.cu), N.ptr(cuk), 1, n, n, 32, 2, 128, 128, n, win, 0.07, None, 0, N.stream()), None,
                     pairs * 32 * 2.0 * (192 + 128))
+                if not win:
+                    case("latent_flash_prefill, gated", lambda: N.call(
+                        "us_latent_flash", N.ptr(q3), 32 * 192, N.ptr(kvx), 32 * 256, N.ptr(rx), N.ptr(att), 32 * 128,
+                        N.ptr(m.cu), N.ptr(cuk), 1, n, n, 32, 2, 128, 128, n, win, 0.07, N.ptr(lgate), 32 * 128,
+                        N.stream()), None, pairs * 32 * 2.0 * (192 + 128))
 
 
 def F_flash(q, k, v, cu, n):
