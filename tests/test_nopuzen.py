@@ -721,6 +721,53 @@ def test_latent_norms_and_scaled_rotation_in_halves_alone(form, H, D, RD, R, Q, 
     settled(dev)
 
 
+@pytest.mark.parametrize("form", FORMS)
+@pytest.mark.parametrize("rows", [1, 3, 9])
+def test_single_rows_over_thousands_of_keys(form, rows):
+    """Both mixers' decode steps with their keys split over many CTAs: a key stands out at the first and
+    last key, at tile and split borders."""
+    dev, dt = form
+    g, n, page, scale = gen(rows), 2120, 16, 0.15
+    lens = [n - 7 * r for r in range(rows)]
+    marks = [0, 1, 15, 16, 63, 64, 127, 128, 131, 132, 255, 256, 511, 512, 1023, 1024, 2047, 2048, n - 70]
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+    m, sl = seq_meta([1] * rows, [t - 1 for t in lens], list(range(rows)), dev), i32(lens)
+    pad = lambda x, w: torch.nn.functional.pad(x, (0, w - x.shape[-1])).contiguous()
+    H, G, D, V = 6, 2, 24, 40
+    k, v = ([as_typed(form, rnd(g, t, G, w, std=0.5)) for t in lens] for w in (D, V))
+    (kp, vp), pt = paged([k, v], page, dev, dt, g)
+    temp, shift = torch.linspace(0.7, 1.3, H), torch.linspace(-9.0, -6.0, H)
+    d, sig = WA.WindowDims(H, G, D, V, scale, 0), WA.SigmoidScores(temp.to(dev), shift.to(dev), 20.0)
+    Hl, R, RD = 20, 64, 16
+    c, r = ([as_typed(form, rnd(g, t, w, std=0.5)) for t in lens] for w in (R, RD))
+    (cp, rp), ptl = paged([[x[:, None] for x in c], [x[:, None] for x in r]], page, dev, dt, g)
+    ld = LA.LatentDims(Hl, 8, RD, 8, R, 8, scale, 0)
+    of = torch.arange(H) // (H // G)
+    for j in marks + [None]:                        # None: every query points along its own key
+        at = [t - 1 if j is None else j for t in lens]
+        q = torch.stack([x[a][of] / x[a][of].norm(dim=-1, keepdim=True) ** 2 * (10.0 / scale) for x, a in zip(k, at)])
+        q = as_typed(form, q)
+        out = torch.zeros(rows, H * V, device=dev, dtype=dt)
+        WA.attend(to(form, pad(q, WA.query_width(d, dt))), kp, vp, m, pt, None, d, out, 1.0, sl, n, sig=sig)
+        want = torch.stack([last_row(a, b, e, scale, temp, 20.0, shift) for a, b, e in zip(q, k, v)])
+        close_rows(out, want.flatten(1), dt, f"sigmoid, key {j}", 0.5)
+        keys = [torch.cat([a, b], -1) for a, b in zip(c, r)]
+        ql = torch.stack([x[a] / x[a].norm() ** 2 * (14.0 / scale) * torch.linspace(0.8, 1.2, Hl)[:, None] for x, a in zip(keys, at)])
+        ql = as_typed(form, ql)
+        qd = to(form, ql)
+        got = LA.latent_attention(qd[..., :R].contiguous(), qd[..., R:].contiguous(), cp, rp, m, ptl, ld, seq_lens=sl, max_k=n)
+        ref = torch.stack([torch.softmax(a @ b.T * scale, -1) @ e for a, b, e in zip(ql, keys, c)])
+        close_rows(got.flatten(1), ref.flatten(1), dt, f"latent, key {j}", 1.0)
+    settled(dev)
+
+
+def last_row(q, k, v, scale, temp, cap, shift):
+    """``sigmoid_attention`` of one query [H, D] that sees every key."""
+    of = torch.arange(q.shape[0]) // (q.shape[0] // k.shape[1])
+    s = torch.einsum("hd,jhd->hj", q, k[:, of]) * scale * temp[:, None]
+    return torch.einsum("hj,jhv->hv", P.sigmoid(cap * torch.tanh(s / cap) + shift[:, None]), v[:, of])
+
+
 # --------------------------------------------------- configuration, loading --
 def test_configuration_and_loading_errors():
     c = CONFIGS["odd"]

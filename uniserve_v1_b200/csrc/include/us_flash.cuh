@@ -97,4 +97,16 @@ __device__ __forceinline__ float max3(float a, float b, float c) {
   return d;
 }
 
+// the largest magnitude of three
+__device__ __forceinline__ float max3_abs(float a, float b, float c) {
+  float d;
+  asm("max.abs.f32 %0, %1, %2, %3;" : "=f"(d) : "f"(a), "f"(b), "f"(c));
+  return d;
+}
+__device__ __forceinline__ float rcpf(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
 }  // namespace flash

@@ -18,6 +18,7 @@ constexpr int kTile = 64;            // keys
 constexpr int kRot = 64;             // rotated channels, padded
 constexpr int kPRow = kTile * 2 + 16;
 constexpr int kSRow = kTile + 8;     // floats of a head's scores (rows apart hit other banks)
+constexpr int kMostSplits = 16;      // more than 8 CTAs to a cluster where the device allows them
 
 struct DecodeArgs {
   const __nv_bfloat16 *ql, *qr;
@@ -270,25 +271,25 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const Decode
   if (a.splits > 1) tc::cluster_sync();
   // every CTA of the cluster finishes a share of the heads' columns, adding the splits in order:
   // first each split's factor per head (in `part`), then the columns
-  float* wgt = part;                                             // [HT][8]
+  float* wgt = part;                                             // [HT][kMostSplits]
   for (int h = tid; h < nh; h += kThreads) {
-    float m[8], l[8], top = -INFINITY, den = 0.f;
+    float m[kMostSplits], l[kMostSplits], top = -INFINITY, den = 0.f;
     const uint32_t am = (uint32_t)__cvta_generic_to_shared(&mx[h]);
     const uint32_t al = (uint32_t)__cvta_generic_to_shared(&sum[h]);
 #pragma unroll
-    for (int p = 0; p < 8; ++p) {
+    for (int p = 0; p < kMostSplits; ++p) {
       m[p] = p < a.splits ? (a.splits > 1 ? tc::ld_dsmem_f32(tc::map_to_cta(am, p)) : mx[h]) : -INFINITY;
       l[p] = p < a.splits ? (a.splits > 1 ? tc::ld_dsmem_f32(tc::map_to_cta(al, p)) : sum[h]) : 0.f;
     }
 #pragma unroll
-    for (int p = 0; p < 8; ++p) top = fmaxf(top, m[p]);
+    for (int p = 0; p < kMostSplits; ++p) top = fmaxf(top, m[p]);
 #pragma unroll
-    for (int p = 0; p < 8; ++p) {
+    for (int p = 0; p < kMostSplits; ++p) {
       m[p] = top > -INFINITY ? ex2(m[p] - top) : 0.f;
       den = fmaf(m[p], l[p], den);
     }
 #pragma unroll
-    for (int p = 0; p < 8; ++p) wgt[h * 8 + p] = den > 0.f ? m[p] / den : 0.f;
+    for (int p = 0; p < kMostSplits; ++p) wgt[h * kMostSplits + p] = den > 0.f ? m[p] / den : 0.f;
   }
   __syncthreads();
   const int cols = a.hso, quads = (cols + 3) / 4;
@@ -298,21 +299,23 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const Decode
     float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
     if (c < RP) {
       const uint32_t ao = (uint32_t)__cvta_generic_to_shared(os + h * RP + c);
-      float4 o4[8];
+      for (int p0 = 0; p0 < a.splits; p0 += 8) {
+        float4 o4[8];
 #pragma unroll
-      for (int p = 0; p < 8; ++p)
-        if (p < a.splits)
-          o4[p] = a.splits > 1 ? tc::ld_dsmem_f32x4(tc::map_to_cta(ao, p))
-                               : *reinterpret_cast<const float4*>(os + h * RP + c);
+        for (int p = 0; p < 8; ++p)
+          if (p0 + p < a.splits)
+            o4[p] = a.splits > 1 ? tc::ld_dsmem_f32x4(tc::map_to_cta(ao, p0 + p))
+                                 : *reinterpret_cast<const float4*>(os + h * RP + c);
 #pragma unroll
-      for (int p = 0; p < 8; ++p)
-        if (p < a.splits) {
-          const float f = wgt[h * 8 + p];
-          v.x = fmaf(f, o4[p].x, v.x);
-          v.y = fmaf(f, o4[p].y, v.y);
-          v.z = fmaf(f, o4[p].z, v.z);
-          v.w = fmaf(f, o4[p].w, v.w);
-        }
+        for (int p = 0; p < 8; ++p)
+          if (p0 + p < a.splits) {
+            const float f = wgt[h * kMostSplits + p0 + p];
+            v.x = fmaf(f, o4[p].x, v.x);
+            v.y = fmaf(f, o4[p].y, v.y);
+            v.z = fmaf(f, o4[p].z, v.z);
+            v.w = fmaf(f, o4[p].w, v.w);
+          }
+      }
     }
     __nv_bfloat16* dst = a.out + t * a.ldo + (long long)(h0 + h) * a.hso + c;
     const float f[4] = {c < a.R ? v.x : 0.f, c + 1 < a.R ? v.y : 0.f, c + 2 < a.R ? v.z : 0.f,
@@ -329,7 +332,7 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const Decode
 }
 
 template <int RP, int MT>
-int launch_decode(const DecodeArgs& a, int rows, cudaStream_t stream) {
+int launch_decode(DecodeArgs a, int rows, cudaStream_t stream) {
   constexpr int PC = RP / 8 + kRot / 8, HT = 16 * MT;
   constexpr size_t smem = 2 * (size_t)kTile * PC * 16 + (8 / MT) * HT * kSRow * 4 + HT * kPRow + 3 * HT * 4;
   static_assert(2 * kTile * PC * 16 >= HT * RP * 4, "partial outputs fit the key tiles");
@@ -339,6 +342,11 @@ int launch_decode(const DecodeArgs& a, int rows, cudaStream_t stream) {
                                        cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     configured = true;
   }
+  if (a.splits > 8) {
+    static const int most = us::cluster_limit(latent_decode_kernel<RP, MT>, kMostSplits, kThreads, smem);
+    if (a.splits > most) a.splits = most;
+  }
+  static_assert((8 / MT) * HT * kSRow >= HT * kMostSplits, "the splits' factors fit the score slices");
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3(a.splits, us::ceil_div(a.H, HT), rows);
   cfg.blockDim = dim3(kThreads);
@@ -369,7 +377,7 @@ US_API int us_latent_decode(const void* ql, long long ldql, int hsql, const void
                             int splits, float scale, void* stream_) {
   US_REQUIRE(ql && qr && cpages && rpages && out && cu && pos && page_table && count >= 0 && B >= 1 &&
              H >= 1 && R >= 1 && RD >= 0 && page >= 1 && hso >= R && ldc >= R && ldr >= RD &&
-             ((uintptr_t)out % 8) == 0 && splits >= 1 && splits <= 8 && count <= 65535 && (rows || count == B));
+             ((uintptr_t)out % 8) == 0 && splits >= 1 && splits <= kMostSplits && count <= 65535 && (rows || count == B));
   US_REQUIRE((ldc % 8) == 0 && (ldr % 8) == 0 && (ldql % 2) == 0 && (hsql % 2) == 0 && (ldqr % 2) == 0 &&
              (hsqr % 2) == 0 && ((uintptr_t)cpages % 16) == 0 && ((uintptr_t)rpages % 16) == 0 &&
              ((uintptr_t)ql % 4) == 0 && ((uintptr_t)qr % 4) == 0);
@@ -380,7 +388,9 @@ US_API int us_latent_decode(const void* ql, long long ldql, int hsql, const void
                (__nv_bfloat16*)out, ldo, hso, rows, cu, pos, seq_lens, page_table, B, H, R, RD, page,
                max_pages, window, splits, scale * 1.4426950408889634f};
   cudaStream_t stream = (cudaStream_t)stream_;
-#define US_LATENT(RP) return H <= 16 ? launch_decode<RP, 1>(a, count, stream) : launch_decode<RP, 2>(a, count, stream)
+  // 16 heads to a CTA while there are few (clusters of one CTA per SM do not fill every SM of a GPC)
+  const bool narrow = H <= 16 || (long long)count * us::ceil_div(H, 16) * splits <= 64;
+#define US_LATENT(RP) return narrow ? launch_decode<RP, 1>(a, count, stream) : launch_decode<RP, 2>(a, count, stream)
   if (ldc <= 64) US_LATENT(64);
   if (ldc <= 128) US_LATENT(128);
   if (ldc <= 256) US_LATENT(256);

@@ -108,16 +108,79 @@ struct FlashArgs {
   float scale, cap;
 };
 
-__device__ __forceinline__ float rcpf(float x) {
-  float y;
-  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
+// tanh(z) / z as polynomials in u = z^2 (least maximum error: 1.3e-8 up to |z| = 1/2, 3.8e-8 up to 6/5)
+constexpr float kTanhNear = 0.5f, kTanhFar = 1.2f;
+__device__ constexpr float kNear[5] = {1.f, -0.33333075046539307f, 0.13324907422065735f, -0.05299423262476921f,
+                                       0.017151299864053726f};
+__device__ constexpr float kFar[8] = {1.f, -0.3333297073841095f, 0.13327667117118835f, -0.053627558052539825f,
+                                      0.020839421078562737f, -0.007092796266078949f, 0.001742084277793765f,
+                                      -0.00021388338063843548f};
+constexpr float kLog2e = 1.4426950408889634f;
+constexpr float kExpMost = 60.f;         // exponents (base 2) up to here keep the product of two sums finite
 
-// tanh(z) / z as a polynomial in u = z^2, u <= 1/4 (least maximum error, 1.3e-8)
-constexpr float kTanhMost = 0.5f;
-constexpr float kT1 = -0.33333075046539307f, kT2 = 0.13324907422065735f, kT3 = -0.05299423262476921f,
-                kT4 = 0.017151299864053726f;
+// Weights of a row's scores, two at a time with one reciprocal: sigmoid(cap tanh(z) + shift), z = score * f.
+struct SigWeights {
+  float near, far;                       // scores up to here take a polynomial; up to `near` no exponent passes kExpMost
+  float f, c, f_shift;                   // exponent (base 2) of the negated argument: c * tanh(score * f) + f_shift
+  __device__ __forceinline__ SigWeights(float f_, float cap, float shift)
+      : f(f_), c(-cap * kLog2e), f_shift(-shift * kLog2e) {
+    near = fminf(kTanhNear, (kExpMost / kLog2e - fabsf(shift)) / cap) / fabsf(f);
+    far = kTanhFar / fabsf(f);
+  }
+  // two exponents -> two weights as bf16
+  static __device__ __forceinline__ uint32_t weigh(float x0, float x1) {
+    float a0, a1;
+    unpack2(add2(pack2(ex2f(x0), ex2f(x1)), pack2(1.f, 1.f)), a0, a1);
+    const float r = rcpf(a0 * a1);
+    return us::pack_bf(r * a1, r * a0);
+  }
+  // score * (k_0 + k_1 score^2 + ..) with the factors of score, cap and base in the coefficients
+  template <int N, bool kClamp>
+  __device__ __forceinline__ void by_polynomial(const uint32_t (&v)[32], uint32_t (&w)[16], const float (&k)[N]) const {
+    unsigned long long b[N];
+    float at = c * f;
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      b[i] = pack2(k[i] * at, k[i] * at);
+      at *= f * f;
+    }
+    const unsigned long long sh = pack2(f_shift, f_shift);
+#pragma unroll
+    for (int i = 0; i < 32; i += 2) {
+      const unsigned long long s = pack2(__uint_as_float(v[i]), __uint_as_float(v[i + 1])), u = mul2(s, s);
+      unsigned long long p = b[N - 1];
+#pragma unroll
+      for (int e = N - 2; e >= 0; --e) p = fma2(p, u, b[e]);
+      float x0, x1;
+      unpack2(fma2(s, p, sh), x0, x1);
+      w[i >> 1] = kClamp ? weigh(fminf(x0, kExpMost), fminf(x1, kExpMost)) : weigh(x0, x1);
+    }
+  }
+  __device__ __forceinline__ void operator()(const uint32_t (&v)[32], uint32_t (&w)[16]) const {
+    float top[2] = {0.f, 0.f};
+#pragma unroll
+    for (int i = 0; i < 32; i += 4)
+#pragma unroll
+      for (int e = 0; e < 2; ++e)
+        top[e] = max3_abs(top[e], __uint_as_float(v[i + 2 * e]), __uint_as_float(v[i + 2 * e + 1]));
+    const float most = fmaxf(top[0], top[1]);
+    if (__all_sync(0xffffffffu, most <= near)) {
+      by_polynomial<5, false>(v, w, {kNear[0], kNear[1], kNear[2], kNear[3], kNear[4]});
+    } else if (__all_sync(0xffffffffu, most <= far)) {
+      by_polynomial<8, true>(v, w, {kFar[0], kFar[1], kFar[2], kFar[3], kFar[4], kFar[5], kFar[6], kFar[7]});
+    } else {
+      const float f_e = 2.f * kLog2e * f;    // e^{2 z} = 2^{score f_e}, tanh(z) = 1 - 2 / (e^{2 z} + 1)
+#pragma unroll
+      for (int i = 0; i < 32; i += 2) {
+        const float e0 = ex2f(fminf(__uint_as_float(v[i]) * f_e, kExpMost)) + 1.f;
+        const float e1 = ex2f(fminf(__uint_as_float(v[i + 1]) * f_e, kExpMost)) + 1.f;
+        const float r = -2.f * rcpf(e0 * e1);
+        const float t0 = fmaf(r, e1, 1.f), t1 = fmaf(r, e0, 1.f);
+        w[i >> 1] = weigh(fminf(fmaf(t0, c, f_shift), kExpMost), fminf(fmaf(t1, c, f_shift), kExpMost));
+      }
+    }
+  }
+};
 
 __device__ __forceinline__ float sigmoid_of(__nv_bfloat16 x) { return 1.f / (1.f + __expf(-us::bf2f(x))); }
 
@@ -310,8 +373,7 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     const int q_idx = q0 + x * kBM + r;
     const int j0 = x ? jb[1] : jb[0], j1 = x ? je[1] : je[0];
     float m_used = -INFINITY, l_sum = 0.f;
-    const float f_z = kSig ? a.scale * a.temp[h] / a.cap : 0.f;
-    const float f_cap = -a.cap * 1.4426950408889634f, f_shift = kSig ? -a.shift[h] * 1.4426950408889634f : 0.f;
+    const SigWeights weights(kSig ? a.scale * a.temp[h] / a.cap : 1.f, kSig ? a.cap : 1.f, kSig ? a.shift[h] : 0.f);
     bool ok = true;
     for (int j = j0; j < j1; ++j) {
       ok = __all_sync(0xffffffffu, tc::mbar_wait(&s_full[x], (uint32_t)(j - j0) & 1u, abort_flag));
@@ -321,65 +383,38 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       const int kbase = (j_lo + j) * kBN, q_rel = q_idx + shift;
       const int lim = min(kv_len, q_rel + 1) - kbase;
       const int low = a.window > 0 ? q_rel - a.window + 1 - kbase : 0;
-      uint32_t v[kBN];
-#pragma unroll
-      for (int c = 0; c < 4; ++c)
-        tc::tmem_ld32(s_tmem + 32 * c, *reinterpret_cast<uint32_t(*)[32]>(v + 32 * c));
-      tc::tmem_ld_wait();
       if constexpr (kSig) {
-        uint32_t pk[kBN / 2];
-        float tops[4] = {0.f, 0.f, 0.f, 0.f};
+        // 32 columns at a time, the next ones on their way; their weights go where scores have been read
+        uint32_t v[2][32];
+        tc::tmem_ld32(s_tmem, v[0]);
 #pragma unroll
-        for (int i = 0; i < 32; ++i)
+        for (int c = 0; c < 4; ++c) {
+          tc::tmem_ld_wait();
 #pragma unroll
-          for (int c = 0; c < 4; ++c) tops[c] = fmaxf(tops[c], fabsf(__uint_as_float(v[32 * c + i])));
-        const float top = fmaxf(fmaxf(tops[0], tops[1]), fmaxf(tops[2], tops[3]));
-        const unsigned long long f2 = pack2(f_z, f_z), sh2 = pack2(f_shift, f_shift), one2 = pack2(1.f, 1.f);
-        // two exponents (base 2) of the negated argument -> two weights with one reciprocal
-        auto weigh = [&](float x0, float x1, int at) {
-          const float u0 = ex2f(fminf(x0, 60.f)), u1 = ex2f(fminf(x1, 60.f));
-          float a0, a1;
-          unpack2(add2(pack2(u0, u1), one2), a0, a1);
-          const float r = rcpf(a0 * a1);
-          pk[at] = us::pack_bf(r * a1, r * a0);
-        };
-        if (__all_sync(0xffffffffu, top * fabsf(f_z) <= kTanhMost)) {
-          const unsigned long long c2 = pack2(f_cap, f_cap);
+          for (int i = 0; i < 32; ++i) asm volatile("" : "+r"(v[c & 1][i]));     // not before the wait
+          if (c < 3) tc::tmem_ld32(s_tmem + 32 * (c + 1), v[(c + 1) & 1]);
+          uint32_t pk[16];
+          weights(v[c & 1], pk);
+          const int l0 = low - 32 * c, l1 = lim - 32 * c;
+          if (l1 < 32 || l0 > 0) {
 #pragma unroll
-          for (int i = 0; i < kBN; i += 2) {
-            const unsigned long long z = mul2(pack2(__uint_as_float(v[i]), __uint_as_float(v[i + 1])), f2);
-            const unsigned long long u = mul2(z, z);
-            unsigned long long p = fma2(pack2(kT4, kT4), u, pack2(kT3, kT3));
-            p = fma2(fma2(p, u, pack2(kT2, kT2)), u, pack2(kT1, kT1));
-            p = fma2(p, u, one2);
-            float x0, x1;
-            unpack2(fma2(mul2(z, c2), p, sh2), x0, x1);
-            weigh(x0, x1, i >> 1);
+            for (int i = 0; i < 32; i += 2) {
+              if (i >= l1 || i < l0) pk[i >> 1] &= 0xffff0000u;
+              if (i + 1 >= l1 || i + 1 < l0) pk[i >> 1] &= 0x0000ffffu;
+            }
           }
-        } else {
-          const float f_e = 2.8853900817779268f * f_z;       // e^{2 z} = 2^{score f_e}
-#pragma unroll
-          for (int i = 0; i < kBN; i += 2) {                  // tanh(z) = 1 - 2 / (e^{2 z} + 1)
-            const float t0 = fmaf(-2.f, rcpf(ex2f(__uint_as_float(v[i]) * f_e) + 1.f), 1.f);
-            const float t1 = fmaf(-2.f, rcpf(ex2f(__uint_as_float(v[i + 1]) * f_e) + 1.f), 1.f);
-            weigh(fmaf(t0, f_cap, f_shift), fmaf(t1, f_cap, f_shift), i >> 1);
-          }
+          tc::tmem_st16(s_tmem + 16 * c, pk);
         }
-        if (lim < kBN || low > 0) {
-#pragma unroll
-          for (int i = 0; i < kBN; i += 2) {
-            if (i >= lim || i < low) pk[i >> 1] &= 0xffff0000u;
-            if (i + 1 >= lim || i + 1 < low) pk[i >> 1] &= 0x0000ffffu;
-          }
-        }
-#pragma unroll
-        for (int c = 0; c < 2; ++c)
-          tc::tmem_st32(s_tmem + 32 * c, *reinterpret_cast<const uint32_t(*)[32]>(pk + 32 * c));
         tc::tmem_st_wait();
         tc::tc_fence_before_sync();
         tc::mbar_arrive(&p_full[x]);
         continue;
       }
+      uint32_t v[kBN];
+#pragma unroll
+      for (int c = 0; c < 4; ++c)
+        tc::tmem_ld32(s_tmem + 32 * c, *reinterpret_cast<uint32_t(*)[32]>(v + 32 * c));
+      tc::tmem_ld_wait();
       if (lim < kBN || low > 0) {
 #pragma unroll
         for (int i = 0; i < kBN; ++i)
@@ -441,41 +476,70 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       tc::mbar_arrive(&p_full[x]);
     }
     if (j1 > j0) {
+      const bool row_ok = q_idx < q_len, wide = ((a.V | (int)a.ldo) & 7) == 0;
+      const long long row = q_start + q_idx;
+      // a gate of every column: fetched in 16-byte pieces while the last value product runs
+      const bool columns = a.gate && a.gate_cols > 1;
+      const bool pieces = columns && wide && (a.ldg & 7) == 0 && ((uintptr_t)a.gate & 15) == 0;
+      const __nv_bfloat16* grow = a.gate ? a.gate + row * a.ldg + (long long)h * a.gate_cols : nullptr;
+      uint4 gp[kDV / 8];
+      if (pieces) {
+#pragma unroll
+        for (int i = 0; i < kDV / 8; ++i)
+          if (row_ok && i * 8 < a.V) gp[i] = __ldg(reinterpret_cast<const uint4*>(grow) + i);
+      }
       if (ok && tc::mbar_wait(&o_full[x], 0, abort_flag)) {
         tc::tc_fence_after_sync();
-        if (a.sink && l_sum > 0.f) l_sum += ex2f(a.sink[h] * 1.4426950408889634f - m_used);
+        if (a.sink && l_sum > 0.f) l_sum += ex2f(a.sink[h] * kLog2e - m_used);
         float inv = kSig ? a.out_scale : l_sum > 0.f ? a.out_scale / l_sum : 0.f;
-        const bool row_ok = q_idx < q_len, wide = ((a.V | (int)a.ldo) & 7) == 0;
-        __nv_bfloat16* orow = a.out + (long long)(q_start + q_idx) * a.ldo + (long long)h * a.V;
-        const __nv_bfloat16* grow = nullptr;     // gate of every column
-        if (a.gate && row_ok) {
-          grow = a.gate + (long long)(q_start + q_idx) * a.ldg + (long long)h * a.gate_cols;
-          if (a.gate_cols == 1) {
-            inv *= sigmoid_of(*grow);
-            grow = nullptr;
-          }
-        }
-#pragma unroll 1
-        for (int c = 0; c < kDV; c += 32) {
-          uint32_t w[32];
-          tc::tmem_ld32(o_tmem + c, w);
-          tc::tmem_ld_wait();
-          if (!row_ok) continue;
+        if (a.gate && !columns && row_ok) inv *= sigmoid_of(*grow);
+        __nv_bfloat16* orow = a.out + row * a.ldo + (long long)h * a.V;
+        if (pieces) {
 #pragma unroll
-          for (int q4 = 0; q4 < 4; ++q4) {
-            us::Pack16 o;
+          for (int c = 0; c < kDV; c += 32) {
+            uint32_t w[32];
+            tc::tmem_ld32(o_tmem + c, w);
+            tc::tmem_ld_wait();
+            if (!row_ok) continue;
 #pragma unroll
-            for (int i = 0; i < 8; ++i) {
-              float f = __uint_as_float(w[q4 * 8 + i]) * inv;
-              if (grow && c + q4 * 8 + i < a.V) f *= sigmoid_of(grow[c + q4 * 8 + i]);
-              o.b[i] = us::f2bf(f);
+            for (int q4 = 0; q4 < 4; ++q4) {
+              if (c + q4 * 8 >= a.V) continue;
+              us::Pack16 o, g;
+              g.u = gp[c / 8 + q4];
+#pragma unroll
+              for (int i = 0; i < 8; i += 2) {         // two sigmoids with one reciprocal
+                const float g0 = ex2f(fminf(us::bf2f(g.b[i]) * -kLog2e, kExpMost)) + 1.f;
+                const float g1 = ex2f(fminf(us::bf2f(g.b[i + 1]) * -kLog2e, kExpMost)) + 1.f;
+                const float r = inv * rcpf(g0 * g1);
+                o.b[i] = us::f2bf(__uint_as_float(w[q4 * 8 + i]) * (r * g1));
+                o.b[i + 1] = us::f2bf(__uint_as_float(w[q4 * 8 + i + 1]) * (r * g0));
+              }
+              *reinterpret_cast<uint4*>(orow + c + q4 * 8) = o.u;
             }
-            if (wide) {
-              if (c + q4 * 8 < a.V) *reinterpret_cast<uint4*>(orow + c + q4 * 8) = o.u;
-            } else {
+          }
+        } else {
+#pragma unroll 1
+          for (int c = 0; c < kDV; c += 32) {
+            uint32_t w[32];
+            tc::tmem_ld32(o_tmem + c, w);
+            tc::tmem_ld_wait();
+            if (!row_ok) continue;
 #pragma unroll
-              for (int i = 0; i < 8; ++i)
-                if (c + q4 * 8 + i < a.V) orow[c + q4 * 8 + i] = o.b[i];
+            for (int q4 = 0; q4 < 4; ++q4) {
+              us::Pack16 o;
+#pragma unroll
+              for (int i = 0; i < 8; ++i) {
+                float f = __uint_as_float(w[q4 * 8 + i]) * inv;
+                if (columns && c + q4 * 8 + i < a.V) f *= sigmoid_of(grow[c + q4 * 8 + i]);
+                o.b[i] = us::f2bf(f);
+              }
+              if (wide) {
+                if (c + q4 * 8 < a.V) *reinterpret_cast<uint4*>(orow + c + q4 * 8) = o.u;
+              } else {
+#pragma unroll
+                for (int i = 0; i < 8; ++i)
+                  if (c + q4 * 8 + i < a.V) orow[c + q4 * 8 + i] = o.b[i];
+              }
             }
           }
         }
@@ -606,7 +670,7 @@ US_API int us_sigmoid_flash(const void* q, long long ldq, const void* k, long lo
   US_REQUIRE(temp && shift && cap >= 0.f);
   // an enormous cap: z is tiny, its tanh z itself, and cap * z the score
   FlashArgs a{cu_q, cu_k, (__nv_bfloat16*)out, ldo, V, window, 0.f, nullptr, 1, nullptr, out_scale,
-              (const __nv_bfloat16*)gate, ldg, 1, temp, shift, scale, cap > 0.f ? cap : 1e12f};
+              (const __nv_bfloat16*)gate, ldg, 1, temp, shift, scale, cap > 0.f ? cap : 1e9f};
   return grouped_flash<true>(a, q, ldq, k, ldk, v, ldv, n_seqs, Tq, Tk, H, G, slabs, dv, max_q,
                              (cudaStream_t)stream_);
 }

@@ -18,6 +18,7 @@ constexpr int kWarps = 4, kThreads = kWarps * 32;
 constexpr int kKeys = 16;            // per tile
 constexpr int kStages = 3;           // tiles in a warp's ring
 constexpr int kHeads = 16;
+constexpr int kMostSplits = 16;      // more than 8 CTAs to a cluster where the device allows them
 
 struct SigDecode {
   const __nv_bfloat16* q;            // [T, H, ..]: rows at ldq, heads at hsq
@@ -216,7 +217,7 @@ __global__ void __launch_bounds__(kThreads) sigmoid_decode_kernel(const SigDecod
 }
 
 template <int DP, int VP>
-int launch(const SigDecode& a, int rows, cudaStream_t stream) {
+int launch(SigDecode a, int rows, cudaStream_t stream) {
   constexpr size_t smem = (size_t)kWarps * kStages * kKeys * (DP + VP) * 2;
   static_assert(smem >= (size_t)kWarps * kHeads * VP * 4, "partial outputs fit the rings");
   static bool configured = false;
@@ -224,6 +225,10 @@ int launch(const SigDecode& a, int rows, cudaStream_t stream) {
     US_CUDA_CHECK(cudaFuncSetAttribute(sigmoid_decode_kernel<DP, VP>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                        (int)smem));
     configured = true;
+  }
+  if (a.splits > 8) {
+    static const int most = us::cluster_limit(sigmoid_decode_kernel<DP, VP>, kMostSplits, kThreads, smem);
+    if (a.splits > most) a.splits = most;
   }
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3(a.splits, a.G * us::ceil_div(a.H / a.G, kHeads), rows);
@@ -255,7 +260,7 @@ US_API int us_sigmoid_decode(const void* q, long long ldq, int hsq, const void* 
                              const float* temp, const float* shift, float cap, float out_scale,
                              const void* gate, long long ldg, void* stream_) {
   US_REQUIRE(q && kpages && vpages && out && cu && pos && page_table && temp && shift && count >= 0 && B >= 1 &&
-             H >= 1 && G >= 1 && H % G == 0 && D >= 8 && V >= 8 && page >= 1 && splits >= 1 && splits <= 8 &&
+             H >= 1 && G >= 1 && H % G == 0 && D >= 8 && V >= 8 && page >= 1 && splits >= 1 && splits <= kMostSplits &&
              count <= 65535 && G * us::ceil_div(H / G, kHeads) <= 65535 && (rows || count == B) &&
              ldo >= (long long)H * V && cap >= 0.f);
   US_REQUIRE((D % 8) == 0 && (V % 8) == 0 && (ldq % 2) == 0 && (hsq % 2) == 0 && ((uintptr_t)q % 4) == 0 &&

@@ -102,8 +102,8 @@ struct StreamRows {
 
 enum Form : int { kOutNorm = 0, kPlain = 1, kLayer = 2 };
 
-template <int NV, int FORM>
-__global__ void __launch_bounds__(256) stream_rows_kernel(const StreamRows a) {
+template <int NV, int FORM, bool MIX>
+__global__ void __launch_bounds__(256, NV <= 2 ? 4 : 1) stream_rows_kernel(const StreamRows a) {
   US_PDL_PROLOGUE();
   __shared__ float buf[64];
   int turn = 0;
@@ -133,11 +133,26 @@ __global__ void __launch_bounds__(256) stream_rows_kernel(const StreamRows a) {
     }
     if (t0 == t1) return;
   }
+  // a mixture's routes of a row (lane k: expert k) and the shared rows' gate, fetched a row ahead
+  int next_p = -1;
+  float next_w = 0.f, next_g = 1.f;
+  auto routes = [&](int t) {
+    const int lane = threadIdx.x & 31;
+    if (t >= t1) return;
+    if (lane < a.top) {
+      next_p = a.perm[(long long)t * a.top + lane];
+      next_w = a.route_w[(long long)t * a.top + lane];
+    }
+    if (FORM == kLayer && a.shared_gate) next_g = 1.f / (1.f + expf(-a.shared_gate[t * a.ld_gate]));
+  };
+  if constexpr (MIX) routes(t0);
   // raw operands of a row: the sublayer's output (or the embedding sum) and the residual
   auto load = [&](int t, float4 (&v)[NV], float4 (&r)[NV]) {
     const long long base = (long long)t * W;
-    if (FORM != kOutNorm && a.y_perm) {
-      const float sg = FORM == kLayer && a.shared_gate ? 1.f / (1.f + expf(-a.shared_gate[t * a.ld_gate])) : 1.f;
+    if constexpr (MIX) {
+      const int p_row = next_p;
+      const float w_row = next_w, sg = next_g;
+      routes(t + 1);
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
         const int c = c0 + i * step;
@@ -147,11 +162,10 @@ __global__ void __launch_bounds__(256) stream_rows_kernel(const StreamRows a) {
         if (FORM == kLayer) v[i] = make_float4(v[i].x * sg, v[i].y * sg, v[i].z * sg, v[i].w * sg);
         r[i] = *reinterpret_cast<const float4*>(a.residual + base + c);
       }
-      const long long k0 = (long long)t * a.top;
 #pragma unroll 4
       for (int k = 0; k < a.top; ++k) {
-        const int p = a.perm[k0 + k];
-        const float wk = a.route_w[k0 + k];
+        const int p = __shfl_sync(0xffffffffu, p_row, k);
+        const float wk = __shfl_sync(0xffffffffu, w_row, k);
         if (p < 0 && !a.ident) continue;
         const void* from = p < 0 ? a.ident : a.y_perm;
         const long long row = (long long)(p < 0 ? t : p) * W;
@@ -405,13 +419,13 @@ int block_threads(int W) { return min(256, (W / 4 + 31) / 32 * 32); }
 
 namespace {
 
-template <int FORM>
+template <int FORM, bool MIX>
 int launch_stream(const StreamRows& a, cudaStream_t stream) {
   const int grid = !a.mu ? us::ceil_div(a.T, a.rows) : a.one_token ? a.T : a.T / kRows + a.B;
   const dim3 block(block_threads(a.W));
   const int nv = us::ceil_div(a.W, 1024);
 #define US_STREAM(N) \
-  US_CUDA_CHECK(us::launch_pdl(stream_rows_kernel<N, FORM>, dim3(grid), block, 0, stream, a))
+  US_CUDA_CHECK(us::launch_pdl(stream_rows_kernel<N, FORM, MIX>, dim3(grid), block, 0, stream, a))
   if (nv <= 1) US_STREAM(1);
   else if (nv <= 2) US_STREAM(2);
   else if (nv <= 4) US_STREAM(4);
@@ -438,7 +452,7 @@ US_API int us_stream_rows(const int* ids, const int* rows2, const void* table, c
   if (T == 0) return US_OK;
   StreamRows a{ids, rows2, table, table2, scale, vocab, n2, y, residual, w, residual_out, w_out, mu,
                state, cu, slots, pos, x, B, T, W, width, bf16, one_token, eps, T >= 2048 ? 4 : 1, us_status_ptr()};
-  return launch_stream<kOutNorm>(a, (cudaStream_t)stream_);
+  return launch_stream<kOutNorm, false>(a, (cudaStream_t)stream_);
 }
 
 // The plain form: residual_out = table row * scale (ids given), or residual + gain * (y, or the mixture
@@ -450,12 +464,12 @@ US_API int us_plain_rows(const int* ids, const void* table, float scale, int voc
                          int bf16, float eps, void* stream_) {
   US_REQUIRE(residual_out && w_out && x && T >= 0 && W >= 8 && (W % 8) == 0 && width >= 1 && width <= W);
   US_REQUIRE(y || y_perm ? residual && residual != residual_out : ids && table);
-  US_REQUIRE(!y_perm || (perm && route_w && top >= 1 && !y));
+  US_REQUIRE(!y_perm || (perm && route_w && top >= 1 && top <= 32 && !y));
   if (T == 0) return US_OK;
   StreamRows a{ids, nullptr, table, nullptr, scale, vocab, 0, y, residual, nullptr, residual_out, w_out, nullptr,
-               nullptr, nullptr, nullptr, nullptr, x, 1, T, W, width, bf16, 0, eps, T >= 2048 ? 4 : 1, us_status_ptr(),
+               nullptr, nullptr, nullptr, nullptr, x, 1, T, W, width, bf16, 0, eps, T >= 2048 ? 2 : 1, us_status_ptr(),
                y || y_perm ? gain : 1.f, y_perm, perm, route_w, top, ident, shared};
-  return launch_stream<kPlain>(a, (cudaStream_t)stream_);
+  return y_perm ? launch_stream<kPlain, true>(a, (cudaStream_t)stream_) : launch_stream<kPlain, false>(a, (cudaStream_t)stream_);
 }
 
 // The layer form: residual_out = table row * scale (ids given), or residual + ln(y, or a mixture of `top`
@@ -468,13 +482,13 @@ US_API int us_layer_rows(const int* ids, const void* table, float scale, int voc
                          int bf16, float eps, void* stream_) {
   US_REQUIRE(residual_out && x && T >= 0 && W >= 8 && (W % 8) == 0 && width >= 1 && width <= W);
   US_REQUIRE(y || y_perm ? residual && residual != residual_out && w && b : ids && table && !residual);
-  US_REQUIRE(!y_perm || (perm && route_w && top >= 1 && !y));
+  US_REQUIRE(!y_perm || (perm && route_w && top >= 1 && top <= 32 && !y));
   US_REQUIRE(!w_out || b_out);
   if (T == 0) return US_OK;
   StreamRows a{ids, nullptr, table, nullptr, scale, vocab, 0, y, residual, w, residual_out, w_out, nullptr,
-               nullptr, nullptr, nullptr, nullptr, x, 1, T, W, width, bf16, 0, eps, T >= 2048 ? 4 : 1, us_status_ptr(),
+               nullptr, nullptr, nullptr, nullptr, x, 1, T, W, width, bf16, 0, eps, T >= 2048 ? 2 : 1, us_status_ptr(),
                1.f, y_perm, perm, route_w, top, nullptr, shared, b, b_out, shared_gate, ld_gate};
-  return launch_stream<kLayer>(a, (cudaStream_t)stream_);
+  return y_perm ? launch_stream<kLayer, true>(a, (cudaStream_t)stream_) : launch_stream<kLayer, false>(a, (cudaStream_t)stream_);
 }
 
 US_API int us_bigram_rows(const int* ids, int* last, const int* cu, const int* slots, const int* pos,

@@ -177,6 +177,102 @@ __global__ void __launch_bounds__(kPrepWarps * 32) window_prep_kernel(const Prep
   }
 }
 
+__device__ __forceinline__ float4 ld4(const void* base, long long i, int bf16) {
+  if (bf16) {
+    us::Pack8 p;
+    p.u = *reinterpret_cast<const uint2*>(reinterpret_cast<const __nv_bfloat16*>(base) + i);
+    return make_float4(us::bf2f(p.b[0]), us::bf2f(p.b[1]), us::bf2f(p.b[2]), us::bf2f(p.b[3]));
+  }
+  return *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(base) + i);
+}
+__device__ __forceinline__ void st4(void* base, long long i, int bf16, float4 v) {
+  if (bf16) {
+    us::Pack8 p;
+    p.b[0] = us::f2bf(v.x); p.b[1] = us::f2bf(v.y); p.b[2] = us::f2bf(v.z); p.b[3] = us::f2bf(v.w);
+    *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(base) + i) = p.u;
+  } else {
+    *reinterpret_cast<float4*>(reinterpret_cast<float*>(base) + i) = v;
+  }
+}
+
+// The same for neighbouring channels: a lane holds both of every pair, four channels at a time, and a
+// warp's heads are loaded together.
+template <int NI>
+__global__ void __launch_bounds__(kPrepWarps * 32) neighbours_prep_kernel(const Prep a) {
+  US_PDL_PROLOGUE();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int units = a.H + a.G, groups = (units + kPrepHeads - 1) / kPrepHeads;
+  const long long item = (long long)blockIdx.x * kPrepWarps + warp;
+  if (item >= (long long)a.T * groups) return;
+  const int t = (int)(item / groups), u0 = (int)(item % groups) * kPrepHeads, pos = a.pos[t];
+  const long long slot = a.slots[t], row = (long long)t * a.ldx;
+  float4 v[kPrepHeads][NI];
+  bool in[kPrepHeads];
+#pragma unroll
+  for (int u = 0; u < kPrepHeads; ++u) {
+    const int unit = u0 + u;
+    in[u] = unit < a.H || (unit < units && slot >= 0);
+    const long long from = row + (unit < a.H ? a.off_q + unit * a.D : a.off_k + (unit - a.H) * a.D);
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      const int d = (i * 32 + lane) * 4;
+      v[u][i] = in[u] && d < a.D ? ld4(a.x, from + d, a.bf16) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+  }
+  float cs[NI][2], sn[NI][2];
+#pragma unroll
+  for (int i = 0; i < NI; ++i)
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int p = (i * 32 + lane) * 2 + e;
+      cs[i][e] = 1.f;
+      sn[i][e] = 0.f;
+      if (p < a.pairs) {
+        turn(pos, a.freq[p], cs[i][e], sn[i][e]);
+        cs[i][e] *= a.mag;
+        sn[i][e] *= a.mag;
+      }
+    }
+  float ss[kPrepHeads];
+#pragma unroll
+  for (int u = 0; u < kPrepHeads; ++u) {
+    ss[u] = 0.f;
+#pragma unroll
+    for (int i = 0; i < NI; ++i)
+      ss[u] += v[u][i].x * v[u][i].x + v[u][i].y * v[u][i].y + v[u][i].z * v[u][i].z + v[u][i].w * v[u][i].w;
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+    for (int u = 0; u < kPrepHeads; ++u) ss[u] += __shfl_xor_sync(0xffffffffu, ss[u], o);
+#pragma unroll
+  for (int u = 0; u < kPrepHeads; ++u) {
+    const int unit = u0 + u, g = unit - a.H;
+    if (!in[u]) continue;
+    const bool is_q = g < 0;
+    const float* w = is_q ? a.wq : a.wk;
+    void* dst = is_q ? a.q : a.kp;
+    const long long to = is_q ? ((long long)t * a.H + unit) * a.Dq : (slot * a.G + g) * a.D;
+    const float inv = 1.f / sqrtf(ss[u] / (float)a.D + a.eps);
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      const int d = (i * 32 + lane) * 4;
+      if (d < a.D) {
+        const float4 w4 = *reinterpret_cast<const float4*>(w + d);
+        const float4 n = make_float4(v[u][i].x * (inv * w4.x), v[u][i].y * (inv * w4.y), v[u][i].z * (inv * w4.z),
+                                     v[u][i].w * (inv * w4.w));
+        st4(dst, to + d, a.bf16, make_float4(n.x * cs[i][0] - n.y * sn[i][0], n.y * cs[i][0] + n.x * sn[i][0],
+                                             n.z * cs[i][1] - n.w * sn[i][1], n.w * cs[i][1] + n.z * sn[i][1]));
+      } else if (is_q && d < a.Dq) {
+        st4(dst, to + d, a.bf16, make_float4(0.f, 0.f, 0.f, 0.f));
+      }
+    }
+    if (is_q) continue;
+    const long long vf = row + a.off_v + (long long)g * a.V, vt = (slot * a.G + g) * a.V;
+    for (int d = lane * 4; d < a.V; d += 128) st4(a.vp, vt + d, a.bf16, ld4(a.x, vf + d, a.bf16));
+  }
+}
+
 template <int VEC>
 int launch_prep(const Prep& a, cudaStream_t stream) {
   const long long items = (long long)a.T * ((a.H + a.G + kPrepHeads - 1) / kPrepHeads);
@@ -380,6 +476,15 @@ US_API int us_window_prep(const void* x, long long ldx, int off_q, int off_k, in
   if (T == 0) return US_OK;
   Prep a{x, ldx, off_q, off_k, off_v, H, G, D, V, pairs, wq, wk, freq, mag, pos, slots, q, Dq, kpages, vpages,
          T, bf16, eps, neighbours};
+  const int sizes = D | V | Dq | off_q | off_k | off_v | (int)(ldx & 3);
+  if (neighbours && (sizes & 3) == 0 && D <= 256 && Dq <= 128 * us::ceil_div(D, 128) && ((uintptr_t)x % 16) == 0 &&
+      ((uintptr_t)wq % 16) == 0 && ((uintptr_t)wk % 16) == 0) {
+    const long long items = (long long)T * ((H + G + kPrepHeads - 1) / kPrepHeads);
+    const dim3 grid((unsigned)((items + kPrepWarps - 1) / kPrepWarps)), block(kPrepWarps * 32);
+    US_CUDA_CHECK(us::launch_pdl(D <= 128 ? neighbours_prep_kernel<1> : neighbours_prep_kernel<2>, grid, block, 0,
+                                 (cudaStream_t)stream_, a));
+    return US_OK;
+  }
   const bool two = even(ldx, off_q, off_k, off_v) && even(D, V, pairs, Dq) && ((uintptr_t)x % 4) == 0;
   return two ? launch_prep<2>(a, (cudaStream_t)stream_) : launch_prep<1>(a, (cudaStream_t)stream_);
 }

@@ -350,6 +350,8 @@ def linear(x, w, bias=None, out_dtype=None, out=None, block_n=None, act=None, ac
                0 if (bias is None or bias.dtype == BF16) else 1, acode, *act_ab, N.stream())
         return out.view(*x.shape[:-1], M)
     bn = block_n or _block_n(rows, False)
+    if block_n is None and M <= 128 and rows > 128:       # few features (a router): more, smaller row tiles
+        bn = 64 if rows <= 64 * 296 else 128
     if acode == 6:
         assert bias is None and out.dtype == BF16
         N.call("us_gemm_wx_act", N.ptr(w), N.ptr(x2), N.ptr(out), 1, M, M, K, rows, w.stride(0), x2.stride(0),

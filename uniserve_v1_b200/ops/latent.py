@@ -132,8 +132,11 @@ def decode_fits(ql, cpages, rpages) -> bool:
 
 
 def decode_splits(rows: int, heads: int, keys: int) -> int:
-    """Key splits per row: one CTA per SM, at least 64 keys each."""
+    """Key splits per row: one CTA per SM, at least 64 keys each.  Sixteen (a cluster that fills a GPC) for
+    few rows with many keys."""
     ctas = rows * -(-heads // (16 if heads <= 16 else 32))
+    if ctas <= 2 and keys >= 2048:
+        return 16
     return max(1, min(148 // ctas, keys // 64, 8))
 
 

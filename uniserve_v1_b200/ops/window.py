@@ -168,6 +168,8 @@ def _sigmoid_decode(q, kpages, vpages, m: SeqMeta, page_table, sig: SigmoidScore
     keys = min(keys, d.window) if d.window > 0 else keys
     ctas = count * G * -(-(H // G) // 16)
     splits = max(1, min(296 // max(1, ctas), keys // 64, 8))          # two CTAs per SM
+    if ctas <= 8 and keys >= 2048:
+        splits = 16
     N.call("us_sigmoid_decode", N.ptr(q), q.stride(0), q.stride(1), N.ptr(kpages), N.ptr(vpages), N.ptr(out),
            out.stride(0), N.ptr(rows), N.ptr(m.cu), N.ptr(m.positions), N.ptr(seq_lens), N.ptr(page_table), count,
            m.cu.shape[0] - 1, H, G, d.dim, d.vdim, page, page_table.shape[1], d.window, splits, d.scale,
