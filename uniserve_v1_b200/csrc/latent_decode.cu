@@ -269,27 +269,26 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const Decode
   }
   __syncthreads();
   if (a.splits > 1) tc::cluster_sync();
-  // every CTA of the cluster finishes a share of the heads' columns, adding the splits in order:
-  // first each split's factor per head (in `part`), then the columns
-  float* wgt = part;                                             // [HT][kMostSplits]
-  for (int h = tid; h < nh; h += kThreads) {
-    float m[kMostSplits], l[kMostSplits], top = -INFINITY, den = 0.f;
+  // every CTA of the cluster finishes a share of the heads' columns, adding the splits in order: first the
+  // splits' maxima and sums side by side (in `part`), then each split's factor per head, then the columns
+  float* mt = part;                                              // [HT][kMostSplits] each
+  float* lt = mt + HT * kMostSplits;
+  float* wgt = lt + HT * kMostSplits;
+  for (int e = tid; e < nh * a.splits; e += kThreads) {
+    const int h = e / a.splits, p = e - h * a.splits;
     const uint32_t am = (uint32_t)__cvta_generic_to_shared(&mx[h]);
     const uint32_t al = (uint32_t)__cvta_generic_to_shared(&sum[h]);
-#pragma unroll
-    for (int p = 0; p < kMostSplits; ++p) {
-      m[p] = p < a.splits ? (a.splits > 1 ? tc::ld_dsmem_f32(tc::map_to_cta(am, p)) : mx[h]) : -INFINITY;
-      l[p] = p < a.splits ? (a.splits > 1 ? tc::ld_dsmem_f32(tc::map_to_cta(al, p)) : sum[h]) : 0.f;
-    }
-#pragma unroll
-    for (int p = 0; p < kMostSplits; ++p) top = fmaxf(top, m[p]);
-#pragma unroll
-    for (int p = 0; p < kMostSplits; ++p) {
-      m[p] = top > -INFINITY ? ex2(m[p] - top) : 0.f;
-      den = fmaf(m[p], l[p], den);
-    }
-#pragma unroll
-    for (int p = 0; p < kMostSplits; ++p) wgt[h * kMostSplits + p] = den > 0.f ? m[p] / den : 0.f;
+    mt[h * kMostSplits + p] = a.splits > 1 ? tc::ld_dsmem_f32(tc::map_to_cta(am, p)) : mx[h];
+    lt[h * kMostSplits + p] = a.splits > 1 ? tc::ld_dsmem_f32(tc::map_to_cta(al, p)) : sum[h];
+  }
+  __syncthreads();
+  for (int h = tid; h < nh; h += kThreads) {
+    const float *m = mt + h * kMostSplits, *l = lt + h * kMostSplits;
+    float top = -INFINITY, den = 0.f;
+    for (int p = 0; p < a.splits; ++p) top = fmaxf(top, m[p]);
+    if (top > -INFINITY)
+      for (int p = 0; p < a.splits; ++p) den = fmaf(ex2(m[p] - top), l[p], den);
+    for (int p = 0; p < a.splits; ++p) wgt[h * kMostSplits + p] = den > 0.f ? ex2(m[p] - top) / den : 0.f;
   }
   __syncthreads();
   const int cols = a.hso, quads = (cols + 3) / 4;
@@ -299,7 +298,7 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const Decode
     float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
     if (c < RP) {
       const uint32_t ao = (uint32_t)__cvta_generic_to_shared(os + h * RP + c);
-      for (int p0 = 0; p0 < a.splits; p0 += 8) {
+      auto add = [&](int p0) {                       // eight splits, fetched together
         float4 o4[8];
 #pragma unroll
         for (int p = 0; p < 8; ++p)
@@ -315,7 +314,9 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const Decode
             v.z = fmaf(f, o4[p].z, v.z);
             v.w = fmaf(f, o4[p].w, v.w);
           }
-      }
+      };
+      add(0);
+      if (a.splits > 8) add(8);
     }
     __nv_bfloat16* dst = a.out + t * a.ldo + (long long)(h0 + h) * a.hso + c;
     const float f[4] = {c < a.R ? v.x : 0.f, c + 1 < a.R ? v.y : 0.f, c + 2 < a.R ? v.z : 0.f,
@@ -346,7 +347,7 @@ int launch_decode(DecodeArgs a, int rows, cudaStream_t stream) {
     static const int most = us::cluster_limit(latent_decode_kernel<RP, MT>, kMostSplits, kThreads, smem);
     if (a.splits > most) a.splits = most;
   }
-  static_assert((8 / MT) * HT * kSRow >= HT * kMostSplits, "the splits' factors fit the score slices");
+  static_assert((8 / MT) * kSRow >= 3 * kMostSplits, "the splits' factors fit the score slices");
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3(a.splits, us::ceil_div(a.H, HT), rows);
   cfg.blockDim = dim3(kThreads);
